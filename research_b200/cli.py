@@ -107,10 +107,7 @@ def cmd_serve(args) -> int:
 
     device = "cuda" if torch.cuda.is_available() else "cpu"
     if os.path.isdir(args.model):
-        from .models.config import ModelConfig
-
-        cfg = ModelConfig.from_hf_dict(json.loads((Path(args.model) / "config.json").read_text()))
-        weights = load_safetensors_dir(args.model)
+        weights, cfg = load_safetensors_dir(args.model)
         tokenizer = None
         try:
             from transformers import AutoTokenizer

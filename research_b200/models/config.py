@@ -13,6 +13,8 @@ import json
 from dataclasses import asdict, dataclass, field, replace
 from pathlib import Path
 
+from .stack import ClampedGluSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, RotarySpec, uniform_stack
+
 
 @dataclass(frozen=True)
 class ModelConfig:
@@ -130,13 +132,18 @@ class ModelConfig:
 
     @staticmethod
     def load(path: str | Path) -> "ModelConfig":
+        """A Hugging Face style ``config.json`` (``registry.load_config`` reads every known kind)."""
         return ModelConfig.from_hf_dict(json.loads((Path(path) / "config.json").read_text()))
 
     def as_dict(self) -> dict:
         return asdict(self)
 
 
-PRESETS: dict[str, ModelConfig] = {
+def _latent(heads: int, dim: int, rot: int, vdim: int, kv_rank: int, q_rank: int, window: int, base: float = 5e5) -> LatentAttentionSpec:
+    return LatentAttentionSpec(heads, dim, rot, vdim, kv_rank, q_rank, (dim + rot) ** -0.5, window, RotarySpec(rot, base))
+
+
+PRESETS: dict[str, ModelConfig | LayerStackConfig] = {
     # tiny CPU plumbing model: Qwen2-style, vocab 4096, 4 layers, d 256, 4q/2kv heads
     "tiny-qwen2": ModelConfig(),
     "tiny-qwen3": ModelConfig(family="qwen3", attention_bias=False, qk_norm=True, tie_word_embeddings=False),
@@ -158,10 +165,19 @@ PRESETS: dict[str, ModelConfig] = {
                                  rope_theta=1e6, max_position_embeddings=40960, tie_word_embeddings=False,
                                  attention_bias=False, qk_norm=True, num_experts=128, num_experts_per_tok=8,
                                  moe_intermediate_size=768, norm_topk_prob=True),
+    # layer stacks: latent attention with a sliding window (two layers of unlike sizes in the tiny one)
+    "tiny-lulezen": LayerStackConfig("Lulezen", 4096, 192, (
+        LayerSpec(_latent(4, 32, 16, 24, 64, 80, 40), ClampedGluSpec(320, 7.0)),
+        LayerSpec(_latent(3, 24, 8, 32, 96, 64, 100, 1e4), None),
+        LayerSpec(_latent(4, 32, 16, 24, 64, 80, 40), ClampedGluSpec(256, 5.0))), logit_softcap=30.0, init_std=0.05),
+    "lulezen-1b": uniform_stack("Lulezen", vocab=128256, width=2048, num_layers=16, mixer=_latent(16, 128, 64, 128, 512, 1024, 4096),
+                                mlp=ClampedGluSpec(8192, 7.0), logit_softcap=30.0),
+    "lulezen-7b": uniform_stack("Lulezen", vocab=128256, width=4096, num_layers=32, mixer=_latent(32, 128, 64, 128, 512, 1536, 4096),
+                                mlp=ClampedGluSpec(14336, 7.0), logit_softcap=30.0),
 }
 
 
-def get_preset(name: str, **overrides) -> ModelConfig:
+def get_preset(name: str, **overrides) -> ModelConfig | LayerStackConfig:
     cfg = PRESETS[name]
     return replace(cfg, **overrides) if overrides else cfg
 

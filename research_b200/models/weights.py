@@ -20,14 +20,27 @@ import numpy as np
 import torch
 
 from .config import ModelConfig
+from .registry import load_config
+from .stack import LayerStackConfig
 
 _DT = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "I64": torch.int64, "I32": torch.int32,
        "U8": torch.uint8, "F64": torch.float64, "BOOL": torch.bool}
 _DT_INV = {v: k for k, v in _DT.items()}
 
 
-def param_shapes(cfg: ModelConfig) -> dict[str, tuple[int, ...]]:
-    """HF parameter names and shapes for ``cfg``."""
+def _fill_value(cfg: ModelConfig | LayerStackConfig, name: str) -> float | None:
+    """Constant a freshly initialised tensor is filled with; None for a random matrix."""
+    if isinstance(cfg, LayerStackConfig):
+        return cfg.fill_value(name)
+    if name.endswith("norm.weight") or name.endswith("layernorm.weight"):
+        return 1.0
+    return 0.0 if name.endswith(".bias") else None
+
+
+def param_shapes(cfg: ModelConfig | LayerStackConfig) -> dict[str, tuple[int, ...]]:
+    """Checkpoint tensor names and shapes for ``cfg`` (HF names for ``ModelConfig`` families)."""
+    if isinstance(cfg, LayerStackConfig):
+        return cfg.param_shapes()
     d = cfg.hidden_size
     shapes: dict[str, tuple[int, ...]] = {"model.embed_tokens.weight": (cfg.vocab_size, d)}
     for i in range(cfg.num_layers):
@@ -72,16 +85,15 @@ def param_shapes(cfg: ModelConfig) -> dict[str, tuple[int, ...]]:
     return shapes
 
 
-def init_random_weights(cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="cpu") -> dict[str, torch.Tensor]:
+def init_random_weights(cfg: ModelConfig | LayerStackConfig, seed: int = 0, dtype=torch.float32, device="cpu") -> dict[str, torch.Tensor]:
     """N(0, init_std) matrices, unit norm weights, zero biases; deterministic in ``seed``."""
     dev = torch.device(device)
     g = torch.Generator(device=dev).manual_seed(seed)
     out: dict[str, torch.Tensor] = {}
     for name, shape in param_shapes(cfg).items():
-        if name.endswith("norm.weight") or name.endswith("layernorm.weight"):
-            t = torch.ones(shape, dtype=dtype, device=dev)
-        elif name.endswith(".bias"):
-            t = torch.zeros(shape, dtype=dtype, device=dev)
+        fill = _fill_value(cfg, name)
+        if fill is not None:
+            t = torch.full(shape, fill, dtype=dtype, device=dev)
         else:
             t = torch.empty(shape, dtype=torch.float32, device=dev).normal_(0.0, cfg.init_std, generator=g).to(dtype)
         out[name] = t
@@ -93,16 +105,15 @@ class LazyRandomWeights(Mapping):
     ``(seed, name)``) and keeps no reference, so loading a 30B-parameter model into an engine needs the engine's own
     buffers plus one tensor, not a second full copy. Values differ from ``init_random_weights`` (per-name streams)."""
 
-    def __init__(self, cfg: ModelConfig, seed: int = 0, dtype=torch.float32, device="cpu"):
+    def __init__(self, cfg: ModelConfig | LayerStackConfig, seed: int = 0, dtype=torch.float32, device="cpu"):
         self.cfg, self.seed, self.dtype, self.device = cfg, seed, dtype, torch.device(device)
         self.shapes = param_shapes(cfg)
 
     def __getitem__(self, name: str) -> torch.Tensor:
         shape = self.shapes[name]
-        if name.endswith("norm.weight") or name.endswith("layernorm.weight"):
-            return torch.ones(shape, dtype=self.dtype, device=self.device)
-        if name.endswith(".bias"):
-            return torch.zeros(shape, dtype=self.dtype, device=self.device)
+        fill = _fill_value(self.cfg, name)
+        if fill is not None:
+            return torch.full(shape, fill, dtype=self.dtype, device=self.device)
         g = torch.Generator(device=self.device).manual_seed((self.seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFF)
         return torch.empty(shape, dtype=torch.float32, device=self.device).normal_(0.0, self.cfg.init_std, generator=g).to(self.dtype)
 
@@ -180,9 +191,9 @@ def save_safetensors_dir(weights: dict[str, torch.Tensor], cfg: ModelConfig, pat
     (path / "model.safetensors.index.json").write_text(json.dumps(index, indent=2))
 
 
-def load_safetensors_dir(path: str | Path, device="cpu") -> tuple[dict[str, torch.Tensor], ModelConfig]:
+def load_safetensors_dir(path: str | Path, device="cpu") -> tuple[dict[str, torch.Tensor], ModelConfig | LayerStackConfig]:
     path = Path(path)
-    cfg = ModelConfig.load(path)
+    cfg = load_config(path)
     files = sorted(path.glob("*.safetensors"))
     if not files:
         raise FileNotFoundError(f"no safetensors files in {path}")
