@@ -39,6 +39,8 @@ LIBRARIES: dict[str, tuple[str, list[str]]] = {
     "rb_gemm2": ("nvcc", ["gemm2_sm100.cu"]),
     "rb_ops": ("nvcc", ["ops_sm100.cu"]),
     "rb_attn": ("nvcc", ["attn_sm100.cu"]),
+    "rb_latent": ("nvcc", ["latent_sm100.cu"]),
+    "rb_gemm_f32": ("nvcc", ["gemm_f32_sm100.cu"]),
     "rb_flash": ("nvcc", ["flash_sm100.cu"]),
     "rb_quant": ("nvcc", ["quant_sm100.cu"]),
     "rb_train": ("nvcc", ["train_sm100.cu"]),

@@ -9,7 +9,8 @@
 //                (decode first, then admit under batch-size / token / block budgets),
 //                preemption by recompute, and the per-step batch builder that writes token
 //                ids, positions, slot mapping, block tables and sampling rows straight into
-//                pinned host buffers.
+//                pinned host buffers. Prompts can be prefilled in portions (prefill_chunk), and
+//                callers can feed given tokens instead of sampling them (rbe_open / rbe_feed).
 //
 // Behaviour it reproduces: rollouts/inference/scheduler.py:15-84 (policy),
 // rollouts/inference/cache/paged.py:57-203 (block table + prefix hits),
@@ -266,7 +267,8 @@ struct KVManager {
 };
 
 // ------------------------------------------------------------------------------------------
-enum SeqStatus { WAITING = 0, RUNNING = 1, FINISHED = 2 };
+// FED: an externally driven sequence (rbe_feed); it is in no queue and nothing is sampled for it.
+enum SeqStatus { WAITING = 0, RUNNING = 1, FINISHED = 2, FED = 3 };
 
 struct Seq {
   i64 id;
@@ -274,6 +276,7 @@ struct Seq {
   std::vector<float> logprobs;    // one per generated token
   int n_prompt = 0;
   int n_computed = 0;             // tokens whose KV is in the cache
+  int n_target = 0;               // tokens whose KV will be in the cache after the scheduled step
   int n_cached = 0;               // prefix tokens served from the cache at the last admission
   std::vector<int> blocks;
   RadixNode* radix_node = nullptr;
@@ -292,6 +295,7 @@ struct Seq {
 struct EngineCore {
   KVManager kv;
   int max_batch, max_tokens_per_batch, max_model_len;
+  int prefill_chunk = 0;          // > 0: a prompt enters the cache at most this many tokens per step
   std::unordered_map<i64, std::unique_ptr<Seq>> seqs;
   std::deque<i64> waiting;
   std::vector<i64> running;
@@ -362,11 +366,14 @@ struct EngineCore {
     }
     s->n_cached = matched * bs;
     s->n_computed = matched * bs;
+    s->n_target = prefill_chunk > 0 ? std::min(n, s->n_computed + prefill_chunk) : n;
+    // only what this step computes is published now; the rest of a prompt that is prefilled in portions is published
+    // as it is committed (hash mode) or when the sequence releases its blocks (radix mode)
+    const int n_full = s->n_target / bs;
     kv.hit_tokens += matched * bs;
     kv.miss_tokens += n - matched * bs;
     if (kv.mode == 1) {
       // publish the hashes of the full blocks this prefill is about to compute
-      const int n_full = n / bs;
       for (int i = s->n_hashed_blocks; i < n_full; ++i) {
         uint64_t h;
         kv.register_hash(s->blocks[i], s->tokens.data() + i * bs, s->chain, h);
@@ -377,7 +384,6 @@ struct EngineCore {
       // Publish the prompt's full blocks right away so sequences admitted later in this same
       // step already share them (their KV is written by this step's prefill before any
       // attention kernel reads it), then pin the path down to the deepest node.
-      const int n_full = n / bs;
       if (n_full > 0) kv.insert_radix(s->tokens.data(), n_full, s->blocks.data());
       std::vector<int> tmp;
       RadixNode* deep = kv.match_radix(s->tokens.data(), n_full, tmp);
@@ -385,6 +391,14 @@ struct EngineCore {
       s->radix_node = deep;
     }
     return true;
+  }
+
+  // sequences of the scheduled batch in row order: which = 1 decode, 2 prefill, 3 decode then prefill
+  std::vector<i64> batch_order(int which) const {
+    std::vector<i64> order;
+    if (which & 1) order = sched_decode;
+    if (which & 2) order.insert(order.end(), sched_prefill.begin(), sched_prefill.end());
+    return order;
   }
 
   void preempt(Seq* s) {
@@ -403,6 +417,7 @@ struct EngineCore {
     std::vector<i64> keep;
     for (size_t i = 0; i < running.size(); ++i) {
       Seq* s = get(running[i]);
+      if (s == nullptr) continue;
       if ((int)keep.size() >= max_batch) { sched_preempted.push_back(s->id); continue; }
       keep.push_back(s->id);
     }
@@ -431,9 +446,19 @@ struct EngineCore {
         s->blocks.push_back(b);
       }
       if (!ok) { sched_preempted.push_back(s->id); preempt(s); continue; }
-      sched_decode.push_back(s->id);
-      batch_tokens += 1;
+      if (n - s->n_computed > 1) {    // in the middle of its prompt: the next portion
+        s->n_target = prefill_chunk > 0 ? std::min(n, s->n_computed + prefill_chunk) : n;
+        sched_prefill.push_back(s->id);
+      } else {
+        s->n_target = n;
+        sched_decode.push_back(s->id);
+      }
+      batch_tokens += s->n_target - s->n_computed;
     }
+    // a sequence preempted above may already hold a portion
+    sched_prefill.erase(std::remove_if(sched_prefill.begin(), sched_prefill.end(),
+                                       [&](i64 id) { Seq* s = get(id); return !s || s->status != RUNNING; }),
+                        sched_prefill.end());
     for (i64 id : sched_preempted) {
       Seq* s = get(id);
       if (s && s->status == RUNNING) preempt(s);
@@ -445,7 +470,7 @@ struct EngineCore {
       Seq* s = get(waiting.front());
       if (s == nullptr) { waiting.pop_front(); continue; }
       if ((int)(sched_prefill.size() + sched_decode.size()) >= max_batch) break;
-      const int n = (int)s->tokens.size();
+      const int n = prefill_chunk > 0 ? std::min((int)s->tokens.size(), prefill_chunk) : (int)s->tokens.size();
       if (batch_tokens + n > max_tokens_per_batch && !(sched_prefill.empty() && sched_decode.empty())) break;
       // sequences preempted in this very step wait for the next one
       if (std::find(sched_preempted.begin(), sched_preempted.end(), s->id) != sched_preempted.end()) break;
@@ -454,7 +479,7 @@ struct EngineCore {
       s->status = RUNNING;
       running.push_back(s->id);
       sched_prefill.push_back(s->id);
-      batch_tokens += n - s->n_computed;
+      batch_tokens += s->n_target - s->n_computed;
     }
   }
 
@@ -496,6 +521,60 @@ i64 rbe_add_request(void* h, const int* tokens, int n, int max_new, float temper
   return id;
 }
 
+// 0: a prompt is prefilled whole. n > 0: at most n of its tokens per step, beside the decoding sequences.
+void rbe_set_prefill_chunk(void* h, int n) { static_cast<EngineCore*>(h)->prefill_chunk = n; }
+
+// ---- externally driven sequences -----------------------------------------------------------
+// A fed sequence gets its tokens from the caller, portion by portion; it uses the same block pool and the same batch
+// builder as the scheduled ones, and is released with rbe_abort.
+i64 rbe_open(void* h) {
+  auto* e = static_cast<EngineCore*>(h);
+  auto s = std::make_unique<Seq>();
+  s->id = e->next_id++;
+  s->status = FED;
+  i64 id = s->id;
+  e->seqs[id] = std::move(s);
+  return id;
+}
+// Appends counts[i] tokens to sequence ids[i] and makes the n sequences the scheduled batch: those that continue with
+// a single token are its decode rows, the others its prefill rows. Blocks are taken from the pool. Returns the number
+// of packed tokens, or -1 unknown sequence, -2 out of blocks, -3 over max_batch / max_tokens_per_batch / max_model_len;
+// after an error nothing has changed.
+int rbe_feed(void* h, const i64* ids, const int* counts, int n, const int* tokens) {
+  auto* e = static_cast<EngineCore*>(h);
+  const int bs = e->kv.pool.block_size;
+  if (n > e->max_batch) return -3;
+  int total = 0, need = 0;
+  for (int i = 0; i < n; ++i) {
+    Seq* s = e->get(ids[i]);
+    if (s == nullptr || s->status != FED || counts[i] <= 0) return -1;
+    const int len = (int)s->tokens.size() + counts[i];
+    if (len > e->max_model_len) return -3;
+    need += (len + bs - 1) / bs - (int)s->blocks.size();
+    total += counts[i];
+  }
+  if (total > e->max_tokens_per_batch) return -3;
+  if (need > e->kv.num_free()) return -2;
+  e->sched_prefill.clear(); e->sched_decode.clear(); e->sched_preempted.clear();
+  for (int i = 0; i < n; ++i) {
+    Seq* s = e->get(ids[i]);
+    s->tokens.insert(s->tokens.end(), tokens, tokens + counts[i]);
+    tokens += counts[i];
+    s->n_prompt = s->n_target = (int)s->tokens.size();
+    while ((int)s->blocks.size() * bs < s->n_target) s->blocks.push_back(e->kv.take_block());
+    if (counts[i] == 1 && s->n_computed > 0) e->sched_decode.push_back(s->id);
+    else e->sched_prefill.push_back(s->id);
+  }
+  return total;
+}
+// The fed batch has run: its tokens are in the cache.
+void rbe_commit_fed(void* h) {
+  auto* e = static_cast<EngineCore*>(h);
+  for (auto* list : {&e->sched_decode, &e->sched_prefill})
+    for (i64 id : *list)
+      if (Seq* s = e->get(id)) s->n_computed = s->n_target;
+}
+
 int rbe_num_waiting(void* h) { return (int)static_cast<EngineCore*>(h)->waiting.size(); }
 int rbe_num_running(void* h) { return (int)static_cast<EngineCore*>(h)->running.size(); }
 int rbe_num_free_blocks(void* h) { return static_cast<EngineCore*>(h)->kv.num_free(); }
@@ -507,7 +586,7 @@ int rbe_schedule(void* h, int* counts) {
   int new_tokens = 0, max_new = 0, max_blocks = 0;
   for (i64 id : e->sched_prefill) {
     Seq* s = e->get(id);
-    int n = (int)s->tokens.size() - s->n_computed;
+    int n = s->n_target - s->n_computed;
     new_tokens += n;
     max_new = std::max(max_new, n);
     max_blocks = std::max(max_blocks, (int)s->blocks.size());
@@ -536,22 +615,22 @@ int rbe_get_scheduled(void* h, i64* prefill, i64* decode, i64* preempted) {
 }
 
 // Builds one packed batch from the last schedule: which = 1 the decode sequences (one new
-// token each), which = 2 the admitted prefill sequences (all tokens not yet in the cache).
-// block_tables is [rows, bt_stride]; rows beyond the batch are left untouched.
+// token each), which = 2 the prefill sequences (this step's portion of the tokens not yet in the
+// cache), which = 3 both, decode rows first. block_tables is [rows, bt_stride]; rows beyond the batch are left untouched.
 // Returns the number of packed tokens, or -1 if a buffer is too small.
 int rbe_build_batch(void* h, int which, int* tokens, int* positions, int* slots, int* cu_q, int* seq_lens,
                     int* block_tables, int bt_stride, float* temps, unsigned long long* seeds, int* sample_rows,
                     int max_tokens, int max_rows) {
   auto* e = static_cast<EngineCore*>(h);
   const int bs = e->kv.pool.block_size;
-  const std::vector<i64>& order = which == 1 ? e->sched_decode : e->sched_prefill;
+  const std::vector<i64> order = e->batch_order(which);
   if ((int)order.size() > max_rows) return -1;
   int t = 0, row = 0;
   cu_q[0] = 0;
   for (i64 id : order) {
     Seq* s = e->get(id);
-    const int n = (int)s->tokens.size();
-    const int start = which == 1 ? n - 1 : s->n_computed;
+    const int n = s->n_target;
+    const int start = s->n_computed;
     if (t + (n - start) > max_tokens) return -1;
     if ((int)s->blocks.size() > bt_stride) return -1;
     for (int p = start; p < n; ++p, ++t) {
@@ -570,19 +649,19 @@ int rbe_build_batch(void* h, int which, int* tokens, int* positions, int* slots,
   return t;
 }
 
-// Appends the sampled token of every row of the decode (which = 1) or prefill (which = 2)
-// batch, publishes blocks that just filled up to the prefix index, and applies the stop
+// Appends the sampled token of every row of the decode (which = 1), prefill (which = 2) or joint
+// (which = 3) batch, except rows whose prompt is not complete yet, publishes blocks that just filled up to the prefix index, and applies the stop
 // rules. Returns the number of sequences that finished.
 int rbe_commit(void* h, int which, const int* sampled, const float* logprobs, int n_rows) {
   auto* e = static_cast<EngineCore*>(h);
   const int bs = e->kv.pool.block_size;
-  const std::vector<i64> order = which == 1 ? e->sched_decode : e->sched_prefill;
+  const std::vector<i64> order = e->batch_order(which);
   if (n_rows != (int)order.size()) return -1;
   int n_fin = 0;
   for (int r = 0; r < n_rows; ++r) {
     Seq* s = e->get(order[r]);
     if (s == nullptr || s->status != RUNNING) continue;
-    s->n_computed = (int)s->tokens.size();
+    s->n_computed = s->n_target;
     if (e->kv.mode == 1) {
       const int n_full = s->n_computed / bs;
       for (int i = s->n_hashed_blocks; i < n_full && i < (int)s->blocks.size(); ++i) {
@@ -592,6 +671,7 @@ int rbe_commit(void* h, int which, const int* sampled, const float* logprobs, in
       }
       s->n_hashed_blocks = std::max(s->n_hashed_blocks, n_full);
     }
+    if (s->n_computed < (int)s->tokens.size()) continue;   // more of the prompt to come
     const int tok = sampled[r];
     s->tokens.push_back(tok);
     s->logprobs.push_back(logprobs[r]);
@@ -636,7 +716,7 @@ int rbe_abort(void* h, i64 id) {
   auto* e = static_cast<EngineCore*>(h);
   Seq* s = e->get(id);
   if (!s) return -1;
-  if (s->status == RUNNING) e->release_blocks(s, false);
+  if (s->status == RUNNING || s->status == FED) e->release_blocks(s, false);
   e->waiting.erase(std::remove(e->waiting.begin(), e->waiting.end(), id), e->waiting.end());
   e->running.erase(std::remove(e->running.begin(), e->running.end(), id), e->running.end());
   e->seqs.erase(id);

@@ -249,6 +249,113 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const __nv_bfloat1
 }
 
 // ------------------------------------------------------------------------------------------
+// Models with a 32-bit residual stream. The stream x is fp32 [T, d]; `xb` is the copy in the activation type TA
+// (bf16 when serving, fp32 in exact mode) that the projections read, row stride ldb, columns d..ldb stay zero.
+// ------------------------------------------------------------------------------------------
+template <typename TA> __device__ __forceinline__ TA to_act(float v);
+template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 to_act<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+__device__ __forceinline__ float from_act(float v) { return v; }
+__device__ __forceinline__ float from_act(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+// Sum over the CTA (blockDim.x a multiple of 32, at most 1024); every thread receives the total.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float t = lane < nw ? red[lane] : 0.f;
+  t = warp_sum(t);
+  __syncthreads();
+  return t;
+}
+
+template <typename TA>
+__global__ void embed_residual_kernel(const int* __restrict__ ids, const TA* __restrict__ table, float* __restrict__ x,
+                                      TA* __restrict__ xb, int d, long long ldb, int vocab, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  int id = ids[t];
+  if (id < 0 || id >= vocab) { if (threadIdx.x == 0) set_status(status, ST_BAD_INDEX); id = 0; }
+  const TA* src = table + (long long)id * ldb;
+  for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    const TA v = src[c];
+    x[t * d + c] = from_act(v);
+    xb[t * ldb + c] = v;
+  }
+}
+
+// Layer norm of fp32 rows with a two-pass variance; the row is kept in shared memory.
+//   y == nullptr : out = LN(x[rows[i]]) * w + b                     (rows == nullptr: row i)
+//   otherwise    : x += LN(y) * w + b, out = x                      (norm on the sublayer's output, residual add)
+// The caller folds a layer scale into w and b.
+template <typename TA>
+__global__ void layernorm_kernel(const float* __restrict__ y, long long ldy, float* __restrict__ x, const int* __restrict__ rows,
+                                 const float* __restrict__ w, const float* __restrict__ b, TA* __restrict__ out, long long ldo,
+                                 int d, float eps, int num_src_rows, int* status) {
+  extern __shared__ float ln_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long r = blockIdx.x;
+  long long xr = r;
+  if (rows != nullptr) {
+    xr = rows[r];
+    if (xr < 0 || xr >= num_src_rows) { if (threadIdx.x == 0) set_status(status, ST_BAD_INDEX); xr = 0; }
+  }
+  const float* src = y != nullptr ? y + r * ldy : x + xr * d;
+  float s = 0.f;
+  for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    const float v = src[c];
+    ln_row[c] = v;
+    s += v;
+  }
+  const float mean = block_sum(s, red) / (float)d;
+  float q = 0.f;
+  for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    const float v = ln_row[c] - mean;
+    q += v * v;
+  }
+  const float rstd = 1.f / sqrtf(block_sum(q, red) / (float)d + eps);
+  for (int c = threadIdx.x; c < d; c += blockDim.x) {
+    float v = fmaf((ln_row[c] - mean) * rstd, w[c], b[c]);
+    if (y != nullptr) {
+      v += x[r * d + c];
+      x[r * d + c] = v;
+    }
+    out[r * ldo + c] = to_act<TA>(v);
+  }
+}
+
+// Clamped gated unit: g = min(gate, limit), u = clamp(up, +-limit), out = g sigmoid(1.702 g) (u + 1). gate|up packed
+// as [T, 2F].
+__device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+template <typename TA>
+__global__ void clamped_glu_kernel(const TA* __restrict__ gu, TA* __restrict__ out, long long T, int F, float limit) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long n = T * F;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / F;
+    const int c = (int)(i - t * F);
+    out[i] = to_act<TA>(clamped_glu(from_act(gu[t * 2 * F + c]), from_act(gu[t * 2 * F + F + c]), limit));
+  }
+}
+
+// logits = cap * tanh(logits / cap), in place.
+__global__ void softcap_kernel(float* __restrict__ x, long long n, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
+    x[i] = cap * tanhf(x[i] / cap);
+}
+
+// ------------------------------------------------------------------------------------------
 // Sampling with log-probabilities, one CTA per row of fp32 logits [B, V].
 //   token  ~ softmax(logits / T)   via the Gumbel-max trick with a counter-based RNG
 //            (temperature == 0 -> argmax)
@@ -558,4 +665,46 @@ extern "C" int rb_transpose_bf16(const void* in, void* out, int rows, int cols, 
   dim3 block(32, 8);
   transpose_bf16_kernel<<<grid, block, 0, stream>>>((const __nv_bfloat16*)in, (__nv_bfloat16*)out, rows, cols);
   return RB_CHECK_LAUNCH();
+}
+
+// dtype of the activations: 0 bf16, 1 fp32
+#define RB_ACT_DISPATCH(dtype, CALL)            \
+  if ((dtype) == 0) { using TA = __nv_bfloat16; CALL } \
+  else if ((dtype) == 1) { using TA = float; CALL }    \
+  else return -1;
+
+extern "C" int rb_embed_residual(const int* ids, const void* table, float* x, void* xb, int dtype, int T, int d, long long ldb,
+                                 int vocab, int* status, cudaStream_t stream) {
+  if (T <= 0 || d <= 0 || ldb < d) return -1;
+  cudaError_t e;
+  RB_ACT_DISPATCH(dtype, e = launch_kernel(embed_residual_kernel<TA>, dim3(T), dim3(256), 0, stream, ids, (const TA*)table, x,
+                                           (TA*)xb, d, ldb, vocab, status);)
+  return e == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int rb_layernorm(const float* y, long long ldy, float* x, const int* rows, const float* w, const float* b, void* out,
+                            long long ldo, int dtype, int n, int d, float eps, int num_src_rows, int* status, cudaStream_t stream) {
+  if (n <= 0 || d <= 0 || d > 12288 || ldo < d || (y != nullptr && rows != nullptr)) return -1;
+  const int threads = d <= 512 ? 128 : 256;
+  cudaError_t e;
+  RB_ACT_DISPATCH(dtype, e = launch_kernel(layernorm_kernel<TA>, dim3(n), dim3(threads), (size_t)d * 4, stream, y, ldy, x, rows, w, b,
+                                           (TA*)out, ldo, d, eps, num_src_rows, status);)
+  return e == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int rb_clamped_glu(const void* gu, void* out, int dtype, long long T, int F, float limit, cudaStream_t stream) {
+  if (T <= 0 || F <= 0) return -1;
+  long long grid = (T * F + 255) / 256;
+  if (grid > 148 * 16) grid = 148 * 16;
+  cudaError_t e;
+  RB_ACT_DISPATCH(dtype, e = launch_kernel(clamped_glu_kernel<TA>, dim3((unsigned)grid), dim3(256), 0, stream, (const TA*)gu, (TA*)out,
+                                           T, F, limit);)
+  return e == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int rb_softcap(float* x, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0 || !(cap > 0.f)) return -1;
+  long long grid = (n + 255) / 256;
+  if (grid > 148 * 16) grid = 148 * 16;
+  return launch_kernel(softcap_kernel, dim3((unsigned)grid), dim3(256), 0, stream, x, n, cap) == cudaSuccess ? 0 : -11;
 }

@@ -40,26 +40,241 @@ class StepBatch:
     max_blocks: int
 
 
+@dataclass
+class PackedBatch:
+    """Device views (and the host copies the planning needs) of one packed batch of new tokens."""
+
+    rows: int
+    num_tokens: int
+    padded: int
+    max_new: int
+    tokens: torch.Tensor
+    positions: torch.Tensor
+    slots: torch.Tensor
+    cu_q: torch.Tensor
+    seq_lens: torch.Tensor
+    block_tables: torch.Tensor
+    host_cu_q: list[int]
+    host_seq_lens: list[int]
+
+
+class RunnerBase:
+    """What every model's runner shares: the static device buffers of a decode step and their pinned host staging, the
+    CUDA graphs per batch-size bucket, packed prefill staging and sampling. A subclass owns weights and cache and supplies
+
+    * ``_decode_body(bk)``: one decode step for ``bk`` staged rows, sampled into ``d_out_*``, logits left in ``a_logits``;
+    * ``_packed_forward(b)``: a packed batch of sequences with any number of new tokens each, up to the final residual;
+    * ``_row_logits(x, rows)``: fp32 logits of some of its rows;
+    * ``load_weights(weights)``, and ``cache_bytes_per_block(cfg, tp_size, dtype)`` for sizing the pool.
+    """
+
+    supports_f32 = False         # runs all in 32-bit on the GPU (EngineConfig.dtype = "float32")
+    joint_steps = False          # decode rows and prompt portions of a step run as one packed batch
+    short_first = False          # wants the packed batch ordered by portion length
+
+    def _init_step_buffers(self, vocab_padded: int) -> None:
+        device, mb = self.device, self.max_batch
+        # one int32 staging vector: tokens | positions | slots | seq_lens | temps | seeds(lo,hi)
+        self.meta_fields = 7
+        self.meta_dev = torch.zeros(self.meta_fields * mb, dtype=torch.int32, device=device)
+        self.meta_host = self._pinned(torch.zeros(self.meta_fields * mb, dtype=torch.int32))
+        self.bt_dev = torch.zeros(mb, self.max_blocks_per_seq, dtype=torch.int32, device=device)
+        self.bt_host = self._pinned(torch.zeros(mb, self.max_blocks_per_seq, dtype=torch.int32))
+        self.out_dev = torch.zeros(2 * mb, dtype=torch.int32, device=device)
+        self.out_host = self._pinned(torch.zeros(2 * mb, dtype=torch.int32))
+        m = self.meta_dev
+        self.d_tokens, self.d_pos, self.d_slots, self.d_lens = m[0:mb], m[mb:2 * mb], m[2 * mb:3 * mb], m[3 * mb:4 * mb]
+        self.d_temps = m[4 * mb:5 * mb].view(torch.float32)
+        self.d_seeds = m[5 * mb:7 * mb].view(torch.int64)
+        self.d_out_tokens = self.out_dev[0:mb]
+        self.d_out_logprobs = self.out_dev[mb:2 * mb].view(torch.float32)
+        self.a_logits = torch.empty(mb, vocab_padded, dtype=torch.float32, device=device)[:, :self.cfg.vocab_size]
+        self.graphs: dict[int, torch.cuda.CUDAGraph] = {}
+        self.launches_per_graph: dict[int, int] = {}
+        self.graph_pool = None
+        # prefill staging (pinned): tokens | positions | slots | cu_q | seq_lens | sample_rows | temps | seeds
+        T = self.max_prefill_tokens
+        self.pf_host = self._pinned(torch.zeros(3 * T + 6 * (mb + 1), dtype=torch.int32))
+        self.pf_dev = torch.zeros_like(self.pf_host, device=device)
+
+    def _init_geometry(self, cfg, *, device, num_kv_blocks: int, max_batch: int, max_model_len: int, max_prefill_tokens: int,
+                       use_cuda_graphs: bool, graph_batch_sizes: tuple[int, ...], dtype: torch.dtype) -> None:
+        # On a CUDA device every op is an sm_100a kernel. On CPU the same call sequence runs the PyTorch reference twins
+        # of the ops (fp32), which is how the scheduler, paged cache and radix reuse are exercised without a GPU.
+        self.on_gpu = device.type == "cuda"
+        assert max_batch % 2 == 0 and max_prefill_tokens % 2 == 0
+        self.cfg = cfg
+        self.device = device
+        self.dtype = dtype
+        self.max_batch = max_batch
+        self.max_model_len = max_model_len
+        self.max_blocks_per_seq = (max_model_len + BLOCK - 1) // BLOCK
+        self.max_prefill_tokens = max_prefill_tokens
+        self.num_kv_blocks = num_kv_blocks
+        self.use_cuda_graphs = use_cuda_graphs and self.on_gpu
+        self.graph_batch_sizes = tuple(sorted(b for b in graph_batch_sizes if b <= max_batch)) or (max_batch,)
+        if self.graph_batch_sizes[-1] < max_batch:
+            self.graph_batch_sizes += (max_batch,)
+        self.launches_per_decode_step = 0
+        self.row_align = 1
+
+    def _pinned(self, t: torch.Tensor) -> torch.Tensor:
+        return t.pin_memory() if self.on_gpu else t
+
+    def _sample(self, logits, temps, seeds, n: int) -> None:
+        if self.on_gpu:
+            ops.sample_with_logprobs(logits, temps, seeds, 0, None, self.d_out_tokens[:n], self.d_out_logprobs[:n])
+            return
+        # CPU twin: one seeded generator per row so a request reproduces in any batch slot
+        for r in range(n):
+            g = torch.Generator().manual_seed(int(seeds[r].item()) & 0x7FFFFFFFFFFFFFFF)
+            tok, lp = ops.sample_with_logprobs_reference(logits[r:r + 1].float(), temps[r:r + 1], g)
+            self.d_out_tokens[r] = int(tok[0])
+            self.d_out_logprobs[r] = float(lp[0])
+
+    def bucket(self, n: int) -> int:
+        for b in self.graph_batch_sizes:
+            if b >= n:
+                return b
+        return self.max_batch
+
+    def capture_graphs(self) -> None:
+        """Capture one decode graph per batch-size bucket (largest first, shared memory pool)."""
+        if not self.use_cuda_graphs:
+            return
+        self.d_lens.zero_()
+        self.d_slots.fill_(-1)
+        torch.cuda.synchronize(self.device)
+        stream = torch.cuda.Stream(self.device)
+        ops.set_pdl(True)  # decode kernels overlap their prologue with the previous kernel's tail
+        with torch.cuda.stream(stream):
+            for bk in sorted(self.graph_batch_sizes, reverse=True):
+                self._decode_body(bk)  # warm-up: sets kernel attributes outside capture
+                stream.synchronize()
+                g = torch.cuda.CUDAGraph()
+                n0 = LAUNCH_COUNT[0]
+                with torch.cuda.graph(g, pool=self.graph_pool, stream=stream):
+                    self._decode_body(bk)
+                self.launches_per_graph[bk] = LAUNCH_COUNT[0] - n0
+                if self.graph_pool is None:
+                    self.graph_pool = g.pool()
+                self.graphs[bk] = g
+        ops.set_pdl(False)
+        torch.cuda.synchronize(self.device)
+        ops.check_status(self.device)
+
+    def decode(self, n: int, max_blocks: int) -> None:
+        """Run one decode step for the ``n`` rows staged in ``meta_host`` / ``bt_host``.
+
+        Host->device: one copy of the packed metadata vector and one 2-D copy of the used
+        block-table columns. Device->host: one copy of tokens|logprobs into ``out_host``.
+        The caller synchronises before reading ``out_host``.
+        """
+        bk = self.bucket(n) if (self.use_cuda_graphs or self.row_align > 1) else max(n, 1)
+        self.meta_dev.copy_(self.meta_host, non_blocking=True)
+        self.bt_dev[:n, :max_blocks].copy_(self.bt_host[:n, :max_blocks], non_blocking=True)
+        g = self.graphs.get(bk)
+        if g is not None:
+            g.replay()
+        else:
+            self._decode_body(bk)
+        self.out_host.copy_(self.out_dev, non_blocking=True)
+
+    def stage_decode_padding(self, n: int) -> None:
+        """Mark rows n..bucket as padding (no KV write, empty context)."""
+        bk = self.bucket(n) if (self.use_cuda_graphs or self.row_align > 1) else max(n, 1)
+        mb = self.max_batch
+        mh = self.meta_host
+        if bk > n:
+            mh[0 * mb + n:0 * mb + bk] = 0
+            mh[1 * mb + n:1 * mb + bk] = 0
+            mh[2 * mb + n:2 * mb + bk] = -1
+            mh[3 * mb + n:3 * mb + bk] = 0
+            mh[4 * mb + n:4 * mb + bk] = 0
+
+    # ------------------------------------------------------------------ packed batches
+    def _stage_packed(self, rows: int, T: int, max_new: int, max_blocks: int) -> "PackedBatch":
+        """Copy the batch staged in ``pf_host`` / ``bt_host`` (filled by the engine core) to the device."""
+        o = self._pf_offsets()
+        ph = self.pf_host
+        Tp = -(-T // self.row_align) * self.row_align  # padded row count (tensor parallel only)
+        if Tp > T:
+            ph[o["tokens"] + T:o["tokens"] + Tp] = 0
+            ph[o["positions"] + T:o["positions"] + Tp] = 0
+            ph[o["slots"] + T:o["slots"] + Tp] = -1   # padding rows never touch the KV cache
+        self.pf_dev.copy_(ph, non_blocking=True)
+        self.bt_dev[:rows, :max_blocks].copy_(self.bt_host[:rows, :max_blocks], non_blocking=True)
+        pd = self.pf_dev
+        return PackedBatch(
+            rows=rows, num_tokens=T, padded=Tp, max_new=max_new, tokens=pd[o["tokens"]:o["tokens"] + Tp],
+            positions=pd[o["positions"]:o["positions"] + Tp], slots=pd[o["slots"]:o["slots"] + Tp],
+            cu_q=pd[o["cu_q"]:o["cu_q"] + rows + 1], seq_lens=pd[o["seq_lens"]:o["seq_lens"] + rows], block_tables=self.bt_dev[:rows],
+            host_cu_q=ph[o["cu_q"]:o["cu_q"] + rows + 1].tolist(), host_seq_lens=ph[o["seq_lens"]:o["seq_lens"] + rows].tolist())
+
+    def prefill(self, rows: int, T: int, max_new: int, max_blocks: int, views: dict[str, torch.Tensor] | None = None) -> None:
+        """Packed varlen pass over ``T`` new tokens of ``rows`` sequences; the last token of each is sampled.
+
+        Results land in ``out_host[:rows]`` / ``out_host[max_batch:max_batch+rows]`` after a synchronise.
+        """
+        b = self._stage_packed(rows, T, max_new, max_blocks)
+        o, pd = self._pf_offsets(), self.pf_dev
+        sample_rows = pd[o["sample_rows"]:o["sample_rows"] + rows]
+        temps = pd[o["temps"]:o["temps"] + rows].view(torch.float32)
+        seeds = pd[o["seeds"]:o["seeds"] + 2 * rows].view(torch.int64)
+        self._sample_rows(self._packed_forward(b), sample_rows, temps, seeds, rows)
+        self.out_host.copy_(self.out_dev, non_blocking=True)
+
+    def _sample_rows(self, x, sample_rows, temps, seeds, rows: int) -> None:
+        self._sample(self._row_logits(x, sample_rows), temps, seeds, rows)
+
+    def packed_logits(self, rows: int, T: int, max_new: int, max_blocks: int, wanted: list[int]) -> torch.Tensor | None:
+        """The same pass without sampling: fp32 logits ``[len(wanted), V]`` of the packed rows ``wanted``."""
+        x = self._packed_forward(self._stage_packed(rows, T, max_new, max_blocks))
+        if not wanted:
+            return None
+        return self._row_logits(x, torch.tensor(wanted, dtype=torch.int32).to(self.device))
+
+    # ------------------------------------------------------------------ teacher forcing
+    def score(self, token_ids: torch.Tensor) -> torch.Tensor:
+        """Full-sequence logits ``[T, V]`` (fp32) for one sequence, without touching live KV blocks.
+
+        Uses the tail of the KV pool as scratch blocks; meant for tests and logprob checks.
+        """
+        T = token_ids.numel()
+        nblk = (T + BLOCK - 1) // BLOCK
+        assert nblk <= self.num_kv_blocks
+        dev = self.device
+        blocks = torch.arange(self.num_kv_blocks - nblk, self.num_kv_blocks, dtype=torch.int32, device=dev)
+        pos = torch.arange(T, dtype=torch.int32, device=dev)
+        slots = blocks[torch.div(pos, BLOCK, rounding_mode="floor").long()] * BLOCK + pos % BLOCK
+        x = self._packed_forward(PackedBatch(
+            rows=1, num_tokens=T, padded=T, max_new=T, tokens=token_ids.to(device=dev, dtype=torch.int32), positions=pos,
+            slots=slots.to(torch.int32), cu_q=torch.tensor([0, T], dtype=torch.int32, device=dev),
+            seq_lens=torch.tensor([T], dtype=torch.int32, device=dev), block_tables=blocks[None].contiguous(),
+            host_cu_q=[0, T], host_seq_lens=[T]))
+        return self._row_logits(x, pos)
+
+    def _pf_offsets(self) -> dict[str, int]:
+        T, mb = self.max_prefill_tokens, self.max_batch
+        return {"tokens": 0, "positions": T, "slots": 2 * T, "cu_q": 3 * T, "seq_lens": 3 * T + (mb + 1),
+                "sample_rows": 3 * T + 2 * (mb + 1), "temps": 3 * T + 3 * (mb + 1), "seeds": 3 * T + 4 * (mb + 1)}
+
+
 class LayerWeights:
     __slots__ = ("ln1", "wqkv", "bqkv", "q_norm", "k_norm", "wo", "ln2", "wgu", "wd", "moe")
 
 
-class ModelRunner:
+class ModelRunner(RunnerBase):
     def __init__(self, cfg: ModelConfig, weights: dict[str, torch.Tensor], *, device: torch.device,
                  num_kv_blocks: int, max_batch: int, max_model_len: int, max_prefill_tokens: int,
                  use_cuda_graphs: bool = True, graph_batch_sizes: tuple[int, ...] = (), tp=None, ep=None,
                  dtype: torch.dtype = torch.bfloat16):
-        # On a CUDA device every op below is an sm_100a kernel. On CPU the same call sequence
-        # runs the PyTorch reference twins of the ops (fp32), which is how the scheduler,
-        # paged cache and radix reuse are exercised without a GPU.
-        self.on_gpu = device.type == "cuda"
-        if self.on_gpu:
+        if device.type == "cuda":
             assert cfg.head_dim in (64, 128), "attention kernels are built for head_dim 64 and 128"
             assert dtype == torch.bfloat16, "the CUDA kernels are bf16"
-        assert max_batch % 2 == 0 and max_prefill_tokens % 2 == 0
-        use_cuda_graphs = use_cuda_graphs and self.on_gpu
-        self.cfg = cfg
-        self.device = device
+        self._init_geometry(cfg, device=device, num_kv_blocks=num_kv_blocks, max_batch=max_batch, max_model_len=max_model_len,
+                            max_prefill_tokens=max_prefill_tokens, use_cuda_graphs=use_cuda_graphs,
+                            graph_batch_sizes=graph_batch_sizes, dtype=dtype)
         self.tp = tp
         # expert parallelism: attention and dense layers stay whole on every rank (each rank serves its own
         # requests), only the experts of the MoE layers are split; ``ep`` carries the peer-memory context
@@ -71,17 +286,7 @@ class ModelRunner:
         self.Hkv = cfg.num_kv_heads // self.tp_size
         self.D = cfg.head_dim
         self.F = (cfg.intermediate_size // self.tp_size) if cfg.intermediate_size else 0
-        self.max_batch = max_batch
-        self.max_model_len = max_model_len
-        self.max_blocks_per_seq = (max_model_len + BLOCK - 1) // BLOCK
-        self.max_prefill_tokens = max_prefill_tokens
-        self.num_kv_blocks = num_kv_blocks
-        self.use_cuda_graphs = use_cuda_graphs
-        self.graph_batch_sizes = tuple(sorted(b for b in graph_batch_sizes if b <= max_batch)) or (max_batch,)
-        if self.graph_batch_sizes[-1] < max_batch:
-            self.graph_batch_sizes += (max_batch,)
         self.scale = 1.0 / math.sqrt(self.D)
-        self.launches_per_decode_step = 0
         # gate|up projection with SwiGLU fused into the GEMM epilogue: weights are stored
         # interleaved in blocks of 128 gate rows + 128 up rows (tile width 256)
         self.swiglu_bn = 256
@@ -114,7 +319,6 @@ class ModelRunner:
             self.graph_batch_sizes = tuple(sorted({-(-b // ra) * ra for b in self.graph_batch_sizes}))
 
         bf = dtype
-        self.dtype = dtype
         d, L = cfg.hidden_size, cfg.num_layers
         self.embed = torch.empty(cfg.vocab_size, d, dtype=bf, device=device)
         self.final_norm = torch.empty(d, dtype=bf, device=device)
@@ -153,20 +357,7 @@ class ModelRunner:
 
         # ---- static decode buffers (graph inputs/outputs) ----
         mb = max_batch
-        # one int32 staging vector: tokens | positions | slots | seq_lens | temps | seeds(lo,hi)
-        self.meta_fields = 7
-        self.meta_dev = torch.zeros(self.meta_fields * mb, dtype=torch.int32, device=device)
-        self.meta_host = self._pinned(torch.zeros(self.meta_fields * mb, dtype=torch.int32))
-        self.bt_dev = torch.zeros(mb, self.max_blocks_per_seq, dtype=torch.int32, device=device)
-        self.bt_host = self._pinned(torch.zeros(mb, self.max_blocks_per_seq, dtype=torch.int32))
-        self.out_dev = torch.zeros(2 * mb, dtype=torch.int32, device=device)
-        self.out_host = self._pinned(torch.zeros(2 * mb, dtype=torch.int32))
-        m = self.meta_dev
-        self.d_tokens, self.d_pos, self.d_slots, self.d_lens = m[0:mb], m[mb:2 * mb], m[2 * mb:3 * mb], m[3 * mb:4 * mb]
-        self.d_temps = m[4 * mb:5 * mb].view(torch.float32)
-        self.d_seeds = m[5 * mb:7 * mb].view(torch.int64)
-        self.d_out_tokens = self.out_dev[0:mb]
-        self.d_out_logprobs = self.out_dev[mb:2 * mb].view(torch.float32)
+        self._init_step_buffers(cfg.vocab_size)
         # activations for decode
         self.a_x = tp.alloc((mb, d), bf) if (tp is not None and self.on_gpu) else torch.empty(mb, d, dtype=bf, device=device)
         self.a_h = torch.empty(mb, d, dtype=bf, device=device)
@@ -180,26 +371,18 @@ class ModelRunner:
         self.a_attn = torch.empty(mb, self.Hq * self.D, dtype=bf, device=device)
         self.a_gu = torch.empty(mb, 2 * self.F, dtype=bf, device=device) if self.F else None
         self.a_act = torch.empty(mb, self.F, dtype=bf, device=device) if self.F else None
-        self.a_logits = torch.empty(mb, cfg.vocab_size, dtype=torch.float32, device=device)
         # off by default: with four epilogue warps per SM the per-element sampling arithmetic (hash, two logs, exp)
         # is latency-bound and the fused launch measured 0.1 ms slower per 0.5B decode step than GEMM + sampler
         self.fused_sample = self.on_gpu and bool(os.environ.get("RB_FUSED_SAMPLE"))
         self.sample_ws = ops.lm_head_sample_workspace(mb, cfg.vocab_size, device) if self.fused_sample else None
         # split-KV partials for small batches (up to 64 rows x 32 splits)
         self.dec_ws = torch.empty(min(mb, 64) * self.Hq * 32 * (self.D + 2), dtype=torch.float32, device=device)
-        self.graphs: dict[int, torch.cuda.CUDAGraph] = {}
-        self.launches_per_graph: dict[int, int] = {}
-        self.graph_pool = None
-
-        # prefill staging (pinned): tokens | positions | slots | cu_q | seq_lens | sample_rows | temps | seeds
-        T = max_prefill_tokens
-        self.pf_host = self._pinned(torch.zeros(3 * T + 6 * (mb + 1), dtype=torch.int32))
-        self.pf_dev = torch.zeros_like(self.pf_host, device=device)
         # residual stream of the prefill pass; symmetric when ranks all-reduce into it
-        self.pf_x = tp.alloc((T + self.row_align, d), bf) if (tp is not None and self.on_gpu) else None
+        self.pf_x = tp.alloc((max_prefill_tokens + self.row_align, d), bf) if (tp is not None and self.on_gpu) else None
 
-    def _pinned(self, t: torch.Tensor) -> torch.Tensor:
-        return t.pin_memory() if self.on_gpu else t
+    @staticmethod
+    def cache_bytes_per_block(cfg: ModelConfig, tp_size: int, dtype: torch.dtype) -> int:
+        return cfg.num_layers * 2 * (cfg.num_kv_heads // tp_size) * BLOCK * cfg.head_dim * 2
 
     # ------------------------------------------------------------------ weights
     def _shard_rows(self, w: torch.Tensor, parts: int, idx: int) -> torch.Tensor:
@@ -376,148 +559,26 @@ class ModelRunner:
         logits = ops.gemm(h, self.lm_head, out=self.a_logits[:n], out_f32=True)
         self._sample(logits, temps, seeds, n)
 
-    def _sample(self, logits, temps, seeds, n: int) -> None:
-        if self.on_gpu:
-            ops.sample_with_logprobs(logits, temps, seeds, 0, None, self.d_out_tokens[:n], self.d_out_logprobs[:n])
-            return
-        # CPU twin: one seeded generator per row so a request reproduces in any batch slot
-        for r in range(n):
-            g = torch.Generator().manual_seed(int(seeds[r].item()) & 0x7FFFFFFFFFFFFFFF)
-            tok, lp = ops.sample_with_logprobs_reference(logits[r:r + 1].float(), temps[r:r + 1], g)
-            self.d_out_tokens[r] = int(tok[0])
-            self.d_out_logprobs[r] = float(lp[0])
-
-    def bucket(self, n: int) -> int:
-        for b in self.graph_batch_sizes:
-            if b >= n:
-                return b
-        return self.max_batch
-
-    def capture_graphs(self) -> None:
-        """Capture one decode graph per batch-size bucket (largest first, shared memory pool)."""
-        if not self.use_cuda_graphs:
-            return
-        self.d_lens.zero_()
-        self.d_slots.fill_(-1)
-        torch.cuda.synchronize(self.device)
-        stream = torch.cuda.Stream(self.device)
-        ops.set_pdl(True)  # decode kernels overlap their prologue with the previous kernel's tail
-        with torch.cuda.stream(stream):
-            for bk in sorted(self.graph_batch_sizes, reverse=True):
-                self._decode_body(bk)  # warm-up: sets kernel attributes outside capture
-                stream.synchronize()
-                g = torch.cuda.CUDAGraph()
-                n0 = LAUNCH_COUNT[0]
-                with torch.cuda.graph(g, pool=self.graph_pool, stream=stream):
-                    self._decode_body(bk)
-                self.launches_per_graph[bk] = LAUNCH_COUNT[0] - n0
-                if self.graph_pool is None:
-                    self.graph_pool = g.pool()
-                self.graphs[bk] = g
-        ops.set_pdl(False)
-        torch.cuda.synchronize(self.device)
-        ops.check_status(self.device)
-
-    def decode(self, n: int, max_blocks: int) -> None:
-        """Run one decode step for the ``n`` rows staged in ``meta_host`` / ``bt_host``.
-
-        Host->device: one copy of the packed metadata vector and one 2-D copy of the used
-        block-table columns. Device->host: one copy of tokens|logprobs into ``out_host``.
-        The caller synchronises before reading ``out_host``.
-        """
-        bk = self.bucket(n) if (self.use_cuda_graphs or self.row_align > 1) else max(n, 1)
-        self.meta_dev.copy_(self.meta_host, non_blocking=True)
-        self.bt_dev[:n, :max_blocks].copy_(self.bt_host[:n, :max_blocks], non_blocking=True)
-        g = self.graphs.get(bk)
-        if g is not None:
-            g.replay()
-        else:
-            self._decode_body(bk)
-        self.out_host.copy_(self.out_dev, non_blocking=True)
-
-    def stage_decode_padding(self, n: int) -> None:
-        """Mark rows n..bucket as padding (no KV write, empty context)."""
-        bk = self.bucket(n) if (self.use_cuda_graphs or self.row_align > 1) else max(n, 1)
-        mb = self.max_batch
-        mh = self.meta_host
-        if bk > n:
-            mh[0 * mb + n:0 * mb + bk] = 0
-            mh[1 * mb + n:1 * mb + bk] = 0
-            mh[2 * mb + n:2 * mb + bk] = -1
-            mh[3 * mb + n:3 * mb + bk] = 0
-            mh[4 * mb + n:4 * mb + bk] = 0
-
-    # ------------------------------------------------------------------ prefill
-    def prefill(self, rows: int, T: int, max_new: int, max_blocks: int, views: dict[str, torch.Tensor]) -> None:
-        """Packed varlen prefill of ``T`` new tokens over ``rows`` sequences.
-
-        ``views`` are slices of ``pf_host`` filled by the engine core. Results land in
-        ``out_host[:rows]`` / ``out_host[max_batch:max_batch+rows]`` after a synchronise.
-        """
+    # ------------------------------------------------------------------ packed batches
+    def _packed_forward(self, b: PackedBatch) -> torch.Tensor:
         cfg = self.cfg
-        dev = self.device
-        o = self._pf_offsets()
-        Tp = -(-T // self.row_align) * self.row_align  # padded row count (tensor parallel only)
-        if Tp > T:
-            ph = self.pf_host
-            ph[o["tokens"] + T:o["tokens"] + Tp] = 0
-            ph[o["positions"] + T:o["positions"] + Tp] = 0
-            ph[o["slots"] + T:o["slots"] + Tp] = -1   # padding rows never touch the KV cache
-        self.pf_dev.copy_(self.pf_host, non_blocking=True)
-        self.bt_dev[:rows, :max_blocks].copy_(self.bt_host[:rows, :max_blocks], non_blocking=True)
-        pd = self.pf_dev
-        tokens = pd[o["tokens"]:o["tokens"] + Tp]
-        positions = pd[o["positions"]:o["positions"] + Tp]
-        slots = pd[o["slots"]:o["slots"] + Tp]
-        cu_q = pd[o["cu_q"]:o["cu_q"] + rows + 1]
-        seq_lens = pd[o["seq_lens"]:o["seq_lens"] + rows]
-        sample_rows = pd[o["sample_rows"]:o["sample_rows"] + rows]
-        temps = pd[o["temps"]:o["temps"] + rows].view(torch.float32)
-        seeds = pd[o["seeds"]:o["seeds"] + 2 * rows].view(torch.int64)
-        x = ops.embedding(tokens, self.embed, out=self.pf_x[:Tp] if self.pf_x is not None else None)
+        T, Tp = b.num_tokens, b.padded
+        x = ops.embedding(b.tokens, self.embed, out=self.pf_x[:Tp] if self.pf_x is not None else None)
         h = torch.empty_like(x)
-        bt = self.bt_dev[:rows]
-        attn_out = torch.zeros(Tp, self.Hq, self.D, dtype=x.dtype, device=dev) if Tp > T else None
+        attn_out = torch.zeros(Tp, self.Hq, self.D, dtype=x.dtype, device=self.device) if Tp > T else None
 
         def attn_fn(li, q):
-            return ops.paged_prefill(q, self.k_cache[li], self.v_cache[li], bt, cu_q, seq_lens, max_new, self.scale,
+            return ops.paged_prefill(q, self.k_cache[li], self.v_cache[li], b.block_tables, b.cu_q, b.seq_lens, b.max_new, self.scale,
                                      cfg.sliding_window, out=attn_out)
 
-        self._forward_layers(x, h, Tp, positions, slots, attn_fn, static=False)
-        last = ops.embedding(sample_rows, x)  # row gather of the last token of every sequence
-        hl = ops.rmsnorm(last, self.final_norm, cfg.rms_norm_eps)
-        self._lm_head_sample(hl, temps, seeds, rows)
-        self.out_host.copy_(self.out_dev, non_blocking=True)
-        _ = dev
+        self._forward_layers(x, h, Tp, b.positions, b.slots, attn_fn, static=False)
+        return x
 
-    def _pf_offsets(self) -> dict[str, int]:
-        T, mb = self.max_prefill_tokens, self.max_batch
-        return {"tokens": 0, "positions": T, "slots": 2 * T, "cu_q": 3 * T, "seq_lens": 3 * T + (mb + 1),
-                "sample_rows": 3 * T + 2 * (mb + 1), "temps": 3 * T + 3 * (mb + 1), "seeds": 3 * T + 4 * (mb + 1)}
+    def _last_norm(self, x, rows) -> torch.Tensor:
+        return ops.rmsnorm(ops.embedding(rows, x), self.final_norm, self.cfg.rms_norm_eps)   # row gather, then the final norm
 
-    # ------------------------------------------------------------------ teacher forcing
-    def score(self, token_ids: torch.Tensor) -> torch.Tensor:
-        """Full-sequence logits ``[T, V]`` (fp32) for one sequence, without touching live KV blocks.
+    def _row_logits(self, x, rows) -> torch.Tensor:
+        return ops.gemm(self._last_norm(x, rows), self.lm_head, out_f32=True)
 
-        Uses the tail of the KV pool as scratch blocks; meant for tests and logprob checks.
-        """
-        T = token_ids.numel()
-        nblk = (T + BLOCK - 1) // BLOCK
-        assert nblk <= self.num_kv_blocks
-        dev = self.device
-        blocks = torch.arange(self.num_kv_blocks - nblk, self.num_kv_blocks, dtype=torch.int32, device=dev)
-        pos = torch.arange(T, dtype=torch.int32, device=dev)
-        slots = blocks[torch.div(pos, BLOCK, rounding_mode="floor").long()] * BLOCK + pos % BLOCK
-        bt = blocks[None].contiguous()
-        cu_q = torch.tensor([0, T], dtype=torch.int32, device=dev)
-        lens = torch.tensor([T], dtype=torch.int32, device=dev)
-        x = ops.embedding(token_ids.to(device=dev, dtype=torch.int32), self.embed)
-        h = torch.empty_like(x)
-
-        def attn_fn(li, q):
-            return ops.paged_prefill(q, self.k_cache[li], self.v_cache[li], bt, cu_q, lens, T, self.scale,
-                                     self.cfg.sliding_window)
-
-        self._forward_layers(x, h, T, pos, slots.to(torch.int32), attn_fn, static=False)
-        hl = ops.rmsnorm(x, self.final_norm, self.cfg.rms_norm_eps)
-        return ops.gemm(hl, self.lm_head, out_f32=True)
+    def _sample_rows(self, x, sample_rows, temps, seeds, rows: int) -> None:
+        self._lm_head_sample(self._last_norm(x, sample_rows), temps, seeds, rows)

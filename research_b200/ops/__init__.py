@@ -11,12 +11,19 @@ from .attention import (
     paged_prefill_reference,
 )
 from .elementwise import (
+    clamped_glu,
+    clamped_glu_reference,
+    embed_residual,
     embedding,
+    layernorm_reference,
+    layernorm_residual,
+    layernorm_rows,
     rmsnorm,
     rmsnorm_reference,
     rope_kv_append,
     rope_kv_append_reference,
     rope_table,
+    softcap,
     swiglu,
     swiglu_backward,
     swiglu_reference,
@@ -30,7 +37,17 @@ from .flash import (
     flash_paged_prefill,
 )
 from . import gemm as gemm_mod
-from .gemm import gemm, gemm_fp8, lm_head_sample, lm_head_sample_workspace, gemm_reference, gemm_symmetric, quantize_fp8, interleave_gate_up, linear
+from .gemm import gemm, gemm_f32, gemm_fp8, lm_head_sample, lm_head_sample_workspace, gemm_reference, gemm_symmetric, quantize_fp8, interleave_gate_up, linear
+from .latent import (
+    LatentGeometry,
+    head_gemm_absorb,
+    head_gemm_expand,
+    latent_append,
+    latent_attention,
+    latent_gather,
+    latent_num_splits,
+    latent_query,
+)
 from .sampling import sample_with_logprobs, sample_with_logprobs_reference, token_logprobs
 
 def set_pdl(on: bool) -> None:
@@ -38,8 +55,10 @@ def set_pdl(on: bool) -> None:
     attention, SwiGLU, embedding, sampling): consecutive kernels overlap prologue and tail."""
     from .. import _native
 
-    for lib, fn in (("rb_gemm", "rb_gemm_set_pdl"), ("rb_ops", "rb_ops_set_pdl"), ("rb_attn", "rb_attn_set_pdl")):
-        getattr(_native.load(lib), fn)(int(on))
+    for lib, fn in (("rb_gemm", "rb_gemm_set_pdl"), ("rb_ops", "rb_ops_set_pdl"), ("rb_attn", "rb_attn_set_pdl"),
+                    ("rb_latent", "rb_latent_set_pdl"), ("rb_gemm_f32", "rb_gemm_f32_set_pdl")):
+        if _native.available(lib):      # a partial build has only the libraries its models need
+            getattr(_native.load(lib), fn)(int(on))
 
 
 __all__ = [
@@ -48,5 +67,7 @@ __all__ = [
     "rmsnorm_reference", "rope_kv_append", "rope_kv_append_reference", "rope_table", "swiglu", "swiglu_backward",
     "swiglu_reference", "transpose", "gemm", "gemm_reference", "linear", "sample_with_logprobs",
     "sample_with_logprobs_reference", "token_logprobs", "set_pdl", "interleave_gate_up", "gemm_mod", "gemm_symmetric", "gemm_fp8", "quantize_fp8", "lm_head_sample", "lm_head_sample_workspace", "flash_attention", "flash_attn_varlen",
-    "flash_attn_varlen_backward", "flash_attn_varlen_reference", "flash_paged_prefill",
+    "flash_attn_varlen_backward", "flash_attn_varlen_reference", "flash_paged_prefill", "clamped_glu", "clamped_glu_reference",
+    "embed_residual", "layernorm_reference", "layernorm_residual", "layernorm_rows", "softcap", "gemm_f32", "LatentGeometry",
+    "head_gemm_absorb", "head_gemm_expand", "latent_append", "latent_attention", "latent_gather", "latent_num_splits", "latent_query",
 ]

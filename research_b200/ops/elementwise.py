@@ -28,7 +28,11 @@ def _lib() -> ctypes.CDLL:
         lib.rb_swiglu_bounded.restype = c_int
         lib.rb_embedding.argtypes = [c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_vp]
         lib.rb_transpose_bf16.argtypes = [c_vp, c_vp, c_int, c_int, c_vp]
-        for f in ("rb_rmsnorm", "rb_rope_kv_append", "rb_swiglu", "rb_swiglu_bwd", "rb_embedding", "rb_transpose_bf16"):
+        lib.rb_embed_residual.argtypes = [c_vp] * 4 + [c_int] * 3 + [c_ll, c_int, c_vp, c_vp]
+        lib.rb_layernorm.argtypes = [c_vp, c_ll] + [c_vp] * 5 + [c_ll, c_int, c_int, c_int, c_float, c_int, c_vp, c_vp]
+        lib.rb_clamped_glu.argtypes = [c_vp, c_vp, c_int, c_ll, c_int, c_float, c_vp]
+        lib.rb_softcap.argtypes = [c_vp, c_ll, c_float, c_vp]
+        for f in ("rb_embed_residual", "rb_layernorm", "rb_clamped_glu", "rb_softcap", "rb_rmsnorm", "rb_rope_kv_append", "rb_swiglu", "rb_swiglu_bwd", "rb_embedding", "rb_transpose_bf16"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -62,8 +66,14 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float = 1e-6, out: torch.Tens
 
 
 # ------------------------------------------------------------------------------- RoPE tables
-def rope_table(max_pos: int, head_dim: int, theta: float, device=None) -> torch.Tensor:
-    """``[max_pos, head_dim/2, 2]`` fp32 table of (cos, sin), HF ``inv_freq`` convention."""
+def rope_table(max_pos: int, head_dim: int, theta: float, device=None, exact: bool = False) -> torch.Tensor:
+    """``[max_pos, head_dim/2, 2]`` fp32 table of (cos, sin), HF ``inv_freq`` convention. ``exact`` forms the angles in
+    float64 first, so that the table is right to fp32 at every position."""
+    if exact:
+        freq = float(theta) ** (-torch.arange(0, head_dim, 2, dtype=torch.float64) / max(head_dim, 1))
+        ang = torch.outer(torch.arange(max_pos, dtype=torch.float64), freq)
+        tab = torch.stack([ang.cos(), ang.sin()], dim=-1).float().contiguous()
+        return tab.to(device) if device is not None else tab
     inv_freq = 1.0 / (theta ** (torch.arange(0, head_dim, 2, dtype=torch.float32) / head_dim))
     pos = torch.arange(max_pos, dtype=torch.float32)
     ang = torch.outer(pos, inv_freq)
@@ -197,3 +207,82 @@ def transpose(x: torch.Tensor) -> torch.Tensor:
     rc = _lib().rb_transpose_bf16(ptr(x), ptr(out), x.shape[0], x.shape[1], stream_handle(x.device))
     check_rc(rc, "rb_transpose_bf16")
     return out
+
+
+# ------------------------------------------------------------------------------- 32-bit residual stream
+_ACT = {torch.bfloat16: 0, torch.float32: 1}
+
+
+def embed_residual(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, xb: torch.Tensor) -> None:
+    """``x[t] = table[ids[t]]`` in fp32 and the same row in the activation type ``xb`` (leading columns; row strides of
+    ``table`` and ``xb`` agree)."""
+    T, d = ids.numel(), x.shape[1]
+    if not table.is_cuda:
+        x[:T] = table[ids.long(), :d].float()
+        xb[:T, :d] = table[ids.long(), :d]
+        return
+    assert ids.dtype == torch.int32 and ids.is_contiguous() and x.is_contiguous() and table.stride(0) == xb.stride(0)
+    rc = _lib().rb_embed_residual(ptr(ids), ptr(table), ptr(x), ptr(xb), _ACT[table.dtype], T, d, xb.stride(0), table.shape[0],
+                                  ptr(status_tensor(table.device)), stream_handle(table.device))
+    check_rc(rc, "rb_embed_residual")
+
+
+def layernorm_reference(v: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float) -> torch.Tensor:
+    c = v.float() - v.float().mean(-1, keepdim=True)
+    return c / torch.sqrt(c.pow(2).mean(-1, keepdim=True) + eps) * w + b
+
+
+def layernorm_residual(y: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float, x: torch.Tensor, xb: torch.Tensor) -> None:
+    """``x += layer_norm(y) * w + b`` on the fp32 stream, and ``xb`` = the new ``x`` in the activation type."""
+    n, d = x.shape
+    if not x.is_cuda:
+        x += layernorm_reference(y[:n, :d], w, b, eps)
+        xb[:n, :d] = x.to(xb.dtype)
+        return
+    assert y.dtype == torch.float32 and y.stride(1) == 1 and x.is_contiguous() and w.dtype == b.dtype == torch.float32
+    rc = _lib().rb_layernorm(ptr(y), y.stride(0), ptr(x), None, ptr(w), ptr(b), ptr(xb), xb.stride(0), _ACT[xb.dtype], n, d, eps, n,
+                             ptr(status_tensor(x.device)), stream_handle(x.device))
+    check_rc(rc, "rb_layernorm")
+
+
+def layernorm_rows(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float, out: torch.Tensor, rows: torch.Tensor | None = None) -> None:
+    """``out[i] = layer_norm(x[rows[i]]) * w + b`` (``rows`` None: all rows in order)."""
+    d = x.shape[1]
+    n = rows.numel() if rows is not None else x.shape[0]
+    if not x.is_cuda:
+        src = x if rows is None else x[rows.long()]
+        out[:n, :d] = layernorm_reference(src, w, b, eps).to(out.dtype)
+        return
+    assert x.is_contiguous() and x.dtype == torch.float32 and (rows is None or rows.dtype == torch.int32)
+    rc = _lib().rb_layernorm(None, 0, ptr(x), ptr(rows), ptr(w), ptr(b), ptr(out), out.stride(0), _ACT[out.dtype], n, d, eps, x.shape[0],
+                             ptr(status_tensor(x.device)), stream_handle(x.device))
+    check_rc(rc, "rb_layernorm")
+
+
+def clamped_glu_reference(gu: torch.Tensor, limit: float) -> torch.Tensor:
+    g, u = gu.float().chunk(2, dim=-1)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1)
+
+
+def clamped_glu(gu: torch.Tensor, limit: float, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, +-limit)`` for ``gu = [gate | up] [T, 2F]``."""
+    T, F2 = gu.shape
+    if out is None:
+        out = torch.empty(T, F2 // 2, dtype=gu.dtype, device=gu.device)
+    if not gu.is_cuda:
+        out.copy_(clamped_glu_reference(gu, limit))
+        return out
+    assert gu.is_contiguous() and out.is_contiguous()
+    check_rc(_lib().rb_clamped_glu(ptr(gu), ptr(out), _ACT[gu.dtype], T, F2 // 2, limit, stream_handle(gu.device)), "rb_clamped_glu")
+    return out
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap * tanh(x / cap)`` in place on fp32."""
+    if not x.is_cuda:
+        x.copy_(cap * torch.tanh(x / cap))
+        return x
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    check_rc(_lib().rb_softcap(ptr(x), x.numel(), cap, stream_handle(x.device)), "rb_softcap")
+    return x

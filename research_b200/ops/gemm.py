@@ -174,6 +174,33 @@ def _gemm2_gather(a, b, bias, residual, out, M, N, K, mn_major: bool, out_f32: b
     return out
 
 
+def _lib_f32() -> ctypes.CDLL:
+    lib = _native.load("rb_gemm_f32")
+    if not getattr(lib, "_rb_typed", False):
+        vp, i, ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
+        lib.rb_gemm_f32.argtypes = [vp] * 3 + [i] * 3 + [ll] * 3 + [i] + [ll] * 3 + [i, vp]
+        lib.rb_gemm_f32.restype = i
+        lib._rb_typed = True
+    return lib
+
+
+def gemm_f32_batched(a, b, out, M: int, N: int, K: int, batch: int, ld: tuple[int, int, int], step: tuple[int, int, int], b_kn: bool = False) -> None:
+    """``batch`` fp32 products ``C = A B^T`` (``b_kn``: ``A B``) at the given leading dimensions and batch strides."""
+    assert a.dtype == b.dtype == out.dtype == torch.float32 and a.is_cuda
+    rc = _lib_f32().rb_gemm_f32(a.data_ptr(), b.data_ptr(), out.data_ptr(), M, N, K, *ld, batch, *step, int(b_kn), stream_handle(a.device))
+    check_rc(rc, "rb_gemm_f32")
+
+
+def gemm_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``A @ B^T`` with fp32 operands, products and sums (no reduced-precision matrix mode)."""
+    assert a.dim() == b.dim() == 2 and a.stride(1) == b.stride(1) == 1 and a.shape[1] == b.shape[1]
+    M, N = a.shape[0], b.shape[0]
+    if out is None:
+        out = torch.empty(M, N, dtype=torch.float32, device=a.device)
+    gemm_f32_batched(a, b, out, M, N, a.shape[1], 1, (a.stride(0), b.stride(0), out.stride(0)), (0, 0, 0))
+    return out
+
+
 def gemm_reference(a, b, bias=None, residual=None, a_mn_major=False, b_mn_major=False, out_dtype=None):
     """fp32 PyTorch reference: ``op(a) @ op(b).T`` (+bias) (+residual)."""
     af = a.float().t() if a_mn_major else a.float()
@@ -258,6 +285,9 @@ def gemm(
             out.copy_(res)
             return out
         return res
+    if a.dtype == torch.float32 and b is not None and b.dtype == torch.float32:
+        assert bias is None and residual is None and not (a_mn_major or b_mn_major or swiglu) and norm_eps is None and alpha == beta == 1.0
+        return gemm_f32(a, b, out)
     if b_gather is not None:
         b = b_gather.staged          # [rows, cols] view of the staging matrix this launch fills
     assert a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16
@@ -624,5 +654,5 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias=None, residual=None, out=
     return y.reshape(*lead, weight.shape[0])
 
 
-__all__ = ["gemm", "gemm2", "lm_head_sample", "lm_head_sample_workspace", "gemm_fp8", "quantize_fp8", "gemm_symmetric", "gemm_reference", "linear", "interleave_gate_up", "swiglu_interleaved_reference", "RbGemmArgs", "EPI_STORE", "EPI_REDUCE_SCATTER", "EPI_ALL_REDUCE", "EPI_ALL_REDUCE_ONESHOT"]
+__all__ = ["gemm", "gemm2", "gemm_f32", "gemm_f32_batched", "lm_head_sample", "lm_head_sample_workspace", "gemm_fp8", "quantize_fp8", "gemm_symmetric", "gemm_reference", "linear", "interleave_gate_up", "swiglu_interleaved_reference", "RbGemmArgs", "EPI_STORE", "EPI_REDUCE_SCATTER", "EPI_ALL_REDUCE", "EPI_ALL_REDUCE_ONESHOT"]
 _ = ptr  # re-exported helper kept for wrappers that build RbGemmArgs themselves
