@@ -296,6 +296,7 @@ struct EngineCore {
   KVManager kv;
   int max_batch, max_tokens_per_batch, max_model_len;
   int prefill_chunk = 0;          // > 0: a prompt enters the cache at most this many tokens per step
+  bool short_first = false;
   std::unordered_map<i64, std::unique_ptr<Seq>> seqs;
   std::deque<i64> waiting;
   std::vector<i64> running;
@@ -331,7 +332,8 @@ struct EngineCore {
 
   // Blocks a waiting sequence needs beyond what the prefix cache can serve is not known until
   // admission; the scheduler budgets with the conservative full count like the reference.
-  bool admit(Seq* s) {
+  // `budget`: tokens this step still has room for (portions only).
+  bool admit(Seq* s, int budget = 1 << 30) {
     const int bs = kv.pool.block_size;
     const int n = (int)s->tokens.size();
     const int need = (n + bs - 1) / bs;
@@ -366,7 +368,7 @@ struct EngineCore {
     }
     s->n_cached = matched * bs;
     s->n_computed = matched * bs;
-    s->n_target = prefill_chunk > 0 ? std::min(n, s->n_computed + prefill_chunk) : n;
+    s->n_target = s->n_computed + portion(n - s->n_computed, budget);
     // only what this step computes is published now; the rest of a prompt that is prefilled in portions is published
     // as it is committed (hash mode) or when the sequence releases its blocks (radix mode)
     const int n_full = s->n_target / bs;
@@ -391,6 +393,20 @@ struct EngineCore {
       s->radix_node = deep;
     }
     return true;
+  }
+
+  // tokens of an unfinished prompt that enter the cache in one step
+  int portion(int remaining, int budget) const {
+    return prefill_chunk > 0 ? std::min(remaining, std::max(1, std::min(prefill_chunk, budget))) : remaining;
+  }
+
+  // Prefill rows in order of their portion's length (stable), for runners that treat short portions differently.
+  void order_prefill() {
+    if (!short_first) return;
+    std::stable_sort(sched_prefill.begin(), sched_prefill.end(), [&](i64 a, i64 b) {
+      const Seq *x = get(a), *y = get(b);
+      return x->n_target - x->n_computed < y->n_target - y->n_computed;
+    });
   }
 
   // sequences of the scheduled batch in row order: which = 1 decode, 2 prefill, 3 decode then prefill
@@ -447,7 +463,8 @@ struct EngineCore {
       }
       if (!ok) { sched_preempted.push_back(s->id); preempt(s); continue; }
       if (n - s->n_computed > 1) {    // in the middle of its prompt: the next portion
-        s->n_target = prefill_chunk > 0 ? std::min(n, s->n_computed + prefill_chunk) : n;
+        const int later = (int)(keep.size() - i) - 1;      // the sequences behind it take a token each
+        s->n_target = s->n_computed + portion(n - s->n_computed, max_tokens_per_batch - batch_tokens - later);
         sched_prefill.push_back(s->id);
       } else {
         s->n_target = n;
@@ -470,17 +487,19 @@ struct EngineCore {
       Seq* s = get(waiting.front());
       if (s == nullptr) { waiting.pop_front(); continue; }
       if ((int)(sched_prefill.size() + sched_decode.size()) >= max_batch) break;
-      const int n = prefill_chunk > 0 ? std::min((int)s->tokens.size(), prefill_chunk) : (int)s->tokens.size();
+      const int n = portion((int)s->tokens.size(), max_tokens_per_batch - batch_tokens);
+      if (prefill_chunk > 0 && batch_tokens >= max_tokens_per_batch) break;
       if (batch_tokens + n > max_tokens_per_batch && !(sched_prefill.empty() && sched_decode.empty())) break;
       // sequences preempted in this very step wait for the next one
       if (std::find(sched_preempted.begin(), sched_preempted.end(), s->id) != sched_preempted.end()) break;
-      if (!admit(s)) break;
+      if (!admit(s, max_tokens_per_batch - batch_tokens)) break;
       waiting.pop_front();
       s->status = RUNNING;
       running.push_back(s->id);
       sched_prefill.push_back(s->id);
       batch_tokens += s->n_target - s->n_computed;
     }
+    order_prefill();
   }
 
   void finish(Seq* s, int reason) {
@@ -521,8 +540,13 @@ i64 rbe_add_request(void* h, const int* tokens, int n, int max_new, float temper
   return id;
 }
 
-// 0: a prompt is prefilled whole. n > 0: at most n of its tokens per step, beside the decoding sequences.
-void rbe_set_prefill_chunk(void* h, int n) { static_cast<EngineCore*>(h)->prefill_chunk = n; }
+// n = 0: a prompt is prefilled whole. n > 0: at most n of its tokens per step, beside the decoding sequences, and no
+// more than the step's token budget leaves. short_first: prefill rows ordered by portion length.
+void rbe_set_prefill(void* h, int n, int short_first) {
+  auto* e = static_cast<EngineCore*>(h);
+  e->prefill_chunk = n;
+  e->short_first = short_first != 0;
+}
 
 // ---- externally driven sequences -----------------------------------------------------------
 // A fed sequence gets its tokens from the caller, portion by portion; it uses the same block pool and the same batch
@@ -565,6 +589,7 @@ int rbe_feed(void* h, const i64* ids, const int* counts, int n, const int* token
     if (counts[i] == 1 && s->n_computed > 0) e->sched_decode.push_back(s->id);
     else e->sched_prefill.push_back(s->id);
   }
+  e->order_prefill();
   return total;
 }
 // The fed batch has run: its tokens are in the cache.
@@ -606,12 +631,13 @@ int rbe_schedule(void* h, int* counts) {
   return counts[0] + counts[1];
 }
 
+// Returns the number of decode rows.
 int rbe_get_scheduled(void* h, i64* prefill, i64* decode, i64* preempted) {
   auto* e = static_cast<EngineCore*>(h);
   if (prefill) std::copy(e->sched_prefill.begin(), e->sched_prefill.end(), prefill);
   if (decode) std::copy(e->sched_decode.begin(), e->sched_decode.end(), decode);
   if (preempted) std::copy(e->sched_preempted.begin(), e->sched_preempted.end(), preempted);
-  return 0;
+  return (int)e->sched_decode.size();
 }
 
 // Builds one packed batch from the last schedule: which = 1 the decode sequences (one new

@@ -20,9 +20,11 @@ import torch
 
 from .. import _native
 from ..models.config import ModelConfig
+from ..models.registry import runner_class
+from ..models.stack import LayerStackConfig
 from ..models.weights import load_safetensors_dir
 from ..ops import check_status
-from .model_runner import BLOCK, ModelRunner
+from .model_runner import BLOCK
 from .types import EngineConfig, SamplingParams, TrainingSample
 
 _LL, _I, _F, _VP, _ULL = ctypes.c_longlong, ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_ulonglong
@@ -37,6 +39,11 @@ def _core_lib():
         lib.rbe_destroy.argtypes = [_VP]
         lib.rbe_add_request.restype = _LL
         lib.rbe_add_request.argtypes = [_VP, _VP, _I, _I, _F, _ULL, _VP, _I, _I]
+        lib.rbe_set_prefill.argtypes = [_VP, _I, _I]
+        lib.rbe_open.restype = _LL
+        lib.rbe_open.argtypes = [_VP]
+        lib.rbe_feed.argtypes = [_VP, _VP, _VP, _I, _VP]
+        lib.rbe_commit_fed.argtypes = [_VP]
         for f in ("rbe_num_waiting", "rbe_num_running", "rbe_num_free_blocks", "rbe_num_finished", "rbe_check_invariants"):
             getattr(lib, f).argtypes = [_VP]
         lib.rbe_schedule.argtypes = [_VP, _VP]
@@ -54,7 +61,7 @@ def _core_lib():
 
 
 class InferenceEngine:
-    def __init__(self, config: EngineConfig, model_config: ModelConfig | None = None,
+    def __init__(self, config: EngineConfig, model_config: ModelConfig | LayerStackConfig | None = None,
                  weights: dict[str, torch.Tensor] | None = None, tokenizer=None,
                  device: torch.device | str | None = None, tp=None, ep=None) -> None:
         assert config.block_size == BLOCK, "the KV kernels use 16-token blocks"
@@ -78,9 +85,15 @@ class InferenceEngine:
                 self.tokenizer = None
         self.max_tokens_per_batch = config.max_tokens_per_batch or min(config.max_batch_size * 512, 16384)
         on_gpu = self.device.type == "cuda"
-        dtype = torch.bfloat16 if on_gpu else torch.float32
-        num_blocks = config.num_kv_blocks or self._size_kv_cache(model_config, tp, ep)
-        self.runner = ModelRunner(
+        runner_type = runner_class(model_config)
+        if config.dtype not in ("bfloat16", "float32"):
+            raise ValueError(f"EngineConfig.dtype {config.dtype!r}: bfloat16 or float32")
+        if on_gpu and config.dtype == "float32" and not runner_type.supports_f32:
+            raise ValueError(f"{runner_type.__name__} has no 32-bit mode on the GPU")
+        dtype = torch.bfloat16 if on_gpu and config.dtype == "bfloat16" else torch.float32
+        self.runner_type = runner_type
+        num_blocks = config.num_kv_blocks or self._size_kv_cache(model_config, tp, ep, dtype)
+        self.runner = runner_type(
             model_config, weights, device=self.device, num_kv_blocks=num_blocks, max_batch=config.max_batch_size,
             max_model_len=config.max_model_len, max_prefill_tokens=self.max_tokens_per_batch + 2 * BLOCK,
             use_cuda_graphs=config.use_cuda_graphs, graph_batch_sizes=config.graph_batch_sizes, tp=tp, ep=ep, dtype=dtype)
@@ -93,6 +106,9 @@ class InferenceEngine:
         self._core = self._lib.rbe_create(num_blocks, BLOCK, _CACHE_MODES[config.cache_type], config.max_batch_size,
                                           self.max_tokens_per_batch, config.max_model_len)
         assert self._core, "engine core allocation failed"
+        # runners that take portions beside decoded tokens get long prompts in pieces that fit a step
+        chunk = config.prefill_chunk or (self.max_tokens_per_batch if runner_type.joint_steps else 0)
+        self._lib.rbe_set_prefill(self._core, chunk, int(runner_type.short_first))
         self.num_kv_blocks = num_blocks
         self.weight_version = 0
         self.steps = 0
@@ -110,9 +126,9 @@ class InferenceEngine:
         self.last_step_rows = (0, 0)
 
     # ---------------------------------------------------------------- sizing
-    def _size_kv_cache(self, cfg: ModelConfig, tp, ep=None) -> int:
+    def _size_kv_cache(self, cfg: ModelConfig | LayerStackConfig, tp, ep=None, dtype: torch.dtype = torch.bfloat16) -> int:
         tp_size = tp.world if tp is not None else 1
-        per_block = cfg.num_layers * 2 * (cfg.num_kv_heads // tp_size) * BLOCK * cfg.head_dim * 2
+        per_block = self.runner_type.cache_bytes_per_block(cfg, tp_size, dtype)
         want_tokens = self.config.max_batch_size * self.config.max_model_len
         want = -(-want_tokens // BLOCK)
         if self.device.type == "cuda":
@@ -205,41 +221,89 @@ class InferenceEngine:
         if n_prefill + n_decode == 0:
             return []
         mb = r.max_batch
-        if n_decode > 0:
-            mh = r.meta_host
-            base = mh.data_ptr()
-            T = lib.rbe_build_batch(
-                core, 1, base, base + 4 * mb, base + 8 * mb, r.pf_host.data_ptr() + 4 * r._pf_offsets()["cu_q"],
-                base + 12 * mb, r.bt_host.data_ptr(), r.max_blocks_per_seq, base + 16 * mb, base + 20 * mb,
-                r.pf_host.data_ptr() + 4 * r._pf_offsets()["sample_rows"], mb, mb)
-            assert T == n_decode, T
-            max_blocks = self._max_blocks_in(r.meta_host[3 * mb:3 * mb + n_decode])
-            r.stage_decode_padding(n_decode)
-            r.decode(n_decode, max_blocks)
-            self._sync()
+        joint = r.joint_steps and n_prefill > 0 and n_decode > 0
+        if n_decode > 0 and not joint:
+            self._run_decode(n_decode)
             out_i = r.out_host
             fin = lib.rbe_commit(core, 1, out_i.data_ptr(), out_i.data_ptr() + 4 * mb, n_decode)
             assert fin >= 0
         if n_prefill > 0:
-            o = r._pf_offsets()
-            base = r.pf_host.data_ptr()
-            T = lib.rbe_build_batch(
-                core, 2, base + 4 * o["tokens"], base + 4 * o["positions"], base + 4 * o["slots"], base + 4 * o["cu_q"],
-                base + 4 * o["seq_lens"], r.bt_host.data_ptr(), r.max_blocks_per_seq, base + 4 * o["temps"],
-                base + 4 * o["seeds"], base + 4 * o["sample_rows"], r.max_prefill_tokens, mb)
-            assert T > 0, f"prefill batch does not fit the staging buffers ({T})"
-            cu = r.pf_host[o["cu_q"]:o["cu_q"] + n_prefill + 1]
-            max_new = int((cu[1:] - cu[:-1]).max())
-            max_blocks = self._max_blocks_in(r.pf_host[o["seq_lens"]:o["seq_lens"] + n_prefill])
-            r.prefill(n_prefill, T, max_new, max_blocks, {})
+            # decode rows of a joint step come first and are sampled in the same pass
+            which, n_rows = (3, n_decode + n_prefill) if joint else (2, n_prefill)
+            r.prefill(*self._build_packed(which, n_rows))
             self._sync()
             out_i = r.out_host
-            fin = lib.rbe_commit(core, 2, out_i.data_ptr(), out_i.data_ptr() + 4 * mb, n_prefill)
+            fin = lib.rbe_commit(core, which, out_i.data_ptr(), out_i.data_ptr() + 4 * mb, n_rows)
             assert fin >= 0
         self.steps += 1
         if self.device.type == "cuda" and self.steps % 256 == 0:
             check_status(self.device)
         return self._collect_finished()
+
+    def _run_decode(self, n: int) -> None:
+        """Stage the scheduled decode rows, run one decode step and wait for it."""
+        r = self.runner
+        mb, o = r.max_batch, r._pf_offsets()
+        base, pf = r.meta_host.data_ptr(), r.pf_host.data_ptr()
+        T = self._lib.rbe_build_batch(
+            self._core, 1, base, base + 4 * mb, base + 8 * mb, pf + 4 * o["cu_q"], base + 12 * mb, r.bt_host.data_ptr(),
+            r.max_blocks_per_seq, base + 16 * mb, base + 20 * mb, pf + 4 * o["sample_rows"], mb, mb)
+        assert T == n, T
+        max_blocks = self._max_blocks_in(r.meta_host[3 * mb:3 * mb + n])
+        r.stage_decode_padding(n)
+        r.decode(n, max_blocks)
+        self._sync()
+
+    def _build_packed(self, which: int, n_rows: int) -> tuple[int, int, int, int]:
+        """Stage the scheduled prefill (2) or decode + prefill (3) rows; returns the arguments of a packed pass."""
+        r = self.runner
+        o, base = r._pf_offsets(), r.pf_host.data_ptr()
+        T = self._lib.rbe_build_batch(
+            self._core, which, base + 4 * o["tokens"], base + 4 * o["positions"], base + 4 * o["slots"], base + 4 * o["cu_q"],
+            base + 4 * o["seq_lens"], r.bt_host.data_ptr(), r.max_blocks_per_seq, base + 4 * o["temps"],
+            base + 4 * o["seeds"], base + 4 * o["sample_rows"], r.max_prefill_tokens, r.max_batch)
+        assert T > 0, f"packed batch does not fit the staging buffers ({T})"
+        cu = r.pf_host[o["cu_q"]:o["cu_q"] + n_rows + 1]
+        return n_rows, T, int((cu[1:] - cu[:-1]).max()), self._max_blocks_in(r.pf_host[o["seq_lens"]:o["seq_lens"] + n_rows])
+
+    # ---------------------------------------------------------------- given tokens instead of sampled ones
+    def open_stream(self) -> int:
+        """A sequence whose tokens the caller supplies with ``feed`` (replaying a trace, scoring); it holds cache blocks
+        until ``close_stream``."""
+        return int(self._lib.rbe_open(self._core))
+
+    def feed(self, entries: list[tuple[int, list[int], list[int]]]) -> torch.Tensor | None:
+        """One step over ``(stream, next tokens, wanted places among them)`` entries, run as one batch from the cache that
+        earlier steps left: portions of any length beside single tokens. Returns fp32 logits ``[wanted, V]`` in the order
+        of the entries and of their places, or None when nothing is wanted."""
+        assert entries and len({e[0] for e in entries}) == len(entries), "one entry per stream"
+        lib, core, r = self._lib, self._core, self.runner
+        n = len(entries)
+        flat = [t for _, toks, _ in entries for t in toks]
+        rc = lib.rbe_feed(core, (_LL * n)(*[e[0] for e in entries]), (_I * n)(*[len(e[1]) for e in entries]), n, (_I * len(flat))(*flat))
+        if rc < 0:
+            raise RuntimeError({-1: "feed: unknown stream or an entry without tokens", -2: "feed: the KV cache is full",
+                                -3: "feed: more tokens than the engine was made for"}[rc])
+        pre, dec = (_LL * n)(), (_LL * n)()
+        n_dec = lib.rbe_get_scheduled(core, pre, dec, None)
+        order = list(dec[:n_dec]) + list(pre[:n - n_dec])
+        count = {e[0]: len(e[1]) for e in entries}
+        first, at = {}, 0                                  # packed row of every stream's first token
+        for s in order:
+            first[s] = at
+            at += count[s]
+        wanted = [first[s] + w for s, _, places in entries for w in places]
+        if n_dec == n:
+            self._run_decode(n)
+            out = r.a_logits[:n].index_select(0, torch.tensor(wanted, device=self.device)) if wanted else None
+        else:
+            out = r.packed_logits(*self._build_packed(3, n), wanted)
+            self._sync()
+        lib.rbe_commit_fed(core)
+        return out
+
+    def close_stream(self, stream: int) -> None:
+        self._lib.rbe_abort(self._core, stream)
 
     def _idle_pass(self) -> None:
         """A decode pass over padding rows only: it feeds every MoE layer one (tiny) batch, which is what the peers'

@@ -88,7 +88,8 @@ class RunnerBase:
         self.d_seeds = m[5 * mb:7 * mb].view(torch.int64)
         self.d_out_tokens = self.out_dev[0:mb]
         self.d_out_logprobs = self.out_dev[mb:2 * mb].view(torch.float32)
-        self.a_logits = torch.empty(mb, vocab_padded, dtype=torch.float32, device=device)[:, :self.cfg.vocab_size]
+        self.logits_padded = torch.empty(mb, vocab_padded, dtype=torch.float32, device=device)
+        self.a_logits = self.logits_padded[:, :self.cfg.vocab_size]
         self.graphs: dict[int, torch.cuda.CUDAGraph] = {}
         self.launches_per_graph: dict[int, int] = {}
         self.graph_pool = None

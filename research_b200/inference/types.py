@@ -67,10 +67,11 @@ class EngineConfig:
     tensor_parallel_size: int = 1
     expert_parallel_size: int = 1
     max_tokens_per_batch: int = 0          # 0: max_batch_size * 512
+    prefill_chunk: int = 0                 # > 0: a prompt enters the cache in portions of at most this many tokens per step
     num_kv_blocks: int = 0                 # 0: sized from gpu_memory_utilization
     use_cuda_graphs: bool = True
     graph_batch_sizes: tuple[int, ...] = DEFAULT_GRAPH_BATCHES
-    dtype: str = "bfloat16"
+    dtype: str = "bfloat16"                # "float32": all in 32-bit on the GPU too, for models whose runner has that mode
     seed: int = 0
     ignore_eos: bool = False
 

@@ -34,6 +34,8 @@ from .flash import (
     flash_attn_varlen,
     flash_attn_varlen_backward,
     flash_attn_varlen_reference,
+    flash_latent_prefill,
+    flash_latent_supported,
     flash_paged_prefill,
 )
 from . import gemm as gemm_mod
@@ -67,7 +69,7 @@ __all__ = [
     "rmsnorm_reference", "rope_kv_append", "rope_kv_append_reference", "rope_table", "swiglu", "swiglu_backward",
     "swiglu_reference", "transpose", "gemm", "gemm_reference", "linear", "sample_with_logprobs",
     "sample_with_logprobs_reference", "token_logprobs", "set_pdl", "interleave_gate_up", "gemm_mod", "gemm_symmetric", "gemm_fp8", "quantize_fp8", "lm_head_sample", "lm_head_sample_workspace", "flash_attention", "flash_attn_varlen",
-    "flash_attn_varlen_backward", "flash_attn_varlen_reference", "flash_paged_prefill", "clamped_glu", "clamped_glu_reference",
+    "flash_attn_varlen_backward", "flash_attn_varlen_reference", "flash_paged_prefill", "flash_latent_prefill", "flash_latent_supported", "clamped_glu", "clamped_glu_reference",
     "embed_residual", "layernorm_reference", "layernorm_residual", "layernorm_rows", "softcap", "gemm_f32", "LatentGeometry",
     "head_gemm_absorb", "head_gemm_expand", "latent_append", "latent_attention", "latent_gather", "latent_num_splits", "latent_query",
 ]

@@ -185,3 +185,33 @@ def flash_attention(q, k, v, cu_q, cu_k, max_seqlen_q: int, max_seqlen_k: int, c
                     scale=None):
     """Autograd entry point used by the training model."""
     return FlashAttnVarlen.apply(q, k, v, cu_q, cu_k, max_seqlen_q, max_seqlen_k, causal, window, scale)
+
+
+# ------------------------------------------------------------------------------- latent attention, expanded form
+def flash_latent_supported(geo) -> bool:
+    """Padded head sizes the tensor-core kernel is built for."""
+    return geo.dp in (64, 128) and geo.rp == 64 and geo.vp in (64, 128)
+
+
+def flash_latent_prefill(q, k, rot, v, geo, cu_q, cu_k, sink, gate, out, *, scale: float, window: int, max_q: int, rows: int) -> None:
+    """Attention of packed new tokens over multiplied-out keys and values: ``q [T, H*(dp+rp)]`` (rotated), ``k [S, H*dp]``,
+    the rotated key part ``rot [S, rp]`` shared by all heads, ``v [S, H*vp]``. Sequence ``b`` owns the query rows
+    ``cu_q[b]..cu_q[b+1]`` (absolute rows of ``q`` and ``out [T, H*vp]``) and the key rows ``cu_k[b]..cu_k[b+1]``, which end with
+    its new tokens; a causal window, ``exp(sink_h)`` in the denominator, head outputs times ``gate [T, H]``."""
+    B, H = cu_q.numel() - 1, geo.heads
+    if not q.is_cuda:
+        for b in range(B):
+            t0, t1, s0, s1 = int(cu_q[b]), int(cu_q[b + 1]), int(cu_k[b]), int(cu_k[b + 1])
+            qb = q[t0:t1].view(t1 - t0, H, geo.dp + geo.rp).float()
+            s = torch.einsum("thd,khd->htk", qb[..., :geo.dp], k[s0:s1].view(-1, H, geo.dp).float())
+            s = (s + torch.einsum("thr,kr->htk", qb[..., geo.dp:], rot[s0:s1].float())) * scale
+            pos = torch.arange(t1 - t0) + (s1 - s0) - (t1 - t0)
+            key = torch.arange(s1 - s0)
+            s = s.masked_fill(((key[None] > pos[:, None]) | (key[None] <= pos[:, None] - window))[None], float("-inf"))
+            p = torch.cat([s, sink.view(H, 1, 1).expand(H, t1 - t0, 1)], -1).softmax(-1)[..., :-1]
+            o = torch.einsum("htk,khv->thv", p, v[s0:s1].view(-1, H, geo.vp).float()) * gate[t0:t1, :, None]
+            out[t0:t1] = o.reshape(t1 - t0, H * geo.vp).to(out.dtype)
+        return
+    rc = _lib().rb_flash_latent(ptr(q), ptr(k), ptr(rot), ptr(v), ptr(out), ptr(cu_q), ptr(cu_k), ptr(sink), ptr(gate), B, H, rows, k.shape[0],
+                                max_q, geo.dp, geo.vp, window, scale, ptr(status_tensor(q.device)), stream_handle(q.device))
+    check_rc(rc, "rb_flash_latent")

@@ -146,14 +146,19 @@ _ROW_DST: dict[tuple, torch.Tensor] = {}
 
 
 def _head_tiles(H: int, n: int, stride: int, N: int, b_step: int, bn: int, device) -> tuple[torch.Tensor, torch.Tensor, int]:
-    """Device tile table of ``H`` products over rows ``[h*stride, h*stride + n)``; cached, so captured graphs keep it."""
+    """Device tile table of ``H`` products over rows ``[h*stride, h*stride + n)``, cached."""
     key = (H, n, stride, N, b_step, bn, device.index)
     if key not in _HEAD_TILES:
-        if len(_HEAD_TILES) > 8192:
-            raise RuntimeError("too many per-head tile tables")
+        if len(_HEAD_TILES) >= 4096:         # captured graphs keep theirs alive through live_tables()
+            _HEAD_TILES.clear()
         rows = [(h * stride + m, min(128, n - m), h * b_step, n0) for h in range(H) for n0 in range(0, N, bn) for m in range(0, n, 128)]
         _HEAD_TILES[key] = (torch.tensor(rows, dtype=torch.int32).to(device), torch.tensor([len(rows)], dtype=torch.int32).to(device), len(rows))
     return _HEAD_TILES[key]
+
+
+def live_tables() -> list:
+    """The device tables made so far; whoever captured launches into a graph holds on to them."""
+    return list(_HEAD_TILES.values()) + list(_ROW_DST.values())
 
 
 def _head_bn(H: int, n: int, N: int, least: int) -> int:
