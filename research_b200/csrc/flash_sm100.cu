@@ -776,6 +776,361 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd2_kernel(const __grid_
   }
 }
 
+// ------------------------------------------------------------------------------------------
+// Forward for latent attention in its expanded form (ops/latent.py): 128 query rows of one head per CTA. A key is the
+// head's own part (DN columns of K) followed by 64 rotated columns shared by all heads, so a key tile is loaded from two
+// tensors; values have DV columns. Sliding window, causal, dense key rows per sequence. The softmax denominator also holds
+// exp(sink[h]), and the output row is scaled by gate[t, h].
+// Same roles and pipeline as flash_fwd_kernel; wider keys leave room for two K slots, one V slot and one P buffer.
+// ------------------------------------------------------------------------------------------
+struct FlashLatentParams {
+  CUtensorMap q_map;    // [T, H*(DN+64)]
+  CUtensorMap k_map;    // [S, H*DN]
+  CUtensorMap r_map;    // [S, 64]
+  CUtensorMap v_map;    // [S, H*DV]
+  __nv_bfloat16* out;   // [T, H*DV]
+  const int* cu_q;
+  const int* cu_k;
+  const float* sink;    // [H]
+  const float* gate;    // [T, H]
+  int H, window;
+  float scale_log2;
+  int* status;
+};
+
+template <int DN, int DV>
+struct FlashLatentCfg {
+  static constexpr int DK = DN + 64;
+  static constexpr int kKBytes = FA_BN * DK * 2;            // a K tile, and the Q tile
+  static constexpr int kVBytes = FA_BN * DV * 2;
+  static constexpr int kPBytes = FA_BM * FA_BN * 2;
+  static constexpr int kSmemBytes = 1024 + 3 * kKBytes + kVBytes + kPBytes;
+};
+
+template <int DN, int DV>
+__global__ void __launch_bounds__(FA_THREADS, 1) flash_latent_kernel(const __grid_constant__ FlashLatentParams p) {
+  using Cfg = FlashLatentCfg<DN, DV>;
+  constexpr int DK = Cfg::DK;
+  constexpr int CHUNK_BYTES = FA_BN * 128;
+  extern __shared__ __align__(128) uint8_t smem_raw[];
+  __shared__ __align__(8) uint64_t q_full, k_full[2], k_empty[2], v_full, v_empty;
+  __shared__ __align__(8) uint64_t s_full[2], s_empty[2], p_full, p_empty, o_done, xch_bar[4];
+  __shared__ float xch[2][2][FA_BM];
+  __shared__ uint32_t tmem_base_smem;
+  __shared__ int abort_flag;
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int b = blockIdx.z, h = blockIdx.y;
+  const int q_tile = gridDim.x - 1 - blockIdx.x;
+  const int q_begin = p.cu_q[b];
+  const int q_len = p.cu_q[b + 1] - q_begin;
+  const int q0 = q_tile * FA_BM;
+  if (q0 >= q_len) return;                                  // uniform per CTA, before any set-up
+  const int k_begin = p.cu_k[b];
+  const int kv_len = p.cu_k[b + 1] - k_begin;
+  const int off = kv_len - q_len;                           // key index of query 0
+  const int hi = min(kv_len, off + q0 + FA_BM);
+  const int lo = max(0, off + q0 - p.window + 1);
+  const int t_begin = lo / FA_BN;
+  const int n_tiles = max((hi + FA_BN - 1) / FA_BN - t_begin, 0);
+
+  const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* smem_al = smem_raw + (smem_base - smem_u32(smem_raw));
+  const uint32_t q_s = smem_base;
+  const uint32_t k_s = q_s + Cfg::kKBytes;
+  const uint32_t v_s = k_s + 2 * Cfg::kKBytes;
+  const uint32_t p_s = v_s + Cfg::kVBytes;
+  uint8_t* p_ptr = smem_al + 3 * Cfg::kKBytes + Cfg::kVBytes;
+
+  if (threadIdx.x == 0) {
+    abort_flag = 0;
+    mbar_init(smem_u32(&q_full), 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(smem_u32(&k_full[i]), 1);
+      mbar_init(smem_u32(&k_empty[i]), 1);
+      mbar_init(smem_u32(&s_full[i]), 1);
+      mbar_init(smem_u32(&s_empty[i]), 8);
+    }
+    mbar_init(smem_u32(&v_full), 1);
+    mbar_init(smem_u32(&v_empty), 1);
+    mbar_init(smem_u32(&p_full), 8);
+    mbar_init(smem_u32(&p_empty), 1);
+    for (int i = 0; i < 4; ++i) mbar_init(smem_u32(&xch_bar[i]), 64);
+    mbar_init(smem_u32(&o_done), 1);
+    fence_mbar_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_smem), FA_TMEM_COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = tmem_base_smem;
+  const uint32_t tmem_o = tmem_base + 2 * FA_BN;
+  volatile int* abortp = &abort_flag;
+
+  if (warp == 0) {
+    // ------------------------------------------------------------------ TMA producer
+    if (elect_one_sync()) {
+      bool ok = true;
+      mbar_expect_tx(smem_u32(&q_full), Cfg::kKBytes);
+#pragma unroll
+      for (int c = 0; c < DK / 64; ++c)
+        tma_load_2d(q_s + c * CHUNK_BYTES, &p.q_map, smem_u32(&q_full), h * DK + c * 64, q_begin + q0);
+      int k_issued = 0, v_issued = 0;
+      auto load_k = [&](int j) -> bool {
+        const int slot = j & 1, row = k_begin + (t_begin + j) * FA_BN;
+        if (!mbar_wait_backoff(smem_u32(&k_empty[slot]), ((j >> 1) & 1u) ^ 1u, abortp, p.status, ST_TIMEOUT_SMEM_EMPTY)) return false;
+        const uint32_t fb = smem_u32(&k_full[slot]), dst = k_s + slot * Cfg::kKBytes;
+        mbar_expect_tx(fb, Cfg::kKBytes);
+#pragma unroll
+        for (int c = 0; c < DN / 64; ++c) tma_load_2d(dst + c * CHUNK_BYTES, &p.k_map, fb, h * DN + c * 64, row);
+        tma_load_2d(dst + (DN / 64) * CHUNK_BYTES, &p.r_map, fb, 0, row);
+        ++k_issued;
+        return true;
+      };
+      auto load_v = [&](int j) -> bool {
+        const int row = k_begin + (t_begin + j) * FA_BN;
+        if (!mbar_wait_backoff(smem_u32(&v_empty), (j & 1u) ^ 1u, abortp, p.status, ST_TIMEOUT_SMEM_EMPTY)) return false;
+        mbar_expect_tx(smem_u32(&v_full), Cfg::kVBytes);
+#pragma unroll
+        for (int c = 0; c < DV / 64; ++c) tma_load_2d(v_s + c * CHUNK_BYTES, &p.v_map, smem_u32(&v_full), h * DV + c * 64, row);
+        ++v_issued;
+        return true;
+      };
+      // order of use: K0, then (K_{j+1}, V_j) for every j
+      if (n_tiles > 0) ok = load_k(0);
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        if (j + 1 < n_tiles) { ok = load_k(j + 1); if (!ok) break; }
+        ok = load_v(j);
+      }
+      if (!ok) {   // drain: no bulk copy may land after the CTA has gone
+        auto drain = [&](uint64_t* bar, uint32_t parity) {
+          const uint64_t t0 = globaltimer_ns();
+          while (!mbar_try_wait(smem_u32(bar), parity))
+            if (globaltimer_ns() - t0 > 50000000ull) break;
+        };
+        drain(&q_full, 0);
+        for (int j = max(0, k_issued - 2); j < k_issued; ++j) drain(&k_full[j & 1], (j >> 1) & 1u);
+        if (v_issued > 0) drain(&v_full, (v_issued - 1) & 1u);
+      }
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (elect_one_sync()) {
+      constexpr uint32_t idesc_s = make_idesc_bf16(FA_BM, FA_BN, 0, 0);    // Q, K both K-major
+      constexpr uint32_t idesc_o = make_idesc_bf16(FA_BM, DV, 0, 1);       // P K-major, V MN-major
+      bool ok = mbar_wait_backoff(smem_u32(&q_full), 0, abortp, p.status, ST_TIMEOUT_SMEM_FULL);
+      auto issue_s = [&](int j) -> bool {
+        const int slot = j & 1;
+        if (!mbar_wait_backoff(smem_u32(&k_full[slot]), (j >> 1) & 1u, abortp, p.status, ST_TIMEOUT_SMEM_FULL)) return false;
+        if (!mbar_wait_backoff(smem_u32(&s_empty[slot]), ((j >> 1) & 1u) ^ 1u, abortp, p.status, ST_TIMEOUT_TMEM_EMPTY)) return false;
+        tc_fence_after();
+        const uint32_t ks = k_s + slot * Cfg::kKBytes;
+#pragma unroll
+        for (int k = 0; k < DK / 16; ++k) {
+          const uint64_t adesc = make_smem_desc_sw128(q_s + (k >> 2) * CHUNK_BYTES + (k & 3) * 32, 16, 1024);
+          const uint64_t bdesc = make_smem_desc_sw128(ks + (k >> 2) * CHUNK_BYTES + (k & 3) * 32, 16, 1024);
+          umma_bf16(tmem_base + slot * FA_BN, adesc, bdesc, idesc_s, k > 0 ? 1u : 0u);
+        }
+        umma_commit(smem_u32(&k_empty[slot]));
+        umma_commit(smem_u32(&s_full[slot]));
+        return true;
+      };
+      if (ok && n_tiles > 0) ok = issue_s(0);
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        if (j + 1 < n_tiles) { ok = issue_s(j + 1); if (!ok) break; }
+        ok = mbar_wait_backoff(smem_u32(&p_full), j & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+        if (!ok) break;
+        ok = mbar_wait_backoff(smem_u32(&v_full), j & 1u, abortp, p.status, ST_TIMEOUT_SMEM_FULL);
+        if (!ok) break;
+        tc_fence_after();
+#pragma unroll
+        for (int k = 0; k < FA_BN / 16; ++k) {
+          const uint64_t adesc = make_smem_desc_sw128(p_s + (k >> 2) * CHUNK_BYTES + (k & 3) * 32, 16, 1024);
+          const uint64_t bdesc = make_smem_desc_sw128(v_s + k * 2048, CHUNK_BYTES, 1024);
+          umma_bf16(tmem_o, adesc, bdesc, idesc_o, (j > 0 || k > 0) ? 1u : 0u);
+        }
+        umma_commit(smem_u32(&v_empty));
+        umma_commit(smem_u32(&p_empty));
+        umma_commit(smem_u32(&o_done));
+      }
+    }
+  } else {
+    // ------------------------------------------------------------------ softmax + epilogue
+    // two threads per query row, as in flash_fwd_kernel: `half` owns 64 of the 128 score columns and half of O's columns
+    constexpr int HC = FA_BN / 2;
+    const int qd = warp & 3;
+    const int half = (warp - 2) >> 2;
+    const int r = qd * 32 + lane;
+    const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
+    const int qpos = off + q0 + r;
+    float m_used = -INFINITY, l = 0.f;
+    bool ok = true;
+    uint32_t xph = 0;
+    auto swap_with_partner = [&](float mine, float& other) -> bool {
+      xch[xph & 1][half][r] = mine;
+      mbar_arrive(smem_u32(&xch_bar[qd]));
+      bool good = mbar_wait_backoff(smem_u32(&xch_bar[qd]), xph & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      other = xch[xph & 1][half ^ 1][r];
+      ++xph;
+      return __all_sync(0xffffffffu, good);
+    };
+    for (int j = 0; j < n_tiles; ++j) {
+      const int k0 = (t_begin + j) * FA_BN;
+      const uint32_t s_addr = tmem_base + (j & 1) * FA_BN + half * HC + lane_addr;
+      ok = mbar_wait_backoff(smem_u32(&s_full[j & 1]), (j >> 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      tc_fence_after();
+      const bool need_mask = k0 + FA_BN > kv_len || k0 + FA_BN - 1 > off + q0 || k0 <= off + q0 + FA_BM - 1 - p.window;
+      uint32_t v[HC];
+#pragma unroll
+      for (int c = 0; c < HC / 32; ++c)
+        tmem_ld_32x32(s_addr + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&v[c * 32]));
+      tmem_ld_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&s_empty[j & 1]));
+      if (need_mask) {
+#pragma unroll
+        for (int i = 0; i < HC; ++i) {
+          const int kj = k0 + half * HC + i;
+          if (kj >= kv_len || kj > qpos || kj <= qpos - p.window) v[i] = 0xff800000u;   // -inf
+        }
+      }
+      float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+      for (int i = 0; i < HC; i += 4) {
+        mx[0] = fmaxf(mx[0], __uint_as_float(v[i]));
+        mx[1] = fmaxf(mx[1], __uint_as_float(v[i + 1]));
+        mx[2] = fmaxf(mx[2], __uint_as_float(v[i + 2]));
+        mx[3] = fmaxf(mx[3], __uint_as_float(v[i + 3]));
+      }
+      const float mine = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+      float other;
+      ok = swap_with_partner(mine, other);
+      if (!ok) break;
+      const float m_new = fmaxf(m_used, fmaxf(mine, other) * p.scale_log2);
+      const bool need = m_new > m_used + FA_RESCALE_THRESHOLD || (m_used == -INFINITY && m_new != -INFINITY);
+      if (__any_sync(0xffffffffu, need)) {   // same rows, same inputs: both warps of a quarter agree
+        if (j > 0) {
+          ok = mbar_wait_backoff(smem_u32(&o_done), (uint32_t)((j - 1) & 1), abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+          ok = __all_sync(0xffffffffu, ok);
+          if (!ok) break;
+          tc_fence_after();
+          const float alpha = need ? fast_exp2((m_used == -INFINITY ? m_new : m_used) - m_new) : 1.f;
+#pragma unroll 1
+          for (int c = half * (DV / 64); c < (half + 1) * (DV / 64); ++c) {
+            uint32_t o[32];
+            tmem_ld_32x32(tmem_o + lane_addr + c * 32, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+            tmem_st_32x32(tmem_o + lane_addr + c * 32, o);
+          }
+          tmem_st_wait();
+          l *= alpha;
+        }
+        if (need) m_used = m_new;
+      }
+      const float mref = m_used == -INFINITY ? 0.f : m_used;
+      float ls[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int i = 0; i < HC; i += 4) {
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+          const float x = fast_exp2(fmaf(__uint_as_float(v[i + t]), p.scale_log2, -mref));
+          ls[t] += x;
+          v[i + t] = __float_as_uint(x);
+        }
+      }
+      l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
+      // bf16 P into shared memory once the previous P V has read the buffer
+      ok = mbar_wait_backoff(smem_u32(&p_empty), (j & 1u) ^ 1u, abortp, p.status, ST_TIMEOUT_SMEM_EMPTY);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      uint8_t* prow = p_ptr + half * CHUNK_BYTES + r * 128;
+#pragma unroll
+      for (int unit = 0; unit < HC / 8; ++unit) {
+        uint4 w;
+        w.x = pack_bf16x2(__uint_as_float(v[unit * 8 + 0]), __uint_as_float(v[unit * 8 + 1]));
+        w.y = pack_bf16x2(__uint_as_float(v[unit * 8 + 2]), __uint_as_float(v[unit * 8 + 3]));
+        w.z = pack_bf16x2(__uint_as_float(v[unit * 8 + 4]), __uint_as_float(v[unit * 8 + 5]));
+        w.w = pack_bf16x2(__uint_as_float(v[unit * 8 + 6]), __uint_as_float(v[unit * 8 + 7]));
+        *reinterpret_cast<uint4*>(prow + ((unit ^ (r & 7)) << 4)) = w;
+      }
+      tc_fence_before();          // a rescale of O above is ordered before the product that reads it
+      fence_proxy_async_smem();   // P was written with ordinary stores and is read by the tensor core
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&p_full));
+    }
+    if (ok && n_tiles > 0) {
+      float l_other;
+      ok = swap_with_partner(l, l_other);   // both halves used the same m_used, so the sums simply add
+      l += l_other;
+    }
+    if (ok && n_tiles > 0) {
+      ok = mbar_wait_backoff(smem_u32(&o_done), (uint32_t)((n_tiles - 1) & 1), abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      ok = __all_sync(0xffffffffu, ok);
+    }
+    if (ok) {
+      tc_fence_after();
+      const bool row_ok = q0 + r < q_len;
+      const long long t = q_begin + q0 + r;
+      float f = 0.f;
+      if (row_ok && n_tiles > 0) {
+        l += exp2f(p.sink[h] * 1.4426950408889634f - m_used);      // the sink: in the denominator, no value
+        f = p.gate[t * p.H + h] / l;
+      }
+      __nv_bfloat16* orow = p.out + t * p.H * DV + h * DV;
+#pragma unroll 1
+      for (int c = half * (DV / 64); c < (half + 1) * (DV / 64); ++c) {
+        uint32_t v[32];
+        if (n_tiles > 0) {
+          tmem_ld_32x32(tmem_o + lane_addr + c * 32, v);
+          tmem_ld_wait();
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[i] = 0u;
+        }
+        if (row_ok) {
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            uint4 w;
+            w.x = pack_bf16x2(__uint_as_float(v[u * 8 + 0]) * f, __uint_as_float(v[u * 8 + 1]) * f);
+            w.y = pack_bf16x2(__uint_as_float(v[u * 8 + 2]) * f, __uint_as_float(v[u * 8 + 3]) * f);
+            w.z = pack_bf16x2(__uint_as_float(v[u * 8 + 4]) * f, __uint_as_float(v[u * 8 + 5]) * f);
+            w.w = pack_bf16x2(__uint_as_float(v[u * 8 + 6]) * f, __uint_as_float(v[u * 8 + 7]) * f);
+            *reinterpret_cast<uint4*>(orow + c * 32 + u * 8) = w;
+          }
+        }
+      }
+      tc_fence_before();
+    }
+  }
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, FA_TMEM_COLS);
+  }
+}
+
+template <int DN, int DV>
+static int launch_flash_latent(const FlashLatentParams& p, int max_q, int B, cudaStream_t stream) {
+  auto kern = flash_latent_kernel<DN, DV>;
+  static bool attr_dev[64] = {};
+  int dev_i = 0;
+  if (cudaGetDevice(&dev_i) != cudaSuccess || dev_i < 0 || dev_i >= 64) return -10;
+  if (!attr_dev[dev_i]) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, FlashLatentCfg<DN, DV>::kSmemBytes) != cudaSuccess) return -10;
+    attr_dev[dev_i] = true;
+  }
+  dim3 grid((max_q + FA_BM - 1) / FA_BM, p.H, B);
+  return launch_kernel(kern, grid, dim3(FA_THREADS), FlashLatentCfg<DN, DV>::kSmemBytes, stream, p) == cudaSuccess ? 0 : -11;
+}
+
 
 // ==========================================================================================
 // Backward. Three kernels, no atomics, deterministic:
@@ -1473,6 +1828,36 @@ int rb_flash_fwd(const void* q, const void* k, const void* v, void* out, float* 
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
   int rc = D == 64 ? launch_flash_fwd<64>(p, max_seqlen_q, B, stream) : launch_flash_fwd<128>(p, max_seqlen_q, B, stream);
+  if (rc != 0) return rc;
+  return cudaGetLastError() == cudaSuccess ? 0 : -12;
+}
+
+// Latent attention, expanded form: see flash_latent_kernel. q [T, H*(DN+64)], k [S, H*DN], rot [S, 64], v [S, H*DV]; the
+// queries of sequence b are rows cu_q[b]..cu_q[b+1] of q and out, its keys rows cu_k[b]..cu_k[b+1].
+int rb_flash_latent(const void* q, const void* k, const void* rot, const void* v, void* out, const int* cu_q, const int* cu_k,
+                    const float* sink, const float* gate, int B, int H, int T, int S, int max_q, int DN, int DV, int window,
+                    float scale, int* status, cudaStream_t stream) {
+  using namespace rb;
+  if (B <= 0 || T <= 0 || S <= 0 || max_q <= 0) return 0;
+  if ((DN != 64 && DN != 128) || (DV != 64 && DV != 128) || window < 1 || B > 65535 || H > 65535) return -1;
+  FlashLatentParams p;
+  const unsigned long long hq = (unsigned long long)H * (DN + 64), hk = (unsigned long long)H * DN, hv = (unsigned long long)H * DV;
+  if (tma_map_2d_bf16(&p.q_map, q, T, hq, hq, FA_BM) != 0) return -20;
+  if (tma_map_2d_bf16(&p.k_map, k, S, hk, hk, FA_BN) != 0) return -21;
+  if (tma_map_2d_bf16(&p.r_map, rot, S, 64, 64, FA_BN) != 0) return -22;
+  if (tma_map_2d_bf16(&p.v_map, v, S, hv, hv, FA_BN) != 0) return -23;
+  p.out = (__nv_bfloat16*)out;
+  p.cu_q = cu_q;
+  p.cu_k = cu_k;
+  p.sink = sink;
+  p.gate = gate;
+  p.H = H;
+  p.window = window;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.status = status;
+  int rc;
+  if (DN == 128) rc = DV == 128 ? launch_flash_latent<128, 128>(p, max_q, B, stream) : launch_flash_latent<128, 64>(p, max_q, B, stream);
+  else rc = DV == 128 ? launch_flash_latent<64, 128>(p, max_q, B, stream) : launch_flash_latent<64, 64>(p, max_q, B, stream);
   if (rc != 0) return rc;
   return cudaGetLastError() == cudaSuccess ? 0 : -12;
 }

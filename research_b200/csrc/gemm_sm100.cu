@@ -106,6 +106,8 @@ struct GemmParams {
   int group_k;            // grouped weight gradient: tiles carry their own K range and output group (see RbGemmArgs::group_mode)
   const unsigned long long* row_dst;
   int swiglu;
+  int glu_kind;           // see RbGemmArgs
+  float glu_limit, softcap;
   int split_k, kb_per_split;
   int cluster_k;   // split-K slices are the CTAs of one thread-block cluster; partial tiles meet in distributed shared memory
   int red_alias;   // cluster split-K, one work unit per CTA: the partial tile reuses the (drained) TMA ring
@@ -168,6 +170,12 @@ __device__ __forceinline__ void epi_store_row_chunk(const GemmParams& p, const f
       }
     }
   }
+}
+
+__device__ __forceinline__ float clamped_glu_epi(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
 }
 
 // Counter-based random stream of the sampler (identical to rb_sample_logprob: splitmix64 row key,
@@ -784,6 +792,12 @@ gemm_bf16_kernel(const __grid_constant__ GemmParams p) {
                 uint32_t o[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
+                  if (p.glu_kind == 1) {
+                    o[e] = pack_bf16x2(
+                        clamped_glu_epi(__uint_as_float(g[j + 2 * e]) * rscale, __uint_as_float(u[j + 2 * e]) * rscale, p.glu_limit),
+                        clamped_glu_epi(__uint_as_float(g[j + 2 * e + 1]) * rscale, __uint_as_float(u[j + 2 * e + 1]) * rscale, p.glu_limit));
+                    continue;
+                  }
                   // same rounding points as the unfused path: bf16(gate), bf16(silu), bf16(up), bf16(product)
                   const float g0 = __bfloat162float(__float2bfloat16_rn(__uint_as_float(g[j + 2 * e]) * rscale));
                   const float g1 = __bfloat162float(__float2bfloat16_rn(__uint_as_float(g[j + 2 * e + 1]) * rscale));
@@ -842,6 +856,11 @@ gemm_bf16_kernel(const __grid_constant__ GemmParams p) {
                   f = unpack_bf16x2(b.w); v[j + 6] = fmaf(rs, f.x, v[j + 6]); v[j + 7] = fmaf(rs, f.y, v[j + 7]);
                 }
               }
+            }
+            if (p.softcap > 0.f) {
+              const float inv_cap = 1.f / p.softcap;
+#pragma unroll
+              for (int j = 0; j < 32; ++j) v[j] = p.softcap * tanhf(v[j] * inv_cap);
             }
             if (p.row_dst != nullptr) {
               // fused combine: this row's home is an arbitrary (possibly remote) address
@@ -1306,6 +1325,11 @@ extern "C" int rb_gemm_bf16_ex(const RbGemmArgs* a, cudaStream_t stream) {
   p.num_tiles_ptr = a->num_tiles_ptr;
   p.row_dst = a->row_dst;
   p.swiglu = a->swiglu;
+  p.glu_kind = a->glu_kind;
+  p.glu_limit = a->glu_limit;
+  p.softcap = a->softcap;
+  if (p.softcap > 0.f && (a->swiglu || a->split_k > 1 || a->tile_table || a->epi_mode != RB_EPI_STORE || a->mirror || a->sample_ws))
+    return -1;
   p.scaled_epilogue = a->scaled_epilogue;
   p.alpha = a->alpha;
   p.beta = a->beta;

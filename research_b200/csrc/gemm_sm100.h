@@ -132,6 +132,12 @@ typedef struct RbGemmArgs {
   // group g is C rows [g * M, (g + 1) * M), and K is the total row count of A and B.
   int group_mode;
   int group_b_rows;
+  // Activation of the fused gate|up epilogue (swiglu set): glu_kind 0 = silu(gate) * up; 1 = clamped unit: gate capped at
+  // glu_limit, up clamped to +-glu_limit, gate * sigmoid(1.702 gate) * (up + 1).
+  int glu_kind;
+  float glu_limit;
+  // > 0: C = softcap * tanh(C / softcap) on the fp32 result (plain store only: no split, grouping or reduce mode).
+  float softcap;
 } RbGemmArgs;
 
 // Token and log-probability from the per-tile records written by the sampling epilogue.

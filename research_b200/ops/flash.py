@@ -30,6 +30,8 @@ def _lib() -> ctypes.CDLL:
         lib.rb_flash_fwd.restype = c_int
         lib.rb_flash_bwd.argtypes = [c_vp] * 13 + [c_int] * 13 + [c_float, c_vp, c_vp]
         lib.rb_flash_bwd.restype = c_int
+        lib.rb_flash_latent.argtypes = [c_vp] * 9 + [c_int] * 8 + [c_float, c_vp, c_vp]
+        lib.rb_flash_latent.restype = c_int
         lib._rb_typed = True
     return lib
 

@@ -92,6 +92,9 @@ class RbGemmArgs(ctypes.Structure):
         ("gather_wait_all", ctypes.c_int),
         ("group_mode", ctypes.c_int),
         ("group_b_rows", ctypes.c_int),
+        ("glu_kind", ctypes.c_int),
+        ("glu_limit", ctypes.c_float),
+        ("softcap", ctypes.c_float),
     ]
 
 
@@ -234,6 +237,8 @@ def gemm(
     b_gather=None,
     carry_gather=None,
     wait_flag: tuple[int, int] | None = None,
+    glu_limit: float | None = None,
+    softcap: float = 0.0,
 ) -> torch.Tensor:
     """``C[M,N] = alpha * op(A) @ op(B)^T (+bias) (+ beta * residual)``.
 
@@ -250,6 +255,9 @@ def gemm(
     ``norm_eps`` folds an RMSNorm of A's rows into the launch: ``C = rstd(row) * (A @ B^T) (+bias)`` with
     ``rstd = rsqrt(mean(A[row]^2) + norm_eps)``; together with the norm weight multiplied into B's columns
     beforehand this equals ``rmsnorm(A) @ B^T`` without a separate normalisation pass.
+
+    ``glu_limit`` makes the fused gate|up epilogue (``swiglu=True``) the clamped unit of ``elementwise.clamped_glu``;
+    ``softcap`` stores ``softcap * tanh(C / softcap)``.
 
     K-major operands are ``[rows, K]`` row-major (a torch ``Linear`` weight is a K-major B);
     MN-major operands are ``[K, rows]`` row-major. On CUDA this launches the tcgen05 kernel;
@@ -280,7 +288,9 @@ def gemm(
         else:
             res = gemm_reference(a, b, bias, residual, a_mn_major, b_mn_major, torch.float32 if out_f32 else None)
         if swiglu:
-            res = swiglu_interleaved_reference(res, bn)
+            res = swiglu_interleaved_reference(res, bn, glu_limit)
+        if softcap > 0:
+            res = softcap * torch.tanh(res / softcap)
         if out is not None:
             out.copy_(res)
             return out
@@ -303,7 +313,10 @@ def gemm(
         N, Kb = b.shape
     assert K == Kb, f"K mismatch: {K} vs {Kb}"
     gather = b_gather if b_gather is not None else carry_gather
-    if (gather is None and wait_flag is None and not swiglu and norm_eps is None and alpha == 1.0 and beta == 1.0 and bn == 0 and max_ctas == 0 and split_k in (0, 1)
+    if softcap > 0:
+        assert not swiglu and split_k in (0, 1), "the soft cap belongs to a plain store"
+        split_k, cluster_split = 1, False
+    if (gather is None and softcap == 0 and wait_flag is None and not swiglu and norm_eps is None and alpha == 1.0 and beta == 1.0 and bn == 0 and max_ctas == 0 and split_k in (0, 1)
             and not cluster_split and _use_pair_kernel(M, N, K, a_mn_major, b_mn_major)):
         return gemm2(a, b, bias, residual, out, a_mn_major=a_mn_major, b_mn_major=b_mn_major, out_f32=out_f32)
     if (gather is not None and _GEMM2_GATHER and wait_flag is None and not swiglu and norm_eps is None and alpha == 1.0 and beta == 1.0
@@ -331,6 +344,9 @@ def gemm(
     args.epi_mode = EPI_STORE
     args.rank, args.world = 0, 1
     args.swiglu = int(swiglu)
+    if glu_limit is not None:
+        args.glu_kind, args.glu_limit = 1, float(glu_limit)
+    args.softcap = float(softcap)
     if norm_eps is not None:
         args.norm_fold, args.norm_eps = 1, float(norm_eps)
     if gather is not None:
@@ -637,11 +653,14 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor, bn: int) -> torch.T
     return torch.stack([gate.view(F // h, h, K), up.view(F // h, h, K)], dim=1).reshape(2 * F, K).contiguous()
 
 
-def swiglu_interleaved_reference(y: torch.Tensor, bn: int) -> torch.Tensor:
-    """``silu(gate) * up`` for GEMM output whose columns are interleaved as ``interleave_gate_up`` packs them."""
+def swiglu_interleaved_reference(y: torch.Tensor, bn: int, glu_limit: float | None = None) -> torch.Tensor:
+    """``silu(gate) * up`` (or the clamped unit) for GEMM output whose columns are interleaved as ``interleave_gate_up`` packs them."""
     M, N2 = y.shape
     h = bn // 2
     yv = y.view(M, N2 // bn, 2, h)
+    if glu_limit is not None:
+        g, u = yv[:, :, 0].clamp(max=glu_limit), yv[:, :, 1].clamp(-glu_limit, glu_limit)
+        return (g * torch.sigmoid(1.702 * g) * (u + 1)).reshape(M, N2 // 2)
     return (torch.nn.functional.silu(yv[:, :, 0]) * yv[:, :, 1]).reshape(M, N2 // 2)
 
 

@@ -145,13 +145,14 @@ _HEAD_TILES: dict[tuple, tuple[torch.Tensor, torch.Tensor, int]] = {}
 _ROW_DST: dict[tuple, torch.Tensor] = {}
 
 
-def _head_tiles(H: int, n: int, stride: int, N: int, b_step: int, bn: int, device) -> tuple[torch.Tensor, torch.Tensor, int]:
+def _head_tiles(H: int, n: int, stride: int, N: int, b_step: int, bn: int, mode: int, device) -> tuple[torch.Tensor, torch.Tensor, int]:
     """Device tile table of ``H`` products over rows ``[h*stride, h*stride + n)``, cached."""
-    key = (H, n, stride, N, b_step, bn, device.index)
+    key = (H, n, stride, N, b_step, bn, mode, device.index)
     if key not in _HEAD_TILES:
         if len(_HEAD_TILES) >= 4096:         # captured graphs keep theirs alive through live_tables()
             _HEAD_TILES.clear()
-        rows = [(h * stride + m, min(128, n - m), h * b_step, n0) for h in range(H) for n0 in range(0, N, bn) for m in range(0, n, 128)]
+        # mode 0 names the tile's first B row, mode 1 the head's first B row (its tile column is n0)
+        rows = [(h * stride + m, min(128, n - m), h * b_step + (n0 if mode == 0 else 0), n0) for h in range(H) for n0 in range(0, N, bn) for m in range(0, n, 128)]
         _HEAD_TILES[key] = (torch.tensor(rows, dtype=torch.int32).to(device), torch.tensor([len(rows)], dtype=torch.int32).to(device), len(rows))
     return _HEAD_TILES[key]
 
@@ -171,7 +172,7 @@ def _head_bn(H: int, n: int, N: int, least: int) -> int:
 
 
 def _grouped(a, w, out, H, n, N, K, b_step, bn, mode, row_dst=None) -> None:
-    table, count, tiles = _head_tiles(H, n, a.shape[1], N, b_step, bn, a.device)
+    table, count, tiles = _head_tiles(H, n, a.shape[1], N, b_step, bn, mode, a.device)
     args = RbGemmArgs()
     args.A[0], args.B[0], args.C = a.data_ptr(), w.data_ptr(), out.data_ptr()
     args.lda, args.ldb, args.ldc = a.stride(1), w.stride(0), out.stride(-2)
