@@ -4,6 +4,7 @@
     chat      talk to a model (any provider) with an agent preset; sessions are stored and resumable
     sessions  list / show / export / slice / import stored sessions
     eval      run a JSONL dataset through an agent and score it with a dotted-path score function
+    replay    feed given tokens through a model step by step and write logits (bin/trace_run)
     bench     the flagship benchmark (same as the repository's bench.py)
     build     compile the native libraries
 """
@@ -120,7 +121,8 @@ def cmd_serve(args) -> int:
         weights = init_random_weights(cfg, seed=0, dtype=torch.bfloat16 if device == "cuda" else torch.float32, device=device)
         tokenizer = None
     ecfg = EngineConfig(cache_type=args.cache, max_batch_size=args.max_batch_size, max_model_len=args.max_model_len,
-                        gpu_memory_utilization=args.gpu_memory_utilization, tensor_parallel_size=args.tp)
+                        gpu_memory_utilization=args.gpu_memory_utilization, tensor_parallel_size=args.tp,
+                        dtype=args.dtype, prefill_chunk=args.prefill_chunk)
     tp = group = None
     if args.tp > 1:       # launched with torch.distributed.run: one rank per GPU, rank 0 serves HTTP
         import torch.distributed as dist
@@ -395,6 +397,7 @@ _DELEGATES = {   # sub-command -> module whose ``main(argv)`` takes the remainin
     "monitor": "research_b200.frontend.training_monitor", "traces": "research_b200.frontend.traces",
     "pretrain": "research_b200.training.pretrain", "infra": "research_b200.infra.cli",
     "kernel-harness": "research_b200.utils.kernel_harness",
+    "replay": "research_b200.inference.trace_replay",
 }
 
 
@@ -415,6 +418,8 @@ def build_parser() -> argparse.ArgumentParser:
     p.add_argument("--cache", default="radix", choices=["paged", "radix", "none"])
     p.add_argument("--max-batch-size", type=int, default=256); p.add_argument("--max-model-len", type=int, default=8192)
     p.add_argument("--gpu-memory-utilization", type=float, default=0.9); p.add_argument("--tp", type=int, default=1)
+    p.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="float32: all in 32-bit, for models that have that mode")
+    p.add_argument("--prefill-chunk", type=int, default=0, help="most prompt tokens of a request per step (0: the engine's own choice)")
     p.set_defaults(fn=cmd_serve)
     p = sub.add_parser("chat")
     _add_endpoint_args(p)

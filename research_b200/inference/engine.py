@@ -302,6 +302,11 @@ class InferenceEngine:
         lib.rbe_commit_fed(core)
         return out
 
+    def check_kernels(self) -> None:
+        """Raise if a kernel recorded a failure (bad index, wait that ran out)."""
+        if self.device.type == "cuda":
+            check_status(self.device)
+
     def close_stream(self, stream: int) -> None:
         self._lib.rbe_abort(self._core, stream)
 

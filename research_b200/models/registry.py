@@ -20,11 +20,14 @@ from .stack import LayerStackConfig
 class Architecture:
     parse: Callable[[dict], object]
     runner: str                        # module:class, imported when an engine is built
+    libraries: tuple[str, ...]         # native libraries its kernels live in (names of ``_native.LIBRARIES``)
 
 
-HF_DECODER = Architecture(ModelConfig.from_hf_dict, "research_b200.inference.model_runner:ModelRunner")
+HF_DECODER = Architecture(ModelConfig.from_hf_dict, "research_b200.inference.model_runner:ModelRunner",
+                          ("rb_engine_core", "rb_gemm", "rb_gemm2", "rb_ops", "rb_attn", "rb_flash", "rb_moe"))
 ARCHITECTURES: dict[str, Architecture] = {
-    "Lulezen": Architecture(LayerStackConfig.from_dict, "research_b200.inference.stack_runner:StackRunner"),
+    "Lulezen": Architecture(LayerStackConfig.from_dict, "research_b200.inference.stack_runner:StackRunner",
+                            ("rb_engine_core", "rb_gemm", "rb_gemm2", "rb_gemm_f32", "rb_ops", "rb_latent", "rb_flash")),
 }
 
 
