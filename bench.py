@@ -785,6 +785,20 @@ def run_reference_train(args) -> dict:
     return _time_train_arm(args, step, world, rank, local, args.impl, extra)
 
 
+def run_stack(args) -> dict:
+    """One GPU: the layer-stack design against its closest neighbour in the framework (``utils/stack_bench.py``)."""
+    from research_b200.utils import stack_bench
+    from research_b200.utils.timing import ClockSampler
+
+    if args.impl != "native" or args.gpus != 1:
+        return {"impl": args.impl, "unavailable": "the stack workload runs natively on one GPU"}
+    sampler = ClockSampler(0)
+    sampler.start()
+    res = stack_bench.run(tuple(x for x in args.sizes.split(",") if x))
+    return {"metric": "prefill and decode of a layer-stack model, tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
+            "higher_is_better": True, "clocks": sampler.stop(), **res}
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -794,10 +808,12 @@ def main() -> None:
                     help="reference = the unmodified reference through its own API (unavailable for training where its imports "
                          "cannot be met); library = HF Llama + FSDP2 + torch AdamW driven by this script; reference-standin = the "
                          "reference's FSDP backend class imported with a stand-in for the missing trio module (context only)")
-    ap.add_argument("--workload", choices=["train", "rollout", "serving"], default="train",
+    ap.add_argument("--workload", choices=["train", "rollout", "serving", "stack"], default="train",
                     help="train = sharded training step on the Llama-3-8B shape, seq 4096, one sequence per GPU (the flagship); "
                          "rollout = engine decode, 1024 requests, prompts U[128,1024], 512 new tokens, batch 256; "
-                         "serving = batch 64, prompts of 2048 tokens, 256 new tokens (the tensor-parallel serving case)")
+                         "serving = batch 64, prompts of 2048 tokens, 256 new tokens (the tensor-parallel serving case); "
+                         "stack = prefill and decode of a layer-stack model beside a Llama-type model of equal size, kernel by kernel")
+    ap.add_argument("--sizes", default="", help="stack: comma-separated sizes (default: all)")
     ap.add_argument("--model", default=None, help="model preset (default: llama-3-8b for train / serving, qwen2.5-0.5b for rollout)")
     ap.add_argument("--seq", type=int, default=TRAIN_SEQ, help="train: tokens per sequence")
     ap.add_argument("--batch", type=int, default=TRAIN_BATCH_PER_GPU, help="train: sequences per GPU per step")
@@ -819,6 +835,8 @@ def main() -> None:
         args.warmup = 3 if args.warmup is None else args.warmup
         out = {"native": run_train, "reference": run_reference_train, "library": run_library_train,
                "reference-standin": run_reference_train}[args.impl](args)
+    elif args.workload == "stack":
+        out = run_stack(args)
     else:
         if args.impl in ("library", "reference-standin"):
             out = {"impl": args.impl, "unavailable": "this arm exists for the train workload only"}

@@ -22,6 +22,9 @@ from dataclasses import asdict, dataclass
 from pathlib import Path
 
 
+NO_WINDOW = 1 << 30          # a window nothing reaches: plain causal attention
+
+
 @dataclass(frozen=True)
 class RotarySpec:
     """Rotation of pairs ``(i, i + dims/2)`` of the first ``dims`` channels by ``position * base^(-2i/dims)``."""
@@ -55,7 +58,7 @@ class LatentAttentionSpec:
     def from_dict(m: dict) -> "LatentAttentionSpec":
         return LatentAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]),
                                    kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]), scale=float(m["scale"]),
-                                   window=int(m["mask"]["size"]),
+                                   window=int((m.get("mask") or {}).get("size") or NO_WINDOW),
                                    rot=RotarySpec(int(m["rot"]["dims"]), float(m["rot"]["base"])))
 
     def to_dict(self) -> dict:
