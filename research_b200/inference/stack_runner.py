@@ -94,7 +94,7 @@ class StackRunner(RunnerBase):
 
     @staticmethod
     def cache_bytes_per_block(cfg: LayerStackConfig, tp_size: int, dtype: torch.dtype) -> int:
-        return sum(latent_geometry(x.mixer).cw for x in cfg.layers) * BLOCK * (4 if dtype == torch.float32 else 2)
+        return sum(latent_geometry(x.mixer).cs for x in cfg.layers) * BLOCK * (4 if dtype == torch.float32 else 2)
 
     # ------------------------------------------------------------------ memory
     def _alloc_weights(self) -> None:
@@ -131,7 +131,7 @@ class StackRunner(RunnerBase):
                 lw.ffp = _up(spec.mlp.ff, self.glu_bn // 2 if self.bf16 else 8)
                 lw.wgu, lw.wd = zeros(2 * lw.ffp, self.wp), zeros(self.wp, lw.ffp)
                 lw.norm2 = (zeros(d, dtype=f32), zeros(d, dtype=f32))
-            lw.cache = zeros(self.num_kv_blocks, BLOCK, g.cw)
+            lw.cache = zeros(self.num_kv_blocks, BLOCK, g.cs)
             self.layers.append(lw)
 
     def _alloc_activations(self) -> None:
@@ -148,13 +148,9 @@ class StackRunner(RunnerBase):
         for lw in self.layers:
             if lw.geo not in self.bufs:
                 self.bufs[lw.geo] = GeometryBuffers(lw.geo, n, self.short_rows, dt, dev)
-        # partial sums of split keys: what the captured decode batches need, and at least 64 MB for packed batches
-        need = 1 << 24
-        for lw in self.layers:
-            for bk in set(self.graph_batch_sizes) | {self.max_batch}:
-                s = ops.latent_num_splits(bk, lw.geo.heads, min(self.max_model_len, lw.spec.mixer.window + BLOCK))
-                need = max(need, bk * lw.geo.heads * s * (lw.geo.rw + 2) if s > 1 else 0)
-        self.attn_ws = torch.empty(need, dtype=torch.float32, device=dev) if self.bf16 else None
+        self.attn_ws = ops.latent_workspace(list(self.bufs), dev) if self.bf16 else None
+        self.kinds = sorted({(lw.geo.heads, lw.spec.mixer.window) for lw in self.layers})    # layers that share an attention plan
+        self.decode_plans = {k: torch.zeros(ops.latent_units(self.max_batch, k[0], 1) + 1, dtype=torch.int32, device=dev) for k in self.kinds}
 
     # ------------------------------------------------------------------ weights
     def load_weights(self, weights: Mapping[str, torch.Tensor]) -> None:
@@ -250,17 +246,26 @@ class StackRunner(RunnerBase):
                 ops.softcap(logits, cap)
         return logits[:, :self.cfg.vocab_size]
 
+    def _short_attention(self, rows: int, max_q: int, cu_q, seq_lens, block_tables, plans: dict | None = None):
+        """Attention on the cached latents for the first ``rows`` rows of the batch."""
+        if self.bf16:
+            n = seq_lens.shape[0]
+            if plans is None:
+                plans = {k: torch.empty(ops.latent_units(n, k[0], max_q) + 1, dtype=torch.int32, device=self.device) for k in self.kinds}
+            for (heads, window), plan in plans.items():
+                ops.latent_plan(cu_q, seq_lens, heads, max_q, window, plan)
+
+        def attend(lw, b):
+            m = lw.spec.mixer
+            ops.latent_attention(b.qa, lw.cache, lw.geo, block_tables, cu_q, seq_lens, lw.sink, b.gate, b.ol, scale=m.scale, window=m.window,
+                                 rows=rows, max_q=max_q, plan=plans[(m.heads, m.window)] if self.bf16 else None, workspace=self.attn_ws)
+
+        return attend
+
     # ------------------------------------------------------------------ decode
     def _decode_body(self, bk: int) -> None:
-        bt, lens = self.bt_dev[:bk], self.d_lens[:bk]
-
-        def short_attn(lw, b):
-            span = min(self.max_model_len, lw.spec.mixer.window + BLOCK)
-            ops.latent_attention(b.qa, lw.cache, lw.geo, bt, None, lens, lw.sink, b.gate, b.ol, scale=lw.spec.mixer.scale,
-                                 window=lw.spec.mixer.window, rows=bk, max_q=1, workspace=self.attn_ws,
-                                 splits=ops.latent_num_splits(bk, lw.geo.heads, span) if self.bf16 else 1)
-
-        self._layers(bk, self.d_tokens[:bk], self.d_pos[:bk], self.d_slots[:bk], bk, short_attn)
+        self._layers(bk, self.d_tokens[:bk], self.d_pos[:bk], self.d_slots[:bk], bk,
+                     self._short_attention(bk, 1, None, self.d_lens[:bk], self.bt_dev[:bk], self.decode_plans))
         ops.layernorm_rows(self.x[:bk], self.final_norm[0], self.final_norm[1], self.cfg.norm_eps, self.hl)
         logits = self._head(self.hl[:bk], self.logits_padded[:bk])
         self._sample(logits, self.d_temps[:bk], self.d_seeds[:bk], bk)
@@ -281,18 +286,9 @@ class StackRunner(RunnerBase):
                 n_seq -= 1
         n_short = b.host_cu_q[n_seq]
         max_q = max(lens[:n_seq], default=1)
-        cu_s, lens_s, bt_s = b.cu_q[:n_seq + 1], b.seq_lens[:n_seq], b.block_tables[:n_seq]
-        longest = max(b.host_seq_lens[:n_seq], default=1)
-
-        def short_attn(lw, buf):
-            g, m = lw.geo, lw.spec.mixer
-            splits = 1
-            if self.bf16:
-                splits = ops.latent_num_splits(n_seq, g.heads, min(longest, m.window + max_q + BLOCK), max_q)
-                splits = max(1, min(splits, self.attn_ws.numel() // (n_short * g.heads * (g.rw + 2))))
-            ops.latent_attention(buf.qa, lw.cache, g, bt_s, cu_s, lens_s, lw.sink, buf.gate, buf.ol, scale=m.scale, window=m.window,
-                                 rows=n_short, max_q=max_q, splits=splits, workspace=self.attn_ws)
-
+        short_attn = None
+        if n_short > 0:
+            short_attn = self._short_attention(n_short, max_q, b.cu_q[:n_seq + 1], b.seq_lens[:n_seq], b.block_tables[:n_seq])
         self._layers(T, b.tokens[:T], b.positions[:T], b.slots[:T], n_short, short_attn,
                      self._long_attention(b, n_seq, n_short) if n_seq < b.rows else None)
         return self.x[:T]

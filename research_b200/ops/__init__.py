@@ -47,8 +47,10 @@ from .latent import (
     latent_append,
     latent_attention,
     latent_gather,
-    latent_num_splits,
+    latent_plan,
     latent_query,
+    latent_units,
+    latent_workspace,
 )
 from .sampling import sample_with_logprobs, sample_with_logprobs_reference, token_logprobs
 
@@ -71,5 +73,5 @@ __all__ = [
     "sample_with_logprobs_reference", "token_logprobs", "set_pdl", "interleave_gate_up", "gemm_mod", "gemm_symmetric", "gemm_fp8", "quantize_fp8", "lm_head_sample", "lm_head_sample_workspace", "flash_attention", "flash_attn_varlen",
     "flash_attn_varlen_backward", "flash_attn_varlen_reference", "flash_paged_prefill", "flash_latent_prefill", "flash_latent_supported", "clamped_glu", "clamped_glu_reference",
     "embed_residual", "layernorm_reference", "layernorm_residual", "layernorm_rows", "softcap", "gemm_f32", "LatentGeometry",
-    "head_gemm_absorb", "head_gemm_expand", "latent_append", "latent_attention", "latent_gather", "latent_num_splits", "latent_query",
+    "head_gemm_absorb", "head_gemm_expand", "latent_append", "latent_attention", "latent_gather", "latent_plan", "latent_query", "latent_units", "latent_workspace",
 ]

@@ -60,8 +60,12 @@ class LatentGeometry:
         return _up(self.kv_rank, 16)
 
     @property
-    def cw(self) -> int:           # cache row
+    def cw(self) -> int:           # used channels of a cache row
         return _up(self.rw + _up(self.rot_dim, 16), 32)
+
+    @property
+    def cs(self) -> int:           # cache row stride: 8 channels apart, so that the attention kernel reads shared memory conflict-free
+        return self.cw + 8
 
     @property
     def qp(self) -> int:           # query latent
@@ -78,9 +82,10 @@ def _lib() -> ctypes.CDLL:
         lib.rb_latent_append.argtypes = ([c_vp, c_ll, c_vp, c_vp, c_float] + [c_vp] * 3 + [c_int, c_int, c_vp, c_ll, c_int, c_int, c_vp, c_ll, c_vp]
                                          + [c_int] * 6 + [c_vp, c_vp])
         lib.rb_latent_query.argtypes = [c_vp] * 3 + [c_int] * 3 + [c_vp, c_vp, c_ll] + [c_int] * 8 + [c_vp, c_vp]
-        lib.rb_latent_attn.argtypes = [c_vp] * 10 + [c_ll] + [c_int] * 9 + [c_float] + [c_int] * 4 + [c_vp, c_vp]
+        lib.rb_latent_attn.argtypes = [c_vp] * 11 + [c_ll] + [c_int] * 8 + [c_float] + [c_int] * 4 + [c_vp, c_vp]
+        lib.rb_latent_plan.argtypes = [c_vp, c_vp] + [c_int] * 4 + [c_vp, c_vp]
         lib.rb_latent_gather.argtypes = [c_vp, c_vp] + [c_int] * 3 + [c_vp, c_vp, c_int, c_int, c_vp, c_vp] + [c_int] * 5 + [c_vp, c_vp]
-        for f in ("rb_latent_append", "rb_latent_query", "rb_latent_attn", "rb_latent_gather"):
+        for f in ("rb_latent_append", "rb_latent_query", "rb_latent_attn", "rb_latent_plan", "rb_latent_gather"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -109,13 +114,13 @@ def latent_append(proj, geo: LatentGeometry, q_norm, kv_norm, eps: float, positi
         gate[:T] = torch.sigmoid(proj[:, r0:r0 + geo.heads])
         ok = slots >= 0
         sl = slots[ok].long()
-        flat = cache.view(-1, geo.cw)
+        flat = cache.view(-1, geo.cs)[:, :geo.cw]
         flat[sl, :geo.kv_rank] = rms(proj[ok][:, q0:k0], kv_norm).to(cache.dtype)
         flat[sl, geo.rw:geo.rw + geo.rot_dim] = _rotate_half_pairs(proj[ok][:, k0:r0], table[positions[ok].long()]).to(cache.dtype)
         return
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and cache.is_contiguous() and gate.dtype == torch.float32
     rc = _lib().rb_latent_append(ptr(proj), proj.stride(0), ptr(q_norm), ptr(kv_norm), eps, ptr(positions), ptr(slots), ptr(table),
-                                 table.shape[0], geo.rot_pairs, ptr(cache), cache.shape[0] * LATENT_BLOCK, geo.cw, geo.rw, ptr(cq),
+                                 table.shape[0], geo.rot_pairs, ptr(cache), cache.shape[0] * LATENT_BLOCK, geo.cs, geo.rw, ptr(cq),
                                  cq.stride(0), ptr(gate), geo.q_rank, geo.kv_rank, geo.rot_dim, geo.heads, T, _DT[cq.dtype],
                                  ptr(status_tensor(proj.device)), stream_handle(proj.device))
     check_rc(rc, "rb_latent_append")
@@ -228,23 +233,39 @@ def head_gemm_expand(a, w, out, n: int) -> None:
 
 
 # ------------------------------------------------------------------------------- attention on the cached rows
-def latent_num_splits(batch: int, heads: int, span: int, max_q: int = 1) -> int:
-    """Key splits per row tile: one CTA occupies an SM, so few tiles are cut until they fill the machine; a split keeps
-    at least 128 keys."""
-    tiles = batch * -(-max_q * heads // (32 if max_q * heads > 16 else 16))
-    return max(1, min(-(-148 // max(tiles, 1)), span // 128, 32))
+def latent_units(B: int, heads: int, max_q: int) -> int:
+    """Row tiles of a batch: 32 (token, head) rows each, or 16 where a sequence has no more."""
+    rows = 32 if max_q * heads > 16 else 16
+    return B * -(-max_q * heads // rows)
+
+
+def latent_workspace(geos, device) -> torch.Tensor:
+    """fp32 room for the partial results of units cut by a CTA boundary, for any batch of these geometries."""
+    sms = torch.cuda.get_device_properties(device).multi_processor_count
+    return torch.empty(2 * sms * 32 * (max(g.rw for g in geos) + 2), dtype=torch.float32, device=device)
+
+
+def latent_plan(cu_q, seq_lens, heads: int, max_q: int, window: int, plan) -> None:
+    """Prefix sums of the row tiles' key tiles -> ``plan [latent_units + 1]`` (int32): how ``latent_attention`` shares its
+    work. One per batch, window and head count; the CPU twin needs none."""
+    if not seq_lens.is_cuda:
+        return
+    B = seq_lens.shape[0]
+    assert plan.dtype == torch.int32 and plan.numel() >= latent_units(B, heads, max_q) + 1
+    check_rc(_lib().rb_latent_plan(ptr(cu_q), ptr(seq_lens), B, heads, max_q, window, ptr(plan), stream_handle(seq_lens.device)), "rb_latent_plan")
 
 
 def latent_attention(qa, cache, geo: LatentGeometry, block_tables, cu_q, seq_lens, sink, gate, out, *, scale: float, window: int,
-                     rows: int, max_q: int, splits: int = 1, workspace=None) -> None:
+                     rows: int, max_q: int, plan=None, workspace=None) -> None:
     """``out[h, t] = gate[t, h] * sum_j p_j c_j`` for the first ``rows`` tokens of ``qa [H, S, cw]``.
 
     ``cu_q`` ``[B+1]`` gives the rows of every sequence (None: one row per sequence); the new tokens are the last of the
-    sequence's ``seq_lens`` keys and already in the cache. ``workspace``: fp32, ``rows * H * splits * (rw + 2)``."""
+    sequence's ``seq_lens`` keys and already in the cache. bf16 on the GPU needs the batch's ``plan`` and a
+    ``latent_workspace``."""
     B = seq_lens.shape[0]
     H, S = qa.shape[0], qa.shape[1]
     if not qa.is_cuda:
-        flat = cache.view(-1, geo.cw)
+        flat = cache.view(-1, geo.cs)[:, :geo.cw]
         for b in range(B):
             t0, t1 = (b, b + 1) if cu_q is None else (int(cu_q[b]), int(cu_q[b + 1]))
             L = int(seq_lens[b])
@@ -262,19 +283,15 @@ def latent_attention(qa, cache, geo: LatentGeometry, block_tables, cu_q, seq_len
             out[:, t0:t1, :geo.rw] = o.to(out.dtype)
         return
     dt = _DT[qa.dtype]
-    if dt == 1:
-        splits = 1
-    part_o = part_ml = None
-    if splits > 1:
-        need = rows * H * splits * (geo.rw + 2)
-        assert workspace is not None and workspace.numel() >= need, "latent attention workspace too small"
-        part_o, part_ml = workspace, workspace[rows * H * splits * geo.rw:]
-    assert qa.is_contiguous() and out.is_contiguous() and sink.dtype == gate.dtype == torch.float32
-    rc = _lib().rb_latent_attn(ptr(qa), ptr(cache), ptr(block_tables), ptr(cu_q), ptr(seq_lens), ptr(sink), ptr(gate), ptr(out),
-                               ptr(part_o), ptr(part_ml), S, H, geo.cw, geo.rw, out.shape[2], geo.rw, block_tables.stride(0),
-                               cache.shape[0], splits, window, scale, B, rows, max_q, dt, ptr(status_tensor(qa.device)),
-                               stream_handle(qa.device))
-    check_rc(rc, "rb_latent_attn", 2 if splits > 1 else 1)
+    part_ml = None
+    if dt == 0:
+        n = workspace.numel() // (geo.rw + 2) * geo.rw
+        part_ml = workspace[n:]
+    assert qa.is_contiguous() and out.is_contiguous() and cache.is_contiguous() and sink.dtype == gate.dtype == torch.float32
+    rc = _lib().rb_latent_attn(ptr(qa), ptr(cache), ptr(block_tables), ptr(cu_q), ptr(seq_lens), ptr(sink), ptr(gate), ptr(out), ptr(plan),
+                               ptr(workspace), ptr(part_ml), S, H, geo.cw, geo.cs, geo.rw, out.shape[2], block_tables.stride(0),
+                               cache.shape[0], window, scale, B, rows, max_q, dt, ptr(status_tensor(qa.device)), stream_handle(qa.device))
+    check_rc(rc, "rb_latent_attn", 2 if dt == 0 else 1)
 
 
 def latent_gather(cache, geo: LatentGeometry, block_tables, bt_row0: int, cu_k, k_lo, n_rows: int, lat, rot) -> None:
@@ -282,7 +299,7 @@ def latent_gather(cache, geo: LatentGeometry, block_tables, bt_row0: int, cu_k, 
     latents -> ``lat [n, rw]``, rotated parts -> ``rot [n, rp]``."""
     B = k_lo.shape[0]
     if not cache.is_cuda:
-        flat = cache.view(-1, geo.cw)
+        flat = cache.view(-1, geo.cs)[:, :geo.cw]
         for b in range(B):
             s, e = int(cu_k[b]), int(cu_k[b + 1])
             key = torch.arange(e - s) + int(k_lo[b])
@@ -292,6 +309,6 @@ def latent_gather(cache, geo: LatentGeometry, block_tables, bt_row0: int, cu_k, 
             rot[s:e, :geo.rot_dim] = rows[:, geo.rw:geo.rw + geo.rot_dim]
         return
     rc = _lib().rb_latent_gather(ptr(cache), ptr(block_tables), bt_row0, block_tables.stride(0), cache.shape[0], ptr(cu_k), ptr(k_lo), B,
-                                 n_rows, ptr(lat), ptr(rot), geo.cw, geo.rw, geo.rp, geo.rw, _up(geo.rot_dim, 16),
+                                 n_rows, ptr(lat), ptr(rot), geo.cs, geo.rw, geo.rp, geo.rw, _up(geo.rot_dim, 16),
                                  ptr(status_tensor(cache.device)), stream_handle(cache.device))
     check_rc(rc, "rb_latent_gather")
