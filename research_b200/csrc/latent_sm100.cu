@@ -1,8 +1,8 @@
 // Attention over a shared latent ("latent attention") on a paged cache, for sm_100a.
 //
 // A token keeps one row in the cache, shared by all heads: the normalised latent c (kv_rank channels) and one rotated
-// key part. Per layer: [num_blocks, 16, CS], a row = c | zeros to a multiple of 16 | rotated part | zeros to CW, a
-// multiple of 32 | 8 unused channels (CS = CW + 8). Head h's key is (W_uk[h] c, rotated part) and its value W_uv[h] c.
+// key part. Per layer: [num_blocks, 16, CW], a row = c | zeros to a multiple of 16 | rotated part | zeros, CW a
+// multiple of 32. Head h's key is (W_uk[h] c, rotated part) and its value W_uv[h] c.
 //
 // Two evaluations of the same attention:
 //   absorbed : q_lat = W_uk[h]^T q, scores = q_lat . c + q_rot . k_rot, output W_uv[h] (sum_j p_j c_j). The cached rows are
@@ -17,6 +17,7 @@
 // All heads of a token form rows of one score tile: row r of a sequence is (token r / H, head r % H). The mask is a
 // causal sliding window; the softmax denominator also contains exp(sink[h]); every head's output is multiplied by a gate.
 #include "common.cuh"
+#include "tma_host.h"
 
 #include <math.h>
 
@@ -49,7 +50,7 @@ template <typename TA>
 __global__ void latent_append_kernel(const float* __restrict__ proj, long long ldp, const float* __restrict__ qn_w,
                                      const float* __restrict__ kn_w, float eps, const int* __restrict__ positions,
                                      const int* __restrict__ slots, const float2* __restrict__ table, int max_pos, int rot_pairs,
-                                     TA* __restrict__ cache, long long num_slots, int CS, int rot_off, TA* __restrict__ cq,
+                                     TA* __restrict__ cache, long long num_slots, int CW, int rot_off, TA* __restrict__ cq,
                                      long long ldq, float* __restrict__ gate, int q_rank, int kv_rank, int rot_dim, int H,
                                      int* status) {
   __shared__ float red[32];
@@ -74,7 +75,7 @@ __global__ void latent_append_kernel(const float* __restrict__ proj, long long l
     if (threadIdx.x == 0) set_status(status, ST_BAD_INDEX);
     return;
   }
-  TA* row = cache + (long long)slot * CS;
+  TA* row = cache + (long long)slot * CW;
   for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) row[i] = lat_cast<TA>(pc[i] * rc * kn_w[i]);
   for (int i = threadIdx.x; i < rot_dim; i += blockDim.x) {
     float v = pr[i];
@@ -129,27 +130,35 @@ __global__ void latent_query_kernel(TA* __restrict__ q, const int* __restrict__ 
 }
 
 // ------------------------------------------------------------------------------------------
-// Absorbed attention, bf16.
+// Absorbed attention, bf16, on the 5th-generation tensor cores.
 //
-// Work is a list of key tiles (32 keys) over all units; a unit is one row tile (16 or 32 rows) of one sequence. Every CTA
-// takes an equal share of the list, so ragged batches and short ones fill the machine alike; a unit cut by a CTA boundary
-// leaves partial results that latent_merge_kernel combines. The prefix sums of the units' tile counts come from
-// latent_plan_kernel, once per step and window.
+// Work is a list of key tiles (KT keys) over all units; a unit is NH (16 or 32) rows of one sequence. Every CTA takes an equal
+// share of the list, so ragged batches and short ones fill the machine alike; a unit cut by a CTA boundary leaves partial
+// results that latent_merge_kernel combines. The prefix sums of the units' tile counts come from latent_plan_kernel, once
+// per step and kind of layer.
 //
-// A CTA is a producer warp, which streams whole cache blocks (16 rows, one contiguous run) through a ring of shared-memory
-// stages, and two groups of four warps. In a group, warp w multiplies a quarter of the row's channels (its query fragments stay
-// in registers), the four partial scores meet in shared memory, every warp forms the same weights and sums a quarter of the
-// latent columns. With 16-row units the groups take alternate tiles and merge at the unit's end; with 32-row units each takes
-// half the rows and both read every tile. Cache rows carry 8 channels of padding, which keeps ldmatrix free of bank conflicts.
+// A tile of cached rows is brought into shared memory once (TMA, 16-row blocks, 128-byte swizzle) and is the operand of two
+// products:
+//   S   [rows, KT]      = Q C^T    : A = Q (K-major), B = the tile (K-major, all CW channels)
+//   O^T [channels, NH] += C^T P^T  : A = the tile read MN-major in blocks of 128 channels, B = P (K-major)
+// With the output transposed the few rows of a unit are the N side, so the accumulators take NH columns per 128 channels.
+// S has M = 128 although only NH rows are queries: the A descriptor runs on into the shared memory behind them, and those
+// rows of S are never read.
+//
+// Warps: 0 TMA producer, 1 MMA issuer + TMEM owner, 2-3 load the queries of the next unit, 4 softmax (one row per lane),
+// 4-7 rescale and store O^T. The running maximum is refreshed only when it grew by more than 2^8. A wait that runs out sets
+// the status and an abort flag that ends all other waits; the steps still run through, so that every barrier is met.
 // ------------------------------------------------------------------------------------------
-constexpr int LAT_KT = 32;                       // keys per tile
-constexpr int LAT_THREADS = 9 * 32;
+constexpr int LAT_THREADS = 256;
 constexpr int LAT_MIN_TILES = 2;                 // least share of a CTA
 constexpr int LAT_MAX_STAGES = 6;
+constexpr float LAT_RESCALE = 8.f;               // log2 units
 
 struct LatentAttnParams {
+  CUtensorMap map;         // cache rows [num_blocks * 16, CW], box 64 x 16
+  CUtensorMap q_map;       // one new token per sequence: qa as [H, S, CW], box 64 channels x 1 token x NH heads
   const void* qa;          // [H][S][CW]
-  const void* cache;       // [num_blocks, 16, CS]
+  const void* cache;       // [num_blocks, 16, CW]
   const int* block_tables; // [B, max_blocks]
   const int* cu_q;         // [B+1] rows of every sequence, or null: sequence b is row b
   const int* seq_lens;     // [B] keys per sequence, this step's tokens included
@@ -160,8 +169,8 @@ struct LatentAttnParams {
   float* part_o;           // [2 * grid][rows][RW]
   float* part_ml;          // [2 * grid][rows][2]
   long long S;
-  int B, H, CW, CS, RW, OW, row_tiles;   // RW: latent columns (a multiple of 16) that are summed
-  int max_blocks, num_blocks, window, stages;
+  int B, H, CW, RW, OW, row_tiles;       // RW: latent columns (a multiple of 16) that are summed
+  int max_blocks, num_blocks, window, stages, q_tma;
   float scale;
   int* status;
 };
@@ -194,7 +203,7 @@ __device__ __forceinline__ LatentUnit latent_unit(const int* cu_q, const int* se
 
 // One CTA: prefix sums of the tile counts of all units.
 __global__ void __launch_bounds__(1024) latent_plan_kernel(const int* __restrict__ cu_q, const int* __restrict__ seq_lens, int B, int H,
-                                                           int rows, int row_tiles, int window, int* __restrict__ plan) {
+                                                           int rows, int row_tiles, int window, int keys, int* __restrict__ plan) {
   __shared__ int warp_tot[32];
   __shared__ int carry;
   pdl_launch_dependents();
@@ -207,7 +216,7 @@ __global__ void __launch_bounds__(1024) latent_plan_kernel(const int* __restrict
     int n = 0;
     if (u < units) {
       const LatentUnit w = latent_unit(cu_q, seq_lens, u, row_tiles, rows, H, window);
-      n = (w.hi - w.lo + LAT_KT - 1) / LAT_KT;
+      n = (w.hi - w.lo + keys - 1) / keys;
     }
     for (int o = 1; o < 32; o <<= 1) {
       const int v = __shfl_up_sync(0xffffffffu, n, o);
@@ -224,313 +233,348 @@ __global__ void __launch_bounds__(1024) latent_plan_kernel(const int* __restrict
   }
 }
 
-// First unit whose tiles reach past `tile` (prefix[u] <= tile < prefix[u+1]).
-__device__ __forceinline__ int latent_find(const int* __restrict__ plan, int units, int tile) {
-  int lo = 0, hi = units;
-  while (hi - lo > 1) {
-    const int mid = (lo + hi) >> 1;
-    if (plan[mid] <= tile) lo = mid; else hi = mid;
-  }
-  return lo;
+// The unit that holds `tile` (plan[u] <= tile < plan[u + 1]), found by all threads of a CTA at once.
+__device__ __forceinline__ int latent_find_cta(const int* __restrict__ plan, int units, int tile, int* shared) {
+  for (int u = threadIdx.x; u < units; u += blockDim.x)
+    if (plan[u] <= tile && tile < plan[u + 1]) *shared = u;
+  __syncthreads();
+  return *shared;
 }
 __device__ __forceinline__ int latent_share(int total, int ctas) { return max((total + ctas - 1) / ctas, LAT_MIN_TILES); }
 
-__device__ __forceinline__ void lat_bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-               ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+__device__ __forceinline__ float lat_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 __device__ __forceinline__ void lat_bar(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
-__device__ __forceinline__ void lat_ldsm4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void lat_ldsm4t(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void lat_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 
-template <int NT, int KW, bool WIDE>
-__global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const LatentAttnParams p) {
-  constexpr int ROWS = WIDE ? 32 : 16;
-  extern __shared__ __align__(128) uint8_t smem[];
-  __shared__ __align__(8) uint64_t full[LAT_MAX_STAGES], empty[LAT_MAX_STAGES];
-  __shared__ int abort_flag;
+template <int NH, int KT>
+__global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __grid_constant__ LatentAttnParams p) {
+  constexpr int CHUNK = KT * 128;                // bytes of 64 channels of a tile
+  constexpr int PAGES = KT / LAT_BLOCK;
+  constexpr uint32_t O_COL = 128;                // TMEM: S at columns 0 and 64, O^T behind
+  extern __shared__ __align__(128) uint8_t smem_raw[];
+  __shared__ __align__(8) uint64_t kv_full[LAT_MAX_STAGES], kv_empty[LAT_MAX_STAGES];
+  __shared__ __align__(8) uint64_t q_full, q_empty, s_full[2], a_full[2], p_full[2], o_done, o_free;
+  __shared__ float s_alpha[2][NH], s_scale[NH];
+  __shared__ int s_flag[2];
+  __shared__ long long s_row[NH];
+  __shared__ uint32_t tmem_base_smem;
+  __shared__ int abort_flag, u_shared;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int tile_bytes = LAT_KT * p.CS * 2, page_bytes = LAT_BLOCK * p.CS * 2;
-  const uint32_t ring = smem_u32(smem);
-  uint8_t* exch = smem + p.stages * tile_bytes;         // partial scores of both groups, or a group's sums at a unit's end
-  if (threadIdx.x == 0) {
-    abort_flag = 0;
-    for (int i = 0; i < p.stages; ++i) {
-      mbar_init(smem_u32(&full[i]), 1);
-      mbar_init(smem_u32(&empty[i]), WIDE ? 8 : 4);
-    }
-    fence_mbar_init();
-  }
+  const int nch = (p.CW + 63) / 64, nblk = (p.RW + 127) / 128, tile_bytes = max(nch, 2 * nblk) * CHUNK;
   pdl_launch_dependents();
-  __syncthreads();
   pdl_wait();
-  volatile int* abortp = &abort_flag;
   const int units = p.B * p.row_tiles, total = p.plan[units];
   const int share = latent_share(total, gridDim.x);
   const int t_begin = min((int)blockIdx.x * share, total), t_end = min(t_begin + share, total);
-  if (t_begin >= t_end) return;                         // uniform per CTA
-  const int u_first = latent_find(p.plan, units, t_begin);
+  if (t_begin >= t_end) return;                  // uniform per CTA, before any set-up
+  const int u_first = latent_find_cta(p.plan, units, t_begin, &u_shared);
 
-  if (warp == 8) {
-    // ---------------------------------------------------------------- producer
-    if (lane == 0) {
-      uint32_t it = 0;
-      bool ok = true;
-      for (int u = u_first, t = t_begin; t < t_end; ++u) {
-        const int u_end = min(p.plan[u + 1], t_end);
-        if (u_end <= t) continue;
-        const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, ROWS, p.H, p.window);
-        const int* bt = p.block_tables + (long long)w.b * p.max_blocks;
-        const int last_page = (w.hi - 1) / LAT_BLOCK;
-        for (int k0 = w.lo + (t - p.plan[u]) * LAT_KT; t < u_end; ++t, k0 += LAT_KT, ++it) {
-          const uint32_t s = it % p.stages;
-          if (ok) ok = mbar_wait_bounded(smem_u32(&empty[s]), ((it / p.stages) & 1u) ^ 1u, abortp, p.status, ST_TIMEOUT_SMEM_EMPTY);
-          if (!ok) break;                               // the consumers' waits end with the abort flag
-          const uint32_t bar = smem_u32(&full[s]);
-          mbar_expect_tx(bar, 2 * page_bytes);
-#pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            // past the last page the tile repeats it: those keys are masked, and their values are finite
-            int blk = bt[min(k0 / LAT_BLOCK + i, last_page)];
-            if (blk < 0 || blk >= p.num_blocks) { set_status(p.status, ST_BAD_INDEX); blk = 0; }
-            lat_bulk_load(ring + s * tile_bytes + i * page_bytes,
-                          reinterpret_cast<const __nv_bfloat16*>(p.cache) + (long long)blk * LAT_BLOCK * p.CS, page_bytes, bar);
-          }
-        }
-        if (!ok) break;
-      }
-      if (!ok) {   // drain: no bulk copy may land after the CTA has gone
-        for (uint32_t j = it > (uint32_t)p.stages ? it - p.stages : 0; j < it; ++j) {
-          const uint64_t c0 = globaltimer_ns();
-          while (!mbar_try_wait(smem_u32(&full[j % p.stages]), (j / p.stages) & 1u))
-            if (globaltimer_ns() - c0 > 50000000ull) break;
-        }
-      }
+  const uint32_t q_s = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* q_ptr = smem_raw + (q_s - smem_u32(smem_raw));
+  const uint32_t p_s = q_s + nch * NH * 128, kv_s = p_s + 2 * NH * 128;
+  uint8_t* p_ptr = q_ptr + nch * NH * 128;
+  if (threadIdx.x == 0) {
+    abort_flag = 0;
+    for (int i = 0; i < p.stages; ++i) {
+      mbar_init(smem_u32(&kv_full[i]), 1);
+      mbar_init(smem_u32(&kv_empty[i]), 1);
     }
-    return;
+    mbar_init(smem_u32(&q_full), p.q_tma ? 1 : 2);
+    mbar_init(smem_u32(&q_empty), 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(smem_u32(&s_full[i]), 1);
+      mbar_init(smem_u32(&a_full[i]), 1);
+      mbar_init(smem_u32(&p_full[i]), 4);
+    }
+    mbar_init(smem_u32(&o_done), 1);
+    mbar_init(smem_u32(&o_free), 4);
+    fence_mbar_init();
   }
+  const uint32_t tmem_cols = O_COL + nblk * NH <= 256 ? 256 : 512;
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_smem), tmem_cols);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = tmem_base_smem, tmem_o = tmem_base + O_COL;
+  volatile int* abortp = &abort_flag;
 
-  // ------------------------------------------------------------------ consumers
-  const int group = warp >> 2, wg = warp & 3, g = lane >> 2, tq = lane & 3;
-  const int ksteps = p.CW / 16, k_per = (ksteps + 3) / 4, k_lo = wg * k_per, k_n = max(0, min(k_per, ksteps - k_lo));
-  const int n16 = p.RW / 16, n_per = (n16 + 3) / 4, col0 = wg * n_per * 16, n_n = max(0, min(n_per, n16 - wg * n_per));   // 16-column pairs
-  const float log2e = 1.4426950408889634f, scale_log2 = p.scale * log2e;
-  float2* my_exch = reinterpret_cast<float2*>(exch + group * (2 * 4 * 8 * 32 * 8));   // [2 buffers][4 warps][8][32 lanes]
-  const int row_bytes = p.CS * 2;
-  uint32_t it = 0, local = 0;
-  for (int u = u_first, t = t_begin; t < t_end; ++u) {
-    const int u_begin = p.plan[u], u_stop = p.plan[u + 1], u_end = min(u_stop, t_end);
-    if (u_end <= t) continue;
-    const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, ROWS, p.H, p.window);
-    const int rg = WIDE ? group * 16 : 0;               // this group's rows: rg + g and rg + g + 8
-    // query fragments of this warp's channels, and the positions of this lane's two rows
-    uint32_t qf[KW][4];
-    int pos[2];
-    float m[2], l[2];
-    {
-      const __nv_bfloat16* src[2];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int r = rg + g + i * 8;
-        const bool ok = r < w.n_rows;
-        const int tok = (w.r0 + (ok ? r : 0)) / p.H, h = (w.r0 + (ok ? r : 0)) - tok * p.H;
-        src[i] = ok ? reinterpret_cast<const __nv_bfloat16*>(p.qa) + ((long long)h * p.S + w.t0 + tok) * p.CW : nullptr;
-        pos[i] = w.L - w.q_len + tok;
-        // the sink enters the running maximum and the sum once, with the unit's first tile
-        const bool sink = t == u_begin && (WIDE || group == 0);
-        m[i] = sink ? p.sink[h] * log2e : -INFINITY;
-        l[i] = sink ? 1.f : 0.f;
-      }
-#pragma unroll
-      for (int k = 0; k < KW; ++k) {
-        const int c = (k_lo + k) * 16 + 2 * tq;
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const bool ok = k < k_n && src[i] != nullptr;
-          qf[k][i] = ok ? *reinterpret_cast<const uint32_t*>(src[i] + c) : 0u;
-          qf[k][i + 2] = ok ? *reinterpret_cast<const uint32_t*>(src[i] + c + 8) : 0u;
+  if (warp == 0) {
+    // ---------------------------------------------------------------- TMA producer: lane i loads boxes i, i + 32, ...
+    uint32_t it = 0;
+    bool ok = true;
+    const int boxes = PAGES * nch;
+    for (int u = u_first, t = t_begin; t < t_end && ok; ++u) {
+      const int u_end = min(p.plan[u + 1], t_end);
+      if (u_end <= t) continue;
+      const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, NH, p.H, p.window);
+      const int* bt = p.block_tables + (long long)w.b * p.max_blocks;
+      const int n_pages = (w.hi + LAT_BLOCK - 1) / LAT_BLOCK;
+      for (int k0 = w.lo + (t - p.plan[u]) * KT; t < u_end && ok; ++t, k0 += KT, ++it) {
+        const uint32_t s = it % p.stages;
+        ok = mbar_wait_bounded(smem_u32(&kv_empty[s]), ((it / p.stages) & 1u) ^ 1u, abortp, p.status, ST_TIMEOUT_SMEM_EMPTY);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        const uint32_t bar = smem_u32(&kv_full[s]), dst = kv_s + s * tile_bytes;
+        if (lane == 0) mbar_expect_tx(bar, boxes * 2048);
+        __syncwarp();
+        for (int i = lane; i < boxes; i += 32) {
+          const int pg = i / nch, c = i - pg * nch;
+          int blk = p.num_blocks;                 // past the sequence's end: the copy fills zeros
+          if (k0 / LAT_BLOCK + pg < n_pages) {
+            blk = bt[k0 / LAT_BLOCK + pg];
+            if (blk < 0 || blk >= p.num_blocks) { set_status(p.status, ST_BAD_INDEX); blk = p.num_blocks; }
+          }
+          tma_load_2d(dst + c * CHUNK + pg * 2048, &p.map, bar, c * 64, blk * LAT_BLOCK);
         }
       }
     }
-    float o[NT][4];
-#pragma unroll
-    for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
-
-    const int t_unit = t;
-    for (int k0 = w.lo + (t - u_begin) * LAT_KT; t < u_end; ++t, k0 += LAT_KT, ++it) {
-      if (!WIDE && (int)(it & 1u) != group) continue;
-      const uint32_t s = it % p.stages;
-      // a wait that runs out sets the status and the abort flag; the remaining (meaningless) steps run through so that every
-      // barrier is met
-      mbar_wait_bounded(smem_u32(&full[s]), (it / p.stages) & 1u, abortp, p.status, ST_TIMEOUT_SMEM_FULL);
-      const uint32_t tile = ring + s * tile_bytes;
-      float acc[4][4];
-#pragma unroll
-      for (int n = 0; n < 4; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-      {
-        const uint32_t ka = tile + (uint32_t)(((lane >> 4) * 8 + (lane & 7)) * row_bytes + (k_lo * 16 + ((lane >> 3) & 1) * 8) * 2);
-#pragma unroll
-        for (int k = 0; k < KW; ++k) {
-          if (k < k_n) {
-            uint32_t b0, b1, b2, b3;
-            lat_ldsm4(ka + k * 32, b0, b1, b2, b3);
-            lat_mma(acc[0], qf[k], b0, b1);
-            lat_mma(acc[1], qf[k], b2, b3);
-            lat_ldsm4(ka + 16 * row_bytes + k * 32, b0, b1, b2, b3);
-            lat_mma(acc[2], qf[k], b0, b1);
-            lat_mma(acc[3], qf[k], b2, b3);
-          }
-        }
+    if (!ok && lane == 0) {   // drain: no bulk copy may land after the CTA has gone
+      for (uint32_t j = it > (uint32_t)p.stages ? it - p.stages : 0; j < it; ++j) {
+        const uint64_t c0 = globaltimer_ns();
+        while (!mbar_try_wait(smem_u32(&kv_full[j % p.stages]), (j / p.stages) & 1u))
+          if (globaltimer_ns() - c0 > 50000000ull) break;
       }
-      // sum the four quarters: every lane reads its own fragment positions of all warps, in the same order everywhere
-      float2* ex = my_exch + (local & 1u) * (4 * 8 * 32);
-      ++local;
-#pragma unroll
-      for (int n = 0; n < 4; ++n) {
-        ex[(wg * 8 + 2 * n) * 32 + lane] = make_float2(acc[n][0], acc[n][1]);
-        ex[(wg * 8 + 2 * n + 1) * 32 + lane] = make_float2(acc[n][2], acc[n][3]);
-      }
-      lat_bar(1 + group, 128);
-#pragma unroll
-      for (int n = 0; n < 8; ++n) {
-        float2 a = ex[n * 32 + lane];
-#pragma unroll
-        for (int i = 1; i < 4; ++i) {
-          const float2 b = ex[(i * 8 + n) * 32 + lane];
-          a.x += b.x;
-          a.y += b.y;
-        }
-        acc[n >> 1][(n & 1) * 2] = a.x;
-        acc[n >> 1][(n & 1) * 2 + 1] = a.y;
-      }
-      // mask, online softmax; row i of the lane has columns 8n + 2tq, +1
-      float alpha[2];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        float mx = -INFINITY;
-#pragma unroll
-        for (int n = 0; n < 4; ++n)
-#pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            const int key = k0 + n * 8 + 2 * tq + j;
-            float v = acc[n][i * 2 + j] * scale_log2;
-            if (key > pos[i] || key <= pos[i] - p.window) v = -INFINITY;
-            acc[n][i * 2 + j] = v;
-            mx = fmaxf(mx, v);
-          }
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        const float m_new = fmaxf(m[i], mx), base = m_new == -INFINITY ? 0.f : m_new;
-        float sum = 0.f;
-#pragma unroll
-        for (int n = 0; n < 4; ++n)
-#pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            const float e = exp2f(acc[n][i * 2 + j] - base);
-            acc[n][i * 2 + j] = e;
-            sum += e;
-          }
-        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-        sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-        alpha[i] = exp2f(m[i] - base);
-        l[i] = l[i] * alpha[i] + sum;
-        m[i] = m_new;
-      }
-      if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
-#pragma unroll
-        for (int n = 0; n < NT; ++n) { o[n][0] *= alpha[0]; o[n][1] *= alpha[0]; o[n][2] *= alpha[1]; o[n][3] *= alpha[1]; }
-      }
-#pragma unroll
-      for (int ks = 0; ks < 2; ++ks) {
-        const uint32_t a[4] = {pack_bf16x2(acc[2 * ks][0], acc[2 * ks][1]), pack_bf16x2(acc[2 * ks][2], acc[2 * ks][3]),
-                               pack_bf16x2(acc[2 * ks + 1][0], acc[2 * ks + 1][1]), pack_bf16x2(acc[2 * ks + 1][2], acc[2 * ks + 1][3])};
-        const uint32_t va = tile + (uint32_t)((ks * 16 + (lane & 15)) * row_bytes + (col0 + (lane >> 4) * 8) * 2);
-#pragma unroll
-        for (int n = 0; n < NT / 2; ++n) {
-          if (n < n_n) {
-            uint32_t b0, b1, b2, b3;
-            lat_ldsm4t(va + n * 32, b0, b1, b2, b3);
-            lat_mma(o[2 * n], a, b0, b1);
-            lat_mma(o[2 * n + 1], a, b2, b3);
-          }
-        }
-      }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(smem_u32(&empty[s]));
     }
-
-    if (!WIDE) {
-      // the groups' sums over alternate tiles meet: group 1 leaves its own in shared memory, group 0 adds them
-      float4* mo = reinterpret_cast<float4*>(exch);               // [4 warps][NT][32 lanes]
-      float4* mml = mo + 4 * NT * 32;                             // [32 lanes] (m, m', l, l')
-      lat_bar(3, 256);                                            // both groups are done with the partial scores
-      if (group == 1) {
-#pragma unroll
-        for (int n = 0; n < NT; ++n) mo[(wg * NT + n) * 32 + lane] = make_float4(o[n][0], o[n][1], o[n][2], o[n][3]);
-        if (wg == 0) mml[lane] = make_float4(m[0], m[1], l[0], l[1]);
-      }
-      lat_bar(3, 256);
-      if (group == 0) {
-        const float4 q4 = mml[lane];
-        float fa[2], fb[2];
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const float mb = i ? q4.y : q4.x, lb = i ? q4.w : q4.z;
-          const float mn = fmaxf(m[i], mb), base = mn == -INFINITY ? 0.f : mn;
-          fa[i] = exp2f(m[i] - base);
-          fb[i] = exp2f(mb - base);
-          l[i] = l[i] * fa[i] + lb * fb[i];
-          m[i] = mn;
+  } else if (warp == 1) {
+    // ---------------------------------------------------------------- MMA issuer
+    if (elect_one_sync()) {
+      constexpr uint32_t idesc_s = make_idesc_bf16(128, KT, 0, 0);
+      constexpr uint32_t idesc_o = make_idesc_bf16(128, NH, 1, 0);
+      const int n = t_end - t_begin, ksteps = p.CW / 16;
+      int uq = 0, u_s = u_first, u_o = u_first;      // units started by the scores / being summed
+      uint32_t o_units = 0;
+      auto issue_s = [&](int j) {
+        const int t = t_begin + j;
+        while (p.plan[u_s + 1] <= t) ++u_s;
+        if (t == t_begin || t == p.plan[u_s])       // a new unit: its queries
+          mbar_wait_bounded(smem_u32(&q_full), (uint32_t)(uq++) & 1u, abortp, p.status, ST_TIMEOUT_SMEM_FULL);
+        const uint32_t s = j % p.stages;
+        mbar_wait_bounded(smem_u32(&kv_full[s]), (j / p.stages) & 1u, abortp, p.status, ST_TIMEOUT_SMEM_FULL);
+        tc_fence_after();
+        const uint32_t tile = kv_s + s * tile_bytes;
+        // descriptors advance by plain additions (addresses in 16-byte units): one thread issues all of this
+        uint64_t ad = make_smem_desc_sw128(q_s, 16, 1024), bd = make_smem_desc_sw128(tile, 16, 1024);
+        const uint32_t d = tmem_base + (j & 1) * 64;
+        umma_bf16(d, ad, bd, idesc_s, 0u);
+        umma_bf16(d, ad + 2, bd + 2, idesc_s, 1u);
+        if (ksteps > 2) {
+          umma_bf16(d, ad + 4, bd + 4, idesc_s, 1u);
+          umma_bf16(d, ad + 6, bd + 6, idesc_s, 1u);
         }
-#pragma unroll
-        for (int n = 0; n < NT; ++n) {
-          const float4 v = mo[(wg * NT + n) * 32 + lane];
-          o[n][0] = o[n][0] * fa[0] + v.x * fb[0];
-          o[n][1] = o[n][1] * fa[0] + v.y * fb[0];
-          o[n][2] = o[n][2] * fa[1] + v.z * fb[1];
-          o[n][3] = o[n][3] * fa[1] + v.w * fb[1];
+#pragma unroll 2
+        for (int c = 1; c < nch; ++c) {
+          ad += (NH * 128) >> 4;
+          bd += CHUNK >> 4;
+          umma_bf16(d, ad, bd, idesc_s, 1u);
+          umma_bf16(d, ad + 2, bd + 2, idesc_s, 1u);
+          if (c * 4 + 2 < ksteps) {              // CW is a multiple of 32: the last chunk may be half
+            umma_bf16(d, ad + 4, bd + 4, idesc_s, 1u);
+            umma_bf16(d, ad + 6, bd + 6, idesc_s, 1u);
+          }
         }
+        umma_commit(smem_u32(&s_full[j & 1]));
+        if (t + 1 == t_end || t + 1 == p.plan[u_s + 1]) umma_commit(smem_u32(&q_empty));   // the unit's last scores
+      };
+      issue_s(0);
+      for (int j = 0; j < n; ++j) {
+        const int t = t_begin + j;
+        while (p.plan[u_o + 1] <= t) ++u_o;
+        const bool first = t == t_begin || t == p.plan[u_o], last = t + 1 == p.plan[u_o + 1];
+        if (j + 1 < n && !last) issue_s(j + 1);     // the next tile's scores overlap this tile's softmax
+        mbar_wait_bounded(smem_u32(&p_full[j & 1]), (j >> 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+        if (first && o_units++ > 0)                 // the previous unit's sums have left TMEM
+          mbar_wait_bounded(smem_u32(&o_free), (o_units - 2) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_EMPTY);
+        tc_fence_after();
+        const uint32_t s = j % p.stages, tile = kv_s + s * tile_bytes;
+        uint64_t ad = make_smem_desc_sw128(tile, CHUNK, 1024);
+        const uint64_t bd = make_smem_desc_sw128(p_s + (j & 1) * (NH * 128), 16, 1024);
+#pragma unroll 2
+        for (int m = 0; m < nblk; ++m, ad += (2 * CHUNK) >> 4)
+#pragma unroll
+          for (int k = 0; k < KT / 16; ++k)
+            umma_bf16(tmem_o + m * NH, ad + k * (2048 >> 4), bd + 2 * k, idesc_o, (!first || k > 0) ? 1u : 0u);
+        umma_commit(smem_u32(&kv_empty[s]));
+        umma_commit(smem_u32(&o_done));
+        if (j + 1 < n && last) issue_s(j + 1);
       }
-      lat_bar(3, 256);
+      // nothing of this CTA is in flight when it frees its TMEM
+      mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(n - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
     }
-    if (WIDE || group == 0) {
-      const bool whole = t_unit == u_begin && u_end == u_stop;
-      const long long slot = 2ll * blockIdx.x + (u_begin > t_begin ? 1 : 0);
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int r = rg + g + i * 8;
-        if (r >= w.n_rows) continue;
-        if (whole) {
+  } else if (warp < 4) {
+    // ---------------------------------------------------------------- query rows of every unit
+    int uq = 0;
+    const int per_row = nch * 8, tid = threadIdx.x - 64;
+    const bool q_tma = p.q_tma != 0;
+    for (int u = u_first, t = t_begin; t < t_end; ++u) {
+      const int u_end = min(p.plan[u + 1], t_end);
+      if (u_end <= t) continue;
+      t = u_end;
+      const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, NH, p.H, p.window);
+      if (uq > 0) mbar_wait_bounded(smem_u32(&q_empty), (uint32_t)(uq - 1) & 1u, abortp, p.status, ST_TIMEOUT_SMEM_EMPTY);
+      if (q_tma) {                                  // the unit's rows are heads r0.. of one token
+        if (warp == 2 && lane == 0) {
+          mbar_expect_tx(smem_u32(&q_full), nch * NH * 128);
+          for (int c = 0; c < nch; ++c) tma_load_3d(q_s + c * (NH * 128), &p.q_map, smem_u32(&q_full), c * 64, w.t0, w.r0);
+        }
+        ++uq;
+        continue;
+      }
+#pragma unroll 4
+      for (int i = tid; i < NH * per_row; i += 64) {
+        const int r = i / per_row, c = i - r * per_row;      // 16-byte unit c of row r
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (r < w.n_rows && c * 8 < p.CW) {
           const int tok = (w.r0 + r) / p.H, h = (w.r0 + r) - tok * p.H;
-          const float f = l[i] > 0.f ? p.gate[(long long)(w.t0 + tok) * p.H + h] / l[i] : 0.f;
-          __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + ((long long)h * p.S + w.t0 + tok) * p.OW + col0 + 2 * tq;
+          v = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.qa) + ((long long)h * p.S + w.t0 + tok) * p.CW + c * 8);
+        }
+        *reinterpret_cast<uint4*>(q_ptr + (c >> 3) * (NH * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+      }
+      fence_proxy_async_smem();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(&q_full));
+      ++uq;
+    }
+  } else {
+    // ---------------------------------------------------------------- softmax (warp 4), O^T (warps 4-7)
+    const int qd = warp - 4;
+    const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
+    const float log2e = 1.4426950408889634f, scale_log2 = p.scale * log2e;
+    int j = 0;
+    for (int u = u_first, t = t_begin; t < t_end; ++u) {
+      const int u_begin = p.plan[u], u_stop = p.plan[u + 1], u_end = min(u_stop, t_end);
+      if (u_end <= t) continue;
+      const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, NH, p.H, p.window);
+      const bool has_first = t == u_begin, whole = has_first && u_end == u_stop, row_ok = lane < w.n_rows;
+      const int tok = (w.r0 + (row_ok ? lane : 0)) / p.H, head = (w.r0 + (row_ok ? lane : 0)) - tok * p.H;
+      const int pos = w.L - w.q_len + tok;
+      const int pos_min = w.L - w.q_len + w.r0 / p.H, pos_max = w.L - w.q_len + (w.r0 + w.n_rows - 1) / p.H;
+      float m_used = -INFINITY, l = 0.f;
+      const int t_piece = t;
+      for (int k0 = w.lo + (t - u_begin) * KT; t < u_end; ++t, k0 += KT, ++j) {
+        const int b = j & 1;
+        const uint32_t ph = (j >> 1) & 1u;
+        if (qd == 0) {
+          mbar_wait_bounded(smem_u32(&s_full[b]), ph, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+          __syncwarp();
+          tc_fence_after();
+          uint32_t v[KT];
+          tmem_ld_32x32(tmem_base + b * 64, *reinterpret_cast<uint32_t(*)[32]>(&v[0]));
+          if constexpr (KT == 48) tmem_ld_32x16(tmem_base + b * 64 + 32, *reinterpret_cast<uint32_t(*)[16]>(&v[32]));
+          tmem_ld_wait();
+          tc_fence_before();
+          if (k0 + KT - 1 > pos_min || k0 <= pos_max - p.window) {
 #pragma unroll
-          for (int n = 0; n < NT; ++n)
-            if (n < 2 * n_n) *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16x2(o[n][2 * i] * f, o[n][2 * i + 1] * f);
+            for (int i = 0; i < KT; ++i)
+              if (k0 + i > pos || k0 + i <= pos - p.window) v[i] = 0xff800000u;   // -inf
+          }
+          float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+          for (int i = 0; i < KT; ++i) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(v[i]));
+          const float m_new = fmaxf(m_used, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale_log2);
+          const bool need = row_ok && (m_new > m_used + LAT_RESCALE || (m_used == -INFINITY && m_new != -INFINITY));
+          const float alpha = need && m_used != -INFINITY ? lat_exp2(m_used - m_new) : 1.f;
+          const int any = __any_sync(0xffffffffu, need && t > t_piece);
+          if (need) { m_used = m_new; l *= alpha; }
+          if (lane < NH) s_alpha[b][lane] = alpha;
+          if (lane == 0) s_flag[b] = any;
+          const float mref = m_used == -INFINITY ? 0.f : m_used;
+          float ls[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+          for (int i = 0; i < KT; ++i) {
+            const float x = lat_exp2(fmaf(__uint_as_float(v[i]), scale_log2, -mref));
+            ls[i & 3] += x;
+            v[i] = __float_as_uint(x);
+          }
+          l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
+          if (lane < NH) {
+            uint8_t* prow = p_ptr + b * (NH * 128) + lane * 128;
+#pragma unroll
+            for (int i = 0; i < KT / 8; ++i) {
+              uint4 o;
+              o.x = row_ok ? pack_bf16x2(__uint_as_float(v[i * 8]), __uint_as_float(v[i * 8 + 1])) : 0u;
+              o.y = row_ok ? pack_bf16x2(__uint_as_float(v[i * 8 + 2]), __uint_as_float(v[i * 8 + 3])) : 0u;
+              o.z = row_ok ? pack_bf16x2(__uint_as_float(v[i * 8 + 4]), __uint_as_float(v[i * 8 + 5])) : 0u;
+              o.w = row_ok ? pack_bf16x2(__uint_as_float(v[i * 8 + 6]), __uint_as_float(v[i * 8 + 7])) : 0u;
+              *reinterpret_cast<uint4*>(prow + ((i ^ (lane & 7)) << 4)) = o;
+            }
+          }
+          fence_proxy_async_smem();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(smem_u32(&a_full[b]));
         } else {
-          float* dst = p.part_o + (slot * ROWS + r) * p.RW + col0 + 2 * tq;
+          mbar_wait_bounded(smem_u32(&a_full[b]), ph, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+          __syncwarp();
+        }
+        if (*(volatile int*)&s_flag[b]) {          // O^T holds the tiles before this one
+          mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+          __syncwarp();
+          tc_fence_after();
+#pragma unroll 1
+          for (int c = 0; c < nblk * NH; c += 32) {
+            uint32_t o[32];
+            tmem_ld_32x32(tmem_o + lane_addr + c, o);
+            tmem_ld_wait();
 #pragma unroll
-          for (int n = 0; n < NT; ++n)
-            if (n < 2 * n_n) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(o[n][2 * i], o[n][2 * i + 1]);
-          if (wg == 0 && tq == 0) {
-            p.part_ml[(slot * ROWS + r) * 2] = m[i];
-            p.part_ml[(slot * ROWS + r) * 2 + 1] = l[i];
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[b][i & (NH - 1)]);
+            tmem_st_32x32(tmem_o + lane_addr + c, o);
+          }
+          tmem_st_wait();
+          tc_fence_before();
+        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&p_full[b]));
+      }
+      // ---- the piece is complete ----
+      const long long slot = 2ll * blockIdx.x + (u_begin > t_begin ? 1 : 0);
+      if (qd == 0 && lane < NH) {
+        float m = m_used, f = 1.f;
+        if (has_first) {                            // the sink: in the denominator once, no value
+          const float sk = p.sink[head] * log2e;
+          m = fmaxf(m_used, sk);
+          f = lat_exp2(m_used - m);
+          l = l * f + lat_exp2(sk - m);
+        }
+        if (whole) f = l > 0.f ? f * p.gate[(long long)(w.t0 + tok) * p.H + head] / l : 0.f;
+        s_scale[lane] = f;
+        s_row[lane] = whole ? ((long long)head * p.S + w.t0 + tok) * p.OW : (slot * NH + lane) * p.RW;
+        if (!whole && row_ok) {
+          p.part_ml[(slot * NH + lane) * 2] = m;
+          p.part_ml[(slot * NH + lane) * 2 + 1] = l;
+        }
+      }
+      mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      lat_bar(1, 128);
+      tc_fence_after();
+#pragma unroll 1
+      for (int c = 0; c < nblk * NH; c += 32) {
+        uint32_t o[32];
+        tmem_ld_32x32(tmem_o + lane_addr + c, o);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const int r = i & (NH - 1), ch = (c + i) / NH * 128 + qd * 32 + lane;
+          if (r < w.n_rows && ch < p.RW) {
+            const float x = __uint_as_float(o[i]) * s_scale[r];
+            if (whole) reinterpret_cast<__nv_bfloat16*>(p.out)[s_row[r] + ch] = __float2bfloat16_rn(x);
+            else p.part_o[s_row[r] + ch] = x;
           }
         }
       }
+      tc_fence_before();
+      lat_bar(1, 128);                              // the row tables are rewritten by the next unit
+      if (lane == 0) mbar_arrive(smem_u32(&o_free));
     }
+  }
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, tmem_cols);
   }
 }
 
@@ -538,10 +582,11 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const Laten
 __global__ void latent_merge_kernel(const LatentAttnParams p, int ctas, int rows) {
   pdl_launch_dependents();
   pdl_wait();
+  __shared__ int u_shared;
   const int units = p.B * p.row_tiles, total = p.plan[units], share = latent_share(total, ctas);
   const long long cut = (long long)(blockIdx.y + 1) * share;
   if (cut >= total) return;
-  const int u = latent_find(p.plan, units, (int)cut), u_begin = p.plan[u], u_stop = p.plan[u + 1];
+  const int u = latent_find_cta(p.plan, units, (int)cut, &u_shared), u_begin = p.plan[u], u_stop = p.plan[u + 1];
   if (u_begin == cut || cut - share > u_begin) return;            // no cut, or an earlier boundary has it
   const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, rows, p.H, p.window);
   const int r = blockIdx.x;
@@ -598,7 +643,7 @@ __global__ void __launch_bounds__(128) latent_attn_f32_kernel(const LatentAttnPa
   for (int key = lo; key < hi; ++key) {
     const int blk = p.block_tables[(long long)b * p.max_blocks + key / LAT_BLOCK];
     if (blk < 0 || blk >= p.num_blocks) { set_status(p.status, ST_BAD_INDEX); continue; }
-    const float* c = reinterpret_cast<const float*>(p.cache) + ((long long)blk * LAT_BLOCK + (key & (LAT_BLOCK - 1))) * p.CS;
+    const float* c = reinterpret_cast<const float*>(p.cache) + ((long long)blk * LAT_BLOCK + (key & (LAT_BLOCK - 1))) * p.CW;
     float kv[LAT_F32_MAX];
     float s = 0.f;
 #pragma unroll
@@ -624,7 +669,7 @@ __global__ void __launch_bounds__(128) latent_attn_f32_kernel(const LatentAttnPa
 // Cached rows [k_lo[b], k_lo[b] + cu_k[b+1] - cu_k[b]) of every sequence, packed: latent part [n, RW], rotated part [n, RP].
 __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_tables, int bt_row0,
                                      int max_blocks, int num_blocks, const int* __restrict__ cu_k, const int* __restrict__ k_lo,
-                                     int B, __nv_bfloat16* __restrict__ lat, __nv_bfloat16* __restrict__ rot, int CS, int RW,
+                                     int B, __nv_bfloat16* __restrict__ lat, __nv_bfloat16* __restrict__ rot, int CW, int RW,
                                      int RP, int rot_off, int rot_cols, int* status) {
   pdl_launch_dependents();
   pdl_wait();
@@ -635,7 +680,7 @@ __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, co
   const int key = k_lo[b] + row - cu_k[b];
   const int blk = block_tables[(long long)(bt_row0 + b) * max_blocks + key / LAT_BLOCK];
   if (blk < 0 || blk >= num_blocks) { if (lane == 0) set_status(status, ST_BAD_INDEX); return; }
-  const __nv_bfloat16* src = cache + ((long long)blk * LAT_BLOCK + (key & (LAT_BLOCK - 1))) * CS;
+  const __nv_bfloat16* src = cache + ((long long)blk * LAT_BLOCK + (key & (LAT_BLOCK - 1))) * CW;
   for (int c = lane; c < RW / 8; c += 32)
     *reinterpret_cast<uint4*>(lat + (long long)row * RW + c * 8) = *reinterpret_cast<const uint4*>(src + c * 8);
   for (int c = lane; c < RP / 8; c += 32)
@@ -653,23 +698,48 @@ static int latent_sms() {
   return n;
 }
 
-template <int NT, bool WIDE>
-static int launch_latent(LatentAttnParams p, int ctas, cudaStream_t stream) {
-  constexpr int KW = NT / 2 + 1;
-  auto kern = latent_attn_kernel<NT, KW, WIDE>;
-  const int tile = LAT_KT * p.CS * 2, limit = 226 * 1024;
-  const int exch = NT * 2048 + 512 > 32768 ? NT * 2048 + 512 : 32768;
-  p.stages = (limit - exch) / tile;
-  if (p.stages > LAT_MAX_STAGES) p.stages = LAT_MAX_STAGES;
-  if (p.stages < 2) return -14;
+// Rows of a unit, keys of a tile and stages of the ring for a batch and a row width.
+struct LatentShape { int rows, row_tiles, keys, stages, smem; };
+static LatentShape latent_shape(int max_q, int H, int CW, int RW) {
+  constexpr int limit = 224 * 1024;
+  LatentShape s;
+  s.rows = max_q * H > 16 ? 32 : 16;
+  s.row_tiles = (max_q * H + s.rows - 1) / s.rows;
+  const int nch = (CW + 63) / 64, nblk = (RW + 127) / 128, fixed = 1024 + nch * s.rows * 128 + 2 * s.rows * 128;
+  const int chunks = nch > 2 * nblk ? nch : 2 * nblk;
+  s.keys = fixed + 3 * chunks * 48 * 128 <= limit ? 48 : 32;
+  s.stages = (limit - fixed) / (chunks * s.keys * 128);
+  if (s.stages > LAT_MAX_STAGES) s.stages = LAT_MAX_STAGES;
+  s.smem = fixed + s.stages * chunks * s.keys * 128;
+  return s;
+}
+
+// qa [H][S][CW] as a 3-D map with boxes of 64 channels x 1 token x `heads` heads (heads past the end read as zero).
+static int latent_q_map(CUtensorMap* out, const void* qa, int H, long long S, int CW, int heads) {
+  EncodeTiledFnT fn = tma_encode_fn();
+  if (fn == nullptr) return -1;
+  if ((reinterpret_cast<uintptr_t>(qa) & 15) != 0 || CW % 8 != 0) return -2;
+  cuuint64_t dims[3] = {(cuuint64_t)CW, (cuuint64_t)S, (cuuint64_t)H};
+  cuuint64_t strides[2] = {(cuuint64_t)CW * 2, (cuuint64_t)S * CW * 2};
+  cuuint32_t box[3] = {64, 1, (cuuint32_t)heads};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(qa), dims, strides, box, estr,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
+}
+
+template <int NH, int KT>
+static int launch_latent(const LatentAttnParams& p, int smem, int ctas, cudaStream_t stream) {
+  auto kern = latent_attn_kernel<NH, KT>;
   static bool attr_dev[64] = {};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
   if (!attr_dev[dev]) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, limit) != cudaSuccess) return -10;
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 224 * 1024) != cudaSuccess) return -10;
     attr_dev[dev] = true;
   }
-  return launch_kernel(kern, dim3(ctas), dim3(LAT_THREADS), (size_t)(p.stages * tile + exch), stream, p) == cudaSuccess ? 0 : -11;
+  return launch_kernel(kern, dim3(ctas), dim3(LAT_THREADS), (size_t)smem, stream, p) == cudaSuccess ? 0 : -11;
 }
 
 }  // namespace rb
@@ -681,19 +751,19 @@ extern "C" void rb_latent_set_pdl(int on) { rb::pdl_enabled() = on != 0; }
 // dtype: 0 bf16, 1 fp32
 extern "C" int rb_latent_append(const float* proj, long long ldp, const float* qn_w, const float* kn_w, float eps,
                                 const int* positions, const int* slots, const float* table, int max_pos, int rot_pairs,
-                                void* cache, long long num_slots, int CS, int rot_off, void* cq, long long ldq, float* gate,
+                                void* cache, long long num_slots, int CW, int rot_off, void* cq, long long ldq, float* gate,
                                 int q_rank, int kv_rank, int rot_dim, int H, int T, int dtype, int* status, cudaStream_t stream) {
-  if (T <= 0 || rot_off < kv_rank || rot_off + rot_dim > CS || 2 * rot_pairs > rot_dim || ldq < q_rank) return -1;
+  if (T <= 0 || rot_off < kv_rank || rot_off + rot_dim > CW || 2 * rot_pairs > rot_dim || ldq < q_rank) return -1;
   if (ldp < (long long)q_rank + kv_rank + rot_dim + H) return -1;
   const int threads = q_rank + kv_rank <= 512 ? 128 : 256;
   cudaError_t e;
   if (dtype == 0)
     e = launch_kernel(latent_append_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, proj, ldp, qn_w, kn_w, eps, positions,
-                      slots, (const float2*)table, max_pos, rot_pairs, (__nv_bfloat16*)cache, num_slots, CS, rot_off,
+                      slots, (const float2*)table, max_pos, rot_pairs, (__nv_bfloat16*)cache, num_slots, CW, rot_off,
                       (__nv_bfloat16*)cq, ldq, gate, q_rank, kv_rank, rot_dim, H, status);
   else
     e = launch_kernel(latent_append_kernel<float>, dim3(T), dim3(threads), 0, stream, proj, ldp, qn_w, kn_w, eps, positions, slots,
-                      (const float2*)table, max_pos, rot_pairs, (float*)cache, num_slots, CS, rot_off, (float*)cq, ldq, gate,
+                      (const float2*)table, max_pos, rot_pairs, (float*)cache, num_slots, CW, rot_off, (float*)cq, ldq, gate,
                       q_rank, kv_rank, rot_dim, H, status);
   return e == cudaSuccess ? 0 : -11;
 }
@@ -715,53 +785,51 @@ extern "C" int rb_latent_query(void* q, const int* positions, const float* table
   return e == cudaSuccess ? 0 : -11;
 }
 
-// Rows of one unit and row tiles per sequence for batches whose longest sequence has max_q new rows.
-static int latent_rows(int max_q, int H) { return max_q * H > 16 ? 32 : 16; }
-extern "C" int rb_latent_units(int B, int H, int max_q) { return B * ((max_q * H + latent_rows(max_q, H) - 1) / latent_rows(max_q, H)); }
-extern "C" int rb_latent_ctas() { return latent_sms(); }
-
-// plan: [units + 1] ints (rb_latent_units).
-extern "C" int rb_latent_plan(const int* cu_q, const int* seq_lens, int B, int H, int max_q, int window, int* plan, cudaStream_t stream) {
+// plan: [B * row tiles + 1] ints; CW and RW as in rb_latent_attn.
+extern "C" int rb_latent_plan(const int* cu_q, const int* seq_lens, int B, int H, int max_q, int window, int CW, int RW, int* plan,
+                              cudaStream_t stream) {
   if (B <= 0 || H <= 0 || max_q <= 0 || window < 1) return -1;
-  const int rows = latent_rows(max_q, H);
-  return launch_kernel(latent_plan_kernel, dim3(1), dim3(1024), 0, stream, cu_q, seq_lens, B, H, rows, (max_q * H + rows - 1) / rows,
-                       window, plan) == cudaSuccess ? 0 : -11;
+  const LatentShape s = latent_shape(max_q, H, CW, RW);
+  return launch_kernel(latent_plan_kernel, dim3(1), dim3(1024), 0, stream, cu_q, seq_lens, B, H, s.rows, s.row_tiles, window, s.keys,
+                       plan) == cudaSuccess ? 0 : -11;
 }
 
 // T rows of B sequences (cu_q null: one row per sequence). max_q: most rows of any sequence. bf16: `plan` from rb_latent_plan
-// for the same batch; part_o [2 * ctas][rows of a unit][RW] and part_ml [.., 2] hold the pieces of cut units.
+// for the same batch; part_o [2 * CTAs][rows of a unit][RW] and part_ml [.., 2] hold the pieces of cut units.
 extern "C" int rb_latent_attn(const void* qa, const void* cache, const int* block_tables, const int* cu_q, const int* seq_lens,
                               const float* sink, const float* gate, void* out, const int* plan, float* part_o, float* part_ml,
-                              long long S, int H, int CW, int CS, int RW, int OW, int max_blocks, int num_blocks, int window,
+                              long long S, int H, int CW, int RW, int OW, int max_blocks, int num_blocks, int window,
                               float scale, int B, int T, int max_q, int dtype, int* status, cudaStream_t stream) {
-  if (T <= 0 || B <= 0 || H <= 0 || window < 1 || RW > OW || RW > CW || CW % 32 != 0 || CS < CW || max_q <= 0) return -1;
-  const int rows = latent_rows(max_q, H);
-  LatentAttnParams p = {qa, cache, block_tables, cu_q, seq_lens, sink, gate, out, plan, part_o, part_ml, S, B, H, CW, CS, RW, OW,
-                        (max_q * H + rows - 1) / rows, max_blocks, num_blocks, window, 2, scale, status};
+  if (T <= 0 || B <= 0 || H <= 0 || window < 1 || RW > OW || RW > CW || CW % 32 != 0 || max_q <= 0) return -1;
+  const LatentShape s = latent_shape(max_q, H, CW, RW);
+  LatentAttnParams p;
+  p.qa = qa; p.cache = cache; p.block_tables = block_tables; p.cu_q = cu_q; p.seq_lens = seq_lens; p.sink = sink; p.gate = gate;
+  p.out = out; p.plan = plan; p.part_o = part_o; p.part_ml = part_ml; p.S = S; p.B = B; p.H = H; p.CW = CW; p.RW = RW; p.OW = OW;
+  p.row_tiles = s.row_tiles; p.max_blocks = max_blocks; p.num_blocks = num_blocks; p.window = window; p.stages = s.stages;
+  p.scale = scale; p.status = status;
   if (dtype == 1) {
     if (CW > 32 * LAT_F32_MAX) return -1;
     return launch_kernel(latent_attn_f32_kernel, dim3((unsigned)(((long long)T * H + 3) / 4)), dim3(128), 0, stream, p, T, B) ==
                    cudaSuccess ? 0 : -11;
   }
-  if (plan == nullptr || part_o == nullptr || part_ml == nullptr || RW % 16 != 0 || OW % 8 != 0 || CS != CW + 8) return -1;
+  if (plan == nullptr || part_o == nullptr || part_ml == nullptr || RW % 16 != 0 || OW % 8 != 0 || RW > 1024 || s.stages < 2) return -1;
+  if (tma_map_2d_bf16(&p.map, cache, (unsigned long long)num_blocks * LAT_BLOCK, CW, CW, LAT_BLOCK) != 0) return -20;
+  p.q_tma = max_q == 1 ? 1 : 0;
+  if (p.q_tma && latent_q_map(&p.q_map, qa, H, S, CW, s.rows) != 0) return -21;
   const int ctas = latent_sms();
-  int rc = -1;
-#define LAT_GO(NT) rc = rows == 32 ? launch_latent<NT, true>(p, ctas, stream) : launch_latent<NT, false>(p, ctas, stream)
-  if (RW <= 128 && CW <= 192) LAT_GO(4);
-  else if (RW <= 256 && CW <= 320) LAT_GO(8);
-  else if (RW <= 512 && CW <= 576) LAT_GO(16);
-  else if (RW <= 1024 && CW <= 1088) LAT_GO(32);
-#undef LAT_GO
+  int rc;
+  if (s.keys == 48) rc = s.rows == 32 ? launch_latent<32, 48>(p, s.smem, ctas, stream) : launch_latent<16, 48>(p, s.smem, ctas, stream);
+  else rc = s.rows == 32 ? launch_latent<32, 32>(p, s.smem, ctas, stream) : launch_latent<16, 32>(p, s.smem, ctas, stream);
   if (rc != 0) return rc;
-  return launch_kernel(latent_merge_kernel, dim3(rows, ctas - 1), dim3(RW >= 256 ? 128 : 64), 0, stream, p, ctas, rows) == cudaSuccess
+  return launch_kernel(latent_merge_kernel, dim3(s.rows, ctas - 1), dim3(RW >= 256 ? 128 : 64), 0, stream, p, ctas, s.rows) == cudaSuccess
              ? 0 : -11;
 }
 
 extern "C" int rb_latent_gather(const void* cache, const int* block_tables, int bt_row0, int max_blocks, int num_blocks,
-                                const int* cu_k, const int* k_lo, int B, int n_rows, void* lat, void* rot, int CS, int RW, int RP,
+                                const int* cu_k, const int* k_lo, int B, int n_rows, void* lat, void* rot, int CW, int RW, int RP,
                                 int rot_off, int rot_cols, int* status, cudaStream_t stream) {
   if (n_rows <= 0 || B <= 0 || RW % 8 != 0 || RP % 8 != 0 || rot_off % 8 != 0) return -1;
   return launch_kernel(latent_gather_kernel, dim3((n_rows + 7) / 8), dim3(256), 0, stream, (const __nv_bfloat16*)cache, block_tables,
-                       bt_row0, max_blocks, num_blocks, cu_k, k_lo, B, (__nv_bfloat16*)lat, (__nv_bfloat16*)rot, CS, RW, RP, rot_off,
+                       bt_row0, max_blocks, num_blocks, cu_k, k_lo, B, (__nv_bfloat16*)lat, (__nv_bfloat16*)rot, CW, RW, RP, rot_off,
                        rot_cols, status) == cudaSuccess ? 0 : -11;
 }

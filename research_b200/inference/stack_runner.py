@@ -94,7 +94,7 @@ class StackRunner(RunnerBase):
 
     @staticmethod
     def cache_bytes_per_block(cfg: LayerStackConfig, tp_size: int, dtype: torch.dtype) -> int:
-        return sum(latent_geometry(x.mixer).cs for x in cfg.layers) * BLOCK * (4 if dtype == torch.float32 else 2)
+        return sum(latent_geometry(x.mixer).cw for x in cfg.layers) * BLOCK * (4 if dtype == torch.float32 else 2)
 
     # ------------------------------------------------------------------ memory
     def _alloc_weights(self) -> None:
@@ -131,7 +131,7 @@ class StackRunner(RunnerBase):
                 lw.ffp = _up(spec.mlp.ff, self.glu_bn // 2 if self.bf16 else 8)
                 lw.wgu, lw.wd = zeros(2 * lw.ffp, self.wp), zeros(self.wp, lw.ffp)
                 lw.norm2 = (zeros(d, dtype=f32), zeros(d, dtype=f32))
-            lw.cache = zeros(self.num_kv_blocks, BLOCK, g.cs)
+            lw.cache = zeros(self.num_kv_blocks, BLOCK, g.cw)
             self.layers.append(lw)
 
     def _alloc_activations(self) -> None:
@@ -149,8 +149,8 @@ class StackRunner(RunnerBase):
             if lw.geo not in self.bufs:
                 self.bufs[lw.geo] = GeometryBuffers(lw.geo, n, self.short_rows, dt, dev)
         self.attn_ws = ops.latent_workspace(list(self.bufs), dev) if self.bf16 else None
-        self.kinds = sorted({(lw.geo.heads, lw.spec.mixer.window) for lw in self.layers})    # layers that share an attention plan
-        self.decode_plans = {k: torch.zeros(ops.latent_units(self.max_batch, k[0], 1) + 1, dtype=torch.int32, device=dev) for k in self.kinds}
+        self.kinds = sorted({(lw.geo, lw.spec.mixer.window) for lw in self.layers}, key=repr)    # layers that share an attention plan
+        self.decode_plans = {k: torch.zeros(ops.latent_units(self.max_batch, k[0].heads, 1) + 1, dtype=torch.int32, device=dev) for k in self.kinds}
 
     # ------------------------------------------------------------------ weights
     def load_weights(self, weights: Mapping[str, torch.Tensor]) -> None:
@@ -251,14 +251,14 @@ class StackRunner(RunnerBase):
         if self.bf16:
             n = seq_lens.shape[0]
             if plans is None:
-                plans = {k: torch.empty(ops.latent_units(n, k[0], max_q) + 1, dtype=torch.int32, device=self.device) for k in self.kinds}
-            for (heads, window), plan in plans.items():
-                ops.latent_plan(cu_q, seq_lens, heads, max_q, window, plan)
+                plans = {k: torch.empty(ops.latent_units(n, k[0].heads, max_q) + 1, dtype=torch.int32, device=self.device) for k in self.kinds}
+            for (geo, window), plan in plans.items():
+                ops.latent_plan(cu_q, seq_lens, geo, max_q, window, plan)
 
         def attend(lw, b):
             m = lw.spec.mixer
             ops.latent_attention(b.qa, lw.cache, lw.geo, block_tables, cu_q, seq_lens, lw.sink, b.gate, b.ol, scale=m.scale, window=m.window,
-                                 rows=rows, max_q=max_q, plan=plans[(m.heads, m.window)] if self.bf16 else None, workspace=self.attn_ws)
+                                 rows=rows, max_q=max_q, plan=plans[(lw.geo, m.window)] if self.bf16 else None, workspace=self.attn_ws)
 
         return attend
 

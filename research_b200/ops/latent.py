@@ -60,12 +60,8 @@ class LatentGeometry:
         return _up(self.kv_rank, 16)
 
     @property
-    def cw(self) -> int:           # used channels of a cache row
+    def cw(self) -> int:           # cache row
         return _up(self.rw + _up(self.rot_dim, 16), 32)
-
-    @property
-    def cs(self) -> int:           # cache row stride: 8 channels apart, so that the attention kernel reads shared memory conflict-free
-        return self.cw + 8
 
     @property
     def qp(self) -> int:           # query latent
@@ -82,8 +78,8 @@ def _lib() -> ctypes.CDLL:
         lib.rb_latent_append.argtypes = ([c_vp, c_ll, c_vp, c_vp, c_float] + [c_vp] * 3 + [c_int, c_int, c_vp, c_ll, c_int, c_int, c_vp, c_ll, c_vp]
                                          + [c_int] * 6 + [c_vp, c_vp])
         lib.rb_latent_query.argtypes = [c_vp] * 3 + [c_int] * 3 + [c_vp, c_vp, c_ll] + [c_int] * 8 + [c_vp, c_vp]
-        lib.rb_latent_attn.argtypes = [c_vp] * 11 + [c_ll] + [c_int] * 8 + [c_float] + [c_int] * 4 + [c_vp, c_vp]
-        lib.rb_latent_plan.argtypes = [c_vp, c_vp] + [c_int] * 4 + [c_vp, c_vp]
+        lib.rb_latent_attn.argtypes = [c_vp] * 11 + [c_ll] + [c_int] * 7 + [c_float] + [c_int] * 4 + [c_vp, c_vp]
+        lib.rb_latent_plan.argtypes = [c_vp, c_vp] + [c_int] * 6 + [c_vp, c_vp]
         lib.rb_latent_gather.argtypes = [c_vp, c_vp] + [c_int] * 3 + [c_vp, c_vp, c_int, c_int, c_vp, c_vp] + [c_int] * 5 + [c_vp, c_vp]
         for f in ("rb_latent_append", "rb_latent_query", "rb_latent_attn", "rb_latent_plan", "rb_latent_gather"):
             getattr(lib, f).restype = c_int
@@ -114,13 +110,13 @@ def latent_append(proj, geo: LatentGeometry, q_norm, kv_norm, eps: float, positi
         gate[:T] = torch.sigmoid(proj[:, r0:r0 + geo.heads])
         ok = slots >= 0
         sl = slots[ok].long()
-        flat = cache.view(-1, geo.cs)[:, :geo.cw]
+        flat = cache.view(-1, geo.cw)
         flat[sl, :geo.kv_rank] = rms(proj[ok][:, q0:k0], kv_norm).to(cache.dtype)
         flat[sl, geo.rw:geo.rw + geo.rot_dim] = _rotate_half_pairs(proj[ok][:, k0:r0], table[positions[ok].long()]).to(cache.dtype)
         return
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and cache.is_contiguous() and gate.dtype == torch.float32
     rc = _lib().rb_latent_append(ptr(proj), proj.stride(0), ptr(q_norm), ptr(kv_norm), eps, ptr(positions), ptr(slots), ptr(table),
-                                 table.shape[0], geo.rot_pairs, ptr(cache), cache.shape[0] * LATENT_BLOCK, geo.cs, geo.rw, ptr(cq),
+                                 table.shape[0], geo.rot_pairs, ptr(cache), cache.shape[0] * LATENT_BLOCK, geo.cw, geo.rw, ptr(cq),
                                  cq.stride(0), ptr(gate), geo.q_rank, geo.kv_rank, geo.rot_dim, geo.heads, T, _DT[cq.dtype],
                                  ptr(status_tensor(proj.device)), stream_handle(proj.device))
     check_rc(rc, "rb_latent_append")
@@ -245,14 +241,14 @@ def latent_workspace(geos, device) -> torch.Tensor:
     return torch.empty(2 * sms * 32 * (max(g.rw for g in geos) + 2), dtype=torch.float32, device=device)
 
 
-def latent_plan(cu_q, seq_lens, heads: int, max_q: int, window: int, plan) -> None:
+def latent_plan(cu_q, seq_lens, geo: LatentGeometry, max_q: int, window: int, plan) -> None:
     """Prefix sums of the row tiles' key tiles -> ``plan [latent_units + 1]`` (int32): how ``latent_attention`` shares its
-    work. One per batch, window and head count; the CPU twin needs none."""
+    work. One per batch, window and geometry; the CPU twin needs none."""
     if not seq_lens.is_cuda:
         return
     B = seq_lens.shape[0]
-    assert plan.dtype == torch.int32 and plan.numel() >= latent_units(B, heads, max_q) + 1
-    check_rc(_lib().rb_latent_plan(ptr(cu_q), ptr(seq_lens), B, heads, max_q, window, ptr(plan), stream_handle(seq_lens.device)), "rb_latent_plan")
+    assert plan.dtype == torch.int32 and plan.numel() >= latent_units(B, geo.heads, max_q) + 1
+    check_rc(_lib().rb_latent_plan(ptr(cu_q), ptr(seq_lens), B, geo.heads, max_q, window, geo.cw, geo.rw, ptr(plan), stream_handle(seq_lens.device)), "rb_latent_plan")
 
 
 def latent_attention(qa, cache, geo: LatentGeometry, block_tables, cu_q, seq_lens, sink, gate, out, *, scale: float, window: int,
@@ -265,7 +261,7 @@ def latent_attention(qa, cache, geo: LatentGeometry, block_tables, cu_q, seq_len
     B = seq_lens.shape[0]
     H, S = qa.shape[0], qa.shape[1]
     if not qa.is_cuda:
-        flat = cache.view(-1, geo.cs)[:, :geo.cw]
+        flat = cache.view(-1, geo.cw)
         for b in range(B):
             t0, t1 = (b, b + 1) if cu_q is None else (int(cu_q[b]), int(cu_q[b + 1]))
             L = int(seq_lens[b])
@@ -289,7 +285,7 @@ def latent_attention(qa, cache, geo: LatentGeometry, block_tables, cu_q, seq_len
         part_ml = workspace[n:]
     assert qa.is_contiguous() and out.is_contiguous() and cache.is_contiguous() and sink.dtype == gate.dtype == torch.float32
     rc = _lib().rb_latent_attn(ptr(qa), ptr(cache), ptr(block_tables), ptr(cu_q), ptr(seq_lens), ptr(sink), ptr(gate), ptr(out), ptr(plan),
-                               ptr(workspace), ptr(part_ml), S, H, geo.cw, geo.cs, geo.rw, out.shape[2], block_tables.stride(0),
+                               ptr(workspace), ptr(part_ml), S, H, geo.cw, geo.rw, out.shape[2], block_tables.stride(0),
                                cache.shape[0], window, scale, B, rows, max_q, dt, ptr(status_tensor(qa.device)), stream_handle(qa.device))
     check_rc(rc, "rb_latent_attn", 2 if dt == 0 else 1)
 
@@ -299,7 +295,7 @@ def latent_gather(cache, geo: LatentGeometry, block_tables, bt_row0: int, cu_k, 
     latents -> ``lat [n, rw]``, rotated parts -> ``rot [n, rp]``."""
     B = k_lo.shape[0]
     if not cache.is_cuda:
-        flat = cache.view(-1, geo.cs)[:, :geo.cw]
+        flat = cache.view(-1, geo.cw)
         for b in range(B):
             s, e = int(cu_k[b]), int(cu_k[b + 1])
             key = torch.arange(e - s) + int(k_lo[b])
@@ -309,6 +305,6 @@ def latent_gather(cache, geo: LatentGeometry, block_tables, bt_row0: int, cu_k, 
             rot[s:e, :geo.rot_dim] = rows[:, geo.rw:geo.rw + geo.rot_dim]
         return
     rc = _lib().rb_latent_gather(ptr(cache), ptr(block_tables), bt_row0, block_tables.stride(0), cache.shape[0], ptr(cu_k), ptr(k_lo), B,
-                                 n_rows, ptr(lat), ptr(rot), geo.cs, geo.rw, geo.rp, geo.rw, _up(geo.rot_dim, 16),
+                                 n_rows, ptr(lat), ptr(rot), geo.cw, geo.rw, geo.rp, geo.rw, _up(geo.rot_dim, 16),
                                  ptr(status_tensor(cache.device)), stream_handle(cache.device))
     check_rc(rc, "rb_latent_gather")

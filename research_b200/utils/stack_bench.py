@@ -154,8 +154,8 @@ def stack_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> d
     if decode:
         bt, lens = r.bt_dev[:T], r.d_lens[:T]
         span = min(context, m.window)
-        plan = r.decode_plans[(H, m.window)]
-        ops.latent_plan(None, lens, H, 1, m.window, plan)
+        plan = r.decode_plans[(g, m.window)]
+        ops.latent_plan(None, lens, g, 1, m.window, plan)
         t.add("absorb W_uk", lambda: ops.head_gemm_absorb(b.qn, lw.wuk, b.qa, T), 2 * H * (g.dp * g.rw + T * (g.dp + g.rw)), 2.0 * T * H * g.dp * g.rw)
         t.add("attention", lambda: ops.latent_attention(b.qa, lw.cache, g, bt, None, lens, lw.sink, b.gate, b.ol, scale=m.scale, window=m.window,
                                                         rows=T, max_q=1, plan=plan, workspace=r.attn_ws),

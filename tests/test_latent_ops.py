@@ -88,17 +88,17 @@ def test_append_query_and_head_products(place, geo):
     table = ops.rope_table(1024, 2 * geo.rot_pairs, base, exact=True)
     proj = rand(T, geo.proj, seed=20)
     qn_w, kn_w = 1 + 0.3 * rand(geo.q_rank, seed=21), 1 + 0.3 * rand(geo.kv_rank, seed=22)
-    cache = torch.zeros(4, 16, geo.cs, dtype=dt, device=dev)
+    cache = torch.zeros(4, 16, geo.cw, dtype=dt, device=dev)
     cq, gate = torch.zeros(T, geo.qp, dtype=dt, device=dev), torch.zeros(T, H, device=dev)
     ops.latent_append(proj.to(dev), geo, qn_w.to(dev), kn_w.to(dev), eps, pos.to(dev), slots.to(dev), table.to(dev), cache, cq, gate)
     p = proj.double()
     close(cq[:, :q0], oracle.rms(p[:, :q0], qn_w.double(), eps), dt, "query latent")
     close(gate, torch.sigmoid(p[:, r0:r0 + H]), torch.float32, "gate")
-    want = torch.zeros(64, geo.cs, dtype=torch.float64)
+    want = torch.zeros(64, geo.cw, dtype=torch.float64)
     ok = slots >= 0
     want[slots[ok].long(), :geo.kv_rank] = oracle.rms(p[ok][:, q0:k0], kn_w.double(), eps)
     want[slots[ok].long(), geo.rw:geo.rw + geo.rot_dim] = oracle.rotate(p[ok][:, k0:r0], pos[ok], 2 * geo.rot_pairs, base)
-    close(cache.view(64, geo.cs), want, dt, "cache rows")
+    close(cache.view(64, geo.cw), want, dt, "cache rows")
 
     q = rand(T, H, geo.dp + geo.rp, seed=23).to(dt)
     turned = oracle.rotate(q[..., geo.dp:geo.dp + geo.rot_dim].double(), pos, 2 * geo.rot_pairs, base)
@@ -151,7 +151,7 @@ def test_attention_on_cached_latents(place, geo, decode):
     new = [1] * 7 if decode else [1, 5, 16, 2, 13, 1, 3]
     T, scale = sum(new), 1.0 / math.sqrt(geo.cw)
     blocks = torch.randperm(64, generator=torch.Generator().manual_seed(1)).int()
-    cache = torch.zeros(64, 16, geo.cs)
+    cache = torch.zeros(64, 16, geo.cw)
     bt, at = torch.zeros(len(lens), 24, dtype=torch.int32), 0
     qa = torch.zeros(H, S, geo.cw)
     sink, gate = rand(H, seed=3) + 1, torch.sigmoid(rand(T, H, seed=4))
@@ -172,7 +172,7 @@ def test_attention_on_cached_latents(place, geo, decode):
         nb = -(-L // 16)
         bt[b, :nb] = blocks[at:at + nb]
         at += nb
-        flat = cache.view(-1, geo.cs)
+        flat = cache.view(-1, geo.cw)
         for k in range(L):
             flat[int(bt[b, k // 16]) * 16 + k % 16, :geo.cw] = keys[k].float()
         rows.append(plain_attention(q.double(), keys.double(), keys[:, :geo.rw].double(), n, window, scale, sink.double(), gate[t0:t0 + n].double()))
@@ -184,7 +184,7 @@ def test_attention_on_cached_latents(place, geo, decode):
     plan = ws = None
     if dev == "cuda" and dt == torch.bfloat16:
         plan = torch.zeros(ops.latent_units(len(lens), H, max(new)) + 1, dtype=torch.int32, device=dev)
-        ops.latent_plan(cu, sl, H, max(new), window, plan)
+        ops.latent_plan(cu, sl, geo, max(new), window, plan)
         ws = ops.latent_workspace([geo], dev)
     ops.latent_attention(qa.to(dt).to(dev), cache.to(dt).to(dev), geo, bt.to(dev), cu, sl, sink.to(dev), gate.to(dev), out, scale=scale,
                          window=window, rows=T, max_q=max(new), plan=plan, workspace=ws)
@@ -203,14 +203,13 @@ def test_attention_shares_cut_anywhere(cuda_device):
         lens[0] = longest
         nb = -(-longest // 16)
         bt = torch.randperm(B * nb, generator=g).int().view(B, nb)
-        cache = rand(B * nb, 16, geo.cs, seed=seed, dtype=dt)
-        cache[..., geo.cw:] = float("nan")                   # the gap between rows is never read as data
+        cache = rand(B * nb, 16, geo.cw, seed=seed, dtype=dt)
         cache[..., geo.kv_rank:geo.rw] = 0
         cache[..., geo.rw + geo.rot_dim:geo.cw] = 0
         qa, sink, gate = rand(geo.heads, B, geo.cw, seed=seed + 9, dtype=dt), rand(geo.heads, seed=1), torch.sigmoid(rand(B, geo.heads, seed=2))
         plan = torch.zeros(B + 1, dtype=torch.int32, device=cuda_device)
         sl = lens.to(cuda_device)
-        ops.latent_plan(None, sl, geo.heads, 1, window, plan)
+        ops.latent_plan(None, sl, geo, 1, window, plan)
         out = torch.zeros(geo.heads, B, geo.rw, dtype=dt, device=cuda_device)
         ops.latent_attention(qa.to(cuda_device), cache.to(cuda_device), geo, bt.to(cuda_device), None, sl, sink.to(cuda_device),
                              gate.to(cuda_device), out, scale=0.1, window=window, rows=B, max_q=1, plan=plan, workspace=ws)
@@ -219,7 +218,7 @@ def test_attention_shares_cut_anywhere(cuda_device):
             if L == 0:
                 continue
             k = torch.arange(L)
-            keys = cache.view(-1, geo.cs)[bt[b, k // 16].long() * 16 + k % 16, :geo.cw].double()
+            keys = cache.view(-1, geo.cw)[bt[b, k // 16].long() * 16 + k % 16, :geo.cw].double()
             want = plain_attention(qa[:, b][None].double(), keys, keys[:, :geo.rw], 1, window, 0.1, sink.double(), gate[b:b + 1].double())
             close(out[:, b], want[0], dt, (B, b, L))
 
@@ -244,10 +243,10 @@ def test_expanded_attention_and_gather(place, geo, window):
     q[..., :geo.dim], q[..., geo.dp:geo.dp + geo.rot_dim] = rand(T, H, geo.dim, seed=3), rand(T, H, geo.rot_dim, seed=4)
     q = q.to(dt)
     sink, gate = rand(H, seed=5) * 2, torch.sigmoid(rand(T, H, seed=6))
-    cache, bt, at, rows = torch.zeros(160, 16, geo.cs), torch.zeros(4, 48, dtype=torch.int32), 0, []
+    cache, bt, at, rows = torch.zeros(160, 16, geo.cw), torch.zeros(4, 48, dtype=torch.int32), 0, []
     perm = torch.randperm(160, generator=torch.Generator().manual_seed(7)).int()
     for b, L in enumerate(lens):
-        c = torch.zeros(L, geo.cs)
+        c = torch.zeros(L, geo.cw)
         c[:, :geo.kv_rank], c[:, geo.rw:geo.rw + geo.rot_dim] = rand(L, geo.kv_rank, seed=20 + b), rand(L, geo.rot_dim, seed=40 + b)
         t_last, pos = new[b] - 1, L - 1
         for h, k in enumerate((pos - window + 1, pos - window, pos - 128, 0)):      # planted in the rotated part, which needs no product
@@ -259,7 +258,7 @@ def test_expanded_attention_and_gather(place, geo, window):
         bt[b, :nb] = perm[at:at + nb]
         at += nb
         k = torch.arange(L)
-        cache.view(-1, geo.cs)[bt[b, k // 16].long() * 16 + k % 16] = c.float()
+        cache.view(-1, geo.cw)[bt[b, k // 16].long() * 16 + k % 16] = c.float()
         rw = lambda w: torch.einsum("kr,hdr->khd", c[:, :geo.rw].double(), w.double().view(H, -1, geo.rw)).to(dt).double()   # noqa: E731
         rot = torch.zeros(L, geo.rp, dtype=torch.float64)
         rot[:, :geo.rot_dim] = c[:, geo.rw:geo.rw + geo.rot_dim].double()
