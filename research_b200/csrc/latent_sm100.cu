@@ -166,7 +166,7 @@ struct LatentAttnParams {
   const float* gate;       // [T, H]
   void* out;               // [H][S][OW] gate * sum_j p_j c_j
   const int* plan;         // [B * row_tiles + 1] prefix sums of the units' tiles
-  float* part_o;           // [2 * grid][rows][RW]
+  float* part_o;           // [2 * grid][RW][rows]
   float* part_ml;          // [2 * grid][rows][2]
   long long S;
   int B, H, CW, RW, OW, row_tiles;       // RW: latent columns (a multiple of 16) that are summed
@@ -242,6 +242,17 @@ __device__ __forceinline__ int latent_find_cta(const int* __restrict__ plan, int
 }
 __device__ __forceinline__ int latent_share(int total, int ctas) { return max((total + ctas - 1) / ctas, LAT_MIN_TILES); }
 
+__device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {     // one look, never waits
+  uint32_t done;
+  asm volatile(
+      "{\n\t.reg .pred P;\n\t"
+      "mbarrier.test_wait.parity.shared::cta.b64 P, [%1], %2;\n\t"
+      "selp.u32 %0, 1, 0, P;\n\t}"
+      : "=r"(done)
+      : "r"(bar), "r"(parity)
+      : "memory");
+  return done != 0;
+}
 __device__ __forceinline__ float lat_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -253,12 +264,13 @@ template <int NH, int KT>
 __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __grid_constant__ LatentAttnParams p) {
   constexpr int CHUNK = KT * 128;                // bytes of 64 channels of a tile
   constexpr int PAGES = KT / LAT_BLOCK;
-  constexpr uint32_t O_COL = 128;                // TMEM: S at columns 0 and 64, O^T behind
+  constexpr int SB = 3;                          // score, weight and alpha buffers
+  constexpr uint32_t O_COL = SB * 64;            // TMEM: S at columns 0, 64, 128, O^T behind
   extern __shared__ __align__(128) uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t kv_full[LAT_MAX_STAGES], kv_empty[LAT_MAX_STAGES];
-  __shared__ __align__(8) uint64_t q_full, q_empty, s_full[2], a_full[2], p_full[2], o_done, o_free;
-  __shared__ float s_alpha[2][NH], s_scale[NH];
-  __shared__ int s_flag[2];
+  __shared__ __align__(8) uint64_t q_full, q_empty, s_full[SB], p_full[SB], o_done, o_free, cmd, cmd_done;
+  __shared__ float s_alpha[NH], s_scale[NH];
+  __shared__ int s_tile;
   __shared__ long long s_row[NH];
   __shared__ uint32_t tmem_base_smem;
   __shared__ int abort_flag, u_shared;
@@ -274,7 +286,7 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
 
   const uint32_t q_s = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* q_ptr = smem_raw + (q_s - smem_u32(smem_raw));
-  const uint32_t p_s = q_s + nch * NH * 128, kv_s = p_s + 2 * NH * 128;
+  const uint32_t p_s = q_s + nch * NH * 128, kv_s = p_s + SB * NH * 128;
   uint8_t* p_ptr = q_ptr + nch * NH * 128;
   if (threadIdx.x == 0) {
     abort_flag = 0;
@@ -284,16 +296,17 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
     }
     mbar_init(smem_u32(&q_full), p.q_tma ? 1 : 2);
     mbar_init(smem_u32(&q_empty), 1);
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < SB; ++i) {
       mbar_init(smem_u32(&s_full[i]), 1);
-      mbar_init(smem_u32(&a_full[i]), 1);
-      mbar_init(smem_u32(&p_full[i]), 4);
+      mbar_init(smem_u32(&p_full[i]), 1);
     }
     mbar_init(smem_u32(&o_done), 1);
     mbar_init(smem_u32(&o_free), 4);
+    mbar_init(smem_u32(&cmd), 1);
+    mbar_init(smem_u32(&cmd_done), 3);
     fence_mbar_init();
   }
-  const uint32_t tmem_cols = O_COL + nblk * NH <= 256 ? 256 : 512;
+  const uint32_t tmem_cols = O_COL + (nblk * NH + 31) / 32 * 32 <= 256 ? 256 : 512;
   if (warp == 1) {
     tmem_alloc(smem_u32(&tmem_base_smem), tmem_cols);
     tmem_relinquish();
@@ -349,10 +362,18 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
       const int n = t_end - t_begin, ksteps = p.CW / 16;
       int uq = 0, u_s = u_first, u_o = u_first;      // units started by the scores / being summed
       uint32_t o_units = 0;
+      auto new_unit = [&](int t) {                   // moves u_s to the unit of tile t
+        while (p.plan[u_s + 1] <= t) ++u_s;
+        return t == t_begin || t == p.plan[u_s];
+      };
+      // the operands of tile j's scores are in shared memory
+      auto s_ready = [&](int j) {
+        if (new_unit(t_begin + j) && !mbar_test(smem_u32(&q_full), (uint32_t)uq & 1u)) return false;
+        return mbar_test(smem_u32(&kv_full[j % p.stages]), (j / p.stages) & 1u);
+      };
       auto issue_s = [&](int j) {
         const int t = t_begin + j;
-        while (p.plan[u_s + 1] <= t) ++u_s;
-        if (t == t_begin || t == p.plan[u_s])       // a new unit: its queries
+        if (new_unit(t))                             // its queries
           mbar_wait_bounded(smem_u32(&q_full), (uint32_t)(uq++) & 1u, abortp, p.status, ST_TIMEOUT_SMEM_FULL);
         const uint32_t s = j % p.stages;
         mbar_wait_bounded(smem_u32(&kv_full[s]), (j / p.stages) & 1u, abortp, p.status, ST_TIMEOUT_SMEM_FULL);
@@ -360,7 +381,7 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
         const uint32_t tile = kv_s + s * tile_bytes;
         // descriptors advance by plain additions (addresses in 16-byte units): one thread issues all of this
         uint64_t ad = make_smem_desc_sw128(q_s, 16, 1024), bd = make_smem_desc_sw128(tile, 16, 1024);
-        const uint32_t d = tmem_base + (j & 1) * 64;
+        const uint32_t d = tmem_base + (j % SB) * 64;
         umma_bf16(d, ad, bd, idesc_s, 0u);
         umma_bf16(d, ad + 2, bd + 2, idesc_s, 1u);
         if (ksteps > 2) {
@@ -378,22 +399,35 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
             umma_bf16(d, ad + 6, bd + 6, idesc_s, 1u);
           }
         }
-        umma_commit(smem_u32(&s_full[j & 1]));
+        umma_commit(smem_u32(&s_full[j % SB]));
         if (t + 1 == t_end || t + 1 == p.plan[u_s + 1]) umma_commit(smem_u32(&q_empty));   // the unit's last scores
       };
-      issue_s(0);
+      const int ahead = min(SB - 1, p.stages - 1);   // scores of later tiles overlap this tile's softmax, as far as stages allow
+      int js = 0;
       for (int j = 0; j < n; ++j) {
         const int t = t_begin + j;
         while (p.plan[u_o + 1] <= t) ++u_o;
-        const bool first = t == t_begin || t == p.plan[u_o], last = t + 1 == p.plan[u_o + 1];
-        if (j + 1 < n && !last) issue_s(j + 1);     // the next tile's scores overlap this tile's softmax
-        mbar_wait_bounded(smem_u32(&p_full[j & 1]), (j >> 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+        const bool first = t == t_begin || t == p.plan[u_o];
+        if (js == j) issue_s(js++);
+        const uint32_t pb = smem_u32(&p_full[j % SB]), pph = (j / SB) & 1u;
+        const uint64_t c0 = globaltimer_ns();
+        for (uint32_t spins = 0; !mbar_test(pb, pph);) {
+          if (js < n && js <= j + ahead && s_ready(js)) { issue_s(js++); continue; }
+          if ((++spins & 0x3f) == 0) {
+            if (*abortp != 0) break;
+            if (globaltimer_ns() - c0 > RB_WAIT_BUDGET_NS) {
+              *abortp = 1;
+              set_status(p.status, ST_TIMEOUT_TMEM_FULL);
+              break;
+            }
+          }
+        }
         if (first && o_units++ > 0)                 // the previous unit's sums have left TMEM
           mbar_wait_bounded(smem_u32(&o_free), (o_units - 2) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_EMPTY);
         tc_fence_after();
         const uint32_t s = j % p.stages, tile = kv_s + s * tile_bytes;
         uint64_t ad = make_smem_desc_sw128(tile, CHUNK, 1024);
-        const uint64_t bd = make_smem_desc_sw128(p_s + (j & 1) * (NH * 128), 16, 1024);
+        const uint64_t bd = make_smem_desc_sw128(p_s + (j % SB) * (NH * 128), 16, 1024);
 #pragma unroll 2
         for (int m = 0; m < nblk; ++m, ad += (2 * CHUNK) >> 4)
 #pragma unroll
@@ -401,7 +435,6 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
             umma_bf16(tmem_o + m * NH, ad + k * (2048 >> 4), bd + 2 * k, idesc_o, (!first || k > 0) ? 1u : 0u);
         umma_commit(smem_u32(&kv_empty[s]));
         umma_commit(smem_u32(&o_done));
-        if (j + 1 < n && last) issue_s(j + 1);
       }
       // nothing of this CTA is in flight when it frees its TMEM
       mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(n - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
@@ -442,9 +475,29 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
     }
   } else {
     // ---------------------------------------------------------------- softmax (warp 4), O^T (warps 4-7)
+    // Warp 4 works alone from tile to tile. It calls the other three through `cmd` when O^T has to be rescaled (s_tile = the
+    // tile) and when a piece is complete (s_tile = -1).
     const int qd = warp - 4;
     const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
     const float log2e = 1.4426950408889634f, scale_log2 = p.scale * log2e;
+    auto rescale = [&](int j) {                     // O^T holds the tiles before tile j
+      mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      __syncwarp();
+      tc_fence_after();
+#pragma unroll 1
+      for (int c = 0; c < nblk * NH; c += 32) {
+        uint32_t o[32];
+        tmem_ld_32x32(tmem_o + lane_addr + c, o);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[i & (NH - 1)]);
+        tmem_st_32x32(tmem_o + lane_addr + c, o);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+    };
+    uint32_t n_cmd = 0, n_rescale = 0;
     int j = 0;
     for (int u = u_first, t = t_begin; t < t_end; ++u) {
       const int u_begin = p.plan[u], u_stop = p.plan[u + 1], u_end = min(u_stop, t_end);
@@ -452,22 +505,22 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
       const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, NH, p.H, p.window);
       const bool has_first = t == u_begin, whole = has_first && u_end == u_stop, row_ok = lane < w.n_rows;
       const int tok = (w.r0 + (row_ok ? lane : 0)) / p.H, head = (w.r0 + (row_ok ? lane : 0)) - tok * p.H;
-      const int pos = w.L - w.q_len + tok;
-      const int pos_min = w.L - w.q_len + w.r0 / p.H, pos_max = w.L - w.q_len + (w.r0 + w.n_rows - 1) / p.H;
-      float m_used = -INFINITY, l = 0.f;
-      const int t_piece = t;
-      for (int k0 = w.lo + (t - u_begin) * KT; t < u_end; ++t, k0 += KT, ++j) {
-        const int b = j & 1;
-        const uint32_t ph = (j >> 1) & 1u;
-        if (qd == 0) {
-          mbar_wait_bounded(smem_u32(&s_full[b]), ph, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      float m_used = -INFINITY, l = 0.f, sink = 0.f, gate = 0.f;
+      if (qd == 0) {
+        sink = p.sink[head] * log2e;
+        gate = p.gate[(long long)(w.t0 + tok) * p.H + head];
+        const int pos = w.L - w.q_len + tok;
+        const int pos_min = w.L - w.q_len + w.r0 / p.H, pos_max = w.L - w.q_len + (w.r0 + w.n_rows - 1) / p.H;
+        const int t_piece = t;
+        for (int k0 = w.lo + (t - u_begin) * KT; t < u_end; ++t, k0 += KT, ++j) {
+          const int b = j % SB;
+          mbar_wait_bounded(smem_u32(&s_full[b]), (j / SB) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
           __syncwarp();
           tc_fence_after();
           uint32_t v[KT];
           tmem_ld_32x32(tmem_base + b * 64, *reinterpret_cast<uint32_t(*)[32]>(&v[0]));
           if constexpr (KT == 48) tmem_ld_32x16(tmem_base + b * 64 + 32, *reinterpret_cast<uint32_t(*)[16]>(&v[32]));
           tmem_ld_wait();
-          tc_fence_before();
           if (k0 + KT - 1 > pos_min || k0 <= pos_max - p.window) {
 #pragma unroll
             for (int i = 0; i < KT; ++i)
@@ -478,11 +531,18 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
           for (int i = 0; i < KT; ++i) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(v[i]));
           const float m_new = fmaxf(m_used, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale_log2);
           const bool need = row_ok && (m_new > m_used + LAT_RESCALE || (m_used == -INFINITY && m_new != -INFINITY));
-          const float alpha = need && m_used != -INFINITY ? lat_exp2(m_used - m_new) : 1.f;
-          const int any = __any_sync(0xffffffffu, need && t > t_piece);
-          if (need) { m_used = m_new; l *= alpha; }
-          if (lane < NH) s_alpha[b][lane] = alpha;
-          if (lane == 0) s_flag[b] = any;
+          const bool any = __any_sync(0xffffffffu, need && t > t_piece);
+          if (any && lane < NH) s_alpha[lane] = need && m_used != -INFINITY ? lat_exp2(m_used - m_new) : 1.f;
+          if (need) {
+            l *= m_used != -INFINITY ? lat_exp2(m_used - m_new) : 1.f;
+            m_used = m_new;
+          }
+          if (any) {
+            if (lane == 0) s_tile = j;
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(&cmd));
+            rescale(j);
+          }
           const float mref = m_used == -INFINITY ? 0.f : m_used;
           float ls[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -497,56 +557,57 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
 #pragma unroll
             for (int i = 0; i < KT / 8; ++i) {
               uint4 o;
-              o.x = row_ok ? pack_bf16x2(__uint_as_float(v[i * 8]), __uint_as_float(v[i * 8 + 1])) : 0u;
-              o.y = row_ok ? pack_bf16x2(__uint_as_float(v[i * 8 + 2]), __uint_as_float(v[i * 8 + 3])) : 0u;
-              o.z = row_ok ? pack_bf16x2(__uint_as_float(v[i * 8 + 4]), __uint_as_float(v[i * 8 + 5])) : 0u;
-              o.w = row_ok ? pack_bf16x2(__uint_as_float(v[i * 8 + 6]), __uint_as_float(v[i * 8 + 7])) : 0u;
+              o.x = pack_bf16x2(__uint_as_float(v[i * 8]), __uint_as_float(v[i * 8 + 1]));
+              o.y = pack_bf16x2(__uint_as_float(v[i * 8 + 2]), __uint_as_float(v[i * 8 + 3]));
+              o.z = pack_bf16x2(__uint_as_float(v[i * 8 + 4]), __uint_as_float(v[i * 8 + 5]));
+              o.w = pack_bf16x2(__uint_as_float(v[i * 8 + 6]), __uint_as_float(v[i * 8 + 7]));
+              if (!row_ok) o = make_uint4(0, 0, 0, 0);
               *reinterpret_cast<uint4*>(prow + ((i ^ (lane & 7)) << 4)) = o;
             }
           }
           fence_proxy_async_smem();
-          __syncwarp();
-          if (lane == 0) mbar_arrive(smem_u32(&a_full[b]));
-        } else {
-          mbar_wait_bounded(smem_u32(&a_full[b]), ph, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
-          __syncwarp();
-        }
-        if (*(volatile int*)&s_flag[b]) {          // O^T holds the tiles before this one
-          mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
-          __syncwarp();
-          tc_fence_after();
-#pragma unroll 1
-          for (int c = 0; c < nblk * NH; c += 32) {
-            uint32_t o[32];
-            tmem_ld_32x32(tmem_o + lane_addr + c, o);
-            tmem_ld_wait();
-#pragma unroll
-            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[b][i & (NH - 1)]);
-            tmem_st_32x32(tmem_o + lane_addr + c, o);
-          }
-          tmem_st_wait();
           tc_fence_before();
+          if (any) {                                // the other quarters of O^T are rescaled too
+            mbar_wait_bounded(smem_u32(&cmd_done), n_rescale & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+            ++n_rescale;
+          }
+          __syncwarp();
+          if (lane == 0) mbar_arrive(smem_u32(&p_full[b]));
         }
-        __syncwarp();
-        if (lane == 0) mbar_arrive(smem_u32(&p_full[b]));
+      } else {
+        j += u_end - t;
+        t = u_end;
+        while (true) {
+          mbar_wait_bounded(smem_u32(&cmd), n_cmd & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+          ++n_cmd;
+          __syncwarp();
+          const int tile = *(volatile int*)&s_tile;
+          if (tile < 0 || *abortp != 0) break;
+          rescale(tile);
+          if (lane == 0) mbar_arrive(smem_u32(&cmd_done));
+        }
       }
       // ---- the piece is complete ----
       const long long slot = 2ll * blockIdx.x + (u_begin > t_begin ? 1 : 0);
       if (qd == 0 && lane < NH) {
         float m = m_used, f = 1.f;
         if (has_first) {                            // the sink: in the denominator once, no value
-          const float sk = p.sink[head] * log2e;
-          m = fmaxf(m_used, sk);
+          m = fmaxf(m_used, sink);
           f = lat_exp2(m_used - m);
-          l = l * f + lat_exp2(sk - m);
+          l = l * f + lat_exp2(sink - m);
         }
-        if (whole) f = l > 0.f ? f * p.gate[(long long)(w.t0 + tok) * p.H + head] / l : 0.f;
+        if (whole) f = l > 0.f ? f * gate / l : 0.f;
         s_scale[lane] = f;
-        s_row[lane] = whole ? ((long long)head * p.S + w.t0 + tok) * p.OW : (slot * NH + lane) * p.RW;
+        s_row[lane] = ((long long)head * p.S + w.t0 + tok) * p.OW;
         if (!whole && row_ok) {
           p.part_ml[(slot * NH + lane) * 2] = m;
           p.part_ml[(slot * NH + lane) * 2 + 1] = l;
         }
+      }
+      if (qd == 0) {
+        if (lane == 0) s_tile = -1;
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&cmd));
       }
       mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
       lat_bar(1, 128);
@@ -556,13 +617,27 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
         uint32_t o[32];
         tmem_ld_32x32(tmem_o + lane_addr + c, o);
         tmem_ld_wait();
+        if (whole) {
+          // a lane holds one channel of 32 rows; neighbours trade, so that each stores two channels of every other row
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          const int r = i & (NH - 1), ch = (c + i) / NH * 128 + qd * 32 + lane;
-          if (r < w.n_rows && ch < p.RW) {
-            const float x = __uint_as_float(o[i]) * s_scale[r];
-            if (whole) reinterpret_cast<__nv_bfloat16*>(p.out)[s_row[r] + ch] = __float2bfloat16_rn(x);
-            else p.part_o[s_row[r] + ch] = x;
+          for (int i = 0; i < 32; i += 2) {
+            const int r = i & (NH - 1), ch = (c + i) / NH * 128 + qd * 32 + (lane & ~1);
+            const float x = __uint_as_float(o[i]) * s_scale[r], y = __uint_as_float(o[i + 1]) * s_scale[r + 1];
+            const float got = __shfl_xor_sync(0xffffffffu, (lane & 1) ? x : y, 1);
+            const int row = r + (lane & 1);
+            if (row < w.n_rows && ch < p.RW)
+              *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + s_row[row] + ch) =
+                  (lane & 1) ? pack_bf16x2(got, y) : pack_bf16x2(x, got);
+          }
+        } else {
+          // pieces are kept transposed, [channel][row]: contiguous for a lane
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) {
+            const int r = i & (NH - 1), ch = (c + i) / NH * 128 + qd * 32 + lane;
+            if (ch < p.RW)
+              *reinterpret_cast<float4*>(p.part_o + (slot * p.RW + ch) * NH + r) =
+                  make_float4(__uint_as_float(o[i]) * s_scale[r], __uint_as_float(o[i + 1]) * s_scale[r + 1],
+                              __uint_as_float(o[i + 2]) * s_scale[r + 2], __uint_as_float(o[i + 3]) * s_scale[r + 3]);
           }
         }
       }
@@ -578,38 +653,58 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
   }
 }
 
-// Combine the pieces of units that a CTA boundary cuts: CTA (row, boundary), for the first boundary inside each such unit.
-__global__ void latent_merge_kernel(const LatentAttnParams p, int ctas, int rows) {
+// Combine the pieces of units that a CTA boundary cuts: blockIdx.x is the boundary (the first one inside such a unit acts),
+// blockIdx.y a range of 128 channels. The pieces' weights are worked out once per row; almost always there are two pieces.
+constexpr int LAT_MERGE_MAX = 160;               // pieces of one unit: at most one per CTA
+__global__ void __launch_bounds__(256) latent_merge_kernel(const LatentAttnParams p, int ctas, int rows) {
+  __shared__ int u_shared;
+  __shared__ float wgt[LAT_MERGE_MAX][32];
+  __shared__ long long dst[32];
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ int u_shared;
   const int units = p.B * p.row_tiles, total = p.plan[units], share = latent_share(total, ctas);
-  const long long cut = (long long)(blockIdx.y + 1) * share;
+  const long long cut = (long long)(blockIdx.x + 1) * share;
   if (cut >= total) return;
   const int u = latent_find_cta(p.plan, units, (int)cut, &u_shared), u_begin = p.plan[u], u_stop = p.plan[u + 1];
   if (u_begin == cut || cut - share > u_begin) return;            // no cut, or an earlier boundary has it
   const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, rows, p.H, p.window);
-  const int r = blockIdx.x;
-  if (r >= w.n_rows) return;
-  const int tok = (w.r0 + r) / p.H, h = (w.r0 + r) - tok * p.H;
-  const int c_first = blockIdx.y, c_last = (u_stop - 1) / share;
-  auto slot = [&](int c) { return (2ll * c + ((long long)u_begin > (long long)c * share ? 1 : 0)) * rows + r; };
-  float m = -INFINITY;
-  for (int c = c_first; c <= c_last; ++c) m = fmaxf(m, p.part_ml[slot(c) * 2]);
-  const float base = m == -INFINITY ? 0.f : m;
-  float l = 0.f;
-  for (int c = c_first; c <= c_last; ++c) l += p.part_ml[slot(c) * 2 + 1] * exp2f(p.part_ml[slot(c) * 2] - base);
-  const float f = l > 0.f ? p.gate[(long long)(w.t0 + tok) * p.H + h] / l : 0.f;
-  __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + ((long long)h * p.S + w.t0 + tok) * p.OW;
-  for (int col = 2 * threadIdx.x; col < p.RW; col += 2 * blockDim.x) {
-    float x = 0.f, y = 0.f;
-    for (int c = c_first; c <= c_last; ++c) {
-      const float wgt = exp2f(p.part_ml[slot(c) * 2] - base);
-      const float2 v = *reinterpret_cast<const float2*>(p.part_o + slot(c) * p.RW + col);
-      x = fmaf(wgt, v.x, x);
-      y = fmaf(wgt, v.y, y);
+  const int c_first = blockIdx.x, n = min((u_stop - 1) / share - c_first + 1, LAT_MERGE_MAX);
+  auto slot = [&](int i) { return 2ll * (c_first + i) + ((long long)u_begin > (long long)(c_first + i) * share ? 1 : 0); };
+  if (threadIdx.x < 32) {
+    const int r = threadIdx.x;
+    if (r < w.n_rows) {
+      const int tok = (w.r0 + r) / p.H, h = (w.r0 + r) - tok * p.H;
+      float m = -INFINITY, l = 0.f;
+      for (int i = 0; i < n; ++i) m = fmaxf(m, p.part_ml[(slot(i) * rows + r) * 2]);
+      const float base = m == -INFINITY ? 0.f : m;
+      for (int i = 0; i < n; ++i) {
+        const float e = exp2f(p.part_ml[(slot(i) * rows + r) * 2] - base);
+        l += p.part_ml[(slot(i) * rows + r) * 2 + 1] * e;
+        wgt[i][r] = e;
+      }
+      const float f = l > 0.f ? p.gate[(long long)(w.t0 + tok) * p.H + h] / l : 0.f;
+      for (int i = 0; i < n; ++i) wgt[i][r] *= f;
+      dst[r] = ((long long)h * p.S + w.t0 + tok) * p.OW;
     }
-    *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16x2(x * f, y * f);
+  }
+  __syncthreads();
+  // a thread takes four rows of one channel; a warp's lanes are neighbouring channels
+  for (int k = threadIdx.x; k < 128 * (rows / 4); k += blockDim.x) {
+    const int ch = blockIdx.y * 128 + (k & 127), r = (k >> 7) * 4;
+    if (ch >= p.RW) continue;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < n; ++i) {
+      const float4 v = __ldcg(reinterpret_cast<const float4*>(p.part_o + (slot(i) * p.RW + ch) * rows + r));
+      acc.x = fmaf(wgt[i][r], v.x, acc.x);
+      acc.y = fmaf(wgt[i][r + 1], v.y, acc.y);
+      acc.z = fmaf(wgt[i][r + 2], v.z, acc.z);
+      acc.w = fmaf(wgt[i][r + 3], v.w, acc.w);
+    }
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + ch;
+    if (r < w.n_rows) out[dst[r]] = __float2bfloat16_rn(acc.x);
+    if (r + 1 < w.n_rows) out[dst[r + 1]] = __float2bfloat16_rn(acc.y);
+    if (r + 2 < w.n_rows) out[dst[r + 2]] = __float2bfloat16_rn(acc.z);
+    if (r + 3 < w.n_rows) out[dst[r + 3]] = __float2bfloat16_rn(acc.w);
   }
 }
 
@@ -705,7 +800,7 @@ static LatentShape latent_shape(int max_q, int H, int CW, int RW) {
   LatentShape s;
   s.rows = max_q * H > 16 ? 32 : 16;
   s.row_tiles = (max_q * H + s.rows - 1) / s.rows;
-  const int nch = (CW + 63) / 64, nblk = (RW + 127) / 128, fixed = 1024 + nch * s.rows * 128 + 2 * s.rows * 128;
+  const int nch = (CW + 63) / 64, nblk = (RW + 127) / 128, fixed = 1024 + nch * s.rows * 128 + 3 * s.rows * 128;
   const int chunks = nch > 2 * nblk ? nch : 2 * nblk;
   s.keys = fixed + 3 * chunks * 48 * 128 <= limit ? 48 : 32;
   s.stages = (limit - fixed) / (chunks * s.keys * 128);
@@ -795,7 +890,7 @@ extern "C" int rb_latent_plan(const int* cu_q, const int* seq_lens, int B, int H
 }
 
 // T rows of B sequences (cu_q null: one row per sequence). max_q: most rows of any sequence. bf16: `plan` from rb_latent_plan
-// for the same batch; part_o [2 * CTAs][rows of a unit][RW] and part_ml [.., 2] hold the pieces of cut units.
+// for the same batch; part_o [2 * CTAs][RW][rows of a unit] and part_ml [2 * CTAs][rows][2] hold the pieces of cut units.
 extern "C" int rb_latent_attn(const void* qa, const void* cache, const int* block_tables, const int* cu_q, const int* seq_lens,
                               const float* sink, const float* gate, void* out, const int* plan, float* part_o, float* part_ml,
                               long long S, int H, int CW, int RW, int OW, int max_blocks, int num_blocks, int window,
@@ -816,13 +911,12 @@ extern "C" int rb_latent_attn(const void* qa, const void* cache, const int* bloc
   if (tma_map_2d_bf16(&p.map, cache, (unsigned long long)num_blocks * LAT_BLOCK, CW, CW, LAT_BLOCK) != 0) return -20;
   p.q_tma = max_q == 1 ? 1 : 0;
   if (p.q_tma && latent_q_map(&p.q_map, qa, H, S, CW, s.rows) != 0) return -21;
-  const int ctas = latent_sms();
+  const int ctas = latent_sms() < LAT_MERGE_MAX ? latent_sms() : LAT_MERGE_MAX;
   int rc;
   if (s.keys == 48) rc = s.rows == 32 ? launch_latent<32, 48>(p, s.smem, ctas, stream) : launch_latent<16, 48>(p, s.smem, ctas, stream);
   else rc = s.rows == 32 ? launch_latent<32, 32>(p, s.smem, ctas, stream) : launch_latent<16, 32>(p, s.smem, ctas, stream);
   if (rc != 0) return rc;
-  return launch_kernel(latent_merge_kernel, dim3(s.rows, ctas - 1), dim3(RW >= 256 ? 128 : 64), 0, stream, p, ctas, s.rows) == cudaSuccess
-             ? 0 : -11;
+  return launch_kernel(latent_merge_kernel, dim3(ctas - 1, (RW + 127) / 128), dim3(256), 0, stream, p, ctas, s.rows) == cudaSuccess ? 0 : -11;
 }
 
 extern "C" int rb_latent_gather(const void* cache, const int* block_tables, int bt_row0, int max_blocks, int num_blocks,
