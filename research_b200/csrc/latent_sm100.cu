@@ -142,11 +142,11 @@ __global__ void latent_query_kernel(TA* __restrict__ q, const int* __restrict__ 
 //   S   [rows, KT]      = Q C^T    : A = Q (K-major), B = the tile (K-major, all CW channels)
 //   O^T [channels, NH] += C^T P^T  : A = the tile read MN-major in blocks of 128 channels, B = P (K-major)
 // With the output transposed the few rows of a unit are the N side, so the accumulators take NH columns per 128 channels.
-// S has M = 128 although only NH rows are queries: the A descriptor runs on into the shared memory behind them, and those
-// rows of S are never read.
+// S has M = 64 although only NH rows are queries: the A descriptor runs on into the shared memory behind them, and those
+// rows of S are never read. (An instruction takes the time of its A operand here, so M = 64 halves the cost of S.)
 //
-// Warps: 0 TMA producer, 1 MMA issuer + TMEM owner, 2-3 load the queries of the next unit, 4 softmax (one row per lane),
-// 4-7 rescale and store O^T. The running maximum is refreshed only when it grew by more than 2^8. A wait that runs out sets
+// Warps: 0 TMA producer, 1 MMA issuer + TMEM owner, 2-3 load the queries of the next unit, 4 (and 5) softmax, one row
+// per lane, 4-7 rescale and store O^T. The running maximum is refreshed only when it grew by more than 2^8. A wait that runs out sets
 // the status and an abort flag that ends all other waits; the steps still run through, so that every barrier is met.
 // ------------------------------------------------------------------------------------------
 constexpr int LAT_THREADS = 256;
@@ -265,12 +265,13 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
   constexpr int CHUNK = KT * 128;                // bytes of 64 channels of a tile
   constexpr int PAGES = KT / LAT_BLOCK;
   constexpr int SB = 3;                          // score, weight and alpha buffers
+  constexpr int SW = NH / 16;                    // softmax warps
   constexpr uint32_t O_COL = SB * 64;            // TMEM: S at columns 0, 64, 128, O^T behind
   extern __shared__ __align__(128) uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t kv_full[LAT_MAX_STAGES], kv_empty[LAT_MAX_STAGES];
-  __shared__ __align__(8) uint64_t q_full, q_empty, s_full[SB], p_full[SB], o_done, o_free, cmd, cmd_done;
-  __shared__ float s_alpha[NH], s_scale[NH];
-  __shared__ int s_tile;
+  __shared__ __align__(8) uint64_t q_full, q_empty, s_full[SB], a_full[SB], p_full[SB], o_done, o_free;
+  __shared__ float s_alpha[SB][NH], s_scale[NH];
+  __shared__ int s_flag[SB][SW];
   __shared__ long long s_row[NH];
   __shared__ uint32_t tmem_base_smem;
   __shared__ int abort_flag, u_shared;
@@ -298,12 +299,11 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
     mbar_init(smem_u32(&q_empty), 1);
     for (int i = 0; i < SB; ++i) {
       mbar_init(smem_u32(&s_full[i]), 1);
-      mbar_init(smem_u32(&p_full[i]), 1);
+      mbar_init(smem_u32(&a_full[i]), SW);
+      mbar_init(smem_u32(&p_full[i]), 4);
     }
     mbar_init(smem_u32(&o_done), 1);
     mbar_init(smem_u32(&o_free), 4);
-    mbar_init(smem_u32(&cmd), 1);
-    mbar_init(smem_u32(&cmd_done), 3);
     fence_mbar_init();
   }
   const uint32_t tmem_cols = O_COL + (nblk * NH + 31) / 32 * 32 <= 256 ? 256 : 512;
@@ -357,7 +357,7 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
   } else if (warp == 1) {
     // ---------------------------------------------------------------- MMA issuer
     if (elect_one_sync()) {
-      constexpr uint32_t idesc_s = make_idesc_bf16(128, KT, 0, 0);
+      constexpr uint32_t idesc_s = make_idesc_bf16(64, KT, 0, 0);
       constexpr uint32_t idesc_o = make_idesc_bf16(128, NH, 1, 0);
       const int n = t_end - t_begin, ksteps = p.CW / 16;
       int uq = 0, u_s = u_first, u_o = u_first;      // units started by the scores / being summed
@@ -474,53 +474,39 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
       ++uq;
     }
   } else {
-    // ---------------------------------------------------------------- softmax (warp 4), O^T (warps 4-7)
-    // Warp 4 works alone from tile to tile. It calls the other three through `cmd` when O^T has to be rescaled (s_tile = the
-    // tile) and when a piece is complete (s_tile = -1).
-    const int qd = warp - 4;
+    // ---------------------------------------------------------------- softmax (warps 4..), O^T (warps 4-7)
+    // S has M = 64: rows 16q .. 16q+15 lie in lanes 0-15 of TMEM quarter q, so warp 4 + q owns rows 16q + lane.
+    const int qd = warp - 4, row = qd * 16 + lane;
+    const bool soft = qd < SW, mine = soft && lane < 16;
     const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
     const float log2e = 1.4426950408889634f, scale_log2 = p.scale * log2e;
-    auto rescale = [&](int j) {                     // O^T holds the tiles before tile j
-      mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
-      __syncwarp();
-      tc_fence_after();
-#pragma unroll 1
-      for (int c = 0; c < nblk * NH; c += 32) {
-        uint32_t o[32];
-        tmem_ld_32x32(tmem_o + lane_addr + c, o);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[i & (NH - 1)]);
-        tmem_st_32x32(tmem_o + lane_addr + c, o);
-      }
-      tmem_st_wait();
-      tc_fence_before();
-      __syncwarp();
-    };
-    uint32_t n_cmd = 0, n_rescale = 0;
     int j = 0;
     for (int u = u_first, t = t_begin; t < t_end; ++u) {
       const int u_begin = p.plan[u], u_stop = p.plan[u + 1], u_end = min(u_stop, t_end);
       if (u_end <= t) continue;
       const LatentUnit w = latent_unit(p.cu_q, p.seq_lens, u, p.row_tiles, NH, p.H, p.window);
-      const bool has_first = t == u_begin, whole = has_first && u_end == u_stop, row_ok = lane < w.n_rows;
-      const int tok = (w.r0 + (row_ok ? lane : 0)) / p.H, head = (w.r0 + (row_ok ? lane : 0)) - tok * p.H;
+      const bool has_first = t == u_begin, whole = has_first && u_end == u_stop, row_ok = mine && row < w.n_rows;
+      const int tok = (w.r0 + (row_ok ? row : 0)) / p.H, head = (w.r0 + (row_ok ? row : 0)) - tok * p.H;
+      const int pos = w.L - w.q_len + tok;
+      const int pos_min = w.L - w.q_len + w.r0 / p.H, pos_max = w.L - w.q_len + (w.r0 + w.n_rows - 1) / p.H;
       float m_used = -INFINITY, l = 0.f, sink = 0.f, gate = 0.f;
-      if (qd == 0) {
+      if (row_ok) {
         sink = p.sink[head] * log2e;
         gate = p.gate[(long long)(w.t0 + tok) * p.H + head];
-        const int pos = w.L - w.q_len + tok;
-        const int pos_min = w.L - w.q_len + w.r0 / p.H, pos_max = w.L - w.q_len + (w.r0 + w.n_rows - 1) / p.H;
-        const int t_piece = t;
-        for (int k0 = w.lo + (t - u_begin) * KT; t < u_end; ++t, k0 += KT, ++j) {
-          const int b = j % SB;
-          mbar_wait_bounded(smem_u32(&s_full[b]), (j / SB) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      }
+      const int t_piece = t;
+      for (int k0 = w.lo + (t - u_begin) * KT; t < u_end; ++t, k0 += KT, ++j) {
+        const int b = j % SB;
+        const uint32_t ph = (j / SB) & 1u;
+        if (soft) {
+          mbar_wait_bounded(smem_u32(&s_full[b]), ph, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
           __syncwarp();
           tc_fence_after();
           uint32_t v[KT];
-          tmem_ld_32x32(tmem_base + b * 64, *reinterpret_cast<uint32_t(*)[32]>(&v[0]));
-          if constexpr (KT == 48) tmem_ld_32x16(tmem_base + b * 64 + 32, *reinterpret_cast<uint32_t(*)[16]>(&v[32]));
+          tmem_ld_32x32(tmem_base + lane_addr + b * 64, *reinterpret_cast<uint32_t(*)[32]>(&v[0]));
+          if constexpr (KT == 48) tmem_ld_32x16(tmem_base + lane_addr + b * 64 + 32, *reinterpret_cast<uint32_t(*)[16]>(&v[32]));
           tmem_ld_wait();
+          tc_fence_before();
           if (k0 + KT - 1 > pos_min || k0 <= pos_max - p.window) {
 #pragma unroll
             for (int i = 0; i < KT; ++i)
@@ -531,18 +517,11 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
           for (int i = 0; i < KT; ++i) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(v[i]));
           const float m_new = fmaxf(m_used, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * scale_log2);
           const bool need = row_ok && (m_new > m_used + LAT_RESCALE || (m_used == -INFINITY && m_new != -INFINITY));
-          const bool any = __any_sync(0xffffffffu, need && t > t_piece);
-          if (any && lane < NH) s_alpha[lane] = need && m_used != -INFINITY ? lat_exp2(m_used - m_new) : 1.f;
-          if (need) {
-            l *= m_used != -INFINITY ? lat_exp2(m_used - m_new) : 1.f;
-            m_used = m_new;
-          }
-          if (any) {
-            if (lane == 0) s_tile = j;
-            __syncwarp();
-            if (lane == 0) mbar_arrive(smem_u32(&cmd));
-            rescale(j);
-          }
+          const float alpha = need && m_used != -INFINITY ? lat_exp2(m_used - m_new) : 1.f;
+          const int any = __any_sync(0xffffffffu, need && t > t_piece);
+          if (need) { m_used = m_new; l *= alpha; }
+          if (mine) s_alpha[b][row] = alpha;
+          if (lane == 0) s_flag[b][qd] = any;
           const float mref = m_used == -INFINITY ? 0.f : m_used;
           float ls[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -552,8 +531,8 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
             v[i] = __float_as_uint(x);
           }
           l += (ls[0] + ls[1]) + (ls[2] + ls[3]);
-          if (lane < NH) {
-            uint8_t* prow = p_ptr + b * (NH * 128) + lane * 128;
+          if (mine) {
+            uint8_t* prow = p_ptr + b * (NH * 128) + row * 128;
 #pragma unroll
             for (int i = 0; i < KT / 8; ++i) {
               uint4 o;
@@ -562,34 +541,40 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
               o.z = pack_bf16x2(__uint_as_float(v[i * 8 + 4]), __uint_as_float(v[i * 8 + 5]));
               o.w = pack_bf16x2(__uint_as_float(v[i * 8 + 6]), __uint_as_float(v[i * 8 + 7]));
               if (!row_ok) o = make_uint4(0, 0, 0, 0);
-              *reinterpret_cast<uint4*>(prow + ((i ^ (lane & 7)) << 4)) = o;
+              *reinterpret_cast<uint4*>(prow + ((i ^ (row & 7)) << 4)) = o;
             }
           }
           fence_proxy_async_smem();
-          tc_fence_before();
-          if (any) {                                // the other quarters of O^T are rescaled too
-            mbar_wait_bounded(smem_u32(&cmd_done), n_rescale & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
-            ++n_rescale;
+          __syncwarp();
+          if (lane == 0) mbar_arrive(smem_u32(&a_full[b]));
+        }
+        mbar_wait_bounded(smem_u32(&a_full[b]), ph, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+        __syncwarp();
+        int flag = 0;
+#pragma unroll
+        for (int i = 0; i < SW; ++i) flag |= *(volatile int*)&s_flag[b][i];
+        if (flag) {                                 // O^T holds the tiles before this one
+          mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+          __syncwarp();
+          tc_fence_after();
+#pragma unroll 1
+          for (int c = 0; c < nblk * NH; c += 32) {
+            uint32_t o[32];
+            tmem_ld_32x32(tmem_o + lane_addr + c, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[b][i & (NH - 1)]);
+            tmem_st_32x32(tmem_o + lane_addr + c, o);
           }
-          __syncwarp();
-          if (lane == 0) mbar_arrive(smem_u32(&p_full[b]));
+          tmem_st_wait();
+          tc_fence_before();
         }
-      } else {
-        j += u_end - t;
-        t = u_end;
-        while (true) {
-          mbar_wait_bounded(smem_u32(&cmd), n_cmd & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
-          ++n_cmd;
-          __syncwarp();
-          const int tile = *(volatile int*)&s_tile;
-          if (tile < 0 || *abortp != 0) break;
-          rescale(tile);
-          if (lane == 0) mbar_arrive(smem_u32(&cmd_done));
-        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&p_full[b]));
       }
       // ---- the piece is complete ----
       const long long slot = 2ll * blockIdx.x + (u_begin > t_begin ? 1 : 0);
-      if (qd == 0 && lane < NH) {
+      if (mine) {
         float m = m_used, f = 1.f;
         if (has_first) {                            // the sink: in the denominator once, no value
           m = fmaxf(m_used, sink);
@@ -597,17 +582,12 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
           l = l * f + lat_exp2(sink - m);
         }
         if (whole) f = l > 0.f ? f * gate / l : 0.f;
-        s_scale[lane] = f;
-        s_row[lane] = ((long long)head * p.S + w.t0 + tok) * p.OW;
+        s_scale[row] = f;
+        s_row[row] = ((long long)head * p.S + w.t0 + tok) * p.OW;
         if (!whole && row_ok) {
-          p.part_ml[(slot * NH + lane) * 2] = m;
-          p.part_ml[(slot * NH + lane) * 2 + 1] = l;
+          p.part_ml[(slot * NH + row) * 2] = m;
+          p.part_ml[(slot * NH + row) * 2 + 1] = l;
         }
-      }
-      if (qd == 0) {
-        if (lane == 0) s_tile = -1;
-        __syncwarp();
-        if (lane == 0) mbar_arrive(smem_u32(&cmd));
       }
       mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
       lat_bar(1, 128);
@@ -624,9 +604,9 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
             const int r = i & (NH - 1), ch = (c + i) / NH * 128 + qd * 32 + (lane & ~1);
             const float x = __uint_as_float(o[i]) * s_scale[r], y = __uint_as_float(o[i + 1]) * s_scale[r + 1];
             const float got = __shfl_xor_sync(0xffffffffu, (lane & 1) ? x : y, 1);
-            const int row = r + (lane & 1);
-            if (row < w.n_rows && ch < p.RW)
-              *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + s_row[row] + ch) =
+            const int ro = r + (lane & 1);
+            if (ro < w.n_rows && ch < p.RW)
+              *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(p.out) + s_row[ro] + ch) =
                   (lane & 1) ? pack_bf16x2(got, y) : pack_bf16x2(x, got);
           }
         } else {
