@@ -31,15 +31,15 @@ template <> __device__ __forceinline__ __nv_bfloat16 lat_cast<__nv_bfloat16>(flo
 __device__ __forceinline__ float lat_f(float v) { return v; }
 __device__ __forceinline__ float lat_f(__nv_bfloat16 v) { return __bfloat162float(v); }
 
-__device__ __forceinline__ float lat_block_sum(float v, float* red) {
-  v = warp_sum(v);
+// Sums of two values over the CTA in one round; every thread receives both.
+__device__ __forceinline__ float2 lat_block_sum2(float a, float b, float2* red) {
+  a = warp_sum(a);
+  b = warp_sum(b);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  if (lane == 0) red[warp] = v;
+  if (lane == 0) red[warp] = make_float2(a, b);
   __syncthreads();
-  float t = lane < nw ? red[lane] : 0.f;
-  t = warp_sum(t);
-  __syncthreads();
-  return t;
+  const float2 t = lane < nw ? red[lane] : make_float2(0.f, 0.f);
+  return make_float2(warp_sum(t.x), warp_sum(t.y));
 }
 
 // ------------------------------------------------------------------------------------------
@@ -53,24 +53,25 @@ __global__ void latent_append_kernel(const float* __restrict__ proj, long long l
                                      TA* __restrict__ cache, long long num_slots, int CW, int rot_off, TA* __restrict__ cq,
                                      long long ldq, float* __restrict__ gate, int q_rank, int kv_rank, int rot_dim, int H,
                                      int* status) {
-  __shared__ float red[32];
+  __shared__ float2 red[32];
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x;
+  const int slot = slots[t], pos = positions[t];
   const float* p = proj + t * ldp;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) ss = fmaf(p[i], p[i], ss);
-  const float rq = 1.f / sqrtf(lat_block_sum(ss, red) / (float)q_rank + eps);
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) cq[t * ldq + i] = lat_cast<TA>(p[i] * rq * qn_w[i]);
   const float* pc = p + q_rank;
-  ss = 0.f;
-  for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) ss = fmaf(pc[i], pc[i], ss);
-  const float rc = 1.f / sqrtf(lat_block_sum(ss, red) / (float)kv_rank + eps);
   const float* pr = pc + kv_rank;
+  float sq = 0.f, sc = 0.f;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) sq = fmaf(p[i], p[i], sq);
+#pragma unroll 2
+  for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) sc = fmaf(pc[i], pc[i], sc);
+  const float2 sums = lat_block_sum2(sq, sc, red);
+  const float rq = 1.f / sqrtf(sums.x / (float)q_rank + eps), rc = 1.f / sqrtf(sums.y / (float)kv_rank + eps);
+#pragma unroll 4
+  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) cq[t * ldq + i] = lat_cast<TA>(p[i] * rq * qn_w[i]);
   for (int h = threadIdx.x; h < H; h += blockDim.x) gate[t * H + h] = 1.f / (1.f + expf(-pr[rot_dim + h]));
-  const int slot = slots[t];
   if (slot < 0) return;
-  int pos = positions[t];
   if (slot >= num_slots || pos < 0 || pos >= max_pos) {
     if (threadIdx.x == 0) set_status(status, ST_BAD_INDEX);
     return;
@@ -269,7 +270,7 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
   constexpr uint32_t O_COL = SB * 64;            // TMEM: S at columns 0, 64, 128, O^T behind
   extern __shared__ __align__(128) uint8_t smem_raw[];
   __shared__ __align__(8) uint64_t kv_full[LAT_MAX_STAGES], kv_empty[LAT_MAX_STAGES];
-  __shared__ __align__(8) uint64_t q_full, q_empty, s_full[SB], a_full[SB], p_full[SB], o_done, o_free;
+  __shared__ __align__(8) uint64_t q_full, q_empty, s_full[SB], a_full[SB], p_full[SB], o_done[SB], o_free;
   __shared__ float s_alpha[SB][NH], s_scale[NH];
   __shared__ int s_flag[SB][SW];
   __shared__ long long s_row[NH];
@@ -301,8 +302,8 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
       mbar_init(smem_u32(&s_full[i]), 1);
       mbar_init(smem_u32(&a_full[i]), SW);
       mbar_init(smem_u32(&p_full[i]), 4);
+      mbar_init(smem_u32(&o_done[i]), 1);
     }
-    mbar_init(smem_u32(&o_done), 1);
     mbar_init(smem_u32(&o_free), 4);
     fence_mbar_init();
   }
@@ -434,10 +435,10 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
           for (int k = 0; k < KT / 16; ++k)
             umma_bf16(tmem_o + m * NH, ad + k * (2048 >> 4), bd + 2 * k, idesc_o, (!first || k > 0) ? 1u : 0u);
         umma_commit(smem_u32(&kv_empty[s]));
-        umma_commit(smem_u32(&o_done));
+        umma_commit(smem_u32(&o_done[j % SB]));
       }
       // nothing of this CTA is in flight when it frees its TMEM
-      mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(n - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      mbar_wait_bounded(smem_u32(&o_done[(n - 1) % SB]), ((n - 1) / SB) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
     }
   } else if (warp < 4) {
     // ---------------------------------------------------------------- query rows of every unit
@@ -480,6 +481,11 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
     const bool soft = qd < SW, mine = soft && lane < 16;
     const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
     const float log2e = 1.4426950408889634f, scale_log2 = p.scale * log2e;
+    // The sums of tile j have been added. One barrier per buffer: its phase before the awaited one is over by then (a tile's
+    // scores are complete only after the sums of three tiles ago), which a single barrier would not guarantee.
+    auto o_wait = [&](int j) {
+      mbar_wait_bounded(smem_u32(&o_done[j % SB]), (j / SB) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+    };
     int j = 0;
     for (int u = u_first, t = t_begin; t < t_end; ++u) {
       const int u_begin = p.plan[u], u_stop = p.plan[u + 1], u_end = min(u_stop, t_end);
@@ -554,7 +560,7 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
 #pragma unroll
         for (int i = 0; i < SW; ++i) flag |= *(volatile int*)&s_flag[b][i];
         if (flag) {                                 // O^T holds the tiles before this one
-          mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+          o_wait(j - 1);
           __syncwarp();
           tc_fence_after();
 #pragma unroll 1
@@ -589,7 +595,7 @@ __global__ void __launch_bounds__(LAT_THREADS, 1) latent_attn_kernel(const __gri
           p.part_ml[(slot * NH + row) * 2 + 1] = l;
         }
       }
-      mbar_wait_bounded(smem_u32(&o_done), (uint32_t)(j - 1) & 1u, abortp, p.status, ST_TIMEOUT_TMEM_FULL);
+      o_wait(j - 1);
       lat_bar(1, 128);
       tc_fence_after();
 #pragma unroll 1
@@ -830,7 +836,7 @@ extern "C" int rb_latent_append(const float* proj, long long ldp, const float* q
                                 int q_rank, int kv_rank, int rot_dim, int H, int T, int dtype, int* status, cudaStream_t stream) {
   if (T <= 0 || rot_off < kv_rank || rot_off + rot_dim > CW || 2 * rot_pairs > rot_dim || ldq < q_rank) return -1;
   if (ldp < (long long)q_rank + kv_rank + rot_dim + H) return -1;
-  const int threads = q_rank + kv_rank <= 512 ? 128 : 256;
+  const int threads = q_rank + kv_rank <= 512 ? 128 : (T <= 512 && q_rank > 1024 ? 512 : 256);
   cudaError_t e;
   if (dtype == 0)
     e = launch_kernel(latent_append_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, proj, ldp, qn_w, kn_w, eps, positions,

@@ -223,6 +223,26 @@ def test_attention_shares_cut_anywhere(cuda_device):
             close(out[:, b], want[0], dt, (B, b, L))
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("heads", [3, 20])
+def test_attention_is_repeatable(cuda_device, heads):
+    """Hand-offs between the kernel's warps: short sequences (few tiles per CTA, cut units) give the same bits every time."""
+    geo, B = LatentGeometry(heads, 24, 8, 4, 20, 40, 36), 5
+    g = torch.Generator().manual_seed(4)
+    bt = torch.randperm(B * 10, generator=g).int().view(B, 10).to(cuda_device)
+    sl = torch.tensor([97, 120, 33, 150, 49], dtype=torch.int32, device=cuda_device)
+    cache, qa = rand(B * 10, 16, geo.cw, seed=1, dtype=torch.bfloat16).to(cuda_device), (3 * rand(heads, B, geo.cw, seed=2)).bfloat16().to(cuda_device)
+    sink, gate = rand(heads, seed=3).to(cuda_device), torch.sigmoid(rand(B, heads, seed=4)).to(cuda_device)
+    plan = torch.zeros(ops.latent_units(B, heads, 1) + 1, dtype=torch.int32, device=cuda_device)
+    ops.latent_plan(None, sl, geo, 1, 1000, plan)
+    ws, first = ops.latent_workspace([geo], cuda_device), None
+    for _ in range(300):
+        out = torch.zeros(heads, B, geo.rw, dtype=torch.bfloat16, device=cuda_device)
+        ops.latent_attention(qa, cache, geo, bt, None, sl, sink, gate, out, scale=0.3, window=1000, rows=B, max_q=1, plan=plan, workspace=ws)
+        first = out if first is None else first
+        assert torch.equal(out, first)
+
+
 @pytest.mark.parametrize("place", [PLACES[0], PLACES[2]])
 @pytest.mark.parametrize("geo", [LatentGeometry(4, 40, 12, 6, 24, 72, 44), LatentGeometry(2, 128, 64, 32, 128, 96, 64),
                                  LatentGeometry(3, 100, 64, 32, 50, 64, 64), LatentGeometry(3, 50, 40, 16, 128, 80, 64)])
