@@ -10,7 +10,11 @@ from .types import EngineConfig, SamplingParams
 
 
 def engine_smoke(device: torch.device) -> None:
-    cfg = get_preset("tiny-qwen2", num_layers=2)
+    _run(device, get_preset("tiny-qwen2", num_layers=2))
+    _run(device, get_preset("tiny-lulezen"))      # latent attention: prefill and decode kernels, 32-bit residual stream
+
+
+def _run(device: torch.device, cfg) -> None:
     w = init_random_weights(cfg, seed=0, dtype=torch.bfloat16, device=device)
     eng = InferenceEngine(EngineConfig(max_batch_size=4, max_model_len=256, num_kv_blocks=64, ignore_eos=True,
                                        graph_batch_sizes=(2, 4)), cfg, w, device=device)

@@ -25,6 +25,7 @@ from ..models.stack import ClampedGluSpec, LatentAttentionSpec, LayerStackConfig
 from ..ops.latent import LatentGeometry, live_tables
 from .model_runner import BLOCK, PackedBatch, RunnerBase
 
+MAX_LATENT, MAX_CACHE_ROW = 1024, 1088
 SHORT_PORTION = 16           # new tokens of a sequence up to which attention runs on the cached latents
 
 
@@ -72,6 +73,10 @@ class StackRunner(RunnerBase):
                  graph_batch_sizes: tuple[int, ...] = (), tp=None, ep=None, dtype: torch.dtype = torch.bfloat16):
         if tp is not None or ep is not None:
             raise ValueError("layer-stack models run on one GPU per engine (no tensor or expert parallelism)")
+        for x in cfg.layers:
+            g = latent_geometry(x.mixer)
+            if g.rw > MAX_LATENT or g.cw > MAX_CACHE_ROW:
+                raise ValueError(f"the latent attention kernels take up to {MAX_LATENT} latent channels and cache rows of {MAX_CACHE_ROW}")
         self.tp = self.ep = None
         self.tp_size, self.tp_rank = 1, 0
         self._init_geometry(cfg, device=device, num_kv_blocks=num_kv_blocks, max_batch=max_batch, max_model_len=max_model_len,

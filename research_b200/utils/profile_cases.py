@@ -214,6 +214,42 @@ def case_moe_train() -> None:
     print("ok")
 
 
+def case_latent_decode() -> None:
+    """Latent attention on the cached rows: 256 sequences x 2048 keys, 32 heads, 512 latent + 64 rotated channels (600 MB)."""
+    from ..ops.latent import LatentGeometry
+
+    geo, B, L = LatentGeometry(32, 128, 64, 32, 128, 512, 1536), 256, 2048
+    cache = torch.randn(B * L // 16, 16, geo.cw, device="cuda").bfloat16()
+    bt = torch.randperm(B * L // 16, device="cuda").int().view(B, L // 16).contiguous()
+    lens = torch.full((B,), L, dtype=torch.int32, device="cuda")
+    qa, out = torch.randn(32, B, geo.cw, device="cuda").bfloat16(), torch.zeros(32, B, geo.rw, dtype=torch.bfloat16, device="cuda")
+    sink, gate = torch.zeros(32, device="cuda"), torch.rand(B, 32, device="cuda")
+    plan = torch.zeros(ops.latent_units(B, 32, 1) + 1, dtype=torch.int32, device="cuda")
+    ops.latent_plan(None, lens, geo, 1, 4096, plan)
+    ws = ops.latent_workspace([geo], "cuda")
+    for _ in range(3):
+        ops.latent_attention(qa, cache, geo, bt, None, lens, sink, gate, out, scale=0.07, window=4096, rows=B, max_q=1, plan=plan, workspace=ws)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def case_latent_prefill() -> None:
+    """Latent attention on multiplied-out keys and values: one prompt of 4096 tokens, 32 heads of 128 + 64 / 128 channels."""
+    from ..ops.latent import LatentGeometry
+
+    geo, T = LatentGeometry(32, 128, 64, 32, 128, 512, 1536), 4096
+    q, k, v = (torch.randn(T, 32 * n, device="cuda").bfloat16() for n in (192, 128, 128))
+    rot, out = torch.randn(T, 64, device="cuda").bfloat16(), torch.empty(T, 32 * 128, dtype=torch.bfloat16, device="cuda")
+    cu = torch.tensor([0, T], dtype=torch.int32, device="cuda")
+    sink, gate = torch.zeros(32, device="cuda"), torch.rand(T, 32, device="cuda")
+    for _ in range(3):
+        ops.flash_latent_prefill(q, k, rot, v, geo, cu, cu, sink, gate, out, scale=0.07, window=4096, max_q=T, rows=T)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
 CASES = {k[5:]: v for k, v in globals().items() if k.startswith("case_")}
 
 if __name__ == "__main__":

@@ -221,7 +221,7 @@ def llama_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> d
     return t.rows
 
 
-def run(sizes: tuple[str, ...] = (), batches: tuple[int, ...] = (1, 64, 256), context: int = 1024, prompts: tuple[int, ...] = (512, 4096),
+def run(sizes: tuple[str, ...] = (), batches: tuple[int, ...] = (1, 64, 256), context: int = 2048, prompts: tuple[int, ...] = (512, 4096),
         kernels: bool = True) -> dict:
     out: dict = {"peaks": dict(zip(("hbm_bytes_s", "bf16_flop_s", "origin"), peaks())), "context": context, "sizes": {}}
     for s in SIZES:

@@ -15,7 +15,8 @@ from research_b200.ops.latent import LatentGeometry
 PLACES = [("cpu", torch.float32), pytest.param(("cuda", torch.float32), marks=pytest.mark.gpu),
           pytest.param(("cuda", torch.bfloat16), marks=pytest.mark.gpu)]
 GEOMETRIES = [LatentGeometry(5, 40, 12, 6, 24, 72, 44), LatentGeometry(1, 7, 2, 1, 5, 9, 10), LatentGeometry(16, 128, 64, 32, 128, 512, 200),
-              LatentGeometry(40, 64, 32, 16, 64, 250, 64), LatentGeometry(3, 16, 8, 2, 16, 600, 24)]
+              LatentGeometry(40, 64, 32, 16, 64, 250, 64), LatentGeometry(3, 16, 8, 2, 16, 600, 24),
+              LatentGeometry(20, 16, 64, 32, 16, 1024, 24)]
 
 
 def close(got, want, dtype, what=""):

@@ -336,6 +336,30 @@ def test_seeded_sampling_weight_update_and_score(place):
     assert eng.generate(p[:1], SamplingParams(temperature=0.0, max_tokens=2))[0].cached_tokens == 0
 
 
+def test_http_front_end_serves_it():
+    from fastapi.testclient import TestClient
+
+    from research_b200.inference.server import EngineService, create_app
+
+    name = "uneven"
+    svc = EngineService(engine(name, ("cpu", "float32"), cache_type="radix", num_kv_blocks=80))
+    try:
+        client = TestClient(create_app(svc, name))
+        ids = tokens_for(CONFIGS[name], 30, 4)
+        r = client.post("/generate", json={"input_ids": ids, "sampling_params": {"temperature": 0.0, "max_new_tokens": 5}}).json()
+        w = {k: v.double() for k, v in weights_for(CONFIGS[name]).items()}
+        for k, tok in enumerate(r["output_ids"]):
+            assert int(oracle.forward(ids + r["output_ids"][:k], w, CONFIGS[name])[-1].argmax()) == tok
+    finally:
+        svc.shutdown()
+
+
+def test_sizes_beyond_the_kernels_are_refused():
+    c = model([(mixer(kv_rank=1500), None)])
+    with pytest.raises(ValueError, match="latent channels"):
+        InferenceEngine(EngineConfig(max_batch_size=2, max_model_len=64, num_kv_blocks=8), config_from_dict(c), weights_for(c), device="cpu")
+
+
 def test_hf_models_take_portions_and_fed_tokens_too():
     """The portioned scheduler and fed streams are not special to layer stacks."""
     from research_b200.models import causal_lm_forward
