@@ -11,8 +11,8 @@
 //              multi-head attention on them (flash_sm100.cu). Long portions of a prompt.
 //
 // This file: the steps between the projections and the attention (norms, rotation, cache append), the absorbed
-// attention (bf16 on mma.sync: one pass over the cached rows is bound by HBM, not by the tensor pipe; fp32 for the exact
-// mode), the merge of its splits, and the gather of cached rows for the expanded form.
+// attention (bf16 on the 5th-generation tensor cores; fp32 for the exact mode), the merge of its pieces, and the gather of
+// cached rows for the expanded form.
 //
 // All heads of a token form rows of one score tile: row r of a sequence is (token r / H, head r % H). The mask is a
 // causal sliding window; the softmax denominator also contains exp(sink[h]); every head's output is multiplied by a gate.
@@ -144,7 +144,7 @@ __global__ void latent_query_kernel(TA* __restrict__ q, const int* __restrict__ 
 //   O^T [channels, NH] += C^T P^T  : A = the tile read MN-major in blocks of 128 channels, B = P (K-major)
 // With the output transposed the few rows of a unit are the N side, so the accumulators take NH columns per 128 channels.
 // S has M = 64 although only NH rows are queries: the A descriptor runs on into the shared memory behind them, and those
-// rows of S are never read. (An instruction takes the time of its A operand here, so M = 64 halves the cost of S.)
+// rows of S are never read.
 //
 // Warps: 0 TMA producer, 1 MMA issuer + TMEM owner, 2-3 load the queries of the next unit, 4 (and 5) softmax, one row
 // per lane, 4-7 rescale and store O^T. The running maximum is refreshed only when it grew by more than 2^8. A wait that runs out sets
