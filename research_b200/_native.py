@@ -40,6 +40,7 @@ LIBRARIES: dict[str, tuple[str, list[str]]] = {
     "rb_ops": ("nvcc", ["ops_sm100.cu"]),
     "rb_attn": ("nvcc", ["attn_sm100.cu"]),
     "rb_latent": ("nvcc", ["latent_sm100.cu"]),
+    "rb_recurrent": ("nvcc", ["recurrent_sm100.cu"]),
     "rb_gemm_f32": ("nvcc", ["gemm_f32_sm100.cu"]),
     "rb_flash": ("nvcc", ["flash_sm100.cu"]),
     "rb_quant": ("nvcc", ["quant_sm100.cu"]),

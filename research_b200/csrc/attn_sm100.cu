@@ -748,6 +748,409 @@ extern "C" int rb_paged_prefill(const void* q, const void* k_cache, const void* 
 }
 
 // ------------------------------------------------------------------------------------------
+// Attention whose values are its keys (ops/keyvalue.py): one cached row per token and kv head, [num_blocks, G, 16, D]. The joint
+// projection of a token is q [H, D] | k [G, D] | gate [H, D]; the softmax denominator also holds exp(sink[h]), and the
+// output is multiplied by sigmoid(gate) element by element.
+// ------------------------------------------------------------------------------------------
+namespace rb {
+
+__device__ __forceinline__ float kv_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float kv_to_f(float v) { return v; }
+__device__ __forceinline__ float kv_to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void kv_store(float* p, float v) { *p = v; }
+__device__ __forceinline__ void kv_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// Queries times 1 + coef ln(floor((p + 1) / every) + 1) in place, keys into the cache. One CTA per token.
+template <typename T>
+__global__ void kv_append_kernel(T* __restrict__ proj, long long ld, const int* __restrict__ positions, const int* __restrict__ slots, float coef,
+                                 int every, T* __restrict__ cache, int num_blocks, int H, int G, int D, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  T* row = proj + t * ld;
+  const float f = 1.f + coef * logf((float)((positions[t] + 1) / every) + 1.f);
+  if (f != 1.f)
+    for (int i = threadIdx.x; i < H * D; i += blockDim.x) kv_store(row + i, kv_to_f(row[i]) * f);
+  const int slot = slots[t];
+  if (slot < 0) return;
+  const int blk = slot / KV_BLOCK;
+  if (blk >= num_blocks) { if (threadIdx.x == 0) set_status(status, ST_BAD_INDEX); return; }
+  for (int i = threadIdx.x; i < G * D; i += blockDim.x)
+    cache[(((long long)blk * G + i / D) * KV_BLOCK + slot % KV_BLOCK) * D + i % D] = row[H * D + i];
+}
+
+// Decode: the structure of paged_decode_tma_kernel with one tile that serves as K and V, up to 16 query heads per CTA
+// (blockIdx.y = kv head x chunk of 16 query heads).
+template <int D>
+__host__ __device__ constexpr int kv_dec_stages() { return D == 64 ? 6 : 6; }
+constexpr int KV_MERGE_LD_PAD = 4;
+
+template <int D>
+__global__ void __launch_bounds__(DEC_WARPS * 32)
+kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_col, const __grid_constant__ CUtensorMap k_map,
+                 const int* __restrict__ block_tables, const int* __restrict__ seq_lens, const float* __restrict__ sink,
+                 __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int H, int Hkv, int bt_stride,
+                 int num_blocks, int num_splits, float scale, int* status) {
+  constexpr int CH = D / 8;
+  constexpr int TILE_BYTES = KV_BLOCK * D * 2;
+  constexpr int ST = kv_dec_stages<D>();
+  extern __shared__ __align__(128) uint8_t smem[];
+  __shared__ __align__(8) uint64_t bars[DEC_WARPS][ST];
+  __shared__ int abort_flag;
+  pdl_launch_dependents();
+  const int G = H / Hkv, chunks = (G + 15) / 16;
+  const int split = blockIdx.x, kvh = blockIdx.y / chunks, b = blockIdx.z;
+  const int h0 = kvh * G + (blockIdx.y % chunks) * 16;      // first query head of this CTA
+  const int rows = min(16, kvh * G + G - h0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const uint32_t ring0 = (smem_u32(smem) + 1023u) & ~1023u;
+  uint8_t* ring_ptr = smem + (ring0 - smem_u32(smem));
+  const uint32_t k_smem = ring0 + warp * (ST * TILE_BYTES);
+  uint8_t* q_ptr = ring_ptr + DEC_WARPS * ST * TILE_BYTES;
+  const uint32_t q_smem = smem_u32(q_ptr);
+  if (threadIdx.x == 0) {
+    abort_flag = 0;
+    for (int w = 0; w < DEC_WARPS; ++w)
+      for (int s2 = 0; s2 < ST; ++s2) mbar_init(smem_u32(&bars[w][s2]), 1);
+    fence_mbar_init();
+  }
+  pdl_wait();
+  const int L = seq_lens[b];
+  const int n_chunks = (L + KV_BLOCK - 1) / KV_BLOCK;
+  const int per = (n_chunks + num_splits - 1) / num_splits;
+  const int c_begin = split * per;
+  const int c_end = min(n_chunks, c_begin + per);
+  for (int i = threadIdx.x; i < 16 * CH; i += blockDim.x) {
+    const int r = i / CH, c = i % CH;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (r < rows) v = *reinterpret_cast<const uint4*>(proj + b * ld + (h0 + r) * D + c * 8);
+    *reinterpret_cast<uint4*>(q_ptr + swz<D>(r, c)) = v;
+  }
+  __syncthreads();
+  uint32_t qf[D / 16][4];
+  {
+    const int mat = lane >> 3, r = lane & 7;
+#pragma unroll
+    for (int ks = 0; ks < D / 16; ++ks)
+      ldsm_x4(q_smem + swz<D>((mat & 1) * 8 + r, 2 * ks + (mat >> 1)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+  }
+  float o[D / 8][4];
+#pragma unroll
+  for (int n = 0; n < D / 8; ++n) { o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f; }
+  RowState st = {-INFINITY, -INFINITY, 0.f, 0.f};
+  const float scale_log2 = scale * 1.4426950408889634f;
+  volatile int* abortp = &abort_flag;
+  const int first = c_begin + warp;
+  const int n_my = first < c_end ? (c_end - first + DEC_WARPS - 1) / DEC_WARPS : 0;
+  const int* bt_row = block_tables + (long long)b * bt_stride;
+  auto load_ids = [&](int round) {
+    const int j = round * 32 + lane;
+    return j < n_my ? __ldg(bt_row + first + j * DEC_WARPS) : 0;
+  };
+  int ids_round = 0, ids = load_ids(0), ids_next = load_ids(1);
+  auto blk_of = [&](int i) {   // all lanes, i uniform and non-decreasing
+    if ((i >> 5) > ids_round) { ids = ids_next; ids_round = i >> 5; ids_next = load_ids(ids_round + 1); }
+    return __shfl_sync(0xffffffffu, ids, i & 31);
+  };
+  auto issue = [&](int i, int blk) {   // lane 0 only
+    const int stage = i % ST;
+    if (blk < 0 || blk >= num_blocks) { set_status(status, ST_BAD_INDEX); blk = num_blocks; }  // OOB -> zeros
+    const uint32_t bar = smem_u32(&bars[warp][stage]), ks = k_smem + stage * TILE_BYTES;
+    mbar_expect_tx(bar, TILE_BYTES);
+#pragma unroll
+    for (int hx = 0; hx < D / 64; ++hx) tma_load_2d(ks + hx * (KV_BLOCK * 128), &k_map, bar, hx * 64, (blk * Hkv + kvh) * KV_BLOCK);
+  };
+  int issued = 0;
+  for (; issued < ST - 1 && issued < n_my; ++issued) {
+    const int blk = blk_of(issued);
+    if (lane == 0) issue(issued, blk);
+  }
+  bool ok = true;
+  const int mat = lane >> 3, rr = lane & 7;
+  for (int i = 0; i < n_my; ++i) {
+    if (issued < n_my) {
+      const int blk = blk_of(issued);
+      if (lane == 0) issue(issued, blk);
+      ++issued;
+    }
+    const int stage = i % ST;
+    ok = mbar_wait_bounded(smem_u32(&bars[warp][stage]), (uint32_t)((i / ST) & 1), abortp, status, ST_TIMEOUT_SMEM_FULL);
+    ok = __all_sync(0xffffffffu, ok);
+    if (!ok) break;
+    const uint32_t ks = k_smem + stage * TILE_BYTES;
+    float s0[4] = {0, 0, 0, 0}, s1[4] = {0, 0, 0, 0};
+#pragma unroll
+    for (int kk = 0; kk < D / 16; ++kk) {
+      uint32_t b0, b1, b2, b3;
+      ldsm_x4(ks + swz_tma<D>((mat >> 1) * 8 + rr, 2 * kk + (mat & 1)), b0, b1, b2, b3);
+      mma_16816(s0, qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b0, b1);
+      mma_16816(s1, qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b2, b3);
+    }
+    const int tok0 = (first + i * DEC_WARPS) * KV_BLOCK + 2 * (lane & 3);
+    if (tok0 >= L) { s0[0] = s0[2] = -INFINITY; }
+    if (tok0 + 1 >= L) { s0[1] = s0[3] = -INFINITY; }
+    if (tok0 + 8 >= L) { s1[0] = s1[2] = -INFINITY; }
+    if (tok0 + 9 >= L) { s1[1] = s1[3] = -INFINITY; }
+    uint32_t p0, p1, p2, p3;
+    softmax_update<D>(s0, s1, st, o, scale_log2, p0, p1, p2, p3);
+#pragma unroll
+    for (int dp = 0; dp < D / 16; ++dp) {
+      uint32_t b0, b1, b2, b3;
+      ldsm_x4_t(ks + swz_tma<D>((mat & 1) * 8 + rr, 2 * dp + (mat >> 1)), b0, b1, b2, b3);
+      mma_16816(o[2 * dp], p0, p1, p2, p3, b0, b1);
+      mma_16816(o[2 * dp + 1], p0, p1, p2, p3, b2, b3);
+    }
+    __syncwarp();   // every lane is done with this stage before lane 0 refills it
+  }
+  if (!ok && lane == 0) {
+    for (int j = max(0, issued - ST); j < issued; ++j) {   // no copy may land after the CTA has gone
+      const uint64_t t0 = globaltimer_ns();
+      while (!mbar_try_wait(smem_u32(&bars[warp][j % ST]), (uint32_t)((j / ST) & 1)))
+        if (globaltimer_ns() - t0 > 50000000ull) break;
+    }
+  }
+  __syncthreads();
+
+  constexpr int LD = D + KV_MERGE_LD_PAD;
+  float* mo = reinterpret_cast<float*>(ring_ptr);                   // [DEC_WARPS][16][LD]
+  float* mml = mo + DEC_WARPS * 16 * LD;                            // [DEC_WARPS][16][2]
+  const int g = lane >> 2, tq = lane & 3;
+#pragma unroll
+  for (int n = 0; n < D / 8; ++n) {
+    *reinterpret_cast<float2*>(mo + (warp * 16 + g) * LD + n * 8 + 2 * tq) = make_float2(o[n][0], o[n][1]);
+    *reinterpret_cast<float2*>(mo + (warp * 16 + g + 8) * LD + n * 8 + 2 * tq) = make_float2(o[n][2], o[n][3]);
+  }
+  if (tq == 0) {
+    mml[(warp * 16 + g) * 2] = st.m0;
+    mml[(warp * 16 + g) * 2 + 1] = st.l0;
+    mml[(warp * 16 + g + 8) * 2] = st.m1;
+    mml[(warp * 16 + g + 8) * 2 + 1] = st.l1;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < rows * D; i += blockDim.x) {
+    const int r = i / D, d = i % D, h = h0 + r;
+    float M = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < DEC_WARPS; ++w) M = fmaxf(M, mml[(w * 16 + r) * 2]);
+    float acc = 0.f, l = 0.f;
+    if (M != -INFINITY) {
+#pragma unroll
+      for (int w = 0; w < DEC_WARPS; ++w) {
+        const float e = exp2f(mml[(w * 16 + r) * 2] - M);
+        acc += e * mo[(w * 16 + r) * LD + d];
+        l += e * mml[(w * 16 + r) * 2 + 1];
+      }
+    }
+    if (num_splits == 1) {
+      float y = 0.f;
+      if (l > 0.f)
+        y = acc / (l + exp2f(sink[h] * 1.4426950408889634f - M)) * kv_sigmoid(__bfloat162float(proj[b * ld + gate_col + h * D + d]));
+      out[((long long)b * H + h) * D + d] = __float2bfloat16_rn(y);
+    } else {
+      const long long pi = ((long long)b * H + h) * num_splits + split;
+      part_o[pi * D + d] = acc;
+      if (d == 0) { part_ml[pi * 2] = M; part_ml[pi * 2 + 1] = l; }
+    }
+  }
+}
+
+template <int D>
+__global__ void kv_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const __nv_bfloat16* __restrict__ proj,
+                                       long long ld, int gate_col, const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int H,
+                                       int num_splits) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, d = threadIdx.x;
+  const long long b = blockIdx.y, bh = b * H + h;
+  float M = -INFINITY;
+  for (int s = 0; s < num_splits; ++s) M = fmaxf(M, part_ml[(bh * num_splits + s) * 2]);
+  float acc = 0.f, l = 0.f, y = 0.f;
+  if (M != -INFINITY) {
+    for (int s = 0; s < num_splits; ++s) {
+      const float e = exp2f(part_ml[(bh * num_splits + s) * 2] - M);
+      acc += e * part_o[(bh * num_splits + s) * D + d];
+      l += e * part_ml[(bh * num_splits + s) * 2 + 1];
+    }
+    y = acc / (l + exp2f(sink[h] * 1.4426950408889634f - M)) * kv_sigmoid(__bfloat162float(proj[b * ld + gate_col + h * D + d]));
+  }
+  out[bh * D + d] = __float2bfloat16_rn(y);
+}
+
+// Any head size up to 512 and either number format, a warp per (token, query head): the exact mode and sizes without a
+// tensor-core kernel. Lanes take one key each for the scores and 1/32 of the channels for the sums.
+constexpr int KVS_WARPS = 4, KVS_MAX_D = 512;
+
+template <typename T>
+__global__ void __launch_bounds__(KVS_WARPS * 32)
+kv_simple_kernel(const T* __restrict__ proj, long long ld, int gate_col, const T* __restrict__ cache, const int* __restrict__ block_tables,
+                 const int* __restrict__ cu_q, const int* __restrict__ seq_lens, const float* __restrict__ sink, T* __restrict__ out, int H, int G,
+                 int D, int bt_stride, int num_blocks, int rows, float scale, int* status) {
+  extern __shared__ float kvs_q[];       // [KVS_WARPS][D]
+  pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y, b = blockIdx.z, kvh = h / (H / G);
+  pdl_wait();
+  int t0 = b, t1 = b + 1;
+  if (cu_q != nullptr) { t0 = cu_q[b]; t1 = cu_q[b + 1]; }
+  const int t = t0 + blockIdx.x * KVS_WARPS + warp;
+  if (t >= t1) return;                                     // (no CTA-wide synchronisation below)
+  if (t >= rows) { if (lane == 0) set_status(status, ST_BAD_INDEX); return; }
+  const int n_keys = seq_lens[b] - (t1 - 1 - t);           // keys this token sees
+  T* dst = out + ((long long)t * H + h) * D;
+  if (n_keys <= 0) {
+    for (int d = lane; d < D; d += 32) kv_store(dst + d, 0.f);
+    return;
+  }
+  float* q = kvs_q + warp * D;
+  for (int d = lane; d < D; d += 32) q[d] = kv_to_f(proj[t * ld + h * D + d]) * scale;
+  __syncwarp();
+  float o[KVS_MAX_D / 32];
+#pragma unroll
+  for (int i = 0; i < KVS_MAX_D / 32; ++i) o[i] = 0.f;
+  float m = sink[h], l = 1.f;                              // the sink: a key of weight exp(sink) without a value
+  for (int k0 = 0; k0 < n_keys; k0 += 32) {
+    const int j = k0 + lane;
+    float s = -INFINITY;
+    long long row = 0;
+    if (j < n_keys) {
+      int blk = block_tables[(long long)b * bt_stride + j / KV_BLOCK];
+      if (blk < 0 || blk >= num_blocks) { set_status(status, ST_BAD_INDEX); blk = 0; }
+      row = (((long long)blk * G + kvh) * KV_BLOCK + j % KV_BLOCK) * D;
+      s = 0.f;
+      for (int d = 0; d < D; ++d) s = fmaf(q[d], kv_to_f(cache[row + d]), s);
+    }
+    const float m_new = fmaxf(m, warp_max(s));
+    const float c = expf(m - m_new), p = j < n_keys ? expf(s - m_new) : 0.f;
+    l = l * c + warp_sum(p);
+    m = m_new;
+#pragma unroll
+    for (int i = 0; i < KVS_MAX_D / 32; ++i) o[i] *= c;
+    const int n = min(32, n_keys - k0);
+    for (int u = 0; u < n; ++u) {
+      const float pu = __shfl_sync(0xffffffffu, p, u);
+      const long long ru = __shfl_sync(0xffffffffu, row, u);
+#pragma unroll
+      for (int i = 0; i < KVS_MAX_D / 32; ++i)
+        if (lane + 32 * i < D) o[i] = fmaf(pu, kv_to_f(cache[ru + lane + 32 * i]), o[i]);
+    }
+  }
+  const T* gate = proj + t * ld + gate_col + h * D;
+#pragma unroll
+  for (int i = 0; i < KVS_MAX_D / 32; ++i) {
+    const int d = lane + 32 * i;
+    if (d < D) kv_store(dst + d, o[i] / l * kv_sigmoid(kv_to_f(gate[d])));
+  }
+}
+
+// out *= sigmoid(gate) * exp(lse) / (exp(lse) + exp(sink)) for token rows [row0, row0 + n): what the plain softmax of the
+// long-portion kernel lacks.
+__global__ void kv_gate_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ lse, const float* __restrict__ sink,
+                               const __nv_bfloat16* __restrict__ gate, long long ld, int H, int D, int row0, int n, int Tq) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int vpr = H * D / 8;
+  const long long total = (long long)n * vpr;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = row0 + i / vpr;
+    const int c = (int)(i % vpr) * 8, h = c / D;
+    const float f = kv_sigmoid(lse[(long long)h * Tq + t] - sink[h]);
+    uint4* po = reinterpret_cast<uint4*>(out + t * H * D + c);
+    const uint4 g = *reinterpret_cast<const uint4*>(gate + t * ld + c);
+    uint4 v = *po;
+    auto one = [&](uint32_t x, uint32_t y) {
+      const float2 a = unpack_bf16x2(x), z = unpack_bf16x2(y);
+      return pack_bf16x2(a.x * f * kv_sigmoid(z.x), a.y * f * kv_sigmoid(z.y));
+    };
+    v.x = one(v.x, g.x); v.y = one(v.y, g.y); v.z = one(v.z, g.z); v.w = one(v.w, g.w);
+    *po = v;
+  }
+}
+
+template <int D>
+constexpr int kv_decode_smem_bytes() {
+  const int ring = DEC_WARPS * kv_dec_stages<D>() * KV_BLOCK * D * 2 + 16 * D * 2;
+  const int merge = DEC_WARPS * 16 * (D + KV_MERGE_LD_PAD + 2) * 4;
+  return 1024 + (ring > merge ? ring : merge);
+}
+
+}  // namespace rb
+
+extern "C" int rb_kv_append(void* proj, long long ld, const int* positions, const int* slots, float coef, int every, void* cache, int num_blocks,
+                            int H, int G, int D, int T, int dtype, int* status, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (every <= 0 || H <= 0 || G <= 0 || D <= 0) return -1;
+  cudaError_t e;
+  if (dtype == 0)
+    e = launch_kernel(kv_append_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, (__nv_bfloat16*)proj, ld, positions, slots, coef, every,
+                      (__nv_bfloat16*)cache, num_blocks, H, G, D, status);
+  else
+    e = launch_kernel(kv_append_kernel<float>, dim3(T), dim3(256), 0, stream, (float*)proj, ld, positions, slots, coef, every, (float*)cache,
+                      num_blocks, H, G, D, status);
+  return e == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int rb_kv_decode(const void* proj, long long ld, int gate_col, const void* cache, const int* block_tables, const int* seq_lens,
+                            const float* sink, void* out, float* workspace, int B, int H, int G, int D, int bt_stride, int num_blocks,
+                            int block_size, int num_splits, float scale, int* status, cudaStream_t stream) {
+  if (B <= 0) return 0;
+  if (block_size != KV_BLOCK || G <= 0 || H % G != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr) || B > 65535) return -1;
+  CUtensorMap kmap;
+  if (tma_map_2d_bf16(&kmap, cache, (unsigned long long)num_blocks * G * KV_BLOCK, D, D, KV_BLOCK) != 0) return -20;
+  float* part_ml = workspace != nullptr ? workspace + (long long)B * H * num_splits * D : nullptr;
+  const dim3 grid(num_splits, G * ((H / G + 15) / 16), B);
+#define LAUNCH_KV(DD)                                                                                          \
+  do {                                                                                                         \
+    static bool attr[RB_MAX_DEVICES] = {};                                                                     \
+    const int dev_ = current_device_index();                                                                   \
+    if (dev_ < 0) return -10;                                                                                  \
+    if (!attr[dev_]) {                                                                                         \
+      if (cudaFuncSetAttribute(kv_decode_kernel<DD>, cudaFuncAttributeMaxDynamicSharedMemorySize,              \
+                               kv_decode_smem_bytes<DD>()) != cudaSuccess) return -10;                         \
+      attr[dev_] = true;                                                                                       \
+    }                                                                                                          \
+    launch_kernel(kv_decode_kernel<DD>, grid, dim3(DEC_WARPS * 32), kv_decode_smem_bytes<DD>(), stream,        \
+                  (const __nv_bfloat16*)proj, ld, gate_col, kmap, block_tables, seq_lens, sink,                \
+                  (__nv_bfloat16*)out, workspace, part_ml, H, G, bt_stride, num_blocks, num_splits, scale, status); \
+    if (num_splits > 1)                                                                                        \
+      launch_kernel(kv_decode_merge_kernel<DD>, dim3(H, B), dim3(DD), 0, stream, (const float*)workspace,      \
+                    (const float*)part_ml, (const __nv_bfloat16*)proj, ld, gate_col, sink, (__nv_bfloat16*)out, H, num_splits); \
+  } while (0)
+  if (D == 64) LAUNCH_KV(64);
+  else if (D == 128) LAUNCH_KV(128);
+  else return -1;
+#undef LAUNCH_KV
+  return cudaGetLastError() == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int rb_kv_simple(const void* proj, long long ld, int gate_col, const void* cache, const int* block_tables, const int* cu_q,
+                            const int* seq_lens, const float* sink, void* out, int H, int G, int D, int bt_stride, int num_blocks, int B, int rows,
+                            int max_q, int dtype, float scale, int* status, cudaStream_t stream) {
+  if (B <= 0 || rows <= 0) return 0;
+  if (D > KVS_MAX_D || G <= 0 || H % G != 0 || H > 65535 || B > 65535) return -1;
+  const dim3 grid((max_q + KVS_WARPS - 1) / KVS_WARPS, H, B);
+  const size_t smem = (size_t)KVS_WARPS * D * 4;
+  cudaError_t e;
+  if (dtype == 0)
+    e = launch_kernel(kv_simple_kernel<__nv_bfloat16>, grid, dim3(KVS_WARPS * 32), smem, stream, (const __nv_bfloat16*)proj, ld, gate_col,
+                      (const __nv_bfloat16*)cache, block_tables, cu_q, seq_lens, sink, (__nv_bfloat16*)out, H, G, D, bt_stride, num_blocks, rows,
+                      scale, status);
+  else
+    e = launch_kernel(kv_simple_kernel<float>, grid, dim3(KVS_WARPS * 32), smem, stream, (const float*)proj, ld, gate_col, (const float*)cache,
+                      block_tables, cu_q, seq_lens, sink, (float*)out, H, G, D, bt_stride, num_blocks, rows, scale, status);
+  return e == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int rb_kv_gate(void* out, const float* lse, const float* sink, const void* gate, long long ld, int H, int D, int row0, int n, int Tq,
+                          cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (D % 8 != 0 || ld % 8 != 0) return -1;
+  long long grid = ((long long)n * (H * D / 8) + 255) / 256;
+  if (grid > 148 * 16) grid = 148 * 16;
+  return launch_kernel(kv_gate_kernel, dim3((unsigned)grid), dim3(256), 0, stream, (__nv_bfloat16*)out, lse, sink, (const __nv_bfloat16*)gate, ld,
+                       H, D, row0, n, Tq) == cudaSuccess ? 0 : -11;
+}
+
+// ------------------------------------------------------------------------------------------
 // Allocation-free variant (see attn_noalloc.h for the contract and for who needs it).
 // ------------------------------------------------------------------------------------------
 #include "attn_noalloc.h"

@@ -11,6 +11,8 @@
 //                ids, positions, slot mapping, block tables and sampling rows straight into
 //                pinned host buffers. Prompts can be prefilled in portions (prefill_chunk), and
 //                callers can feed given tokens instead of sampling them (rbe_open / rbe_feed).
+//   StateSlots   for models with recurrent layers: one slot of fixed size per admitted sequence,
+//                taken with its first blocks and given back with them
 //
 // Behaviour it reproduces: rollouts/inference/scheduler.py:15-84 (policy),
 // rollouts/inference/cache/paged.py:57-203 (block table + prefix hits),
@@ -67,6 +69,27 @@ struct BlockPool {
     unlink(b);
     return b;
   }
+};
+
+// ------------------------------------------------------------------------------------------
+// Slots of the recurrent state. A slot is not cleared when it changes hands: a sequence whose first new token is at
+// position 0 starts from zero in the kernels.
+struct StateSlots {
+  std::vector<int> free_list;    // taken from the back
+  int total = 0;
+  void reset(int n) {
+    total = n;
+    free_list.clear();
+    for (int i = n - 1; i >= 0; --i) free_list.push_back(i);
+  }
+  bool available() const { return total == 0 || !free_list.empty(); }
+  int take() {
+    if (free_list.empty()) return -1;
+    int s = free_list.back();
+    free_list.pop_back();
+    return s;
+  }
+  void give(int s) { if (s >= 0) free_list.push_back(s); }
 };
 
 // ------------------------------------------------------------------------------------------
@@ -279,6 +302,7 @@ struct Seq {
   int n_target = 0;               // tokens whose KV will be in the cache after the scheduled step
   int n_cached = 0;               // prefix tokens served from the cache at the last admission
   std::vector<int> blocks;
+  int slot = -1;                  // recurrent state (models that keep one)
   RadixNode* radix_node = nullptr;
   uint64_t chain = 0;             // hash chain over full blocks (hash mode)
   int n_hashed_blocks = 0;
@@ -294,6 +318,7 @@ struct Seq {
 
 struct EngineCore {
   KVManager kv;
+  StateSlots slots;               // empty for models without recurrent layers
   int max_batch, max_tokens_per_batch, max_model_len;
   int prefill_chunk = 0;          // > 0: a prompt enters the cache at most this many tokens per step
   bool short_first = false;
@@ -325,6 +350,8 @@ struct EngineCore {
     }
     for (int i = (int)s->blocks.size() - 1; i >= 0; --i) kv.unref(s->blocks[i]);
     s->blocks.clear();
+    slots.give(s->slot);
+    s->slot = -1;
     s->n_computed = 0;
     s->n_hashed_blocks = 0;
     s->chain = 0;
@@ -334,6 +361,7 @@ struct EngineCore {
   // admission; the scheduler budgets with the conservative full count like the reference.
   // `budget`: tokens this step still has room for (portions only).
   bool admit(Seq* s, int budget = 1 << 30) {
+    if (!slots.available()) return false;
     const int bs = kv.pool.block_size;
     const int n = (int)s->tokens.size();
     const int need = (n + bs - 1) / bs;
@@ -366,6 +394,7 @@ struct EngineCore {
       }
       s->blocks.push_back(b);
     }
+    s->slot = slots.take();
     s->n_cached = matched * bs;
     s->n_computed = matched * bs;
     s->n_target = s->n_computed + portion(n - s->n_computed, budget);
@@ -548,6 +577,9 @@ void rbe_set_prefill(void* h, int n, int short_first) {
   e->short_first = short_first != 0;
 }
 
+// Models with recurrent layers: n slots (at most n sequences admitted at a time; none may be admitted yet).
+void rbe_set_state_slots(void* h, int n) { static_cast<EngineCore*>(h)->slots.reset(n); }
+
 // ---- externally driven sequences -----------------------------------------------------------
 // A fed sequence gets its tokens from the caller, portion by portion; it uses the same block pool and the same batch
 // builder as the scheduled ones, and is released with rbe_abort.
@@ -562,29 +594,32 @@ i64 rbe_open(void* h) {
 }
 // Appends counts[i] tokens to sequence ids[i] and makes the n sequences the scheduled batch: those that continue with
 // a single token are its decode rows, the others its prefill rows. Blocks are taken from the pool. Returns the number
-// of packed tokens, or -1 unknown sequence, -2 out of blocks, -3 over max_batch / max_tokens_per_batch / max_model_len;
-// after an error nothing has changed.
+// of packed tokens, or -1 unknown sequence, -2 out of blocks, -3 over max_batch / max_tokens_per_batch / max_model_len,
+// -4 out of state slots; after an error nothing has changed.
 int rbe_feed(void* h, const i64* ids, const int* counts, int n, const int* tokens) {
   auto* e = static_cast<EngineCore*>(h);
   const int bs = e->kv.pool.block_size;
   if (n > e->max_batch) return -3;
-  int total = 0, need = 0;
+  int total = 0, need = 0, need_slots = 0;
   for (int i = 0; i < n; ++i) {
     Seq* s = e->get(ids[i]);
     if (s == nullptr || s->status != FED || counts[i] <= 0) return -1;
     const int len = (int)s->tokens.size() + counts[i];
     if (len > e->max_model_len) return -3;
     need += (len + bs - 1) / bs - (int)s->blocks.size();
+    need_slots += s->slot < 0;
     total += counts[i];
   }
   if (total > e->max_tokens_per_batch) return -3;
   if (need > e->kv.num_free()) return -2;
+  if (e->slots.total > 0 && need_slots > (int)e->slots.free_list.size()) return -4;
   e->sched_prefill.clear(); e->sched_decode.clear(); e->sched_preempted.clear();
   for (int i = 0; i < n; ++i) {
     Seq* s = e->get(ids[i]);
     s->tokens.insert(s->tokens.end(), tokens, tokens + counts[i]);
     tokens += counts[i];
     s->n_prompt = s->n_target = (int)s->tokens.size();
+    if (s->slot < 0) s->slot = e->slots.take();
     while ((int)s->blocks.size() * bs < s->n_target) s->blocks.push_back(e->kv.take_block());
     if (counts[i] == 1 && s->n_computed > 0) e->sched_decode.push_back(s->id);
     else e->sched_prefill.push_back(s->id);
@@ -675,6 +710,12 @@ int rbe_build_batch(void* h, int which, int* tokens, int* positions, int* slots,
   return t;
 }
 
+// State slots of the rows of a batch, in the order of rbe_build_batch (-1: the model keeps no state).
+void rbe_batch_slots(void* h, int which, int* out) {
+  auto* e = static_cast<EngineCore*>(h);
+  for (i64 id : e->batch_order(which)) *out++ = e->get(id)->slot;
+}
+
 // Appends the sampled token of every row of the decode (which = 1), prefill (which = 2) or joint
 // (which = 3) batch, except rows whose prompt is not complete yet, publishes blocks that just filled up to the prefix index, and applies the stop
 // rules. Returns the number of sequences that finished.
@@ -758,7 +799,7 @@ void rbe_stats(void* h, i64* stats) {
 }
 
 // Allocator invariants: every refcount >= 0, a block is on the free list iff refcount == 0,
-// and free + referenced == total. Returns 0 when they hold.
+// and free + referenced == total; every state slot is free or held by exactly one sequence. Returns 0 when they hold.
 int rbe_check_invariants(void* h) {
   auto* e = static_cast<EngineCore*>(h);
   const BlockPool& p = e->kv.pool;
@@ -770,6 +811,13 @@ int rbe_check_invariants(void* h) {
   }
   if (free_n != p.free_count) return 3;
   if (free_n + used != p.num_blocks) return 4;
+  std::vector<char> seen(e->slots.total, 0);
+  int held = 0;
+  auto once = [&](int s) { return s >= 0 && s < e->slots.total && !seen[s]++; };
+  for (int s : e->slots.free_list) if (!once(s)) return 5;
+  for (auto& kv : e->seqs)
+    if (kv.second->slot >= 0) { if (!once(kv.second->slot)) return 6; ++held; }
+  if (held + (int)e->slots.free_list.size() != e->slots.total) return 7;
   return 0;
 }
 

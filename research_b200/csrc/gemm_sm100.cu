@@ -1390,7 +1390,7 @@ extern "C" int rb_gemm_bf16_ex(const RbGemmArgs* a, cudaStream_t stream) {
   }
   if (p.swiglu) {
     if (a->bn < 64 || a->N % a->bn != 0 || a->b_parts != 1 || a->out_f32 || p.epi_mode != RB_EPI_STORE || a->bias ||
-        a->residual || a->tile_table)
+        a->residual || (a->tile_table && (a->group_mode != 0 || a->row_dst || a->group_n % a->bn != 0)))
       return -1;
   }
   if (p.tile_table != nullptr) {

@@ -27,11 +27,13 @@ constexpr int MAX_E_PER_LANE = 8;  // up to 256 experts
 // n_group > 1 (sigmoid router only): group-limited routing. Experts form n_group contiguous groups, a group scores
 // the sum of its two best choice values, the topk_group best groups stay eligible and the choice values of the
 // other experts become 0 (glm4_moe_functional.py:278-301).
-__global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int T, int E,
+__global__ void moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ bias, int T, int E,
                                  int k, int sigmoid_router, int norm_topk, float scaling, int* __restrict__ topk_idx,
                                  float* __restrict__ topk_w, int* __restrict__ counts /*[E] histogram, may be null*/,
                                  int n_group, int topk_group) {
   __shared__ int hist[256];
+  pdl_launch_dependents();
+  pdl_wait();
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (counts != nullptr) {
@@ -44,7 +46,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
   float mx = -INFINITY;
   for (int i = 0; i < per; ++i) {
     const int e = lane + 32 * i;
-    const float x = e < E ? logits[(long long)t * E + e] : -INFINITY;
+    const float x = e < E ? logits[t * ld + e] : -INFINITY;
     score[i] = x;
     mx = fmaxf(mx, x);
   }
@@ -157,8 +159,11 @@ __global__ void moe_plan_kernel(const int* __restrict__ counts_all, int world, i
                                 int* __restrict__ expert_offset /*[E_local+1]*/, int n_gu, int bn_gu,
                                 int4* __restrict__ tiles_gu, int* __restrict__ ntiles_gu, int n_dn, int bn_dn,
                                 int4* __restrict__ tiles_dn, int* __restrict__ ntiles_dn, int max_tiles,
-                                int* status, int rank, int* __restrict__ cursor /*[2E] or null: [E..2E) = send bases*/) {
+                                int* status, int rank, int* __restrict__ cursor /*[2E] or null: [E..2E) = send bases*/,
+                                int* clear /*world = 1: counts_all itself, zeroed for the next histogram (else null)*/) {
   __shared__ int cnt[256], off[257], tb_gu[257], tb_dn[257];
+  pdl_launch_dependents();
+  pdl_wait();
   const int EL = e_hi - e_lo;
   if (cursor != nullptr) {
     // where this rank's rows for expert e start in the owner's expert-ordered receive buffer: the rows of the
@@ -201,6 +206,8 @@ __global__ void moe_plan_kernel(const int* __restrict__ counts_all, int world, i
     *ntiles_gu = tg; *ntiles_dn = td;
   }
   __syncthreads();
+  if (clear != nullptr)
+    for (int e = threadIdx.x; e < E; e += blockDim.x) { clear[e] = 0; cursor[e] = 0; }
   for (int i = threadIdx.x; i <= EL; i += blockDim.x) expert_offset[i] = off[i];
   const int ngu = (n_gu + bn_gu - 1) / bn_gu, ndn = (n_dn + bn_dn - 1) / bn_dn;
   for (int i = threadIdx.x; i < EL; i += blockDim.x) {
@@ -231,6 +238,29 @@ __global__ void moe_count_kernel(const int* __restrict__ topk_idx, int n, int E,
   __syncthreads();
   for (int i = threadIdx.x; i < E; i += blockDim.x)
     if (h[i]) atomicAdd(&counts[i], h[i]);
+}
+
+// Local dispatch: row (t, j) of any 16-byte-multiple width to the next free row of its expert's block (cursor as left by the
+// plan), and the address its result goes to. One warp per pair.
+__global__ void moe_gather_rows_kernel(const uint4* __restrict__ x, long long ld_vec, const int* __restrict__ topk_idx, int n_pairs, int k,
+                                       int row_vec, int E, int* __restrict__ cursor, uint4* __restrict__ xp,
+                                       unsigned long long* __restrict__ ret, unsigned long long y, long long y_row_bytes, int cap,
+                                       int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int i = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (i >= n_pairs) return;
+  const int e = topk_idx[i];
+  if (e < 0 || e >= E) { set_status(status, ST_BAD_INDEX); return; }
+  int pos = 0;
+  if (lane == 0) pos = cursor[E + e] + atomicAdd(&cursor[e], 1);
+  pos = __shfl_sync(0xffffffffu, pos, 0);
+  if (pos < 0 || pos >= cap) { set_status(status, ST_BAD_INDEX); return; }
+  const uint4* src = x + (long long)(i / k) * ld_vec;
+  uint4* dst = xp + (long long)pos * row_vec;
+  for (int v = lane; v < row_vec; v += 32) dst[v] = src[v];
+  if (lane == 0) ret[pos] = y + (unsigned long long)i * (unsigned long long)y_row_bytes;
 }
 
 struct PeerPtrs { void* p[RB_MAX_RANKS]; };
@@ -535,7 +565,7 @@ extern "C" int rb_moe_route(const float* logits, const float* bias, int T, int E
                             int norm_topk, float scaling, int* topk_idx, float* topk_w, cudaStream_t s) {
   if (T <= 0) return 0;
   if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E) return -1;
-  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, bias, T, E, k, sigmoid_router, norm_topk, scaling, topk_idx, topk_w, nullptr, 1, 1);
+  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, E, bias, T, E, k, sigmoid_router, norm_topk, scaling, topk_idx, topk_w, nullptr, 1, 1);
   return RB_OK();
 }
 // Routing plus the per-expert histogram of the choices (added into counts[E], which the caller zeroes).
@@ -543,7 +573,7 @@ extern "C" int rb_moe_route_count(const float* logits, const float* bias, int T,
                                   int norm_topk, float scaling, int* topk_idx, float* topk_w, int* counts, cudaStream_t s) {
   if (T <= 0) return 0;
   if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E || counts == nullptr) return -1;
-  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, bias, T, E, k, sigmoid_router, norm_topk, scaling, topk_idx, topk_w, counts, 1, 1);
+  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, E, bias, T, E, k, sigmoid_router, norm_topk, scaling, topk_idx, topk_w, counts, 1, 1);
   return RB_OK();
 }
 // The same with group-limited routing (n_group groups of E / n_group >= 2 experts, topk_group of them eligible).
@@ -554,7 +584,7 @@ extern "C" int rb_moe_route_groups(const float* logits, const float* bias, int T
   if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E) return -1;
   if (n_group < 1 || n_group > 32 || topk_group < 1 || topk_group > n_group || E % n_group != 0) return -1;
   if (n_group > 1 && E / n_group < 2) return -1;
-  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, bias, T, E, k, 1, norm_topk, scaling, topk_idx, topk_w, counts, n_group,
+  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, E, bias, T, E, k, 1, norm_topk, scaling, topk_idx, topk_w, counts, n_group,
                                                topk_group);
   return RB_OK();
 }
@@ -576,7 +606,7 @@ extern "C" int rb_moe_plan(const int* counts_all, int world, int E, int e_lo, in
                            int* ntiles_dn, int max_tiles, int* status, cudaStream_t s) {
   if (e_hi - e_lo > 256 || e_hi <= e_lo) return -1;
   moe_plan_kernel<<<1, 256, 0, s>>>(counts_all, world, E, e_lo, e_hi, expert_offset, n_gu, bn_gu, (int4*)tiles_gu,
-                                    ntiles_gu, n_dn, bn_dn, (int4*)tiles_dn, ntiles_dn, max_tiles, status, 0, nullptr);
+                                    ntiles_gu, n_dn, bn_dn, (int4*)tiles_dn, ntiles_dn, max_tiles, status, 0, nullptr, nullptr);
   return RB_OK();
 }
 // The same plus the dispatch bases of rb_moe_permute_planned (cursor[E..2E)).
@@ -585,7 +615,7 @@ extern "C" int rb_moe_plan_dispatch(const int* counts_all, int world, int E, int
                                     int* ntiles_dn, int max_tiles, int* status, int rank, int* cursor, cudaStream_t s) {
   if (e_hi - e_lo > 256 || e_hi <= e_lo || E % world != 0 || cursor == nullptr) return -1;
   moe_plan_kernel<<<1, 256, 0, s>>>(counts_all, world, E, e_lo, e_hi, expert_offset, n_gu, bn_gu, (int4*)tiles_gu,
-                                    ntiles_gu, n_dn, bn_dn, (int4*)tiles_dn, ntiles_dn, max_tiles, status, rank, cursor);
+                                    ntiles_gu, n_dn, bn_dn, (int4*)tiles_dn, ntiles_dn, max_tiles, status, rank, cursor, nullptr);
   return RB_OK();
 }
 extern "C" int rb_moe_permute(const void* x, const int* topk_idx, int T, int k, int d, int E, int world, int rank,
@@ -627,6 +657,33 @@ extern "C" int rb_moe_combine(const void* y, const float* w, int T, int k, int d
   if (grid > 148 * 8) grid = 148 * 8;
   moe_combine_kernel<<<(unsigned)grid, 256, 0, s>>>((const __nv_bfloat16*)y, w, T, k, d, (__nv_bfloat16*)out, accumulate);
   return RB_OK();
+}
+
+// ---------------------------------------------------------------- local expert layer of layer-stack models (ops/experts.py)
+extern "C" void rb_moe_set_pdl(int on) { rb::pdl_enabled() = on != 0; }
+
+// Softmax router on logits with a row stride, chosen scores divided by their sum, histogram added into counts.
+extern "C" int rb_experts_route(const float* logits, long long ld, int T, int E, int k, int* topk_idx, float* topk_w, int* counts,
+                                cudaStream_t s) {
+  if (T <= 0) return 0;
+  if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E || counts == nullptr) return -1;
+  return launch_kernel(moe_route_kernel, dim3((T + 7) / 8), dim3(256), 0, s, logits, ld, nullptr, T, E, k, 0, 1, 1.f, topk_idx, topk_w, counts,
+                       1, 1) == cudaSuccess ? 0 : -11;
+}
+// Offsets, tile tables and dispatch bases from the histogram, which is zeroed again.
+extern "C" int rb_experts_plan(int* counts, int E, int* expert_offset, int n_gu, int bn_gu, void* tiles_gu, int* ntiles_gu, int n_dn, int bn_dn,
+                               void* tiles_dn, int* ntiles_dn, int max_tiles, int* cursor, int* status, cudaStream_t s) {
+  if (E > 256 || E <= 0 || cursor == nullptr) return -1;
+  return launch_kernel(moe_plan_kernel, dim3(1), dim3(256), 0, s, counts, 1, E, 0, E, expert_offset, n_gu, bn_gu, (int4*)tiles_gu, ntiles_gu,
+                       n_dn, bn_dn, (int4*)tiles_dn, ntiles_dn, max_tiles, status, 0, cursor, counts) == cudaSuccess ? 0 : -11;
+}
+extern "C" int rb_experts_gather(const void* x, long long ld_bytes, const int* topk_idx, int T, int k, int row_bytes, int E, int* cursor, void* xp,
+                                 void* ret, void* y, long long y_row_bytes, int cap, int* status, cudaStream_t s) {
+  if (T <= 0) return 0;
+  if (ld_bytes % 16 != 0 || row_bytes % 16 != 0) return -1;
+  const int n = T * k;
+  return launch_kernel(moe_gather_rows_kernel, dim3((n + 7) / 8), dim3(256), 0, s, (const uint4*)x, ld_bytes / 16, topk_idx, n, k, row_bytes / 16, E,
+                       cursor, (uint4*)xp, (unsigned long long*)ret, (unsigned long long)y, y_row_bytes, cap, status) == cudaSuccess ? 0 : -11;
 }
 
 // ---------------------------------------------------------------- training (expert-grouped rows, padded to 64)

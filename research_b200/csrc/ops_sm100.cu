@@ -270,19 +270,108 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return t;
 }
 
+// Embedding row into the fp32 stream and up to two copies of it in the activation type (all strides in elements).
 template <typename TA>
-__global__ void embed_residual_kernel(const int* __restrict__ ids, const TA* __restrict__ table, float* __restrict__ x,
-                                      TA* __restrict__ xb, int d, long long ldb, int vocab, int* status) {
+__global__ void stream_embed_kernel(const int* __restrict__ ids, const TA* __restrict__ table, long long ldt, float* __restrict__ x,
+                                    long long ldx, TA* __restrict__ a, long long lda, TA* __restrict__ b, long long ldb, int d, int vocab,
+                                    int* status) {
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x;
   int id = ids[t];
   if (id < 0 || id >= vocab) { if (threadIdx.x == 0) set_status(status, ST_BAD_INDEX); id = 0; }
-  const TA* src = table + (long long)id * ldb;
+  const TA* src = table + (long long)id * ldt;
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     const TA v = src[c];
-    x[t * d + c] = from_act(v);
-    xb[t * ldb + c] = v;
+    x[t * ldx + c] = from_act(v);
+    if (a != nullptr) a[t * lda + c] = v;
+    if (b != nullptr) b[t * ldb + c] = v;
+  }
+}
+
+__device__ __forceinline__ float4 load_act4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load_act4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = unpack_bf16x2(u.x), hi = unpack_bf16x2(u.y);
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+__device__ __forceinline__ void store_act4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_act4(__nv_bfloat16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+// One pass over the fp32 residual stream between two layers, a CTA per row:
+//   x += y1 + y2 + sum_j w[j] e[row * k + j]     (absent terms are null; nothing is written back when all are)
+//   copy = x in the activation type,  h = x / rms(x) * weight
+// rows != null: h[i] comes from row rows[i] (no update). Columns are padded to a multiple of 4 with zeros.
+struct StreamNormParams {
+  float* x;
+  long long ldx;
+  const float* y1;
+  const float* y2;
+  long long ldy;
+  const void* e;
+  const float* w;
+  long long lde;
+  int k;
+  void* copy;
+  long long ldc;
+  void* h;
+  long long ldh;
+  const float* weight;
+  const int* rows;
+  int num_src_rows, d, dp;
+  float eps;
+  int* status;
+};
+
+template <typename TA>
+__global__ void __launch_bounds__(256) stream_norm_kernel(const StreamNormParams p) {
+  extern __shared__ float4 sn_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long r = blockIdx.x;
+  long long xr = r;
+  if (p.rows != nullptr) {
+    xr = p.rows[r];
+    if (xr < 0 || xr >= p.num_src_rows) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); xr = 0; }
+  }
+  float* x = p.x + xr * p.ldx;
+  const bool update = p.y1 != nullptr || p.y2 != nullptr || p.e != nullptr;
+  const TA* e = reinterpret_cast<const TA*>(p.e) + r * p.k * p.lde;
+  float ss = 0.f;
+  for (int c = threadIdx.x * 4; c < p.dp; c += blockDim.x * 4) {
+    float4 v = *reinterpret_cast<const float4*>(x + c);
+    if (p.y1 != nullptr) {
+      const float4 y = *reinterpret_cast<const float4*>(p.y1 + r * p.ldy + c);
+      v.x += y.x; v.y += y.y; v.z += y.z; v.w += y.w;
+    }
+    if (p.y2 != nullptr) {
+      const float4 y = *reinterpret_cast<const float4*>(p.y2 + r * p.ldy + c);
+      v.x += y.x; v.y += y.y; v.z += y.z; v.w += y.w;
+    }
+    if (p.e != nullptr) {
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int j = 0; j < p.k; ++j) {
+        const float w = __ldg(p.w + r * p.k + j);
+        const float4 y = load_act4(e + j * p.lde + c);
+        a.x = fmaf(w, y.x, a.x); a.y = fmaf(w, y.y, a.y); a.z = fmaf(w, y.z, a.z); a.w = fmaf(w, y.w, a.w);
+      }
+      v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+    }
+    if (update) *reinterpret_cast<float4*>(x + c) = v;
+    if (p.copy != nullptr) store_act4(reinterpret_cast<TA*>(p.copy) + r * p.ldc + c, v);
+    sn_row[c >> 2] = v;
+    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  if (p.h == nullptr) return;
+  const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)p.d + p.eps);
+  TA* h = reinterpret_cast<TA*>(p.h) + r * p.ldh;
+  for (int c = threadIdx.x * 4; c < p.dp; c += blockDim.x * 4) {
+    const float4 v = sn_row[c >> 2];
+    const float4 w = *reinterpret_cast<const float4*>(p.weight + c);
+    store_act4(h + c, make_float4(v.x * rs * w.x, v.y * rs * w.y, v.z * rs * w.z, v.w * rs * w.w));
   }
 }
 
@@ -291,7 +380,8 @@ __global__ void embed_residual_kernel(const int* __restrict__ ids, const TA* __r
 //   otherwise    : x += LN(y) * w + b, out = x                      (norm on the sublayer's output, residual add)
 // The caller folds a layer scale into w and b.
 template <typename TA>
-__global__ void layernorm_kernel(const float* __restrict__ y, long long ldy, float* __restrict__ x, const int* __restrict__ rows,
+__global__ void layernorm_kernel(const float* __restrict__ y, long long ldy, float* __restrict__ x, long long ldx,
+                                 const int* __restrict__ rows,
                                  const float* __restrict__ w, const float* __restrict__ b, TA* __restrict__ out, long long ldo,
                                  int d, float eps, int num_src_rows, int* status) {
   extern __shared__ float ln_row[];
@@ -304,7 +394,7 @@ __global__ void layernorm_kernel(const float* __restrict__ y, long long ldy, flo
     xr = rows[r];
     if (xr < 0 || xr >= num_src_rows) { if (threadIdx.x == 0) set_status(status, ST_BAD_INDEX); xr = 0; }
   }
-  const float* src = y != nullptr ? y + r * ldy : x + xr * d;
+  const float* src = y != nullptr ? y + r * ldy : x + xr * ldx;
   float s = 0.f;
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     const float v = src[c];
@@ -321,8 +411,8 @@ __global__ void layernorm_kernel(const float* __restrict__ y, long long ldy, flo
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     float v = fmaf((ln_row[c] - mean) * rstd, w[c], b[c]);
     if (y != nullptr) {
-      v += x[r * d + c];
-      x[r * d + c] = v;
+      v += x[r * ldx + c];
+      x[r * ldx + c] = v;
     }
     out[r * ldo + c] = to_act<TA>(v);
   }
@@ -673,21 +763,33 @@ extern "C" int rb_transpose_bf16(const void* in, void* out, int rows, int cols, 
   else if ((dtype) == 1) { using TA = float; CALL }    \
   else return -1;
 
-extern "C" int rb_embed_residual(const int* ids, const void* table, float* x, void* xb, int dtype, int T, int d, long long ldb,
-                                 int vocab, int* status, cudaStream_t stream) {
-  if (T <= 0 || d <= 0 || ldb < d) return -1;
+extern "C" int rb_stream_embed(const int* ids, const void* table, long long ldt, float* x, long long ldx, void* a, long long lda, void* b,
+                               long long ldb, int dtype, int T, int d, int vocab, int* status, cudaStream_t stream) {
+  if (T <= 0 || d <= 0) return -1;
   cudaError_t e;
-  RB_ACT_DISPATCH(dtype, e = launch_kernel(embed_residual_kernel<TA>, dim3(T), dim3(256), 0, stream, ids, (const TA*)table, x,
-                                           (TA*)xb, d, ldb, vocab, status);)
+  RB_ACT_DISPATCH(dtype, e = launch_kernel(stream_embed_kernel<TA>, dim3(T), dim3(256), 0, stream, ids, (const TA*)table, ldt, x, ldx, (TA*)a,
+                                           lda, (TA*)b, ldb, d, vocab, status);)
   return e == cudaSuccess ? 0 : -11;
 }
 
-extern "C" int rb_layernorm(const float* y, long long ldy, float* x, const int* rows, const float* w, const float* b, void* out,
+extern "C" int rb_stream_norm(float* x, long long ldx, const float* y1, const float* y2, long long ldy, const void* e, const float* w,
+                              long long lde, int k, void* copy, long long ldc, void* h, long long ldh, const float* weight, const int* rows,
+                              int num_src_rows, int dtype, int n, int d, int dp, float eps, int* status, cudaStream_t stream) {
+  const bool update = y1 != nullptr || y2 != nullptr || e != nullptr;
+  if (n <= 0 || d <= 0 || dp < d || dp % 4 != 0 || dp > 12288 || (rows != nullptr && update) || (ldx | ldy | lde | ldc | ldh) % 4 != 0) return -1;
+  const StreamNormParams p{x, ldx, y1, y2, ldy, e, w, lde, k, copy, ldc, h, ldh, weight, rows, num_src_rows, d, dp, eps, status};
+  const int threads = dp <= 512 ? 128 : 256;
+  cudaError_t err;
+  RB_ACT_DISPATCH(dtype, err = launch_kernel(stream_norm_kernel<TA>, dim3(n), dim3(threads), (size_t)dp * 4, stream, p);)
+  return err == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int rb_layernorm(const float* y, long long ldy, float* x, long long ldx, const int* rows, const float* w, const float* b, void* out,
                             long long ldo, int dtype, int n, int d, float eps, int num_src_rows, int* status, cudaStream_t stream) {
   if (n <= 0 || d <= 0 || d > 12288 || ldo < d || (y != nullptr && rows != nullptr)) return -1;
   const int threads = d <= 512 ? 128 : 256;
   cudaError_t e;
-  RB_ACT_DISPATCH(dtype, e = launch_kernel(layernorm_kernel<TA>, dim3(n), dim3(threads), (size_t)d * 4, stream, y, ldy, x, rows, w, b,
+  RB_ACT_DISPATCH(dtype, e = launch_kernel(layernorm_kernel<TA>, dim3(n), dim3(threads), (size_t)d * 4, stream, y, ldy, x, ldx, rows, w, b,
                                            (TA*)out, ldo, d, eps, num_src_rows, status);)
   return e == cudaSuccess ? 0 : -11;
 }

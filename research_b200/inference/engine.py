@@ -40,6 +40,8 @@ def _core_lib():
         lib.rbe_add_request.restype = _LL
         lib.rbe_add_request.argtypes = [_VP, _VP, _I, _I, _F, _ULL, _VP, _I, _I]
         lib.rbe_set_prefill.argtypes = [_VP, _I, _I]
+        lib.rbe_set_state_slots.argtypes = [_VP, _I]
+        lib.rbe_batch_slots.argtypes = [_VP, _I, _VP]
         lib.rbe_open.restype = _LL
         lib.rbe_open.argtypes = [_VP]
         lib.rbe_feed.argtypes = [_VP, _VP, _VP, _I, _VP]
@@ -92,6 +94,9 @@ class InferenceEngine:
             raise ValueError(f"{runner_type.__name__} has no 32-bit mode on the GPU")
         dtype = torch.bfloat16 if on_gpu and config.dtype == "bfloat16" else torch.float32
         self.runner_type = runner_type
+        # sequences with recurrent state cannot start from cached blocks alone, so such models share no prefixes
+        self.state_slots = config.max_batch_size if runner_type.state_bytes_per_slot(model_config, dtype) > 0 else 0
+        self.cache_type = "none" if self.state_slots else config.cache_type
         num_blocks = config.num_kv_blocks or self._size_kv_cache(model_config, tp, ep, dtype)
         self.runner = runner_type(
             model_config, weights, device=self.device, num_kv_blocks=num_blocks, max_batch=config.max_batch_size,
@@ -103,11 +108,12 @@ class InferenceEngine:
         self.peers_pending = False
         self.idle_passes = 0
         self._lib = _core_lib()
-        self._core = self._lib.rbe_create(num_blocks, BLOCK, _CACHE_MODES[config.cache_type], config.max_batch_size,
+        self._core = self._lib.rbe_create(num_blocks, BLOCK, _CACHE_MODES[self.cache_type], config.max_batch_size,
                                           self.max_tokens_per_batch, config.max_model_len)
         assert self._core, "engine core allocation failed"
         # runners that take portions beside decoded tokens get long prompts in pieces that fit a step
         chunk = config.prefill_chunk or (self.max_tokens_per_batch if runner_type.joint_steps else 0)
+        self._lib.rbe_set_state_slots(self._core, self.state_slots)
         self._lib.rbe_set_prefill(self._core, chunk, int(runner_type.short_first))
         self.num_kv_blocks = num_blocks
         self.weight_version = 0
@@ -128,7 +134,7 @@ class InferenceEngine:
     # ---------------------------------------------------------------- sizing
     def _size_kv_cache(self, cfg: ModelConfig | LayerStackConfig, tp, ep=None, dtype: torch.dtype = torch.bfloat16) -> int:
         tp_size = tp.world if tp is not None else 1
-        per_block = self.runner_type.cache_bytes_per_block(cfg, tp_size, dtype)
+        per_block = max(self.runner_type.cache_bytes_per_block(cfg, tp_size, dtype), 1)     # (0: recurrent layers only)
         want_tokens = self.config.max_batch_size * self.config.max_model_len
         want = -(-want_tokens // BLOCK)
         if self.device.type == "cuda":
@@ -138,7 +144,8 @@ class InferenceEngine:
                 experts = (cfg.num_layers - cfg.first_k_dense_replace) * cfg.num_experts * 3 * cfg.hidden_size * cfg.moe_intermediate_size
                 params -= experts - experts // ep.world
             weights_bytes = params * 2 // tp_size
-            budget = int(free * self.config.gpu_memory_utilization) - weights_bytes - (4 << 30)
+            state_bytes = self.state_slots * self.runner_type.state_bytes_per_slot(cfg, dtype)
+            budget = int(free * self.config.gpu_memory_utilization) - weights_bytes - state_bytes - (4 << 30)
             cap = max(budget // per_block, 64)
             return int(max(64, min(want, cap, (48 << 30) // per_block)))
         return int(min(want, 4096))
@@ -249,6 +256,7 @@ class InferenceEngine:
             self._core, 1, base, base + 4 * mb, base + 8 * mb, pf + 4 * o["cu_q"], base + 12 * mb, r.bt_host.data_ptr(),
             r.max_blocks_per_seq, base + 16 * mb, base + 20 * mb, pf + 4 * o["sample_rows"], mb, mb)
         assert T == n, T
+        self._lib.rbe_batch_slots(self._core, 1, base + 28 * mb)
         max_blocks = self._max_blocks_in(r.meta_host[3 * mb:3 * mb + n])
         r.stage_decode_padding(n)
         r.decode(n, max_blocks)
@@ -262,6 +270,7 @@ class InferenceEngine:
             self._core, which, base + 4 * o["tokens"], base + 4 * o["positions"], base + 4 * o["slots"], base + 4 * o["cu_q"],
             base + 4 * o["seq_lens"], r.bt_host.data_ptr(), r.max_blocks_per_seq, base + 4 * o["temps"],
             base + 4 * o["seeds"], base + 4 * o["sample_rows"], r.max_prefill_tokens, r.max_batch)
+        self._lib.rbe_batch_slots(self._core, which, base + 4 * o["state_slots"])
         assert T > 0, f"packed batch does not fit the staging buffers ({T})"
         cu = r.pf_host[o["cu_q"]:o["cu_q"] + n_rows + 1]
         return n_rows, T, int((cu[1:] - cu[:-1]).max()), self._max_blocks_in(r.pf_host[o["seq_lens"]:o["seq_lens"] + n_rows])
@@ -283,7 +292,7 @@ class InferenceEngine:
         rc = lib.rbe_feed(core, (_LL * n)(*[e[0] for e in entries]), (_I * n)(*[len(e[1]) for e in entries]), n, (_I * len(flat))(*flat))
         if rc < 0:
             raise RuntimeError({-1: "feed: unknown stream or an entry without tokens", -2: "feed: the KV cache is full",
-                                -3: "feed: more tokens than the engine was made for"}[rc])
+                                -3: "feed: more tokens than the engine was made for", -4: "feed: every state slot is taken"}[rc])
         pre, dec = (_LL * n)(), (_LL * n)()
         n_dec = lib.rbe_get_scheduled(core, pre, dec, None)
         order = list(dec[:n_dec]) + list(pre[:n - n_dec])

@@ -56,6 +56,12 @@ class PackedBatch:
     block_tables: torch.Tensor
     host_cu_q: list[int]
     host_seq_lens: list[int]
+    state_slots: torch.Tensor | None = None      # recurrent state of every sequence
+    n_single: int = 0                            # leading sequences with one new token each
+
+
+def leading_singles(cu_q: list[int]) -> int:
+    return next((i for i in range(len(cu_q) - 1) if cu_q[i + 1] - cu_q[i] != 1), len(cu_q) - 1)
 
 
 class RunnerBase:
@@ -72,10 +78,15 @@ class RunnerBase:
     joint_steps = False          # decode rows and prompt portions of a step run as one packed batch
     short_first = False          # wants the packed batch ordered by portion length
 
+    @staticmethod
+    def state_bytes_per_slot(cfg, dtype: torch.dtype) -> int:
+        """Recurrent state of one sequence (0: the model keeps none)."""
+        return 0
+
     def _init_step_buffers(self, vocab_padded: int) -> None:
         device, mb = self.device, self.max_batch
-        # one int32 staging vector: tokens | positions | slots | seq_lens | temps | seeds(lo,hi)
-        self.meta_fields = 7
+        # one int32 staging vector: tokens | positions | slots | seq_lens | temps | seeds(lo,hi) | state slots
+        self.meta_fields = 8
         self.meta_dev = torch.zeros(self.meta_fields * mb, dtype=torch.int32, device=device)
         self.meta_host = self._pinned(torch.zeros(self.meta_fields * mb, dtype=torch.int32))
         self.bt_dev = torch.zeros(mb, self.max_blocks_per_seq, dtype=torch.int32, device=device)
@@ -86,6 +97,7 @@ class RunnerBase:
         self.d_tokens, self.d_pos, self.d_slots, self.d_lens = m[0:mb], m[mb:2 * mb], m[2 * mb:3 * mb], m[3 * mb:4 * mb]
         self.d_temps = m[4 * mb:5 * mb].view(torch.float32)
         self.d_seeds = m[5 * mb:7 * mb].view(torch.int64)
+        self.d_state_slots = m[7 * mb:8 * mb]
         self.d_out_tokens = self.out_dev[0:mb]
         self.d_out_logprobs = self.out_dev[mb:2 * mb].view(torch.float32)
         self.logits_padded = torch.empty(mb, vocab_padded, dtype=torch.float32, device=device)
@@ -93,9 +105,9 @@ class RunnerBase:
         self.graphs: dict[int, torch.cuda.CUDAGraph] = {}
         self.launches_per_graph: dict[int, int] = {}
         self.graph_pool = None
-        # prefill staging (pinned): tokens | positions | slots | cu_q | seq_lens | sample_rows | temps | seeds
+        # prefill staging (pinned): tokens | positions | slots | cu_q | seq_lens | sample_rows | temps | seeds | state slots
         T = self.max_prefill_tokens
-        self.pf_host = self._pinned(torch.zeros(3 * T + 6 * (mb + 1), dtype=torch.int32))
+        self.pf_host = self._pinned(torch.zeros(3 * T + 7 * (mb + 1), dtype=torch.int32))
         self.pf_dev = torch.zeros_like(self.pf_host, device=device)
 
     def _init_geometry(self, cfg, *, device, num_kv_blocks: int, max_batch: int, max_model_len: int, max_prefill_tokens: int,
@@ -118,6 +130,7 @@ class RunnerBase:
             self.graph_batch_sizes += (max_batch,)
         self.launches_per_decode_step = 0
         self.row_align = 1
+        self.scratch_state_slot = max_batch      # one more than the scheduled sequences use: score()
 
     def _pinned(self, t: torch.Tensor) -> torch.Tensor:
         return t.pin_memory() if self.on_gpu else t
@@ -145,6 +158,7 @@ class RunnerBase:
             return
         self.d_lens.zero_()
         self.d_slots.fill_(-1)
+        self.d_state_slots.fill_(-1)
         torch.cuda.synchronize(self.device)
         stream = torch.cuda.Stream(self.device)
         ops.set_pdl(True)  # decode kernels overlap their prologue with the previous kernel's tail
@@ -192,6 +206,7 @@ class RunnerBase:
             mh[2 * mb + n:2 * mb + bk] = -1
             mh[3 * mb + n:3 * mb + bk] = 0
             mh[4 * mb + n:4 * mb + bk] = 0
+            mh[7 * mb + n:7 * mb + bk] = -1
 
     # ------------------------------------------------------------------ packed batches
     def _stage_packed(self, rows: int, T: int, max_new: int, max_blocks: int) -> "PackedBatch":
@@ -206,11 +221,13 @@ class RunnerBase:
         self.pf_dev.copy_(ph, non_blocking=True)
         self.bt_dev[:rows, :max_blocks].copy_(self.bt_host[:rows, :max_blocks], non_blocking=True)
         pd = self.pf_dev
+        cu = ph[o["cu_q"]:o["cu_q"] + rows + 1].tolist()
         return PackedBatch(
             rows=rows, num_tokens=T, padded=Tp, max_new=max_new, tokens=pd[o["tokens"]:o["tokens"] + Tp],
             positions=pd[o["positions"]:o["positions"] + Tp], slots=pd[o["slots"]:o["slots"] + Tp],
             cu_q=pd[o["cu_q"]:o["cu_q"] + rows + 1], seq_lens=pd[o["seq_lens"]:o["seq_lens"] + rows], block_tables=self.bt_dev[:rows],
-            host_cu_q=ph[o["cu_q"]:o["cu_q"] + rows + 1].tolist(), host_seq_lens=ph[o["seq_lens"]:o["seq_lens"] + rows].tolist())
+            host_cu_q=cu, host_seq_lens=ph[o["seq_lens"]:o["seq_lens"] + rows].tolist(),
+            state_slots=pd[o["state_slots"]:o["state_slots"] + rows], n_single=leading_singles(cu))
 
     def prefill(self, rows: int, T: int, max_new: int, max_blocks: int, views: dict[str, torch.Tensor] | None = None) -> None:
         """Packed varlen pass over ``T`` new tokens of ``rows`` sequences; the last token of each is sampled.
@@ -252,13 +269,14 @@ class RunnerBase:
             rows=1, num_tokens=T, padded=T, max_new=T, tokens=token_ids.to(device=dev, dtype=torch.int32), positions=pos,
             slots=slots.to(torch.int32), cu_q=torch.tensor([0, T], dtype=torch.int32, device=dev),
             seq_lens=torch.tensor([T], dtype=torch.int32, device=dev), block_tables=blocks[None].contiguous(),
-            host_cu_q=[0, T], host_seq_lens=[T]))
+            host_cu_q=[0, T], host_seq_lens=[T], state_slots=torch.tensor([self.scratch_state_slot], dtype=torch.int32, device=dev),
+            n_single=int(T == 1)))
         return self._row_logits(x, pos)
 
     def _pf_offsets(self) -> dict[str, int]:
         T, mb = self.max_prefill_tokens, self.max_batch
         return {"tokens": 0, "positions": T, "slots": 2 * T, "cu_q": 3 * T, "seq_lens": 3 * T + (mb + 1),
-                "sample_rows": 3 * T + 2 * (mb + 1), "temps": 3 * T + 3 * (mb + 1), "seeds": 3 * T + 4 * (mb + 1)}
+                "sample_rows": 3 * T + 2 * (mb + 1), "temps": 3 * T + 3 * (mb + 1), "seeds": 3 * T + 4 * (mb + 1), "state_slots": 3 * T + 6 * (mb + 1)}
 
 
 class LayerWeights:

@@ -1,0 +1,15 @@
+"""Building blocks of layer-stack models on the engine: one class per kind of mixer and feed-forward.
+
+A part is made once per runner and kind. It knows the limits of its kernels, allocates and loads the padded weights of
+every layer of its kind (``make`` / ``load``), the cache or state of every run of such a layer (``new_cache``) and the shared
+activations (``allocate``), plans a step for all its layers at once (``plan``) and runs one layer (``forward``).
+"""
+
+from ...models.stack import ClampedGluSpec, ExpertsSpec, KeyValueAttentionSpec, LatentAttentionSpec, LightningSpec, MatrixMemorySpec
+from .feedforward import DensePart, ExpertsPart
+from .keyvalue import KeyValuePart
+from .latent import LatentPart
+from .recurrent import RecurrentPart
+
+MIXER_PARTS = {LatentAttentionSpec: LatentPart, KeyValueAttentionSpec: KeyValuePart, LightningSpec: RecurrentPart, MatrixMemorySpec: RecurrentPart}
+FEED_FORWARD_PARTS = {ClampedGluSpec: DensePart, ExpertsSpec: ExpertsPart}

@@ -1,0 +1,86 @@
+"""Recurrent mixers (``ops/recurrent.py``) as a part of a layer stack: one joint projection (queries, keys, values, output
+gate), the recurrence over the sequences' state slots, one norm-and-gate kernel, the output projection. Gate logits of the
+recurrence come from the layer's narrow fp32 projection."""
+
+from __future__ import annotations
+
+import torch
+
+from ... import ops
+from ...models.stack import LightningSpec, MatrixMemorySpec
+from ...ops.recurrent import MAX_DIM, RecurrentGeometry, RecurrentState
+from .base import Part, load_head_columns, load_head_vector, load_heads
+
+
+def recurrent_geometry(m: LightningSpec | MatrixMemorySpec) -> RecurrentGeometry:
+    gated = isinstance(m, MatrixMemorySpec)
+    return RecurrentGeometry(m.heads, m.dim, m.vdim, silu=not gated, gated=gated)
+
+
+class RecurrentWeights:
+    __slots__ = ("geo", "spec", "wproj", "wo", "norm", "decay", "bias_i", "bias_f", "cap")
+
+
+class RecurrentPart(Part):
+    @staticmethod
+    def state_floats(spec) -> int:
+        return recurrent_geometry(spec).state_floats
+
+    @staticmethod
+    def small_rows(spec) -> int:
+        return 2 * spec.heads if isinstance(spec, MatrixMemorySpec) else 0
+
+    def make(self, spec) -> RecurrentWeights:
+        g, f32 = recurrent_geometry(spec), torch.float32
+        if g.kp > MAX_DIM:
+            raise ValueError(f"the recurrent kernels take up to {MAX_DIM} key channels per head")
+        w = RecurrentWeights()
+        w.spec, w.geo = spec, g
+        w.wproj, w.wo = self.zeros(g.proj, self.r.wp), self.zeros(self.r.wp, g.heads * g.vp)
+        w.norm = self.zeros(g.heads * g.vp, dtype=f32)
+        w.decay = w.bias_i = w.bias_f = None
+        w.cap = 1.0
+        if g.gated:
+            w.bias_i, w.bias_f, w.cap = self.zeros(g.heads, dtype=f32), self.zeros(g.heads, dtype=f32), spec.gate_cap
+        else:
+            w.decay = torch.tensor(spec.decay, dtype=f32, device=self.r.device)
+        self.layers.append(w)
+        return w
+
+    def new_cache(self, w) -> RecurrentState:
+        return RecurrentState.zeros(w.geo, self.r.scratch_state_slot + 1, self.r.device)
+
+    def allocate(self) -> None:
+        r = self.r
+        self.proj = self.zeros(r.rows * max(w.geo.proj for w in self.layers))
+        most = r.rows * max(w.geo.heads * w.geo.vp for w in self.layers)
+        self.o = self.zeros(most, dtype=torch.float32)
+        self.out = self.zeros(most)
+
+    def load(self, w: RecurrentWeights, get, p: str) -> None:
+        g = w.geo
+        H, (_, ok, ov, og) = g.heads, g.offsets
+        load_heads(w.wproj[:ok], get(p + "q"), H, g.dim, g.kp)
+        load_heads(w.wproj[ok:ov], get(p + "k"), H, g.dim, g.kp)
+        load_heads(w.wproj[ov:og], get(p + "v"), H, g.vdim, g.vp)
+        load_heads(w.wproj[og:], get(p + "g"), H, g.vdim, g.vp)
+        load_head_columns(w.wo, get(p + "o"), H, g.vdim, g.vp)
+        load_head_vector(w.norm, get(p + "norm").float(), H, g.vdim, g.vp)
+        if g.gated:
+            w.bias_i.copy_(get(p + "i.b").float())
+            w.bias_f.copy_(get(p + "f.b").float())
+
+    def load_small(self, w: RecurrentWeights, get, p: str, dst: torch.Tensor) -> None:
+        if w.geo.gated:
+            dst[:w.geo.heads, :self.r.cfg.hidden_size].copy_(get(p + "i"))
+            dst[w.geo.heads:2 * w.geo.heads, :self.r.cfg.hidden_size].copy_(get(p + "f"))
+
+    def forward(self, w: RecurrentWeights, state: RecurrentState, inp, y, b, plan, small=None) -> None:
+        T, g = b.num_tokens, w.geo
+        n = g.heads * g.vp
+        proj = self.proj[:T * g.proj].view(T, g.proj)
+        o, out = self.o[:T * n].view(T, n), self.out[:T * n].view(T, n)
+        ops.gemm(inp, w.wproj, out=proj)
+        ops.recurrent_scan(proj, small, g, w.decay, w.bias_i, w.bias_f, w.cap, state, b.state_slots, b.cu_q, b.seq_lens, o, T, b.rows)
+        ops.gated_norm(o, w.norm, proj[:, g.offsets[3]:], g, self.r.cfg.norm_eps, out, g.gated)
+        ops.gemm(out, w.wo, out=y, out_f32=True)

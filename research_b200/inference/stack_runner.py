@@ -1,15 +1,16 @@
-"""Kernel-backed execution of layer-stack models (``LayerStackConfig``) over the engine's paged cache.
+"""Kernel-backed execution of layer-stack models (``LayerStackConfig``) over the engine's paged cache and state slots.
 
-Step buffers, graph capture, packed batches and sampling come from ``RunnerBase``; this file has the weights, the cache
-tensors and the layer sequence. The residual stream is fp32 with a copy in the activation type for the projections; a
-sublayer reads the stream itself and its output is layer-normalised on the way back (the layer scale is folded into that
-norm's weight and bias in fp32).
+Step buffers, graph capture, packed batches and sampling come from ``RunnerBase``, mixers and feed-forwards from
+``stack_parts``; this file puts layers together. The residual stream is fp32; projections read activations in the serving
+type. Two kinds of layer (``Design.block``):
 
-Per layer on the GPU: one joint down projection (query latent, kv latent, rotated key part, gate logits), one fused
-norm / rotation / cache-append kernel, the query up projection, attention, the output projection, norm + residual, and
-the feed-forward as gate|up with the clamped unit in the GEMM epilogue, down projection, norm + residual. Attention has
-two forms (``ops/latent.py``): on the cached latents themselves for decoded tokens and portions of at most
-``SHORT_PORTION`` tokens, on multiplied-out keys and values for longer portions. Both kinds run in one packed batch.
+* post_norm: a sublayer reads the stream itself (a copy in the activation type) and its output is layer-normalised on the way
+  back; the layer scale is folded into that norm's weight and bias in fp32;
+* parallel: mixer and feed-forward read one RMS norm of the stream; the residual add, the sum over a token's experts and
+  the next layer's norm are one kernel.
+
+Looped layers run several times with the same weights; every run has a cache or state of its own, and a pass starts with a
+product that mixes the embedding output into the stream.
 
 ``dtype`` bf16 serves; fp32 runs the same sequence with every product in 32-bit.
 """
@@ -17,50 +18,36 @@ two forms (``ops/latent.py``): on the cached latents themselves for decoded toke
 from __future__ import annotations
 
 from collections.abc import Mapping
+from dataclasses import dataclass
+from typing import Any
 
 import torch
 
 from .. import ops
-from ..models.stack import ClampedGluSpec, LatentAttentionSpec, LayerStackConfig
-from ..ops.latent import LatentGeometry, live_tables
+from ..models.stack import LayerSpec, LayerStackConfig
+from ..ops.latent import live_tables
 from .model_runner import BLOCK, PackedBatch, RunnerBase
-
-MAX_LATENT, MAX_CACHE_ROW = 1024, 1088
-SHORT_PORTION = 16           # new tokens of a sequence up to which attention runs on the cached latents
-
-
-def _up(n: int, m: int) -> int:
-    return -(-n // m) * m
-
-
-def latent_geometry(m: LatentAttentionSpec) -> LatentGeometry:
-    return LatentGeometry(m.heads, m.dim, m.rot_dim, m.rot.dims // 2, m.vdim, m.kv_rank, m.q_rank)
+from .stack_parts import FEED_FORWARD_PARTS, MIXER_PARTS
+from .stack_parts.base import Part, up
 
 
 class StackLayer:
-    """Padded device weights of one layer."""
+    """Weights of one layer: those of its mixer and feed-forward parts, the norms, the narrow fp32 projection."""
 
-    __slots__ = ("geo", "spec", "table", "wproj", "q_norm", "kv_norm", "wuq", "wuk", "wuv", "wo", "sink", "norm1", "norm2", "glu",
-                 "wgu", "wd", "ffp", "cache")
+    __slots__ = ("spec", "mixer", "mix", "feed_forward", "ff", "norm1", "norm2", "wsmall", "mix_small")
 
 
-class GeometryBuffers:
-    """Activations whose padding depends on a layer's geometry; layers of equal geometry share them."""
+@dataclass
+class StackRun:
+    """One execution of a layer in a step, with the cache or state that belongs to it."""
 
-    def __init__(self, geo: LatentGeometry, rows: int, short_rows: int, dtype: torch.dtype, device: torch.device):
-        H = geo.heads
+    layer: StackLayer
+    cache: Any
+    enters: bool
 
-        def zeros(*shape, dt=dtype):
-            return torch.zeros(*shape, dtype=dt, device=device)
 
-        self.cq = zeros(rows, geo.qp)
-        self.gate = zeros(rows, H, dt=torch.float32)
-        self.qn = zeros(H, short_rows, geo.dp)
-        self.qa = zeros(H, short_rows, geo.cw)
-        self.ol = zeros(H, short_rows, geo.rw)
-        self.q = zeros(rows, H * (geo.dp + geo.rp))
-        self.attn = zeros(rows, H * geo.vp)
-        self.proj = zeros(rows, geo.proj, dt=torch.float32)
+def _mixer_part(spec: LayerSpec):
+    return MIXER_PARTS[type(spec.mixer)]
 
 
 class StackRunner(RunnerBase):
@@ -73,25 +60,17 @@ class StackRunner(RunnerBase):
                  graph_batch_sizes: tuple[int, ...] = (), tp=None, ep=None, dtype: torch.dtype = torch.bfloat16):
         if tp is not None or ep is not None:
             raise ValueError("layer-stack models run on one GPU per engine (no tensor or expert parallelism)")
-        for x in cfg.layers:
-            g = latent_geometry(x.mixer)
-            if g.rw > MAX_LATENT or g.cw > MAX_CACHE_ROW:
-                raise ValueError(f"the latent attention kernels take up to {MAX_LATENT} latent channels and cache rows of {MAX_CACHE_ROW}")
         self.tp = self.ep = None
         self.tp_size, self.tp_rank = 1, 0
         self._init_geometry(cfg, device=device, num_kv_blocks=num_kv_blocks, max_batch=max_batch, max_model_len=max_model_len,
                             max_prefill_tokens=max_prefill_tokens, use_cuda_graphs=use_cuda_graphs,
                             graph_batch_sizes=graph_batch_sizes, dtype=dtype)
         self.bf16 = self.on_gpu and dtype == torch.bfloat16
-        d = cfg.hidden_size
-        self.wp = _up(d, 8)
-        self.vp = _up(cfg.vocab_size, 8)
+        self.parallel = cfg.design.block == "parallel"
+        self.wp = up(cfg.hidden_size, 8)
+        self.vp = up(cfg.vocab_size, 8)
         self.rows = max(max_prefill_tokens, max_batch)
-        self.glu_bn = 256                               # tile width of the fused gate|up launch
-        # multiplied-out keys and values need bf16 tensor-core tiles of a size the kernel has; otherwise (and in exact
-        # mode) every token attends on the cached latents
-        self.expand = (self.bf16 or not self.on_gpu) and all(ops.flash_latent_supported(latent_geometry(x.mixer)) for x in cfg.layers)
-        self.short_rows = min(self.rows, max_batch * SHORT_PORTION) if self.expand else self.rows
+        self.parts: dict[type, Part] = {}
         self._alloc_weights()
         self.load_weights(weights)
         self._init_step_buffers(self.vp)
@@ -99,63 +78,63 @@ class StackRunner(RunnerBase):
 
     @staticmethod
     def cache_bytes_per_block(cfg: LayerStackConfig, tp_size: int, dtype: torch.dtype) -> int:
-        return sum(latent_geometry(x.mixer).cw for x in cfg.layers) * BLOCK * (4 if dtype == torch.float32 else 2)
+        rows = sum(_mixer_part(cfg.layers[x.layer]).cache_row_elements(cfg.layers[x.layer].mixer) for x in cfg.runs)
+        return rows * BLOCK * (4 if dtype == torch.float32 else 2)
+
+    @staticmethod
+    def state_bytes_per_slot(cfg: LayerStackConfig, dtype: torch.dtype) -> int:
+        return 4 * sum(_mixer_part(cfg.layers[x.layer]).state_floats(cfg.layers[x.layer].mixer) for x in cfg.runs)
 
     # ------------------------------------------------------------------ memory
+    def _part(self, cls: type) -> Part:
+        if cls not in self.parts:
+            self.parts[cls] = cls(self)
+        return self.parts[cls]
+
     def _alloc_weights(self) -> None:
         cfg, dev, dt = self.cfg, self.device, self.dtype
 
         def zeros(*shape, dtype=dt):
             return torch.zeros(*shape, dtype=dtype, device=dev)
 
-        f32 = torch.float32
-        d = cfg.hidden_size
-        self.embed = zeros(cfg.vocab_size, self.wp)
-        self.head = zeros(self.vp, self.wp)
-        self.final_norm = (zeros(d, dtype=f32), zeros(d, dtype=f32))
-        tables: dict = {}
+        def norm():
+            return zeros(self.wp, dtype=torch.float32), zeros(self.wp, dtype=torch.float32)
+
+        # (a tied head reads the embedding table itself, whose rows are padded like the head's)
+        self.embed = zeros(self.vp, self.wp)
+        self.head = self.embed if cfg.design.tied else zeros(self.vp, self.wp)
+        self.final_norm = norm()
+        self.loop_in = zeros(self.wp, 2 * self.wp) if cfg.loop is not None else None
         self.layers: list[StackLayer] = []
         for spec in cfg.layers:
-            m, g = spec.mixer, latent_geometry(spec.mixer)
             lw = StackLayer()
-            lw.spec, lw.geo = spec, g
-            if m.rot not in tables:
-                tables[m.rot] = ops.rope_table(self.max_model_len, m.rot.dims, m.rot.base, device=dev, exact=True)
-            lw.table = tables[m.rot]
-            lw.wproj = zeros(g.proj, self.wp)
-            lw.q_norm, lw.kv_norm, lw.sink = zeros(g.q_rank, dtype=f32), zeros(g.kv_rank, dtype=f32), zeros(g.heads, dtype=f32)
-            lw.wuq = zeros(g.heads * (g.dp + g.rp), g.qp)
-            lw.wuk = zeros(g.heads * g.dp, g.rw)
-            lw.wuv = zeros(g.heads * g.vp, g.rw)
-            lw.wo = zeros(self.wp, g.heads * g.vp)
-            lw.norm1 = (zeros(d, dtype=f32), zeros(d, dtype=f32))
-            lw.glu: ClampedGluSpec | None = spec.mlp
-            lw.wgu = lw.wd = lw.norm2 = None
-            lw.ffp = 0
+            lw.spec = spec
+            lw.mixer = self._part(_mixer_part(spec))
+            lw.mix = lw.mixer.make(spec.mixer)
+            lw.norm1, lw.norm2 = norm(), None
+            lw.feed_forward = lw.ff = None
+            lw.mix_small = up(lw.mixer.small_rows(spec.mixer), 8)
+            ff_small = 0
             if spec.mlp is not None:
-                lw.ffp = _up(spec.mlp.ff, self.glu_bn // 2 if self.bf16 else 8)
-                lw.wgu, lw.wd = zeros(2 * lw.ffp, self.wp), zeros(self.wp, lw.ffp)
-                lw.norm2 = (zeros(d, dtype=f32), zeros(d, dtype=f32))
-            lw.cache = zeros(self.num_kv_blocks, BLOCK, g.cw)
+                lw.feed_forward = self._part(FEED_FORWARD_PARTS[type(spec.mlp)])
+                lw.ff = lw.feed_forward.make(spec.mlp)
+                lw.norm2 = None if self.parallel else norm()
+                ff_small = up(lw.feed_forward.small_rows(spec.mlp), 8)
+            lw.wsmall = zeros(lw.mix_small + ff_small, self.wp) if lw.mix_small + ff_small else None
             self.layers.append(lw)
+        self.runs = [StackRun(self.layers[x.layer], self.layers[x.layer].mixer.new_cache(self.layers[x.layer].mix), x.enters) for x in cfg.runs]
 
     def _alloc_activations(self) -> None:
         dev, dt, n = self.device, self.dtype, self.rows
-        d = self.cfg.hidden_size
-        self.x = torch.zeros(n, d, dtype=torch.float32, device=dev)
-        self.xb = torch.zeros(n, self.wp, dtype=dt, device=dev)
+        self.x = torch.zeros(n, self.wp, dtype=torch.float32, device=dev)
+        self.xb = torch.zeros(n, self.wp, dtype=dt, device=dev)          # what the sublayers read
         self.y = torch.zeros(n, self.wp, dtype=torch.float32, device=dev)
+        self.y2 = torch.zeros(n, self.wp, dtype=torch.float32, device=dev)
         self.hl = torch.zeros(self.max_batch, self.wp, dtype=dt, device=dev)
-        ffp = max([lw.ffp for lw in self.layers] + [8])
-        self._gu = None if self.bf16 else torch.zeros(n * 2 * ffp, dtype=dt, device=dev)
-        self._act = torch.zeros(n * ffp, dtype=dt, device=dev)
-        self.bufs: dict[LatentGeometry, GeometryBuffers] = {}
-        for lw in self.layers:
-            if lw.geo not in self.bufs:
-                self.bufs[lw.geo] = GeometryBuffers(lw.geo, n, self.short_rows, dt, dev)
-        self.attn_ws = ops.latent_workspace(list(self.bufs), dev) if self.bf16 else None
-        self.kinds = sorted({(lw.geo, lw.spec.mixer.window) for lw in self.layers}, key=repr)    # layers that share an attention plan
-        self.decode_plans = {k: torch.zeros(ops.latent_units(self.max_batch, k[0].heads, 1) + 1, dtype=torch.int32, device=dev) for k in self.kinds}
+        self.x_loop = torch.zeros(n, 2 * self.wp, dtype=dt, device=dev) if self.loop_in is not None else None     # stream | embedding output
+        self._small = torch.zeros(n * max([lw.wsmall.shape[0] for lw in self.layers if lw.wsmall is not None], default=0), dtype=torch.float32, device=dev)
+        for part in self.parts.values():
+            part.allocate()
 
     # ------------------------------------------------------------------ weights
     def load_weights(self, weights: Mapping[str, torch.Tensor]) -> None:
@@ -169,76 +148,106 @@ class StackRunner(RunnerBase):
         def f32(name: str) -> torch.Tensor:
             return get(name).float()
 
-        def norm_into(dst, name: str, scale: torch.Tensor | None) -> None:
+        def norm_into(dst, name: str, scale: torch.Tensor | None = None) -> None:
+            if self.parallel:          # RMS norm, weight stored around zero
+                dst[0][:d].copy_(1 + f32(name))
+                return
             w, b = f32(name), f32(name + ".b")
-            dst[0].copy_(w if scale is None else w * scale)
-            dst[1].copy_(b if scale is None else b * scale)
+            dst[0][:d].copy_(w if scale is None else w * scale)
+            dst[1][:d].copy_(b if scale is None else b * scale)
 
-        self.embed[:, :d].copy_(get("embed"))
-        self.head[:cfg.vocab_size, :d].copy_(get("head"))
-        norm_into(self.final_norm, "final.norm", None)
+        self.embed[:cfg.vocab_size, :d].copy_(get("embed"))
+        if not cfg.design.tied:
+            self.head[:cfg.vocab_size, :d].copy_(get("head"))
+        if self.loop_in is not None:
+            w = get("loop.in")
+            self.loop_in[:d, :d].copy_(w[:, :d])
+            self.loop_in[:d, self.wp:self.wp + d].copy_(w[:, d:])
+        norm_into(self.final_norm, "final.norm")
         for i, lw in enumerate(self.layers):
-            p, g = f"l{i}.", lw.geo
-            m = p + "mix."
-            H, r0 = g.heads, g.q_rank
-            r1 = r0 + g.kv_rank + g.rot_dim
-            lw.wproj[:r0, :d].copy_(get(m + "dq"))
-            lw.wproj[r0:r1, :d].copy_(get(m + "dkv"))
-            lw.wproj[r1:r1 + H, :d].copy_(get(m + "g"))
-            lw.q_norm.copy_(f32(m + "dq.norm"))
-            lw.kv_norm.copy_(f32(m + "dkv.norm"))
-            lw.sink.copy_(f32(m + "sink"))
-            uq = get(m + "uq").view(H, g.dim + g.rot_dim, g.q_rank)
-            wuq = lw.wuq.view(H, g.dp + g.rp, g.qp)
-            wuq[:, :g.dim, :g.q_rank].copy_(uq[:, :g.dim])
-            wuq[:, g.dp:g.dp + g.rot_dim, :g.q_rank].copy_(uq[:, g.dim:])
-            lw.wuk.view(H, g.dp, g.rw)[:, :g.dim, :g.kv_rank].copy_(get(m + "uk").view(H, g.dim, g.kv_rank))
-            lw.wuv.view(H, g.vp, g.rw)[:, :g.vdim, :g.kv_rank].copy_(get(m + "uv").view(H, g.vdim, g.kv_rank))
-            lw.wo.view(self.wp, H, g.vp)[:d, :, :g.vdim].copy_(get(m + "o").view(d, H, g.vdim))
-            norm_into(lw.norm1, p + "norm1", f32(p + "ls1"))
-            if lw.glu is not None:
-                gate, up = get(p + "mlp.gate"), get(p + "mlp.up")
-                ff = lw.glu.ff
-                if self.bf16:        # interleaved blocks for the fused epilogue; padding rows give 0
-                    pad = torch.zeros(2, lw.ffp, self.wp, dtype=self.dtype, device=dev)
-                    pad[0, :ff, :d], pad[1, :ff, :d] = gate, up
-                    lw.wgu.copy_(ops.interleave_gate_up(pad[0], pad[1], self.glu_bn))
-                else:
-                    lw.wgu[:ff, :d].copy_(gate)
-                    lw.wgu[lw.ffp:lw.ffp + ff, :d].copy_(up)
-                lw.wd[:d, :ff].copy_(get(p + "mlp.down"))
-                norm_into(lw.norm2, p + "norm2", f32(p + "ls2"))
+            p = f"l{i}."
+            lw.mixer.load(lw.mix, get, p + "mix.")
+            norm_into(lw.norm1, p + "norm1", None if self.parallel else f32(p + "ls1"))
+            if lw.mix_small:
+                lw.mixer.load_small(lw.mix, get, p + "mix.", lw.wsmall[:lw.mix_small])
+            if lw.ff is not None:
+                lw.feed_forward.load(lw.ff, get, p + "mlp.")
+                if lw.wsmall is not None:
+                    lw.feed_forward.load_small(lw.ff, get, p + "mlp.", lw.wsmall[lw.mix_small:])
+                if not self.parallel:
+                    norm_into(lw.norm2, p + "norm2", f32(p + "ls2"))
 
     # ------------------------------------------------------------------ layers
-    def _layers(self, T: int, tokens, positions, slots, n_short: int, short_attn, long_attn=None) -> None:
-        """All layers over the first ``T`` rows. ``short_attn(lw, bufs)`` fills ``bufs.ol`` for the first ``n_short`` rows,
-        ``long_attn(lw, bufs)`` the remaining rows of ``bufs.attn``."""
-        eps = self.cfg.norm_eps
+    def _small_rows(self, inp: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        """The narrow projections of ``inp``, fp32."""
+        T, n = inp.shape[0], w.shape[0]
+        return ops.gemm(inp, w, out=self._small[:T * n].view(T, n), out_f32=True)
+
+    def _layers(self, b: PackedBatch) -> None:
+        """All layer runs over the batch's rows; leaves the residual stream in ``self.x``."""
+        plans = {part: part.plan(b) for part in self.parts.values()}
+        if self.parallel:
+            self._parallel_layers(b, plans)
+        else:
+            self._post_norm_layers(b, plans)
+
+    def _enter_pass(self, T: int) -> None:
+        """``x = W [x; embedding output]``: a pass of the loop begins (the stream's copy is in ``x_loop`` already)."""
+        ops.gemm(self.x_loop[:T], self.loop_in, out=self.x[:T], out_f32=True)
+
+    def _embed(self, b: PackedBatch, first_copy: torch.Tensor | None) -> None:
+        """Embedding output into the stream, its second half of ``x_loop`` and, if given, another copy."""
+        x0 = self.x_loop[:, self.wp:] if self.x_loop is not None else None
+        ops.stream_embed(b.tokens[:b.num_tokens], self.embed[:self.cfg.vocab_size], self.cfg.hidden_size, self.x, x0, first_copy)
+
+    def _parallel_layers(self, b: PackedBatch, plans: dict) -> None:
+        T, d, eps = b.num_tokens, self.cfg.hidden_size, self.cfg.norm_eps
+        x, h, y = self.x[:T], self.xb[:T], self.y[:T]
+        xl = self.x_loop[:T, :self.wp] if self.x_loop is not None else None
+        self._embed(b, xl)
+        add: dict = {}                                 # what the layer before leaves for the stream
+        for run in self.runs:
+            lw = run.layer
+            if run.enters:
+                if add:
+                    ops.stream_norm(x, d, **add, copy=xl)
+                    add = {}
+                self._enter_pass(T)
+            ops.stream_norm(x, d, **add, weight=lw.norm1[0], eps=eps, h=h)
+            small = self._small_rows(h, lw.wsmall) if lw.wsmall is not None else None
+            lw.mixer.forward(lw.mix, run.cache, h, y, b, plans[lw.mixer], small)
+            add = {"y1": y}
+            if lw.ff is not None:
+                add.update(lw.feed_forward.forward(lw.ff, h, self.y2[:T], small[:, lw.mix_small:] if small is not None else None))
+        ops.stream_norm(x, d, **add)
+
+    def _post_norm_layers(self, b: PackedBatch, plans: dict) -> None:
+        T, d, eps = b.num_tokens, self.cfg.hidden_size, self.cfg.norm_eps
         x, xb, y = self.x[:T], self.xb[:T], self.y[:T]
-        ops.embed_residual(tokens, self.embed, x, xb)
-        for lw in self.layers:
-            g, b = lw.geo, self.bufs[lw.geo]
-            ops.gemm(xb, lw.wproj, out=b.proj[:T], out_f32=True)
-            ops.latent_append(b.proj[:T], g, lw.q_norm, lw.kv_norm, eps, positions, slots, lw.table, lw.cache, b.cq, b.gate)
-            q = ops.gemm(b.cq[:T], lw.wuq, out=b.q[:T])
-            ops.latent_query(q, g, positions, lw.table, n_short, b.qn, b.qa)
-            if n_short > 0:
-                ops.head_gemm_absorb(b.qn, lw.wuk, b.qa, n_short)
-                short_attn(lw, b)
-                ops.head_gemm_expand(b.ol, lw.wuv, b.attn, n_short)
-            if n_short < T:
-                long_attn(lw, b)
-            ops.gemm(b.attn[:T], lw.wo, out=y, out_f32=True)
-            ops.layernorm_residual(y, lw.norm1[0], lw.norm1[1], eps, x, xb)
-            if lw.glu is not None:
-                act = self._act[:T * lw.ffp].view(T, lw.ffp)
-                if self.bf16:
-                    ops.gemm(xb, lw.wgu, out=act, bn=self.glu_bn, swiglu=True, glu_limit=lw.glu.limit)
-                else:
-                    gu = ops.gemm(xb, lw.wgu, out=self._gu[:T * 2 * lw.ffp].view(T, 2 * lw.ffp))
-                    ops.clamped_glu(gu, lw.glu.limit, out=act)
-                ops.gemm(act, lw.wd, out=y, out_f32=True)
-                ops.layernorm_residual(y, lw.norm2[0], lw.norm2[1], eps, x, xb)
+        self._embed(b, xb)
+        for run in self.runs:
+            lw = run.layer
+            if run.enters:
+                ops.stream_norm(x, d, copy=self.x_loop[:T, :self.wp])
+                self._enter_pass(T)
+                ops.stream_norm(x, d, copy=xb)
+            small = self._small_rows(xb, lw.wsmall[:lw.mix_small]) if lw.mix_small else None
+            lw.mixer.forward(lw.mix, run.cache, xb, y, b, plans[lw.mixer], small)
+            ops.layernorm_residual(y, lw.norm1[0], lw.norm1[1], eps, x, xb, d)
+            if lw.ff is not None:
+                small = self._small_rows(xb, lw.wsmall[lw.mix_small:]) if lw.wsmall is not None and lw.wsmall.shape[0] > lw.mix_small else None
+                add = lw.feed_forward.forward(lw.ff, xb, y, small)
+                if "experts" in add:
+                    y.zero_()
+                    ops.stream_norm(y, d, **add)
+                ops.layernorm_residual(y, lw.norm2[0], lw.norm2[1], eps, x, xb, d)
+
+    def _final_rows(self, x: torch.Tensor, out: torch.Tensor, rows: torch.Tensor | None = None) -> None:
+        d, eps = self.cfg.hidden_size, self.cfg.norm_eps
+        if self.parallel:
+            ops.stream_norm(x, d, weight=self.final_norm[0], eps=eps, h=out, rows=rows)
+        else:
+            ops.layernorm_rows(x, self.final_norm[0], self.final_norm[1], eps, out, rows, d)
 
     def _head(self, h: torch.Tensor, logits: torch.Tensor) -> torch.Tensor:
         """``logits`` (rows padded to ``vp`` columns) of the final-normed rows ``h``, soft-capped."""
@@ -251,27 +260,15 @@ class StackRunner(RunnerBase):
                 ops.softcap(logits, cap)
         return logits[:, :self.cfg.vocab_size]
 
-    def _short_attention(self, rows: int, max_q: int, cu_q, seq_lens, block_tables, plans: dict | None = None):
-        """Attention on the cached latents for the first ``rows`` rows of the batch."""
-        if self.bf16:
-            n = seq_lens.shape[0]
-            if plans is None:
-                plans = {k: torch.empty(ops.latent_units(n, k[0].heads, max_q) + 1, dtype=torch.int32, device=self.device) for k in self.kinds}
-            for (geo, window), plan in plans.items():
-                ops.latent_plan(cu_q, seq_lens, geo, max_q, window, plan)
-
-        def attend(lw, b):
-            m = lw.spec.mixer
-            ops.latent_attention(b.qa, lw.cache, lw.geo, block_tables, cu_q, seq_lens, lw.sink, b.gate, b.ol, scale=m.scale, window=m.window,
-                                 rows=rows, max_q=max_q, plan=plans[(lw.geo, m.window)] if self.bf16 else None, workspace=self.attn_ws)
-
-        return attend
-
     # ------------------------------------------------------------------ decode
+    def _decode_batch(self, bk: int) -> PackedBatch:
+        return PackedBatch(rows=bk, num_tokens=bk, padded=bk, max_new=1, tokens=self.d_tokens[:bk], positions=self.d_pos[:bk], slots=self.d_slots[:bk],
+                           cu_q=None, seq_lens=self.d_lens[:bk], block_tables=self.bt_dev[:bk], host_cu_q=[], host_seq_lens=[],
+                           state_slots=self.d_state_slots[:bk], n_single=bk)
+
     def _decode_body(self, bk: int) -> None:
-        self._layers(bk, self.d_tokens[:bk], self.d_pos[:bk], self.d_slots[:bk], bk,
-                     self._short_attention(bk, 1, None, self.d_lens[:bk], self.bt_dev[:bk], self.decode_plans))
-        ops.layernorm_rows(self.x[:bk], self.final_norm[0], self.final_norm[1], self.cfg.norm_eps, self.hl)
+        self._layers(self._decode_batch(bk))
+        self._final_rows(self.x[:bk], self.hl)
         logits = self._head(self.hl[:bk], self.logits_padded[:bk])
         self._sample(logits, self.d_temps[:bk], self.d_seeds[:bk], bk)
 
@@ -283,50 +280,12 @@ class StackRunner(RunnerBase):
     def _packed_forward(self, b: PackedBatch) -> torch.Tensor:
         T = b.num_tokens
         assert T <= self.rows, f"packed batch of {T} tokens, buffers hold {self.rows}"
-        lens = [b.host_cu_q[i + 1] - b.host_cu_q[i] for i in range(b.rows)]
-        n_seq = b.rows                                      # sequences attending on the cached latents: a prefix of the batch
-        if self.expand:
-            n_seq = next((i for i, n in enumerate(lens) if n > SHORT_PORTION), b.rows)
-            while b.host_cu_q[n_seq] > self.short_rows:     # (score() and other batches that are not ordered by length)
-                n_seq -= 1
-        n_short = b.host_cu_q[n_seq]
-        max_q = max(lens[:n_seq], default=1)
-        short_attn = None
-        if n_short > 0:
-            short_attn = self._short_attention(n_short, max_q, b.cu_q[:n_seq + 1], b.seq_lens[:n_seq], b.block_tables[:n_seq])
-        self._layers(T, b.tokens[:T], b.positions[:T], b.slots[:T], n_short, short_attn,
-                     self._long_attention(b, n_seq, n_short) if n_seq < b.rows else None)
+        b.tokens, b.positions, b.slots = b.tokens[:T], b.positions[:T], b.slots[:T]
+        self._layers(b)
         return self.x[:T]
-
-    def _long_attention(self, b: PackedBatch, first: int, n_short: int):
-        """Plan of the expanded form for the sequences ``first..``: per window, which cached rows they can see."""
-        n_seq = b.rows - first
-        plans: dict[int, tuple] = {}
-        for w in {lw.spec.mixer.window for lw in self.layers}:
-            lo, cu, most = [], [0], 0
-            for i in range(first, b.rows):
-                L, q = b.host_seq_lens[i], b.host_cu_q[i + 1] - b.host_cu_q[i]
-                lo.append(max(0, L - q - w + 1))
-                cu.append(cu[-1] + L - lo[-1])
-                most = max(most, q)
-            meta = torch.tensor(lo + cu, dtype=torch.int32).to(self.device)
-            plans[w] = (meta[:n_seq], meta[n_seq:], cu[-1], most)
-        cu_q = b.cu_q[first:]
-
-        def long_attn(lw, buf):
-            g, m = lw.geo, lw.spec.mixer
-            k_lo, cu_k, n, max_q = plans[m.window]
-            lat = torch.empty(n, g.rw, dtype=self.dtype, device=self.device)
-            rot = torch.empty(n, g.rp, dtype=self.dtype, device=self.device)
-            ops.latent_gather(lw.cache, g, b.block_tables, first, cu_k, k_lo, n, lat, rot)
-            k, v = ops.gemm(lat, lw.wuk), ops.gemm(lat, lw.wuv)
-            ops.flash_latent_prefill(buf.q, k, rot, v, g, cu_q, cu_k, lw.sink, buf.gate, buf.attn, scale=m.scale, window=m.window,
-                                     max_q=max_q, rows=b.num_tokens)
-
-        return long_attn
 
     def _row_logits(self, x, rows) -> torch.Tensor:
         n = rows.numel()
         h = self.hl if n <= self.max_batch else torch.zeros(n, self.wp, dtype=self.dtype, device=self.device)
-        ops.layernorm_rows(x, self.final_norm[0], self.final_norm[1], self.cfg.norm_eps, h, rows)
+        self._final_rows(x, h, rows)
         return self._head(h[:n], torch.empty(n, self.vp, dtype=torch.float32, device=self.device))

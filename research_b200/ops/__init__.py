@@ -13,7 +13,6 @@ from .attention import (
 from .elementwise import (
     clamped_glu,
     clamped_glu_reference,
-    embed_residual,
     embedding,
     layernorm_reference,
     layernorm_residual,
@@ -24,11 +23,14 @@ from .elementwise import (
     rope_kv_append_reference,
     rope_table,
     softcap,
+    stream_embed,
+    stream_norm,
     swiglu,
     swiglu_backward,
     swiglu_reference,
     transpose,
 )
+from .experts import ExpertsGeometry, ExpertsScratch, experts_forward, pack_experts
 from .flash import (
     flash_attention,
     flash_attn_varlen,
@@ -52,6 +54,8 @@ from .latent import (
     latent_units,
     latent_workspace,
 )
+from .keyvalue import KeyValueGeometry, kv_append, kv_attention, kv_workspace
+from .recurrent import RecurrentGeometry, RecurrentState, gated_norm, recurrent_scan
 from .sampling import sample_with_logprobs, sample_with_logprobs_reference, token_logprobs
 
 def set_pdl(on: bool) -> None:
@@ -60,7 +64,8 @@ def set_pdl(on: bool) -> None:
     from .. import _native
 
     for lib, fn in (("rb_gemm", "rb_gemm_set_pdl"), ("rb_ops", "rb_ops_set_pdl"), ("rb_attn", "rb_attn_set_pdl"),
-                    ("rb_latent", "rb_latent_set_pdl"), ("rb_gemm_f32", "rb_gemm_f32_set_pdl")):
+                    ("rb_latent", "rb_latent_set_pdl"), ("rb_gemm_f32", "rb_gemm_f32_set_pdl"),
+                    ("rb_recurrent", "rb_recurrent_set_pdl"), ("rb_moe", "rb_moe_set_pdl")):
         if _native.available(lib):      # a partial build has only the libraries its models need
             getattr(_native.load(lib), fn)(int(on))
 
@@ -72,6 +77,8 @@ __all__ = [
     "swiglu_reference", "transpose", "gemm", "gemm_reference", "linear", "sample_with_logprobs",
     "sample_with_logprobs_reference", "token_logprobs", "set_pdl", "interleave_gate_up", "gemm_mod", "gemm_symmetric", "gemm_fp8", "quantize_fp8", "lm_head_sample", "lm_head_sample_workspace", "flash_attention", "flash_attn_varlen",
     "flash_attn_varlen_backward", "flash_attn_varlen_reference", "flash_paged_prefill", "flash_latent_prefill", "flash_latent_supported", "clamped_glu", "clamped_glu_reference",
-    "embed_residual", "layernorm_reference", "layernorm_residual", "layernorm_rows", "softcap", "gemm_f32", "LatentGeometry",
+    "layernorm_reference", "layernorm_residual", "layernorm_rows", "softcap", "gemm_f32", "LatentGeometry",
     "head_gemm_absorb", "head_gemm_expand", "latent_append", "latent_attention", "latent_gather", "latent_plan", "latent_query", "latent_units", "latent_workspace",
+    "ExpertsGeometry", "ExpertsScratch", "experts_forward", "pack_experts", "KeyValueGeometry", "kv_append", "kv_attention", "kv_workspace",
+    "RecurrentGeometry", "RecurrentState", "gated_norm", "recurrent_scan", "stream_embed", "stream_norm",
 ]

@@ -28,11 +28,13 @@ def _lib() -> ctypes.CDLL:
         lib.rb_swiglu_bounded.restype = c_int
         lib.rb_embedding.argtypes = [c_vp, c_vp, c_vp, c_int, c_int, c_int, c_vp, c_vp]
         lib.rb_transpose_bf16.argtypes = [c_vp, c_vp, c_int, c_int, c_vp]
-        lib.rb_embed_residual.argtypes = [c_vp] * 4 + [c_int] * 3 + [c_ll, c_int, c_vp, c_vp]
-        lib.rb_layernorm.argtypes = [c_vp, c_ll] + [c_vp] * 5 + [c_ll, c_int, c_int, c_int, c_float, c_int, c_vp, c_vp]
+        lib.rb_layernorm.argtypes = [c_vp, c_ll, c_vp, c_ll] + [c_vp] * 4 + [c_ll, c_int, c_int, c_int, c_float, c_int, c_vp, c_vp]
         lib.rb_clamped_glu.argtypes = [c_vp, c_vp, c_int, c_ll, c_int, c_float, c_vp]
         lib.rb_softcap.argtypes = [c_vp, c_ll, c_float, c_vp]
-        for f in ("rb_embed_residual", "rb_layernorm", "rb_clamped_glu", "rb_softcap", "rb_rmsnorm", "rb_rope_kv_append", "rb_swiglu", "rb_swiglu_bwd", "rb_embedding", "rb_transpose_bf16"):
+        lib.rb_stream_embed.argtypes = [c_vp, c_vp, c_ll, c_vp, c_ll, c_vp, c_ll, c_vp, c_ll] + [c_int] * 4 + [c_vp, c_vp]
+        lib.rb_stream_norm.argtypes = ([c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_vp, c_ll, c_int, c_vp, c_ll, c_vp, c_ll, c_vp, c_vp] + [c_int] * 5
+                                       + [c_float, c_vp, c_vp])
+        for f in ("rb_stream_embed", "rb_stream_norm", "rb_layernorm", "rb_clamped_glu", "rb_softcap", "rb_rmsnorm", "rb_rope_kv_append", "rb_swiglu", "rb_swiglu_bwd", "rb_embedding", "rb_transpose_bf16"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -213,18 +215,53 @@ def transpose(x: torch.Tensor) -> torch.Tensor:
 _ACT = {torch.bfloat16: 0, torch.float32: 1}
 
 
-def embed_residual(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, xb: torch.Tensor) -> None:
-    """``x[t] = table[ids[t]]`` in fp32 and the same row in the activation type ``xb`` (leading columns; row strides of
-    ``table`` and ``xb`` agree)."""
-    T, d = ids.numel(), x.shape[1]
+def stream_embed(ids: torch.Tensor, table: torch.Tensor, d: int, x: torch.Tensor, a: torch.Tensor | None = None,
+                 b: torch.Tensor | None = None) -> None:
+    """``x[t, :d] = table[ids[t]]`` in fp32 and the same row in ``a`` and ``b`` (activation type, any row stride)."""
+    T = ids.numel()
     if not table.is_cuda:
-        x[:T] = table[ids.long(), :d].float()
-        xb[:T, :d] = table[ids.long(), :d]
+        row = table[ids.long(), :d]
+        for dst in (x, a, b):
+            if dst is not None:
+                dst[:T, :d] = row.to(dst.dtype)
         return
-    assert ids.dtype == torch.int32 and ids.is_contiguous() and x.is_contiguous() and table.stride(0) == xb.stride(0)
-    rc = _lib().rb_embed_residual(ptr(ids), ptr(table), ptr(x), ptr(xb), _ACT[table.dtype], T, d, xb.stride(0), table.shape[0],
-                                  ptr(status_tensor(table.device)), stream_handle(table.device))
-    check_rc(rc, "rb_embed_residual")
+    assert ids.dtype == torch.int32 and ids.is_contiguous() and x.dtype == torch.float32
+    rc = _lib().rb_stream_embed(ptr(ids), ptr(table), table.stride(0), ptr(x), x.stride(0), ptr(a), a.stride(0) if a is not None else 0, ptr(b),
+                                b.stride(0) if b is not None else 0, _ACT[table.dtype], T, d, table.shape[0], ptr(status_tensor(table.device)),
+                                stream_handle(table.device))
+    check_rc(rc, "rb_stream_embed")
+
+
+def stream_norm(x: torch.Tensor, d: int, *, y1=None, y2=None, experts=None, expert_weights=None, copy=None, weight=None, eps: float = 0.0,
+                h=None, rows=None) -> None:
+    """What happens to the fp32 stream ``x [n, dp]`` (``d`` channels and zero padding) between two layers, in one pass:
+    ``x += y1 + y2 + sum_j expert_weights[t, j] experts[t, j]`` (the terms that are given), ``copy = x`` and
+    ``h = x / rms(x) * weight`` in the activation type. With ``rows`` only ``h[i]`` of row ``rows[i]``."""
+    n = rows.numel() if rows is not None else x.shape[0]
+    if not x.is_cuda:
+        src = x if rows is None else x[rows.long()]
+        assert rows is None or (y1 is None and y2 is None and experts is None)
+        for y in (y1, y2):
+            if y is not None:
+                x += y[:n]
+        if experts is not None:
+            k = expert_weights.shape[1]
+            x += (experts[:n * k].view(n, k, -1).float() * expert_weights[:n, :, None]).sum(1)
+        if copy is not None:
+            copy[:n] = x.to(copy.dtype)
+        if h is not None:
+            h[:n] = (src * torch.rsqrt(src.pow(2).sum(-1, keepdim=True) / d + eps) * weight).to(h.dtype)
+        return
+    act = next((t for t in (h, copy, experts) if t is not None), x)
+    assert x.dtype == torch.float32 and x.stride(1) == 1 and (rows is None or rows.dtype == torch.int32)
+    assert all(t is None or t.stride(-1) == 1 for t in (y1, y2, experts, copy, h)) and (y1 is None or y2 is None or y1.stride(0) == y2.stride(0))
+    y = y1 if y1 is not None else y2
+    rc = _lib().rb_stream_norm(ptr(x), x.stride(0), ptr(y1), ptr(y2), y.stride(0) if y is not None else 0, ptr(experts), ptr(expert_weights),
+                               experts.stride(0) if experts is not None else 0, expert_weights.shape[1] if experts is not None else 0,
+                               ptr(copy), copy.stride(0) if copy is not None else 0, ptr(h), h.stride(0) if h is not None else 0, ptr(weight),
+                               ptr(rows), x.shape[0], _ACT[act.dtype], n, d, x.shape[1], eps, ptr(status_tensor(x.device)),
+                               stream_handle(x.device))
+    check_rc(rc, "rb_stream_norm")
 
 
 def layernorm_reference(v: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float) -> torch.Tensor:
@@ -232,29 +269,32 @@ def layernorm_reference(v: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: 
     return c / torch.sqrt(c.pow(2).mean(-1, keepdim=True) + eps) * w + b
 
 
-def layernorm_residual(y: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float, x: torch.Tensor, xb: torch.Tensor) -> None:
-    """``x += layer_norm(y) * w + b`` on the fp32 stream, and ``xb`` = the new ``x`` in the activation type."""
-    n, d = x.shape
+def layernorm_residual(y: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float, x: torch.Tensor, xb: torch.Tensor,
+                       d: int | None = None) -> None:
+    """``x += layer_norm(y) * w + b`` on the first ``d`` (default: all) channels of the fp32 stream, and ``xb`` = the new ``x`` in
+    the activation type."""
+    n, d = x.shape[0], x.shape[1] if d is None else d
     if not x.is_cuda:
-        x += layernorm_reference(y[:n, :d], w, b, eps)
-        xb[:n, :d] = x.to(xb.dtype)
+        x[:, :d] += layernorm_reference(y[:n, :d], w[:d], b[:d], eps)
+        xb[:n, :d] = x[:, :d].to(xb.dtype)
         return
-    assert y.dtype == torch.float32 and y.stride(1) == 1 and x.is_contiguous() and w.dtype == b.dtype == torch.float32
-    rc = _lib().rb_layernorm(ptr(y), y.stride(0), ptr(x), None, ptr(w), ptr(b), ptr(xb), xb.stride(0), _ACT[xb.dtype], n, d, eps, n,
+    assert y.dtype == torch.float32 and y.stride(1) == 1 and x.stride(1) == 1 and w.dtype == b.dtype == torch.float32
+    rc = _lib().rb_layernorm(ptr(y), y.stride(0), ptr(x), x.stride(0), None, ptr(w), ptr(b), ptr(xb), xb.stride(0), _ACT[xb.dtype], n, d, eps, n,
                              ptr(status_tensor(x.device)), stream_handle(x.device))
     check_rc(rc, "rb_layernorm")
 
 
-def layernorm_rows(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float, out: torch.Tensor, rows: torch.Tensor | None = None) -> None:
-    """``out[i] = layer_norm(x[rows[i]]) * w + b`` (``rows`` None: all rows in order)."""
-    d = x.shape[1]
+def layernorm_rows(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float, out: torch.Tensor, rows: torch.Tensor | None = None,
+                   d: int | None = None) -> None:
+    """``out[i] = layer_norm(x[rows[i]]) * w + b`` over the first ``d`` (default: all) channels (``rows`` None: all rows in order)."""
+    d = x.shape[1] if d is None else d
     n = rows.numel() if rows is not None else x.shape[0]
     if not x.is_cuda:
         src = x if rows is None else x[rows.long()]
-        out[:n, :d] = layernorm_reference(src, w, b, eps).to(out.dtype)
+        out[:n, :d] = layernorm_reference(src[:, :d], w[:d], b[:d], eps).to(out.dtype)
         return
-    assert x.is_contiguous() and x.dtype == torch.float32 and (rows is None or rows.dtype == torch.int32)
-    rc = _lib().rb_layernorm(None, 0, ptr(x), ptr(rows), ptr(w), ptr(b), ptr(out), out.stride(0), _ACT[out.dtype], n, d, eps, x.shape[0],
+    assert x.stride(1) == 1 and x.dtype == torch.float32 and (rows is None or rows.dtype == torch.int32)
+    rc = _lib().rb_layernorm(None, 0, ptr(x), x.stride(0), ptr(rows), ptr(w), ptr(b), ptr(out), out.stride(0), _ACT[out.dtype], n, d, eps, x.shape[0],
                              ptr(status_tensor(x.device)), stream_handle(x.device))
     check_rc(rc, "rb_layernorm")
 

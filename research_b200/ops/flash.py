@@ -104,14 +104,14 @@ def flash_paged_prefill(q, k_cache, v_cache, block_tables, cu_q, seq_lens, max_n
     Unwritten cache slots must hold finite numbers (the cache is allocated zero-filled)."""
     T, Hq, D = q.shape
     nb, Hkv, bs, _ = k_cache.shape
-    assert bs == 16 and q.is_contiguous() and cu_q.dtype == torch.int32 and seq_lens.dtype == torch.int32
+    assert bs == 16 and q.stride(2) == 1 and q.stride(1) == D and cu_q.dtype == torch.int32 and seq_lens.dtype == torch.int32
     scale = scale or 1.0 / math.sqrt(D)
     if out is None:
         out = torch.empty_like(q)
     B = seq_lens.shape[0]
     rc = _lib().rb_flash_fwd(ptr(q), ptr(k_cache), ptr(v_cache), ptr(out), ptr(lse), ptr(cu_q), None, ptr(seq_lens),
                              ptr(block_tables), B, T, nb, Hq, Hkv, D, q.stride(0), 0, 0, max_new,
-                             block_tables.shape[1], 1, int(window), 1, scale, ptr(status_tensor(q.device)),
+                             block_tables.stride(0), 1, int(window), 1, scale, ptr(status_tensor(q.device)),
                              stream_handle(q.device))
     check_rc(rc, "rb_flash_fwd(paged)")
     return out

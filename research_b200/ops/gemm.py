@@ -181,26 +181,28 @@ def _lib_f32() -> ctypes.CDLL:
     lib = _native.load("rb_gemm_f32")
     if not getattr(lib, "_rb_typed", False):
         vp, i, ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
-        lib.rb_gemm_f32.argtypes = [vp] * 3 + [i] * 3 + [ll] * 3 + [i] + [ll] * 3 + [i, vp]
-        lib.rb_gemm_f32.restype = i
+        lib.rb_gemm_f32.argtypes = [vp] * 4 + [i] * 3 + [ll] * 3 + [i] + [ll] * 3 + [i, vp]
+        lib.rb_gemm_f32_grouped.argtypes = [vp] * 3 + [i] + [ll] * 3 + [vp, vp, i, i, vp, vp]
+        lib.rb_gemm_f32.restype = lib.rb_gemm_f32_grouped.restype = i
         lib._rb_typed = True
     return lib
 
 
-def gemm_f32_batched(a, b, out, M: int, N: int, K: int, batch: int, ld: tuple[int, int, int], step: tuple[int, int, int], b_kn: bool = False) -> None:
-    """``batch`` fp32 products ``C = A B^T`` (``b_kn``: ``A B``) at the given leading dimensions and batch strides."""
+def gemm_f32_batched(a, b, out, M: int, N: int, K: int, batch: int, ld: tuple[int, int, int], step: tuple[int, int, int], b_kn: bool = False,
+                     bias=None) -> None:
+    """``batch`` fp32 products ``C = A B^T (+ bias)`` (``b_kn``: ``A B``) at the given leading dimensions and batch strides."""
     assert a.dtype == b.dtype == out.dtype == torch.float32 and a.is_cuda
-    rc = _lib_f32().rb_gemm_f32(a.data_ptr(), b.data_ptr(), out.data_ptr(), M, N, K, *ld, batch, *step, int(b_kn), stream_handle(a.device))
+    rc = _lib_f32().rb_gemm_f32(a.data_ptr(), b.data_ptr(), out.data_ptr(), bias.data_ptr() if bias is not None else None, M, N, K, *ld, batch, *step, int(b_kn), stream_handle(a.device))
     check_rc(rc, "rb_gemm_f32")
 
 
-def gemm_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+def gemm_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> torch.Tensor:
     """``A @ B^T`` with fp32 operands, products and sums (no reduced-precision matrix mode)."""
     assert a.dim() == b.dim() == 2 and a.stride(1) == b.stride(1) == 1 and a.shape[1] == b.shape[1]
     M, N = a.shape[0], b.shape[0]
     if out is None:
         out = torch.empty(M, N, dtype=torch.float32, device=a.device)
-    gemm_f32_batched(a, b, out, M, N, a.shape[1], 1, (a.stride(0), b.stride(0), out.stride(0)), (0, 0, 0))
+    gemm_f32_batched(a, b, out, M, N, a.shape[1], 1, (a.stride(0), b.stride(0), out.stride(0)), (0, 0, 0), bias=bias)
     return out
 
 
@@ -296,8 +298,8 @@ def gemm(
             return out
         return res
     if a.dtype == torch.float32 and b is not None and b.dtype == torch.float32:
-        assert bias is None and residual is None and not (a_mn_major or b_mn_major or swiglu) and norm_eps is None and alpha == beta == 1.0
-        return gemm_f32(a, b, out)
+        assert residual is None and (bias is None or bias.dtype == torch.float32) and not (a_mn_major or b_mn_major or swiglu) and norm_eps is None and alpha == beta == 1.0
+        return gemm_f32(a, b, out, bias)
     if b_gather is not None:
         b = b_gather.staged          # [rows, cols] view of the staging matrix this launch fills
     assert a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16

@@ -1,0 +1,176 @@
+"""Recurrent mixers with a matrix state per head (csrc/recurrent_sm100.cu) and their PyTorch twins.
+
+Both kinds write ``k v^T`` into a state that decays and read it with ``q``::
+
+    S_t = a_t S_(t-1) + b_t k_t v_t^T          o_t = S_t^T q_t
+
+* lightning: ``a`` is a constant of the head, ``b = 1``; queries, keys and values pass through SiLU;
+* matrix memory (mLSTM): capped gate logits ``i``, ``f``; ``log a = logsigmoid(f)``, ``b = exp(i)``, held relative to a running
+  maximum ``m`` (from 0) so that nothing overflows; a second state ``n`` takes ``k`` alone and divides the output by
+  ``max(|n . q|, exp(-m)) + 1e-6``.
+
+A sequence owns a slot of the state; one whose first new token is at position 0 starts from zero whatever the slot holds.
+The state, the decays, the gates and the outputs are fp32; queries, keys and values come in the activation type.
+"""
+
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+
+import torch
+
+from .. import _native
+from ._util import check_rc, ptr, status_tensor, stream_handle
+
+c_int, c_ll, c_float, c_vp = ctypes.c_int, ctypes.c_longlong, ctypes.c_float, ctypes.c_void_p
+_DT = {torch.bfloat16: 0, torch.float32: 1}
+MAX_DIM = 512
+STATE_COLS = 32              # value channels of one state tile; every tile carries its own n and m
+
+
+def _up(n: int, m: int) -> int:
+    return -(-n // m) * m
+
+
+@dataclass(frozen=True)
+class RecurrentGeometry:
+    """Padded sizes of one recurrent layer and its activation. Padding channels are zero in the weights."""
+
+    heads: int
+    dim: int
+    vdim: int
+    silu: bool                   # on q, k, v
+    gated: bool                  # mLSTM gates and normaliser (otherwise a constant decay)
+
+    @property
+    def kp(self) -> int:
+        return _up(self.dim, 64)
+
+    @property
+    def vp(self) -> int:
+        return _up(self.vdim, 64)
+
+    @property
+    def tiles(self) -> int:      # state tiles of a head
+        return self.vp // STATE_COLS
+
+    @property
+    def proj(self) -> int:       # joint projection: q | k | v | output gate
+        return self.heads * (2 * self.kp + 2 * self.vp)
+
+    @property
+    def offsets(self) -> tuple[int, int, int, int]:
+        a, b = self.heads * self.kp, self.heads * self.vp
+        return 0, a, 2 * a, 2 * a + b
+
+    @property
+    def state_floats(self) -> int:       # one sequence
+        return self.heads * self.tiles * (self.kp * (STATE_COLS + 1) + 1)
+
+
+@dataclass
+class RecurrentState:
+    """State of every slot: ``s [slots, H, tiles, kp, 32]``, ``n [slots, H, tiles, kp]``, ``m [slots, H, tiles]``."""
+
+    s: torch.Tensor
+    n: torch.Tensor
+    m: torch.Tensor
+
+    @staticmethod
+    def zeros(geo: RecurrentGeometry, slots: int, device) -> "RecurrentState":
+        lead = (slots, geo.heads, geo.tiles)
+        return RecurrentState(*(torch.zeros(*lead, *tail, dtype=torch.float32, device=device) for tail in ((geo.kp, STATE_COLS), (geo.kp,), ())))
+
+
+def _lib() -> ctypes.CDLL:
+    lib = _native.load("rb_recurrent")
+    if not getattr(lib, "_rb_typed", False):
+        lib.rb_recurrent_scan.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float, c_float] + [c_vp] * 6
+                                          + [c_vp, c_ll] + [c_int] * 10 + [c_vp, c_vp])
+        lib.rb_gated_norm.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_ll] + [c_int] * 6 + [c_float, c_vp]
+        for f in ("rb_recurrent_scan", "rb_gated_norm"):
+            getattr(lib, f).restype = c_int
+        lib._rb_typed = True
+    return lib
+
+
+def capped_gates(small, bias_i, bias_f, cap: float) -> tuple[torch.Tensor, torch.Tensor]:
+    """Logarithms of input and forget gate from ``small [T, i | f]``."""
+    H = bias_i.shape[0]
+    i = cap * torch.tanh((small[:, :H] + bias_i) / cap)
+    f = torch.nn.functional.logsigmoid(cap * torch.tanh((small[:, H:2 * H] + bias_f) / cap))
+    return i, f
+
+
+def _split(proj, geo: RecurrentGeometry):
+    T, (oq, ok, ov, og) = proj.shape[0], geo.offsets
+    q, k, v = proj[:, oq:ok], proj[:, ok:ov], proj[:, ov:og]
+    q, k, v = (t.float().reshape(T, geo.heads, -1) for t in (q, k, v))
+    if geo.silu:
+        q, k, v = (torch.nn.functional.silu(t) for t in (q, k, v))
+    return q * (geo.dim ** -0.5 if geo.gated else 1.0), k, v
+
+
+def recurrent_scan(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, cap: float, state: RecurrentState, slots, cu_q, seq_lens,
+                   out, rows: int, n_seq: int) -> None:
+    """Token-by-token form for the first ``n_seq`` sequences (``rows`` packed tokens): ``out [T, H*vp]`` fp32, state updated.
+
+    ``proj [T, q | k | v | gate]``, ``small [T, i | f]`` fp32 (gated kinds), ``slots [B]`` (negative: padding), ``cu_q``
+    ``[B+1]`` (None: one row per sequence), ``seq_lens [B]`` with the new tokens."""
+    H, KP, VP = geo.heads, geo.kp, geo.vp
+    if not proj.is_cuda:
+        q, k, v = _split(proj[:rows], geo)
+        if geo.gated:
+            gi, gf = capped_gates(small[:rows], bias_i, bias_f, cap)
+        for b in range(n_seq):
+            t0, t1 = (b, b + 1) if cu_q is None else (int(cu_q[b]), int(cu_q[b + 1]))
+            slot = int(slots[b])
+            if slot < 0:
+                out[t0:t1] = 0
+                continue
+            if int(seq_lens[b]) == t1 - t0:
+                state.s[slot], state.n[slot], state.m[slot] = 0, 0, 0
+            S = state.s[slot].permute(0, 2, 1, 3).reshape(H, KP, VP)
+            n, m = state.n[slot, :, 0], state.m[slot, :, 0]
+            for t in range(t0, t1):
+                if geo.gated:
+                    new = torch.maximum(gf[t] + m, gi[t])
+                    a, w = torch.exp(gf[t] + m - new), torch.exp(gi[t] - new)
+                    m = new
+                else:
+                    a, w = decay, torch.ones_like(decay)
+                kw = k[t] * w[:, None]
+                S = a[:, None, None] * S + kw[:, :, None] * v[t][:, None, :]
+                o = torch.einsum("hkv,hk->hv", S, q[t])
+                if geo.gated:
+                    n = a[:, None] * n + kw
+                    o = o / (torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6)[:, None]
+                out[t] = o.reshape(-1)
+            state.s[slot] = S.view(H, KP, geo.tiles, STATE_COLS).permute(0, 2, 1, 3)
+            state.n[slot], state.m[slot] = n[:, None], m[:, None]
+        return
+    oq, ok, ov, _ = geo.offsets
+    assert proj.stride(1) == 1 and out.dtype == torch.float32 and out.stride(1) == 1 and geo.kp <= MAX_DIM
+    rc = _lib().rb_recurrent_scan(ptr(proj), proj.stride(0), oq, ok, ov, ptr(small), small.stride(0) if small is not None else 0, ptr(decay),
+                                  ptr(bias_i), ptr(bias_f), cap, geo.dim ** -0.5 if geo.gated else 1.0, ptr(state.s), ptr(state.n), ptr(state.m),
+                                  ptr(slots), ptr(cu_q), ptr(seq_lens), ptr(out), out.stride(0), H, geo.dim, KP, VP, n_seq, state.s.shape[0],
+                                  int(geo.silu), int(geo.gated), rows, _DT[proj.dtype], ptr(status_tensor(proj.device)),
+                                  stream_handle(proj.device))
+    check_rc(rc, "rb_recurrent_scan")
+
+
+def gated_norm(o, weight, gate, geo: RecurrentGeometry, eps: float, out, per_head: bool) -> None:
+    """``out = o / rms(o) * weight * sigmoid(gate)`` on ``[T, H*vp]``; the mean square is taken over one head's ``vdim`` channels
+    (``per_head``) or over all heads'."""
+    T, H, VP = o.shape[0], geo.heads, geo.vp
+    if not o.is_cuda:
+        x = o.view(T, H, VP)
+        ms = x.pow(2).sum(-1) / geo.vdim if per_head else (x.pow(2).sum((1, 2)) / (H * geo.vdim))[:, None].expand(T, H)
+        y = x * torch.rsqrt(ms + eps)[..., None] * weight.view(1, H, VP) * torch.sigmoid(gate.float().view(T, H, VP))
+        out[:T] = y.reshape(T, H * VP).to(out.dtype)
+        return
+    assert o.dtype == torch.float32 and o.stride(1) == gate.stride(1) == out.stride(1) == 1 and gate.dtype == out.dtype
+    rc = _lib().rb_gated_norm(ptr(o), o.stride(0), ptr(weight), ptr(gate), gate.stride(0), ptr(out), out.stride(0), H, geo.vdim, VP, int(per_head),
+                              T, _DT[out.dtype], eps, stream_handle(o.device))
+    check_rc(rc, "rb_gated_norm")
