@@ -786,7 +786,7 @@ def run_reference_train(args) -> dict:
 
 
 def run_stack(args) -> dict:
-    """One GPU: the layer-stack design against its closest neighbour in the framework (``utils/stack_bench.py``)."""
+    """One GPU: the layer-stack designs against their closest neighbours in the framework (``utils/stack_bench.py``)."""
     from research_b200.utils import stack_bench
     from research_b200.utils.timing import ClockSampler
 
@@ -794,7 +794,7 @@ def run_stack(args) -> dict:
         return {"impl": args.impl, "unavailable": "the stack workload runs natively on one GPU"}
     sampler = ClockSampler(0)
     sampler.start()
-    res = stack_bench.run(tuple(x for x in args.sizes.split(",") if x))
+    res = stack_bench.run(tuple(x for x in args.sizes.split(",") if x), designs=tuple(x for x in args.designs.split(",") if x))
     return {"metric": "prefill and decode of a layer-stack model, tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
             "higher_is_better": True, "clocks": sampler.stop(), **res}
 
@@ -812,8 +812,9 @@ def main() -> None:
                     help="train = sharded training step on the Llama-3-8B shape, seq 4096, one sequence per GPU (the flagship); "
                          "rollout = engine decode, 1024 requests, prompts U[128,1024], 512 new tokens, batch 256; "
                          "serving = batch 64, prompts of 2048 tokens, 256 new tokens (the tensor-parallel serving case); "
-                         "stack = prefill and decode of a layer-stack model beside a Llama-type model of equal size, kernel by kernel")
+                         "stack = prefill and decode of layer-stack models beside the closest model of equal size, kernel by kernel")
     ap.add_argument("--sizes", default="", help="stack: comma-separated sizes (default: all)")
+    ap.add_argument("--designs", default="", help="stack: comma-separated designs, lulezen or zamusun (default: both)")
     ap.add_argument("--model", default=None, help="model preset (default: llama-3-8b for train / serving, qwen2.5-0.5b for rollout)")
     ap.add_argument("--seq", type=int, default=TRAIN_SEQ, help="train: tokens per sequence")
     ap.add_argument("--batch", type=int, default=TRAIN_BATCH_PER_GPU, help="train: sequences per GPU per step")

@@ -2,6 +2,7 @@
 
 from __future__ import annotations
 
+import weakref
 from typing import Any, Callable
 
 import torch
@@ -18,7 +19,7 @@ class Part:
     feed-forwards, fills ``y [T, wp]`` (fp32)."""
 
     def __init__(self, runner):
-        self.r = runner
+        self.r = weakref.proxy(runner)       # no cycle: the runner's graphs go when its engine does
         self.layers: list[Any] = []          # weights made so far
         self.specs: list[Any] = []
 

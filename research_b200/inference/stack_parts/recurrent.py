@@ -81,6 +81,10 @@ class RecurrentPart(Part):
         proj = self.proj[:T * g.proj].view(T, g.proj)
         o, out = self.o[:T * n].view(T, n), self.out[:T * n].view(T, n)
         ops.gemm(inp, w.wproj, out=proj)
-        ops.recurrent_scan(proj, small, g, w.decay, w.bias_i, w.bias_f, w.cap, state, b.state_slots, b.cu_q, b.seq_lens, o, T, b.rows)
+        self.recur(w, state, proj, small, o, b, plan)
         ops.gated_norm(o, w.norm, proj[:, g.offsets[3]:], g, self.r.cfg.norm_eps, out, g.gated)
         ops.gemm(out, w.wo, out=y, out_f32=True)
+
+    def recur(self, w: RecurrentWeights, state: RecurrentState, proj, small, o, b, plan) -> None:
+        """``o`` from the projected rows, and the state of the batch's sequences moved on."""
+        ops.recurrent_scan(proj, small, w.geo, w.decay, w.bias_i, w.bias_f, w.cap, state, b.state_slots, b.cu_q, b.seq_lens, o, b.num_tokens, b.rows)

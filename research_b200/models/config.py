@@ -13,7 +13,8 @@ import json
 from dataclasses import asdict, dataclass, field, replace
 from pathlib import Path
 
-from .stack import ClampedGluSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, RotarySpec, uniform_stack
+from .stack import (ClampedGluSpec, ExpertsSpec, KeyValueAttentionSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec, LoopSpec,
+                    MatrixMemorySpec, QueryTemperature, RotarySpec, uniform_stack)
 
 
 @dataclass(frozen=True)
@@ -143,6 +144,18 @@ def _latent(heads: int, dim: int, rot: int, vdim: int, kv_rank: int, q_rank: int
     return LatentAttentionSpec(heads, dim, rot, vdim, kv_rank, q_rank, (dim + rot) ** -0.5, window, RotarySpec(rot, base))
 
 
+def _memory(heads: int, dim: int, vdim: int) -> MatrixMemorySpec:
+    return MatrixMemorySpec(heads, dim, vdim, 15.0)
+
+
+def _lightning(heads: int, dim: int, vdim: int) -> LightningSpec:
+    return LightningSpec(heads, dim, vdim, tuple(1 - 2.0 ** -(2 + 6 * h / heads) for h in range(heads)))
+
+
+def _keyvalue(heads: int, kv_heads: int, dim: int, every: int) -> KeyValueAttentionSpec:
+    return KeyValueAttentionSpec(heads, kv_heads, dim, dim ** -0.5, QueryTemperature(0.1, every))
+
+
 PRESETS: dict[str, ModelConfig | LayerStackConfig] = {
     # tiny CPU plumbing model: Qwen2-style, vocab 4096, 4 layers, d 256, 4q/2kv heads
     "tiny-qwen2": ModelConfig(),
@@ -174,6 +187,14 @@ PRESETS: dict[str, ModelConfig | LayerStackConfig] = {
                                 mlp=ClampedGluSpec(8192, 7.0), logit_softcap=30.0),
     "lulezen-7b": uniform_stack("Lulezen", vocab=128256, width=4096, num_layers=32, mixer=_latent(32, 128, 64, 128, 512, 1536, 4096),
                                 mlp=ClampedGluSpec(14336, 7.0), logit_softcap=30.0),
+    # layer stacks with recurrent mixers, keys-as-values attention, routed experts and a looped pair of layers
+    "tiny-zamusun": LayerStackConfig("Zamusun", 4096, 160, (
+        LayerSpec(_memory(3, 40, 24), ExpertsSpec(5, 2, ClampedGluSpec(96, 4.0))),
+        LayerSpec(_lightning(4, 24, 36), None),
+        LayerSpec(_keyvalue(6, 2, 40, 64), ExpertsSpec(5, 2, ClampedGluSpec(96, 4.0)))), loop=LoopSpec(1, 3, 2), init_std=0.05),
+    "zamusun-4b": LayerStackConfig("Zamusun", 128256, 2048, tuple(
+        LayerSpec((_memory(16, 128, 128), _lightning(16, 128, 128), _keyvalue(16, 4, 128, 1024))[i % 3], ExpertsSpec(64, 8, ClampedGluSpec(768, 7.0)))
+        for i in range(12)), loop=LoopSpec(0, 3, 2)),
 }
 
 

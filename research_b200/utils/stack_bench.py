@@ -1,8 +1,9 @@
-"""Prefill and decode throughput of a layer-stack model beside the closest Hugging Face style model of equal size.
+"""Prefill and decode throughput of layer-stack models beside the closest Hugging Face style model of equal size.
 
-``bench.py --workload stack`` runs it. For every size two engines are built with random weights: the latent-attention
-stack and a Llama-type model with the same width, layers, feed-forward, vocabulary and heads (grouped queries, head size
-128). Measured with CUDA events, after warm-up:
+``bench.py --workload stack`` runs it (``--designs``, ``--sizes`` choose). For every size two engines are built with random
+weights: Lulezen (latent attention) beside a Llama-type model, Zamusun (recurrent mixers, keys-as-values attention, routed
+experts, a looped pair of layers) beside a Qwen3-MoE-type model, each with the same width, layer runs, feed-forward,
+vocabulary and heads (grouped queries, head size 128). Measured with CUDA events, after warm-up:
 
 * decode: one captured decode step at the given batch and context, replayed;
 * prefill: one packed pass over a whole prompt;
@@ -23,7 +24,9 @@ from .. import ops
 from ..inference import EngineConfig, InferenceEngine
 from ..models import LazyRandomWeights
 from ..models.config import ModelConfig
-from ..models.stack import ClampedGluSpec, LatentAttentionSpec, RotarySpec, uniform_stack
+from ..models.stack import (ClampedGluSpec, ExpertsSpec, KeyValueAttentionSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec,
+                            LoopSpec, MatrixMemorySpec, QueryTemperature, RotarySpec, uniform_stack)
+from ..ops import experts as ex
 from .timing import flush_l2, time_cuda
 
 
@@ -42,6 +45,22 @@ class Size:
 
 
 SIZES = (Size("1b", 2048, 8, 16, 4, 8192, 32000, 1024), Size("7b", 4096, 8, 32, 8, 14336, 32000, 1536))
+
+
+@dataclass(frozen=True)
+class ExpertSize:
+    name: str
+    width: int
+    runs: int                # layer runs; two of the layers are looped twice, so there are runs - 2 layers
+    heads: int
+    kv_heads: int
+    experts: int
+    top: int
+    ff: int
+    vocab: int
+
+
+EXPERT_SIZES = (ExpertSize("w2048", 2048, 8, 16, 4, 64, 8, 768, 32000), ExpertSize("w4096", 4096, 8, 32, 8, 16, 2, 4096, 32000))
 
 
 def peaks() -> tuple[float, float, str]:
@@ -63,6 +82,19 @@ def configs(s: Size):
     return stack, llama
 
 
+def expert_configs(s: ExpertSize):
+    H = s.heads
+    memory, linear = MatrixMemorySpec(H, 128, 128, 15.0), LightningSpec(H, 128, 128, tuple(1 - 2.0 ** -(2 + 6 * h / H) for h in range(H)))
+    attention = KeyValueAttentionSpec(H, s.kv_heads, 128, 128 ** -0.5, QueryTemperature(0.1, 1024))
+    mlp = ExpertsSpec(s.experts, s.top, ClampedGluSpec(s.ff, 7.0))
+    kinds = (memory, linear, attention)
+    stack = LayerStackConfig("Zamusun", s.vocab, s.width, tuple(LayerSpec(kinds[i % 3], mlp) for i in range(s.runs - 2)), loop=LoopSpec(0, 2, 2))
+    moe = ModelConfig(family="qwen3_moe", vocab_size=s.vocab, hidden_size=s.width, num_layers=s.runs, num_heads=H, num_kv_heads=s.kv_heads,
+                      head_dim=128, intermediate_size=s.ff, rope_theta=5e5, tie_word_embeddings=True, attention_bias=False, qk_norm=True,
+                      num_experts=s.experts, num_experts_per_tok=s.top, moe_intermediate_size=s.ff)
+    return stack, moe
+
+
 def _engine(cfg, batch: int, context: int, prompt: int) -> InferenceEngine:
     w = LazyRandomWeights(cfg, seed=0, dtype=torch.bfloat16, device="cuda")
     blocks = batch * (-(-context // 16)) + 2 * (-(-prompt // 16))
@@ -82,6 +114,7 @@ def _stage_decode(r, batch: int, context: int) -> None:
     m[mb:mb + batch] = context - 1
     m[2 * mb:2 * mb + batch] = perm[:, (context - 1) // 16] * 16 + (context - 1) % 16
     m[3 * mb:3 * mb + batch] = context
+    m[7 * mb:7 * mb + batch] = torch.arange(batch, dtype=torch.int32)
     r.meta_dev.copy_(m)
 
 
@@ -115,6 +148,7 @@ def time_prefill(eng: InferenceEngine, prompt: int, iters: int = 8) -> float:
     ph[o["cu_q"]:o["cu_q"] + 2] = torch.tensor([0, n], dtype=torch.int32)
     ph[o["seq_lens"]] = n
     ph[o["sample_rows"]] = n - 1
+    ph[o["state_slots"]] = 0
     r.bt_host[0, :-(-n // 16)] = torch.arange(-(-n // 16), dtype=torch.int32)
     return time_cuda(lambda: r.prefill(1, n, n, -(-n // 16)), iters=iters, flush=False)["median_ms"]
 
@@ -134,11 +168,12 @@ class _Table:
         self.add(name, call, 2 * (M * K + N * K) + out_bytes * M * (out_cols or N), 2.0 * M * N * K)
 
 
-def stack_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict:
+def latent_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict:
     """Time every kernel of the first layer at ``T`` rows: decode rows with ``context`` keys each, or one prompt of T tokens."""
     r, cfg, t = eng.runner, eng.runner.cfg, _Table()
-    lw = r.layers[0]
-    g, b, m = lw.geo, r.bufs[lw.geo], lw.spec.mixer
+    layer = r.layers[0]
+    lw, part, cache = layer.mix, layer.mixer, r.runs[0].cache
+    g, b, m = lw.geo, part.bufs[lw.geo], lw.spec
     H, d = g.heads, cfg.hidden_size
     x, xb, y = r.x[:T], r.xb[:T], r.y[:T]
     pos = torch.full((T,), context - 1, dtype=torch.int32, device="cuda") if decode else torch.arange(T, dtype=torch.int32, device="cuda")
@@ -146,7 +181,7 @@ def stack_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> d
     n_short = T if decode else 0
     t.gemm("joint down projection", T, g.proj, r.wp, lambda: ops.gemm(xb, lw.wproj, out=b.proj[:T], out_f32=True), 4)
     t.add("norms + rotation + append", lambda: ops.latent_append(b.proj[:T], g, lw.q_norm, lw.kv_norm, cfg.norm_eps, pos, slots, lw.table,
-                                                                 lw.cache, b.cq, b.gate), T * (4 * g.proj + 2 * g.qp + 2 * g.cw), 0)
+                                                                 cache, b.cq, b.gate), T * (4 * g.proj + 2 * g.qp + 2 * g.cw), 0)
     q = b.q[:T]
     t.gemm("query up projection", T, q.shape[1], g.qp, lambda: ops.gemm(b.cq[:T], lw.wuq, out=q))
     rot_bytes = T * H * (2 * 2 * (g.dp + g.rp) if decode else 2 * 2 * g.rp)
@@ -154,11 +189,11 @@ def stack_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> d
     if decode:
         bt, lens = r.bt_dev[:T], r.d_lens[:T]
         span = min(context, m.window)
-        plan = r.decode_plans[(g, m.window)]
+        plan = part.decode_plans[(g, m.window)]
         ops.latent_plan(None, lens, g, 1, m.window, plan)
         t.add("absorb W_uk", lambda: ops.head_gemm_absorb(b.qn, lw.wuk, b.qa, T), 2 * H * (g.dp * g.rw + T * (g.dp + g.rw)), 2.0 * T * H * g.dp * g.rw)
-        t.add("attention", lambda: ops.latent_attention(b.qa, lw.cache, g, bt, None, lens, lw.sink, b.gate, b.ol, scale=m.scale, window=m.window,
-                                                        rows=T, max_q=1, plan=plan, workspace=r.attn_ws),
+        t.add("attention", lambda: ops.latent_attention(b.qa, cache, g, bt, None, lens, lw.sink, b.gate, b.ol, scale=m.scale, window=m.window,
+                                                        rows=T, max_q=1, plan=plan, workspace=part.workspace),
               2 * T * (span * g.cw + H * (g.cw + g.rw)), 2.0 * T * H * span * (g.cw + g.rw))
         t.add("expand W_uv", lambda: ops.head_gemm_expand(b.ol, lw.wuv, b.attn, T), 2 * H * (g.vp * g.rw + T * (g.vp + g.rw)), 2.0 * T * H * g.vp * g.rw)
     else:
@@ -167,7 +202,7 @@ def stack_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> d
         lo = torch.zeros(1, dtype=torch.int32, device="cuda")
         lat = torch.empty(T, g.rw, dtype=torch.bfloat16, device="cuda")
         rot = torch.empty(T, g.rp, dtype=torch.bfloat16, device="cuda")
-        t.add("gather latents", lambda: ops.latent_gather(lw.cache, g, bt, 0, cu, lo, T, lat, rot), 2 * 2 * T * g.cw, 0)
+        t.add("gather latents", lambda: ops.latent_gather(cache, g, bt, 0, cu, lo, T, lat, rot), 2 * 2 * T * g.cw, 0)
         k, v = ops.gemm(lat, lw.wuk), ops.gemm(lat, lw.wuv)
         t.gemm("keys", T, k.shape[1], g.rw, lambda: ops.gemm(lat, lw.wuk, out=k))
         t.gemm("values", T, v.shape[1], g.rw, lambda: ops.gemm(lat, lw.wuv, out=v))
@@ -176,17 +211,95 @@ def stack_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> d
                                                             max_q=T, rows=T),
               2 * T * H * (2 * g.dp + g.rp + 2 * g.vp), 2.0 * pairs * H * (g.dp + g.rp + g.vp))
     t.gemm("output projection", T, r.wp, H * g.vp, lambda: ops.gemm(b.attn[:T], lw.wo, out=y, out_f32=True), 4)
-    t.add("norm + residual", lambda: ops.layernorm_residual(y, lw.norm1[0], lw.norm1[1], cfg.norm_eps, x, xb), T * d * 14, 0)
-    act = r._act[:T * lw.ffp].view(T, lw.ffp)
-    t.gemm("gate|up + unit", T, 2 * lw.ffp, r.wp, lambda: ops.gemm(xb, lw.wgu, out=act, bn=r.glu_bn, swiglu=True, glu_limit=lw.glu.limit), 2, lw.ffp)
-    t.gemm("down projection", T, r.wp, lw.ffp, lambda: ops.gemm(act, lw.wd, out=y, out_f32=True), 4)
+    t.add("norm + residual", lambda: ops.layernorm_residual(y, layer.norm1[0], layer.norm1[1], cfg.norm_eps, x, xb, d), T * d * 14, 0)
+    ff = layer.ff
+    act = layer.feed_forward.act[:T * ff.ffp].view(T, ff.ffp)
+    t.gemm("gate|up + unit", T, 2 * ff.ffp, r.wp, lambda: ops.gemm(xb, ff.wgu, out=act, bn=256, swiglu=True, glu_limit=ff.spec.limit), 2, ff.ffp)
+    t.gemm("down projection", T, r.wp, ff.ffp, lambda: ops.gemm(act, ff.wd, out=y, out_f32=True), 4)
     if decode:
         lg = r.logits_padded[:T]
         t.gemm("head + cap", T, r.vp, r.wp, lambda: r._head(r.hl[:T], lg), 4)
     return t.rows
 
 
-def llama_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict:
+def _routed(t: _Table, T: int, E: int, k: int, d: int, ff: int, up, down, unit=None, others: dict | None = None) -> None:
+    """Rows of the routed experts: ``others`` are the small launches around the two grouped products."""
+    n = T * k
+    active = min(E, n)
+    for name, (fn, nbytes) in (others or {}).items():
+        t.add(name, fn, nbytes, 0)
+    t.add("experts gate|up", up, 2 * (n * d + active * 2 * ff * d + n * (ff if unit is None else 2 * ff)), 4.0 * n * d * ff)
+    if unit is not None:
+        t.add("experts unit", unit, 2 * 3 * n * ff, 0)
+    t.add("experts down", down, 2 * (n * ff + active * ff * d + n * d), 2.0 * n * d * ff)
+
+
+def expert_stack_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict:
+    """The first layer of every kind of mixer, the routed experts and what joins them."""
+    r, cfg, t = eng.runner, eng.runner.cfg, _Table()
+    d, eps = cfg.hidden_size, cfg.norm_eps
+    x, h, y = r.x[:T], r.xb[:T], r.y[:T]
+    h.normal_()
+    i32 = dict(dtype=torch.int32, device="cuda")
+    if decode:
+        b = r._decode_batch(T)
+    else:
+        pos = torch.arange(T, **i32)
+        b = type(r._decode_batch(2))(rows=1, num_tokens=T, padded=T, max_new=T, tokens=pos, positions=pos, slots=pos, cu_q=torch.tensor([0, T], **i32),
+                                     seq_lens=torch.tensor([T], **i32), block_tables=torch.arange(-(-T // 16), **i32)[None].contiguous(),
+                                     host_cu_q=[0, T], host_seq_lens=[T], state_slots=torch.zeros(1, **i32), n_single=0)
+    seen = set()
+    for run in r.runs:
+        lw = run.layer
+        w, part, kind = lw.mix, lw.mixer, lw.spec.mixer.type
+        if kind in seen:
+            continue
+        seen.add(kind)
+        g, plan = w.geo, part.plan(b)
+        proj = part.proj[:T * g.proj].view(T, g.proj)
+        t.gemm(f"{kind}: joint projection", T, g.proj, r.wp, lambda: ops.gemm(h, w.wproj, bias=getattr(w, "bproj", None), out=proj))
+        if kind == "attention":
+            H, G, D, m = g.heads, g.kv_heads, g.dp, w.spec
+            out = part.out[:T * H * D].view(T, H * D)
+            t.add("attention: temperature + append", lambda: ops.kv_append(proj, g, b.positions, b.slots, m.q_temp.coef, m.q_temp.every, run.cache),
+                  2 * T * D * (2 * H + 2 * G), 0)
+            fn = lambda: ops.kv_attention(proj, g, run.cache, b.block_tables, b.cu_q, b.seq_lens, w.sink, out, scale=m.scale, rows=T, max_q=b.max_new,
+                                          n_single=b.n_single, workspace=part.workspace, splits=plan.get(g, 1))
+            if decode:
+                t.add("attention: attention", fn, 2 * T * (context * G * D + 3 * H * D), 4.0 * T * H * context * D)
+            else:
+                t.add("attention: attention", fn, 2 * T * D * (3 * H + G), 4.0 * (T * (T + 1) / 2) * H * D)
+            n = H * D
+        else:
+            H, n = g.heads, g.heads * g.vp
+            o, out = part.o[:T * n].view(T, n), part.out[:T * n].view(T, n)
+            small = r._small_rows(h, lw.wsmall)
+            io = T * H * (2 * (2 * g.kp + g.vp) + 4 * g.vp)
+            state = 2 * 4 * H * g.kp * (g.vp + (1 if g.gated else 0))
+            t.add(f"{kind}: recurrence", lambda: part.recur(w, run.cache, proj, small, o, b, plan), io + state * b.rows,
+                  T * H * (4.0 * g.kp * g.vp + (0 if decode else 2.0 * 64 * (g.kp + g.vp))))
+            t.add(f"{kind}: norm + gate", lambda: ops.gated_norm(o, w.norm, proj[:, g.offsets[3]:], g, eps, out, g.gated), T * n * 8, 0)
+        t.gemm(f"{kind}: output projection", T, r.wp, n, lambda: ops.gemm(out, w.wo, bias=getattr(w, "bo", None), out=y, out_f32=True), 4)
+    lw = r.layers[0]
+    t.gemm("gate logits + router", T, lw.wsmall.shape[0], r.wp, lambda: r._small_rows(h, lw.wsmall), 4)
+    logits = r._small_rows(h, lw.wsmall)[:, lw.mix_small:]
+    w, g = lw.ff, lw.ff.geo
+    sc = lw.feed_forward.scratch[g]
+    _routed(t, T, g.experts, g.top, d, g.ff, lambda: ex.experts_up(g, sc, w.wgu, T), lambda: ex.experts_down(g, sc, w.wd), None,
+            {"experts route + plan": (lambda: ex.experts_plan(logits, g, sc), T * (4 * g.experts + 8 * g.top)),
+             "experts gather": (lambda: (ex.experts_plan(logits, g, sc), ex.experts_gather(h, g, sc)), 2 * 2 * T * g.top * d)})
+    t.add("residual + experts' sum + norm", lambda: ops.stream_norm(x, d, y1=y, experts=sc.y[:T * g.top], expert_weights=sc.w[:T], weight=lw.norm1[0],
+                                                                     eps=eps, h=h), T * d * (4 * 3 + 2 + 2 * g.top), 0)
+    if r.loop_in is not None:
+        t.gemm("loop entry", T, r.wp, 2 * r.wp, lambda: r._enter_pass(T), 4)
+    if decode:
+        lg = r.logits_padded[:T]
+        t.gemm("head", T, r.vp, r.wp, lambda: r._head(r.hl[:T], lg), 4)
+    return t.rows
+
+
+def hf_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict:
+    """The first layer of a Hugging Face style model (dense or routed experts)."""
     r, cfg, t = eng.runner, eng.runner.cfg, _Table()
     lw = r.layers[0]
     d, Hq, Hkv, D = cfg.hidden_size, r.Hq, r.Hkv, r.D
@@ -213,40 +326,62 @@ def llama_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> d
               2 * T * D * (2 * Hq + 2 * Hkv), 4.0 * (T * (T + 1) / 2) * Hq * D)
     t.gemm("output projection", T, d, Hq * D, lambda: ops.gemm(o.view(T, Hq * D), lw.wo, residual=x, out=x))
     t.add("norm", lambda: ops.rmsnorm(x, lw.ln2, eps, out=h), 4 * T * d, 0)
-    act = torch.empty(T, r.F, dtype=torch.bfloat16, device="cuda")
-    t.gemm("gate|up + unit", T, 2 * r.F, d, lambda: ops.gemm(h, lw.wgu, out=act, bn=r.swiglu_bn, swiglu=True, norm_eps=fold), 2, r.F)
-    t.gemm("down projection", T, d, r.F, lambda: ops.gemm(act, lw.wd, residual=x, out=x))
+    if lw.moe is not None:
+        m = lw.moe
+        h.normal_()
+        m.forward(h, x)
+        n = T * m.k
+        t.add("experts layer, all launches", lambda: m.forward(h, x), 2 * (min(m.E, n) * 3 * m.F * d + 2 * T * d), 6.0 * n * d * m.F)
+        t.gemm("router", T, m.E, d, lambda: ops.gemm(h, m.gate, out=m.logits[:T], out_f32=True), 4)
+        _routed(t, T, m.E, m.k, d, m.F, lambda: m._grouped(m.xp, m.wgu, m.gu, 2 * m.F, d, m.BN_GU, m.tiles_gu, m.ntiles.data_ptr(), None),
+                lambda: m._grouped(m.act, m.wd, None, d, m.F, m.BN_DN, m.tiles_dn, m.ntiles.data_ptr() + 4, m.ret),
+                lambda: ops.swiglu(m.gu[:n], out=m.act[:n]))
+    else:
+        act = torch.empty(T, r.F, dtype=torch.bfloat16, device="cuda")
+        t.gemm("gate|up + unit", T, 2 * r.F, d, lambda: ops.gemm(h, lw.wgu, out=act, bn=r.swiglu_bn, swiglu=True, norm_eps=fold), 2, r.F)
+        t.gemm("down projection", T, d, r.F, lambda: ops.gemm(act, lw.wd, residual=x, out=x))
     if decode:
         t.gemm("head", T, cfg.vocab_size, d, lambda: ops.gemm(h, r.lm_head, out=r.a_logits[:T], out_f32=True), 4)
     return t.rows
 
 
+# design -> (sizes, pair of configurations, labels and kernel tables)
+DESIGNS = {"lulezen": (SIZES, configs, (("lulezen", latent_kernels), ("llama", hf_kernels))),
+           "zamusun": (EXPERT_SIZES, expert_configs, (("zamusun", expert_stack_kernels), ("qwen3_moe", hf_kernels)))}
+
+
 def run(sizes: tuple[str, ...] = (), batches: tuple[int, ...] = (1, 64, 256), context: int = 2048, prompts: tuple[int, ...] = (512, 4096),
-        kernels: bool = True) -> dict:
+        kernels: bool = True, designs: tuple[str, ...] = ()) -> dict:
     out: dict = {"peaks": dict(zip(("hbm_bytes_s", "bf16_flop_s", "origin"), peaks())), "context": context, "sizes": {}}
-    for s in SIZES:
-        if sizes and s.name not in sizes:
+    for design, (all_sizes, make, sides) in DESIGNS.items():
+        if designs and design not in designs:
             continue
-        res: dict = {"shape": {k: getattr(s, k) for k in ("width", "layers", "heads", "kv_heads", "ff", "vocab", "q_rank", "kv_rank", "window")}}
-        for label, cfg in zip(("lulezen", "llama"), configs(s)):
-            one: dict = {"params_m": round(cfg.num_params() / 1e6), "decode": {}, "prefill": {}, "decode_kernels": {}, "prefill_kernels": {}}
-            table = stack_kernels if label == "lulezen" else llama_kernels
-            for B in batches:
-                eng = _engine(cfg, max(B, 2), context, max(prompts))
-                ms = time_decode(eng, B, context)
-                one["decode"][B] = {"ms": round(ms, 4), "tok_s": round(B / ms * 1e3)}
-                if B == batches[-1]:
-                    if kernels:
-                        one["decode_kernels"] = table(eng, B, context, True)
-                    for n in prompts:
-                        ms = time_prefill(eng, n)
-                        one["prefill"][n] = {"ms": round(ms, 3), "tok_s": round(n / ms * 1e3)}
-                    if kernels:
-                        one["prefill_kernels"] = table(eng, prompts[-1], context, False)
-                ops.check_status()
-                eng.shutdown()
-                del eng
-                torch.cuda.empty_cache()
-            res[label] = one
-        out["sizes"][s.name] = res
+        for s in all_sizes:
+            if sizes and s.name not in sizes:
+                continue
+            res: dict = {"shape": {k: v for k, v in s.__dict__.items() if k != "name"}}
+            for (label, table), cfg in zip(sides, make(s)):
+                res[label] = _measure(cfg, table, batches, context, prompts, kernels)
+            out["sizes"][f"{design} {s.name}"] = res
     return out
+
+
+def _measure(cfg, table, batches, context: int, prompts, kernels: bool) -> dict:
+    one: dict = {"params_m": round(cfg.num_params() / 1e6), "decode": {}, "prefill": {}, "decode_kernels": {}, "prefill_kernels": {}}
+    for B in batches:
+        eng = _engine(cfg, max(B, 2), context, max(prompts))
+        ms = time_decode(eng, B, context)
+        one["decode"][B] = {"ms": round(ms, 4), "tok_s": round(B / ms * 1e3)}
+        if B == batches[-1]:
+            if kernels:
+                one["decode_kernels"] = table(eng, B, context, True)
+            for n in prompts:
+                ms = time_prefill(eng, n)
+                one["prefill"][n] = {"ms": round(ms, 3), "tok_s": round(n / ms * 1e3)}
+            if kernels:
+                one["prefill_kernels"] = table(eng, prompts[-1], context, False)
+        ops.check_status()
+        eng.shutdown()
+        del eng
+        torch.cuda.empty_cache()
+    return one

@@ -185,7 +185,7 @@ def test_whole_prompts_portions_and_single_tokens(name, place):
         assert error(feed_all(eng, toks, portions), want) < TOL[place[1]], portions
     assert eng.check_invariants() == 0 and eng.cache_stats()["free_blocks"] == 64
     if place == ("cuda", "bfloat16"):
-        assert eng.runner.expand == (name != "no_expand")
+        assert eng.runner.layers[0].mixer.expand == (name != "no_expand")
 
 
 @pytest.mark.parametrize("place", PLACES)
