@@ -5,6 +5,9 @@
 //   scan        token by token: decoded tokens, short portions and the exact mode. One CTA per (sequence, head, 32 value
 //               channels); the state tile stays in registers over the tokens of the portion. A decoded token reads and writes
 //               the state once, which is what bounds it.
+//   chunked     long portions, 128 tokens at a time on the tensor cores (tcgen05), in three launches: what every chunk adds to the
+//               state (all chunks at once), the state in front of every chunk (one pass over the chunks), the outputs (all
+//               chunks at once)
 //   gated_norm  RMS norm per head or over all heads, times sigmoid(gate), to the activation type
 //
 // State: s [slots, H, tiles, KP, 32], n [slots, H, tiles, KP], m [slots, H, tiles], all fp32. A tile of 32 value channels keeps its
@@ -182,6 +185,569 @@ static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
 }
 
 // ------------------------------------------------------------------------------------------
+// Chunked form. In a chunk of up to CH tokens of one sequence let F_t be the sum of the logarithms of the decays up to and
+// including token t, g_j = log b_j - F_j, and (m, S, n) the state in front of the chunk. Then with B_t = max(m, max_{j<=t} g_j)
+//
+//   numerator_t   = sum_{j<=t} exp(g_j - B_t) (q_t . k_j) v_j  +  exp(m - B_t) S^T q_t
+//   normaliser_t  = the same with v_j = 1 and n for S,           m_t = F_t + B_t
+//
+// and with G = max_j g_j the chunk itself contributes U = sum_j exp(g_j - G) k_j v_j^T (relative to exp(F_C + G)) to the state
+// behind it. A constant decay has no normaliser and no maximum: there B_t = -F_t, G = -F_C and m = 0 throughout.
+//
+// Products on the tensor cores take bf16 operands; the incoming state and the weighted keys are split into two bf16 parts
+// each, so that what is carried from chunk to chunk keeps 16 bits of mantissa per product and fp32 sums.
+// ------------------------------------------------------------------------------------------
+constexpr int CH = 128;                   // tokens of a chunk
+constexpr int CHT = 256;                  // threads
+constexpr int CH_ROWB = 128;              // bytes of a swizzled row: 64 bf16
+constexpr int CH_CHUNK = CH * CH_ROWB;    // 64 columns of a [CH, .] tile
+constexpr float LOG2E = 1.4426950408889634f;
+
+struct ChunkParams {
+  const __nv_bfloat16* proj;
+  long long ld;
+  int q_col, k_col, v_col;
+  const float* small;
+  long long ld_small;
+  const float* decay;
+  const float* bias_i;
+  const float* bias_f;
+  float cap, q_scale;
+  const int4* chunks;      // {first packed row, tokens, sequence, 1 when it starts the sequence's portion}
+  const int* seq_chunks;   // [n_seq + 1] first chunk of every sequence
+  const int* slots;        // [n_seq]
+  const int* seq_lens;     // [n_seq]
+  const int* cu_q;         // [n_seq + 1]
+  float* s;
+  float* n;
+  float* m;
+  float* u;                // [chunks, H, tiles, KP, 32]
+  float* un;               // [chunks, H, KP]
+  float2* um;              // [chunks, H] {F_C, F_C + G}
+  __nv_bfloat16* s_hi;     // [chunks, H, VP/64, KP, 64] state in front of the chunk
+  __nv_bfloat16* s_lo;
+  float* s_n;              // [chunks, H, KP]
+  float* s_m;              // [chunks, H]
+  float* out;
+  long long ldo;
+  int H, dk, KP, VP, num_slots, silu, gated;
+  int* status;
+};
+
+__device__ __forceinline__ float chunk_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// g_j and F_j of the chunk's tokens (in units of log2), by the first warp: four tokens per lane. Invalid tokens get g = -inf.
+// gs[t] = g_t, bs[t] = running maximum of g (gated) or -F_t, fs[t] = F_t. Returns {F_C, max g} in every lane of the warp.
+__device__ __forceinline__ float2 chunk_gates(const ChunkParams& p, int h, int row0, int n, float* gs, float* bs, float* fs = nullptr) {
+  const int lane = threadIdx.x & 31;
+  float lf[4], li[4], F[4], run = 0.f;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int t = lane * 4 + i;
+    lf[i] = 0.f;
+    li[i] = 0.f;
+    if (t < n) {
+      if (p.gated) {
+        const float* g = p.small + (long long)(row0 + t) * p.ld_small;
+        li[i] = p.cap * tanhf((g[h] + p.bias_i[h]) / p.cap) * LOG2E;
+        lf[i] = log_sigmoid_f(p.cap * tanhf((g[p.H + h] + p.bias_f[h]) / p.cap)) * LOG2E;
+      } else {
+        lf[i] = logf(fmaxf(p.decay[h], 1e-30f)) * LOG2E;
+      }
+    }
+    run += lf[i];
+    F[i] = run;
+  }
+  float before = run;                                      // exclusive scan of the lanes' sums
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float y = __shfl_up_sync(0xffffffffu, before, o);
+    if (lane >= o) before += y;
+  }
+  const float total = __shfl_sync(0xffffffffu, before, 31);
+  before -= run;
+  float mx = -INFINITY, g[4], top[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    F[i] += before;
+    g[i] = lane * 4 + i < n ? li[i] - F[i] : -INFINITY;
+    mx = fmaxf(mx, g[i]);
+    top[i] = mx;
+  }
+  float up = mx;                                           // running maximum over the lanes before this one
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float y = __shfl_up_sync(0xffffffffu, up, o);
+    if (lane >= o) up = fmaxf(up, y);
+  }
+  const float all = __shfl_sync(0xffffffffu, up, 31);
+  float prev = __shfl_up_sync(0xffffffffu, up, 1);
+  if (lane == 0) prev = -INFINITY;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    gs[lane * 4 + i] = g[i];
+    bs[lane * 4 + i] = p.gated ? fmaxf(prev, top[i]) : -F[i];
+    if (fs != nullptr) fs[lane * 4 + i] = F[i];
+  }
+  return make_float2(total, all);
+}
+
+// 16-byte unit u (8 columns) of row r in a [rows, 64] swizzled chunk
+__device__ __forceinline__ uint32_t chunk_addr(int r, int u) { return (uint32_t)(r * CH_ROWB + ((u ^ (r & 7)) << 4)); }
+
+__device__ __forceinline__ uint4 silu8(uint4 v) {
+  auto one = [](uint32_t x) {
+    const float2 f = unpack_bf16x2(x);
+    return pack_bf16x2(silu_f(f.x), silu_f(f.y));
+  };
+  return make_uint4(one(v.x), one(v.y), one(v.z), one(v.w));
+}
+
+// [CH, DK] columns of a projection into swizzled chunks; rows past n are zero
+template <int DK>
+__device__ __forceinline__ void chunk_load(uint8_t* dst, const __nv_bfloat16* src, long long ld, int n, bool silu) {
+#pragma unroll 4
+  for (int i = threadIdx.x; i < CH * (DK / 8); i += CHT) {
+    const int r = i / (DK / 8), u = i % (DK / 8);
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (r < n) {
+      v = *reinterpret_cast<const uint4*>(src + r * ld + u * 8);
+      if (silu) v = silu8(v);
+    }
+    *reinterpret_cast<uint4*>(dst + (u >> 3) * CH_CHUNK + chunk_addr(r, u & 7)) = v;
+  }
+}
+
+// What a chunk adds to the state: U [KP, 64 value channels] of one head. blockIdx: chunk, head, 64 value channels.
+template <int DK>
+struct ChunkStateCfg {
+  static constexpr int kKBytes = CH * DK * 2;
+  static constexpr int kSmem = 1024 + 2 * kKBytes + CH_CHUNK;
+  static constexpr int kCols = DK > 128 ? 128 : 64;
+};
+
+template <int DK>
+__global__ void __launch_bounds__(CHT) recurrent_chunk_state_kernel(const ChunkParams p) {
+  using Cfg = ChunkStateCfg<DK>;
+  extern __shared__ __align__(128) uint8_t smem_raw[];
+  __shared__ float gs[CH], bs[CH], nred[4][DK];
+  __shared__ __align__(8) uint64_t done;
+  __shared__ uint32_t tmem_base_smem;
+  __shared__ int abort_flag;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* hi = smem_raw + (base - smem_u32(smem_raw));
+  uint8_t* lo = hi + Cfg::kKBytes;
+  uint8_t* vt = lo + Cfg::kKBytes;
+  if (threadIdx.x == 0) {
+    abort_flag = 0;
+    mbar_init(smem_u32(&done), 1);
+    fence_mbar_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_smem), Cfg::kCols);
+    tmem_relinquish();
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  const int4 ck = p.chunks[c];
+  const int row0 = ck.x, n = ck.y;
+  if (warp == 0) {
+    const float2 t = chunk_gates(p, h, row0, n, gs, bs);
+    const float G = p.gated ? t.y : -t.x;
+    gs[lane * 4] -= G; gs[lane * 4 + 1] -= G; gs[lane * 4 + 2] -= G; gs[lane * 4 + 3] -= G;
+    if (lane == 0 && z == 0) p.um[(long long)c * p.H + h] = make_float2(t.x, t.x + G);
+  }
+  chunk_load<64>(vt, p.proj + row0 * p.ld + p.v_col + h * p.VP + z * 64, p.ld, n, p.silu);
+  __syncthreads();
+  const __nv_bfloat16* k = p.proj + row0 * p.ld + p.k_col + h * p.KP;
+#pragma unroll 2
+  for (int i = threadIdx.x; i < CH * (DK / 8); i += CHT) {
+    const int r = i / (DK / 8), u = i % (DK / 8);
+    uint4 a = make_uint4(0u, 0u, 0u, 0u), b = a;
+    if (r < n) {
+      const uint4 v = *reinterpret_cast<const uint4*>(k + r * p.ld + u * 8);
+      const float w = chunk_exp2(gs[r]);
+      auto one = [&](uint32_t x, uint32_t& l) {
+        float2 f = unpack_bf16x2(x);
+        if (p.silu) { f.x = silu_f(f.x); f.y = silu_f(f.y); }
+        f.x *= w; f.y *= w;
+        const uint32_t o = pack_bf16x2(f.x, f.y);
+        const float2 back = unpack_bf16x2(o);
+        l = pack_bf16x2(f.x - back.x, f.y - back.y);
+        return o;
+      };
+      a.x = one(v.x, b.x); a.y = one(v.y, b.y); a.z = one(v.z, b.z); a.w = one(v.w, b.w);
+    }
+    const uint32_t at = (u >> 3) * CH_CHUNK + chunk_addr(r, u & 7);
+    *reinterpret_cast<uint4*>(hi + at) = a;
+    *reinterpret_cast<uint4*>(lo + at) = b;
+  }
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_base_smem;
+  if (warp == 0 && elect_one_sync()) {
+    const uint32_t v_s = base + 2 * Cfg::kKBytes;
+#pragma unroll
+    for (int m0 = 0; m0 < DK; m0 += 128) {
+      constexpr int kFull = 128;
+      const uint32_t idesc = make_idesc_bf16(DK - m0 >= kFull ? 128 : 64, 64, 1, 1);
+#pragma unroll
+      for (int part = 0; part < 2; ++part)
+#pragma unroll
+        for (int kk = 0; kk < CH / 16; ++kk) {
+          const uint64_t a = make_smem_desc_sw128(base + part * Cfg::kKBytes + (m0 / 64) * CH_CHUNK + kk * 2048, CH_CHUNK, 1024);
+          const uint64_t b = make_smem_desc_sw128(v_s + kk * 2048, CH_CHUNK, 1024);
+          umma_bf16(tmem + (m0 / 128) * 64, a, b, idesc, (part | kk) ? 1u : 0u);
+        }
+    }
+    umma_commit(smem_u32(&done));
+  }
+  if (p.gated && z == 0) {       // the normaliser's part, while the tensor cores work: column sums of the weighted keys
+    constexpr int PAIRS = DK / 2, GROUPS = 4;
+    for (int i = threadIdx.x; i < PAIRS * GROUPS; i += CHT) {
+      const int pr = i % PAIRS, g = i / PAIRS;
+      float sx = 0.f, sy = 0.f;
+      for (int r = g * (CH / GROUPS); r < (g + 1) * (CH / GROUPS); ++r) {
+        const uint32_t at = (pr >> 5) * CH_CHUNK + chunk_addr(r, (pr & 31) >> 2) + (pr & 3) * 4;
+        const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(hi + at)), y = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(lo + at));
+        sx += x.x + y.x;
+        sy += x.y + y.y;
+      }
+      nred[g][2 * pr] = sx;
+      nred[g][2 * pr + 1] = sy;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < DK; i += CHT)
+      p.un[((long long)c * p.H + h) * p.KP + i] = (nred[0][i] + nred[1][i]) + (nred[2][i] + nred[3][i]);
+  }
+  bool ok = mbar_wait_bounded(smem_u32(&done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
+  ok = __all_sync(0xffffffffu, ok);
+  tc_fence_after();
+  if (ok) {
+    const int qd = warp & 3, half = warp >> 2;       // lanes of a TMEM quarter; the two warps of a quarter split the columns
+    float* u = p.u + (((long long)c * p.H + h) * (p.VP / 32) + z * 2 + half) * p.KP * 32;
+#pragma unroll
+    for (int m0 = 0; m0 < DK; m0 += 128) {
+      uint32_t v[32];
+      tmem_ld_32x32(tmem + (m0 / 128) * 64 + half * 32 + ((uint32_t)(qd * 32) << 16), v);
+      tmem_ld_wait();
+      // a 128-row product has row 32 q + lane in quarter q, a 64-row one row 16 q + lane in its first 16 lanes
+      const bool full = DK - m0 >= 128;
+      const int r = m0 + (full ? qd * 32 + lane : qd * 16 + lane);
+      if (full || lane < 16) {
+        float4* dst = reinterpret_cast<float4*>(u + (long long)r * 32);
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          dst[i] = make_float4(__uint_as_float(v[4 * i]), __uint_as_float(v[4 * i + 1]), __uint_as_float(v[4 * i + 2]), __uint_as_float(v[4 * i + 3]));
+      }
+    }
+    tc_fence_before();
+  }
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, Cfg::kCols);
+  }
+}
+
+// The state in front of every chunk, as two bf16 parts, and the state behind the portion. Every thread carries four value
+// channels of one key row over the chunks. blockIdx: 32 key rows, tile of 32 value channels + head, sequence.
+constexpr int CHAIN_AHEAD = 8;
+
+__global__ void __launch_bounds__(256) recurrent_chunk_chain_kernel(const ChunkParams p) {
+  pdl_launch_dependents();
+  const int tiles = p.VP / SC_COLS;
+  const int tile = blockIdx.y % tiles, h = blockIdx.y / tiles, b = blockIdx.z;
+  const int c4 = threadIdx.x & 7, r = blockIdx.x * 32 + (threadIdx.x >> 3);
+  pdl_wait();
+  const int slot = p.slots[b];
+  if (slot < 0 || slot >= p.num_slots) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); return; }
+  const bool fresh = p.seq_lens[b] == p.cu_q[b + 1] - p.cu_q[b];
+  const int c0 = p.seq_chunks[b], c1 = p.seq_chunks[b + 1];
+  const long long unit = ((long long)slot * p.H + h) * tiles + tile;
+  float4* st = reinterpret_cast<float4*>(p.s + (unit * p.KP + r) * SC_COLS) + c4;
+  float* nt = p.n + unit * p.KP + r;
+  const bool live = r < p.dk;
+  float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+  float n = 0.f, m = 0.f;
+  if (!fresh) {
+    if (live) S = *st;
+    if (p.gated) {
+      if (live) n = *nt;
+      m = p.m[unit] * LOG2E;
+    }
+  }
+  const bool owns_n = p.gated && tile == 0 && c4 == 0;
+  for (int cb = c0; cb < c1; cb += CHAIN_AHEAD) {
+    float4 U[CHAIN_AHEAD];
+    float un[CHAIN_AHEAD];
+    float2 um[CHAIN_AHEAD];
+#pragma unroll
+    for (int i = 0; i < CHAIN_AHEAD; ++i) {
+      const int c = cb + i;
+      if (c < c1) {
+        U[i] = *(reinterpret_cast<const float4*>(p.u + ((((long long)c * p.H + h) * tiles + tile) * p.KP + r) * SC_COLS) + c4);
+        un[i] = p.gated ? p.un[((long long)c * p.H + h) * p.KP + r] : 0.f;
+        um[i] = p.um[(long long)c * p.H + h];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < CHAIN_AHEAD; ++i) {
+      const int c = cb + i;
+      if (c < c1) {
+        const long long ch = (long long)c * p.H + h;
+        const uint32_t h0 = pack_bf16x2(S.x, S.y), h1 = pack_bf16x2(S.z, S.w);
+        const float2 b0 = unpack_bf16x2(h0), b1 = unpack_bf16x2(h1);
+        const long long at = ((ch * (p.VP / 64) + (tile >> 1)) * p.KP + r) * 64 + (tile & 1) * 32 + c4 * 4;
+        *reinterpret_cast<uint2*>(p.s_hi + at) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2*>(p.s_lo + at) = make_uint2(pack_bf16x2(S.x - b0.x, S.y - b0.y), pack_bf16x2(S.z - b1.x, S.w - b1.y));
+        if (owns_n) {
+          p.s_n[ch * p.KP + r] = n;
+          if (r == 0) p.s_m[ch] = m;
+        }
+        float a, w = 1.f;
+        if (p.gated) {
+          const float m_new = fmaxf(um[i].x + m, um[i].y);
+          a = exp2f(um[i].x + m - m_new);
+          w = exp2f(um[i].y - m_new);
+          m = m_new;
+        } else {
+          a = exp2f(um[i].x);
+        }
+        S.x = fmaf(a, S.x, w * U[i].x);
+        S.y = fmaf(a, S.y, w * U[i].y);
+        S.z = fmaf(a, S.z, w * U[i].z);
+        S.w = fmaf(a, S.w, w * U[i].w);
+        n = fmaf(a, n, w * un[i]);
+      }
+    }
+  }
+  if (live) {
+    *st = S;
+    if (p.gated && c4 == 0) *nt = n;
+  }
+  if (p.gated && r == 0 && c4 == 0) p.m[unit] = m / LOG2E;
+}
+
+// Outputs of a chunk: 64 value channels of one head. blockIdx: chunk, head, 64 value channels.
+template <int DK>
+struct ChunkOutCfg {
+  static constexpr int kQBytes = CH * DK * 2;
+  static constexpr int kKpBytes = CH * (DK > 128 ? DK : 128) * 2;             // K, then the weights P [CH, CH]
+  static constexpr int kSBytes = DK * CH_ROWB;                                // one part of the state
+  static constexpr int kSvBytes = kSBytes > CH_CHUNK ? kSBytes : CH_CHUNK;    // state (first part), then V
+  static constexpr int kSmem = 1024 + kQBytes + kKpBytes + kSvBytes + kSBytes;
+  static constexpr int kCols = 256;                                           // scores 128 | P V 64 | Q S 64
+};
+
+template <int DK>
+__global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkParams p) {
+  using Cfg = ChunkOutCfg<DK>;
+  extern __shared__ __align__(128) uint8_t smem_raw[];
+  __shared__ float gs[CH], bs[CH], fs[CH], row_sum[2][CH];
+  __shared__ __align__(16) float ns[DK];
+  __shared__ float m_in;
+  __shared__ __align__(8) uint64_t s_done, o_done;
+  __shared__ uint32_t tmem_base_smem;
+  __shared__ int abort_flag;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* q_p = smem_raw + (base - smem_u32(smem_raw));
+  uint8_t* k_p = q_p + Cfg::kQBytes;
+  uint8_t* sv_p = k_p + Cfg::kKpBytes;
+  uint8_t* sl_p = sv_p + Cfg::kSvBytes;
+  const uint32_t q_s = base, k_s = q_s + Cfg::kQBytes, sv_s = k_s + Cfg::kKpBytes, sl_s = sv_s + Cfg::kSvBytes;
+  if (threadIdx.x == 0) {
+    abort_flag = 0;
+    mbar_init(smem_u32(&s_done), 1);
+    mbar_init(smem_u32(&o_done), 1);
+    fence_mbar_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_smem), Cfg::kCols);
+    tmem_relinquish();
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  const int4 ck = p.chunks[c];
+  const int row0 = ck.x, n = ck.y;
+  const long long ch = (long long)c * p.H + h;
+  const __nv_bfloat16* rows = p.proj + row0 * p.ld;
+  if (warp == 0) {
+    chunk_gates(p, h, row0, n, gs, bs, fs);
+    if (lane == 0) m_in = p.gated ? p.s_m[ch] : 0.f;
+  }
+  if (p.gated)
+    for (int i = threadIdx.x; i < DK; i += CHT) ns[i] = p.s_n[ch * p.KP + i];
+  {
+    const long long at = (ch * (p.VP / 64) + z) * p.KP * 64;
+    const uint4* gh = reinterpret_cast<const uint4*>(p.s_hi + at);
+    const uint4* gl = reinterpret_cast<const uint4*>(p.s_lo + at);
+#pragma unroll 2
+    for (int i = threadIdx.x; i < DK * 8; i += CHT) {
+      const uint32_t a = chunk_addr(i >> 3, i & 7);
+      *reinterpret_cast<uint4*>(sv_p + a) = gh[i];
+      *reinterpret_cast<uint4*>(sl_p + a) = gl[i];
+    }
+  }
+  chunk_load<DK>(q_p, rows + p.q_col + h * p.KP, p.ld, n, p.silu);
+  chunk_load<DK>(k_p, rows + p.k_col + h * p.KP, p.ld, n, p.silu);
+  uint4 vr[CH * 8 / CHT];                            // V waits in registers until the state's shared memory is free
+#pragma unroll
+  for (int i = 0; i < CH * 8 / CHT; ++i) {
+    const int e = threadIdx.x + i * CHT, r = e >> 3, u = e & 7;
+    vr[i] = make_uint4(0u, 0u, 0u, 0u);
+    if (r < n) vr[i] = *reinterpret_cast<const uint4*>(rows + r * p.ld + p.v_col + h * p.VP + z * 64 + u * 8);
+  }
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_base_smem, t_o = tmem + 128, t_s = tmem + 192;
+  if (warp == 0 && elect_one_sync()) {
+    constexpr uint32_t idesc_s = make_idesc_bf16(CH, CH, 0, 0), idesc_o = make_idesc_bf16(CH, 64, 0, 1);
+#pragma unroll
+    for (int kk = 0; kk < DK / 16; ++kk) {
+      const uint64_t a = make_smem_desc_sw128(q_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+      const uint64_t b = make_smem_desc_sw128(k_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+      umma_bf16(tmem, a, b, idesc_s, kk ? 1u : 0u);
+    }
+#pragma unroll
+    for (int part = 0; part < 2; ++part)
+#pragma unroll
+      for (int kk = 0; kk < DK / 16; ++kk) {
+        const uint64_t a = make_smem_desc_sw128(q_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+        const uint64_t b = make_smem_desc_sw128((part ? sl_s : sv_s) + kk * 2048, CH_CHUNK, 1024);
+        umma_bf16(t_s, a, b, idesc_o, (part | kk) ? 1u : 0u);
+      }
+    umma_commit(smem_u32(&s_done));
+  }
+  const int qd = warp & 3, half = warp >> 2;
+  const int t = qd * 32 + lane;                      // this thread's token; the two warps of a quarter split the columns
+  const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
+  const float B = p.gated ? fmaxf(m_in, bs[t]) : bs[t];
+  float qn = 0.f;
+  if (p.gated) {                                     // half of q . n of the incoming state
+    constexpr int U = DK / 16;                       // 16-byte units per half
+#pragma unroll 4
+    for (int u = half * U; u < (half + 1) * U; ++u) {
+      const uint4 v = *reinterpret_cast<const uint4*>(q_p + (u >> 3) * CH_CHUNK + chunk_addr(t, u & 7));
+      const float* w = ns + u * 8;
+      float2 f;
+      f = unpack_bf16x2(v.x); qn = fmaf(f.x, w[0], fmaf(f.y, w[1], qn));
+      f = unpack_bf16x2(v.y); qn = fmaf(f.x, w[2], fmaf(f.y, w[3], qn));
+      f = unpack_bf16x2(v.z); qn = fmaf(f.x, w[4], fmaf(f.y, w[5], qn));
+      f = unpack_bf16x2(v.w); qn = fmaf(f.x, w[6], fmaf(f.y, w[7], qn));
+    }
+  }
+  const float c_in = chunk_exp2(m_in - B);
+  bool ok = mbar_wait_bounded(smem_u32(&s_done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
+  ok = __all_sync(0xffffffffu, ok);
+  tc_fence_after();
+  float sum = 0.f;
+  if (ok) {
+    uint8_t* prow = k_p + half * CH_CHUNK;           // K has been read
+#pragma unroll
+    for (int cc = 0; cc < 2; ++cc) {
+      uint32_t v[32];
+      tmem_ld_32x32(tmem + half * 64 + cc * 32 + lane_addr, v);
+      tmem_ld_wait();
+      float x[32];
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        const int j = half * 64 + cc * 32 + i;
+        x[i] = j <= t ? __uint_as_float(v[i]) * chunk_exp2(gs[j] - B) : 0.f;
+        sum += x[i];
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        *reinterpret_cast<uint4*>(prow + chunk_addr(t, cc * 4 + u)) =
+            make_uint4(pack_bf16x2(x[u * 8], x[u * 8 + 1]), pack_bf16x2(x[u * 8 + 2], x[u * 8 + 3]), pack_bf16x2(x[u * 8 + 4], x[u * 8 + 5]),
+                       pack_bf16x2(x[u * 8 + 6], x[u * 8 + 7]));
+    }
+    // V over the state's first part, which has been read too
+#pragma unroll
+    for (int i = 0; i < CH * 8 / CHT; ++i) {
+      const int e = threadIdx.x + i * CHT;
+      *reinterpret_cast<uint4*>(sv_p + chunk_addr(e >> 3, e & 7)) = p.silu ? silu8(vr[i]) : vr[i];
+    }
+  }
+  row_sum[half][t] = sum + c_in * qn;
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  if (ok && warp == 0 && elect_one_sync()) {
+    constexpr uint32_t idesc_o = make_idesc_bf16(CH, 64, 0, 1);
+#pragma unroll
+    for (int kk = 0; kk < CH / 16; ++kk) {
+      const uint64_t a = make_smem_desc_sw128(k_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+      const uint64_t b = make_smem_desc_sw128(sv_s + kk * 2048, CH_CHUNK, 1024);
+      umma_bf16(t_o, a, b, idesc_o, kk ? 1u : 0u);
+    }
+    umma_commit(smem_u32(&o_done));
+  }
+  if (ok) {
+    ok = mbar_wait_bounded(smem_u32(&o_done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
+    ok = __all_sync(0xffffffffu, ok);
+  }
+  tc_fence_after();
+  if (ok) {
+    float f = p.q_scale;
+    if (p.gated) {
+      const float nq = fabsf((row_sum[0][t] + row_sum[1][t]) * p.q_scale);
+      f /= fmaxf(nq, chunk_exp2(-(fs[t] + B))) + 1e-6f;
+    }
+    uint32_t a[32], b[32];
+    tmem_ld_32x32(t_o + half * 32 + lane_addr, a);
+    tmem_ld_32x32(t_s + half * 32 + lane_addr, b);
+    tmem_ld_wait();
+    tc_fence_before();
+    if (t < n) {
+      float4* dst = reinterpret_cast<float4*>(p.out + (long long)(row0 + t) * p.ldo + h * p.VP + z * 64 + half * 32);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        float y[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[e] = f * fmaf(c_in, __uint_as_float(b[4 * i + e]), __uint_as_float(a[4 * i + e]));
+        dst[i] = make_float4(y[0], y[1], y[2], y[3]);
+      }
+    }
+  }
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, Cfg::kCols);
+  }
+}
+
+template <int DK>
+static int launch_chunks(const ChunkParams& p, int n_chunks, int n_seq, cudaStream_t stream) {
+  static bool attr_dev[64] = {};
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
+  if (!attr_dev[dev]) {
+    if (cudaFuncSetAttribute(recurrent_chunk_state_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkStateCfg<DK>::kSmem) != cudaSuccess ||
+        cudaFuncSetAttribute(recurrent_chunk_out_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkOutCfg<DK>::kSmem) != cudaSuccess)
+      return -10;
+    attr_dev[dev] = true;
+  }
+  const dim3 grid(n_chunks, p.H, p.VP / 64);
+  if (launch_kernel(recurrent_chunk_state_kernel<DK>, grid, dim3(CHT), ChunkStateCfg<DK>::kSmem, stream, p) != cudaSuccess) return -11;
+  if (launch_kernel(recurrent_chunk_chain_kernel, dim3(DK / 32, p.H * (p.VP / SC_COLS), n_seq), dim3(256), 0, stream, p) != cudaSuccess) return -12;
+  return launch_kernel(recurrent_chunk_out_kernel<DK>, grid, dim3(CHT), ChunkOutCfg<DK>::kSmem, stream, p) == cudaSuccess ? 0 : -13;
+}
+
+// ------------------------------------------------------------------------------------------
 // out = o / rms * weight * sigmoid(gate). One CTA per token; a warp takes whole heads. Padding channels of o are zero.
 template <typename T>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ weight,
@@ -247,6 +813,46 @@ int rb_recurrent_scan(const void* proj, long long ld, int q_col, int k_col, int 
   const ScanParams p{proj, ld, q_col, k_col, v_col, small, ld_small, decay, bias_i, bias_f, cap, q_scale, s, n, m, slots, cu_q, seq_lens,
                      out, ldo, H, dk, KP, VP, num_slots, silu, gated, rows, status};
   return dtype == 0 ? launch_scan<__nv_bfloat16>(p, B, stream) : launch_scan<float>(p, B, stream);
+}
+
+// Workspace of the chunked form in bytes.
+long long rb_recurrent_chunk_workspace(int n_chunks, int H, int KP, int VP) {
+  const long long ch = (long long)n_chunks * H;
+  return ch * ((long long)KP * VP * 8 + KP * 8 + 16) + 256;
+}
+
+// Sequences of any length, `chunks` [n_chunks] and `seq_chunks` [n_seq + 1] as ChunkParams describes; slots, seq_lens and cu_q belong to
+// the same n_seq sequences. Activations in bf16.
+int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, int v_col, const float* small, long long ld_small, const float* decay,
+                        const float* bias_i, const float* bias_f, float cap, float q_scale, float* s, float* n, float* m, const void* chunks,
+                        const int* seq_chunks, const int* slots, const int* cu_q, const int* seq_lens, float* out, long long ldo, void* workspace,
+                        int n_chunks, int n_seq, int H, int dk, int KP, int VP, int num_slots, int silu, int gated, int* status, cudaStream_t stream) {
+  if (n_chunks <= 0 || n_seq <= 0) return 0;
+  if (H <= 0 || H > 65535 || n_seq > 65535 || dk <= 0 || dk > KP || KP % 64 != 0 || VP % 64 != 0 || ld % 8 != 0 || ldo % 4 != 0 ||
+      (gated ? small == nullptr : decay == nullptr) || workspace == nullptr)
+    return -1;
+  const long long ch = (long long)n_chunks * H;
+  ChunkParams p{};
+  p.proj = (const __nv_bfloat16*)proj; p.ld = ld; p.q_col = q_col; p.k_col = k_col; p.v_col = v_col;
+  p.small = small; p.ld_small = ld_small; p.decay = decay; p.bias_i = bias_i; p.bias_f = bias_f; p.cap = cap; p.q_scale = q_scale;
+  p.chunks = (const int4*)chunks; p.seq_chunks = seq_chunks; p.slots = slots; p.seq_lens = seq_lens; p.cu_q = cu_q;
+  p.s = s; p.n = n; p.m = m; p.out = out; p.ldo = ldo;
+  p.H = H; p.dk = dk; p.KP = KP; p.VP = VP; p.num_slots = num_slots; p.silu = silu; p.gated = gated; p.status = status;
+  float* w = (float*)workspace;
+  p.u = w; w += ch * KP * VP;
+  p.s_hi = (__nv_bfloat16*)w; w += ch * KP * VP / 2;
+  p.s_lo = (__nv_bfloat16*)w; w += ch * KP * VP / 2;
+  p.un = w; w += ch * KP;
+  p.s_n = w; w += ch * KP;
+  p.um = (float2*)w; w += ch * 2;
+  p.s_m = w;
+  switch (KP) {
+    case 64: return launch_chunks<64>(p, n_chunks, n_seq, stream);
+    case 128: return launch_chunks<128>(p, n_chunks, n_seq, stream);
+    case 192: return launch_chunks<192>(p, n_chunks, n_seq, stream);
+    case 256: return launch_chunks<256>(p, n_chunks, n_seq, stream);
+    default: return -1;
+  }
 }
 
 int rb_gated_norm(const float* o, long long ldo, const float* weight, const void* gate, long long ldg, void* out, long long ldy, int H, int dv,

@@ -1,6 +1,7 @@
 """Recurrent mixers (``ops/recurrent.py``) as a part of a layer stack: one joint projection (queries, keys, values, output
 gate), the recurrence over the sequences' state slots, one norm-and-gate kernel, the output projection. Gate logits of the
-recurrence come from the layer's narrow fp32 projection."""
+recurrence come from the layer's narrow fp32 projection. Decoded tokens and portions of at most ``SCAN_PORTION`` tokens run
+token by token, longer ones in chunks on the tensor cores, in one batch."""
 
 from __future__ import annotations
 
@@ -8,8 +9,10 @@ import torch
 
 from ... import ops
 from ...models.stack import LightningSpec, MatrixMemorySpec
-from ...ops.recurrent import MAX_DIM, RecurrentGeometry, RecurrentState
+from ...ops.recurrent import MAX_DIM, ChunkTable, RecurrentGeometry, RecurrentState, chunk_workspace, chunked_supported
 from .base import Part, load_head_columns, load_head_vector, load_heads
+
+SCAN_PORTION = 16            # new tokens of a sequence up to which the recurrence runs token by token
 
 
 def recurrent_geometry(m: LightningSpec | MatrixMemorySpec) -> RecurrentGeometry:
@@ -85,6 +88,22 @@ class RecurrentPart(Part):
         ops.gated_norm(o, w.norm, proj[:, g.offsets[3]:], g, self.r.cfg.norm_eps, out, g.gated)
         ops.gemm(out, w.wo, out=y, out_f32=True)
 
+    def plan(self, b):
+        """(sequences and rows that run token by token, chunk table of the rest)"""
+        if b.cu_q is None or not self.r.bf16:
+            return b.rows, b.num_tokens, None
+        first = next((i for i in range(b.rows) if b.host_cu_q[i + 1] - b.host_cu_q[i] > SCAN_PORTION), b.rows)
+        return first, b.host_cu_q[first], ChunkTable.make(b.host_cu_q, first, self.r.device) if first < b.rows else None
+
     def recur(self, w: RecurrentWeights, state: RecurrentState, proj, small, o, b, plan) -> None:
         """``o`` from the projected rows, and the state of the batch's sequences moved on."""
-        ops.recurrent_scan(proj, small, w.geo, w.decay, w.bias_i, w.bias_f, w.cap, state, b.state_slots, b.cu_q, b.seq_lens, o, b.num_tokens, b.rows)
+        g = w.geo
+        n_seq, rows, table = plan
+        if table is not None and not chunked_supported(g):
+            n_seq, rows, table = b.rows, b.num_tokens, None
+        args = (proj, small, g, w.decay, w.bias_i, w.bias_f, w.cap, state, b.state_slots, b.cu_q, b.seq_lens, o)
+        if n_seq > 0:
+            ops.recurrent_scan(*args, rows, n_seq)
+        if table is not None:
+            room = torch.empty(chunk_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=o.device)
+            ops.recurrent_chunks(*args, table, room)

@@ -55,7 +55,7 @@ from .latent import (
     latent_workspace,
 )
 from .keyvalue import KeyValueGeometry, kv_append, kv_attention, kv_workspace
-from .recurrent import RecurrentGeometry, RecurrentState, gated_norm, recurrent_scan
+from .recurrent import ChunkTable, RecurrentGeometry, RecurrentState, gated_norm, recurrent_chunks, recurrent_scan
 from .sampling import sample_with_logprobs, sample_with_logprobs_reference, token_logprobs
 
 def set_pdl(on: bool) -> None:
@@ -80,5 +80,5 @@ __all__ = [
     "layernorm_reference", "layernorm_residual", "layernorm_rows", "softcap", "gemm_f32", "LatentGeometry",
     "head_gemm_absorb", "head_gemm_expand", "latent_append", "latent_attention", "latent_gather", "latent_plan", "latent_query", "latent_units", "latent_workspace",
     "ExpertsGeometry", "ExpertsScratch", "experts_forward", "pack_experts", "KeyValueGeometry", "kv_append", "kv_attention", "kv_workspace",
-    "RecurrentGeometry", "RecurrentState", "gated_norm", "recurrent_scan", "stream_embed", "stream_norm",
+    "ChunkTable", "RecurrentGeometry", "RecurrentState", "gated_norm", "recurrent_chunks", "recurrent_scan", "stream_embed", "stream_norm",
 ]

@@ -26,6 +26,7 @@ from ._util import check_rc, ptr, status_tensor, stream_handle
 c_int, c_ll, c_float, c_vp = ctypes.c_int, ctypes.c_longlong, ctypes.c_float, ctypes.c_void_p
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 MAX_DIM = 512
+CHUNK = 128                  # tokens the chunked form takes at a time
 STATE_COLS = 32              # value channels of one state tile; every tile carries its own n and m
 
 
@@ -88,8 +89,11 @@ def _lib() -> ctypes.CDLL:
     if not getattr(lib, "_rb_typed", False):
         lib.rb_recurrent_scan.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float, c_float] + [c_vp] * 6
                                           + [c_vp, c_ll] + [c_int] * 10 + [c_vp, c_vp])
+        lib.rb_recurrent_chunks.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float, c_float] + [c_vp] * 9 + [c_ll, c_vp]
+                                            + [c_int] * 9 + [c_vp, c_vp])
+        lib.rb_recurrent_chunk_workspace.argtypes, lib.rb_recurrent_chunk_workspace.restype = [c_int] * 4, c_ll
         lib.rb_gated_norm.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_ll] + [c_int] * 6 + [c_float, c_vp]
-        for f in ("rb_recurrent_scan", "rb_gated_norm"):
+        for f in ("rb_recurrent_scan", "rb_recurrent_chunks", "rb_gated_norm"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -158,6 +162,51 @@ def recurrent_scan(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, c
                                   int(geo.silu), int(geo.gated), rows, _DT[proj.dtype], ptr(status_tensor(proj.device)),
                                   stream_handle(proj.device))
     check_rc(rc, "rb_recurrent_scan")
+
+
+@dataclass
+class ChunkTable:
+    """Device tables of the chunked form: ``chunks [n, 4]`` (first packed row, tokens, sequence, starts a portion) and
+    ``seq_chunks [B + 1]`` for the packed sequences ``first ..`` of a batch."""
+
+    chunks: torch.Tensor
+    seq_chunks: torch.Tensor
+    first: int
+
+    @staticmethod
+    def make(host_cu_q: list[int], first: int, device) -> "ChunkTable":
+        rows, starts = [], [0]
+        for i in range(first, len(host_cu_q) - 1):
+            for t in range(host_cu_q[i], host_cu_q[i + 1], CHUNK):
+                rows.append((t, min(CHUNK, host_cu_q[i + 1] - t), i - first, int(t == host_cu_q[i])))
+            starts.append(len(rows))
+        flat = torch.tensor([x for r in rows for x in r] + starts, dtype=torch.int32).to(device)
+        return ChunkTable(flat[:4 * len(rows)].view(-1, 4), flat[4 * len(rows):], first)
+
+
+def chunked_supported(geo: RecurrentGeometry) -> bool:
+    """Padded key sizes the tensor-core kernels are built for."""
+    return geo.kp <= 256
+
+
+def recurrent_chunks(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, cap: float, state: RecurrentState, slots, cu_q, seq_lens, out,
+                     table: ChunkTable, workspace) -> None:
+    """The recurrence over the sequences of ``table`` in chunks of 128 tokens (bf16 activations on the GPU): rows
+    ``cu_q[first] ..`` of ``out``, state updated. ``workspace``: ``chunk_workspace`` bytes."""
+    _, ok, ov, _ = geo.offsets
+    n, B, f = table.chunks.shape[0], table.seq_chunks.shape[0] - 1, table.first
+    assert proj.is_cuda and proj.dtype == torch.bfloat16 and proj.stride(1) == out.stride(1) == 1 and out.dtype == torch.float32
+    assert workspace.numel() * workspace.element_size() >= chunk_workspace(n, geo)
+    rc = _lib().rb_recurrent_chunks(ptr(proj), proj.stride(0), 0, ok, ov, ptr(small), small.stride(0) if small is not None else 0, ptr(decay), ptr(bias_i),
+                                    ptr(bias_f), cap, geo.dim ** -0.5 if geo.gated else 1.0, ptr(state.s), ptr(state.n), ptr(state.m),
+                                    ptr(table.chunks), ptr(table.seq_chunks), ptr(slots[f:]), ptr(cu_q[f:]), ptr(seq_lens[f:]), ptr(out),
+                                    out.stride(0), ptr(workspace), n, B, geo.heads, geo.dim, geo.kp, geo.vp, state.s.shape[0], int(geo.silu),
+                                    int(geo.gated), ptr(status_tensor(proj.device)), stream_handle(proj.device))
+    check_rc(rc, "rb_recurrent_chunks", 3)
+
+
+def chunk_workspace(n_chunks: int, geo: RecurrentGeometry) -> int:
+    return int(_lib().rb_recurrent_chunk_workspace(n_chunks, geo.heads, geo.kp, geo.vp))
 
 
 def gated_norm(o, weight, gate, geo: RecurrentGeometry, eps: float, out, per_head: bool) -> None:
