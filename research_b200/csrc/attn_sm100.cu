@@ -755,34 +755,48 @@ extern "C" int rb_paged_prefill(const void* q, const void* k_cache, const void* 
 namespace rb {
 
 __device__ __forceinline__ float kv_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float kv_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float kv_to_f(float v) { return v; }
 __device__ __forceinline__ float kv_to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void kv_store(float* p, float v) { *p = v; }
 __device__ __forceinline__ void kv_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
-// Queries times 1 + coef ln(floor((p + 1) / every) + 1) in place, keys into the cache. One CTA per token.
+// Queries times 1 + coef ln(floor((p + 1) / every) + 1) in place, keys into the cache. One CTA per token, 16 bytes at a time.
 template <typename T>
 __global__ void kv_append_kernel(T* __restrict__ proj, long long ld, const int* __restrict__ positions, const int* __restrict__ slots, float coef,
                                  int every, T* __restrict__ cache, int num_blocks, int H, int G, int D, int* status) {
+  constexpr int V = 16 / sizeof(T);
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x;
   T* row = proj + t * ld;
+  const int slot = slots[t];
   const float f = 1.f + coef * logf((float)((positions[t] + 1) / every) + 1.f);
   if (f != 1.f)
-    for (int i = threadIdx.x; i < H * D; i += blockDim.x) kv_store(row + i, kv_to_f(row[i]) * f);
-  const int slot = slots[t];
+    for (int i = threadIdx.x * V; i < H * D; i += blockDim.x * V) {
+      union { uint4 u; T e[V]; } x;
+      x.u = *reinterpret_cast<const uint4*>(row + i);
+#pragma unroll
+      for (int j = 0; j < V; ++j) kv_store(&x.e[j], kv_to_f(x.e[j]) * f);
+      *reinterpret_cast<uint4*>(row + i) = x.u;
+    }
   if (slot < 0) return;
   const int blk = slot / KV_BLOCK;
   if (blk >= num_blocks) { if (threadIdx.x == 0) set_status(status, ST_BAD_INDEX); return; }
-  for (int i = threadIdx.x; i < G * D; i += blockDim.x)
-    cache[(((long long)blk * G + i / D) * KV_BLOCK + slot % KV_BLOCK) * D + i % D] = row[H * D + i];
+  for (int i = threadIdx.x * V; i < G * D; i += blockDim.x * V)
+    *reinterpret_cast<uint4*>(cache + (((long long)blk * G + i / D) * KV_BLOCK + slot % KV_BLOCK) * D + i % D) =
+        *reinterpret_cast<const uint4*>(row + H * D + i);
 }
 
-// Decode: the structure of paged_decode_tma_kernel with one tile that serves as K and V, up to 16 query heads per CTA
-// (blockIdx.y = kv head x chunk of 16 query heads).
+// Decode: the structure of paged_decode_tma_kernel with one tile that serves as K and V, two blocks (32 keys) per stage, up to
+// 16 query heads per CTA (blockIdx.y = kv head x chunk of 16 query heads). The sums of weights stay per thread until the
+// end, and the accumulators are rescaled only when a row's maximum moves.
 template <int D>
-__host__ __device__ constexpr int kv_dec_stages() { return D == 64 ? 6 : 6; }
+__host__ __device__ constexpr int kv_dec_stages() { return D == 64 ? 4 : 3; }      // 64 / 96 KB of ring per CTA
 constexpr int KV_MERGE_LD_PAD = 4;
 
 template <int D>
@@ -792,7 +806,7 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
                  __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int H, int Hkv, int bt_stride,
                  int num_blocks, int num_splits, float scale, int* status) {
   constexpr int CH = D / 8;
-  constexpr int TILE_BYTES = KV_BLOCK * D * 2;
+  constexpr int BLK_BYTES = KV_BLOCK * D * 2, TILE_BYTES = 2 * BLK_BYTES;
   constexpr int ST = kv_dec_stages<D>();
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ __align__(8) uint64_t bars[DEC_WARPS][ST];
@@ -816,7 +830,7 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
   }
   pdl_wait();
   const int L = seq_lens[b];
-  const int n_chunks = (L + KV_BLOCK - 1) / KV_BLOCK;
+  const int n_blocks = (L + KV_BLOCK - 1) / KV_BLOCK, n_chunks = (n_blocks + 1) / 2;
   const int per = (n_chunks + num_splits - 1) / num_splits;
   const int c_begin = split * per;
   const int c_end = min(n_chunks, c_begin + per);
@@ -844,32 +858,35 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
   const int n_my = first < c_end ? (c_end - first + DEC_WARPS - 1) / DEC_WARPS : 0;
   const int* bt_row = block_tables + (long long)b * bt_stride;
   auto load_ids = [&](int round) {
-    const int j = round * 32 + lane;
-    return j < n_my ? __ldg(bt_row + first + j * DEC_WARPS) : 0;
+    const int j = round * 32 + lane, blk = 2 * (first + (j >> 1) * DEC_WARPS) + (j & 1);
+    return (j >> 1) < n_my && blk < n_blocks ? __ldg(bt_row + blk) : num_blocks;     // past the end: out of bounds, zeros
   };
   int ids_round = 0, ids = load_ids(0), ids_next = load_ids(1);
-  auto blk_of = [&](int i) {   // all lanes, i uniform and non-decreasing
-    if ((i >> 5) > ids_round) { ids = ids_next; ids_round = i >> 5; ids_next = load_ids(ids_round + 1); }
-    return __shfl_sync(0xffffffffu, ids, i & 31);
+  auto blocks_of = [&](int i) {   // all lanes, i uniform and non-decreasing
+    if ((i >> 4) > ids_round) { ids = ids_next; ids_round = i >> 4; ids_next = load_ids(ids_round + 1); }
+    return make_int2(__shfl_sync(0xffffffffu, ids, (2 * i) & 31), __shfl_sync(0xffffffffu, ids, (2 * i + 1) & 31));
   };
-  auto issue = [&](int i, int blk) {   // lane 0 only
+  auto issue = [&](int i, int2 blk) {   // lane 0 only
     const int stage = i % ST;
-    if (blk < 0 || blk >= num_blocks) { set_status(status, ST_BAD_INDEX); blk = num_blocks; }  // OOB -> zeros
+    if (blk.x < 0 || blk.x > num_blocks || blk.y < 0 || blk.y > num_blocks) { set_status(status, ST_BAD_INDEX); blk.x = blk.y = num_blocks; }
     const uint32_t bar = smem_u32(&bars[warp][stage]), ks = k_smem + stage * TILE_BYTES;
     mbar_expect_tx(bar, TILE_BYTES);
 #pragma unroll
-    for (int hx = 0; hx < D / 64; ++hx) tma_load_2d(ks + hx * (KV_BLOCK * 128), &k_map, bar, hx * 64, (blk * Hkv + kvh) * KV_BLOCK);
+    for (int hx = 0; hx < D / 64; ++hx) {
+      tma_load_2d(ks + hx * (KV_BLOCK * 128), &k_map, bar, hx * 64, (blk.x * Hkv + kvh) * KV_BLOCK);
+      tma_load_2d(ks + BLK_BYTES + hx * (KV_BLOCK * 128), &k_map, bar, hx * 64, (blk.y * Hkv + kvh) * KV_BLOCK);
+    }
   };
   int issued = 0;
   for (; issued < ST - 1 && issued < n_my; ++issued) {
-    const int blk = blk_of(issued);
+    const int2 blk = blocks_of(issued);
     if (lane == 0) issue(issued, blk);
   }
   bool ok = true;
   const int mat = lane >> 3, rr = lane & 7;
   for (int i = 0; i < n_my; ++i) {
     if (issued < n_my) {
-      const int blk = blk_of(issued);
+      const int2 blk = blocks_of(issued);
       if (lane == 0) issue(issued, blk);
       ++issued;
     }
@@ -878,28 +895,61 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
     ok = __all_sync(0xffffffffu, ok);
     if (!ok) break;
     const uint32_t ks = k_smem + stage * TILE_BYTES;
-    float s0[4] = {0, 0, 0, 0}, s1[4] = {0, 0, 0, 0};
+    float sc[4][4] = {};
 #pragma unroll
-    for (int kk = 0; kk < D / 16; ++kk) {
-      uint32_t b0, b1, b2, b3;
-      ldsm_x4(ks + swz_tma<D>((mat >> 1) * 8 + rr, 2 * kk + (mat & 1)), b0, b1, b2, b3);
-      mma_16816(s0, qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b0, b1);
-      mma_16816(s1, qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b2, b3);
-    }
-    const int tok0 = (first + i * DEC_WARPS) * KV_BLOCK + 2 * (lane & 3);
-    if (tok0 >= L) { s0[0] = s0[2] = -INFINITY; }
-    if (tok0 + 1 >= L) { s0[1] = s0[3] = -INFINITY; }
-    if (tok0 + 8 >= L) { s1[0] = s1[2] = -INFINITY; }
-    if (tok0 + 9 >= L) { s1[1] = s1[3] = -INFINITY; }
-    uint32_t p0, p1, p2, p3;
-    softmax_update<D>(s0, s1, st, o, scale_log2, p0, p1, p2, p3);
+    for (int kk = 0; kk < D / 16; ++kk)
 #pragma unroll
-    for (int dp = 0; dp < D / 16; ++dp) {
-      uint32_t b0, b1, b2, b3;
-      ldsm_x4_t(ks + swz_tma<D>((mat & 1) * 8 + rr, 2 * dp + (mat >> 1)), b0, b1, b2, b3);
-      mma_16816(o[2 * dp], p0, p1, p2, p3, b0, b1);
-      mma_16816(o[2 * dp + 1], p0, p1, p2, p3, b2, b3);
+      for (int half = 0; half < 2; ++half) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4(ks + half * BLK_BYTES + swz_tma<D>((mat >> 1) * 8 + rr, 2 * kk + (mat & 1)), b0, b1, b2, b3);
+        mma_16816(sc[2 * half], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b0, b1);
+        mma_16816(sc[2 * half + 1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b2, b3);
+      }
+    const int tok0 = (first + i * DEC_WARPS) * 2 * KV_BLOCK + 2 * (lane & 3);
+    if (tok0 - 2 * (lane & 3) + 2 * KV_BLOCK > L) {
+#pragma unroll
+      for (int n8 = 0; n8 < 4; ++n8) {
+        if (tok0 + 8 * n8 >= L) sc[n8][0] = sc[n8][2] = -INFINITY;
+        if (tok0 + 8 * n8 + 1 >= L) sc[n8][1] = sc[n8][3] = -INFINITY;
+      }
     }
+    float mx0 = -INFINITY, mx1 = -INFINITY;
+#pragma unroll
+    for (int n8 = 0; n8 < 4; ++n8) {
+      mx0 = fmaxf(mx0, fmaxf(sc[n8][0], sc[n8][1]));
+      mx1 = fmaxf(mx1, fmaxf(sc[n8][2], sc[n8][3]));
+    }
+    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2)) * scale_log2;
+    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2)) * scale_log2;
+    if (__any_sync(0xffffffffu, mx0 > st.m0 || mx1 > st.m1)) {      // (the tile's first key is valid: the maximum is finite)
+      const float n0 = fmaxf(st.m0, mx0), n1 = fmaxf(st.m1, mx1);
+      const float c0 = exp2f(st.m0 - n0), c1 = exp2f(st.m1 - n1);
+      st.m0 = n0; st.m1 = n1;
+      st.l0 *= c0; st.l1 *= c1;
+#pragma unroll
+      for (int n8 = 0; n8 < D / 8; ++n8) { o[n8][0] *= c0; o[n8][1] *= c0; o[n8][2] *= c1; o[n8][3] *= c1; }
+    }
+    uint32_t pk[4][2];
+#pragma unroll
+    for (int n8 = 0; n8 < 4; ++n8) {
+      const float e0 = kv_exp2(fmaf(sc[n8][0], scale_log2, -st.m0)), e1 = kv_exp2(fmaf(sc[n8][1], scale_log2, -st.m0));
+      const float f0 = kv_exp2(fmaf(sc[n8][2], scale_log2, -st.m1)), f1 = kv_exp2(fmaf(sc[n8][3], scale_log2, -st.m1));
+      st.l0 += e0 + e1;
+      st.l1 += f0 + f1;
+      pk[n8][0] = pack_bf16x2(e0, e1);
+      pk[n8][1] = pack_bf16x2(f0, f1);
+    }
+#pragma unroll
+    for (int dp = 0; dp < D / 16; ++dp)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4_t(ks + half * BLK_BYTES + swz_tma<D>((mat & 1) * 8 + rr, 2 * dp + (mat >> 1)), b0, b1, b2, b3);
+        mma_16816(o[2 * dp], pk[2 * half][0], pk[2 * half][1], pk[2 * half + 1][0], pk[2 * half + 1][1], b0, b1);
+        mma_16816(o[2 * dp + 1], pk[2 * half][0], pk[2 * half][1], pk[2 * half + 1][0], pk[2 * half + 1][1], b2, b3);
+      }
     __syncwarp();   // every lane is done with this stage before lane 0 refills it
   }
   if (!ok && lane == 0) {
@@ -915,6 +965,10 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
   float* mo = reinterpret_cast<float*>(ring_ptr);                   // [DEC_WARPS][16][LD]
   float* mml = mo + DEC_WARPS * 16 * LD;                            // [DEC_WARPS][16][2]
   const int g = lane >> 2, tq = lane & 3;
+  st.l0 += __shfl_xor_sync(0xffffffffu, st.l0, 1);
+  st.l1 += __shfl_xor_sync(0xffffffffu, st.l1, 1);
+  st.l0 += __shfl_xor_sync(0xffffffffu, st.l0, 2);
+  st.l1 += __shfl_xor_sync(0xffffffffu, st.l1, 2);
 #pragma unroll
   for (int n = 0; n < D / 8; ++n) {
     *reinterpret_cast<float2*>(mo + (warp * 16 + g) * LD + n * 8 + 2 * tq) = make_float2(o[n][0], o[n][1]);
@@ -1068,7 +1122,7 @@ __global__ void kv_gate_kernel(__nv_bfloat16* __restrict__ out, const float* __r
 
 template <int D>
 constexpr int kv_decode_smem_bytes() {
-  const int ring = DEC_WARPS * kv_dec_stages<D>() * KV_BLOCK * D * 2 + 16 * D * 2;
+  const int ring = DEC_WARPS * kv_dec_stages<D>() * 2 * KV_BLOCK * D * 2 + 16 * D * 2;
   const int merge = DEC_WARPS * 16 * (D + KV_MERGE_LD_PAD + 2) * 4;
   return 1024 + (ring > merge ? ring : merge);
 }
@@ -1078,10 +1132,10 @@ constexpr int kv_decode_smem_bytes() {
 extern "C" int rb_kv_append(void* proj, long long ld, const int* positions, const int* slots, float coef, int every, void* cache, int num_blocks,
                             int H, int G, int D, int T, int dtype, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (every <= 0 || H <= 0 || G <= 0 || D <= 0) return -1;
+  if (every <= 0 || H <= 0 || G <= 0 || D <= 0 || D % 8 != 0 || ld % 8 != 0) return -1;
   cudaError_t e;
   if (dtype == 0)
-    e = launch_kernel(kv_append_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, (__nv_bfloat16*)proj, ld, positions, slots, coef, every,
+    e = launch_kernel(kv_append_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, stream, (__nv_bfloat16*)proj, ld, positions, slots, coef, every,
                       (__nv_bfloat16*)cache, num_blocks, H, G, D, status);
   else
     e = launch_kernel(kv_append_kernel<float>, dim3(T), dim3(256), 0, stream, (float*)proj, ld, positions, slots, coef, every, (float*)cache,

@@ -314,6 +314,8 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
 // ---- programmatic dependent launch -----------------------------------------------------------
 // A kernel launched with the programmatic-serialization attribute may start while its
 // predecessor on the stream is still running; it must execute pdl_wait() before it touches any

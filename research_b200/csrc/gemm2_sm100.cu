@@ -52,6 +52,9 @@ struct G2Params {
   long long ldr;
   const __nv_bfloat16* bias;
   int out_f32;
+  int silu_cols, tail_col;            // as in RbGemmArgs
+  float* tail;
+  long long tail_ld;
   int* status;
   // Fused all-gather of a row-sharded matrix (GATHER instantiations; same contract as the one-CTA kernel): part r is
   // gather_part_bytes at gather_src[r] (rank r's shard, peer memory); the gather warps of every CTA copy an
@@ -344,6 +347,17 @@ __global__ void __launch_bounds__(GATHER ? G2_THREADS_GATHER : G2_THREADS, 1) ge
               }
             }
           }
+          if (p.tail != nullptr && col >= p.tail_col) {
+            float* dst = p.tail + row * p.tail_ld + (col - p.tail_col);
+#pragma unroll
+            for (int j = 0; j < 32; j += 4)
+              if (j < ncols) *reinterpret_cast<float4*>(dst + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+            continue;
+          }
+          if (col < p.silu_cols) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = silu_fast(v[j]);
+          }
           if (p.out_f32) {
             float* dst = reinterpret_cast<float*>(p.C) + row * p.ldc + col;
 #pragma unroll
@@ -432,7 +446,8 @@ extern "C" int rb_gemm2_pairs() {
 // [K, rows] with rows contiguous (as in rb_gemm_bf16). bn: 256 or 128 output columns per tile (0 = choose).
 extern "C" int rb_gemm2_bf16(const void* A, const void* B, void* C, const void* bias, const void* residual, int M, int N,
                              int K, long long lda, long long ldb, long long ldc, long long ldr, int a_mn_major,
-                             int b_mn_major, int out_f32, int bn, int* status, cudaStream_t stream) {
+                             int b_mn_major, int out_f32, int bn, int silu_cols, float* tail, int tail_col, long long tail_ld,
+                             int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0 || N % 8 != 0) return -1;
   if ((!a_mn_major || !b_mn_major) && K % 8 != 0) return -1;
   if (a_mn_major && !b_mn_major) return -12;         // not used by forward, dgrad or wgrad
@@ -450,6 +465,8 @@ extern "C" int rb_gemm2_bf16(const void* A, const void* B, void* C, const void* 
   p.residual = reinterpret_cast<const __nv_bfloat16*>(residual); p.ldr = ldr;
   p.bias = reinterpret_cast<const __nv_bfloat16*>(bias);
   p.out_f32 = out_f32;
+  p.silu_cols = silu_cols; p.tail = tail; p.tail_col = tail_col; p.tail_ld = tail_ld;
+  if (silu_cols % 32 != 0 || (tail != nullptr && (tail_col % 32 != 0 || tail_ld % 4 != 0))) return -1;
   p.status = status;
   int rc = a_mn_major ? tma_map_2d_bf16(&p.a_map, A, K, M, lda, G2_BK) : tma_map_2d_bf16(&p.a_map, A, M, K, lda, G2_BM);
   if (rc != 0) return -20 + rc;

@@ -19,7 +19,8 @@ struct F32Group {
 
 __global__ void __launch_bounds__(F32_THREADS)
 gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ B, float* __restrict__ C, const float* __restrict__ bias, int M, int N, int K,
-                long long lda, long long ldb, long long ldc, long long sa, long long sb, long long sc, int b_kn, F32Group grp) {
+                long long lda, long long ldb, long long ldc, long long sa, long long sb, long long sc, int b_kn, int silu_cols,
+                F32Group grp) {
   __shared__ float as[F32_BK][F32_BM + 4];
   __shared__ float bs[F32_BK][F32_BM + 4];
   pdl_launch_dependents();
@@ -76,7 +77,8 @@ gemm_f32_kernel(const float* __restrict__ A, const float* __restrict__ B, float*
       const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
       if (m < M && n < N) {
         float* dst = grp.row_dst != nullptr ? reinterpret_cast<float*>(grp.row_dst[m]) : C + (long long)m * ldc;
-        dst[n + col0] = acc[i][j] + (bias != nullptr ? bias[n + col0] : 0.f);
+        const float v = acc[i][j] + (bias != nullptr ? bias[n + col0] : 0.f);
+        dst[n + col0] = n < silu_cols ? v / (1.f + expf(-v)) : v;
       }
     }
 }
@@ -88,11 +90,12 @@ using namespace rb;
 extern "C" void rb_gemm_f32_set_pdl(int on) { rb::pdl_enabled() = on != 0; }
 
 extern "C" int rb_gemm_f32(const float* A, const float* B, float* C, const float* bias, int M, int N, int K, long long lda, long long ldb,
-                           long long ldc, int batch, long long sa, long long sb, long long sc, int b_kn, cudaStream_t stream) {
+                           long long ldc, int batch, long long sa, long long sb, long long sc, int b_kn, int silu_cols,
+                           cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0 || batch <= 0 || batch > 65535) return -1;
   const dim3 grid((N + F32_BM - 1) / F32_BM, (M + F32_BM - 1) / F32_BM, batch);
   if (grid.y > 65535) return -1;
-  return launch_kernel(gemm_f32_kernel, grid, dim3(F32_THREADS), 0, stream, A, B, C, bias, M, N, K, lda, ldb, ldc, sa, sb, sc, b_kn,
+  return launch_kernel(gemm_f32_kernel, grid, dim3(F32_THREADS), 0, stream, A, B, C, bias, M, N, K, lda, ldb, ldc, sa, sb, sc, b_kn, silu_cols,
                        F32Group{nullptr, nullptr, 0, nullptr}) == cudaSuccess ? 0 : -11;
 }
 
@@ -100,6 +103,6 @@ extern "C" int rb_gemm_f32(const float* A, const float* B, float* C, const float
 extern "C" int rb_gemm_f32_grouped(const float* A, const float* B, float* C, int K, long long lda, long long ldb, long long ldc, const void* tiles,
                                    const int* num_tiles, int max_tiles, int group_n, const unsigned long long* row_dst, cudaStream_t stream) {
   if (K <= 0 || max_tiles <= 0 || group_n <= 0 || tiles == nullptr || num_tiles == nullptr) return -1;
-  return launch_kernel(gemm_f32_kernel, dim3(max_tiles, 2, 1), dim3(F32_THREADS), 0, stream, A, B, C, nullptr, 0, 0, K, lda, ldb, ldc, 0, 0, 0, 0,
+  return launch_kernel(gemm_f32_kernel, dim3(max_tiles, 2, 1), dim3(F32_THREADS), 0, stream, A, B, C, nullptr, 0, 0, K, lda, ldb, ldc, 0, 0, 0, 0, 0,
                        F32Group{(const int4*)tiles, num_tiles, group_n, row_dst}) == cudaSuccess ? 0 : -11;
 }

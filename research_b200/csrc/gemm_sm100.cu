@@ -108,6 +108,9 @@ struct GemmParams {
   int swiglu;
   int glu_kind;           // see RbGemmArgs
   float glu_limit, softcap;
+  int silu_cols, tail_col;   // see RbGemmArgs
+  float* tail;
+  long long tail_ld;
   int split_k, kb_per_split;
   int cluster_k;   // split-K slices are the CTAs of one thread-block cluster; partial tiles meet in distributed shared memory
   int red_alias;   // cluster split-K, one work unit per CTA: the partial tile reuses the (drained) TMA ring
@@ -150,6 +153,29 @@ struct GemmParams {
 __device__ __forceinline__ void epi_store_row_chunk(const GemmParams& p, const float* v,
                                                     long long row, int col, int ncols) {
   // v holds 32 fp32 values for (row, col..col+31); ncols valid (multiple of 8).
+  if (p.tail != nullptr && col >= p.tail_col) {
+    float* dst = p.tail + row * p.tail_ld + (col - p.tail_col);
+#pragma unroll
+    for (int j = 0; j < 32; j += 4) {
+      if (j < ncols) *reinterpret_cast<float4*>(dst + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+    }
+    return;
+  }
+  if (col < p.silu_cols) {
+    __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.C) + row * p.ldc + col;
+#pragma unroll
+    for (int j = 0; j < 32; j += 8) {
+      if (j < ncols) {
+        uint4 o;
+        o.x = pack_bf16x2(silu_fast(v[j]), silu_fast(v[j + 1]));
+        o.y = pack_bf16x2(silu_fast(v[j + 2]), silu_fast(v[j + 3]));
+        o.z = pack_bf16x2(silu_fast(v[j + 4]), silu_fast(v[j + 5]));
+        o.w = pack_bf16x2(silu_fast(v[j + 6]), silu_fast(v[j + 7]));
+        *reinterpret_cast<uint4*>(dst + j) = o;
+      }
+    }
+    return;
+  }
   if (p.out_f32) {
     float* dst = reinterpret_cast<float*>(p.C) + row * p.ldc + col;
 #pragma unroll
@@ -1329,6 +1355,11 @@ extern "C" int rb_gemm_bf16_ex(const RbGemmArgs* a, cudaStream_t stream) {
   p.glu_limit = a->glu_limit;
   p.softcap = a->softcap;
   if (p.softcap > 0.f && (a->swiglu || a->split_k > 1 || a->tile_table || a->epi_mode != RB_EPI_STORE || a->mirror || a->sample_ws))
+    return -1;
+  p.silu_cols = a->silu_cols;
+  p.tail = a->tail; p.tail_col = a->tail_col; p.tail_ld = a->tail_ld;
+  if ((p.silu_cols > 0 || p.tail != nullptr) && (a->swiglu || a->tile_table || a->epi_mode != RB_EPI_STORE || a->mirror || a->sample_ws || a->out_f32 ||
+                                                 a->silu_cols % 32 != 0 || a->tail_col % 32 != 0 || (p.tail != nullptr && a->tail_ld % 4 != 0)))
     return -1;
   p.scaled_epilogue = a->scaled_epilogue;
   p.alpha = a->alpha;

@@ -138,6 +138,12 @@ typedef struct RbGemmArgs {
   float glu_limit;
   // > 0: C = softcap * tanh(C / softcap) on the fp32 result (plain store only: no split, grouping or reduce mode).
   float softcap;
+  // Plain store only: columns below silu_cols (a multiple of 32) become silu(C); with tail set, columns from tail_col (a
+  // multiple of 32) on go to the fp32 matrix tail [M, tail_ld] instead of C (narrow projections that ride along).
+  int silu_cols;
+  int tail_col;
+  float* tail;
+  long long tail_ld;
 } RbGemmArgs;
 
 // Token and log-probability from the per-tile records written by the sampling epilogue.

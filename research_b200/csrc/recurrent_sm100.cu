@@ -2,12 +2,12 @@
 //
 //   S_t = a_t S_(t-1) + b_t k_t v_t^T,   o_t = S_t^T q_t        (see ops/recurrent.py)
 //
-//   scan        token by token: decoded tokens, short portions and the exact mode. One CTA per (sequence, head, 32 value
-//               channels); the state tile stays in registers over the tokens of the portion. A decoded token reads and writes
-//               the state once, which is what bounds it.
-//   chunked     long portions, 128 tokens at a time on the tensor cores (tcgen05), in three launches: what every chunk adds to the
-//               state (all chunks at once), the state in front of every chunk (one pass over the chunks), the outputs (all
-//               chunks at once)
+//   scan        token by token: short portions and long ones of the exact mode. One CTA per (sequence, head, 32 value channels);
+//               the state tile stays in registers over the tokens of the portion.
+//   decode      one token per sequence: persistent CTAs stream state tiles through a ring of bulk copies
+//   chunked     long portions, 128 tokens at a time on the tensor cores (tcgen05), in four launches: the gates, what every chunk
+//               adds to the state (all chunks at once), the state in front of every chunk (one pass over the chunks), the
+//               outputs (all chunks at once)
 //   gated_norm  RMS norm per head or over all heads, times sigmoid(gate), to the activation type
 //
 // State: s [slots, H, tiles, KP, 32], n [slots, H, tiles, KP], m [slots, H, tiles], all fp32. A tile of 32 value channels keeps its
@@ -29,7 +29,6 @@ template <>
 __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 // log(sigmoid(z)) without cancellation at either end
 __device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
@@ -51,7 +50,7 @@ struct ScanParams {
   const int* seq_lens;     // [B]
   float* out;              // [T, ldo]
   long long ldo;
-  int H, dk, KP, VP, num_slots, silu, gated, rows;
+  int H, dk, KP, VP, num_slots, gated, rows;
   int* status;
 };
 
@@ -99,14 +98,11 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
   for (int t = t0; t < t1; ++t) {
     const T* row = proj + t * p.ld;
     for (int i = tid; i < p.dk; i += SC_THREADS) {
-      float q = to_f<T>(row[p.q_col + h * p.KP + i]), k = to_f<T>(row[p.k_col + h * p.KP + i]);
-      if (p.silu) { q = silu_f(q); k = silu_f(k); }
-      qs[i] = q * p.q_scale;
-      ks[i] = k;
+      qs[i] = to_f<T>(row[p.q_col + h * p.KP + i]) * p.q_scale;
+      ks[i] = to_f<T>(row[p.k_col + h * p.KP + i]);
     }
     if (tid < SC_COLS) {
-      const float v = to_f<T>(row[p.v_col + h * p.VP + tile * SC_COLS + tid]);
-      vs[tid] = p.silu ? silu_f(v) : v;
+      vs[tid] = to_f<T>(row[p.v_col + h * p.VP + tile * SC_COLS + tid]);
     }
     float a = decay, w = 1.f;
     if (p.gated) {
@@ -185,6 +181,203 @@ static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
 }
 
 // ------------------------------------------------------------------------------------------
+// One token per sequence (row b of the batch is sequence b). The state is read and written once, which is all the time it
+// takes: persistent CTAs walk over the (sequence, head, tile) units with RD_STAGES tiles in flight, bulk copies in both
+// directions, the update in shared memory. The unit's vectors are fetched one unit ahead.
+// ------------------------------------------------------------------------------------------
+constexpr int RD_THREADS = 128, RD_STAGES = 3, RD_VEC = 3;
+constexpr int RD_MAX_DK = 384;                    // key rows: a ring of larger tiles does not fit
+
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar)
+               : "memory");
+}
+__device__ __forceinline__ void bulk_store(void* dst, uint32_t src, uint32_t bytes) {
+  asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst), "r"(src), "r"(bytes) : "memory");
+  asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+}
+
+template <typename T>
+__global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const ScanParams p, int units) {
+  extern __shared__ __align__(128) uint8_t smem_raw[];       // RD_STAGES x [dk, 32] fp32
+  __shared__ float qs[RD_MAX_DK], ks[RD_MAX_DK];
+  __shared__ __align__(16) float vs[SC_COLS];
+  __shared__ __align__(16) float red[RD_THREADS / 32][SC_COLS];
+  __shared__ float red_n[RD_THREADS / 32];
+  __shared__ __align__(8) uint64_t full[RD_STAGES];
+  __shared__ int abort_flag;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c4 = tid & 7, r0 = tid >> 3;
+  const int tiles = p.VP / SC_COLS;
+  const uint32_t ring = smem_u32(smem_raw), tile_bytes = (uint32_t)p.dk * SC_COLS * 4;
+  if (tid == 0) {
+    abort_flag = 0;
+    for (int i = 0; i < RD_STAGES; ++i) mbar_init(smem_u32(&full[i]), 1);
+    fence_mbar_init();
+  }
+  __syncthreads();
+  pdl_launch_dependents();
+  pdl_wait();
+  struct Unit { int b, h, tile, slot; };
+  auto unit_of = [&](int u) {
+    Unit x;
+    x.tile = u % tiles;
+    x.h = (u / tiles) % p.H;
+    x.b = u / tiles / p.H;
+    x.slot = p.slots[x.b];
+    if (x.slot >= p.num_slots) { set_status(p.status, ST_BAD_INDEX); x.slot = -1; }
+    return x;
+  };
+  auto state_index = [&](const Unit& x) { return ((long long)max(x.slot, 0) * p.H + x.h) * tiles + x.tile; };   // padding rows read slot 0
+  int issued = 0;                                            // thread 0
+  auto load = [&](int i) {                                   // thread 0: tile of this CTA's i-th unit
+    const int u = blockIdx.x + i * gridDim.x;
+    if (u >= units) return;
+    const Unit x = unit_of(u);
+    const uint32_t bar = smem_u32(&full[i % RD_STAGES]);
+    mbar_expect_tx(bar, tile_bytes);
+    bulk_load(ring + (i % RD_STAGES) * tile_bytes, p.s + state_index(x) * p.KP * SC_COLS, tile_bytes, bar);
+    issued = i + 1;
+  };
+  if (tid == 0)
+    for (int i = 0; i < RD_STAGES - 1; ++i) load(i);
+  float q[RD_VEC], k[RD_VEC], n[RD_VEC], v = 0.f, gi = 0.f, gf = 0.f, m0 = 0.f;
+  Unit x{};
+  bool fresh = false;
+  auto fetch = [&](int u) {
+    x = unit_of(u);
+    fresh = p.seq_lens[x.b] == 1;
+    const T* row = reinterpret_cast<const T*>(p.proj) + x.b * p.ld;
+    const float* nt = p.n + state_index(x) * p.KP;
+#pragma unroll
+    for (int i = 0; i < RD_VEC; ++i) {
+      const int r = tid + i * RD_THREADS;
+      q[i] = k[i] = n[i] = 0.f;
+      if (r < p.dk) {
+        q[i] = to_f<T>(row[p.q_col + x.h * p.KP + r]) * p.q_scale;
+        k[i] = to_f<T>(row[p.k_col + x.h * p.KP + r]);
+        if (p.gated && !fresh) n[i] = nt[r];
+      }
+    }
+    if (tid < SC_COLS) v = to_f<T>(row[p.v_col + x.h * p.VP + x.tile * SC_COLS + tid]);
+    if (p.gated) {
+      gi = p.small[x.b * p.ld_small + x.h];
+      gf = p.small[x.b * p.ld_small + p.H + x.h];
+      m0 = fresh ? 0.f : p.m[state_index(x)];
+    }
+  };
+  if ((int)blockIdx.x < units) fetch(blockIdx.x);
+  bool ok = true;
+  int it = 0;
+  for (int u = blockIdx.x; u < units; u += gridDim.x, ++it) {
+    const Unit cur = x;
+    const bool zero = fresh;
+    float a, w = 1.f, m = 0.f;
+    if (p.gated) {
+      gi = p.cap * tanhf((gi + p.bias_i[cur.h]) / p.cap);
+      gf = log_sigmoid_f(p.cap * tanhf((gf + p.bias_f[cur.h]) / p.cap));
+      m = fmaxf(gf + m0, gi);
+      a = expf(gf + m0 - m);
+      w = expf(gi - m);
+    } else {
+      a = p.decay[cur.h];
+    }
+    const long long si = state_index(cur);
+    float nq = 0.f;
+#pragma unroll
+    for (int i = 0; i < RD_VEC; ++i) {
+      const int r = tid + i * RD_THREADS;
+      if (r < p.dk) {
+        const float kw = w * k[i];
+        qs[r] = q[i];
+        ks[r] = kw;
+        if (p.gated) {
+          const float nn = fmaf(a, n[i], kw);
+          nq = fmaf(q[i], nn, nq);
+          if (cur.slot >= 0) p.n[si * p.KP + r] = nn;
+        }
+      }
+    }
+    if (tid < SC_COLS) vs[tid] = v;
+    if (p.gated && tid == 0 && cur.slot >= 0) p.m[si] = m;
+    __syncthreads();
+    if (u + (int)gridDim.x < units) fetch(u + gridDim.x);
+    const int stage = it % RD_STAGES;
+    ok = mbar_wait_bounded(smem_u32(&full[stage]), (uint32_t)((it / RD_STAGES) & 1), &abort_flag, p.status, ST_TIMEOUT_SMEM_FULL);
+    ok = __syncthreads_and(ok);
+    if (!ok) break;
+    float4* S = reinterpret_cast<float4*>(smem_raw + stage * tile_bytes);
+    const float4 vv = *reinterpret_cast<const float4*>(&vs[c4 * 4]);
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int r = r0; r < p.dk; r += RD_THREADS / 8) {
+      float4 s = zero ? make_float4(0.f, 0.f, 0.f, 0.f) : S[r * (SC_COLS / 4) + c4];
+      const float kw = ks[r], qr = qs[r];
+      s.x = fmaf(a, s.x, kw * vv.x);
+      s.y = fmaf(a, s.y, kw * vv.y);
+      s.z = fmaf(a, s.z, kw * vv.z);
+      s.w = fmaf(a, s.w, kw * vv.w);
+      acc.x = fmaf(qr, s.x, acc.x);
+      acc.y = fmaf(qr, s.y, acc.y);
+      acc.z = fmaf(qr, s.z, acc.z);
+      acc.w = fmaf(qr, s.w, acc.w);
+      S[r * (SC_COLS / 4) + c4] = s;
+    }
+    fence_proxy_async_smem();
+#pragma unroll
+    for (int o = 8; o < 32; o <<= 1) {
+      acc.x += __shfl_xor_sync(0xffffffffu, acc.x, o);
+      acc.y += __shfl_xor_sync(0xffffffffu, acc.y, o);
+      acc.z += __shfl_xor_sync(0xffffffffu, acc.z, o);
+      acc.w += __shfl_xor_sync(0xffffffffu, acc.w, o);
+    }
+    if (p.gated) nq = warp_sum(nq);
+    if (lane < 8) *reinterpret_cast<float4*>(&red[warp][lane * 4]) = acc;
+    if (lane == 0) red_n[warp] = nq;
+    __syncthreads();
+    if (tid == 0) {
+      if (cur.slot >= 0) bulk_store(p.s + si * p.KP * SC_COLS, ring + stage * tile_bytes, tile_bytes);
+      else asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+      asm volatile("cp.async.bulk.wait_group.read 1;" ::: "memory");     // the tile stored one unit ago has left its stage
+      load(it + RD_STAGES - 1);
+    }
+    if (tid < SC_COLS) {
+      float o = 0.f, d = 0.f;
+#pragma unroll
+      for (int i = 0; i < RD_THREADS / 32; ++i) { o += red[i][tid]; d += red_n[i]; }
+      if (p.gated) o /= fmaxf(fabsf(d), expf(-m)) + 1e-6f;
+      p.out[cur.b * p.ldo + cur.h * p.VP + cur.tile * SC_COLS + tid] = cur.slot < 0 ? 0.f : o;
+    }
+  }
+  if (tid == 0) {
+    if (!ok)                                                 // no copy may land after the CTA has gone
+      for (int i = it; i < issued; ++i) {
+        const uint64_t t0 = globaltimer_ns();
+        while (!mbar_try_wait(smem_u32(&full[i % RD_STAGES]), (uint32_t)((i / RD_STAGES) & 1)))
+          if (globaltimer_ns() - t0 > 50000000ull) break;
+      }
+    asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+  }
+}
+
+template <typename T>
+static int launch_decode(const ScanParams& p, int B, cudaStream_t stream) {
+  static int sms[64] = {};
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
+  const int smem = RD_STAGES * p.dk * SC_COLS * 4;
+  if (sms[dev] == 0) {
+    int n = 0;
+    if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess ||
+        cudaFuncSetAttribute(recurrent_decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, RD_STAGES * RD_MAX_DK * SC_COLS * 4) != cudaSuccess)
+      return -10;
+    sms[dev] = n;
+  }
+  const int per_sm = 200 * 1024 / (smem + 7 * 1024) > 6 ? 6 : 200 * 1024 / (smem + 7 * 1024);
+  const int units = B * p.H * (p.VP / SC_COLS), grid = units < sms[dev] * per_sm ? units : sms[dev] * per_sm;
+  return launch_kernel(recurrent_decode_kernel<T>, dim3(grid), dim3(RD_THREADS), smem, stream, p, units) == cudaSuccess ? 0 : -11;
+}
+
+// ------------------------------------------------------------------------------------------
 // Chunked form. In a chunk of up to CH tokens of one sequence let F_t be the sum of the logarithms of the decays up to and
 // including token t, g_j = log b_j - F_j, and (m, S, n) the state in front of the chunk. Then with B_t = max(m, max_{j<=t} g_j)
 //
@@ -224,13 +417,14 @@ struct ChunkParams {
   float* u;                // [chunks, H, tiles, KP, 32]
   float* un;               // [chunks, H, KP]
   float2* um;              // [chunks, H] {F_C, F_C + G}
+  float* gates;            // [chunks, H, 3, CH] see recurrent_chunk_gates_kernel
   __nv_bfloat16* s_hi;     // [chunks, H, VP/64, KP, 64] state in front of the chunk
   __nv_bfloat16* s_lo;
   float* s_n;              // [chunks, H, KP]
   float* s_m;              // [chunks, H]
   float* out;
   long long ldo;
-  int H, dk, KP, VP, num_slots, silu, gated;
+  int H, dk, KP, VP, num_slots, gated;
   int* status;
 };
 
@@ -240,9 +434,9 @@ __device__ __forceinline__ float chunk_exp2(float x) {
   return y;
 }
 
-// g_j and F_j of the chunk's tokens (in units of log2), by the first warp: four tokens per lane. Invalid tokens get g = -inf.
+// g_j and F_j of the chunk's tokens (in units of log2), by one warp: four tokens per lane. Invalid tokens get g = -inf.
 // gs[t] = g_t, bs[t] = running maximum of g (gated) or -F_t, fs[t] = F_t. Returns {F_C, max g} in every lane of the warp.
-__device__ __forceinline__ float2 chunk_gates(const ChunkParams& p, int h, int row0, int n, float* gs, float* bs, float* fs = nullptr) {
+__device__ __forceinline__ float2 chunk_gates(const ChunkParams& p, int h, int row0, int n, float* gs, float* bs, float* fs) {
   const int lane = threadIdx.x & 31;
   float lf[4], li[4], F[4], run = 0.f;
 #pragma unroll
@@ -291,7 +485,7 @@ __device__ __forceinline__ float2 chunk_gates(const ChunkParams& p, int h, int r
   for (int i = 0; i < 4; ++i) {
     gs[lane * 4 + i] = g[i];
     bs[lane * 4 + i] = p.gated ? fmaxf(prev, top[i]) : -F[i];
-    if (fs != nullptr) fs[lane * 4 + i] = F[i];
+    fs[lane * 4 + i] = F[i];
   }
   return make_float2(total, all);
 }
@@ -299,27 +493,33 @@ __device__ __forceinline__ float2 chunk_gates(const ChunkParams& p, int h, int r
 // 16-byte unit u (8 columns) of row r in a [rows, 64] swizzled chunk
 __device__ __forceinline__ uint32_t chunk_addr(int r, int u) { return (uint32_t)(r * CH_ROWB + ((u ^ (r & 7)) << 4)); }
 
-__device__ __forceinline__ uint4 silu8(uint4 v) {
-  auto one = [](uint32_t x) {
-    const float2 f = unpack_bf16x2(x);
-    return pack_bf16x2(silu_f(f.x), silu_f(f.y));
-  };
-  return make_uint4(one(v.x), one(v.y), one(v.z), one(v.w));
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {     // zeros when not valid
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
 }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-// [CH, DK] columns of a projection into swizzled chunks; rows past n are zero
+// [CH, DK] columns of a projection into swizzled chunks, asynchronously; rows past n are zero
 template <int DK>
-__device__ __forceinline__ void chunk_load(uint8_t* dst, const __nv_bfloat16* src, long long ld, int n, bool silu) {
-#pragma unroll 4
+__device__ __forceinline__ void chunk_load(uint32_t dst, const __nv_bfloat16* src, long long ld, int n) {
+#pragma unroll
   for (int i = threadIdx.x; i < CH * (DK / 8); i += CHT) {
     const int r = i / (DK / 8), u = i % (DK / 8);
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < n) {
-      v = *reinterpret_cast<const uint4*>(src + r * ld + u * 8);
-      if (silu) v = silu8(v);
-    }
-    *reinterpret_cast<uint4*>(dst + (u >> 3) * CH_CHUNK + chunk_addr(r, u & 7)) = v;
+    cp_async16(dst + (u >> 3) * CH_CHUNK + chunk_addr(r, u & 7), src + (r < n ? r : 0) * ld + u * 8, r < n);
   }
+}
+
+// Gates of every chunk and head, a warp each: g, B' (running maximum of g, or -F) and F per token in units of log2.
+__global__ void __launch_bounds__(256) recurrent_chunk_gates_kernel(const ChunkParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5);
+  if (h >= p.H) return;
+  const int4 ck = p.chunks[c];
+  const long long ch = (long long)c * p.H + h;
+  float* g = p.gates + ch * 3 * CH;
+  const float2 t = chunk_gates(p, h, ck.x, ck.y, g, g + CH, g + 2 * CH);
+  const float G = p.gated ? t.y : -t.x;
+  if ((threadIdx.x & 31) == 0) p.um[ch] = make_float2(t.x, t.x + G);
 }
 
 // What a chunk adds to the state: U [KP, 64 value channels] of one head. blockIdx: chunk, head, 64 value channels.
@@ -334,7 +534,7 @@ template <int DK>
 __global__ void __launch_bounds__(CHT) recurrent_chunk_state_kernel(const ChunkParams p) {
   using Cfg = ChunkStateCfg<DK>;
   extern __shared__ __align__(128) uint8_t smem_raw[];
-  __shared__ float gs[CH], bs[CH], nred[4][DK];
+  __shared__ float gs[CH], nred[4][DK];
   __shared__ __align__(8) uint64_t done;
   __shared__ uint32_t tmem_base_smem;
   __shared__ int abort_flag;
@@ -343,7 +543,6 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_state_kernel(const ChunkP
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* hi = smem_raw + (base - smem_u32(smem_raw));
   uint8_t* lo = hi + Cfg::kKBytes;
-  uint8_t* vt = lo + Cfg::kKBytes;
   if (threadIdx.x == 0) {
     abort_flag = 0;
     mbar_init(smem_u32(&done), 1);
@@ -357,37 +556,45 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_state_kernel(const ChunkP
   pdl_wait();
   const int4 ck = p.chunks[c];
   const int row0 = ck.x, n = ck.y;
-  if (warp == 0) {
-    const float2 t = chunk_gates(p, h, row0, n, gs, bs);
-    const float G = p.gated ? t.y : -t.x;
-    gs[lane * 4] -= G; gs[lane * 4 + 1] -= G; gs[lane * 4 + 2] -= G; gs[lane * 4 + 3] -= G;
-    if (lane == 0 && z == 0) p.um[(long long)c * p.H + h] = make_float2(t.x, t.x + G);
+  const long long ch = (long long)c * p.H + h;
+  chunk_load<64>(base + 2 * Cfg::kKBytes, p.proj + row0 * p.ld + p.v_col + h * p.VP + z * 64, p.ld, n);
+  if (threadIdx.x < CH) {
+    const float2 t = p.um[ch];
+    gs[threadIdx.x] = chunk_exp2(p.gates[ch * 3 * CH + threadIdx.x] - (t.y - t.x));     // weights relative to exp(F_C + G)
   }
-  chunk_load<64>(vt, p.proj + row0 * p.ld + p.v_col + h * p.VP + z * 64, p.ld, n, p.silu);
-  __syncthreads();
   const __nv_bfloat16* k = p.proj + row0 * p.ld + p.k_col + h * p.KP;
-#pragma unroll 2
-  for (int i = threadIdx.x; i < CH * (DK / 8); i += CHT) {
-    const int r = i / (DK / 8), u = i % (DK / 8);
-    uint4 a = make_uint4(0u, 0u, 0u, 0u), b = a;
-    if (r < n) {
-      const uint4 v = *reinterpret_cast<const uint4*>(k + r * p.ld + u * 8);
-      const float w = chunk_exp2(gs[r]);
+  constexpr int UNITS = CH * (DK / 8) / CHT, BATCH = UNITS % 8 == 0 ? 8 : 4;
+  static_assert(UNITS % BATCH == 0, "whole batches");
+  __syncthreads();
+#pragma unroll 1
+  for (int i0 = 0; i0 < UNITS; i0 += BATCH) {
+    uint4 raw[BATCH];
+#pragma unroll
+    for (int i = 0; i < BATCH; ++i) {
+      const int e = threadIdx.x + (i0 + i) * CHT, r = e / (DK / 8), u = e % (DK / 8);
+      raw[i] = make_uint4(0u, 0u, 0u, 0u);
+      if (r < n) raw[i] = *reinterpret_cast<const uint4*>(k + r * p.ld + u * 8);
+    }
+#pragma unroll
+    for (int i = 0; i < BATCH; ++i) {
+      const int e = threadIdx.x + (i0 + i) * CHT, r = e / (DK / 8), u = e % (DK / 8);
+      const float w = gs[r];
+      uint4 a, b;
       auto one = [&](uint32_t x, uint32_t& l) {
         float2 f = unpack_bf16x2(x);
-        if (p.silu) { f.x = silu_f(f.x); f.y = silu_f(f.y); }
         f.x *= w; f.y *= w;
         const uint32_t o = pack_bf16x2(f.x, f.y);
         const float2 back = unpack_bf16x2(o);
         l = pack_bf16x2(f.x - back.x, f.y - back.y);
         return o;
       };
-      a.x = one(v.x, b.x); a.y = one(v.y, b.y); a.z = one(v.z, b.z); a.w = one(v.w, b.w);
+      a.x = one(raw[i].x, b.x); a.y = one(raw[i].y, b.y); a.z = one(raw[i].z, b.z); a.w = one(raw[i].w, b.w);
+      const uint32_t at = (u >> 3) * CH_CHUNK + chunk_addr(r, u & 7);
+      *reinterpret_cast<uint4*>(hi + at) = a;
+      *reinterpret_cast<uint4*>(lo + at) = b;
     }
-    const uint32_t at = (u >> 3) * CH_CHUNK + chunk_addr(r, u & 7);
-    *reinterpret_cast<uint4*>(hi + at) = a;
-    *reinterpret_cast<uint4*>(lo + at) = b;
   }
+  cp_async_wait_all();
   fence_proxy_async_smem();
   tc_fence_before();
   __syncthreads();
@@ -426,14 +633,14 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_state_kernel(const ChunkP
     }
     __syncthreads();
     for (int i = threadIdx.x; i < DK; i += CHT)
-      p.un[((long long)c * p.H + h) * p.KP + i] = (nred[0][i] + nred[1][i]) + (nred[2][i] + nred[3][i]);
+      p.un[ch * p.KP + i] = (nred[0][i] + nred[1][i]) + (nred[2][i] + nred[3][i]);
   }
   bool ok = mbar_wait_bounded(smem_u32(&done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
   ok = __all_sync(0xffffffffu, ok);
   tc_fence_after();
   if (ok) {
     const int qd = warp & 3, half = warp >> 2;       // lanes of a TMEM quarter; the two warps of a quarter split the columns
-    float* u = p.u + (((long long)c * p.H + h) * (p.VP / 32) + z * 2 + half) * p.KP * 32;
+    float* u = p.u + (ch * (p.VP / 32) + z * 2 + half) * p.KP * 32;
 #pragma unroll
     for (int m0 = 0; m0 < DK; m0 += 128) {
       uint32_t v[32];
@@ -564,7 +771,6 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkPar
   uint8_t* q_p = smem_raw + (base - smem_u32(smem_raw));
   uint8_t* k_p = q_p + Cfg::kQBytes;
   uint8_t* sv_p = k_p + Cfg::kKpBytes;
-  uint8_t* sl_p = sv_p + Cfg::kSvBytes;
   const uint32_t q_s = base, k_s = q_s + Cfg::kQBytes, sv_s = k_s + Cfg::kKpBytes, sl_s = sv_s + Cfg::kSvBytes;
   if (threadIdx.x == 0) {
     abort_flag = 0;
@@ -582,25 +788,26 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkPar
   const int row0 = ck.x, n = ck.y;
   const long long ch = (long long)c * p.H + h;
   const __nv_bfloat16* rows = p.proj + row0 * p.ld;
-  if (warp == 0) {
-    chunk_gates(p, h, row0, n, gs, bs, fs);
-    if (lane == 0) m_in = p.gated ? p.s_m[ch] : 0.f;
-  }
-  if (p.gated)
-    for (int i = threadIdx.x; i < DK; i += CHT) ns[i] = p.s_n[ch * p.KP + i];
+  chunk_load<DK>(q_s, rows + p.q_col + h * p.KP, p.ld, n);
+  chunk_load<DK>(k_s, rows + p.k_col + h * p.KP, p.ld, n);
   {
     const long long at = (ch * (p.VP / 64) + z) * p.KP * 64;
-    const uint4* gh = reinterpret_cast<const uint4*>(p.s_hi + at);
-    const uint4* gl = reinterpret_cast<const uint4*>(p.s_lo + at);
-#pragma unroll 2
+#pragma unroll
     for (int i = threadIdx.x; i < DK * 8; i += CHT) {
       const uint32_t a = chunk_addr(i >> 3, i & 7);
-      *reinterpret_cast<uint4*>(sv_p + a) = gh[i];
-      *reinterpret_cast<uint4*>(sl_p + a) = gl[i];
+      cp_async16(sv_s + a, p.s_hi + at + i * 8, true);
+      cp_async16(sl_s + a, p.s_lo + at + i * 8, true);
     }
   }
-  chunk_load<DK>(q_p, rows + p.q_col + h * p.KP, p.ld, n, p.silu);
-  chunk_load<DK>(k_p, rows + p.k_col + h * p.KP, p.ld, n, p.silu);
+  if (threadIdx.x < CH) {
+    const float* g = p.gates + ch * 3 * CH + threadIdx.x;
+    gs[threadIdx.x] = g[0];
+    bs[threadIdx.x] = g[CH];
+    fs[threadIdx.x] = g[2 * CH];
+  }
+  if (threadIdx.x == CH) m_in = p.gated ? p.s_m[ch] : 0.f;
+  if (p.gated)
+    for (int i = threadIdx.x; i < DK; i += CHT) ns[i] = p.s_n[ch * p.KP + i];
   uint4 vr[CH * 8 / CHT];                            // V waits in registers until the state's shared memory is free
 #pragma unroll
   for (int i = 0; i < CH * 8 / CHT; ++i) {
@@ -608,6 +815,7 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkPar
     vr[i] = make_uint4(0u, 0u, 0u, 0u);
     if (r < n) vr[i] = *reinterpret_cast<const uint4*>(rows + r * p.ld + p.v_col + h * p.VP + z * 64 + u * 8);
   }
+  cp_async_wait_all();
   fence_proxy_async_smem();
   tc_fence_before();
   __syncthreads();
@@ -678,7 +886,7 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkPar
 #pragma unroll
     for (int i = 0; i < CH * 8 / CHT; ++i) {
       const int e = threadIdx.x + i * CHT;
-      *reinterpret_cast<uint4*>(sv_p + chunk_addr(e >> 3, e & 7)) = p.silu ? silu8(vr[i]) : vr[i];
+      *reinterpret_cast<uint4*>(sv_p + chunk_addr(e >> 3, e & 7)) = vr[i];
     }
   }
   row_sum[half][t] = sum + c_in * qn;
@@ -742,6 +950,7 @@ static int launch_chunks(const ChunkParams& p, int n_chunks, int n_seq, cudaStre
     attr_dev[dev] = true;
   }
   const dim3 grid(n_chunks, p.H, p.VP / 64);
+  if (launch_kernel(recurrent_chunk_gates_kernel, dim3(n_chunks, (p.H + 7) / 8), dim3(256), 0, stream, p) != cudaSuccess) return -14;
   if (launch_kernel(recurrent_chunk_state_kernel<DK>, grid, dim3(CHT), ChunkStateCfg<DK>::kSmem, stream, p) != cudaSuccess) return -11;
   if (launch_kernel(recurrent_chunk_chain_kernel, dim3(DK / 32, p.H * (p.VP / SC_COLS), n_seq), dim3(256), 0, stream, p) != cudaSuccess) return -12;
   return launch_kernel(recurrent_chunk_out_kernel<DK>, grid, dim3(CHT), ChunkOutCfg<DK>::kSmem, stream, p) == cudaSuccess ? 0 : -13;
@@ -807,18 +1016,20 @@ void rb_recurrent_set_pdl(int on) { rb::pdl_enabled() = on != 0; }
 int rb_recurrent_scan(const void* proj, long long ld, int q_col, int k_col, int v_col, const float* small, long long ld_small, const float* decay,
                       const float* bias_i, const float* bias_f, float cap, float q_scale, float* s, float* n, float* m, const int* slots,
                       const int* cu_q, const int* seq_lens, float* out, long long ldo, int H, int dk, int KP, int VP, int B, int num_slots,
-                      int silu, int gated, int rows, int dtype, int* status, cudaStream_t stream) {
+                      int gated, int rows, int dtype, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (H <= 0 || H > 65535 || B > 65535 || dk <= 0 || dk > KP || VP % SC_COLS != 0 || (gated ? small == nullptr : decay == nullptr)) return -1;
   const ScanParams p{proj, ld, q_col, k_col, v_col, small, ld_small, decay, bias_i, bias_f, cap, q_scale, s, n, m, slots, cu_q, seq_lens,
-                     out, ldo, H, dk, KP, VP, num_slots, silu, gated, rows, status};
+                     out, ldo, H, dk, KP, VP, num_slots, gated, rows, status};
+  if (cu_q == nullptr && dk <= RD_MAX_DK)
+    return dtype == 0 ? launch_decode<__nv_bfloat16>(p, B, stream) : launch_decode<float>(p, B, stream);
   return dtype == 0 ? launch_scan<__nv_bfloat16>(p, B, stream) : launch_scan<float>(p, B, stream);
 }
 
 // Workspace of the chunked form in bytes.
 long long rb_recurrent_chunk_workspace(int n_chunks, int H, int KP, int VP) {
   const long long ch = (long long)n_chunks * H;
-  return ch * ((long long)KP * VP * 8 + KP * 8 + 16) + 256;
+  return ch * ((long long)KP * VP * 8 + KP * 8 + 3 * CH * 4 + 16) + 256;
 }
 
 // Sequences of any length, `chunks` [n_chunks] and `seq_chunks` [n_seq + 1] as ChunkParams describes; slots, seq_lens and cu_q belong to
@@ -826,7 +1037,7 @@ long long rb_recurrent_chunk_workspace(int n_chunks, int H, int KP, int VP) {
 int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, int v_col, const float* small, long long ld_small, const float* decay,
                         const float* bias_i, const float* bias_f, float cap, float q_scale, float* s, float* n, float* m, const void* chunks,
                         const int* seq_chunks, const int* slots, const int* cu_q, const int* seq_lens, float* out, long long ldo, void* workspace,
-                        int n_chunks, int n_seq, int H, int dk, int KP, int VP, int num_slots, int silu, int gated, int* status, cudaStream_t stream) {
+                        int n_chunks, int n_seq, int H, int dk, int KP, int VP, int num_slots, int gated, int* status, cudaStream_t stream) {
   if (n_chunks <= 0 || n_seq <= 0) return 0;
   if (H <= 0 || H > 65535 || n_seq > 65535 || dk <= 0 || dk > KP || KP % 64 != 0 || VP % 64 != 0 || ld % 8 != 0 || ldo % 4 != 0 ||
       (gated ? small == nullptr : decay == nullptr) || workspace == nullptr)
@@ -837,7 +1048,7 @@ int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, in
   p.small = small; p.ld_small = ld_small; p.decay = decay; p.bias_i = bias_i; p.bias_f = bias_f; p.cap = cap; p.q_scale = q_scale;
   p.chunks = (const int4*)chunks; p.seq_chunks = seq_chunks; p.slots = slots; p.seq_lens = seq_lens; p.cu_q = cu_q;
   p.s = s; p.n = n; p.m = m; p.out = out; p.ldo = ldo;
-  p.H = H; p.dk = dk; p.KP = KP; p.VP = VP; p.num_slots = num_slots; p.silu = silu; p.gated = gated; p.status = status;
+  p.H = H; p.dk = dk; p.KP = KP; p.VP = VP; p.num_slots = num_slots; p.gated = gated; p.status = status;
   float* w = (float*)workspace;
   p.u = w; w += ch * KP * VP;
   p.s_hi = (__nv_bfloat16*)w; w += ch * KP * VP / 2;
@@ -845,6 +1056,7 @@ int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, in
   p.un = w; w += ch * KP;
   p.s_n = w; w += ch * KP;
   p.um = (float2*)w; w += ch * 2;
+  p.gates = w; w += ch * 3 * CH;
   p.s_m = w;
   switch (KP) {
     case 64: return launch_chunks<64>(p, n_chunks, n_seq, stream);

@@ -18,6 +18,10 @@ class Part:
     """A kind of mixer or feed-forward in one runner. ``forward`` reads the activations ``inp [T, wp]`` and, for mixers and dense
     feed-forwards, fills ``y [T, wp]`` (fp32)."""
 
+    # mixers: the layer's narrow fp32 projection rides along as the last rows of the mixer's joint projection (``make`` is told how
+    # many) and ``project`` fills it; otherwise the runner multiplies it on its own
+    fuses_tail = False
+
     def __init__(self, runner):
         self.r = weakref.proxy(runner)       # no cycle: the runner's graphs go when its engine does
         self.layers: list[Any] = []          # weights made so far
@@ -43,7 +47,7 @@ class Part:
     def zeros(self, *shape: int, dtype: torch.dtype | None = None) -> torch.Tensor:
         return torch.zeros(*shape, dtype=dtype or self.r.dtype, device=self.r.device)
 
-    def make(self, spec):
+    def make(self, spec, tail: int = 0):
         raise NotImplementedError
 
     def new_cache(self, w):
@@ -62,6 +66,9 @@ class Part:
     # ---- one step
     def plan(self, b) -> Any:
         return None
+
+    def project(self, w, inp: torch.Tensor, tail: torch.Tensor | None) -> None:
+        """First half of a mixer: its projections of ``inp``, and the narrow one into ``tail`` (fp32)."""
 
 
 def load_heads(dst: torch.Tensor, src: torch.Tensor, heads: int, dim: int, padded: int) -> None:

@@ -23,18 +23,20 @@ class KeyValueWeights:
 
 
 class KeyValuePart(Part):
+    fuses_tail = True
+
     @staticmethod
     def cache_row_elements(spec) -> int:
         g = keyvalue_geometry(spec)
         return g.kv_heads * g.dp
 
-    def make(self, spec: KeyValueAttentionSpec) -> KeyValueWeights:
+    def make(self, spec: KeyValueAttentionSpec, tail: int = 0) -> KeyValueWeights:
         g = keyvalue_geometry(spec)
         if g.dp > MAX_HEAD:
             raise ValueError(f"the attention kernels take heads of up to {MAX_HEAD} channels")
         w = KeyValueWeights()
         w.spec, w.geo = spec, g
-        w.wproj, w.bproj = self.zeros(g.proj, self.r.wp), self.zeros(g.proj)
+        w.wproj, w.bproj = self.zeros(g.proj + tail, self.r.wp), self.zeros(g.proj + tail)
         w.wo, w.bo = self.zeros(self.r.wp, g.heads * g.dp), self.zeros(self.r.wp)
         w.sink = self.zeros(g.heads, dtype=torch.float32)
         self.layers.append(w)
@@ -57,7 +59,7 @@ class KeyValuePart(Part):
         H, G, D, d = g.heads, g.kv_heads, g.dim, g.dp
         load_heads(w.wproj[:g.k_col], get(p + "q"), H, D, d)
         load_heads(w.wproj[g.k_col:g.gate_col], get(p + "k"), G, D, d)
-        load_heads(w.wproj[g.gate_col:], get(p + "g"), H, D, d)
+        load_heads(w.wproj[g.gate_col:g.proj], get(p + "g"), H, D, d)
         load_head_vector(w.bproj[:g.k_col], get(p + "q.b"), H, D, d)
         load_head_vector(w.bproj[g.k_col:g.gate_col], get(p + "k.b"), G, D, d)
         load_head_columns(w.wo, get(p + "o"), H, D, d)
@@ -68,11 +70,16 @@ class KeyValuePart(Part):
         single = b.rows if b.cu_q is None else b.n_single
         return self.splits.get(single, {})
 
+    def _projected(self, w: KeyValueWeights, T: int) -> torch.Tensor:
+        return self.proj[:T * w.geo.proj].view(T, w.geo.proj)
+
+    def project(self, w: KeyValueWeights, inp, tail) -> None:
+        ops.gemm(inp, w.wproj, bias=w.bproj, out=self._projected(w, inp.shape[0]), tail=tail)
+
     def forward(self, w: KeyValueWeights, cache, inp, y, b, splits, small=None) -> None:
         T, g, m = b.num_tokens, w.geo, w.spec
-        proj = self.proj[:T * g.proj].view(T, g.proj)
+        proj = self._projected(w, T)
         out = self.out[:T * g.heads * g.dp].view(T, g.heads * g.dp)
-        ops.gemm(inp, w.wproj, bias=w.bproj, out=proj)
         ops.kv_append(proj, g, b.positions, b.slots, m.q_temp.coef, m.q_temp.every, cache)
         ops.kv_attention(proj, g, cache, b.block_tables, b.cu_q, b.seq_lens, w.sink, out, scale=m.scale, rows=T, max_q=b.max_new,
                          n_single=b.n_single, workspace=self.workspace, splits=splits.get(g, 1))

@@ -55,7 +55,7 @@ class LatentPart(Part):
     def cache_row_elements(spec) -> int:
         return latent_geometry(spec).cw
 
-    def make(self, spec: LatentAttentionSpec) -> LatentWeights:
+    def make(self, spec: LatentAttentionSpec, tail: int = 0) -> LatentWeights:
         r, f32 = self.r, torch.float32
         g = latent_geometry(spec)
         if g.rw > MAX_LATENT or g.cw > MAX_CACHE_ROW:

@@ -25,6 +25,8 @@ class RecurrentWeights:
 
 
 class RecurrentPart(Part):
+    fuses_tail = True
+
     @staticmethod
     def state_floats(spec) -> int:
         return recurrent_geometry(spec).state_floats
@@ -33,13 +35,13 @@ class RecurrentPart(Part):
     def small_rows(spec) -> int:
         return 2 * spec.heads if isinstance(spec, MatrixMemorySpec) else 0
 
-    def make(self, spec) -> RecurrentWeights:
+    def make(self, spec, tail: int = 0) -> RecurrentWeights:
         g, f32 = recurrent_geometry(spec), torch.float32
         if g.kp > MAX_DIM:
             raise ValueError(f"the recurrent kernels take up to {MAX_DIM} key channels per head")
         w = RecurrentWeights()
         w.spec, w.geo = spec, g
-        w.wproj, w.wo = self.zeros(g.proj, self.r.wp), self.zeros(self.r.wp, g.heads * g.vp)
+        w.wproj, w.wo = self.zeros(g.proj + tail, self.r.wp), self.zeros(self.r.wp, g.heads * g.vp)
         w.norm = self.zeros(g.heads * g.vp, dtype=f32)
         w.decay = w.bias_i = w.bias_f = None
         w.cap = 1.0
@@ -66,7 +68,7 @@ class RecurrentPart(Part):
         load_heads(w.wproj[:ok], get(p + "q"), H, g.dim, g.kp)
         load_heads(w.wproj[ok:ov], get(p + "k"), H, g.dim, g.kp)
         load_heads(w.wproj[ov:og], get(p + "v"), H, g.vdim, g.vp)
-        load_heads(w.wproj[og:], get(p + "g"), H, g.vdim, g.vp)
+        load_heads(w.wproj[og:g.proj], get(p + "g"), H, g.vdim, g.vp)
         load_head_columns(w.wo, get(p + "o"), H, g.vdim, g.vp)
         load_head_vector(w.norm, get(p + "norm").float(), H, g.vdim, g.vp)
         if g.gated:
@@ -78,12 +80,17 @@ class RecurrentPart(Part):
             dst[:w.geo.heads, :self.r.cfg.hidden_size].copy_(get(p + "i"))
             dst[w.geo.heads:2 * w.geo.heads, :self.r.cfg.hidden_size].copy_(get(p + "f"))
 
+    def _projected(self, w: RecurrentWeights, T: int) -> torch.Tensor:
+        return self.proj[:T * w.geo.proj].view(T, w.geo.proj)
+
+    def project(self, w: RecurrentWeights, inp, tail) -> None:
+        ops.gemm(inp, w.wproj, out=self._projected(w, inp.shape[0]), silu_cols=w.geo.silu_cols, tail=tail)
+
     def forward(self, w: RecurrentWeights, state: RecurrentState, inp, y, b, plan, small=None) -> None:
         T, g = b.num_tokens, w.geo
         n = g.heads * g.vp
-        proj = self.proj[:T * g.proj].view(T, g.proj)
+        proj = self._projected(w, T)
         o, out = self.o[:T * n].view(T, n), self.out[:T * n].view(T, n)
-        ops.gemm(inp, w.wproj, out=proj)
         self.recur(w, state, proj, small, o, b, plan)
         ops.gated_norm(o, w.norm, proj[:, g.offsets[3]:], g, self.r.cfg.norm_eps, out, g.gated)
         ops.gemm(out, w.wo, out=y, out_f32=True)
@@ -101,9 +108,11 @@ class RecurrentPart(Part):
         n_seq, rows, table = plan
         if table is not None and not chunked_supported(g):
             n_seq, rows, table = b.rows, b.num_tokens, None
-        args = (proj, small, g, w.decay, w.bias_i, w.bias_f, w.cap, state, b.state_slots, b.cu_q, b.seq_lens, o)
-        if n_seq > 0:
-            ops.recurrent_scan(*args, rows, n_seq)
+        args = (proj, small, g, w.decay, w.bias_i, w.bias_f, w.cap, state, b.state_slots)
+        if b.n_single > 0:
+            ops.recurrent_scan(*args, None, b.seq_lens, o, b.n_single, b.n_single)
+        if n_seq > b.n_single:
+            ops.recurrent_scan(*args, b.cu_q, b.seq_lens, o, rows, n_seq, b.n_single)
         if table is not None:
             room = torch.empty(chunk_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=o.device)
-            ops.recurrent_chunks(*args, table, room)
+            ops.recurrent_chunks(*args, b.cu_q, b.seq_lens, o, table, room)

@@ -34,7 +34,7 @@ from .stack_parts.base import Part, up
 class StackLayer:
     """Weights of one layer: those of its mixer and feed-forward parts, the norms, the narrow fp32 projection."""
 
-    __slots__ = ("spec", "mixer", "mix", "feed_forward", "ff", "norm1", "norm2", "wsmall", "mix_small")
+    __slots__ = ("spec", "mixer", "mix", "feed_forward", "ff", "norm1", "norm2", "wsmall", "wsmall_ff", "mix_small")
 
 
 @dataclass
@@ -110,7 +110,6 @@ class StackRunner(RunnerBase):
             lw = StackLayer()
             lw.spec = spec
             lw.mixer = self._part(_mixer_part(spec))
-            lw.mix = lw.mixer.make(spec.mixer)
             lw.norm1, lw.norm2 = norm(), None
             lw.feed_forward = lw.ff = None
             lw.mix_small = up(lw.mixer.small_rows(spec.mixer), 8)
@@ -120,7 +119,11 @@ class StackRunner(RunnerBase):
                 lw.ff = lw.feed_forward.make(spec.mlp)
                 lw.norm2 = None if self.parallel else norm()
                 ff_small = up(lw.feed_forward.small_rows(spec.mlp), 8)
-            lw.wsmall = zeros(lw.mix_small + ff_small, self.wp) if lw.mix_small + ff_small else None
+            # the mixer's gate logits and, where both read the same activations, the router
+            n = lw.mix_small + (ff_small if self.parallel else 0)
+            lw.mix = lw.mixer.make(spec.mixer, n)
+            lw.wsmall = None if n == 0 else lw.mix.wproj[-n:] if lw.mixer.fuses_tail else zeros(n, self.wp)
+            lw.wsmall_ff = None if ff_small == 0 else lw.wsmall[lw.mix_small:] if self.parallel else zeros(ff_small, self.wp)
             self.layers.append(lw)
         self.runs = [StackRun(self.layers[x.layer], self.layers[x.layer].mixer.new_cache(self.layers[x.layer].mix), x.enters) for x in cfg.runs]
 
@@ -132,7 +135,8 @@ class StackRunner(RunnerBase):
         self.y2 = torch.zeros(n, self.wp, dtype=torch.float32, device=dev)
         self.hl = torch.zeros(self.max_batch, self.wp, dtype=dt, device=dev)
         self.x_loop = torch.zeros(n, 2 * self.wp, dtype=dt, device=dev) if self.loop_in is not None else None     # stream | embedding output
-        self._small = torch.zeros(n * max([lw.wsmall.shape[0] for lw in self.layers if lw.wsmall is not None], default=0), dtype=torch.float32, device=dev)
+        most = max([w.shape[0] for lw in self.layers for w in (lw.wsmall, lw.wsmall_ff) if w is not None], default=0)
+        self._small = torch.zeros(n * most, dtype=torch.float32, device=dev)
         for part in self.parts.values():
             part.allocate()
 
@@ -172,16 +176,27 @@ class StackRunner(RunnerBase):
                 lw.mixer.load_small(lw.mix, get, p + "mix.", lw.wsmall[:lw.mix_small])
             if lw.ff is not None:
                 lw.feed_forward.load(lw.ff, get, p + "mlp.")
-                if lw.wsmall is not None:
-                    lw.feed_forward.load_small(lw.ff, get, p + "mlp.", lw.wsmall[lw.mix_small:])
+                if lw.wsmall_ff is not None:
+                    lw.feed_forward.load_small(lw.ff, get, p + "mlp.", lw.wsmall_ff)
                 if not self.parallel:
                     norm_into(lw.norm2, p + "norm2", f32(p + "ls2"))
 
     # ------------------------------------------------------------------ layers
     def _small_rows(self, inp: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         """The narrow projections of ``inp``, fp32."""
-        T, n = inp.shape[0], w.shape[0]
-        return ops.gemm(inp, w, out=self._small[:T * n].view(T, n), out_f32=True)
+        return ops.gemm(inp, w, out=self._small_buffer(inp.shape[0], w), out_f32=True)
+
+    def _small_buffer(self, T: int, w: torch.Tensor) -> torch.Tensor:
+        return self._small[:T * w.shape[0]].view(T, w.shape[0])
+
+    def _project(self, lw: StackLayer, inp: torch.Tensor) -> torch.Tensor | None:
+        """The mixer's projections; returns the narrow fp32 one."""
+        if lw.wsmall is None or lw.mixer.fuses_tail:
+            small = self._small_buffer(inp.shape[0], lw.wsmall) if lw.wsmall is not None else None
+            lw.mixer.project(lw.mix, inp, small)
+            return small
+        lw.mixer.project(lw.mix, inp, None)
+        return self._small_rows(inp, lw.wsmall)
 
     def _layers(self, b: PackedBatch) -> None:
         """All layer runs over the batch's rows; leaves the residual stream in ``self.x``."""
@@ -214,7 +229,7 @@ class StackRunner(RunnerBase):
                     add = {}
                 self._enter_pass(T)
             ops.stream_norm(x, d, **add, weight=lw.norm1[0], eps=eps, h=h)
-            small = self._small_rows(h, lw.wsmall) if lw.wsmall is not None else None
+            small = self._project(lw, h)
             lw.mixer.forward(lw.mix, run.cache, h, y, b, plans[lw.mixer], small)
             add = {"y1": y}
             if lw.ff is not None:
@@ -231,11 +246,11 @@ class StackRunner(RunnerBase):
                 ops.stream_norm(x, d, copy=self.x_loop[:T, :self.wp])
                 self._enter_pass(T)
                 ops.stream_norm(x, d, copy=xb)
-            small = self._small_rows(xb, lw.wsmall[:lw.mix_small]) if lw.mix_small else None
+            small = self._project(lw, xb)
             lw.mixer.forward(lw.mix, run.cache, xb, y, b, plans[lw.mixer], small)
             ops.layernorm_residual(y, lw.norm1[0], lw.norm1[1], eps, x, xb, d)
             if lw.ff is not None:
-                small = self._small_rows(xb, lw.wsmall[lw.mix_small:]) if lw.wsmall is not None and lw.wsmall.shape[0] > lw.mix_small else None
+                small = self._small_rows(xb, lw.wsmall_ff) if lw.wsmall_ff is not None else None
                 add = lw.feed_forward.forward(lw.ff, xb, y, small)
                 if "experts" in add:
                     y.zero_()

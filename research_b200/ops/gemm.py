@@ -95,6 +95,10 @@ class RbGemmArgs(ctypes.Structure):
         ("glu_kind", ctypes.c_int),
         ("glu_limit", ctypes.c_float),
         ("softcap", ctypes.c_float),
+        ("silu_cols", ctypes.c_int),
+        ("tail_col", ctypes.c_int),
+        ("tail", ctypes.c_void_p),
+        ("tail_ld", ctypes.c_longlong),
     ]
 
 
@@ -113,7 +117,7 @@ def _lib2() -> ctypes.CDLL:
     lib = _native.load("rb_gemm2")
     if not getattr(lib, "_rb_typed", False):
         vp, i, ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
-        lib.rb_gemm2_bf16.argtypes = [vp] * 5 + [i, i, i, ll, ll, ll, ll, i, i, i, i, vp, vp]
+        lib.rb_gemm2_bf16.argtypes = [vp] * 5 + [i, i, i, ll, ll, ll, ll, i, i, i, i, i, vp, i, ll, vp, vp]
         lib.rb_gemm2_bf16.restype = i
         lib.rb_gemm2_pairs.restype = i
         lib.rb_gemm2_bf16_gather.argtypes = ([vp] * 5 + [i, i, i, ll, ll, ll, ll, i, i, i] +
@@ -141,21 +145,22 @@ def _use_pair_kernel(M: int, N: int, K: int, a_mn_major: bool, b_mn_major: bool)
 
 
 def gemm2(a: torch.Tensor, b: torch.Tensor, bias=None, residual=None, out=None, *, a_mn_major=False, b_mn_major=False,
-          out_f32=False, bn: int = 0) -> torch.Tensor:
+          out_f32=False, bn: int = 0, silu_cols: int = 0, tail: torch.Tensor | None = None) -> torch.Tensor:
     """``C = op(A) @ op(B)^T (+bias) (+residual)`` on the two-CTA (``cta_group::2``) kernel; same operand conventions
-    as ``gemm``. ``bn``: 256 or 128 output columns per tile (0 = fewest waves)."""
+    as ``gemm`` (``silu_cols`` and ``tail`` too). ``bn``: 256 or 128 output columns per tile (0 = fewest waves)."""
     assert a.is_cuda and a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16 and a.dim() == 2 and b.dim() == 2
     assert a.stride(1) == 1 and b.stride(1) == 1
     K, M = a.shape if a_mn_major else a.shape[::-1]
     Kb, N = b.shape if b_mn_major else b.shape[::-1]
     assert K == Kb, f"K mismatch: {K} vs {Kb}"
     if out is None:
-        out = torch.empty(M, N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=a.device)
+        out = torch.empty(M, N - (tail.shape[1] if tail is not None else 0), dtype=torch.float32 if out_f32 else torch.bfloat16, device=a.device)
     assert out.stride(1) == 1 and (residual is None or residual.stride(1) == 1)
     rc = _lib2().rb_gemm2_bf16(a.data_ptr(), b.data_ptr(), out.data_ptr(), bias.data_ptr() if bias is not None else None,
                                residual.data_ptr() if residual is not None else None, M, N, K, a.stride(0), b.stride(0),
                                out.stride(0), residual.stride(0) if residual is not None else 0, int(a_mn_major),
-                               int(b_mn_major), int(out_f32), bn, status_tensor(a.device).data_ptr(), stream_handle(a.device))
+                               int(b_mn_major), int(out_f32), bn, silu_cols, tail.data_ptr() if tail is not None else None,
+                               N - tail.shape[1] if tail is not None else 0, tail.stride(0) if tail is not None else 0, status_tensor(a.device).data_ptr(), stream_handle(a.device))
     check_rc(rc, "rb_gemm2_bf16")
     return out
 
@@ -181,7 +186,7 @@ def _lib_f32() -> ctypes.CDLL:
     lib = _native.load("rb_gemm_f32")
     if not getattr(lib, "_rb_typed", False):
         vp, i, ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
-        lib.rb_gemm_f32.argtypes = [vp] * 4 + [i] * 3 + [ll] * 3 + [i] + [ll] * 3 + [i, vp]
+        lib.rb_gemm_f32.argtypes = [vp] * 4 + [i] * 3 + [ll] * 3 + [i] + [ll] * 3 + [i, i, vp]
         lib.rb_gemm_f32_grouped.argtypes = [vp] * 3 + [i] + [ll] * 3 + [vp, vp, i, i, vp, vp]
         lib.rb_gemm_f32.restype = lib.rb_gemm_f32_grouped.restype = i
         lib._rb_typed = True
@@ -189,20 +194,21 @@ def _lib_f32() -> ctypes.CDLL:
 
 
 def gemm_f32_batched(a, b, out, M: int, N: int, K: int, batch: int, ld: tuple[int, int, int], step: tuple[int, int, int], b_kn: bool = False,
-                     bias=None) -> None:
+                     bias=None, silu_cols: int = 0) -> None:
     """``batch`` fp32 products ``C = A B^T (+ bias)`` (``b_kn``: ``A B``) at the given leading dimensions and batch strides."""
     assert a.dtype == b.dtype == out.dtype == torch.float32 and a.is_cuda
-    rc = _lib_f32().rb_gemm_f32(a.data_ptr(), b.data_ptr(), out.data_ptr(), bias.data_ptr() if bias is not None else None, M, N, K, *ld, batch, *step, int(b_kn), stream_handle(a.device))
+    rc = _lib_f32().rb_gemm_f32(a.data_ptr(), b.data_ptr(), out.data_ptr(), bias.data_ptr() if bias is not None else None, M, N, K, *ld, batch, *step, int(b_kn), silu_cols, stream_handle(a.device))
     check_rc(rc, "rb_gemm_f32")
 
 
-def gemm_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> torch.Tensor:
+def gemm_f32(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor | None = None, bias: torch.Tensor | None = None,
+             silu_cols: int = 0) -> torch.Tensor:
     """``A @ B^T`` with fp32 operands, products and sums (no reduced-precision matrix mode)."""
     assert a.dim() == b.dim() == 2 and a.stride(1) == b.stride(1) == 1 and a.shape[1] == b.shape[1]
     M, N = a.shape[0], b.shape[0]
     if out is None:
         out = torch.empty(M, N, dtype=torch.float32, device=a.device)
-    gemm_f32_batched(a, b, out, M, N, a.shape[1], 1, (a.stride(0), b.stride(0), out.stride(0)), (0, 0, 0), bias=bias)
+    gemm_f32_batched(a, b, out, M, N, a.shape[1], 1, (a.stride(0), b.stride(0), out.stride(0)), (0, 0, 0), bias=bias, silu_cols=silu_cols)
     return out
 
 
@@ -241,6 +247,8 @@ def gemm(
     wait_flag: tuple[int, int] | None = None,
     glu_limit: float | None = None,
     softcap: float = 0.0,
+    silu_cols: int = 0,
+    tail: torch.Tensor | None = None,
 ) -> torch.Tensor:
     """``C[M,N] = alpha * op(A) @ op(B)^T (+bias) (+ beta * residual)``.
 
@@ -259,7 +267,8 @@ def gemm(
     beforehand this equals ``rmsnorm(A) @ B^T`` without a separate normalisation pass.
 
     ``glu_limit`` makes the fused gate|up epilogue (``swiglu=True``) the clamped unit of ``elementwise.clamped_glu``;
-    ``softcap`` stores ``softcap * tanh(C / softcap)``.
+    ``softcap`` stores ``softcap * tanh(C / softcap)``. ``silu_cols``: the first so many columns are stored as ``silu(C)``.
+    ``tail`` (fp32 ``[M, n]``) receives the last ``n`` columns of the product, which ``out`` then lacks.
 
     K-major operands are ``[rows, K]`` row-major (a torch ``Linear`` weight is a K-major B);
     MN-major operands are ``[K, rows]`` row-major. On CUDA this launches the tcgen05 kernel;
@@ -293,13 +302,22 @@ def gemm(
             res = swiglu_interleaved_reference(res, bn, glu_limit)
         if softcap > 0:
             res = softcap * torch.tanh(res / softcap)
+        if silu_cols > 0:
+            res[:, :silu_cols] = torch.nn.functional.silu(res[:, :silu_cols].float()).to(res.dtype)
+        if tail is not None:
+            tail.copy_(res[:, -tail.shape[1]:])
+            res = res[:, :-tail.shape[1]]
         if out is not None:
             out.copy_(res)
             return out
         return res
     if a.dtype == torch.float32 and b is not None and b.dtype == torch.float32:
         assert residual is None and (bias is None or bias.dtype == torch.float32) and not (a_mn_major or b_mn_major or swiglu) and norm_eps is None and alpha == beta == 1.0
-        return gemm_f32(a, b, out, bias)
+        if tail is None:
+            return gemm_f32(a, b, out, bias, silu_cols)
+        n = b.shape[0] - tail.shape[1]
+        gemm_f32(a, b[n:], tail, bias[n:] if bias is not None else None)
+        return gemm_f32(a, b[:n], out, bias, silu_cols)
     if b_gather is not None:
         b = b_gather.staged          # [rows, cols] view of the staging matrix this launch fills
     assert a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16
@@ -320,14 +338,17 @@ def gemm(
         split_k, cluster_split = 1, False
     if (gather is None and softcap == 0 and wait_flag is None and not swiglu and norm_eps is None and alpha == 1.0 and beta == 1.0 and bn == 0 and max_ctas == 0 and split_k in (0, 1)
             and not cluster_split and _use_pair_kernel(M, N, K, a_mn_major, b_mn_major)):
-        return gemm2(a, b, bias, residual, out, a_mn_major=a_mn_major, b_mn_major=b_mn_major, out_f32=out_f32)
+        return gemm2(a, b, bias, residual, out, a_mn_major=a_mn_major, b_mn_major=b_mn_major, out_f32=out_f32, silu_cols=silu_cols, tail=tail)
+    if silu_cols or tail is not None:
+        assert gather is None and wait_flag is None and not swiglu and norm_eps is None and alpha == beta == 1.0 and not out_f32 and softcap == 0, \
+            "silu_cols and tail belong to a plain store"
     if (gather is not None and _GEMM2_GATHER and wait_flag is None and not swiglu and norm_eps is None and alpha == 1.0 and beta == 1.0
             and bn == 0 and max_ctas == 0 and split_k in (0, 1) and not cluster_split and a_mn_major == b_mn_major
             and _use_pair_kernel(M, N, K, a_mn_major, b_mn_major)
             and (b_gather is None or (N % gather.world == 0 and (N // gather.world) % 256 == 0))):
         return _gemm2_gather(a, b, bias, residual, out, M, N, K, a_mn_major, out_f32, gather, b_gather is not None)
     if out is None:
-        out = torch.empty(M, N // 2 if swiglu else N, dtype=torch.float32 if out_f32 else torch.bfloat16, device=a.device)
+        out = torch.empty(M, N // 2 if swiglu else N - (tail.shape[1] if tail is not None else 0), dtype=torch.float32 if out_f32 else torch.bfloat16, device=a.device)
     assert out.stride(1) == 1
     args = RbGemmArgs()
     args.A[0] = a.data_ptr()
@@ -349,6 +370,10 @@ def gemm(
     if glu_limit is not None:
         args.glu_kind, args.glu_limit = 1, float(glu_limit)
     args.softcap = float(softcap)
+    args.silu_cols = silu_cols
+    if tail is not None:
+        assert tail.dtype == torch.float32 and tail.stride(1) == 1
+        args.tail, args.tail_col, args.tail_ld = tail.data_ptr(), N - tail.shape[1], tail.stride(0)
     if norm_eps is not None:
         args.norm_fold, args.norm_eps = 1, float(norm_eps)
     if gather is not None:

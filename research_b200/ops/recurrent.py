@@ -4,7 +4,7 @@ Both kinds write ``k v^T`` into a state that decays and read it with ``q``::
 
     S_t = a_t S_(t-1) + b_t k_t v_t^T          o_t = S_t^T q_t
 
-* lightning: ``a`` is a constant of the head, ``b = 1``; queries, keys and values pass through SiLU;
+* lightning: ``a`` is a constant of the head, ``b = 1`` (queries, keys and values come through SiLU, applied by the projection);
 * matrix memory (mLSTM): capped gate logits ``i``, ``f``; ``log a = logsigmoid(f)``, ``b = exp(i)``, held relative to a running
   maximum ``m`` (from 0) so that nothing overflows; a second state ``n`` takes ``k`` alone and divides the output by
   ``max(|n . q|, exp(-m)) + 1e-6``.
@@ -41,7 +41,7 @@ class RecurrentGeometry:
     heads: int
     dim: int
     vdim: int
-    silu: bool                   # on q, k, v
+    silu: bool                   # q, k and v come through SiLU (the projection applies it)
     gated: bool                  # mLSTM gates and normaliser (otherwise a constant decay)
 
     @property
@@ -66,6 +66,10 @@ class RecurrentGeometry:
         return 0, a, 2 * a, 2 * a + b
 
     @property
+    def silu_cols(self) -> int:          # columns of the joint projection that are activated
+        return self.offsets[3] if self.silu else 0
+
+    @property
     def state_floats(self) -> int:       # one sequence
         return self.heads * self.tiles * (self.kp * (STATE_COLS + 1) + 1)
 
@@ -88,9 +92,9 @@ def _lib() -> ctypes.CDLL:
     lib = _native.load("rb_recurrent")
     if not getattr(lib, "_rb_typed", False):
         lib.rb_recurrent_scan.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float, c_float] + [c_vp] * 6
-                                          + [c_vp, c_ll] + [c_int] * 10 + [c_vp, c_vp])
+                                          + [c_vp, c_ll] + [c_int] * 9 + [c_vp, c_vp])
         lib.rb_recurrent_chunks.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float, c_float] + [c_vp] * 9 + [c_ll, c_vp]
-                                            + [c_int] * 9 + [c_vp, c_vp])
+                                            + [c_int] * 8 + [c_vp, c_vp])
         lib.rb_recurrent_chunk_workspace.argtypes, lib.rb_recurrent_chunk_workspace.restype = [c_int] * 4, c_ll
         lib.rb_gated_norm.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_ll] + [c_int] * 6 + [c_float, c_vp]
         for f in ("rb_recurrent_scan", "rb_recurrent_chunks", "rb_gated_norm"):
@@ -111,14 +115,13 @@ def _split(proj, geo: RecurrentGeometry):
     T, (oq, ok, ov, og) = proj.shape[0], geo.offsets
     q, k, v = proj[:, oq:ok], proj[:, ok:ov], proj[:, ov:og]
     q, k, v = (t.float().reshape(T, geo.heads, -1) for t in (q, k, v))
-    if geo.silu:
-        q, k, v = (torch.nn.functional.silu(t) for t in (q, k, v))
     return q * (geo.dim ** -0.5 if geo.gated else 1.0), k, v
 
 
 def recurrent_scan(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, cap: float, state: RecurrentState, slots, cu_q, seq_lens,
-                   out, rows: int, n_seq: int) -> None:
-    """Token-by-token form for the first ``n_seq`` sequences (``rows`` packed tokens): ``out [T, H*vp]`` fp32, state updated.
+                   out, rows: int, n_seq: int, first: int = 0) -> None:
+    """Token-by-token form for the sequences ``first .. n_seq - 1`` (the last one ends at packed row ``rows``): ``out [T, H*vp]``
+    fp32, state updated.
 
     ``proj [T, q | k | v | gate]``, ``small [T, i | f]`` fp32 (gated kinds), ``slots [B]`` (negative: padding), ``cu_q``
     ``[B+1]`` (None: one row per sequence), ``seq_lens [B]`` with the new tokens."""
@@ -127,7 +130,7 @@ def recurrent_scan(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, c
         q, k, v = _split(proj[:rows], geo)
         if geo.gated:
             gi, gf = capped_gates(small[:rows], bias_i, bias_f, cap)
-        for b in range(n_seq):
+        for b in range(first, n_seq):
             t0, t1 = (b, b + 1) if cu_q is None else (int(cu_q[b]), int(cu_q[b + 1]))
             slot = int(slots[b])
             if slot < 0:
@@ -155,11 +158,12 @@ def recurrent_scan(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, c
             state.n[slot], state.m[slot] = n[:, None], m[:, None]
         return
     oq, ok, ov, _ = geo.offsets
-    assert proj.stride(1) == 1 and out.dtype == torch.float32 and out.stride(1) == 1 and geo.kp <= MAX_DIM
+    assert proj.stride(1) == 1 and out.dtype == torch.float32 and out.stride(1) == 1 and (cu_q is not None or first == 0) and geo.kp <= MAX_DIM
     rc = _lib().rb_recurrent_scan(ptr(proj), proj.stride(0), oq, ok, ov, ptr(small), small.stride(0) if small is not None else 0, ptr(decay),
                                   ptr(bias_i), ptr(bias_f), cap, geo.dim ** -0.5 if geo.gated else 1.0, ptr(state.s), ptr(state.n), ptr(state.m),
-                                  ptr(slots), ptr(cu_q), ptr(seq_lens), ptr(out), out.stride(0), H, geo.dim, KP, VP, n_seq, state.s.shape[0],
-                                  int(geo.silu), int(geo.gated), rows, _DT[proj.dtype], ptr(status_tensor(proj.device)),
+                                  ptr(slots[first:]), ptr(cu_q[first:]) if cu_q is not None else None, ptr(seq_lens[first:]), ptr(out), out.stride(0), H, geo.dim, KP, VP,
+                                  n_seq - first, state.s.shape[0],
+                                  int(geo.gated), rows, _DT[proj.dtype], ptr(status_tensor(proj.device)),
                                   stream_handle(proj.device))
     check_rc(rc, "rb_recurrent_scan")
 
@@ -200,9 +204,8 @@ def recurrent_chunks(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f,
     rc = _lib().rb_recurrent_chunks(ptr(proj), proj.stride(0), 0, ok, ov, ptr(small), small.stride(0) if small is not None else 0, ptr(decay), ptr(bias_i),
                                     ptr(bias_f), cap, geo.dim ** -0.5 if geo.gated else 1.0, ptr(state.s), ptr(state.n), ptr(state.m),
                                     ptr(table.chunks), ptr(table.seq_chunks), ptr(slots[f:]), ptr(cu_q[f:]), ptr(seq_lens[f:]), ptr(out),
-                                    out.stride(0), ptr(workspace), n, B, geo.heads, geo.dim, geo.kp, geo.vp, state.s.shape[0], int(geo.silu),
-                                    int(geo.gated), ptr(status_tensor(proj.device)), stream_handle(proj.device))
-    check_rc(rc, "rb_recurrent_chunks", 3)
+                                    out.stride(0), ptr(workspace), n, B, geo.heads, geo.dim, geo.kp, geo.vp, state.s.shape[0], int(geo.gated), ptr(status_tensor(proj.device)), stream_handle(proj.device))
+    check_rc(rc, "rb_recurrent_chunks", 4)
 
 
 def chunk_workspace(n_chunks: int, geo: RecurrentGeometry) -> int:

@@ -257,7 +257,7 @@ def expert_stack_kernels(eng: InferenceEngine, T: int, context: int, decode: boo
         seen.add(kind)
         g, plan = w.geo, part.plan(b)
         proj = part.proj[:T * g.proj].view(T, g.proj)
-        t.gemm(f"{kind}: joint projection", T, g.proj, r.wp, lambda: ops.gemm(h, w.wproj, bias=getattr(w, "bproj", None), out=proj))
+        t.gemm(f"{kind}: joint projection", T, w.wproj.shape[0], r.wp, lambda: r._project(lw, h))
         if kind == "attention":
             H, G, D, m = g.heads, g.kv_heads, g.dp, w.spec
             out = part.out[:T * H * D].view(T, H * D)
@@ -273,7 +273,7 @@ def expert_stack_kernels(eng: InferenceEngine, T: int, context: int, decode: boo
         else:
             H, n = g.heads, g.heads * g.vp
             o, out = part.o[:T * n].view(T, n), part.out[:T * n].view(T, n)
-            small = r._small_rows(h, lw.wsmall)
+            small = r._project(lw, h)
             io = T * H * (2 * (2 * g.kp + g.vp) + 4 * g.vp)
             state = 2 * 4 * H * g.kp * (g.vp + (1 if g.gated else 0))
             t.add(f"{kind}: recurrence", lambda: part.recur(w, run.cache, proj, small, o, b, plan), io + state * b.rows,
@@ -281,8 +281,7 @@ def expert_stack_kernels(eng: InferenceEngine, T: int, context: int, decode: boo
             t.add(f"{kind}: norm + gate", lambda: ops.gated_norm(o, w.norm, proj[:, g.offsets[3]:], g, eps, out, g.gated), T * n * 8, 0)
         t.gemm(f"{kind}: output projection", T, r.wp, n, lambda: ops.gemm(out, w.wo, bias=getattr(w, "bo", None), out=y, out_f32=True), 4)
     lw = r.layers[0]
-    t.gemm("gate logits + router", T, lw.wsmall.shape[0], r.wp, lambda: r._small_rows(h, lw.wsmall), 4)
-    logits = r._small_rows(h, lw.wsmall)[:, lw.mix_small:]
+    logits = r._project(lw, h)[:, lw.mix_small:]
     w, g = lw.ff, lw.ff.geo
     sc = lw.feed_forward.scratch[g]
     _routed(t, T, g.experts, g.top, d, g.ff, lambda: ex.experts_up(g, sc, w.wgu, T), lambda: ex.experts_down(g, sc, w.wd), None,
