@@ -186,6 +186,7 @@ static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
 // directions, the update in shared memory. The unit's vectors are fetched one unit ahead.
 // ------------------------------------------------------------------------------------------
 constexpr int RD_THREADS = 128, RD_STAGES = 3, RD_VEC = 3;
+constexpr int RD_MAX_B = 4096;
 constexpr int RD_MAX_DK = 384;                    // key rows: a ring of larger tiles does not fit
 
 __device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
@@ -198,8 +199,8 @@ __device__ __forceinline__ void bulk_store(void* dst, uint32_t src, uint32_t byt
 }
 
 template <typename T>
-__global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const ScanParams p, int units) {
-  extern __shared__ __align__(128) uint8_t smem_raw[];       // RD_STAGES x [dk, 32] fp32
+__global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const ScanParams p, int B, int units) {
+  extern __shared__ __align__(128) uint8_t smem_raw[];       // RD_STAGES x [dk, 32] fp32, then the sequences' slots
   __shared__ float qs[RD_MAX_DK], ks[RD_MAX_DK];
   __shared__ __align__(16) float vs[SC_COLS];
   __shared__ __align__(16) float red[RD_THREADS / 32][SC_COLS];
@@ -217,14 +218,22 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
   __syncthreads();
   pdl_launch_dependents();
   pdl_wait();
-  struct Unit { int b, h, tile, slot; };
+  int* slots = reinterpret_cast<int*>(smem_raw + RD_STAGES * tile_bytes);      // -1: padding; bit 30: starts from zero
+  for (int b = tid; b < B; b += RD_THREADS) {
+    int s = p.slots[b];
+    if (s >= p.num_slots) { set_status(p.status, ST_BAD_INDEX); s = -1; }
+    slots[b] = s < 0 ? -1 : s | (p.seq_lens[b] == 1 ? 1 << 30 : 0);
+  }
+  __syncthreads();
+  struct Unit { int b, h, tile, slot; bool fresh; };
   auto unit_of = [&](int u) {
     Unit x;
     x.tile = u % tiles;
     x.h = (u / tiles) % p.H;
     x.b = u / tiles / p.H;
-    x.slot = p.slots[x.b];
-    if (x.slot >= p.num_slots) { set_status(p.status, ST_BAD_INDEX); x.slot = -1; }
+    const int s = slots[x.b];
+    x.fresh = s >= 0 && (s >> 30) != 0;
+    x.slot = s < 0 ? -1 : s & ((1 << 30) - 1);
     return x;
   };
   auto state_index = [&](const Unit& x) { return ((long long)max(x.slot, 0) * p.H + x.h) * tiles + x.tile; };   // padding rows read slot 0
@@ -242,10 +251,8 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
     for (int i = 0; i < RD_STAGES - 1; ++i) load(i);
   float q[RD_VEC], k[RD_VEC], n[RD_VEC], v = 0.f, gi = 0.f, gf = 0.f, m0 = 0.f;
   Unit x{};
-  bool fresh = false;
   auto fetch = [&](int u) {
     x = unit_of(u);
-    fresh = p.seq_lens[x.b] == 1;
     const T* row = reinterpret_cast<const T*>(p.proj) + x.b * p.ld;
     const float* nt = p.n + state_index(x) * p.KP;
 #pragma unroll
@@ -255,14 +262,14 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
       if (r < p.dk) {
         q[i] = to_f<T>(row[p.q_col + x.h * p.KP + r]) * p.q_scale;
         k[i] = to_f<T>(row[p.k_col + x.h * p.KP + r]);
-        if (p.gated && !fresh) n[i] = nt[r];
+        if (p.gated) n[i] = nt[r];
       }
     }
     if (tid < SC_COLS) v = to_f<T>(row[p.v_col + x.h * p.VP + x.tile * SC_COLS + tid]);
     if (p.gated) {
       gi = p.small[x.b * p.ld_small + x.h];
       gf = p.small[x.b * p.ld_small + p.H + x.h];
-      m0 = fresh ? 0.f : p.m[state_index(x)];
+      m0 = p.m[state_index(x)];
     }
   };
   if ((int)blockIdx.x < units) fetch(blockIdx.x);
@@ -270,7 +277,8 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
   int it = 0;
   for (int u = blockIdx.x; u < units; u += gridDim.x, ++it) {
     const Unit cur = x;
-    const bool zero = fresh;
+    const bool zero = cur.fresh;
+    if (zero) m0 = n[0] = n[1] = n[2] = 0.f;
     float a, w = 1.f, m = 0.f;
     if (p.gated) {
       gi = p.cap * tanhf((gi + p.bias_i[cur.h]) / p.cap);
@@ -299,12 +307,11 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
     }
     if (tid < SC_COLS) vs[tid] = v;
     if (p.gated && tid == 0 && cur.slot >= 0) p.m[si] = m;
-    __syncthreads();
-    if (u + (int)gridDim.x < units) fetch(u + gridDim.x);
     const int stage = it % RD_STAGES;
     ok = mbar_wait_bounded(smem_u32(&full[stage]), (uint32_t)((it / RD_STAGES) & 1), &abort_flag, p.status, ST_TIMEOUT_SMEM_FULL);
     ok = __syncthreads_and(ok);
     if (!ok) break;
+    if (u + (int)gridDim.x < units) fetch(u + gridDim.x);
     float4* S = reinterpret_cast<float4*>(smem_raw + stage * tile_bytes);
     const float4 vv = *reinterpret_cast<const float4*>(&vs[c4 * 4]);
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -364,17 +371,17 @@ static int launch_decode(const ScanParams& p, int B, cudaStream_t stream) {
   static int sms[64] = {};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
-  const int smem = RD_STAGES * p.dk * SC_COLS * 4;
+  const int smem = RD_STAGES * p.dk * SC_COLS * 4 + B * 4;
   if (sms[dev] == 0) {
     int n = 0;
     if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess ||
-        cudaFuncSetAttribute(recurrent_decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, RD_STAGES * RD_MAX_DK * SC_COLS * 4) != cudaSuccess)
+        cudaFuncSetAttribute(recurrent_decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, RD_STAGES * RD_MAX_DK * SC_COLS * 4 + RD_MAX_B * 4) != cudaSuccess)
       return -10;
     sms[dev] = n;
   }
   const int per_sm = 200 * 1024 / (smem + 7 * 1024) > 6 ? 6 : 200 * 1024 / (smem + 7 * 1024);
   const int units = B * p.H * (p.VP / SC_COLS), grid = units < sms[dev] * per_sm ? units : sms[dev] * per_sm;
-  return launch_kernel(recurrent_decode_kernel<T>, dim3(grid), dim3(RD_THREADS), smem, stream, p, units) == cudaSuccess ? 0 : -11;
+  return launch_kernel(recurrent_decode_kernel<T>, dim3(grid), dim3(RD_THREADS), smem, stream, p, B, units) == cudaSuccess ? 0 : -11;
 }
 
 // ------------------------------------------------------------------------------------------
@@ -442,17 +449,21 @@ __device__ __forceinline__ float2 chunk_gates(const ChunkParams& p, int h, int r
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     const int t = lane * 4 + i;
-    lf[i] = 0.f;
-    li[i] = 0.f;
-    if (t < n) {
-      if (p.gated) {
-        const float* g = p.small + (long long)(row0 + t) * p.ld_small;
-        li[i] = p.cap * tanhf((g[h] + p.bias_i[h]) / p.cap) * LOG2E;
-        lf[i] = log_sigmoid_f(p.cap * tanhf((g[p.H + h] + p.bias_f[h]) / p.cap)) * LOG2E;
-      } else {
-        lf[i] = logf(fmaxf(p.decay[h], 1e-30f)) * LOG2E;
-      }
+    const float* g = p.small + (long long)(row0 + min(t, n - 1)) * p.ld_small;
+    li[i] = p.gated ? g[h] : 0.f;
+    lf[i] = p.gated ? g[p.H + h] : 0.f;
+  }
+  const float bias_i = p.gated ? p.bias_i[h] : 0.f, bias_f = p.gated ? p.bias_f[h] : 0.f;
+  const float fixed = p.gated ? 0.f : logf(fmaxf(p.decay[h], 1e-30f)) * LOG2E;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    if (p.gated) {
+      li[i] = p.cap * tanhf((li[i] + bias_i) / p.cap) * LOG2E;
+      lf[i] = log_sigmoid_f(p.cap * tanhf((lf[i] + bias_f) / p.cap)) * LOG2E;
+    } else {
+      lf[i] = fixed;
     }
+    if (lane * 4 + i >= n) lf[i] = 0.f;
     run += lf[i];
     F[i] = run;
   }
@@ -501,7 +512,7 @@ __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wai
 // [CH, DK] columns of a projection into swizzled chunks, asynchronously; rows past n are zero
 template <int DK>
 __device__ __forceinline__ void chunk_load(uint32_t dst, const __nv_bfloat16* src, long long ld, int n) {
-#pragma unroll
+#pragma unroll 4
   for (int i = threadIdx.x; i < CH * (DK / 8); i += CHT) {
     const int r = i / (DK / 8), u = i % (DK / 8);
     cp_async16(dst + (u >> 3) * CH_CHUNK + chunk_addr(r, u & 7), src + (r < n ? r : 0) * ld + u * 8, r < n);
@@ -522,28 +533,47 @@ __global__ void __launch_bounds__(256) recurrent_chunk_gates_kernel(const ChunkP
   if ((threadIdx.x & 31) == 0) p.um[ch] = make_float2(t.x, t.x + G);
 }
 
-// What a chunk adds to the state: U [KP, 64 value channels] of one head. blockIdx: chunk, head, 64 value channels.
+// A work unit of the two kernels below: 64 value channels of one head of one chunk. Persistent CTAs walk over the units, the
+// value channels of a head next to each other (they share its keys and queries in L2), and fetch a unit ahead.
+struct ChunkUnit {
+  int c, h, z, row0, n;
+  long long ch;
+};
+__device__ __forceinline__ ChunkUnit chunk_unit(const ChunkParams& p, int u) {
+  ChunkUnit x;
+  const int zs = p.VP / 64;
+  x.z = u % zs;
+  x.h = (u / zs) % p.H;
+  x.c = u / zs / p.H;
+  const int4 ck = p.chunks[x.c];
+  x.row0 = ck.x;
+  x.n = ck.y;
+  x.ch = (long long)x.c * p.H + x.h;
+  return x;
+}
+
+// What a chunk adds to the state: U [KP, 64 value channels].
 template <int DK>
 struct ChunkStateCfg {
   static constexpr int kKBytes = CH * DK * 2;
-  static constexpr int kSmem = 1024 + 2 * kKBytes + CH_CHUNK;
+  static constexpr int kSmem = 1024 + 2 * kKBytes + 2 * CH_CHUNK;      // weighted keys in two parts, two V tiles
   static constexpr int kCols = DK > 128 ? 128 : 64;
 };
 
 template <int DK>
-__global__ void __launch_bounds__(CHT) recurrent_chunk_state_kernel(const ChunkParams p) {
+__global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_state_kernel(const ChunkParams p, int units) {
   using Cfg = ChunkStateCfg<DK>;
+  constexpr int UNITS = CH * (DK / 8) / CHT;          // 16-byte pieces of K per thread
   extern __shared__ __align__(128) uint8_t smem_raw[];
   __shared__ float gs[CH], nred[4][DK];
   __shared__ __align__(8) uint64_t done;
   __shared__ uint32_t tmem_base_smem;
   __shared__ int abort_flag;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int c = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* hi = smem_raw + (base - smem_u32(smem_raw));
   uint8_t* lo = hi + Cfg::kKBytes;
-  if (threadIdx.x == 0) {
+  if (tid == 0) {
     abort_flag = 0;
     mbar_init(smem_u32(&done), 1);
     fence_mbar_init();
@@ -552,36 +582,44 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_state_kernel(const ChunkP
     tmem_alloc(smem_u32(&tmem_base_smem), Cfg::kCols);
     tmem_relinquish();
   }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_base_smem;
   pdl_launch_dependents();
   pdl_wait();
-  const int4 ck = p.chunks[c];
-  const int row0 = ck.x, n = ck.y;
-  const long long ch = (long long)c * p.H + h;
-  chunk_load<64>(base + 2 * Cfg::kKBytes, p.proj + row0 * p.ld + p.v_col + h * p.VP + z * 64, p.ld, n);
-  if (threadIdx.x < CH) {
-    const float2 t = p.um[ch];
-    gs[threadIdx.x] = chunk_exp2(p.gates[ch * 3 * CH + threadIdx.x] - (t.y - t.x));     // weights relative to exp(F_C + G)
-  }
-  const __nv_bfloat16* k = p.proj + row0 * p.ld + p.k_col + h * p.KP;
-  constexpr int UNITS = CH * (DK / 8) / CHT, BATCH = UNITS % 8 == 0 ? 8 : 4;
-  static_assert(UNITS % BATCH == 0, "whole batches");
-  __syncthreads();
-#pragma unroll 1
-  for (int i0 = 0; i0 < UNITS; i0 += BATCH) {
-    uint4 raw[BATCH];
+  uint4 raw[UNITS];
+  float weight = 0.f;
+  auto fetch = [&](const ChunkUnit& x, int buf) {
+    chunk_load<64>(base + 2 * Cfg::kKBytes + buf * CH_CHUNK, p.proj + x.row0 * p.ld + p.v_col + x.h * p.VP + x.z * 64, p.ld, x.n);
+    const __nv_bfloat16* k = p.proj + x.row0 * p.ld + p.k_col + x.h * p.KP;
 #pragma unroll
-    for (int i = 0; i < BATCH; ++i) {
-      const int e = threadIdx.x + (i0 + i) * CHT, r = e / (DK / 8), u = e % (DK / 8);
+    for (int i = 0; i < UNITS; ++i) {
+      const int e = tid + i * CHT, r = e / (DK / 8), u = e % (DK / 8);
       raw[i] = make_uint4(0u, 0u, 0u, 0u);
-      if (r < n) raw[i] = *reinterpret_cast<const uint4*>(k + r * p.ld + u * 8);
+      if (r < x.n) raw[i] = *reinterpret_cast<const uint4*>(k + r * p.ld + u * 8);
     }
+    if (tid < CH) {
+      const float2 t = p.um[x.ch];
+      weight = p.gates[x.ch * 3 * CH + tid] - (t.y - t.x);             // relative to exp(F_C + G)
+    }
+  };
+  ChunkUnit x{};
+  if ((int)blockIdx.x < units) { x = chunk_unit(p, blockIdx.x); fetch(x, 0); }
+  bool ok = true;
+  int it = 0;
+  for (int u = blockIdx.x; u < units; u += gridDim.x, ++it) {
+    const ChunkUnit cur = x;
+    if (tid < CH) gs[tid] = chunk_exp2(weight);
+    ok = __syncthreads_and(ok);                        // also: everyone is done with the unit before
+    if (!ok) break;
 #pragma unroll
-    for (int i = 0; i < BATCH; ++i) {
-      const int e = threadIdx.x + (i0 + i) * CHT, r = e / (DK / 8), u = e % (DK / 8);
+    for (int i = 0; i < UNITS; ++i) {
+      const int e = tid + i * CHT, r = e / (DK / 8), uu = e % (DK / 8);
       const float w = gs[r];
       uint4 a, b;
-      auto one = [&](uint32_t x, uint32_t& l) {
-        float2 f = unpack_bf16x2(x);
+      auto one = [&](uint32_t v, uint32_t& l) {
+        float2 f = unpack_bf16x2(v);
         f.x *= w; f.y *= w;
         const uint32_t o = pack_bf16x2(f.x, f.y);
         const float2 back = unpack_bf16x2(o);
@@ -589,75 +627,76 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_state_kernel(const ChunkP
         return o;
       };
       a.x = one(raw[i].x, b.x); a.y = one(raw[i].y, b.y); a.z = one(raw[i].z, b.z); a.w = one(raw[i].w, b.w);
-      const uint32_t at = (u >> 3) * CH_CHUNK + chunk_addr(r, u & 7);
+      const uint32_t at = (uu >> 3) * CH_CHUNK + chunk_addr(r, uu & 7);
       *reinterpret_cast<uint4*>(hi + at) = a;
       *reinterpret_cast<uint4*>(lo + at) = b;
     }
+    cp_async_wait_all();
+    fence_proxy_async_smem();
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (warp == 0 && elect_one_sync()) {
+      const uint32_t v_s = base + 2 * Cfg::kKBytes + (it & 1) * CH_CHUNK;
+#pragma unroll
+      for (int m0 = 0; m0 < DK; m0 += 128) {
+        const uint32_t idesc = make_idesc_bf16(DK - m0 >= 128 ? 128 : 64, 64, 1, 1);
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int kk = 0; kk < CH / 16; ++kk) {
+            const uint64_t a = make_smem_desc_sw128(base + part * Cfg::kKBytes + (m0 / 64) * CH_CHUNK + kk * 2048, CH_CHUNK, 1024);
+            const uint64_t b = make_smem_desc_sw128(v_s + kk * 2048, CH_CHUNK, 1024);
+            umma_bf16(tmem + (m0 / 128) * 64, a, b, idesc, (part | kk) ? 1u : 0u);
+          }
+      }
+      umma_commit(smem_u32(&done));
+    }
+    __syncwarp();
+    if (u + (int)gridDim.x < units) { x = chunk_unit(p, u + gridDim.x); fetch(x, (it + 1) & 1); }
+    if (p.gated && cur.z == 0) {       // the normaliser's part, while the tensor cores work: column sums of the weighted keys
+      constexpr int PAIRS = DK / 2, GROUPS = 4;
+      for (int i = tid; i < PAIRS * GROUPS; i += CHT) {
+        const int pr = i % PAIRS, g = i / PAIRS;
+        float sx = 0.f, sy = 0.f;
+#pragma unroll 8
+        for (int r = g * (CH / GROUPS); r < (g + 1) * (CH / GROUPS); ++r) {
+          const uint32_t at = (pr >> 5) * CH_CHUNK + chunk_addr(r, (pr & 31) >> 2) + (pr & 3) * 4;
+          const float2 a = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(hi + at)), b = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(lo + at));
+          sx += a.x + b.x;
+          sy += a.y + b.y;
+        }
+        nred[g][2 * pr] = sx;
+        nred[g][2 * pr + 1] = sy;
+      }
+      __syncthreads();
+      for (int i = tid; i < DK; i += CHT) p.un[cur.ch * p.KP + i] = (nred[0][i] + nred[1][i]) + (nred[2][i] + nred[3][i]);
+    }
+    ok = mbar_wait_bounded(smem_u32(&done), it & 1, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
+    ok = __all_sync(0xffffffffu, ok);
+    tc_fence_after();
+    if (ok) {
+      const int qd = warp & 3, half = warp >> 2;       // lanes of a TMEM quarter; the two warps of a quarter split the columns
+      float* dstu = p.u + (cur.ch * (p.VP / 32) + cur.z * 2 + half) * p.KP * 32;
+#pragma unroll
+      for (int m0 = 0; m0 < DK; m0 += 128) {
+        uint32_t v[32];
+        tmem_ld_32x32(tmem + (m0 / 128) * 64 + half * 32 + ((uint32_t)(qd * 32) << 16), v);
+        tmem_ld_wait();
+        // a 128-row product has row 32 q + lane in quarter q, a 64-row one row 16 q + lane in its first 16 lanes
+        const bool full = DK - m0 >= 128;
+        const int r = m0 + (full ? qd * 32 + lane : qd * 16 + lane);
+        if (full || lane < 16) {
+          float4* dst = reinterpret_cast<float4*>(dstu + (long long)r * 32);
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            dst[i] = make_float4(__uint_as_float(v[4 * i]), __uint_as_float(v[4 * i + 1]), __uint_as_float(v[4 * i + 2]), __uint_as_float(v[4 * i + 3]));
+        }
+      }
+      tc_fence_before();
+    }
   }
   cp_async_wait_all();
-  fence_proxy_async_smem();
-  tc_fence_before();
-  __syncthreads();
-  tc_fence_after();
-  const uint32_t tmem = tmem_base_smem;
-  if (warp == 0 && elect_one_sync()) {
-    const uint32_t v_s = base + 2 * Cfg::kKBytes;
-#pragma unroll
-    for (int m0 = 0; m0 < DK; m0 += 128) {
-      constexpr int kFull = 128;
-      const uint32_t idesc = make_idesc_bf16(DK - m0 >= kFull ? 128 : 64, 64, 1, 1);
-#pragma unroll
-      for (int part = 0; part < 2; ++part)
-#pragma unroll
-        for (int kk = 0; kk < CH / 16; ++kk) {
-          const uint64_t a = make_smem_desc_sw128(base + part * Cfg::kKBytes + (m0 / 64) * CH_CHUNK + kk * 2048, CH_CHUNK, 1024);
-          const uint64_t b = make_smem_desc_sw128(v_s + kk * 2048, CH_CHUNK, 1024);
-          umma_bf16(tmem + (m0 / 128) * 64, a, b, idesc, (part | kk) ? 1u : 0u);
-        }
-    }
-    umma_commit(smem_u32(&done));
-  }
-  if (p.gated && z == 0) {       // the normaliser's part, while the tensor cores work: column sums of the weighted keys
-    constexpr int PAIRS = DK / 2, GROUPS = 4;
-    for (int i = threadIdx.x; i < PAIRS * GROUPS; i += CHT) {
-      const int pr = i % PAIRS, g = i / PAIRS;
-      float sx = 0.f, sy = 0.f;
-      for (int r = g * (CH / GROUPS); r < (g + 1) * (CH / GROUPS); ++r) {
-        const uint32_t at = (pr >> 5) * CH_CHUNK + chunk_addr(r, (pr & 31) >> 2) + (pr & 3) * 4;
-        const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(hi + at)), y = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(lo + at));
-        sx += x.x + y.x;
-        sy += x.y + y.y;
-      }
-      nred[g][2 * pr] = sx;
-      nred[g][2 * pr + 1] = sy;
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < DK; i += CHT)
-      p.un[ch * p.KP + i] = (nred[0][i] + nred[1][i]) + (nred[2][i] + nred[3][i]);
-  }
-  bool ok = mbar_wait_bounded(smem_u32(&done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
-  ok = __all_sync(0xffffffffu, ok);
-  tc_fence_after();
-  if (ok) {
-    const int qd = warp & 3, half = warp >> 2;       // lanes of a TMEM quarter; the two warps of a quarter split the columns
-    float* u = p.u + (ch * (p.VP / 32) + z * 2 + half) * p.KP * 32;
-#pragma unroll
-    for (int m0 = 0; m0 < DK; m0 += 128) {
-      uint32_t v[32];
-      tmem_ld_32x32(tmem + (m0 / 128) * 64 + half * 32 + ((uint32_t)(qd * 32) << 16), v);
-      tmem_ld_wait();
-      // a 128-row product has row 32 q + lane in quarter q, a 64-row one row 16 q + lane in its first 16 lanes
-      const bool full = DK - m0 >= 128;
-      const int r = m0 + (full ? qd * 32 + lane : qd * 16 + lane);
-      if (full || lane < 16) {
-        float4* dst = reinterpret_cast<float4*>(u + (long long)r * 32);
-#pragma unroll
-        for (int i = 0; i < 8; ++i)
-          dst[i] = make_float4(__uint_as_float(v[4 * i]), __uint_as_float(v[4 * i + 1]), __uint_as_float(v[4 * i + 2]), __uint_as_float(v[4 * i + 3]));
-      }
-    }
-    tc_fence_before();
-  }
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
@@ -723,11 +762,11 @@ __global__ void __launch_bounds__(256) recurrent_chunk_chain_kernel(const ChunkP
         float a, w = 1.f;
         if (p.gated) {
           const float m_new = fmaxf(um[i].x + m, um[i].y);
-          a = exp2f(um[i].x + m - m_new);
-          w = exp2f(um[i].y - m_new);
+          a = chunk_exp2(um[i].x + m - m_new);
+          w = chunk_exp2(um[i].y - m_new);
           m = m_new;
         } else {
-          a = exp2f(um[i].x);
+          a = chunk_exp2(um[i].x);
         }
         S.x = fmaf(a, S.x, w * U[i].x);
         S.y = fmaf(a, S.y, w * U[i].y);
@@ -744,7 +783,7 @@ __global__ void __launch_bounds__(256) recurrent_chunk_chain_kernel(const ChunkP
   if (p.gated && r == 0 && c4 == 0) p.m[unit] = m / LOG2E;
 }
 
-// Outputs of a chunk: 64 value channels of one head. blockIdx: chunk, head, 64 value channels.
+// Outputs of a chunk.
 template <int DK>
 struct ChunkOutCfg {
   static constexpr int kQBytes = CH * DK * 2;
@@ -756,23 +795,22 @@ struct ChunkOutCfg {
 };
 
 template <int DK>
-__global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkParams p) {
+__global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_out_kernel(const ChunkParams p, int units) {
   using Cfg = ChunkOutCfg<DK>;
+  constexpr int VPT = CH * 8 / CHT;                  // 16-byte pieces of V per thread
   extern __shared__ __align__(128) uint8_t smem_raw[];
-  __shared__ float gs[CH], bs[CH], fs[CH], row_sum[2][CH];
-  __shared__ __align__(16) float ns[DK];
+  __shared__ __align__(16) float gs[CH], bs[CH], fs[CH], row_sum[2][CH], ns[DK];
   __shared__ float m_in;
   __shared__ __align__(8) uint64_t s_done, o_done;
   __shared__ uint32_t tmem_base_smem;
   __shared__ int abort_flag;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int c = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* q_p = smem_raw + (base - smem_u32(smem_raw));
   uint8_t* k_p = q_p + Cfg::kQBytes;
   uint8_t* sv_p = k_p + Cfg::kKpBytes;
   const uint32_t q_s = base, k_s = q_s + Cfg::kQBytes, sv_s = k_s + Cfg::kKpBytes, sl_s = sv_s + Cfg::kSvBytes;
-  if (threadIdx.x == 0) {
+  if (tid == 0) {
     abort_flag = 0;
     mbar_init(smem_u32(&s_done), 1);
     mbar_init(smem_u32(&o_done), 1);
@@ -782,146 +820,183 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkPar
     tmem_alloc(smem_u32(&tmem_base_smem), Cfg::kCols);
     tmem_relinquish();
   }
-  pdl_launch_dependents();
-  pdl_wait();
-  const int4 ck = p.chunks[c];
-  const int row0 = ck.x, n = ck.y;
-  const long long ch = (long long)c * p.H + h;
-  const __nv_bfloat16* rows = p.proj + row0 * p.ld;
-  chunk_load<DK>(q_s, rows + p.q_col + h * p.KP, p.ld, n);
-  chunk_load<DK>(k_s, rows + p.k_col + h * p.KP, p.ld, n);
-  {
-    const long long at = (ch * (p.VP / 64) + z) * p.KP * 64;
-#pragma unroll
-    for (int i = threadIdx.x; i < DK * 8; i += CHT) {
-      const uint32_t a = chunk_addr(i >> 3, i & 7);
-      cp_async16(sv_s + a, p.s_hi + at + i * 8, true);
-      cp_async16(sl_s + a, p.s_lo + at + i * 8, true);
-    }
-  }
-  if (threadIdx.x < CH) {
-    const float* g = p.gates + ch * 3 * CH + threadIdx.x;
-    gs[threadIdx.x] = g[0];
-    bs[threadIdx.x] = g[CH];
-    fs[threadIdx.x] = g[2 * CH];
-  }
-  if (threadIdx.x == CH) m_in = p.gated ? p.s_m[ch] : 0.f;
-  if (p.gated)
-    for (int i = threadIdx.x; i < DK; i += CHT) ns[i] = p.s_n[ch * p.KP + i];
-  uint4 vr[CH * 8 / CHT];                            // V waits in registers until the state's shared memory is free
-#pragma unroll
-  for (int i = 0; i < CH * 8 / CHT; ++i) {
-    const int e = threadIdx.x + i * CHT, r = e >> 3, u = e & 7;
-    vr[i] = make_uint4(0u, 0u, 0u, 0u);
-    if (r < n) vr[i] = *reinterpret_cast<const uint4*>(rows + r * p.ld + p.v_col + h * p.VP + z * 64 + u * 8);
-  }
-  cp_async_wait_all();
-  fence_proxy_async_smem();
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = tmem_base_smem, t_o = tmem + 128, t_s = tmem + 192;
-  if (warp == 0 && elect_one_sync()) {
-    constexpr uint32_t idesc_s = make_idesc_bf16(CH, CH, 0, 0), idesc_o = make_idesc_bf16(CH, 64, 0, 1);
+  pdl_launch_dependents();
+  pdl_wait();
+  // A unit's operands arrive in two parts, as the shared memory of the unit before becomes free; its vectors and V wait in
+  // registers.
+  float r_g = 0.f, r_b = 0.f, r_f = 0.f, r_n = 0.f, r_m = 0.f;
+  uint4 vr[VPT];
+  auto load_state = [&](uint32_t dst, const __nv_bfloat16* part, const ChunkUnit& x) {
+    const __nv_bfloat16* src = part + (x.ch * (p.VP / 64) + x.z) * p.KP * 64;
+#pragma unroll 4
+    for (int i = tid; i < DK * 8; i += CHT) cp_async16(dst + chunk_addr(i >> 3, i & 7), src + i * 8, true);
+  };
+  auto fetch_first = [&](const ChunkUnit& x) {       // Q, the state's second part, the vectors, V
+    const __nv_bfloat16* rows = p.proj + x.row0 * p.ld;
+    chunk_load<DK>(q_s, rows + p.q_col + x.h * p.KP, p.ld, x.n);
+    load_state(sl_s, p.s_lo, x);
 #pragma unroll
-    for (int kk = 0; kk < DK / 16; ++kk) {
-      const uint64_t a = make_smem_desc_sw128(q_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
-      const uint64_t b = make_smem_desc_sw128(k_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
-      umma_bf16(tmem, a, b, idesc_s, kk ? 1u : 0u);
+    for (int i = 0; i < VPT; ++i) {
+      const int e = tid + i * CHT, r = e >> 3;
+      vr[i] = make_uint4(0u, 0u, 0u, 0u);
+      if (r < x.n) vr[i] = *reinterpret_cast<const uint4*>(rows + r * p.ld + p.v_col + x.h * p.VP + x.z * 64 + (e & 7) * 8);
     }
-#pragma unroll
-    for (int part = 0; part < 2; ++part)
-#pragma unroll
-      for (int kk = 0; kk < DK / 16; ++kk) {
-        const uint64_t a = make_smem_desc_sw128(q_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
-        const uint64_t b = make_smem_desc_sw128((part ? sl_s : sv_s) + kk * 2048, CH_CHUNK, 1024);
-        umma_bf16(t_s, a, b, idesc_o, (part | kk) ? 1u : 0u);
-      }
-    umma_commit(smem_u32(&s_done));
+    if (tid < CH) {
+      const float* g = p.gates + x.ch * 3 * CH + tid;
+      r_g = g[0];
+      r_b = g[CH];
+      r_f = g[2 * CH];
+    }
+    if (p.gated) {
+      if (tid < DK) r_n = p.s_n[x.ch * p.KP + tid];
+      r_m = p.s_m[x.ch];
+    }
+  };
+  auto fetch_second = [&](const ChunkUnit& x) {      // K, the state's first part
+    chunk_load<DK>(k_s, p.proj + x.row0 * p.ld + p.k_col + x.h * p.KP, p.ld, x.n);
+    load_state(sv_s, p.s_hi, x);
+  };
+  ChunkUnit x{};
+  if ((int)blockIdx.x < units) {
+    x = chunk_unit(p, blockIdx.x);
+    fetch_first(x);
+    fetch_second(x);
   }
   const int qd = warp & 3, half = warp >> 2;
   const int t = qd * 32 + lane;                      // this thread's token; the two warps of a quarter split the columns
   const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
-  const float B = p.gated ? fmaxf(m_in, bs[t]) : bs[t];
-  float qn = 0.f;
-  if (p.gated) {                                     // half of q . n of the incoming state
-    constexpr int U = DK / 16;                       // 16-byte units per half
-#pragma unroll 4
-    for (int u = half * U; u < (half + 1) * U; ++u) {
-      const uint4 v = *reinterpret_cast<const uint4*>(q_p + (u >> 3) * CH_CHUNK + chunk_addr(t, u & 7));
-      const float* w = ns + u * 8;
-      float2 f;
-      f = unpack_bf16x2(v.x); qn = fmaf(f.x, w[0], fmaf(f.y, w[1], qn));
-      f = unpack_bf16x2(v.y); qn = fmaf(f.x, w[2], fmaf(f.y, w[3], qn));
-      f = unpack_bf16x2(v.z); qn = fmaf(f.x, w[4], fmaf(f.y, w[5], qn));
-      f = unpack_bf16x2(v.w); qn = fmaf(f.x, w[6], fmaf(f.y, w[7], qn));
-    }
-  }
-  const float c_in = chunk_exp2(m_in - B);
-  bool ok = mbar_wait_bounded(smem_u32(&s_done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
-  ok = __all_sync(0xffffffffu, ok);
-  tc_fence_after();
-  float sum = 0.f;
-  if (ok) {
-    uint8_t* prow = k_p + half * CH_CHUNK;           // K has been read
+  bool ok = true;
+  int it = 0;
+  for (int u = blockIdx.x; u < units; u += gridDim.x, ++it) {
+    const ChunkUnit cur = x;
+    if (tid < CH) { gs[tid] = r_g; bs[tid] = r_b; fs[tid] = r_f; }
+    if (p.gated && tid < DK) ns[tid] = r_n;
+    if (tid == 0) m_in = r_m;
+    cp_async_wait_all();
+    fence_proxy_async_smem();
+    tc_fence_before();
+    ok = __syncthreads_and(ok);
+    if (!ok) break;
+    tc_fence_after();
+    if (warp == 0 && elect_one_sync()) {
+      constexpr uint32_t idesc_s = make_idesc_bf16(CH, CH, 0, 0), idesc_o = make_idesc_bf16(CH, 64, 0, 1);
 #pragma unroll
-    for (int cc = 0; cc < 2; ++cc) {
-      uint32_t v[32];
-      tmem_ld_32x32(tmem + half * 64 + cc * 32 + lane_addr, v);
-      tmem_ld_wait();
-      float x[32];
-#pragma unroll
-      for (int i = 0; i < 32; ++i) {
-        const int j = half * 64 + cc * 32 + i;
-        x[i] = j <= t ? __uint_as_float(v[i]) * chunk_exp2(gs[j] - B) : 0.f;
-        sum += x[i];
+      for (int kk = 0; kk < DK / 16; ++kk) {
+        const uint64_t a = make_smem_desc_sw128(q_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+        const uint64_t b = make_smem_desc_sw128(k_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+        umma_bf16(tmem, a, b, idesc_s, kk ? 1u : 0u);
       }
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
-        *reinterpret_cast<uint4*>(prow + chunk_addr(t, cc * 4 + u)) =
-            make_uint4(pack_bf16x2(x[u * 8], x[u * 8 + 1]), pack_bf16x2(x[u * 8 + 2], x[u * 8 + 3]), pack_bf16x2(x[u * 8 + 4], x[u * 8 + 5]),
-                       pack_bf16x2(x[u * 8 + 6], x[u * 8 + 7]));
-    }
-    // V over the state's first part, which has been read too
+      for (int part = 0; part < 2; ++part)
 #pragma unroll
-    for (int i = 0; i < CH * 8 / CHT; ++i) {
-      const int e = threadIdx.x + i * CHT;
-      *reinterpret_cast<uint4*>(sv_p + chunk_addr(e >> 3, e & 7)) = vr[i];
+        for (int kk = 0; kk < DK / 16; ++kk) {
+          const uint64_t a = make_smem_desc_sw128(q_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+          const uint64_t b = make_smem_desc_sw128((part ? sl_s : sv_s) + kk * 2048, CH_CHUNK, 1024);
+          umma_bf16(t_s, a, b, idesc_o, (part | kk) ? 1u : 0u);
+        }
+      umma_commit(smem_u32(&s_done));
     }
-  }
-  row_sum[half][t] = sum + c_in * qn;
-  fence_proxy_async_smem();
-  tc_fence_before();
-  __syncthreads();
-  tc_fence_after();
-  if (ok && warp == 0 && elect_one_sync()) {
-    constexpr uint32_t idesc_o = make_idesc_bf16(CH, 64, 0, 1);
-#pragma unroll
-    for (int kk = 0; kk < CH / 16; ++kk) {
-      const uint64_t a = make_smem_desc_sw128(k_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
-      const uint64_t b = make_smem_desc_sw128(sv_s + kk * 2048, CH_CHUNK, 1024);
-      umma_bf16(t_o, a, b, idesc_o, kk ? 1u : 0u);
+    __syncwarp();
+    const bool more = u + (int)gridDim.x < units;
+    if (more) x = chunk_unit(p, u + gridDim.x);
+    const float B = p.gated ? fmaxf(m_in, bs[t]) : bs[t], F = fs[t];
+    float qn = 0.f;
+    if (p.gated) {                                   // half of q . n of the incoming state
+      constexpr int U = DK / 16;                     // 16-byte units per half
+#pragma unroll 4
+      for (int w = half * U; w < (half + 1) * U; ++w) {
+        const uint4 v = *reinterpret_cast<const uint4*>(q_p + (w >> 3) * CH_CHUNK + chunk_addr(t, w & 7));
+        const float4 n0 = *reinterpret_cast<const float4*>(ns + w * 8), n1 = *reinterpret_cast<const float4*>(ns + w * 8 + 4);
+        float2 f;
+        f = unpack_bf16x2(v.x); qn = fmaf(f.x, n0.x, fmaf(f.y, n0.y, qn));
+        f = unpack_bf16x2(v.y); qn = fmaf(f.x, n0.z, fmaf(f.y, n0.w, qn));
+        f = unpack_bf16x2(v.z); qn = fmaf(f.x, n1.x, fmaf(f.y, n1.y, qn));
+        f = unpack_bf16x2(v.w); qn = fmaf(f.x, n1.z, fmaf(f.y, n1.w, qn));
+      }
     }
-    umma_commit(smem_u32(&o_done));
-  }
-  if (ok) {
-    ok = mbar_wait_bounded(smem_u32(&o_done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
+    const float c_in = chunk_exp2(m_in - B);
+    ok = mbar_wait_bounded(smem_u32(&s_done), it & 1, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
     ok = __all_sync(0xffffffffu, ok);
-  }
-  tc_fence_after();
-  if (ok) {
-    float f = p.q_scale;
-    if (p.gated) {
-      const float nq = fabsf((row_sum[0][t] + row_sum[1][t]) * p.q_scale);
-      f /= fmaxf(nq, chunk_exp2(-(fs[t] + B))) + 1e-6f;
+    tc_fence_after();
+    float sum = 0.f;
+    if (ok) {
+      uint8_t* prow = k_p + half * CH_CHUNK;         // K has been read
+#pragma unroll
+      for (int cc = 0; cc < 2; ++cc) {
+        const int j0 = half * 64 + cc * 32;
+        float y[32];
+        if (j0 <= qd * 32 + 31) {                    // (uniform per warp: a block on the diagonal or below it)
+          uint32_t v[32];
+          tmem_ld_32x32(tmem + j0 + lane_addr, v);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) {
+            const float4 g = *reinterpret_cast<const float4*>(gs + j0 + i);
+            y[i] = __uint_as_float(v[i]) * chunk_exp2(g.x - B);
+            y[i + 1] = __uint_as_float(v[i + 1]) * chunk_exp2(g.y - B);
+            y[i + 2] = __uint_as_float(v[i + 2]) * chunk_exp2(g.z - B);
+            y[i + 3] = __uint_as_float(v[i + 3]) * chunk_exp2(g.w - B);
+          }
+          if (j0 + 31 > qd * 32) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (j0 + i > t) y[i] = 0.f;
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) y[i] = 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < 32; ++i) sum += y[i];
+#pragma unroll
+        for (int w = 0; w < 4; ++w)
+          *reinterpret_cast<uint4*>(prow + chunk_addr(t, cc * 4 + w)) =
+              make_uint4(pack_bf16x2(y[w * 8], y[w * 8 + 1]), pack_bf16x2(y[w * 8 + 2], y[w * 8 + 3]), pack_bf16x2(y[w * 8 + 4], y[w * 8 + 5]),
+                         pack_bf16x2(y[w * 8 + 6], y[w * 8 + 7]));
+      }
+      // V over the state's first part, which has been read too
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int e = tid + i * CHT;
+        *reinterpret_cast<uint4*>(sv_p + chunk_addr(e >> 3, e & 7)) = vr[i];
+      }
     }
+    row_sum[half][t] = sum + c_in * qn;
+    fence_proxy_async_smem();
+    tc_fence_before();
+    ok = __syncthreads_and(ok);
+    if (!ok) break;
+    tc_fence_after();
+    if (warp == 0 && elect_one_sync()) {
+      constexpr uint32_t idesc_o = make_idesc_bf16(CH, 64, 0, 1);
+#pragma unroll
+      for (int kk = 0; kk < CH / 16; ++kk) {
+        const uint64_t a = make_smem_desc_sw128(k_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+        const uint64_t b = make_smem_desc_sw128(sv_s + kk * 2048, CH_CHUNK, 1024);
+        umma_bf16(t_o, a, b, idesc_o, kk ? 1u : 0u);
+      }
+      umma_commit(smem_u32(&o_done));
+    }
+    __syncwarp();
+    if (more) fetch_first(x);
+    float f = p.q_scale;
+    if (p.gated) f /= fmaxf(fabsf((row_sum[0][t] + row_sum[1][t]) * p.q_scale), chunk_exp2(-(F + B))) + 1e-6f;
+    ok = mbar_wait_bounded(smem_u32(&o_done), it & 1, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
+    ok = __all_sync(0xffffffffu, ok);
+    tc_fence_after();
+    if (!ok) continue;                               // (the next unit's first barrier ends the loop for all)
+    if (more) fetch_second(x);
     uint32_t a[32], b[32];
     tmem_ld_32x32(t_o + half * 32 + lane_addr, a);
     tmem_ld_32x32(t_s + half * 32 + lane_addr, b);
     tmem_ld_wait();
     tc_fence_before();
-    if (t < n) {
-      float4* dst = reinterpret_cast<float4*>(p.out + (long long)(row0 + t) * p.ldo + h * p.VP + z * 64 + half * 32);
+    if (t < cur.n) {
+      float4* dst = reinterpret_cast<float4*>(p.out + (long long)(cur.row0 + t) * p.ldo + cur.h * p.VP + cur.z * 64 + half * 32);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         float y[4];
@@ -931,6 +1006,7 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkPar
       }
     }
   }
+  cp_async_wait_all();
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
@@ -940,20 +1016,26 @@ __global__ void __launch_bounds__(CHT) recurrent_chunk_out_kernel(const ChunkPar
 
 template <int DK>
 static int launch_chunks(const ChunkParams& p, int n_chunks, int n_seq, cudaStream_t stream) {
-  static bool attr_dev[64] = {};
+  static int sms[64] = {};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
-  if (!attr_dev[dev]) {
+  if (sms[dev] == 0) {
+    int n = 0;
+    if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) return -10;
     if (cudaFuncSetAttribute(recurrent_chunk_state_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkStateCfg<DK>::kSmem) != cudaSuccess ||
         cudaFuncSetAttribute(recurrent_chunk_out_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, ChunkOutCfg<DK>::kSmem) != cudaSuccess)
       return -10;
-    attr_dev[dev] = true;
+    sms[dev] = n;
   }
-  const dim3 grid(n_chunks, p.H, p.VP / 64);
+  const int units = n_chunks * p.H * (p.VP / 64);
+  auto grid = [&](int smem) {                        // two CTAs per SM where they fit (and their TMEM does)
+    const int g = sms[dev] * (smem + 5 * 1024 <= 113 * 1024 ? 2 : 1);
+    return dim3(units < g ? units : g);
+  };
   if (launch_kernel(recurrent_chunk_gates_kernel, dim3(n_chunks, (p.H + 7) / 8), dim3(256), 0, stream, p) != cudaSuccess) return -14;
-  if (launch_kernel(recurrent_chunk_state_kernel<DK>, grid, dim3(CHT), ChunkStateCfg<DK>::kSmem, stream, p) != cudaSuccess) return -11;
+  if (launch_kernel(recurrent_chunk_state_kernel<DK>, grid(ChunkStateCfg<DK>::kSmem), dim3(CHT), ChunkStateCfg<DK>::kSmem, stream, p, units) != cudaSuccess) return -11;
   if (launch_kernel(recurrent_chunk_chain_kernel, dim3(DK / 32, p.H * (p.VP / SC_COLS), n_seq), dim3(256), 0, stream, p) != cudaSuccess) return -12;
-  return launch_kernel(recurrent_chunk_out_kernel<DK>, grid, dim3(CHT), ChunkOutCfg<DK>::kSmem, stream, p) == cudaSuccess ? 0 : -13;
+  return launch_kernel(recurrent_chunk_out_kernel<DK>, grid(ChunkOutCfg<DK>::kSmem), dim3(CHT), ChunkOutCfg<DK>::kSmem, stream, p, units) == cudaSuccess ? 0 : -13;
 }
 
 // ------------------------------------------------------------------------------------------
@@ -1021,7 +1103,7 @@ int rb_recurrent_scan(const void* proj, long long ld, int q_col, int k_col, int 
   if (H <= 0 || H > 65535 || B > 65535 || dk <= 0 || dk > KP || VP % SC_COLS != 0 || (gated ? small == nullptr : decay == nullptr)) return -1;
   const ScanParams p{proj, ld, q_col, k_col, v_col, small, ld_small, decay, bias_i, bias_f, cap, q_scale, s, n, m, slots, cu_q, seq_lens,
                      out, ldo, H, dk, KP, VP, num_slots, gated, rows, status};
-  if (cu_q == nullptr && dk <= RD_MAX_DK)
+  if (cu_q == nullptr && dk <= RD_MAX_DK && B <= RD_MAX_B)
     return dtype == 0 ? launch_decode<__nv_bfloat16>(p, B, stream) : launch_decode<float>(p, B, stream);
   return dtype == 0 ? launch_scan<__nv_bfloat16>(p, B, stream) : launch_scan<float>(p, B, stream);
 }

@@ -49,7 +49,7 @@ class KeyValuePart(Part):
         r = self.r
         self.proj = self.zeros(r.rows * max(w.geo.proj for w in self.layers))
         self.out = self.zeros(r.rows * max(w.geo.heads * w.geo.dp for w in self.layers))
-        self.splits = {b: {w.geo: ops.decode_num_splits(b, w.geo.kv_heads, r.max_model_len, head_dim=w.geo.dp) for w in self.layers}
+        self.splits = {b: {w.geo: ops.decode_num_splits(b, w.geo.kv_heads, r.max_model_len, head_dim=w.geo.dp) if b <= 64 else 1 for w in self.layers}
                        for b in sorted({*r.graph_batch_sizes, *range(1, min(r.max_batch, 64) + 1)})}
         need = max(ops.kv_workspace(g, b, n) for b, by in self.splits.items() for g, n in by.items())
         self.workspace = self.zeros(need, dtype=torch.float32) if r.bf16 else None

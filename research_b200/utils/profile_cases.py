@@ -250,6 +250,59 @@ def case_latent_prefill() -> None:
     print("ok")
 
 
+def _recurrent(T: int, seqs: int, gated: bool):
+    from ..ops.recurrent import RecurrentGeometry, RecurrentState
+
+    geo = RecurrentGeometry(16, 128, 128, silu=not gated, gated=gated)
+    proj = torch.randn(T, geo.proj, device="cuda").bfloat16()
+    small, bias, decay = torch.randn(T, 32, device="cuda"), torch.ones(16, device="cuda"), torch.full((16,), 0.97, device="cuda")
+    return (proj, small, geo, decay, bias, bias, 15.0, RecurrentState.zeros(geo, seqs, "cuda"), torch.arange(seqs, dtype=torch.int32, device="cuda"))
+
+
+def case_recurrent_decode() -> None:
+    """Matrix memory, one token for each of 256 sequences: 16 heads of 128 x 128 (268 MB of state)."""
+    a, out = _recurrent(256, 256, True), torch.empty(256, 2048, device="cuda")
+    lens = torch.full((256,), 100, dtype=torch.int32, device="cuda")
+    for _ in range(3):
+        ops.recurrent_scan(*a, None, lens, out, 256, 256)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def case_recurrent_prefill() -> None:
+    """Matrix memory in chunks: one portion of 4096 tokens, 16 heads of 128 x 128."""
+    from ..ops.recurrent import ChunkTable, chunk_workspace
+
+    T = 4096
+    a, out = _recurrent(T, 1, True), torch.empty(T, 2048, device="cuda")
+    cu, lens = torch.tensor([0, T], dtype=torch.int32, device="cuda"), torch.tensor([T], dtype=torch.int32, device="cuda")
+    table = ChunkTable.make([0, T], 0, "cuda")
+    room = torch.empty(chunk_workspace(table.chunks.shape[0], a[2]), dtype=torch.uint8, device="cuda")
+    for _ in range(3):
+        ops.recurrent_chunks(*a, cu, lens, out, table, room)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def case_keyvalue_decode() -> None:
+    """Keys-as-values attention: 256 sequences x 2048 keys, 16 query heads on 4 kv heads of 128 channels (537 MB of cache)."""
+    from ..ops.keyvalue import KeyValueGeometry
+
+    geo, B, L = KeyValueGeometry(16, 4, 128), 256, 2048
+    proj = torch.randn(B, geo.proj, device="cuda").bfloat16()
+    cache = torch.randn(B * L // 16, 4, 16, 128, device="cuda").bfloat16()
+    bt = torch.randperm(B * L // 16, device="cuda").int().view(B, -1)
+    lens, sink = torch.full((B,), L, dtype=torch.int32, device="cuda"), torch.zeros(16, device="cuda")
+    out = torch.empty(B, 2048, dtype=torch.bfloat16, device="cuda")
+    for _ in range(3):
+        ops.kv_attention(proj, geo, cache, bt, None, lens, sink, out, scale=0.09, rows=B, max_q=1, n_single=B)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
 CASES = {k[5:]: v for k, v in globals().items() if k.startswith("case_")}
 
 if __name__ == "__main__":
