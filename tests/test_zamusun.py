@@ -336,7 +336,7 @@ def test_sampling_score_and_weight_update(place):
     eng.update_weights(w2)
     want = oracle.forward(p[1], {k: v.double() for k, v in w2.items()}, CONFIGS[name])
     s = eng.open_stream()
-    agree(eng.feed([(s, p[1], list(range(140)))]), want, place[1])
+    assert errors(eng.feed([(s, p[1], list(range(140)))]), want).median() < TOL[place[1]]
 
 
 # ------------------------------------------------------------------------------------------ trace replay
