@@ -16,6 +16,7 @@
 // Behaviour replaced: rollouts/inference/attention/flex_backend.py:144-279 (SDPA prefill and
 // the host-loop gather decode). Numerics oracle: qwen_functional.py:173-248.
 #include "common.cuh"
+#include "history.cuh"
 #include "tma_host.h"
 
 #include <stdlib.h>
@@ -792,22 +793,53 @@ __global__ void kv_append_kernel(T* __restrict__ proj, long long ld, const int* 
         *reinterpret_cast<const uint4*>(row + H * D + i);
 }
 
-// Decode: the structure of paged_decode_tma_kernel with one tile that serves as K and V, two blocks (32 keys) per stage, up to
-// 16 query heads per CTA (blockIdx.y = kv head x chunk of 16 query heads). The sums of weights stay per thread until the
-// end, and the accumulators are rescaled only when a row's maximum moves.
-template <int D>
-__host__ __device__ constexpr int kv_dec_stages() { return D == 64 ? 4 : 3; }      // 64 / 96 KB of ring per CTA
+// Which keys j <= i a query at position i sees: all, the last `size` (window), or those of its own chunk of `size` positions.
+struct KeySpan {
+  int window, chunk;       // 0: none
+};
+__device__ __forceinline__ int first_key(const KeySpan& s, int position) {
+  if (s.window > 0) return max(0, position - s.window + 1);
+  return s.chunk > 0 ? position - position % s.chunk : 0;
+}
+
+// What multiplies a head's output: the sigmoid of one number per channel (activation type) or per head (fp32), or nothing;
+// times a constant.
+struct OutputGate {
+  const void* channels;    // [T, ld_channels], H * D of a row
+  long long ld_channels;
+  const float* heads;      // [T, ld_heads], H of a row
+  long long ld_heads;
+  float scale;
+};
+template <typename T>
+__device__ __forceinline__ float output_gate(const OutputGate& g, long long t, int h, int D, int d) {
+  if (g.channels != nullptr) return g.scale * kv_sigmoid(kv_to_f(reinterpret_cast<const T*>(g.channels)[t * g.ld_channels + h * D + d]));
+  return g.heads != nullptr ? g.scale * kv_sigmoid(g.heads[t * g.ld_heads + h]) : g.scale;
+}
+
+// Weight of the softmax sink relative to the maximum M (base 2); no sink: none.
+__device__ __forceinline__ float sink_weight(const float* sink, int h, float M) {
+  return sink != nullptr ? exp2f(sink[h] * 1.4426950408889634f - M) : 0.f;
+}
+
+// Decode: the structure of paged_decode_tma_kernel for up to 16 query heads per CTA (blockIdx.y = kv head x chunk of 16 query
+// heads). SHARED: values are keys, one tile serves as both, two blocks (32 keys) per stage; otherwise a stage is a block of
+// keys and one of values. The sums of weights stay per thread until the end, and the accumulators are rescaled only when a
+// row's maximum moves.
+template <int D, bool SHARED>
+__host__ __device__ constexpr int kv_dec_stages() { return SHARED && D == 64 ? 4 : 3; }      // 64 / 96 KB of ring per CTA, 48 / 96 KB
 constexpr int KV_MERGE_LD_PAD = 4;
 
-template <int D>
+template <int D, bool SHARED>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
-kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_col, const __grid_constant__ CUtensorMap k_map,
-                 const int* __restrict__ block_tables, const int* __restrict__ seq_lens, const float* __restrict__ sink,
-                 __nv_bfloat16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml, int H, int Hkv, int bt_stride,
-                 int num_blocks, int num_splits, float scale, int* status) {
+kv_decode_kernel(const __nv_bfloat16* __restrict__ q, long long ld, const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
+                 const int* __restrict__ block_tables, const int* __restrict__ seq_lens, const float* __restrict__ sink, const OutputGate gate,
+                 __nv_bfloat16* __restrict__ out, long long ldo, float* __restrict__ part_o, float* __restrict__ part_ml, int H, int Hkv,
+                 int bt_stride, int num_blocks, int num_splits, const KeySpan span, float scale, int* status) {
   constexpr int CH = D / 8;
+  constexpr int NB = SHARED ? 2 : 1;                               // blocks of keys in a stage
   constexpr int BLK_BYTES = KV_BLOCK * D * 2, TILE_BYTES = 2 * BLK_BYTES;
-  constexpr int ST = kv_dec_stages<D>();
+  constexpr int ST = kv_dec_stages<D, SHARED>();
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ __align__(8) uint64_t bars[DEC_WARPS][ST];
   __shared__ int abort_flag;
@@ -830,14 +862,15 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
   }
   pdl_wait();
   const int L = seq_lens[b];
-  const int n_blocks = (L + KV_BLOCK - 1) / KV_BLOCK, n_chunks = (n_blocks + 1) / 2;
-  const int per = (n_chunks + num_splits - 1) / num_splits;
-  const int c_begin = split * per;
+  const int n_blocks = (L + KV_BLOCK - 1) / KV_BLOCK, n_chunks = (n_blocks + NB - 1) / NB;
+  const int key0 = L > 0 ? first_key(span, L - 1) : 0, c_first = key0 / (NB * KV_BLOCK);
+  const int per = (n_chunks - c_first + num_splits - 1) / num_splits;
+  const int c_begin = c_first + split * per;
   const int c_end = min(n_chunks, c_begin + per);
   for (int i = threadIdx.x; i < 16 * CH; i += blockDim.x) {
     const int r = i / CH, c = i % CH;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < rows) v = *reinterpret_cast<const uint4*>(proj + b * ld + (h0 + r) * D + c * 8);
+    if (r < rows) v = *reinterpret_cast<const uint4*>(q + b * ld + (h0 + r) * D + c * 8);
     *reinterpret_cast<uint4*>(q_ptr + swz<D>(r, c)) = v;
   }
   __syncthreads();
@@ -858,13 +891,13 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
   const int n_my = first < c_end ? (c_end - first + DEC_WARPS - 1) / DEC_WARPS : 0;
   const int* bt_row = block_tables + (long long)b * bt_stride;
   auto load_ids = [&](int round) {
-    const int j = round * 32 + lane, blk = 2 * (first + (j >> 1) * DEC_WARPS) + (j & 1);
-    return (j >> 1) < n_my && blk < n_blocks ? __ldg(bt_row + blk) : num_blocks;     // past the end: out of bounds, zeros
+    const int j = round * 32 + lane, blk = NB * (first + (j / NB) * DEC_WARPS) + j % NB;
+    return j / NB < n_my && blk < n_blocks ? __ldg(bt_row + blk) : num_blocks;     // past the end: out of bounds, zeros
   };
   int ids_round = 0, ids = load_ids(0), ids_next = load_ids(1);
   auto blocks_of = [&](int i) {   // all lanes, i uniform and non-decreasing
-    if ((i >> 4) > ids_round) { ids = ids_next; ids_round = i >> 4; ids_next = load_ids(ids_round + 1); }
-    return make_int2(__shfl_sync(0xffffffffu, ids, (2 * i) & 31), __shfl_sync(0xffffffffu, ids, (2 * i + 1) & 31));
+    if (i / (32 / NB) > ids_round) { ids = ids_next; ids_round = i / (32 / NB); ids_next = load_ids(ids_round + 1); }
+    return make_int2(__shfl_sync(0xffffffffu, ids, (NB * i) & 31), __shfl_sync(0xffffffffu, ids, (NB * i + NB - 1) & 31));
   };
   auto issue = [&](int i, int2 blk) {   // lane 0 only
     const int stage = i % ST;
@@ -874,7 +907,7 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
 #pragma unroll
     for (int hx = 0; hx < D / 64; ++hx) {
       tma_load_2d(ks + hx * (KV_BLOCK * 128), &k_map, bar, hx * 64, (blk.x * Hkv + kvh) * KV_BLOCK);
-      tma_load_2d(ks + BLK_BYTES + hx * (KV_BLOCK * 128), &k_map, bar, hx * 64, (blk.y * Hkv + kvh) * KV_BLOCK);
+      tma_load_2d(ks + BLK_BYTES + hx * (KV_BLOCK * 128), SHARED ? &k_map : &v_map, bar, hx * 64, (blk.y * Hkv + kvh) * KV_BLOCK);
     }
   };
   int issued = 0;
@@ -894,28 +927,28 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
     ok = mbar_wait_bounded(smem_u32(&bars[warp][stage]), (uint32_t)((i / ST) & 1), abortp, status, ST_TIMEOUT_SMEM_FULL);
     ok = __all_sync(0xffffffffu, ok);
     if (!ok) break;
-    const uint32_t ks = k_smem + stage * TILE_BYTES;
-    float sc[4][4] = {};
+    const uint32_t ks = k_smem + stage * TILE_BYTES, vs = SHARED ? ks : ks + BLK_BYTES;
+    float sc[2 * NB][4] = {};
 #pragma unroll
     for (int kk = 0; kk < D / 16; ++kk)
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
+      for (int half = 0; half < NB; ++half) {
         uint32_t b0, b1, b2, b3;
         ldsm_x4(ks + half * BLK_BYTES + swz_tma<D>((mat >> 1) * 8 + rr, 2 * kk + (mat & 1)), b0, b1, b2, b3);
         mma_16816(sc[2 * half], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b0, b1);
         mma_16816(sc[2 * half + 1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], b2, b3);
       }
-    const int tok0 = (first + i * DEC_WARPS) * 2 * KV_BLOCK + 2 * (lane & 3);
-    if (tok0 - 2 * (lane & 3) + 2 * KV_BLOCK > L) {
+    const int tile0 = (first + i * DEC_WARPS) * NB * KV_BLOCK, tok0 = tile0 + 2 * (lane & 3);
+    if (tile0 + NB * KV_BLOCK > L || tile0 < key0) {
 #pragma unroll
-      for (int n8 = 0; n8 < 4; ++n8) {
-        if (tok0 + 8 * n8 >= L) sc[n8][0] = sc[n8][2] = -INFINITY;
-        if (tok0 + 8 * n8 + 1 >= L) sc[n8][1] = sc[n8][3] = -INFINITY;
+      for (int n8 = 0; n8 < 2 * NB; ++n8) {
+        if (tok0 + 8 * n8 >= L || tok0 + 8 * n8 < key0) sc[n8][0] = sc[n8][2] = -INFINITY;
+        if (tok0 + 8 * n8 + 1 >= L || tok0 + 8 * n8 + 1 < key0) sc[n8][1] = sc[n8][3] = -INFINITY;
       }
     }
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
-    for (int n8 = 0; n8 < 4; ++n8) {
+    for (int n8 = 0; n8 < 2 * NB; ++n8) {
       mx0 = fmaxf(mx0, fmaxf(sc[n8][0], sc[n8][1]));
       mx1 = fmaxf(mx1, fmaxf(sc[n8][2], sc[n8][3]));
     }
@@ -923,7 +956,7 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
     mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
     mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2)) * scale_log2;
     mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2)) * scale_log2;
-    if (__any_sync(0xffffffffu, mx0 > st.m0 || mx1 > st.m1)) {      // (the tile's first key is valid: the maximum is finite)
+    if (__any_sync(0xffffffffu, mx0 > st.m0 || mx1 > st.m1)) {      // (every tile has a visible key: the maximum is finite)
       const float n0 = fmaxf(st.m0, mx0), n1 = fmaxf(st.m1, mx1);
       const float c0 = exp2f(st.m0 - n0), c1 = exp2f(st.m1 - n1);
       st.m0 = n0; st.m1 = n1;
@@ -931,9 +964,9 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
 #pragma unroll
       for (int n8 = 0; n8 < D / 8; ++n8) { o[n8][0] *= c0; o[n8][1] *= c0; o[n8][2] *= c1; o[n8][3] *= c1; }
     }
-    uint32_t pk[4][2];
+    uint32_t pk[2 * NB][2];
 #pragma unroll
-    for (int n8 = 0; n8 < 4; ++n8) {
+    for (int n8 = 0; n8 < 2 * NB; ++n8) {
       const float e0 = kv_exp2(fmaf(sc[n8][0], scale_log2, -st.m0)), e1 = kv_exp2(fmaf(sc[n8][1], scale_log2, -st.m0));
       const float f0 = kv_exp2(fmaf(sc[n8][2], scale_log2, -st.m1)), f1 = kv_exp2(fmaf(sc[n8][3], scale_log2, -st.m1));
       st.l0 += e0 + e1;
@@ -944,9 +977,9 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
 #pragma unroll
     for (int dp = 0; dp < D / 16; ++dp)
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
+      for (int half = 0; half < NB; ++half) {
         uint32_t b0, b1, b2, b3;
-        ldsm_x4_t(ks + half * BLK_BYTES + swz_tma<D>((mat & 1) * 8 + rr, 2 * dp + (mat >> 1)), b0, b1, b2, b3);
+        ldsm_x4_t(vs + half * BLK_BYTES + swz_tma<D>((mat & 1) * 8 + rr, 2 * dp + (mat >> 1)), b0, b1, b2, b3);
         mma_16816(o[2 * dp], pk[2 * half][0], pk[2 * half][1], pk[2 * half + 1][0], pk[2 * half + 1][1], b0, b1);
         mma_16816(o[2 * dp + 1], pk[2 * half][0], pk[2 * half][1], pk[2 * half + 1][0], pk[2 * half + 1][1], b2, b3);
       }
@@ -997,9 +1030,8 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
     }
     if (num_splits == 1) {
       float y = 0.f;
-      if (l > 0.f)
-        y = acc / (l + exp2f(sink[h] * 1.4426950408889634f - M)) * kv_sigmoid(__bfloat162float(proj[b * ld + gate_col + h * D + d]));
-      out[((long long)b * H + h) * D + d] = __float2bfloat16_rn(y);
+      if (l > 0.f) y = acc / (l + sink_weight(sink, h, M)) * output_gate<__nv_bfloat16>(gate, b, h, D, d);
+      out[b * ldo + h * D + d] = __float2bfloat16_rn(y);
     } else {
       const long long pi = ((long long)b * H + h) * num_splits + split;
       part_o[pi * D + d] = acc;
@@ -1009,9 +1041,8 @@ kv_decode_kernel(const __nv_bfloat16* __restrict__ proj, long long ld, int gate_
 }
 
 template <int D>
-__global__ void kv_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const __nv_bfloat16* __restrict__ proj,
-                                       long long ld, int gate_col, const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int H,
-                                       int num_splits) {
+__global__ void kv_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const OutputGate gate,
+                                       const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, long long ldo, int H, int num_splits) {
   pdl_launch_dependents();
   pdl_wait();
   const int h = blockIdx.x, d = threadIdx.x;
@@ -1025,9 +1056,9 @@ __global__ void kv_decode_merge_kernel(const float* __restrict__ part_o, const f
       acc += e * part_o[(bh * num_splits + s) * D + d];
       l += e * part_ml[(bh * num_splits + s) * 2 + 1];
     }
-    y = acc / (l + exp2f(sink[h] * 1.4426950408889634f - M)) * kv_sigmoid(__bfloat162float(proj[b * ld + gate_col + h * D + d]));
+    y = acc / (l + sink_weight(sink, h, M)) * output_gate<__nv_bfloat16>(gate, b, h, D, d);
   }
-  out[bh * D + d] = __float2bfloat16_rn(y);
+  out[b * ldo + h * D + d] = __float2bfloat16_rn(y);
 }
 
 // Any head size up to 512 and either number format, a warp per (token, query head): the exact mode and sizes without a
@@ -1036,9 +1067,10 @@ constexpr int KVS_WARPS = 4, KVS_MAX_D = 512;
 
 template <typename T>
 __global__ void __launch_bounds__(KVS_WARPS * 32)
-kv_simple_kernel(const T* __restrict__ proj, long long ld, int gate_col, const T* __restrict__ cache, const int* __restrict__ block_tables,
-                 const int* __restrict__ cu_q, const int* __restrict__ seq_lens, const float* __restrict__ sink, T* __restrict__ out, int H, int G,
-                 int D, int bt_stride, int num_blocks, int rows, float scale, int* status) {
+kv_simple_kernel(const T* __restrict__ qrows, long long ld, const T* __restrict__ keys, const T* __restrict__ values,
+                 const int* __restrict__ block_tables, const int* __restrict__ cu_q, const int* __restrict__ seq_lens, const float* __restrict__ sink,
+                 const OutputGate gate, T* __restrict__ out, long long ldo, int H, int G, int D, int bt_stride, int num_blocks, int rows,
+                 const KeySpan span, float scale, int* status) {
   extern __shared__ float kvs_q[];       // [KVS_WARPS][D]
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -1050,19 +1082,20 @@ kv_simple_kernel(const T* __restrict__ proj, long long ld, int gate_col, const T
   if (t >= t1) return;                                     // (no CTA-wide synchronisation below)
   if (t >= rows) { if (lane == 0) set_status(status, ST_BAD_INDEX); return; }
   const int n_keys = seq_lens[b] - (t1 - 1 - t);           // keys this token sees
-  T* dst = out + ((long long)t * H + h) * D;
+  T* dst = out + t * ldo + h * D;
   if (n_keys <= 0) {
     for (int d = lane; d < D; d += 32) kv_store(dst + d, 0.f);
     return;
   }
   float* q = kvs_q + warp * D;
-  for (int d = lane; d < D; d += 32) q[d] = kv_to_f(proj[t * ld + h * D + d]) * scale;
+  for (int d = lane; d < D; d += 32) q[d] = kv_to_f(qrows[t * ld + h * D + d]) * scale;
   __syncwarp();
   float o[KVS_MAX_D / 32];
 #pragma unroll
   for (int i = 0; i < KVS_MAX_D / 32; ++i) o[i] = 0.f;
-  float m = sink[h], l = 1.f;                              // the sink: a key of weight exp(sink) without a value
-  for (int k0 = 0; k0 < n_keys; k0 += 32) {
+  float m = -INFINITY, l = 0.f;
+  if (sink != nullptr) { m = sink[h]; l = 1.f; }           // the sink: a key of weight exp(sink) without a value
+  for (int k0 = first_key(span, n_keys - 1); k0 < n_keys; k0 += 32) {
     const int j = k0 + lane;
     float s = -INFINITY;
     long long row = 0;
@@ -1071,7 +1104,7 @@ kv_simple_kernel(const T* __restrict__ proj, long long ld, int gate_col, const T
       if (blk < 0 || blk >= num_blocks) { set_status(status, ST_BAD_INDEX); blk = 0; }
       row = (((long long)blk * G + kvh) * KV_BLOCK + j % KV_BLOCK) * D;
       s = 0.f;
-      for (int d = 0; d < D; ++d) s = fmaf(q[d], kv_to_f(cache[row + d]), s);
+      for (int d = 0; d < D; ++d) s = fmaf(q[d], kv_to_f(keys[row + d]), s);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float c = expf(m - m_new), p = j < n_keys ? expf(s - m_new) : 0.f;
@@ -1085,14 +1118,13 @@ kv_simple_kernel(const T* __restrict__ proj, long long ld, int gate_col, const T
       const long long ru = __shfl_sync(0xffffffffu, row, u);
 #pragma unroll
       for (int i = 0; i < KVS_MAX_D / 32; ++i)
-        if (lane + 32 * i < D) o[i] = fmaf(pu, kv_to_f(cache[ru + lane + 32 * i]), o[i]);
+        if (lane + 32 * i < D) o[i] = fmaf(pu, kv_to_f(values[ru + lane + 32 * i]), o[i]);
     }
   }
-  const T* gate = proj + t * ld + gate_col + h * D;
 #pragma unroll
   for (int i = 0; i < KVS_MAX_D / 32; ++i) {
     const int d = lane + 32 * i;
-    if (d < D) kv_store(dst + d, o[i] / l * kv_sigmoid(kv_to_f(gate[d])));
+    if (d < D) kv_store(dst + d, o[i] / l * output_gate<T>(gate, t, h, D, d));
   }
 }
 
@@ -1120,14 +1152,225 @@ __global__ void kv_gate_kernel(__nv_bfloat16* __restrict__ out, const float* __r
   }
 }
 
-template <int D>
+// ------------------------------------------------------------------------------------------
+// Grouped attention with cached keys and values: everything between the joint projection and the attention, one CTA per token.
+// Every projected channel goes through its causal convolution (if there is one), queries and keys through the norm and the rotation;
+// queries land in a buffer with heads padded to DP channels, keys and values in the cache. Look back: history.cuh, over the raw
+// projected values.
+// ------------------------------------------------------------------------------------------
+constexpr int GA_THREADS = 256, GA_MAX_DP = 512;
+enum { GA_NORM_NONE = 0, GA_NORM_PROJECTION = 1, GA_NORM_HEAD = 2 };
+
+struct GroupedAppend {
+  const void* proj;        // [T, ld]: q at 0, k at k_col, v at v_col (multiples of 8); `channels` columns in all
+  long long ld;
+  int k_col, v_col, channels;
+  const float* conv;       // [taps, channels] or null
+  int taps;
+  void* hist;              // [slots, taps - 1, channels]
+  History rows;
+  const int* slots;        // [T] places in the cache, negative: not stored
+  const float* q_norm;     // [H * dim], projection norm
+  const float* k_norm;     // [G * dim]
+  int norm;
+  float eps;
+  const float* table;      // [positions, half, 2] cos, sin
+  int half, interleaved, max_pos;
+  void* q;                 // [T, H * DP]
+  void* keys;              // [num_blocks, G, 16, DP]
+  void* values;
+  int num_blocks, H, G, dim, vdim, DP, T;
+  int* status;
+};
+
+template <typename T>
+__device__ __forceinline__ void load8(const T* p, float (&x)[8]) {
+  constexpr int V = 16 / sizeof(T);
+#pragma unroll
+  for (int i = 0; i < 8 / V; ++i) {
+    union { uint4 u; T e[V]; } a;
+    a.u = reinterpret_cast<const uint4*>(p)[i];
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[i * V + j] = kv_to_f(a.e[j]);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(GA_THREADS) grouped_append_kernel(const GroupedAppend p) {
+  extern __shared__ float ga_row[];                       // q and k channels, laid out as in the projection
+  __shared__ float red[2][GA_THREADS / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* rows = reinterpret_cast<const T*>(p.proj);
+  T* hist = reinterpret_cast<T*>(p.hist);
+  RowPlace place{0, p.rows.positions[t], -1};
+  if (p.taps > 1) place = row_place(p.rows, t, p.status);
+  int slot = p.slots[t];
+  if (slot >= 0 && slot / KV_BLOCK >= p.num_blocks) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); slot = -1; }
+  const long long krow = slot >= 0 ? ((long long)(slot / KV_BLOCK) * p.G * KV_BLOCK + slot % KV_BLOCK) * p.DP : 0;
+  T* vcache = reinterpret_cast<T*>(p.values) + krow;      // + head * 16 * DP
+  float ssq = 0.f, ssk = 0.f;
+  const int nq = p.H * p.dim, nk = p.G * p.dim, nv = p.G * p.vdim;
+  for (int c = threadIdx.x * 8; c < p.channels; c += GA_THREADS * 8) {
+    float x[8];
+    load8(rows + (long long)t * p.ld + c, x);
+    if (p.conv != nullptr) {
+      float u[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) { u[i] = x[i]; x[i] *= p.conv[(long long)(p.taps - 1) * p.channels + c + i]; }
+      for (int d = 1; d < p.taps; ++d) {
+        const T* back = row_before(place, d, rows, p.ld, t, (const T*)hist, p.taps - 1, p.channels);
+        if (back == nullptr) break;                       // (nothing further back either)
+        float y[8];
+        load8(back + c, y);
+        const float* w = p.conv + (long long)(p.taps - 1 - d) * p.channels + c;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] = fmaf(w[i], y[i], x[i]);
+      }
+      if (p.taps > 1 && p.rows.cu_q == nullptr && place.slot >= 0) {    // one row per sequence: this thread moves its own channels on
+        T* mine = hist + (long long)place.slot * (p.taps - 1) * p.channels + c;
+        for (int d = p.taps - 2; d >= 1; --d)
+#pragma unroll
+          for (int i = 0; i < (int)(8 * sizeof(T) / 16); ++i)
+            reinterpret_cast<uint4*>(mine + (long long)d * p.channels)[i] = reinterpret_cast<const uint4*>(mine + (long long)(d - 1) * p.channels)[i];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) kv_store(mine + i, u[i]);
+      }
+    }
+    if (c >= p.v_col) {
+      const int v0 = c - p.v_col;
+      if (slot >= 0) {
+        if (p.vdim % 8 == 0) {
+          if (v0 < nv) {
+            T* dst = vcache + (long long)(v0 / p.vdim) * KV_BLOCK * p.DP + v0 % p.vdim;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) kv_store(dst + i, x[i]);
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            if (v0 + i < nv) kv_store(vcache + (long long)((v0 + i) / p.vdim) * KV_BLOCK * p.DP + (v0 + i) % p.vdim, x[i]);
+        }
+      }
+    } else {
+      const bool is_k = c >= p.k_col;
+      const int n = is_k ? nk : nq, c0 = c - (is_k ? p.k_col : 0);
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        ga_row[c + i] = x[i];
+        if (c0 + i < n) s = fmaf(x[i], x[i], s);
+      }
+      if (is_k) ssk += s; else ssq += s;
+    }
+  }
+  if (p.norm == GA_NORM_PROJECTION) {
+    ssq = warp_sum(ssq);
+    ssk = warp_sum(ssk);
+    if (lane == 0) { red[0][warp] = ssq; red[1][warp] = ssk; }
+  }
+  __syncthreads();
+  float rq = 1.f, rk = 1.f;
+  if (p.norm == GA_NORM_PROJECTION) {
+    ssq = ssk = 0.f;
+#pragma unroll
+    for (int i = 0; i < GA_THREADS / 32; ++i) { ssq += red[0][i]; ssk += red[1][i]; }
+    rq = 1.f / sqrtf(ssq / (float)nq + p.eps);
+    rk = 1.f / sqrtf(ssk / (float)nk + p.eps);
+  }
+  int pos = place.position;
+  if (pos < 0 || pos >= p.max_pos) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); pos = 0; }
+  const float2* table = reinterpret_cast<const float2*>(p.table) + (long long)pos * p.half;
+  // a warp per head, two channels per lane and step
+  for (int hd = warp; hd < p.H + p.G; hd += GA_THREADS / 32) {
+    const bool is_k = hd >= p.H;
+    const int head = is_k ? hd - p.H : hd;
+    if (is_k && slot < 0) continue;
+    const float* src = ga_row + (is_k ? p.k_col : 0) + head * p.dim;
+    const float* w = p.norm == GA_NORM_PROJECTION ? (is_k ? p.k_norm : p.q_norm) + head * p.dim : nullptr;
+    const float r = is_k ? rk : rq;
+    auto at = [&](int d) { return w != nullptr ? src[d] * r * w[d] : src[d]; };
+    auto rotated = [&](int d) {
+      if (d >= 2 * p.half) return d < p.dim ? at(d) : 0.f;
+      const int i = p.interleaved ? d >> 1 : d < p.half ? d : d - p.half;
+      const bool first = p.interleaved ? (d & 1) == 0 : d < p.half;
+      const float2 cs = table[i];
+      const float u = at(p.interleaved ? 2 * i : i), v = at(p.interleaved ? 2 * i + 1 : i + p.half);
+      return first ? u * cs.x - v * cs.y : v * cs.x + u * cs.y;
+    };
+    float y[GA_MAX_DP / 64][2], ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < GA_MAX_DP / 64; ++j) {
+      const int d = lane * 2 + j * 64;
+      y[j][0] = y[j][1] = 0.f;
+      if (d < p.DP) {
+        y[j][0] = rotated(d);
+        y[j][1] = rotated(d + 1);
+        ss += y[j][0] * y[j][0] + y[j][1] * y[j][1];
+      }
+    }
+    float f = 1.f;
+    if (p.norm == GA_NORM_HEAD) f = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+    T* dst = is_k ? reinterpret_cast<T*>(p.keys) + krow + (long long)head * KV_BLOCK * p.DP
+                  : reinterpret_cast<T*>(p.q) + ((long long)t * p.H + head) * p.DP;
+#pragma unroll
+    for (int j = 0; j < GA_MAX_DP / 64; ++j) {
+      const int d = lane * 2 + j * 64;
+      if (d < p.DP) { kv_store(dst + d, y[j][0] * f); kv_store(dst + d + 1, y[j][1] * f); }
+    }
+  }
+}
+
+template <int D, bool SHARED>
 constexpr int kv_decode_smem_bytes() {
-  const int ring = DEC_WARPS * kv_dec_stages<D>() * 2 * KV_BLOCK * D * 2 + 16 * D * 2;
+  const int ring = DEC_WARPS * kv_dec_stages<D, SHARED>() * 2 * KV_BLOCK * D * 2 + 16 * D * 2;
   const int merge = DEC_WARPS * 16 * (D + KV_MERGE_LD_PAD + 2) * 4;
   return 1024 + (ring > merge ? ring : merge);
 }
 
 }  // namespace rb
+
+struct GroupedAppendArgs {       // mirrored by ops/grouped.py
+  const void* proj; const float* conv; void* hist; const int* cu_q; const int* positions; const int* state_slots; const int* slots;
+  const float* q_norm; const float* k_norm; const float* table; void* q; void* keys; void* values; int* status;
+  long long ld;
+  int k_col, v_col, channels, taps, B, num_state_slots, norm, half, interleaved, max_pos, num_blocks, H, G, dim, vdim, DP, T, dtype;
+  float eps;
+};
+
+// Norm, rotation, convolution and cache append of a batch; with cu_q also moves the convolution's histories on (a second launch).
+extern "C" int rb_grouped_append(const GroupedAppendArgs* a, cudaStream_t stream) {
+  if (a->T <= 0) return 0;
+  if (a->DP > GA_MAX_DP || a->DP % 64 != 0 || a->dim > a->DP || a->vdim > a->DP || a->G <= 0 || a->H % a->G != 0 || a->taps < 1) return -1;
+  if (a->taps > 1 && (a->conv == nullptr || a->hist == nullptr || a->state_slots == nullptr)) return -1;
+  if (a->k_col % 8 != 0 || a->v_col % 8 != 0 || a->channels % 8 != 0 || a->ld % 8 != 0 || 2 * a->half > a->dim) return -1;
+  const size_t smem = (size_t)a->v_col * 4;
+  if (smem > 200 * 1024) return -1;
+  GroupedAppend p;
+  p.proj = a->proj; p.ld = a->ld; p.k_col = a->k_col; p.v_col = a->v_col; p.channels = a->channels;
+  p.conv = a->conv; p.taps = a->taps; p.hist = a->hist;
+  p.rows = History{a->cu_q, a->positions, a->state_slots, a->B, a->taps - 1, a->num_state_slots};
+  p.slots = a->slots; p.q_norm = a->q_norm; p.k_norm = a->k_norm; p.norm = a->norm; p.eps = a->eps;
+  p.table = a->table; p.half = a->half; p.interleaved = a->interleaved; p.max_pos = a->max_pos;
+  p.q = a->q; p.keys = a->keys; p.values = a->values; p.num_blocks = a->num_blocks;
+  p.H = a->H; p.G = a->G; p.dim = a->dim; p.vdim = a->vdim; p.DP = a->DP; p.T = a->T; p.status = a->status;
+  const int dev = current_device_index();
+  if (dev < 0) return -10;
+  static bool attr[RB_MAX_DEVICES] = {};
+  if (!attr[dev]) {
+    if (cudaFuncSetAttribute(grouped_append_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess ||
+        cudaFuncSetAttribute(grouped_append_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+      return -10;
+    attr[dev] = true;
+  }
+  cudaError_t e = a->dtype == 0 ? launch_kernel(grouped_append_kernel<__nv_bfloat16>, dim3(a->T), dim3(GA_THREADS), smem, stream, p)
+                                : launch_kernel(grouped_append_kernel<float>, dim3(a->T), dim3(GA_THREADS), smem, stream, p);
+  if (e == cudaSuccess && a->cu_q != nullptr && a->taps > 1)
+    e = a->dtype == 0 ? launch_history_update((const __nv_bfloat16*)a->proj, a->ld, p.rows, (__nv_bfloat16*)a->hist, a->channels, stream)
+                      : launch_history_update((const float*)a->proj, a->ld, p.rows, (float*)a->hist, a->channels, stream);
+  return e == cudaSuccess ? 0 : -11;
+}
 
 extern "C" int rb_kv_append(void* proj, long long ld, const int* positions, const int* slots, float coef, int every, void* cache, int num_blocks,
                             int H, int G, int D, int T, int dtype, int* status, cudaStream_t stream) {
@@ -1143,54 +1386,68 @@ extern "C" int rb_kv_append(void* proj, long long ld, const int* positions, cons
   return e == cudaSuccess ? 0 : -11;
 }
 
-extern "C" int rb_kv_decode(const void* proj, long long ld, int gate_col, const void* cache, const int* block_tables, const int* seq_lens,
-                            const float* sink, void* out, float* workspace, int B, int H, int G, int D, int bt_stride, int num_blocks,
-                            int block_size, int num_splits, float scale, int* status, cudaStream_t stream) {
+// Gates of rb_kv_decode / rb_kv_simple: gate_channels (activation type, H * D per row) or gate_heads (fp32, H per row), or neither;
+// sink may be null. values null (or equal to keys): values are keys. window / chunk: see KeySpan.
+extern "C" int rb_kv_decode(const void* q, long long ld, const void* keys, const void* values, const int* block_tables, const int* seq_lens,
+                            const float* sink, const void* gate_channels, long long ld_gate_channels, const float* gate_heads, long long ld_gate_heads,
+                            float gate_scale, void* out, long long ldo, float* workspace, int B, int H, int G, int D, int bt_stride, int num_blocks,
+                            int block_size, int num_splits, int window, int chunk, float scale, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (block_size != KV_BLOCK || G <= 0 || H % G != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr) || B > 65535) return -1;
-  CUtensorMap kmap;
-  if (tma_map_2d_bf16(&kmap, cache, (unsigned long long)num_blocks * G * KV_BLOCK, D, D, KV_BLOCK) != 0) return -20;
+  CUtensorMap kmap, vmap;
+  const bool shared = values == nullptr || values == keys;
+  const unsigned long long rows = (unsigned long long)num_blocks * G * KV_BLOCK;
+  if (tma_map_2d_bf16(&kmap, keys, rows, D, D, KV_BLOCK) != 0) return -20;
+  if (tma_map_2d_bf16(&vmap, shared ? keys : values, rows, D, D, KV_BLOCK) != 0) return -20;
   float* part_ml = workspace != nullptr ? workspace + (long long)B * H * num_splits * D : nullptr;
   const dim3 grid(num_splits, G * ((H / G + 15) / 16), B);
-#define LAUNCH_KV(DD)                                                                                          \
+  const OutputGate gate{gate_channels, ld_gate_channels, gate_heads, ld_gate_heads, gate_scale};
+  const KeySpan span{window, chunk};
+#define LAUNCH_KV(DD, SH)                                                                                      \
   do {                                                                                                         \
     static bool attr[RB_MAX_DEVICES] = {};                                                                     \
     const int dev_ = current_device_index();                                                                   \
     if (dev_ < 0) return -10;                                                                                  \
     if (!attr[dev_]) {                                                                                         \
-      if (cudaFuncSetAttribute(kv_decode_kernel<DD>, cudaFuncAttributeMaxDynamicSharedMemorySize,              \
-                               kv_decode_smem_bytes<DD>()) != cudaSuccess) return -10;                         \
+      if (cudaFuncSetAttribute(kv_decode_kernel<DD, SH>, cudaFuncAttributeMaxDynamicSharedMemorySize,          \
+                               kv_decode_smem_bytes<DD, SH>()) != cudaSuccess) return -10;                     \
       attr[dev_] = true;                                                                                       \
     }                                                                                                          \
-    launch_kernel(kv_decode_kernel<DD>, grid, dim3(DEC_WARPS * 32), kv_decode_smem_bytes<DD>(), stream,        \
-                  (const __nv_bfloat16*)proj, ld, gate_col, kmap, block_tables, seq_lens, sink,                \
-                  (__nv_bfloat16*)out, workspace, part_ml, H, G, bt_stride, num_blocks, num_splits, scale, status); \
+    launch_kernel(kv_decode_kernel<DD, SH>, grid, dim3(DEC_WARPS * 32), kv_decode_smem_bytes<DD, SH>(), stream, \
+                  (const __nv_bfloat16*)q, ld, kmap, vmap, block_tables, seq_lens, sink, gate,                 \
+                  (__nv_bfloat16*)out, ldo, workspace, part_ml, H, G, bt_stride, num_blocks, num_splits, span, scale, status); \
     if (num_splits > 1)                                                                                        \
       launch_kernel(kv_decode_merge_kernel<DD>, dim3(H, B), dim3(DD), 0, stream, (const float*)workspace,      \
-                    (const float*)part_ml, (const __nv_bfloat16*)proj, ld, gate_col, sink, (__nv_bfloat16*)out, H, num_splits); \
+                    (const float*)part_ml, gate, sink, (__nv_bfloat16*)out, ldo, H, num_splits);               \
   } while (0)
-  if (D == 64) LAUNCH_KV(64);
-  else if (D == 128) LAUNCH_KV(128);
+  if (D == 64 && shared) LAUNCH_KV(64, true);
+  else if (D == 128 && shared) LAUNCH_KV(128, true);
+  else if (D == 64) LAUNCH_KV(64, false);
+  else if (D == 128) LAUNCH_KV(128, false);
   else return -1;
 #undef LAUNCH_KV
   return cudaGetLastError() == cudaSuccess ? 0 : -11;
 }
 
-extern "C" int rb_kv_simple(const void* proj, long long ld, int gate_col, const void* cache, const int* block_tables, const int* cu_q,
-                            const int* seq_lens, const float* sink, void* out, int H, int G, int D, int bt_stride, int num_blocks, int B, int rows,
-                            int max_q, int dtype, float scale, int* status, cudaStream_t stream) {
+extern "C" int rb_kv_simple(const void* q, long long ld, const void* keys, const void* values, const int* block_tables, const int* cu_q,
+                            const int* seq_lens, const float* sink, const void* gate_channels, long long ld_gate_channels, const float* gate_heads,
+                            long long ld_gate_heads, float gate_scale, void* out, long long ldo, int H, int G, int D, int bt_stride, int num_blocks,
+                            int B, int rows, int max_q, int window, int chunk, int dtype, float scale, int* status, cudaStream_t stream) {
   if (B <= 0 || rows <= 0) return 0;
   if (D > KVS_MAX_D || G <= 0 || H % G != 0 || H > 65535 || B > 65535) return -1;
   const dim3 grid((max_q + KVS_WARPS - 1) / KVS_WARPS, H, B);
   const size_t smem = (size_t)KVS_WARPS * D * 4;
+  const OutputGate gate{gate_channels, ld_gate_channels, gate_heads, ld_gate_heads, gate_scale};
+  const KeySpan span{window, chunk};
+  if (values == nullptr) values = keys;
   cudaError_t e;
   if (dtype == 0)
-    e = launch_kernel(kv_simple_kernel<__nv_bfloat16>, grid, dim3(KVS_WARPS * 32), smem, stream, (const __nv_bfloat16*)proj, ld, gate_col,
-                      (const __nv_bfloat16*)cache, block_tables, cu_q, seq_lens, sink, (__nv_bfloat16*)out, H, G, D, bt_stride, num_blocks, rows,
-                      scale, status);
+    e = launch_kernel(kv_simple_kernel<__nv_bfloat16>, grid, dim3(KVS_WARPS * 32), smem, stream, (const __nv_bfloat16*)q, ld,
+                      (const __nv_bfloat16*)keys, (const __nv_bfloat16*)values, block_tables, cu_q, seq_lens, sink, gate, (__nv_bfloat16*)out, ldo, H, G,
+                      D, bt_stride, num_blocks, rows, span, scale, status);
   else
-    e = launch_kernel(kv_simple_kernel<float>, grid, dim3(KVS_WARPS * 32), smem, stream, (const float*)proj, ld, gate_col, (const float*)cache,
-                      block_tables, cu_q, seq_lens, sink, (float*)out, H, G, D, bt_stride, num_blocks, rows, scale, status);
+    e = launch_kernel(kv_simple_kernel<float>, grid, dim3(KVS_WARPS * 32), smem, stream, (const float*)q, ld, (const float*)keys, (const float*)values,
+                      block_tables, cu_q, seq_lens, sink, gate, (float*)out, ldo, H, G, D, bt_stride, num_blocks, rows, span, scale, status);
   return e == cudaSuccess ? 0 : -11;
 }
 

@@ -83,10 +83,22 @@ struct FlashFwdParams {
   const int* block_tables;  // [B, max_blocks] (paged)
   int max_blocks, num_blocks;
   int Hq, Hkv, Tq;
-  int causal, window, paged;
+  int causal, window, chunk, paged;     // window: the last so many keys; chunk: keys of the query's own run of so many positions (0: none)
+  const float* gate;   // [Tq, ld_gate] or null: a head's output is multiplied by gate_scale * sigmoid(gate)
+  long long ld_gate, ldo;
+  float gate_scale;
   float scale_log2;
   int* status;
 };
+
+// First key the query at position i sees.
+__device__ __forceinline__ int flash_first_key(const FlashFwdParams& p, int i) {
+  if (p.window > 0) return max(0, i - p.window + 1);
+  return p.chunk > 0 ? i - i % p.chunk : 0;
+}
+__device__ __forceinline__ float flash_gate(const FlashFwdParams& p, long long row, int h) {
+  return p.gate != nullptr ? p.gate_scale / (1.f + __expf(-p.gate[row * p.ld_gate + h])) : 1.f;
+}
 
 template <int D>
 struct FlashCfg {
@@ -120,8 +132,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd_kernel(const __grid_c
   const int kvh = h / (p.Hq / p.Hkv);
   // keys this tile can see
   int hi = p.causal ? min(kv_len, off + q0 + FA_BM) : kv_len;
-  int lo = 0;
-  if (p.window > 0) lo = max(0, off + q0 - p.window + 1);
+  const int lo = flash_first_key(p, off + q0);
   const int t_begin = lo / FA_BN;
   const int t_end = (hi + FA_BN - 1) / FA_BN;
   const int n_tiles = max(t_end - t_begin, 0);
@@ -277,6 +288,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd_kernel(const __grid_c
     const int r = qd * 32 + lane;                // query row inside the tile
     const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
     const int qpos = off + q0 + r;               // key position of this query
+    const int k_first = flash_first_key(p, qpos), last_first = flash_first_key(p, off + q0 + FA_BM - 1);
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
     uint32_t xph = 0;                            // phase of the pair barrier
@@ -296,7 +308,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd_kernel(const __grid_c
       if (!ok) break;
       tc_fence_after();
       const bool need_mask = (k0 + FA_BN > kv_len) || (p.causal && k0 + FA_BN - 1 > off + q0) ||
-                             (p.window > 0 && k0 <= off + q0 + FA_BM - 1 - p.window);
+                             k0 < last_first;
       // this thread's 64 score columns go to registers with one wait; then the S buffer is free again
       uint32_t v[HC];
 #pragma unroll
@@ -310,7 +322,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd_kernel(const __grid_c
 #pragma unroll
         for (int i = 0; i < HC; ++i) {
           const int kj = k0 + half * HC + i;
-          const bool dead = kj >= kv_len || (p.causal && kj > qpos) || (p.window > 0 && kj <= qpos - p.window);
+          const bool dead = kj >= kv_len || (p.causal && kj > qpos) || kj < k_first;
           if (dead) v[i] = 0xff800000u;   // -inf
         }
       }
@@ -393,8 +405,8 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd_kernel(const __grid_c
     if (ok) {
       tc_fence_after();
       const bool row_ok = q0 + r < q_len;
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* orow = p.out + ((long long)(q_begin + q0 + r) * p.Hq + h) * D;
+      const float inv = l > 0.f && row_ok ? flash_gate(p, q_begin + q0 + r, h) / l : 0.f;
+      __nv_bfloat16* orow = p.out + (long long)(q_begin + q0 + r) * p.ldo + h * D;
 #pragma unroll 1
       for (int c = half * (D / 64); c < (half + 1) * (D / 64); ++c) {   // each warpgroup stores half the columns
         uint32_t v[32];
@@ -469,7 +481,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd2_kernel(const __grid_
   const int kvh = h / (p.Hq / p.Hkv);
   const bool has_b = q0 + FA_BM < q_len;
   // key tiles: both query tiles start at tile a's first visible tile; each stops at its own last one
-  const int lo = p.window > 0 ? max(0, off + q0 - p.window + 1) : 0;
+  const int lo = flash_first_key(p, off + q0);
   const int t_begin = lo / FA_BN;
   const int hi_a = p.causal ? min(kv_len, off + q0 + FA_BM) : kv_len;
   const int hi_b = p.causal ? min(kv_len, off + q0 + 2 * FA_BM) : kv_len;
@@ -643,6 +655,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd2_kernel(const __grid_
     const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
     const int q0x = q0 + x * FA_BM;
     const int qpos = off + q0x + r;
+    const int k_first = flash_first_key(p, qpos), last_first = flash_first_key(p, off + q0x + FA_BM - 1);
     const int n_mine = x == 0 ? n_a : n_b;
     const uint32_t tmem_s = tmem_base + x * FA_BN + lane_addr;
     const uint32_t tmem_o = tmem_base + 2 * FA_BN + x * D + lane_addr;
@@ -656,7 +669,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd2_kernel(const __grid_
       if (!ok) break;
       tc_fence_after();
       const bool need_mask = (k0 + FA_BN > kv_len) || (p.causal && k0 + FA_BN - 1 > off + q0x) ||
-                             (p.window > 0 && k0 <= off + q0x + FA_BM - 1 - p.window);
+                             k0 < last_first;
       uint32_t v[FA_BN];
 #pragma unroll
       for (int c = 0; c < FA_BN / 32; ++c)
@@ -669,7 +682,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd2_kernel(const __grid_
 #pragma unroll
         for (int i = 0; i < FA_BN; ++i) {
           const int kj = k0 + i;
-          const bool dead = kj >= kv_len || (p.causal && kj > qpos) || (p.window > 0 && kj <= qpos - p.window);
+          const bool dead = kj >= kv_len || (p.causal && kj > qpos) || kj < k_first;
           if (dead) v[i] = 0xff800000u;
         }
       }
@@ -740,8 +753,8 @@ __global__ void __launch_bounds__(FA_THREADS, 1) flash_fwd2_kernel(const __grid_
     if (ok && (x == 0 || has_b)) {
       tc_fence_after();
       const bool row_ok = q0x + r < q_len;
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* orow = p.out + ((long long)(q_begin + q0x + r) * p.Hq + h) * D;
+      const float inv = l > 0.f && row_ok ? flash_gate(p, q_begin + q0x + r, h) / l : 0.f;
+      __nv_bfloat16* orow = p.out + (long long)(q_begin + q0x + r) * p.ldo + h * D;
 #pragma unroll 1
       for (int c = 0; c < D / 32; ++c) {
         uint32_t o[32];
@@ -1794,13 +1807,15 @@ extern "C" {
 // ldk, ldv (elements) and cu_k gives the key ranges. Paged mode: k, v are the cache
 // [num_blocks, Hkv, 16, D] (kv_rows = num_blocks), keys of sequence b are the first seq_lens[b]
 // slots of its block table and its queries are the LAST (cu_q[b+1]-cu_q[b]) positions.
-int rb_flash_fwd(const void* q, const void* k, const void* v, void* out, float* lse, const int* cu_q,
-                 const int* cu_k, const int* seq_lens, const int* block_tables, int B, int Tq, int kv_rows,
-                 int Hq, int Hkv, int D, int ldq, int ldk, int ldv, int max_seqlen_q, int max_blocks, int causal,
-                 int window, int paged, float scale, int* status, cudaStream_t stream) {
+// Rows of out are ldo apart. chunk > 0: a query sees the keys of its own run of `chunk` positions; gate: see FlashFwdParams.
+int rb_flash_fwd_ex(const void* q, const void* k, const void* v, void* out, long long ldo, float* lse, const int* cu_q,
+                    const int* cu_k, const int* seq_lens, const int* block_tables, int B, int Tq, int kv_rows,
+                    int Hq, int Hkv, int D, int ldq, int ldk, int ldv, int max_seqlen_q, int max_blocks, int causal,
+                    int window, int chunk, int paged, const float* gate, long long ld_gate, float gate_scale, float scale, int* status,
+                    cudaStream_t stream) {
   using namespace rb;
   if (B <= 0 || Tq <= 0 || max_seqlen_q <= 0) return 0;
-  if ((D != 64 && D != 128) || Hq % Hkv != 0) return -1;
+  if ((D != 64 && D != 128) || Hq % Hkv != 0 || ldo % 8 != 0 || (window > 0 && chunk > 0)) return -1;
   FlashFwdParams p;
   if (tma_map_2d_bf16(&p.q_map, q, Tq, (unsigned long long)Hq * D, ldq, FA_BM) != 0) return -20;
   if (!paged) {
@@ -1824,12 +1839,25 @@ int rb_flash_fwd(const void* q, const void* k, const void* v, void* out, float* 
   p.Tq = Tq;
   p.causal = causal;
   p.window = window;
+  p.chunk = chunk;
+  p.gate = gate;
+  p.ld_gate = ld_gate;
+  p.gate_scale = gate_scale;
+  p.ldo = ldo;
   p.paged = paged;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
   int rc = D == 64 ? launch_flash_fwd<64>(p, max_seqlen_q, B, stream) : launch_flash_fwd<128>(p, max_seqlen_q, B, stream);
   if (rc != 0) return rc;
   return cudaGetLastError() == cudaSuccess ? 0 : -12;
+}
+
+int rb_flash_fwd(const void* q, const void* k, const void* v, void* out, float* lse, const int* cu_q,
+                 const int* cu_k, const int* seq_lens, const int* block_tables, int B, int Tq, int kv_rows,
+                 int Hq, int Hkv, int D, int ldq, int ldk, int ldv, int max_seqlen_q, int max_blocks, int causal,
+                 int window, int paged, float scale, int* status, cudaStream_t stream) {
+  return rb_flash_fwd_ex(q, k, v, out, (long long)Hq * D, lse, cu_q, cu_k, seq_lens, block_tables, B, Tq, kv_rows, Hq, Hkv, D, ldq, ldk, ldv,
+                         max_seqlen_q, max_blocks, causal, window, 0, paged, nullptr, 0, 1.f, scale, status, stream);
 }
 
 // Latent attention, expanded form: see flash_latent_kernel. q [T, H*(DN+64)], k [S, H*DN], rot [S, 64], v [S, H*DV]; the

@@ -53,7 +53,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
   if (sigmoid_router) {
     for (int i = 0; i < per; ++i) {
       const int e = lane + 32 * i;
-      score[i] = e < E ? 1.f / (1.f + __expf(-score[i])) : -INFINITY;
+      score[i] = e < E ? 1.f / (1.f + expf(-score[i])) : -INFINITY;
       choice[i] = e < E ? score[i] + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
     }
     if (n_group > 1 && topk_group < n_group) {
@@ -241,11 +241,12 @@ __global__ void moe_count_kernel(const int* __restrict__ topk_idx, int n, int E,
 }
 
 // Local dispatch: row (t, j) of any 16-byte-multiple width to the next free row of its expert's block (cursor as left by the
-// plan), and the address its result goes to. One warp per pair.
+// plan), and the address its result goes to. One warp per pair. With weights (act: 0 bf16, 1 fp32) the row is multiplied by the
+// pair's weight on the way.
 __global__ void moe_gather_rows_kernel(const uint4* __restrict__ x, long long ld_vec, const int* __restrict__ topk_idx, int n_pairs, int k,
                                        int row_vec, int E, int* __restrict__ cursor, uint4* __restrict__ xp,
                                        unsigned long long* __restrict__ ret, unsigned long long y, long long y_row_bytes, int cap,
-                                       int* status) {
+                                       const float* __restrict__ weights, int act, int* status) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -259,7 +260,22 @@ __global__ void moe_gather_rows_kernel(const uint4* __restrict__ x, long long ld
   if (pos < 0 || pos >= cap) { set_status(status, ST_BAD_INDEX); return; }
   const uint4* src = x + (long long)(i / k) * ld_vec;
   uint4* dst = xp + (long long)pos * row_vec;
-  for (int v = lane; v < row_vec; v += 32) dst[v] = src[v];
+  if (weights == nullptr) {
+    for (int v = lane; v < row_vec; v += 32) dst[v] = src[v];
+  } else {
+    const float w = weights[i];
+    auto pair = [&](uint32_t u) {
+      const float2 f = unpack_bf16x2(u);
+      return pack_bf16x2(w * f.x, w * f.y);
+    };
+    auto single = [&](uint32_t u) { return __float_as_uint(w * __uint_as_float(u)); };
+    for (int v = lane; v < row_vec; v += 32) {
+      uint4 u = src[v];
+      if (act == 0) u = make_uint4(pair(u.x), pair(u.y), pair(u.z), pair(u.w));
+      else u = make_uint4(single(u.x), single(u.y), single(u.z), single(u.w));
+      dst[v] = u;
+    }
+  }
   if (lane == 0) ret[pos] = y + (unsigned long long)i * (unsigned long long)y_row_bytes;
 }
 
@@ -662,12 +678,13 @@ extern "C" int rb_moe_combine(const void* y, const float* w, int T, int k, int d
 // ---------------------------------------------------------------- local expert layer of layer-stack models (ops/experts.py)
 extern "C" void rb_moe_set_pdl(int on) { rb::pdl_enabled() = on != 0; }
 
-// Softmax router on logits with a row stride, chosen scores divided by their sum, histogram added into counts.
-extern "C" int rb_experts_route(const float* logits, long long ld, int T, int E, int k, int* topk_idx, float* topk_w, int* counts,
-                                cudaStream_t s) {
+// Router on logits with a row stride: softmax or sigmoid scores, the chosen ones divided by their sum or not; histogram added
+// into counts.
+extern "C" int rb_experts_route(const float* logits, long long ld, int T, int E, int k, int sigmoid, int normalize, int* topk_idx, float* topk_w,
+                                int* counts, cudaStream_t s) {
   if (T <= 0) return 0;
   if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E || counts == nullptr) return -1;
-  return launch_kernel(moe_route_kernel, dim3((T + 7) / 8), dim3(256), 0, s, logits, ld, nullptr, T, E, k, 0, 1, 1.f, topk_idx, topk_w, counts,
+  return launch_kernel(moe_route_kernel, dim3((T + 7) / 8), dim3(256), 0, s, logits, ld, nullptr, T, E, k, sigmoid, normalize, 1.f, topk_idx, topk_w, counts,
                        1, 1) == cudaSuccess ? 0 : -11;
 }
 // Offsets, tile tables and dispatch bases from the histogram, which is zeroed again.
@@ -678,12 +695,12 @@ extern "C" int rb_experts_plan(int* counts, int E, int* expert_offset, int n_gu,
                        n_dn, bn_dn, (int4*)tiles_dn, ntiles_dn, max_tiles, status, 0, cursor, counts) == cudaSuccess ? 0 : -11;
 }
 extern "C" int rb_experts_gather(const void* x, long long ld_bytes, const int* topk_idx, int T, int k, int row_bytes, int E, int* cursor, void* xp,
-                                 void* ret, void* y, long long y_row_bytes, int cap, int* status, cudaStream_t s) {
+                                 void* ret, void* y, long long y_row_bytes, int cap, const float* weights, int act, int* status, cudaStream_t s) {
   if (T <= 0) return 0;
   if (ld_bytes % 16 != 0 || row_bytes % 16 != 0) return -1;
   const int n = T * k;
   return launch_kernel(moe_gather_rows_kernel, dim3((n + 7) / 8), dim3(256), 0, s, (const uint4*)x, ld_bytes / 16, topk_idx, n, k, row_bytes / 16, E,
-                       cursor, (uint4*)xp, (unsigned long long*)ret, (unsigned long long)y, y_row_bytes, cap, status) == cudaSuccess ? 0 : -11;
+                       cursor, (uint4*)xp, (unsigned long long*)ret, (unsigned long long)y, y_row_bytes, cap, weights, act, status) == cudaSuccess ? 0 : -11;
 }
 
 // ---------------------------------------------------------------- training (expert-grouped rows, padded to 64)

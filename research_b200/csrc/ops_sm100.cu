@@ -301,7 +301,8 @@ __device__ __forceinline__ void store_act4(__nv_bfloat16* p, float4 v) {
 }
 
 // One pass over the fp32 residual stream between two layers, a CTA per row:
-//   x += y1 + y2 + sum_j w[j] e[row * k + j]     (absent terms are null; nothing is written back when all are)
+//   x += mult * (y1 + y2 + sum_j w[j] e[row * k + j] + side / rms(side) * side_weight)
+//                                                (absent terms are null; nothing is written back when all are; w null: ones)
 //   copy = x in the activation type,  h = x / rms(x) * weight
 // rows != null: h[i] comes from row rows[i] (no update). Columns are padded to a multiple of 4 with zeros.
 struct StreamNormParams {
@@ -319,9 +320,12 @@ struct StreamNormParams {
   void* h;
   long long ldh;
   const float* weight;
+  const float* side;
+  long long ld_side;
+  const float* side_weight;
   const int* rows;
   int num_src_rows, d, dp;
-  float eps;
+  float eps, mult;
   int* status;
 };
 
@@ -338,11 +342,19 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamNormParams
     if (xr < 0 || xr >= p.num_src_rows) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); xr = 0; }
   }
   float* x = p.x + xr * p.ldx;
-  const bool update = p.y1 != nullptr || p.y2 != nullptr || p.e != nullptr;
+  const bool update = p.y1 != nullptr || p.y2 != nullptr || p.e != nullptr || p.side != nullptr;
   const TA* e = reinterpret_cast<const TA*>(p.e) + r * p.k * p.lde;
-  float ss = 0.f;
+  float ss = 0.f, side_scale = 0.f;
+  if (p.side != nullptr) {
+    float sq = 0.f;
+    for (int c = threadIdx.x * 4; c < p.dp; c += blockDim.x * 4) {
+      const float4 y = *reinterpret_cast<const float4*>(p.side + r * p.ld_side + c);
+      sq += y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+    }
+    side_scale = 1.f / sqrtf(block_sum(sq, red) / (float)p.d + p.eps);
+  }
   for (int c = threadIdx.x * 4; c < p.dp; c += blockDim.x * 4) {
-    float4 v = *reinterpret_cast<const float4*>(x + c);
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (p.y1 != nullptr) {
       const float4 y = *reinterpret_cast<const float4*>(p.y1 + r * p.ldy + c);
       v.x += y.x; v.y += y.y; v.z += y.z; v.w += y.w;
@@ -354,12 +366,19 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamNormParams
     if (p.e != nullptr) {
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
       for (int j = 0; j < p.k; ++j) {
-        const float w = __ldg(p.w + r * p.k + j);
+        const float w = p.w != nullptr ? __ldg(p.w + r * p.k + j) : 1.f;
         const float4 y = load_act4(e + j * p.lde + c);
         a.x = fmaf(w, y.x, a.x); a.y = fmaf(w, y.y, a.y); a.z = fmaf(w, y.z, a.z); a.w = fmaf(w, y.w, a.w);
       }
       v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
     }
+    if (p.side != nullptr) {
+      const float4 y = *reinterpret_cast<const float4*>(p.side + r * p.ld_side + c);
+      const float4 w = *reinterpret_cast<const float4*>(p.side_weight + c);
+      v.x += y.x * side_scale * w.x; v.y += y.y * side_scale * w.y; v.z += y.z * side_scale * w.z; v.w += y.w * side_scale * w.w;
+    }
+    const float4 old = *reinterpret_cast<const float4*>(x + c);
+    v.x = fmaf(p.mult, v.x, old.x); v.y = fmaf(p.mult, v.y, old.y); v.z = fmaf(p.mult, v.z, old.z); v.w = fmaf(p.mult, v.w, old.w);
     if (update) *reinterpret_cast<float4*>(x + c) = v;
     if (p.copy != nullptr) store_act4(reinterpret_cast<TA*>(p.copy) + r * p.ldc + c, v);
     sn_row[c >> 2] = v;
@@ -418,9 +437,28 @@ __global__ void layernorm_kernel(const float* __restrict__ y, long long ldy, flo
   }
 }
 
-// Clamped gated unit: g = min(gate, limit), u = clamp(up, +-limit), out = g sigmoid(1.702 g) (u + 1). gate|up packed
-// as [T, 2F].
+// a[t, c] = gelu_tanh(z[t, c]) * table[ids[t], col0 + c]: the gate of a per-layer token embedding.
+template <typename TA>
+__global__ void token_side_kernel(const float* __restrict__ z, long long ldz, const int* __restrict__ ids, const TA* __restrict__ table,
+                                  long long ldt, int col0, TA* __restrict__ a, long long lda, int n, int T, int vocab, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long total = (long long)T * n;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / n;
+    const int c = (int)(i - t * n);
+    int id = ids[t];
+    if (id < 0 || id >= vocab) { set_status(status, ST_BAD_INDEX); id = 0; }
+    const float x = z[t * ldz + c];
+    const float g = 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+    a[t * lda + c] = to_act<TA>(g * from_act(table[(long long)id * ldt + col0 + c]));
+  }
+}
+
+// Gated unit on gate|up packed as [T, 2F]. limit > 0: g = min(gate, limit), u = clamp(up, +-limit), out = g sigmoid(1.702 g) (u + 1);
+// otherwise out = silu(gate) * up.
 __device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
+  if (!(limit > 0.f)) return g / (1.f + expf(-g)) * u;
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
@@ -773,14 +811,27 @@ extern "C" int rb_stream_embed(const int* ids, const void* table, long long ldt,
 }
 
 extern "C" int rb_stream_norm(float* x, long long ldx, const float* y1, const float* y2, long long ldy, const void* e, const float* w,
-                              long long lde, int k, void* copy, long long ldc, void* h, long long ldh, const float* weight, const int* rows,
-                              int num_src_rows, int dtype, int n, int d, int dp, float eps, int* status, cudaStream_t stream) {
-  const bool update = y1 != nullptr || y2 != nullptr || e != nullptr;
-  if (n <= 0 || d <= 0 || dp < d || dp % 4 != 0 || dp > 12288 || (rows != nullptr && update) || (ldx | ldy | lde | ldc | ldh) % 4 != 0) return -1;
-  const StreamNormParams p{x, ldx, y1, y2, ldy, e, w, lde, k, copy, ldc, h, ldh, weight, rows, num_src_rows, d, dp, eps, status};
+                              long long lde, int k, const float* side, long long ld_side, const float* side_weight, float mult, void* copy,
+                              long long ldc, void* h, long long ldh, const float* weight, const int* rows, int num_src_rows, int dtype, int n, int d,
+                              int dp, float eps, int* status, cudaStream_t stream) {
+  const bool update = y1 != nullptr || y2 != nullptr || e != nullptr || side != nullptr;
+  if (n <= 0 || d <= 0 || dp < d || dp % 4 != 0 || dp > 12288 || (rows != nullptr && update) || (ldx | ldy | lde | ldc | ldh | ld_side) % 4 != 0) return -1;
+  const StreamNormParams p{x, ldx, y1, y2, ldy, e, w, lde, k, copy, ldc, h, ldh, weight, side, ld_side, side_weight, rows, num_src_rows, d, dp, eps, mult,
+                           status};
   const int threads = dp <= 512 ? 128 : 256;
   cudaError_t err;
   RB_ACT_DISPATCH(dtype, err = launch_kernel(stream_norm_kernel<TA>, dim3(n), dim3(threads), (size_t)dp * 4, stream, p);)
+  return err == cudaSuccess ? 0 : -11;
+}
+
+extern "C" int rb_token_side(const float* z, long long ldz, const int* ids, const void* table, long long ldt, int col0, void* a, long long lda, int n,
+                             int T, int vocab, int dtype, int* status, cudaStream_t stream) {
+  if (T <= 0 || n <= 0) return -1;
+  long long grid = ((long long)T * n + 255) / 256;
+  if (grid > 148 * 16) grid = 148 * 16;
+  cudaError_t err;
+  RB_ACT_DISPATCH(dtype, err = launch_kernel(token_side_kernel<TA>, dim3((unsigned)grid), dim3(256), 0, stream, z, ldz, ids, (const TA*)table, ldt,
+                                             col0, (TA*)a, lda, n, T, vocab, status);)
   return err == cudaSuccess ? 0 : -11;
 }
 

@@ -1,6 +1,7 @@
 // Recurrent mixers with a matrix state per head, for sm_100a.
 //
 //   S_t = a_t S_(t-1) + b_t k_t v_t^T,   o_t = S_t^T q_t        (see ops/recurrent.py)
+//   S_t = diag(w_t) S_(t-1) + k_t v_t^T, o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t        (time mixing: a decay per key channel)
 //
 //   scan        token by token: short portions and long ones of the exact mode. One CTA per (sequence, head, 32 value channels);
 //               the state tile stays in registers over the tokens of the portion.
@@ -14,6 +15,7 @@
 // own copy of n and m, so that the CTAs of a head never share anything they write. Only the first `dk` of the KP rows are
 // touched. A slot holds whatever its last user left: a portion that starts at position 0 starts from zero.
 #include "common.cuh"
+#include "history.cuh"
 
 namespace rb {
 
@@ -51,13 +53,20 @@ struct ScanParams {
   float* out;              // [T, ldo]
   long long ldo;
   int H, dk, KP, VP, num_slots, gated, rows;
+  const float* z;          // [T, ldz] time mixing: w = exp(-exp(z + w0)), column h * KP + key channel
+  long long ldz;
+  const float* w0;         // [H * KP]
+  const float* bonus;      // [H * KP]
   int* status;
 };
 
-// NR: key rows held by a thread (dk <= NR * SC_ROWS)
-template <typename T, int NR>
+__device__ __forceinline__ float channel_decay(float z) { return expf(-expf(z)); }
+
+// NR: key rows held by a thread (dk <= NR * SC_ROWS); MIX: time mixing
+template <typename T, int NR, bool MIX>
 __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanParams p) {
   __shared__ float qs[NR * SC_ROWS], ks[NR * SC_ROWS], vs[SC_COLS];
+  __shared__ float ws[MIX ? NR * SC_ROWS : 1];
   __shared__ float red[SC_THREADS / 32][SC_COLS];
   __shared__ float red_n[SC_THREADS / 32];
   pdl_launch_dependents();
@@ -94,12 +103,17 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
   }
   float m = fresh || !p.gated ? 0.f : p.m[unit];
   const T* proj = reinterpret_cast<const T*>(p.proj);
-  const float decay = p.gated ? 0.f : p.decay[h];
+  const float decay = p.gated || MIX ? 0.f : p.decay[h];
+  float bonus[MIX ? NR : 1];
+  if (MIX)
+#pragma unroll
+    for (int i = 0; i < NR; ++i) bonus[i] = r0 + i * SC_ROWS < p.dk ? p.bonus[h * p.KP + r0 + i * SC_ROWS] : 0.f;
   for (int t = t0; t < t1; ++t) {
     const T* row = proj + t * p.ld;
     for (int i = tid; i < p.dk; i += SC_THREADS) {
       qs[i] = to_f<T>(row[p.q_col + h * p.KP + i]) * p.q_scale;
       ks[i] = to_f<T>(row[p.k_col + h * p.KP + i]);
+      if (MIX) ws[i] = channel_decay(p.z[t * p.ldz + h * p.KP + i] + p.w0[h * p.KP + i]);
     }
     if (tid < SC_COLS) {
       vs[tid] = to_f<T>(row[p.v_col + h * p.VP + tile * SC_COLS + tid]);
@@ -121,7 +135,19 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
       const int r = r0 + i * SC_ROWS;
-      if (r < p.dk) {
+      if (MIX && r < p.dk) {
+        const float k = ks[r], q = qs[r], d = ws[r], u = bonus[MIX ? i : 0];
+        const float4 kv = make_float4(k * v.x, k * v.y, k * v.z, k * v.w);
+        acc.x = fmaf(q, fmaf(u, kv.x, S[i].x), acc.x);
+        acc.y = fmaf(q, fmaf(u, kv.y, S[i].y), acc.y);
+        acc.z = fmaf(q, fmaf(u, kv.z, S[i].z), acc.z);
+        acc.w = fmaf(q, fmaf(u, kv.w, S[i].w), acc.w);
+        S[i].x = fmaf(d, S[i].x, kv.x);
+        S[i].y = fmaf(d, S[i].y, kv.y);
+        S[i].z = fmaf(d, S[i].z, kv.z);
+        S[i].w = fmaf(d, S[i].w, kv.w);
+      }
+      if (!MIX && r < p.dk) {
         const float kw = w * ks[r], q = qs[r];
         S[i].x = fmaf(a, S[i].x, kw * v.x);
         S[i].y = fmaf(a, S[i].y, kw * v.y);
@@ -166,16 +192,16 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
   if (p.gated && tid == 0) p.m[unit] = m;
 }
 
-template <typename T>
+template <typename T, bool MIX>
 static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
   const dim3 grid(p.VP / SC_COLS, p.H, B);
   const int need = (p.dk + SC_ROWS - 1) / SC_ROWS;
   cudaError_t e;
-  if (need <= 1) e = launch_kernel(recurrent_scan_kernel<T, 1>, grid, dim3(SC_THREADS), 0, stream, p);
-  else if (need <= 2) e = launch_kernel(recurrent_scan_kernel<T, 2>, grid, dim3(SC_THREADS), 0, stream, p);
-  else if (need <= 4) e = launch_kernel(recurrent_scan_kernel<T, 4>, grid, dim3(SC_THREADS), 0, stream, p);
-  else if (need <= 8) e = launch_kernel(recurrent_scan_kernel<T, 8>, grid, dim3(SC_THREADS), 0, stream, p);
-  else if (need <= 16) e = launch_kernel(recurrent_scan_kernel<T, 16>, grid, dim3(SC_THREADS), 0, stream, p);
+  if (need <= 1) e = launch_kernel(recurrent_scan_kernel<T, 1, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
+  else if (need <= 2) e = launch_kernel(recurrent_scan_kernel<T, 2, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
+  else if (need <= 4) e = launch_kernel(recurrent_scan_kernel<T, 4, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
+  else if (need <= 8) e = launch_kernel(recurrent_scan_kernel<T, 8, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
+  else if (need <= 16) e = launch_kernel(recurrent_scan_kernel<T, 16, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
   else return -1;
   return e == cudaSuccess ? 0 : -11;
 }
@@ -198,10 +224,11 @@ __device__ __forceinline__ void bulk_store(void* dst, uint32_t src, uint32_t byt
   asm volatile("cp.async.bulk.commit_group;" ::: "memory");
 }
 
-template <typename T>
+template <typename T, bool MIX>
 __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const ScanParams p, int B, int units) {
   extern __shared__ __align__(128) uint8_t smem_raw[];       // RD_STAGES x [dk, 32] fp32, then the sequences' slots
   __shared__ float qs[RD_MAX_DK], ks[RD_MAX_DK];
+  __shared__ float ws[MIX ? RD_MAX_DK : 1], us[MIX ? RD_MAX_DK : 1];
   __shared__ __align__(16) float vs[SC_COLS];
   __shared__ __align__(16) float red[RD_THREADS / 32][SC_COLS];
   __shared__ float red_n[RD_THREADS / 32];
@@ -250,6 +277,7 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
   if (tid == 0)
     for (int i = 0; i < RD_STAGES - 1; ++i) load(i);
   float q[RD_VEC], k[RD_VEC], n[RD_VEC], v = 0.f, gi = 0.f, gf = 0.f, m0 = 0.f;
+  float z[MIX ? RD_VEC : 1], bonus[MIX ? RD_VEC : 1];
   Unit x{};
   auto fetch = [&](int u) {
     x = unit_of(u);
@@ -263,6 +291,10 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
         q[i] = to_f<T>(row[p.q_col + x.h * p.KP + r]) * p.q_scale;
         k[i] = to_f<T>(row[p.k_col + x.h * p.KP + r]);
         if (p.gated) n[i] = nt[r];
+        if (MIX) {
+          z[i] = p.z[x.b * p.ldz + x.h * p.KP + r] + p.w0[x.h * p.KP + r];
+          bonus[i] = p.bonus[x.h * p.KP + r];
+        }
       }
     }
     if (tid < SC_COLS) v = to_f<T>(row[p.v_col + x.h * p.VP + x.tile * SC_COLS + tid]);
@@ -279,14 +311,14 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
     const Unit cur = x;
     const bool zero = cur.fresh;
     if (zero) m0 = n[0] = n[1] = n[2] = 0.f;
-    float a, w = 1.f, m = 0.f;
+    float a = 0.f, w = 1.f, m = 0.f;
     if (p.gated) {
       gi = p.cap * tanhf((gi + p.bias_i[cur.h]) / p.cap);
       gf = log_sigmoid_f(p.cap * tanhf((gf + p.bias_f[cur.h]) / p.cap));
       m = fmaxf(gf + m0, gi);
       a = expf(gf + m0 - m);
       w = expf(gi - m);
-    } else {
+    } else if (!MIX) {
       a = p.decay[cur.h];
     }
     const long long si = state_index(cur);
@@ -298,6 +330,7 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
         const float kw = w * k[i];
         qs[r] = q[i];
         ks[r] = kw;
+        if (MIX) { ws[r] = channel_decay(z[i]); us[r] = bonus[i]; }
         if (p.gated) {
           const float nn = fmaf(a, n[i], kw);
           nq = fmaf(q[i], nn, nq);
@@ -319,14 +352,24 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
     for (int r = r0; r < p.dk; r += RD_THREADS / 8) {
       float4 s = zero ? make_float4(0.f, 0.f, 0.f, 0.f) : S[r * (SC_COLS / 4) + c4];
       const float kw = ks[r], qr = qs[r];
+      if (MIX) {                                             // the state in front of the token, and the token with its bonus
+        const float bo = us[r];
+        acc.x = fmaf(qr, fmaf(bo, kw * vv.x, s.x), acc.x);
+        acc.y = fmaf(qr, fmaf(bo, kw * vv.y, s.y), acc.y);
+        acc.z = fmaf(qr, fmaf(bo, kw * vv.z, s.z), acc.z);
+        acc.w = fmaf(qr, fmaf(bo, kw * vv.w, s.w), acc.w);
+        a = ws[r];
+      }
       s.x = fmaf(a, s.x, kw * vv.x);
       s.y = fmaf(a, s.y, kw * vv.y);
       s.z = fmaf(a, s.z, kw * vv.z);
       s.w = fmaf(a, s.w, kw * vv.w);
-      acc.x = fmaf(qr, s.x, acc.x);
-      acc.y = fmaf(qr, s.y, acc.y);
-      acc.z = fmaf(qr, s.z, acc.z);
-      acc.w = fmaf(qr, s.w, acc.w);
+      if (!MIX) {
+        acc.x = fmaf(qr, s.x, acc.x);
+        acc.y = fmaf(qr, s.y, acc.y);
+        acc.z = fmaf(qr, s.z, acc.z);
+        acc.w = fmaf(qr, s.w, acc.w);
+      }
       S[r * (SC_COLS / 4) + c4] = s;
     }
     fence_proxy_async_smem();
@@ -366,7 +409,7 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
   }
 }
 
-template <typename T>
+template <typename T, bool MIX>
 static int launch_decode(const ScanParams& p, int B, cudaStream_t stream) {
   static int sms[64] = {};
   int dev = 0;
@@ -375,13 +418,13 @@ static int launch_decode(const ScanParams& p, int B, cudaStream_t stream) {
   if (sms[dev] == 0) {
     int n = 0;
     if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess ||
-        cudaFuncSetAttribute(recurrent_decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, RD_STAGES * RD_MAX_DK * SC_COLS * 4 + RD_MAX_B * 4) != cudaSuccess)
+        cudaFuncSetAttribute(recurrent_decode_kernel<T, MIX>, cudaFuncAttributeMaxDynamicSharedMemorySize, RD_STAGES * RD_MAX_DK * SC_COLS * 4 + RD_MAX_B * 4) != cudaSuccess)
       return -10;
     sms[dev] = n;
   }
   const int per_sm = 200 * 1024 / (smem + 7 * 1024) > 6 ? 6 : 200 * 1024 / (smem + 7 * 1024);
   const int units = B * p.H * (p.VP / SC_COLS), grid = units < sms[dev] * per_sm ? units : sms[dev] * per_sm;
-  return launch_kernel(recurrent_decode_kernel<T>, dim3(grid), dim3(RD_THREADS), smem, stream, p, B, units) == cudaSuccess ? 0 : -11;
+  return launch_kernel(recurrent_decode_kernel<T, MIX>, dim3(grid), dim3(RD_THREADS), smem, stream, p, B, units) == cudaSuccess ? 0 : -11;
 }
 
 // ------------------------------------------------------------------------------------------
@@ -1039,11 +1082,11 @@ static int launch_chunks(const ChunkParams& p, int n_chunks, int n_seq, cudaStre
 }
 
 // ------------------------------------------------------------------------------------------
-// out = o / rms * weight * sigmoid(gate). One CTA per token; a warp takes whole heads. Padding channels of o are zero.
+// out = o / rms * weight * sigmoid(gate), or silu(gate). One CTA per token; a warp takes whole heads. Padding channels of o are zero.
 template <typename T>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ weight,
                                                          const T* __restrict__ gate, long long ldg, T* __restrict__ out, long long ldy,
-                                                         int H, int dv, int VP, int per_head, float eps) {
+                                                         int H, int dv, int VP, int per_head, int silu, float eps) {
   __shared__ float part[8];
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -1079,10 +1122,72 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
       const float4 v = *reinterpret_cast<const float4*>(x + c);
       const float4 w = *reinterpret_cast<const float4*>(weight + c);
       const T* g = gate + t * ldg + c;
-      const float y0 = v.x * rs * w.x * sigmoid_f(to_f<T>(g[0])), y1 = v.y * rs * w.y * sigmoid_f(to_f<T>(g[1]));
-      const float y2 = v.z * rs * w.z * sigmoid_f(to_f<T>(g[2])), y3 = v.w * rs * w.w * sigmoid_f(to_f<T>(g[3]));
+      auto gated = [&](float z) { return silu ? z * sigmoid_f(z) : sigmoid_f(z); };
+      const float y0 = v.x * rs * w.x * gated(to_f<T>(g[0])), y1 = v.y * rs * w.y * gated(to_f<T>(g[1]));
+      const float y2 = v.z * rs * w.z * gated(to_f<T>(g[2])), y3 = v.w * rs * w.w * gated(to_f<T>(g[3]));
       if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(out + t * ldy + c) = make_float4(y0, y1, y2, y3);
       else *reinterpret_cast<uint2*>(out + t * ldy + c) = make_uint2(pack_bf16x2(y0, y1), pack_bf16x2(y2, y3));
+    }
+  }
+}
+
+// mix[s][t] = h_t + (h_(t-1) - h_t) mu[s] for the `mixes` projections of a token; 8 channels per thread. With one row per sequence
+// (rows.cu_q null) the history moves on in the same pass.
+template <typename T>
+__global__ void __launch_bounds__(256) token_shift_kernel(const T* __restrict__ h, long long ld, const float* __restrict__ mu, int mixes, T* __restrict__ out,
+                                                          long long step, long long ldo, T* __restrict__ hist, const History rows, int width, int n,
+                                                          int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int V = 16 / sizeof(T);
+  union Vec { uint4 u[8 / V]; T e[8]; };
+  const int per = width / 8;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < (long long)n * per; i += (long long)gridDim.x * blockDim.x) {
+    const int t = (int)(i / per), c = (int)(i % per) * 8;
+    const RowPlace place = row_place(rows, t, status);
+    const T* back = row_before(place, 1, h, ld, t, (const T*)hist, 1, width);
+    Vec x, y;
+#pragma unroll
+    for (int j = 0; j < 8 / V; ++j) {
+      x.u[j] = reinterpret_cast<const uint4*>(h + t * ld + c)[j];
+      y.u[j] = back != nullptr ? reinterpret_cast<const uint4*>(back + c)[j] : make_uint4(0u, 0u, 0u, 0u);
+    }
+    if (rows.cu_q == nullptr && place.slot >= 0)
+#pragma unroll
+      for (int j = 0; j < 8 / V; ++j) reinterpret_cast<uint4*>(hist + (long long)place.slot * width + c)[j] = x.u[j];
+    float a[8], d[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) { a[j] = to_f<T>(x.e[j]); d[j] = to_f<T>(y.e[j]) - a[j]; }
+    for (int s = 0; s < mixes; ++s) {
+      const float4* m4 = reinterpret_cast<const float4*>(mu + (long long)s * width + c);
+      const float4 m0 = m4[0], m1 = m4[1];
+      const float m[8] = {m0.x, m0.y, m0.z, m0.w, m1.x, m1.y, m1.z, m1.w};
+      Vec r;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float v = fmaf(d[j], m[j], a[j]);
+        if constexpr (sizeof(T) == 4) r.e[j] = v; else r.e[j] = __float2bfloat16_rn(v);
+      }
+#pragma unroll
+      for (int j = 0; j < 8 / V; ++j) reinterpret_cast<uint4*>(out + s * step + t * ldo + c)[j] = r.u[j];
+    }
+  }
+}
+
+// tanh of fp32 rows as operand of a product that is to lose nothing: fp32 as it is, bf16 as two parts side by side.
+__global__ void tanh_parts_kernel(const float* __restrict__ x, int n, __nv_bfloat16* __restrict__ parts, float* __restrict__ whole, long long total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const float v = tanhf(x[i]);
+    if (whole != nullptr) {
+      whole[i] = v;
+    } else {
+      const long long r = i / n;
+      const int c = (int)(i - r * n);
+      const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+      parts[r * 2 * n + c] = hi;
+      parts[r * 2 * n + n + c] = __float2bfloat16_rn(v - __bfloat162float(hi));
     }
   }
 }
@@ -1093,19 +1198,55 @@ using namespace rb;
 
 extern "C" {
 
+// h [n, ld] -> out [mixes][n rows of ldo, `step` apart]; hist [num_slots, width]. cu_q null: one row per sequence.
+int rb_token_shift(const void* h, long long ld, const float* mu, int mixes, void* out, long long step, long long ldo, void* hist, const int* cu_q,
+                   const int* positions, const int* slots, int B, int num_slots, int width, int n, int dtype, int* status, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (width % 8 != 0 || ld % 8 != 0 || ldo % 8 != 0 || step % 8 != 0 || mixes <= 0 || B <= 0) return -1;
+  const History rows{cu_q, positions, slots, B, 1, num_slots};
+  long long grid = ((long long)n * (width / 8) + 255) / 256;
+  if (grid > 148 * 16) grid = 148 * 16;
+  cudaError_t e;
+  if (dtype == 0) {
+    e = launch_kernel(token_shift_kernel<__nv_bfloat16>, dim3((unsigned)grid), dim3(256), 0, stream, (const __nv_bfloat16*)h, ld, mu, mixes,
+                      (__nv_bfloat16*)out, step, ldo, (__nv_bfloat16*)hist, rows, width, n, status);
+    if (e == cudaSuccess && cu_q != nullptr) e = launch_history_update((const __nv_bfloat16*)h, ld, rows, (__nv_bfloat16*)hist, width, stream);
+  } else {
+    e = launch_kernel(token_shift_kernel<float>, dim3((unsigned)grid), dim3(256), 0, stream, (const float*)h, ld, mu, mixes, (float*)out, step, ldo,
+                      (float*)hist, rows, width, n, status);
+    if (e == cudaSuccess && cu_q != nullptr) e = launch_history_update((const float*)h, ld, rows, (float*)hist, width, stream);
+  }
+  return e == cudaSuccess ? 0 : -11;
+}
+
+// x [rows, n] fp32 -> tanh as fp32 [rows, n] (whole) or as bf16 [rows, 2n] (high parts, then what they lack).
+int rb_tanh_parts(const float* x, int n, void* parts, float* whole, int rows, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (n <= 0 || (parts == nullptr) == (whole == nullptr)) return -1;
+  const long long total = (long long)rows * n;
+  long long grid = (total + 255) / 256;
+  if (grid > 148 * 8) grid = 148 * 8;
+  return launch_kernel(tanh_parts_kernel, dim3((unsigned)grid), dim3(256), 0, stream, x, n, (__nv_bfloat16*)parts, whole, total) == cudaSuccess ? 0 : -11;
+}
+
 void rb_recurrent_set_pdl(int on) { rb::pdl_enabled() = on != 0; }
 
 int rb_recurrent_scan(const void* proj, long long ld, int q_col, int k_col, int v_col, const float* small, long long ld_small, const float* decay,
                       const float* bias_i, const float* bias_f, float cap, float q_scale, float* s, float* n, float* m, const int* slots,
                       const int* cu_q, const int* seq_lens, float* out, long long ldo, int H, int dk, int KP, int VP, int B, int num_slots,
-                      int gated, int rows, int dtype, int* status, cudaStream_t stream) {
+                      int gated, int rows, const float* z, long long ldz, const float* w0, const float* bonus, int dtype, int* status,
+                      cudaStream_t stream) {
   if (B <= 0) return 0;
-  if (H <= 0 || H > 65535 || B > 65535 || dk <= 0 || dk > KP || VP % SC_COLS != 0 || (gated ? small == nullptr : decay == nullptr)) return -1;
+  const bool mix = z != nullptr;
+  if (H <= 0 || H > 65535 || B > 65535 || dk <= 0 || dk > KP || VP % SC_COLS != 0) return -1;
+  if (mix ? (gated || w0 == nullptr || bonus == nullptr) : (gated ? small == nullptr : decay == nullptr)) return -1;
   const ScanParams p{proj, ld, q_col, k_col, v_col, small, ld_small, decay, bias_i, bias_f, cap, q_scale, s, n, m, slots, cu_q, seq_lens,
-                     out, ldo, H, dk, KP, VP, num_slots, gated, rows, status};
+                     out, ldo, H, dk, KP, VP, num_slots, gated, rows, z, ldz, w0, bonus, status};
   if (cu_q == nullptr && dk <= RD_MAX_DK && B <= RD_MAX_B)
-    return dtype == 0 ? launch_decode<__nv_bfloat16>(p, B, stream) : launch_decode<float>(p, B, stream);
-  return dtype == 0 ? launch_scan<__nv_bfloat16>(p, B, stream) : launch_scan<float>(p, B, stream);
+    return mix ? (dtype == 0 ? launch_decode<__nv_bfloat16, true>(p, B, stream) : launch_decode<float, true>(p, B, stream))
+               : (dtype == 0 ? launch_decode<__nv_bfloat16, false>(p, B, stream) : launch_decode<float, false>(p, B, stream));
+  return mix ? (dtype == 0 ? launch_scan<__nv_bfloat16, true>(p, B, stream) : launch_scan<float, true>(p, B, stream))
+             : (dtype == 0 ? launch_scan<__nv_bfloat16, false>(p, B, stream) : launch_scan<float, false>(p, B, stream));
 }
 
 // Workspace of the chunked form in bytes.
@@ -1150,16 +1291,16 @@ int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, in
 }
 
 int rb_gated_norm(const float* o, long long ldo, const float* weight, const void* gate, long long ldg, void* out, long long ldy, int H, int dv,
-                  int VP, int per_head, int T, int dtype, float eps, cudaStream_t stream) {
+                  int VP, int per_head, int silu, int T, int dtype, float eps, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (VP % 4 != 0 || ldo % 4 != 0 || ldy % 4 != 0) return -1;
   cudaError_t e;
   if (dtype == 0)
     e = launch_kernel(gated_norm_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, o, ldo, weight, (const __nv_bfloat16*)gate, ldg,
-                      (__nv_bfloat16*)out, ldy, H, dv, VP, per_head, eps);
+                      (__nv_bfloat16*)out, ldy, H, dv, VP, per_head, silu, eps);
   else
     e = launch_kernel(gated_norm_kernel<float>, dim3(T), dim3(256), 0, stream, o, ldo, weight, (const float*)gate, ldg, (float*)out, ldy, H, dv, VP,
-                      per_head, eps);
+                      per_head, silu, eps);
   return e == cudaSuccess ? 0 : -11;
 }
 

@@ -5,11 +5,15 @@ every layer of its kind (``make`` / ``load``), the cache or state of every run o
 activations (``allocate``), plans a step for all its layers at once (``plan``) and runs one layer (``forward``).
 """
 
-from ...models.stack import ClampedGluSpec, ExpertsSpec, KeyValueAttentionSpec, LatentAttentionSpec, LightningSpec, MatrixMemorySpec
+from ...models.stack import (ClampedGluSpec, ExpertsSpec, GluSpec, GroupedAttentionSpec, KeyValueAttentionSpec, LatentAttentionSpec, LightningSpec,
+                             MatrixMemorySpec, ParallelSpec, TimeMixSpec)
 from .feedforward import DensePart, ExpertsPart
+from .grouped import GroupedPart
 from .keyvalue import KeyValuePart
 from .latent import LatentPart
-from .recurrent import RecurrentPart
+from .parallel import ParallelPart
+from .recurrent import RecurrentPart, TimeMixPart
 
-MIXER_PARTS = {LatentAttentionSpec: LatentPart, KeyValueAttentionSpec: KeyValuePart, LightningSpec: RecurrentPart, MatrixMemorySpec: RecurrentPart}
-FEED_FORWARD_PARTS = {ClampedGluSpec: DensePart, ExpertsSpec: ExpertsPart}
+MIXER_PARTS = {LatentAttentionSpec: LatentPart, KeyValueAttentionSpec: KeyValuePart, LightningSpec: RecurrentPart, MatrixMemorySpec: RecurrentPart,
+               GroupedAttentionSpec: GroupedPart, TimeMixSpec: TimeMixPart, ParallelSpec: ParallelPart}
+FEED_FORWARD_PARTS = {ClampedGluSpec: DensePart, GluSpec: DensePart, ExpertsSpec: ExpertsPart}

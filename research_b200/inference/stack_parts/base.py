@@ -25,6 +25,7 @@ class Part:
     def __init__(self, runner):
         self.r = weakref.proxy(runner)       # no cycle: the runner's graphs go when its engine does
         self.layers: list[Any] = []          # weights made so far
+        self._planned: tuple = (None, None)
         self.specs: list[Any] = []
 
     # ---- sizing, before a runner exists
@@ -67,13 +68,19 @@ class Part:
     def plan(self, b) -> Any:
         return None
 
+    def planned(self, b) -> Any:
+        """``plan(b)``, made once per batch (a part may also belong to another one)."""
+        if self._planned[0] is not b:
+            self._planned = (b, self.plan(b))
+        return self._planned[1]
+
     def project(self, w, inp: torch.Tensor, tail: torch.Tensor | None) -> None:
         """First half of a mixer: its projections of ``inp``, and the narrow one into ``tail`` (fp32)."""
 
 
 def load_heads(dst: torch.Tensor, src: torch.Tensor, heads: int, dim: int, padded: int) -> None:
     """``src [heads*dim, d]`` into the leading rows of every head's block of ``dst [heads*padded, >= d]``."""
-    dst.view(heads, padded, -1)[:, :dim, :src.shape[1]].copy_(src.view(heads, dim, -1))
+    dst.unflatten(0, (heads, padded))[:, :dim, :src.shape[1]].copy_(src.view(heads, dim, -1))
 
 
 def load_head_vector(dst: torch.Tensor, src: torch.Tensor, heads: int, dim: int, padded: int) -> None:
@@ -83,4 +90,4 @@ def load_head_vector(dst: torch.Tensor, src: torch.Tensor, heads: int, dim: int,
 def load_head_columns(dst: torch.Tensor, src: torch.Tensor, heads: int, dim: int, padded: int) -> None:
     """``src [d, heads*dim]`` into the leading columns of every head's block of ``dst [>= d, heads*padded]``."""
     d = src.shape[0]
-    dst[:d].view(d, heads, padded)[:, :, :dim].copy_(src.view(d, heads, dim))
+    dst[:d].unflatten(1, (heads, padded))[:, :, :dim].copy_(src.view(d, heads, dim))

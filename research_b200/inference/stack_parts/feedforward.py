@@ -1,12 +1,12 @@
-"""Feed-forwards as parts of a layer stack: the clamped gated unit, dense (gate|up with the unit in the GEMM's epilogue, down)
-or as routed experts (``ops/experts.py``)."""
+"""Feed-forwards as parts of a layer stack: a gated unit, clamped or plain SiLU, dense (gate|up with the unit in the GEMM's epilogue,
+down) or as routed experts (``ops/experts.py``) with or without a shared one."""
 
 from __future__ import annotations
 
 import torch
 
 from ... import ops
-from ...models.stack import ClampedGluSpec, ExpertsSpec
+from ...models.stack import ClampedGluSpec, ExpertsSpec, GluSpec
 from ...ops.experts import ExpertsGeometry, ExpertsScratch
 from .base import Part, up
 
@@ -18,7 +18,7 @@ class DenseWeights:
 
 
 class DensePart(Part):
-    def make(self, spec: ClampedGluSpec) -> DenseWeights:
+    def make(self, spec: ClampedGluSpec | GluSpec) -> DenseWeights:
         r = self.r
         w = DenseWeights()
         w.spec = spec
@@ -58,7 +58,7 @@ class DensePart(Part):
 
 
 class ExpertsWeights:
-    __slots__ = ("spec", "geo", "wgu", "wd")
+    __slots__ = ("spec", "geo", "wgu", "wd", "shared")
 
 
 class ExpertsPart(Part):
@@ -70,7 +70,9 @@ class ExpertsPart(Part):
         r = self.r
         w = ExpertsWeights()
         w.spec = spec
-        w.geo = ExpertsGeometry.make(spec.experts, spec.top, spec.expert.ff, r.wp, spec.expert.limit, r.dtype)
+        how = spec.routing
+        w.geo = ExpertsGeometry.make(spec.experts, spec.top, spec.expert.ff, r.wp, spec.expert.limit, r.dtype, how.scores, how.normalize, how.scale_input)
+        w.shared = r._part(DensePart).make(spec.shared) if spec.shared is not None else None
         w.wgu, w.wd = self.zeros(spec.experts * 2 * w.geo.ffp, r.wp), self.zeros(spec.experts * r.wp, w.geo.ffp)
         self.layers.append(w)
         return w
@@ -81,10 +83,13 @@ class ExpertsPart(Part):
     def load(self, w: ExpertsWeights, get, p: str) -> None:
         n = range(w.spec.experts)
         ops.pack_experts((get(f"{p}e{e}.gate") for e in n), (get(f"{p}e{e}.up") for e in n), (get(f"{p}e{e}.down") for e in n), w.geo, w.wgu, w.wd)
+        if w.shared is not None:
+            self.r._part(DensePart).load(w.shared, get, p + "shared.")
 
     def load_small(self, w: ExpertsWeights, get, p: str, dst: torch.Tensor) -> None:
         dst[:w.spec.experts, :self.r.cfg.hidden_size].copy_(get(p + "router"))
 
     def forward(self, w: ExpertsWeights, inp, y, small) -> dict:
         e, p = ops.experts_forward(inp, small, w.geo, self.scratch[w.geo], w.wgu, w.wd)
-        return {"experts": e, "expert_weights": p}
+        add = {"experts": e, "expert_weights": p, "top": w.geo.top}
+        return {**self.r._part(DensePart).forward(w.shared, inp, y), **add} if w.shared is not None else add

@@ -5,12 +5,14 @@ token by token, longer ones in chunks on the tensor cores, in one batch."""
 
 from __future__ import annotations
 
+from dataclasses import dataclass
+
 import torch
 
 from ... import ops
-from ...models.stack import LightningSpec, MatrixMemorySpec
-from ...ops.recurrent import MAX_DIM, ChunkTable, RecurrentGeometry, RecurrentState, chunk_workspace, chunked_supported
-from .base import Part, load_head_columns, load_head_vector, load_heads
+from ...models.stack import LightningSpec, MatrixMemorySpec, TimeMixSpec
+from ...ops.recurrent import MAX_DIM, ChunkTable, RecurrentGeometry, RecurrentState, TimeMix, chunk_workspace, chunked_supported
+from .base import Part, load_head_columns, load_head_vector, load_heads, up
 
 SCAN_PORTION = 16            # new tokens of a sequence up to which the recurrence runs token by token
 
@@ -116,3 +118,113 @@ class RecurrentPart(Part):
         if table is not None:
             room = torch.empty(chunk_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=o.device)
             ops.recurrent_chunks(*args, b.cu_q, b.seq_lens, o, table, room)
+
+
+MIXES = "rkvgw"              # what reads a mix of its own: the joint projection's four parts and the decay
+WIDE_BATCH = 512             # rows from which the four projections are products of their own
+
+
+class TimeMixWeights:
+    __slots__ = ("geo", "spec", "wproj", "w1", "w2", "w0", "bonus", "mu", "norm", "wo", "rank")
+
+
+@dataclass
+class TimeMixState:
+    state: RecurrentState
+    history: torch.Tensor        # [slots, 1, wp], the last input of every sequence
+
+
+class TimeMixPart(Part):
+    @staticmethod
+    def geometry(spec: TimeMixSpec) -> RecurrentGeometry:
+        return RecurrentGeometry(spec.heads, spec.dim, spec.dim, silu=False, gated=False)
+
+    @staticmethod
+    def state_floats(spec) -> int:
+        return TimeMixPart.geometry(spec).state_floats
+
+    def make(self, spec: TimeMixSpec, tail: int = 0, output: bool = True) -> TimeMixWeights:
+        g, r, f32 = self.geometry(spec), self.r, torch.float32
+        if g.kp > MAX_DIM:
+            raise ValueError(f"the recurrent kernels take up to {MAX_DIM} key channels per head")
+        w = TimeMixWeights()
+        w.spec, w.geo, w.rank = spec, g, up(spec.decay_rank, 8)
+        n = g.heads * g.kp
+        w.wproj = self.zeros(4 * n, r.wp)
+        w.w1, w.w2 = self.zeros(w.rank, r.wp), self.zeros(n, w.rank * self.parts)
+        w.w0, w.bonus, w.norm = (self.zeros(n, dtype=f32) for _ in range(3))
+        w.mu = self.zeros(len(MIXES), r.wp, dtype=f32)
+        w.wo = self.zeros(r.wp, n) if output else None
+        self.layers.append(w)
+        return w
+
+    @property
+    def parts(self) -> int:      # how many activations carry one value of the decay's inner product exactly enough
+        return 1 if self.r.dtype == torch.float32 else 2
+
+    def new_cache(self, w: TimeMixWeights) -> TimeMixState:
+        slots = self.r.scratch_state_slot + 1
+        return TimeMixState(RecurrentState.zeros(w.geo, slots, self.r.device), self.zeros(slots, 1, self.r.wp))
+
+    def allocate(self) -> None:
+        r, f32 = self.r, torch.float32
+        n, rank = max(w.geo.heads * w.geo.kp for w in self.layers), max(w.rank for w in self.layers)
+        self.mixed = self.zeros(len(MIXES), r.rows, r.wp)
+        self.proj = self.zeros(r.rows * 4 * n)
+        self.inner, self.tanh = self.zeros(r.rows * rank, dtype=f32), self.zeros(r.rows * rank * self.parts)
+        self.z, self.o = self.zeros(r.rows * n, dtype=f32), self.zeros(r.rows * n, dtype=f32)
+        self.out = self.zeros(r.rows * max([w.geo.heads * w.geo.vp for w in self.layers if w.wo is not None], default=0))
+
+    def load(self, w: TimeMixWeights, get, p: str, factor: float = 1.0) -> None:
+        """``factor`` of the output, carried by the norm's weight."""
+        g, d = w.geo, self.r.cfg.hidden_size
+        for i, s in enumerate(MIXES):
+            w.mu[i, :d].copy_(get(f"{p}mu.{s}").float())
+            if s != "w":
+                load_heads(w.wproj[i * g.heads * g.kp:(i + 1) * g.heads * g.kp], get(p + s), g.heads, g.dim, g.kp)
+        rank = w.spec.decay_rank
+        w.w1[:rank, :d].copy_(get(p + "w1"))
+        for i in range(self.parts):
+            load_heads(w.w2[:, i * w.rank:], get(p + "w2"), g.heads, g.dim, g.kp)
+        load_head_vector(w.w0, get(p + "w0").float(), g.heads, g.dim, g.kp)
+        load_head_vector(w.bonus, get(p + "u").float().reshape(-1), g.heads, g.dim, g.kp)
+        load_head_vector(w.norm, get(p + "norm").float() * factor, g.heads, g.vdim, g.vp)
+        if w.wo is not None:
+            self.load_output(w, get, p, w.wo)
+
+    def load_output(self, w: TimeMixWeights, get, p: str, dst: torch.Tensor) -> None:
+        load_head_columns(dst, get(p + "o"), w.geo.heads, w.geo.vdim, w.geo.vp)
+
+    plan = RecurrentPart.plan
+
+    def mix(self, w: TimeMixWeights, cache: TimeMixState, inp, out, b, plan) -> None:
+        """Normed and gated heads' outputs into ``out [T, H * vp]``."""
+        T, g = b.num_tokens, w.geo
+        n = g.heads * g.kp
+        ops.token_shift(inp, w.mu, self.mixed, cache.history, b.cu_q, b.positions, b.state_slots)
+        proj = self.proj[:self.r.rows * 4 * n].view(-1, 4 * n)
+        if T < WIDE_BATCH:
+            ops.head_gemm_expand(self.mixed[:4], w.wproj, proj, T)       # (the whole buffer: its destination table is kept)
+        proj = proj[:T]
+        if T >= WIDE_BATCH:
+            for i in range(4):
+                ops.gemm(self.mixed[i, :T], w.wproj[i * n:(i + 1) * n], out=proj[:, i * n:(i + 1) * n])
+        inner, tanh = self.inner[:T * w.rank].view(T, -1), self.tanh[:T * w.rank * self.parts].view(T, -1)
+        z, o = self.z[:T * n].view(T, n), self.o[:T * n].view(T, n)
+        ops.gemm(self.mixed[4, :T], w.w1, out=inner, out_f32=True)
+        ops.tanh_parts(inner, tanh)
+        ops.gemm(tanh, w.w2, out=z, out_f32=True)
+        mix = TimeMix(z, w.w0, w.bonus)
+        args = (proj, None, g, None, None, None, 1.0, cache.state, b.state_slots)
+        if b.cu_q is None or b.n_single > 0:
+            single = b.rows if b.cu_q is None else b.n_single
+            ops.recurrent_scan(*args, None, b.seq_lens, o, single, single, mix=mix)
+        if b.cu_q is not None and b.rows > b.n_single:
+            ops.recurrent_scan(*args, b.cu_q, b.seq_lens, o, T, b.rows, b.n_single, mix=mix)
+        ops.gated_norm(o, w.norm, proj[:, g.offsets[3]:], g, self.r.cfg.norm_eps, out, True, silu=True)
+
+    def forward(self, w: TimeMixWeights, cache: TimeMixState, inp, y, b, plan, small=None) -> None:
+        T, n = b.num_tokens, w.geo.heads * w.geo.vp
+        out = self.out[:T * n].view(T, n)
+        self.mix(w, cache, inp, out, b, plan)
+        ops.gemm(out, w.wo, out=y, out_f32=True)

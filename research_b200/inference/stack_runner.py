@@ -7,7 +7,8 @@ type. Two kinds of layer (``Design.block``):
 * post_norm: a sublayer reads the stream itself (a copy in the activation type) and its output is layer-normalised on the way
   back; the layer scale is folded into that norm's weight and bias in fp32;
 * parallel: mixer and feed-forward read one RMS norm of the stream; the residual add, the sum over a token's experts and
-  the next layer's norm are one kernel.
+  the next layer's norm are one kernel. A per-layer token input (``TokenSideSpec``) enters between the add and that norm: two narrow
+  products over the stream, and its own norm in the same kernel as the next layer's.
 
 Looped layers run several times with the same weights; every run has a cache or state of its own, and a pass starts with a
 product that mixes the embedding output into the stream.
@@ -34,7 +35,18 @@ from .stack_parts.base import Part, up
 class StackLayer:
     """Weights of one layer: those of its mixer and feed-forward parts, the norms, the narrow fp32 projection."""
 
-    __slots__ = ("spec", "mixer", "mix", "feed_forward", "ff", "norm1", "norm2", "wsmall", "wsmall_ff", "mix_small")
+    __slots__ = ("spec", "mixer", "mix", "feed_forward", "ff", "norm1", "norm2", "wsmall", "wsmall_ff", "mix_small", "side")
+
+
+@dataclass
+class SideWeights:
+    """Per-layer token input: the gate ``[sp, wp]``, the projection back ``[wp, sp]``, the norm's weight, the layer's columns of the side
+    embedding."""
+
+    gate: torch.Tensor
+    proj: torch.Tensor
+    norm: torch.Tensor
+    col: int
 
 
 @dataclass
@@ -62,6 +74,7 @@ class StackRunner(RunnerBase):
             raise ValueError("layer-stack models run on one GPU per engine (no tensor or expert parallelism)")
         self.tp = self.ep = None
         self.tp_size, self.tp_rank = 1, 0
+        cfg = cfg.fitted(weights)
         self._init_geometry(cfg, device=device, num_kv_blocks=num_kv_blocks, max_batch=max_batch, max_model_len=max_model_len,
                             max_prefill_tokens=max_prefill_tokens, use_cuda_graphs=use_cuda_graphs,
                             graph_batch_sizes=graph_batch_sizes, dtype=dtype)
@@ -105,6 +118,9 @@ class StackRunner(RunnerBase):
         self.head = self.embed if cfg.design.tied else zeros(self.vp, self.wp)
         self.final_norm = norm()
         self.loop_in = zeros(self.wp, 2 * self.wp) if cfg.loop is not None else None
+        self.side_dim = cfg.token_side.dim if cfg.token_side is not None else 0
+        self.sp = up(self.side_dim, 8)
+        self.side_embed = zeros(cfg.vocab_size, cfg.num_layers * self.side_dim) if self.side_dim else None
         self.layers: list[StackLayer] = []
         for spec in cfg.layers:
             lw = StackLayer()
@@ -124,6 +140,8 @@ class StackRunner(RunnerBase):
             lw.mix = lw.mixer.make(spec.mixer, n)
             lw.wsmall = None if n == 0 else lw.mix.wproj[-n:] if lw.mixer.fuses_tail else zeros(n, self.wp)
             lw.wsmall_ff = None if ff_small == 0 else lw.wsmall[lw.mix_small:] if self.parallel else zeros(ff_small, self.wp)
+            lw.side = SideWeights(zeros(self.sp, self.wp), zeros(self.wp, self.sp), zeros(self.wp, dtype=torch.float32),
+                                  len(self.layers) * self.side_dim) if self.side_dim else None
             self.layers.append(lw)
         self.runs = [StackRun(self.layers[x.layer], self.layers[x.layer].mixer.new_cache(self.layers[x.layer].mix), x.enters) for x in cfg.runs]
 
@@ -135,6 +153,8 @@ class StackRunner(RunnerBase):
         self.y2 = torch.zeros(n, self.wp, dtype=torch.float32, device=dev)
         self.hl = torch.zeros(self.max_batch, self.wp, dtype=dt, device=dev)
         self.x_loop = torch.zeros(n, 2 * self.wp, dtype=dt, device=dev) if self.loop_in is not None else None     # stream | embedding output
+        self.side_z = torch.zeros(n, self.sp, dtype=torch.float32, device=dev)
+        self.side_a = torch.zeros(n, self.sp, dtype=dt, device=dev)
         most = max([w.shape[0] for lw in self.layers for w in (lw.wsmall, lw.wsmall_ff) if w is not None], default=0)
         self._small = torch.zeros(n * most, dtype=torch.float32, device=dev)
         for part in self.parts.values():
@@ -153,8 +173,8 @@ class StackRunner(RunnerBase):
             return get(name).float()
 
         def norm_into(dst, name: str, scale: torch.Tensor | None = None) -> None:
-            if self.parallel:          # RMS norm, weight stored around zero
-                dst[0][:d].copy_(1 + f32(name))
+            if self.parallel:          # RMS norm
+                dst[0][:d].copy_(f32(name) + float(cfg.design.unit_norms))
                 return
             w, b = f32(name), f32(name + ".b")
             dst[0][:d].copy_(w if scale is None else w * scale)
@@ -167,6 +187,8 @@ class StackRunner(RunnerBase):
             w = get("loop.in")
             self.loop_in[:d, :d].copy_(w[:, :d])
             self.loop_in[:d, self.wp:self.wp + d].copy_(w[:, d:])
+        if self.side_embed is not None:
+            self.side_embed.copy_(get("side.embed"))
         norm_into(self.final_norm, "final.norm")
         for i, lw in enumerate(self.layers):
             p = f"l{i}."
@@ -180,6 +202,10 @@ class StackRunner(RunnerBase):
                     lw.feed_forward.load_small(lw.ff, get, p + "mlp.", lw.wsmall_ff)
                 if not self.parallel:
                     norm_into(lw.norm2, p + "norm2", f32(p + "ls2"))
+            if lw.side is not None:
+                lw.side.gate[:self.side_dim, :d].copy_(get(p + "side.gate"))
+                lw.side.proj[:d, :self.side_dim].copy_(get(p + "side.proj"))
+                lw.side.norm[:d].copy_(f32(p + "side.norm"))
 
     # ------------------------------------------------------------------ layers
     def _small_rows(self, inp: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -200,7 +226,7 @@ class StackRunner(RunnerBase):
 
     def _layers(self, b: PackedBatch) -> None:
         """All layer runs over the batch's rows; leaves the residual stream in ``self.x``."""
-        plans = {part: part.plan(b) for part in self.parts.values()}
+        plans = {part: part.planned(b) for part in self.parts.values()}
         if self.parallel:
             self._parallel_layers(b, plans)
         else:
@@ -216,7 +242,7 @@ class StackRunner(RunnerBase):
         ops.stream_embed(b.tokens[:b.num_tokens], self.embed[:self.cfg.vocab_size], self.cfg.hidden_size, self.x, x0, first_copy)
 
     def _parallel_layers(self, b: PackedBatch, plans: dict) -> None:
-        T, d, eps = b.num_tokens, self.cfg.hidden_size, self.cfg.norm_eps
+        T, d, eps, m = b.num_tokens, self.cfg.hidden_size, self.cfg.norm_eps, self.cfg.residual_mult
         x, h, y = self.x[:T], self.xb[:T], self.y[:T]
         xl = self.x_loop[:T, :self.wp] if self.x_loop is not None else None
         self._embed(b, xl)
@@ -225,16 +251,28 @@ class StackRunner(RunnerBase):
             lw = run.layer
             if run.enters:
                 if add:
-                    ops.stream_norm(x, d, **add, copy=xl)
+                    ops.stream_norm(x, d, **add, mult=m, eps=eps, copy=xl)
                     add = {}
                 self._enter_pass(T)
-            ops.stream_norm(x, d, **add, weight=lw.norm1[0], eps=eps, h=h)
+            ops.stream_norm(x, d, **add, mult=m, weight=lw.norm1[0], eps=eps, h=h)
             small = self._project(lw, h)
             lw.mixer.forward(lw.mix, run.cache, h, y, b, plans[lw.mixer], small)
             add = {"y1": y}
             if lw.ff is not None:
                 add.update(lw.feed_forward.forward(lw.ff, h, self.y2[:T], small[:, lw.mix_small:] if small is not None else None))
-        ops.stream_norm(x, d, **add)
+            if lw.side is not None:
+                ops.stream_norm(x, d, **add, mult=m, copy=h)
+                self._token_side(lw.side, b, h, y)
+                add = {"side": y, "side_weight": lw.side.norm}
+        ops.stream_norm(x, d, **add, mult=m, eps=eps)
+
+    def _token_side(self, w: SideWeights, b: PackedBatch, xb: torch.Tensor, y: torch.Tensor) -> None:
+        """``y = W_proj (gelu_tanh(W_gate x) * e)`` with the layer's part ``e`` of the tokens' side embedding."""
+        T = b.num_tokens
+        z, a = self.side_z[:T], self.side_a[:T]
+        ops.gemm(xb, w.gate, out=z, out_f32=True)
+        ops.token_side(z, b.tokens[:T], self.side_embed, w.col, a, self.side_dim)
+        ops.gemm(a, w.proj, out=y, out_f32=True)
 
     def _post_norm_layers(self, b: PackedBatch, plans: dict) -> None:
         T, d, eps = b.num_tokens, self.cfg.hidden_size, self.cfg.norm_eps

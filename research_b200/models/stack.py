@@ -2,9 +2,8 @@
 
 ``ModelConfig`` holds one set of sizes for the whole model. A ``LayerStackConfig`` instead lists its layers; each names
 the mixer it uses (with that layer's own sizes, window and rotation) and its feed-forward, or none. Mixers and
-feed-forwards are small value types that know their ``config.json`` form and their tensors; a further kind is a new class
-registered in ``MIXERS`` or ``FEED_FORWARDS``. How a layer is put together around them (norms, residual, head) is a
-property of the design, a row of ``DESIGNS``.
+feed-forwards are small value types that know their ``config.json`` form and their tensors. Which of them a design has, and how
+a layer is put together around them (norms, residual, head), is a row of ``DESIGNS``.
 
 ``config.json`` form::
 
@@ -12,28 +11,91 @@ property of the design, a row of ``DESIGNS``.
      "loop": {"start": a, "stop": b, "times": n},
      "layers": [{"type": "latent_attention", "mixer": {...}, "mlp": {"kind": "dense", ...} or null}, ...]}
 
+``type`` and ``kind`` are names within a design: ``Design.mixers`` and ``Design.feed_forwards`` say what they stand for.
+
 Tensors are named ``embed``, ``l<i>.norm1`` / ``.mix.*`` / ``.mlp.*``, ``final.norm``; matrices are stored ``[out, in]``.
 Post-norm designs add ``.norm1.b`` / ``.ls1`` (and ``norm2`` / ``norm2.b`` / ``ls2`` for the feed-forward) and
-``final.norm.b``; designs without tied embeddings have ``head``; looped stacks have ``loop.in``.
+``final.norm.b``; designs without tied embeddings have ``head``; looped stacks have ``loop.in``; stacks with a per-layer token
+input have ``side.embed`` and ``l<i>.side.gate`` / ``.proj`` / ``.norm``.
 """
 
 from __future__ import annotations
 
 import json
 import math
-from dataclasses import asdict, dataclass
+from collections.abc import Mapping
+from dataclasses import asdict, dataclass, replace
+from functools import partial
 from pathlib import Path
+from typing import Callable
 
 
 NO_WINDOW = 1 << 30          # a window nothing reaches: plain causal attention
 
 
 @dataclass(frozen=True)
+class BandScaling:
+    """Long waves slowed by ``factor``, short ones kept, a blend in between: with the wavelength ``l = 2 pi / f``, frequencies of
+    ``l < original/high`` stay, those of ``l > original/low`` are divided, the others are mixed linearly in ``original/l``."""
+
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    amplitude = 1.0
+
+    def frequencies(self, rot: "RotarySpec") -> list[float]:
+        out = []
+        for f in rot.plain_frequencies():
+            turns = self.original * f / (2 * math.pi)          # of one wave over the original context
+            keep = 1.0 if turns > self.high else 0.0 if turns < self.low else (turns - self.low) / (self.high - self.low)
+            out.append(f * (keep + (1 - keep) / self.factor))
+        return out
+
+
+@dataclass(frozen=True)
+class YarnScaling:
+    """YaRN: channels that turn more than ``fast`` times over the ``original`` context keep their frequency, those below
+    ``slow`` turns are divided by ``factor``, a linear ramp over the channels between; cos and sin are scaled by ``amplitude``."""
+
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    @property
+    def amplitude(self) -> float:
+        return 0.1 * math.log(self.factor) + 1
+
+    def frequencies(self, rot: "RotarySpec") -> list[float]:
+        def channel(turns: float) -> float:
+            return rot.dims * math.log(self.original / (2 * math.pi * turns)) / (2 * math.log(rot.base))
+
+        lo, hi = max(math.floor(channel(self.fast)), 0), min(math.ceil(channel(self.slow)), rot.dims - 1)
+        ramps = (min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(rot.dims // 2))
+        return [f * (1 - r + r / self.factor) for f, r in zip(rot.plain_frequencies(), ramps)]
+
+
+@dataclass(frozen=True)
 class RotarySpec:
-    """Rotation of pairs ``(i, i + dims/2)`` of the first ``dims`` channels by ``position * base^(-2i/dims)``."""
+    """Rotation of pairs of the first ``dims`` channels by ``position * base^(-2i/dims)``: channels ``(i, i + dims/2)``, or
+    ``(2i, 2i+1)`` when ``interleaved``; ``scaling`` changes the frequencies."""
 
     dims: int
     base: float
+    interleaved: bool = False
+    scaling: BandScaling | YarnScaling | None = None
+
+    def plain_frequencies(self) -> list[float]:
+        return [self.base ** (-2 * i / self.dims) for i in range(self.dims // 2)]
+
+    def frequencies(self) -> list[float]:
+        return self.scaling.frequencies(self) if self.scaling is not None else self.plain_frequencies()
+
+    @property
+    def amplitude(self) -> float:
+        return self.scaling.amplitude if self.scaling is not None else 1.0
 
 
 @dataclass(frozen=True)
@@ -194,13 +256,44 @@ class KeyValueAttentionSpec:
 
 
 @dataclass(frozen=True)
+class GluSpec:
+    """``silu(gate) * up``."""
+
+    ff: int
+
+    kind = "dense"
+    limit = None
+
+    @staticmethod
+    def from_dict(m: dict) -> "GluSpec":
+        return GluSpec(ff=int(m["ff"]))
+
+    def to_dict(self) -> dict:
+        return {"kind": self.kind, "ff": self.ff}
+
+    param_shapes = ClampedGluSpec.param_shapes
+
+
+@dataclass(frozen=True)
+class ExpertsRouting:
+    """How a design weighs the chosen experts: ``scores`` is "softmax" or "sigmoid" of the router's logits; ``normalize``
+    divides the chosen scores by their sum; the weight multiplies an expert's output, or its input with ``scale_input``."""
+
+    scores: str = "softmax"
+    normalize: bool = True
+    scale_input: bool = False
+
+
+@dataclass(frozen=True)
 class ExpertsSpec:
-    """``experts`` clamped gated units of which every token uses the ``top`` with the largest softmax score, weighted by
-    their scores divided by the chosen scores' sum."""
+    """``experts`` gated units of which every token uses the ``top`` with the largest score, weighed as ``routing`` says;
+    ``shared`` is a further unit that every token passes."""
 
     experts: int
     top: int
-    expert: ClampedGluSpec
+    expert: ClampedGluSpec | GluSpec
+    routing: ExpertsRouting = ExpertsRouting()
+    shared: GluSpec | None = None
 
     kind = "moe"
 
@@ -208,50 +301,212 @@ class ExpertsSpec:
         assert 1 <= self.top <= self.experts
 
     @staticmethod
-    def from_dict(m: dict) -> "ExpertsSpec":
-        return ExpertsSpec(int(m["router"]["experts"]), int(m["router"]["top"]), ClampedGluSpec.from_dict(m["expert"]))
+    def from_dict(m: dict, unit=ClampedGluSpec, routing: ExpertsRouting = ExpertsRouting()) -> "ExpertsSpec":
+        shared = m.get("shared")
+        return ExpertsSpec(int(m["router"]["experts"]), int(m["router"]["top"]), unit.from_dict(m["expert"]), routing,
+                           unit.from_dict(shared) if shared else None)
 
     def to_dict(self) -> dict:
-        return {"kind": self.kind, "router": {"experts": self.experts, "top": self.top},
-                "expert": {"ff": self.expert.ff, "limit": self.expert.limit}}
+        def unit(u) -> dict:
+            return {k: v for k, v in u.to_dict().items() if k != "kind"}
+
+        d = {"kind": self.kind, "router": {"experts": self.experts, "top": self.top}, "expert": unit(self.expert)}
+        return {**d, "shared": unit(self.shared)} if self.shared is not None else d
 
     def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
         out = {p + "router": (self.experts, width)}
         for e in range(self.experts):
             out.update(self.expert.param_shapes(f"{p}e{e}.", width))
+        if self.shared is not None:
+            out.update(self.shared.param_shapes(p + "shared.", width))
         return out
 
 
-MIXERS = {c.type: c for c in (LatentAttentionSpec, LightningSpec, MatrixMemorySpec, KeyValueAttentionSpec)}
-FEED_FORWARDS = {c.kind: c for c in (ClampedGluSpec, ExpertsSpec)}
+@dataclass(frozen=True)
+class AttentionForm:
+    """What a design fixes about a kind of grouped attention; sizes and constants are in ``GroupedAttentionSpec``.
+
+    ``norm``: "projection" (RMS norm over all heads at once with weights, before the rotation), "head" (every head divided by its
+    root mean square after the rotation) or "". ``span``: which keys ``j <= i`` a query sees, "all", "window" (``i - j < size``) or
+    "chunk" (the same ``floor(position / size)``)."""
+
+    type: str
+    bias: bool = False
+    conv: bool = False                 # a short causal convolution on every projected channel
+    norm: str = ""
+    interleaved: bool = False
+    scaling: type | None = None        # BandScaling or YarnScaling
+    span: str = "all"
+    gate: bool = False                 # every head's output times the sigmoid of one projected number
+
+    def from_dict(self, m: dict) -> "GroupedAttentionSpec":
+        rot, scaling = m["rot"], None
+        if self.scaling is not None and rot.get("scaling"):
+            scaling = self.scaling(**{k: float(v) for k, v in rot["scaling"].items()})
+        return GroupedAttentionSpec(self, int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                    RotarySpec(int(rot["dims"]), float(rot["base"]), self.interleaved, scaling),
+                                    int(m["conv"]) if self.conv else 1, int(m["mask"]["size"]) if self.span != "all" else 0)
+
+
+@dataclass(frozen=True)
+class GroupedAttentionSpec:
+    """Causal attention with grouped heads and cached keys and values (see ``ops/grouped.py``). ``taps`` of the convolution (1: the
+    projection itself), ``size`` of the window or chunk."""
+
+    form: AttentionForm
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotarySpec
+    taps: int = 1
+    size: int = 0
+
+    def __post_init__(self):
+        assert self.heads % self.kv_heads == 0, "query heads share kv heads evenly"
+        assert self.rot.dims % 2 == 0 and self.rot.dims <= self.dim, "the rotation covers an even part of a head"
+        assert self.taps >= 1 and (self.form.span == "all" or self.size >= 1)
+
+    @property
+    def type(self) -> str:
+        return self.form.type
+
+    @property
+    def rows(self) -> tuple[int, int, int]:
+        """Projected channels of queries, keys and values."""
+        return self.heads * self.dim, self.kv_heads * self.dim, self.kv_heads * self.vdim
+
+    def to_dict(self) -> dict:
+        rot = {"dims": self.rot.dims, "base": self.rot.base}
+        if self.rot.scaling is not None:
+            rot["scaling"] = asdict(self.rot.scaling)
+        d = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale, "rot": rot}
+        if self.form.conv:
+            d["conv"] = self.taps
+        if self.form.span != "all":
+            d["mask"] = {"size": self.size}
+        return d
+
+    def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
+        out: dict[str, tuple[int, ...]] = {}
+        for name, n in zip("qkv", self.rows):
+            out[p + name] = (n, width)
+            if self.form.bias:
+                out[p + name + ".b"] = (n,)
+            if self.form.conv:
+                out[p + name + ".conv"] = (n, self.taps)
+            if self.form.norm == "projection" and name != "v":
+                out[p + name + ".norm"] = (n,)
+        if self.form.gate:
+            out[p + "g"] = (self.heads, width)
+        return {**out, p + "o": (width, self.heads * self.vdim)}
+
+
+@dataclass(frozen=True)
+class TimeMixSpec:
+    """RWKV-style time mixing (see ``ops/recurrent.py``): projections of mixes with the previous token, a decay per key channel
+    through a narrow product of ``decay_rank`` channels (0: as wide as the checkpoint's tensor), a bonus for the current token,
+    an RMS norm per head, a SiLU gate."""
+
+    heads: int
+    dim: int
+    decay_rank: int = 0
+
+    type = "time_mix"
+    DEFAULT_RANK = 32                  # of freshly initialised weights
+
+    @staticmethod
+    def from_dict(m: dict) -> "TimeMixSpec":
+        return TimeMixSpec(int(m["heads"]), int(m["dim"]), int(m.get("decay_rank", 0)))
+
+    def to_dict(self) -> dict:
+        d = {"heads": self.heads, "dim": self.dim}
+        return {**d, "decay_rank": self.decay_rank} if self.decay_rank else d
+
+    def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
+        n, r = self.heads * self.dim, self.decay_rank or self.DEFAULT_RANK
+        out = {f"{p}mu.{s}": (width,) for s in "rkvgw"}
+        out.update({p + s: (n, width) for s in "rkvg"})
+        return {**out, p + "w1": (r, width), p + "w2": (n, r), p + "w0": (n,), p + "u": (self.heads, self.dim), p + "norm": (n,), p + "o": (width, n)}
+
+    def fitted(self, shapes: Callable[[str], tuple[int, ...]], p: str) -> "TimeMixSpec":
+        rank = shapes(p + "w1")[0]
+        assert self.decay_rank in (0, rank), f"{p}w1 has {rank} rows, the configuration says {self.decay_rank}"
+        return replace(self, decay_rank=rank)
+
+
+@dataclass(frozen=True)
+class ParallelForm:
+    """Which mixers a design puts side by side."""
+
+    type: str
+    left: AttentionForm
+    right: type
+
+    def from_dict(self, m: dict) -> "ParallelSpec":
+        return ParallelSpec(self.type, self.left.from_dict(m["left"]), self.right.from_dict(m["right"]), float(m["left_scale"]), float(m["right_scale"]))
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers that read the same activations: ``left_scale * left + right_scale * right``."""
+
+    type: str
+    left: GroupedAttentionSpec
+    right: TimeMixSpec
+    left_scale: float
+    right_scale: float
+
+    def to_dict(self) -> dict:
+        return {"left": self.left.to_dict(), "right": self.right.to_dict(), "left_scale": self.left_scale, "right_scale": self.right_scale}
+
+    def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
+        return {**self.left.param_shapes(p + "left.", width), **self.right.param_shapes(p + "right.", width)}
+
+    def fitted(self, shapes: Callable[[str], tuple[int, ...]], p: str) -> "ParallelSpec":
+        return replace(self, right=self.right.fitted(shapes, p + "right."))
 
 
 @dataclass(frozen=True)
 class Design:
     """What all models of a design share. ``block`` is "post_norm" (sublayers read the stream; layer norm with bias and layer
-    scale on their outputs) or "parallel" (mixer and feed-forward read one RMS norm whose weight is stored around zero, and
-    both are added)."""
+    scale on their outputs) or "parallel" (mixer and feed-forward read one RMS norm, and both are added)."""
 
     block: str
     tied: bool                         # the head is the embedding table
+    mixers: dict                       # "type" in config.json -> what reads the layer's "mixer"
+    feed_forwards: dict                # "kind" -> function that reads "mlp"
+    unit_norms: bool = False           # norm weights are stored around zero
 
 
-DESIGNS = {"Lulezen": Design("post_norm", False), "Zamusun": Design("parallel", True)}
+WINDOW_ATTENTION = AttentionForm("window_attention", norm="projection", interleaved=True, span="window", gate=True)
+
+DESIGNS = {
+    "Lulezen": Design("post_norm", False, {"latent_attention": LatentAttentionSpec}, {"dense": ClampedGluSpec.from_dict}),
+    "Zamusun": Design("parallel", True, {"lightning": LightningSpec, "mlstm": MatrixMemorySpec, "attention": KeyValueAttentionSpec},
+                      {"dense": ClampedGluSpec.from_dict, "moe": ExpertsSpec.from_dict}, unit_norms=True),
+    "Fogurax": Design("parallel", True,
+                      {f.type: f for f in (AttentionForm("attention", bias=True, conv=True, norm="head", interleaved=True, scaling=BandScaling, gate=True),
+                                           AttentionForm("attention_2", norm="projection", scaling=YarnScaling, span="chunk"),
+                                           ParallelForm("parallel", WINDOW_ATTENTION, TimeMixSpec))},
+                      {"dense": GluSpec.from_dict, "moe": partial(ExpertsSpec.from_dict, unit=GluSpec, routing=ExpertsRouting("sigmoid", False, True))}),
+}
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentAttentionSpec | LightningSpec | MatrixMemorySpec | KeyValueAttentionSpec
-    mlp: ClampedGluSpec | ExpertsSpec | None = None
+    mixer: LatentAttentionSpec | LightningSpec | MatrixMemorySpec | KeyValueAttentionSpec | GroupedAttentionSpec | ParallelSpec
+    mlp: ClampedGluSpec | GluSpec | ExpertsSpec | None = None
 
     @staticmethod
-    def from_dict(e: dict) -> "LayerSpec":
-        if e["type"] not in MIXERS:
-            raise ValueError(f"unknown mixer {e['type']!r}; known: {sorted(MIXERS)}")
+    def from_dict(e: dict, design: Design) -> "LayerSpec":
+        if e["type"] not in design.mixers:
+            raise ValueError(f"unknown mixer {e['type']!r}; known: {sorted(design.mixers)}")
         mlp = e.get("mlp")
-        if mlp is not None and mlp["kind"] not in FEED_FORWARDS:
-            raise ValueError(f"unknown feed-forward {mlp['kind']!r}; known: {sorted(FEED_FORWARDS)}")
-        return LayerSpec(MIXERS[e["type"]].from_dict(e["mixer"]), FEED_FORWARDS[mlp["kind"]].from_dict(mlp) if mlp is not None else None)
+        if mlp is not None and mlp["kind"] not in design.feed_forwards:
+            raise ValueError(f"unknown feed-forward {mlp['kind']!r}; known: {sorted(design.feed_forwards)}")
+        return LayerSpec(design.mixers[e["type"]].from_dict(e["mixer"]), design.feed_forwards[mlp["kind"]](mlp) if mlp is not None else None)
 
     def to_dict(self) -> dict:
         return {"type": self.mixer.type, "mixer": self.mixer.to_dict(), "mlp": self.mlp.to_dict() if self.mlp is not None else None}
@@ -265,6 +520,14 @@ class LoopSpec:
     start: int
     stop: int
     times: int
+
+
+@dataclass(frozen=True)
+class TokenSideSpec:
+    """A second embedding of every token, ``dim`` channels for each layer, that enters the stream after the layer's sublayers:
+    ``y = W_proj (gelu_tanh(W_gate x) * e)``, ``x += residual_mult * y / rms(y) * norm``."""
+
+    dim: int
 
 
 @dataclass(frozen=True)
@@ -287,11 +550,14 @@ class LayerStackConfig:
     max_position_embeddings: int = 8192
     init_std: float = 0.02
     loop: LoopSpec | None = None
+    residual_mult: float = 1.0         # factor of everything that is added to the stream
+    token_side: TokenSideSpec | None = None
 
     # what the engine asks of every model configuration
     is_moe = False                     # (expert-parallel engines shard ModelConfig models only)
 
     def __post_init__(self):
+        assert (self.residual_mult == 1.0 and self.token_side is None) or self.design.block == "parallel", "parallel blocks only"
         if self.loop is not None:
             assert 0 <= self.loop.start < self.loop.stop <= len(self.layers) and self.loop.times >= 1, "loop range"
 
@@ -330,6 +596,10 @@ class LayerStackConfig:
                 elif n == "1":
                     out[p + "norm1"] = (d,)
                 out.update(spec.param_shapes(p + sub, d))
+            if self.token_side is not None:
+                out.update({p + "side.gate": (self.token_side.dim, d), p + "side.proj": (d, self.token_side.dim), p + "side.norm": (d,)})
+        if self.token_side is not None:
+            out["side.embed"] = (self.vocab_size, self.num_layers * self.token_side.dim)
         out["final.norm"] = (d,)
         if post:
             out["final.norm.b"] = (d,)
@@ -343,8 +613,17 @@ class LayerStackConfig:
         if last == "b" or last == "sink":
             return 0.0
         if last.startswith("norm") or last.startswith("ls"):
-            return 0.0 if self.design.block == "parallel" and ".mix." not in name else 1.0
-        return None
+            return 0.0 if self.design.unit_norms and ".mix." not in name else 1.0
+        if ".mu." in name or last == "conv":
+            return 0.5
+        return -3.0 if last == "w0" else None
+
+    def fitted(self, weights: Mapping) -> "LayerStackConfig":
+        """This configuration with the sizes that only the checkpoint's tensors tell."""
+        def mixer(i: int, spec):
+            return spec.fitted(lambda name: tuple(weights[name].shape), f"l{i}.mix.") if hasattr(spec, "fitted") else spec
+
+        return replace(self, layers=tuple(replace(x, mixer=mixer(i, x.mixer)) for i, x in enumerate(self.layers)))
 
     def num_params(self) -> int:
         return sum(math.prod(s) for s in self.param_shapes().values())
@@ -352,12 +631,13 @@ class LayerStackConfig:
     # ---- config.json -----------------------------------------------------------------------
     @staticmethod
     def from_dict(d: dict) -> "LayerStackConfig":
-        loop = d.get("loop")
+        loop, side = d.get("loop"), d.get("token_side")
         return LayerStackConfig(architecture=d["architecture"], vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
-                                layers=tuple(LayerSpec.from_dict(e) for e in d["layers"]), norm_eps=float(d["norm"]["eps"]),
+                                layers=tuple(LayerSpec.from_dict(e, DESIGNS[d["architecture"]]) for e in d["layers"]), norm_eps=float(d["norm"]["eps"]),
                                 logit_softcap=float(d.get("logit_softcap") or 0.0),
                                 eos_token_id=int(d.get("eos_token_id", -1)),
-                                loop=LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None)
+                                loop=LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None,
+                                residual_mult=float(d.get("residual_mult", 1.0)), token_side=TokenSideSpec(int(side["dim"])) if side else None)
 
     def to_dict(self) -> dict:
         d = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
@@ -366,6 +646,10 @@ class LayerStackConfig:
             d["logit_softcap"] = self.logit_softcap
         if self.loop is not None:
             d["loop"] = asdict(self.loop)
+        if self.residual_mult != 1.0:
+            d["residual_mult"] = self.residual_mult
+        if self.token_side is not None:
+            d["token_side"] = asdict(self.token_side)
         if self.eos_token_id >= 0:
             d["eos_token_id"] = self.eos_token_id
         return d

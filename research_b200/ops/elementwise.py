@@ -32,9 +32,10 @@ def _lib() -> ctypes.CDLL:
         lib.rb_clamped_glu.argtypes = [c_vp, c_vp, c_int, c_ll, c_int, c_float, c_vp]
         lib.rb_softcap.argtypes = [c_vp, c_ll, c_float, c_vp]
         lib.rb_stream_embed.argtypes = [c_vp, c_vp, c_ll, c_vp, c_ll, c_vp, c_ll, c_vp, c_ll] + [c_int] * 4 + [c_vp, c_vp]
-        lib.rb_stream_norm.argtypes = ([c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_vp, c_ll, c_int, c_vp, c_ll, c_vp, c_ll, c_vp, c_vp] + [c_int] * 5
-                                       + [c_float, c_vp, c_vp])
-        for f in ("rb_stream_embed", "rb_stream_norm", "rb_layernorm", "rb_clamped_glu", "rb_softcap", "rb_rmsnorm", "rb_rope_kv_append", "rb_swiglu", "rb_swiglu_bwd", "rb_embedding", "rb_transpose_bf16"):
+        lib.rb_stream_norm.argtypes = ([c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_vp, c_ll, c_int, c_vp, c_ll, c_vp, c_float, c_vp, c_ll, c_vp, c_ll, c_vp,
+                                        c_vp] + [c_int] * 5 + [c_float, c_vp, c_vp])
+        lib.rb_token_side.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_int, c_vp, c_ll] + [c_int] * 4 + [c_vp, c_vp]
+        for f in ("rb_token_side", "rb_stream_embed", "rb_stream_norm", "rb_layernorm", "rb_clamped_glu", "rb_softcap", "rb_rmsnorm", "rb_rope_kv_append", "rb_swiglu", "rb_swiglu_bwd", "rb_embedding", "rb_transpose_bf16"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -81,6 +82,12 @@ def rope_table(max_pos: int, head_dim: int, theta: float, device=None, exact: bo
     ang = torch.outer(pos, inv_freq)
     tab = torch.stack([ang.cos(), ang.sin()], dim=-1).contiguous()
     return tab.to(device) if device is not None else tab
+
+
+def frequency_table(max_pos: int, frequencies: list[float], amplitude: float = 1.0, device=None) -> torch.Tensor:
+    """``[max_pos, n, 2]`` fp32 table of ``amplitude`` times (cos, sin) of position times frequency, angles formed in float64."""
+    ang = torch.outer(torch.arange(max_pos, dtype=torch.float64), torch.tensor(frequencies, dtype=torch.float64))
+    return (amplitude * torch.stack([ang.cos(), ang.sin()], dim=-1)).float().contiguous().to(device or "cpu")
 
 
 def _rotate_reference(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
@@ -232,21 +239,25 @@ def stream_embed(ids: torch.Tensor, table: torch.Tensor, d: int, x: torch.Tensor
     check_rc(rc, "rb_stream_embed")
 
 
-def stream_norm(x: torch.Tensor, d: int, *, y1=None, y2=None, experts=None, expert_weights=None, copy=None, weight=None, eps: float = 0.0,
-                h=None, rows=None) -> None:
+def stream_norm(x: torch.Tensor, d: int, *, y1=None, y2=None, experts=None, expert_weights=None, top: int = 0, side=None, side_weight=None,
+                mult: float = 1.0, copy=None, weight=None, eps: float = 0.0, h=None, rows=None) -> None:
     """What happens to the fp32 stream ``x [n, dp]`` (``d`` channels and zero padding) between two layers, in one pass:
-    ``x += y1 + y2 + sum_j expert_weights[t, j] experts[t, j]`` (the terms that are given), ``copy = x`` and
-    ``h = x / rms(x) * weight`` in the activation type. With ``rows`` only ``h[i]`` of row ``rows[i]``."""
+    ``x += mult (y1 + y2 + sum_j expert_weights[t, j] experts[t, j] + side / rms(side) * side_weight)`` (the terms that are given),
+    ``copy = x`` and ``h = x / rms(x) * weight`` in the activation type. Without ``expert_weights`` the ``top`` results of a token
+    are added as they are. With ``rows`` only ``h[i]`` of row ``rows[i]``."""
     n = rows.numel() if rows is not None else x.shape[0]
     if not x.is_cuda:
         src = x if rows is None else x[rows.long()]
-        assert rows is None or (y1 is None and y2 is None and experts is None)
+        assert rows is None or (y1 is None and y2 is None and experts is None and side is None)
         for y in (y1, y2):
             if y is not None:
-                x += y[:n]
+                x += mult * y[:n]
         if experts is not None:
-            k = expert_weights.shape[1]
-            x += (experts[:n * k].view(n, k, -1).float() * expert_weights[:n, :, None]).sum(1)
+            k = top if expert_weights is None else expert_weights.shape[1]
+            e = experts[:n * k].view(n, k, -1).float()
+            x += mult * (e if expert_weights is None else e * expert_weights[:n, :, None]).sum(1)
+        if side is not None:
+            x += mult * side[:n] * torch.rsqrt(side[:n].pow(2).sum(-1, keepdim=True) / d + eps) * side_weight
         if copy is not None:
             copy[:n] = x.to(copy.dtype)
         if h is not None:
@@ -256,12 +267,26 @@ def stream_norm(x: torch.Tensor, d: int, *, y1=None, y2=None, experts=None, expe
     assert x.dtype == torch.float32 and x.stride(1) == 1 and (rows is None or rows.dtype == torch.int32)
     assert all(t is None or t.stride(-1) == 1 for t in (y1, y2, experts, copy, h)) and (y1 is None or y2 is None or y1.stride(0) == y2.stride(0))
     y = y1 if y1 is not None else y2
+    k = top if expert_weights is None else expert_weights.shape[1]
     rc = _lib().rb_stream_norm(ptr(x), x.stride(0), ptr(y1), ptr(y2), y.stride(0) if y is not None else 0, ptr(experts), ptr(expert_weights),
-                               experts.stride(0) if experts is not None else 0, expert_weights.shape[1] if experts is not None else 0,
-                               ptr(copy), copy.stride(0) if copy is not None else 0, ptr(h), h.stride(0) if h is not None else 0, ptr(weight),
+                               experts.stride(0) if experts is not None else 0, k, ptr(side), side.stride(0) if side is not None else 0,
+                               ptr(side_weight), mult, ptr(copy), copy.stride(0) if copy is not None else 0, ptr(h), h.stride(0) if h is not None else 0, ptr(weight),
                                ptr(rows), x.shape[0], _ACT[act.dtype], n, d, x.shape[1], eps, ptr(status_tensor(x.device)),
                                stream_handle(x.device))
     check_rc(rc, "rb_stream_norm")
+
+
+def token_side(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col: int, out: torch.Tensor, n: int) -> None:
+    """``out[t, :n] = gelu_tanh(z[t, :n]) * table[ids[t], col : col + n]``, ``z`` in fp32."""
+    T = ids.numel()
+    if not z.is_cuda:
+        g = torch.nn.functional.gelu(z[:T, :n], approximate="tanh")
+        out[:T, :n] = (g * table[ids.long(), col:col + n].float()).to(out.dtype)
+        return
+    assert z.dtype == torch.float32 and z.stride(1) == out.stride(1) == table.stride(1) == 1 and out.dtype == table.dtype and ids.is_contiguous()
+    rc = _lib().rb_token_side(ptr(z), z.stride(0), ptr(ids), ptr(table), table.stride(0), col, ptr(out), out.stride(0), n, T, table.shape[0],
+                              _ACT[out.dtype], ptr(status_tensor(z.device)), stream_handle(z.device))
+    check_rc(rc, "rb_token_side")
 
 
 def layernorm_reference(v: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float) -> torch.Tensor:
@@ -299,14 +324,17 @@ def layernorm_rows(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float
     check_rc(rc, "rb_layernorm")
 
 
-def clamped_glu_reference(gu: torch.Tensor, limit: float) -> torch.Tensor:
+def clamped_glu_reference(gu: torch.Tensor, limit: float | None) -> torch.Tensor:
     g, u = gu.float().chunk(2, dim=-1)
+    if limit is None:
+        return torch.nn.functional.silu(g) * u
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
     return g * torch.sigmoid(1.702 * g) * (u + 1)
 
 
-def clamped_glu(gu: torch.Tensor, limit: float, out: torch.Tensor | None = None) -> torch.Tensor:
-    """``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, +-limit)`` for ``gu = [gate | up] [T, 2F]``."""
+def clamped_glu(gu: torch.Tensor, limit: float | None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, +-limit)`` for ``gu = [gate | up] [T, 2F]``;
+    without a limit ``silu(gate) * up``."""
     T, F2 = gu.shape
     if out is None:
         out = torch.empty(T, F2 // 2, dtype=gu.dtype, device=gu.device)
@@ -314,7 +342,7 @@ def clamped_glu(gu: torch.Tensor, limit: float, out: torch.Tensor | None = None)
         out.copy_(clamped_glu_reference(gu, limit))
         return out
     assert gu.is_contiguous() and out.is_contiguous()
-    check_rc(_lib().rb_clamped_glu(ptr(gu), ptr(out), _ACT[gu.dtype], T, F2 // 2, limit, stream_handle(gu.device)), "rb_clamped_glu")
+    check_rc(_lib().rb_clamped_glu(ptr(gu), ptr(out), _ACT[gu.dtype], T, F2 // 2, limit or 0.0, stream_handle(gu.device)), "rb_clamped_glu")
     return out
 
 

@@ -1,9 +1,9 @@
 """Routed experts on one GPU (``csrc/moe_sm100.cu`` routing and row movement, grouped GEMMs) with a PyTorch twin.
 
-A router's logits -> the ``top`` largest softmax scores divided by their sum; rows are gathered expert by expert, the
-clamped gated unit runs as two grouped products (tile tables made on the device, so the layer fits a CUDA graph) and the
-second one stores every result row at its ``(token, choice)`` place. The weighted sum over the choices is left to whoever
-adds the result to the residual stream (``elementwise.stream_norm``).
+A router's logits -> the ``top`` largest softmax or sigmoid scores, divided by their sum or not; rows are gathered expert by
+expert (times their weight, when it belongs to the input), the gated unit runs as two grouped products (tile tables made on the
+device, so the layer fits a CUDA graph) and the second one stores every result row at its ``(token, choice)`` place. The
+weighted sum over the choices is left to whoever adds the result to the residual stream (``elementwise.stream_norm``).
 """
 
 from __future__ import annotations
@@ -29,9 +29,9 @@ def _up(n: int, m: int) -> int:
 def _lib() -> ctypes.CDLL:
     lib = _native.load("rb_moe")
     if not getattr(lib, "_rb_experts_typed", False):
-        lib.rb_experts_route.argtypes = [c_vp, c_ll] + [c_int] * 3 + [c_vp] * 4
+        lib.rb_experts_route.argtypes = [c_vp, c_ll] + [c_int] * 5 + [c_vp] * 4
         lib.rb_experts_plan.argtypes = [c_vp, c_int, c_vp, c_int, c_int, c_vp, c_vp, c_int, c_int, c_vp, c_vp, c_int, c_vp, c_vp, c_vp]
-        lib.rb_experts_gather.argtypes = [c_vp, c_ll, c_vp] + [c_int] * 4 + [c_vp] * 4 + [c_ll, c_int, c_vp, c_vp]
+        lib.rb_experts_gather.argtypes = [c_vp, c_ll, c_vp] + [c_int] * 4 + [c_vp] * 4 + [c_ll, c_int, c_vp, c_int, c_vp, c_vp]
         for f in ("rb_experts_route", "rb_experts_plan", "rb_experts_gather"):
             getattr(lib, f).restype = c_int
         lib._rb_experts_typed = True
@@ -44,19 +44,24 @@ class ExpertsGeometry:
     top: int
     ff: int
     width: int           # padded row width of the stream
-    limit: float
+    limit: float | None  # of the clamped unit; None: silu(gate) * up
     bn: int              # tile width of the grouped products (gate and up rows are interleaved in halves of it when it is fused)
     fused: bool          # the unit runs in the first product's epilogue
+    scores: str = "softmax"
+    normalize: bool = True
+    scale_input: bool = False    # a choice's weight multiplies the expert's input, not its output
 
     @property
     def ffp(self) -> int:
         return _up(self.ff, self.bn // 2 if self.fused else 8)
 
     @staticmethod
-    def make(experts: int, top: int, ff: int, width: int, limit: float, dtype: torch.dtype) -> "ExpertsGeometry":
+    def make(experts: int, top: int, ff: int, width: int, limit: float | None, dtype: torch.dtype, scores: str = "softmax", normalize: bool = True,
+             scale_input: bool = False) -> "ExpertsGeometry":
         if experts > MAX_EXPERTS or top > MAX_TOP:
             raise ValueError(f"the expert kernels take up to {MAX_EXPERTS} experts, {MAX_TOP} per token")
-        return ExpertsGeometry(experts, top, ff, width, limit, 128 if dtype == torch.bfloat16 else 64, dtype == torch.bfloat16)
+        return ExpertsGeometry(experts, top, ff, width, limit, 128 if dtype == torch.bfloat16 else 64, dtype == torch.bfloat16, scores, normalize,
+                               scale_input)
 
 
 class ExpertsScratch:
@@ -91,9 +96,10 @@ def pack_experts(gates, ups, downs, geo: ExpertsGeometry, wgu: torch.Tensor, wd:
         wd3[e, :dn.shape[0], :geo.ff].copy_(dn)
 
 
-def route_reference(logits: torch.Tensor, top: int) -> tuple[torch.Tensor, torch.Tensor]:
-    w, idx = logits.float().softmax(-1).topk(top, -1)
-    return idx.to(torch.int32), w / (w.sum(-1, keepdim=True) + 1e-20)
+def route_reference(logits: torch.Tensor, top: int, scores: str = "softmax", normalize: bool = True) -> tuple[torch.Tensor, torch.Tensor]:
+    s = logits.float().softmax(-1) if scores == "softmax" else torch.sigmoid(logits.float())
+    w, idx = s.topk(top, -1)
+    return idx.to(torch.int32), w / (w.sum(-1, keepdim=True) + 1e-20) if normalize else w
 
 
 def _grouped(a, b, c, geo: ExpertsGeometry, sc: ExpertsScratch, group_n: int, K: int, tiles, count, unit: bool, row_dst) -> None:
@@ -114,7 +120,7 @@ def _grouped(a, b, c, geo: ExpertsGeometry, sc: ExpertsScratch, group_n: int, K:
     args.tile_table, args.num_tiles_ptr = tiles.data_ptr(), count.data_ptr()
     args.group_n, args.max_tiles = group_n, sc.max_tiles
     if unit:
-        args.swiglu, args.glu_kind, args.glu_limit = 1, 1, geo.limit
+        args.swiglu, args.glu_kind, args.glu_limit = 1, int(geo.limit is not None), geo.limit or 0.0
     args.row_dst = row_dst.data_ptr() if row_dst is not None else None
     check_rc(_gemm_lib().rb_gemm_bf16_ex(ctypes.byref(args), stream_handle(a.device)), "rb_gemm_bf16_ex(experts)")
 
@@ -122,7 +128,8 @@ def _grouped(a, b, c, geo: ExpertsGeometry, sc: ExpertsScratch, group_n: int, K:
 def experts_plan(logits, geo: ExpertsGeometry, sc: ExpertsScratch) -> None:
     """Choices and weights of every token, the experts' row ranges and the tile tables of both products."""
     T, s, st = logits.shape[0], stream_handle(logits.device), ptr(status_tensor(logits.device))
-    check_rc(_lib().rb_experts_route(ptr(logits), logits.stride(0), T, geo.experts, geo.top, ptr(sc.idx), ptr(sc.w), ptr(sc.counts), s), "rb_experts_route")
+    check_rc(_lib().rb_experts_route(ptr(logits), logits.stride(0), T, geo.experts, geo.top, int(geo.scores == "sigmoid"), int(geo.normalize), ptr(sc.idx),
+                                     ptr(sc.w), ptr(sc.counts), s), "rb_experts_route")
     check_rc(_lib().rb_experts_plan(ptr(sc.counts), geo.experts, ptr(sc.offsets), 2 * geo.ffp, geo.bn, ptr(sc.tiles_gu), ptr(sc.ntiles), geo.width,
                                     geo.bn, ptr(sc.tiles_dn), sc.ntiles.data_ptr() + 4, sc.max_tiles, ptr(sc.cursor), st, s), "rb_experts_plan")
 
@@ -130,7 +137,8 @@ def experts_plan(logits, geo: ExpertsGeometry, sc: ExpertsScratch) -> None:
 def experts_gather(h, geo: ExpertsGeometry, sc: ExpertsScratch) -> None:
     es = h.element_size()
     check_rc(_lib().rb_experts_gather(ptr(h), h.stride(0) * es, ptr(sc.idx), h.shape[0], geo.top, geo.width * es, geo.experts, ptr(sc.cursor), ptr(sc.xp),
-                                      ptr(sc.ret), ptr(sc.y), geo.width * es, sc.cap, ptr(status_tensor(h.device)), stream_handle(h.device)),
+                                      ptr(sc.ret), ptr(sc.y), geo.width * es, sc.cap, ptr(sc.w) if geo.scale_input else None, int(es == 4),
+                                       ptr(status_tensor(h.device)), stream_handle(h.device)),
              "rb_experts_gather")
 
 
@@ -145,9 +153,9 @@ def experts_down(geo: ExpertsGeometry, sc: ExpertsScratch, wd) -> None:
     _grouped(sc.act, wd, sc.y, geo, sc, geo.width, geo.ffp, sc.tiles_dn, sc.ntiles[1:], False, sc.ret)
 
 
-def experts_forward(h, logits, geo: ExpertsGeometry, sc: ExpertsScratch, wgu, wd) -> tuple[torch.Tensor, torch.Tensor]:
-    """Results ``[T * top, width]`` of every token's chosen experts and their weights ``[T, top]`` for ``h [T, width]`` and the
-    router's logits ``[T, >= experts]`` (fp32)."""
+def experts_forward(h, logits, geo: ExpertsGeometry, sc: ExpertsScratch, wgu, wd) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """Results ``[T * top, width]`` of every token's chosen experts and the weights ``[T, top]`` they are still to be multiplied by
+    (None with ``scale_input``) for ``h [T, width]`` and the router's logits ``[T, >= experts]`` (fp32)."""
     T, k = h.shape[0], geo.top
     assert T * k <= sc.cap and logits.dtype == torch.float32
     if h.is_cuda:
@@ -155,13 +163,14 @@ def experts_forward(h, logits, geo: ExpertsGeometry, sc: ExpertsScratch, wgu, wd
         experts_gather(h, geo, sc)
         experts_up(geo, sc, wgu, T)
         experts_down(geo, sc, wd)
-        return sc.y[:T * k], sc.w[:T]
-    idx, w = route_reference(logits[:, :geo.experts], k)
+        return sc.y[:T * k], None if geo.scale_input else sc.w[:T]
+    idx, w = route_reference(logits[:, :geo.experts], k, geo.scores, geo.normalize)
     sc.idx[:T], sc.w[:T] = idx, w
     y = sc.y[:T * k].view(T, k, geo.width)
     gu3, wd3 = wgu.view(geo.experts, 2 * geo.ffp, -1), wd.view(geo.experts, geo.width, geo.ffp)
     for e in range(geo.experts):
         tok, slot = (idx == e).nonzero(as_tuple=True)
         if tok.numel():
-            y[tok, slot] = (clamped_glu_reference(h[tok].float() @ gu3[e].float().T, geo.limit) @ wd3[e].float().T).to(y.dtype)
-    return sc.y[:T * k], sc.w[:T]
+            x = h[tok].float() * w[tok, slot, None] if geo.scale_input else h[tok].float()
+            y[tok, slot] = (clamped_glu_reference(x @ gu3[e].float().T, geo.limit) @ wd3[e].float().T).to(y.dtype)
+    return sc.y[:T * k], None if geo.scale_input else sc.w[:T]

@@ -52,8 +52,9 @@ def _lib() -> ctypes.CDLL:
     lib = _native.load("rb_attn")
     if not getattr(lib, "_rb_kv_typed", False):
         lib.rb_kv_append.argtypes = [c_vp, c_ll, c_vp, c_vp, c_float, c_int, c_vp] + [c_int] * 6 + [c_vp, c_vp]
-        lib.rb_kv_decode.argtypes = [c_vp, c_ll, c_int, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp] + [c_int] * 8 + [c_float, c_vp, c_vp]
-        lib.rb_kv_simple.argtypes = [c_vp, c_ll, c_int, c_vp, c_vp, c_vp, c_vp, c_vp, c_vp] + [c_int] * 9 + [c_float, c_vp, c_vp]
+        gate = [c_vp, c_ll, c_vp, c_ll, c_float]
+        lib.rb_kv_decode.argtypes = [c_vp, c_ll] + [c_vp] * 5 + gate + [c_vp, c_ll, c_vp] + [c_int] * 10 + [c_float, c_vp, c_vp]
+        lib.rb_kv_simple.argtypes = [c_vp, c_ll] + [c_vp] * 6 + gate + [c_vp, c_ll] + [c_int] * 11 + [c_float, c_vp, c_vp]
         lib.rb_kv_gate.argtypes = [c_vp, c_vp, c_vp, c_vp, c_ll] + [c_int] * 5 + [c_vp]
         for f in ("rb_kv_append", "rb_kv_decode", "rb_kv_simple", "rb_kv_gate"):
             getattr(lib, f).restype = c_int
@@ -107,17 +108,18 @@ def kv_attention(proj, geo: KeyValueGeometry, cache, block_tables, cu_q, seq_len
         return
     H, G, D, B, dev = geo.heads, geo.kv_heads, geo.dp, seq_lens.shape[0], proj.device
     assert cache.is_contiguous() and block_tables.stride(1) == 1 and out.is_contiguous() and sink.dtype == torch.float32
+    gate = (proj.data_ptr() + proj.element_size() * geo.gate_col, proj.stride(0), None, 0, 1.0)
     if proj.dtype == torch.float32 or not geo.tensor_core:
-        rc = _lib().rb_kv_simple(ptr(proj), proj.stride(0), geo.gate_col, ptr(cache), ptr(block_tables), ptr(cu_q), ptr(seq_lens), ptr(sink), ptr(out),
-                                 H, G, D, block_tables.stride(0), cache.shape[0], B, rows, max_q, _DT[proj.dtype], scale,
+        rc = _lib().rb_kv_simple(ptr(proj), proj.stride(0), ptr(cache), None, ptr(block_tables), ptr(cu_q), ptr(seq_lens), ptr(sink), *gate, ptr(out),
+                                 out.stride(0), H, G, D, block_tables.stride(0), cache.shape[0], B, rows, max_q, 0, 0, _DT[proj.dtype], scale,
                                  ptr(status_tensor(dev)), stream_handle(dev))
         check_rc(rc, "rb_kv_simple")
         return
     if cu_q is None:
         n_single = B
     if n_single > 0:
-        rc = _lib().rb_kv_decode(ptr(proj), proj.stride(0), geo.gate_col, ptr(cache), ptr(block_tables), ptr(seq_lens), ptr(sink), ptr(out),
-                                 ptr(workspace), n_single, H, G, D, block_tables.stride(0), cache.shape[0], KV_BLOCK, splits, scale,
+        rc = _lib().rb_kv_decode(ptr(proj), proj.stride(0), ptr(cache), None, ptr(block_tables), ptr(seq_lens), ptr(sink), *gate, ptr(out),
+                                 out.stride(0), ptr(workspace), n_single, H, G, D, block_tables.stride(0), cache.shape[0], KV_BLOCK, splits, 0, 0, scale,
                                  ptr(status_tensor(dev)), stream_handle(dev))
         check_rc(rc, "rb_kv_decode", 2 if splits > 1 else 1)
     if n_single < B:

@@ -1,13 +1,16 @@
 """Recurrent mixers with a matrix state per head (csrc/recurrent_sm100.cu) and their PyTorch twins.
 
-Both kinds write ``k v^T`` into a state that decays and read it with ``q``::
+All kinds write ``k v^T`` into a state that decays and read it with ``q``::
 
     S_t = a_t S_(t-1) + b_t k_t v_t^T          o_t = S_t^T q_t
 
 * lightning: ``a`` is a constant of the head, ``b = 1`` (queries, keys and values come through SiLU, applied by the projection);
 * matrix memory (mLSTM): capped gate logits ``i``, ``f``; ``log a = logsigmoid(f)``, ``b = exp(i)``, held relative to a running
   maximum ``m`` (from 0) so that nothing overflows; a second state ``n`` takes ``k`` alone and divides the output by
-  ``max(|n . q|, exp(-m)) + 1e-6``.
+  ``max(|n . q|, exp(-m)) + 1e-6``;
+* time mixing (RWKV): ``a`` is a vector, ``exp(-exp(z_t + w0))`` per key channel, ``b = 1``; ``o_t`` reads the state in front of the
+  token and the token's own ``k v^T`` times a bonus ``u`` per key channel. Its projections read mixes of a token with the one
+  before (``token_shift``).
 
 A sequence owns a slot of the state; one whose first new token is at position 0 starts from zero whatever the slot holds.
 The state, the decays, the gates and the outputs are fp32; queries, keys and values come in the activation type.
@@ -22,6 +25,7 @@ import torch
 
 from .. import _native
 from ._util import check_rc, ptr, status_tensor, stream_handle
+from .grouped import look_back, move_history
 
 c_int, c_ll, c_float, c_vp = ctypes.c_int, ctypes.c_longlong, ctypes.c_float, ctypes.c_void_p
 _DT = {torch.bfloat16: 0, torch.float32: 1}
@@ -42,7 +46,7 @@ class RecurrentGeometry:
     dim: int
     vdim: int
     silu: bool                   # q, k and v come through SiLU (the projection applies it)
-    gated: bool                  # mLSTM gates and normaliser (otherwise a constant decay)
+    gated: bool                  # mLSTM gates and normaliser (otherwise a decay per head or key channel)
 
     @property
     def kp(self) -> int:
@@ -88,16 +92,27 @@ class RecurrentState:
         return RecurrentState(*(torch.zeros(*lead, *tail, dtype=torch.float32, device=device) for tail in ((geo.kp, STATE_COLS), (geo.kp,), ())))
 
 
+@dataclass
+class TimeMix:
+    """What time mixing adds to a recurrence: ``z [T, H*kp]`` fp32 with the decay ``exp(-exp(z + w0))``, the bonus of the current token."""
+
+    z: torch.Tensor
+    w0: torch.Tensor             # [H*kp]
+    bonus: torch.Tensor          # [H*kp]
+
+
 def _lib() -> ctypes.CDLL:
     lib = _native.load("rb_recurrent")
     if not getattr(lib, "_rb_typed", False):
         lib.rb_recurrent_scan.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float, c_float] + [c_vp] * 6
-                                          + [c_vp, c_ll] + [c_int] * 9 + [c_vp, c_vp])
+                                          + [c_vp, c_ll] + [c_int] * 8 + [c_vp, c_ll, c_vp, c_vp, c_int, c_vp, c_vp])
+        lib.rb_token_shift.argtypes = [c_vp, c_ll, c_vp, c_int, c_vp, c_ll, c_ll, c_vp, c_vp, c_vp, c_vp] + [c_int] * 5 + [c_vp, c_vp]
+        lib.rb_tanh_parts.argtypes = [c_vp, c_int, c_vp, c_vp, c_int, c_vp]
         lib.rb_recurrent_chunks.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float, c_float] + [c_vp] * 9 + [c_ll, c_vp]
                                             + [c_int] * 8 + [c_vp, c_vp])
         lib.rb_recurrent_chunk_workspace.argtypes, lib.rb_recurrent_chunk_workspace.restype = [c_int] * 4, c_ll
-        lib.rb_gated_norm.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_ll] + [c_int] * 6 + [c_float, c_vp]
-        for f in ("rb_recurrent_scan", "rb_recurrent_chunks", "rb_gated_norm"):
+        lib.rb_gated_norm.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_ll] + [c_int] * 7 + [c_float, c_vp]
+        for f in ("rb_recurrent_scan", "rb_recurrent_chunks", "rb_gated_norm", "rb_token_shift", "rb_tanh_parts"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -119,15 +134,18 @@ def _split(proj, geo: RecurrentGeometry):
 
 
 def recurrent_scan(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, cap: float, state: RecurrentState, slots, cu_q, seq_lens,
-                   out, rows: int, n_seq: int, first: int = 0) -> None:
+                   out, rows: int, n_seq: int, first: int = 0, mix: TimeMix | None = None) -> None:
     """Token-by-token form for the sequences ``first .. n_seq - 1`` (the last one ends at packed row ``rows``): ``out [T, H*vp]``
     fp32, state updated.
 
     ``proj [T, q | k | v | gate]``, ``small [T, i | f]`` fp32 (gated kinds), ``slots [B]`` (negative: padding), ``cu_q``
-    ``[B+1]`` (None: one row per sequence), ``seq_lens [B]`` with the new tokens."""
+    ``[B+1]`` (None: one row per sequence), ``seq_lens [B]`` with the new tokens; ``mix`` for time mixing."""
     H, KP, VP = geo.heads, geo.kp, geo.vp
     if not proj.is_cuda:
         q, k, v = _split(proj[:rows], geo)
+        if mix is not None:
+            keep = torch.exp(-torch.exp(mix.z[:rows] + mix.w0)).view(-1, H, KP)
+            bonus = mix.bonus.view(H, KP, 1)
         if geo.gated:
             gi, gf = capped_gates(small[:rows], bias_i, bias_f, cap)
         for b in range(first, n_seq):
@@ -141,6 +159,11 @@ def recurrent_scan(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, c
             S = state.s[slot].permute(0, 2, 1, 3).reshape(H, KP, VP)
             n, m = state.n[slot, :, 0], state.m[slot, :, 0]
             for t in range(t0, t1):
+                if mix is not None:
+                    kv = k[t][:, :, None] * v[t][:, None, :]
+                    out[t] = torch.einsum("hkv,hk->hv", S + bonus * kv, q[t]).reshape(-1)
+                    S = keep[t][:, :, None] * S + kv
+                    continue
                 if geo.gated:
                     new = torch.maximum(gf[t] + m, gi[t])
                     a, w = torch.exp(gf[t] + m - new), torch.exp(gi[t] - new)
@@ -163,8 +186,9 @@ def recurrent_scan(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f, c
                                   ptr(bias_i), ptr(bias_f), cap, geo.dim ** -0.5 if geo.gated else 1.0, ptr(state.s), ptr(state.n), ptr(state.m),
                                   ptr(slots[first:]), ptr(cu_q[first:]) if cu_q is not None else None, ptr(seq_lens[first:]), ptr(out), out.stride(0), H, geo.dim, KP, VP,
                                   n_seq - first, state.s.shape[0],
-                                  int(geo.gated), rows, _DT[proj.dtype], ptr(status_tensor(proj.device)),
-                                  stream_handle(proj.device))
+                                  int(geo.gated), rows, ptr(mix.z) if mix is not None else None, mix.z.stride(0) if mix is not None else 0,
+                                  ptr(mix.w0) if mix is not None else None, ptr(mix.bonus) if mix is not None else None, _DT[proj.dtype],
+                                  ptr(status_tensor(proj.device)), stream_handle(proj.device))
     check_rc(rc, "rb_recurrent_scan")
 
 
@@ -212,17 +236,50 @@ def chunk_workspace(n_chunks: int, geo: RecurrentGeometry) -> int:
     return int(_lib().rb_recurrent_chunk_workspace(n_chunks, geo.heads, geo.kp, geo.vp))
 
 
-def gated_norm(o, weight, gate, geo: RecurrentGeometry, eps: float, out, per_head: bool) -> None:
-    """``out = o / rms(o) * weight * sigmoid(gate)`` on ``[T, H*vp]``; the mean square is taken over one head's ``vdim`` channels
-    (``per_head``) or over all heads'."""
+def token_shift(h, mu, out, history, cu_q, positions, state_slots) -> None:
+    """``out[s, t] = h_t + (h_(t-1) - h_t) mu[s]`` for the packed rows ``h [T, w]``, ``mu [mixes, w]`` fp32, ``out [mixes, >= T, w]``. The token
+    before a portion comes from ``history [slots, 1, w]`` (zeros before a sequence), which moves on."""
+    T = h.shape[0]
+    if not h.is_cuda:
+        back = look_back(h, 1, history, cu_q, positions, state_slots)[:, 0].float()
+        for s in range(mu.shape[0]):
+            out[s, :T] = (h.float() + (back - h.float()) * mu[s]).to(out.dtype)
+        move_history(h, history, cu_q, state_slots)
+        return
+    assert h.stride(1) == out.stride(2) == 1 and mu.is_contiguous() and history.is_contiguous() and mu.dtype == torch.float32
+    rc = _lib().rb_token_shift(ptr(h), h.stride(0), ptr(mu), mu.shape[0], ptr(out), out.stride(0), out.stride(1), ptr(history), ptr(cu_q), ptr(positions),
+                               ptr(state_slots), T if cu_q is None else cu_q.numel() - 1, history.shape[0], h.shape[1], T, _DT[h.dtype],
+                               ptr(status_tensor(h.device)), stream_handle(h.device))
+    check_rc(rc, "rb_token_shift", 1 if cu_q is None else 2)
+
+
+def tanh_parts(x, out) -> None:
+    """``tanh`` of contiguous fp32 rows ``x [T, n]`` as operand of an exact product: fp32 ``out [T, n]``, or bf16 ``out [T, 2n]`` with what
+    the first ``n`` columns lack in the others."""
+    T, n = x.shape
+    assert out.shape[1] == (n if out.dtype == torch.float32 else 2 * n)
+    if not x.is_cuda:
+        v = torch.tanh(x)
+        out[:T, :n] = v.to(out.dtype)
+        if out.dtype != torch.float32:
+            out[:T, n:] = (v - out[:T, :n].float()).to(out.dtype)
+        return
+    assert x.is_contiguous() and out.is_contiguous()
+    f32 = out.dtype == torch.float32
+    check_rc(_lib().rb_tanh_parts(ptr(x), n, None if f32 else ptr(out), ptr(out) if f32 else None, T, stream_handle(x.device)), "rb_tanh_parts")
+
+
+def gated_norm(o, weight, gate, geo: RecurrentGeometry, eps: float, out, per_head: bool, silu: bool = False) -> None:
+    """``out = o / rms(o) * weight * sigmoid(gate)`` (``silu``: times ``silu(gate)``) on ``[T, H*vp]``; the mean square is taken over one
+    head's ``vdim`` channels (``per_head``) or over all heads'."""
     T, H, VP = o.shape[0], geo.heads, geo.vp
     if not o.is_cuda:
         x = o.view(T, H, VP)
         ms = x.pow(2).sum(-1) / geo.vdim if per_head else (x.pow(2).sum((1, 2)) / (H * geo.vdim))[:, None].expand(T, H)
-        y = x * torch.rsqrt(ms + eps)[..., None] * weight.view(1, H, VP) * torch.sigmoid(gate.float().view(T, H, VP))
+        y = x * torch.rsqrt(ms + eps)[..., None] * weight.view(1, H, VP) * (torch.nn.functional.silu if silu else torch.sigmoid)(gate.float().reshape(T, H, VP))
         out[:T] = y.reshape(T, H * VP).to(out.dtype)
         return
     assert o.dtype == torch.float32 and o.stride(1) == gate.stride(1) == out.stride(1) == 1 and gate.dtype == out.dtype
     rc = _lib().rb_gated_norm(ptr(o), o.stride(0), ptr(weight), ptr(gate), gate.stride(0), ptr(out), out.stride(0), H, geo.vdim, VP, int(per_head),
-                              T, _DT[out.dtype], eps, stream_handle(o.device))
+                              int(silu), T, _DT[out.dtype], eps, stream_handle(o.device))
     check_rc(rc, "rb_gated_norm")
