@@ -9,6 +9,7 @@
 //   chunked     long portions, 128 tokens at a time on the tensor cores (tcgen05), in four launches: the gates, what every chunk
 //               adds to the state (all chunks at once), the state in front of every chunk (one pass over the chunks), the
 //               outputs (all chunks at once)
+//   time mixing of long portions: chunked in the same way, in three launches
 //   gated_norm  RMS norm per head or over all heads, times sigmoid(gate), to the activation type
 //
 // State: s [slots, H, tiles, KP, 32], n [slots, H, tiles, KP], m [slots, H, tiles], all fp32. A tile of 32 value channels keeps its
@@ -1082,6 +1083,473 @@ static int launch_chunks(const ChunkParams& p, int n_chunks, int n_seq, cudaStre
 }
 
 // ------------------------------------------------------------------------------------------
+// Time mixing in chunks. With A_t the summed log2 decays of a key channel up to and including token t of the chunk (A_-1 = 0), all
+// of them <= 0 and falling, and S the state in front of the chunk,
+//
+//   o_t = (r_t 2^A_(t-1))^T S + sum_{j<t} P_tj v_j + P_tt v_t,   P_tj = sum_c r_t k_j 2^(A_(t-1) - A_j),   P_tt = sum_c r_t u k_t
+//   S'  = diag(2^A_last) S + sum_j (k_j 2^(A_last - A_j)) v_j^T
+//
+// Every exponent above is <= 0, but P does not factor over t and j without one that is not: 2^-A_j overflows. So P is made in
+// blocks of 16 x 16 below the diagonal, whose two factors are taken relative to the token in front of the block row, both <= 1
+// (mma.sync, their operands are made in registers); of a block on the diagonal the lower left quarter goes the same way
+// and the two 8 x 8 triangles pair by pair in fp32. P V and the state's part run on tcgen05. Three launches: what every chunk
+// adds to the state (z becomes A on the way), the chain of states, outputs with the head's norm and the output gate.
+// ------------------------------------------------------------------------------------------
+constexpr float MIX_MOST = 64.f;      // a token that keeps less than 2^-64 keeps nothing; larger sums would cost A its last digits
+
+struct MixParams {
+  const __nv_bfloat16* proj;     // [T, ld]: r | k | v | gate
+  long long ld;
+  int k_col, v_col, g_col;
+  float* z;                      // [T, ldz] decay logits, then A
+  long long ldz;
+  const float* w0;               // [H * KP]
+  const float* bonus;            // [H * KP]
+  const int4* chunks;
+  const int* seq_chunks;
+  const int* slots;
+  const int* seq_lens;
+  const int* cu_q;
+  float* s;                      // [slots, H, tiles, KP, 32]
+  float* u;                      // [chunks, H, tiles, KP, 32]
+  float* last;                   // [chunks, H, KP] A of the chunk's last token
+  __nv_bfloat16* s_hi;           // [chunks, H, VP/64, KP, 64]
+  __nv_bfloat16* s_lo;
+  const float* norm;             // [H * VP]
+  float eps;
+  __nv_bfloat16* out;            // [T, ldo]
+  long long ldo;
+  int H, dk, KP, VP, num_slots;
+  int* status;
+};
+
+template <int DK>
+struct MixStateCfg {
+  static constexpr int kKBytes = CH * DK * 2;
+  static constexpr int kSmem = 1024 + 2 * kKBytes + DK / 64 * CH_CHUNK;      // weighted keys in two parts, V
+  static constexpr int kCols = DK;
+};
+
+// What a chunk of one head adds to the state, and A. VP == KP == DK.
+template <int DK>
+__global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_state_kernel(const MixParams p) {
+  using Cfg = MixStateCfg<DK>;
+  constexpr int SEGS = CHT / DK, SEG = CH / SEGS;       // a thread has one channel of SEG tokens
+  extern __shared__ __align__(128) uint8_t smem_raw[];
+  __shared__ float sums[SEGS][DK];
+  __shared__ __align__(8) uint64_t done;
+  __shared__ uint32_t tmem_base_smem;
+  __shared__ int abort_flag;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* hi = smem_raw + (base - smem_u32(smem_raw));
+  uint8_t* lo = hi + Cfg::kKBytes;
+  const uint32_t v_s = base + 2 * Cfg::kKBytes;
+  if (tid == 0) {
+    abort_flag = 0;
+    mbar_init(smem_u32(&done), 1);
+    fence_mbar_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_smem), Cfg::kCols);
+    tmem_relinquish();
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x / p.H, h = blockIdx.x % p.H;
+  const int4 ck = p.chunks[c];
+  const int row0 = ck.x, n = ck.y;
+  const long long ch = (long long)c * p.H + h;
+  const __nv_bfloat16* rows = p.proj + (long long)row0 * p.ld;
+  chunk_load<DK>(v_s, rows + p.v_col + h * p.VP, p.ld, n);
+  const int col = tid % DK, seg = tid / DK, t0 = seg * SEG;
+  float* z = p.z + (long long)row0 * p.ldz + h * p.KP + col;
+  const __nv_bfloat16* k = rows + p.k_col + h * p.KP + col;
+  const float w0 = p.w0[h * p.KP + col];
+  float A[SEG], run = 0.f;
+#pragma unroll
+  for (int i = 0; i < SEG; ++i) A[i] = t0 + i < n ? z[(long long)(t0 + i) * p.ldz] : 0.f;
+#pragma unroll
+  for (int i = 0; i < SEG; ++i) {
+    if (t0 + i < n) run -= fminf(expf(A[i] + w0) * LOG2E, MIX_MOST);
+    A[i] = run;
+  }
+  sums[seg][col] = run;
+  __syncthreads();
+  float before = 0.f, total = 0.f;
+#pragma unroll
+  for (int i = 0; i < SEGS; ++i) {
+    if (i < seg) before += sums[i][col];
+    total += sums[i][col];
+  }
+  if (seg == 0) p.last[ch * p.KP + col] = total;
+#pragma unroll
+  for (int i = 0; i < SEG; ++i) {
+    const int t = t0 + i;
+    float x = 0.f;
+    if (t < n) {
+      A[i] += before;
+      z[(long long)t * p.ldz] = A[i];
+      x = __bfloat162float(k[(long long)t * p.ld]) * chunk_exp2(total - A[i]);
+    }
+    const __nv_bfloat16 a = __float2bfloat16_rn(x);
+    const uint32_t at = (col >> 6) * CH_CHUNK + chunk_addr(t, (col & 63) >> 3) + (col & 7) * 2;
+    *reinterpret_cast<__nv_bfloat16*>(hi + at) = a;
+    *reinterpret_cast<__nv_bfloat16*>(lo + at) = __float2bfloat16_rn(x - __bfloat162float(a));
+  }
+  cp_async_wait_all();
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_base_smem;
+  if (warp == 0 && elect_one_sync()) {
+    constexpr uint32_t idesc = make_idesc_bf16(DK, 64, 1, 1);
+#pragma unroll
+    for (int z64 = 0; z64 < DK / 64; ++z64)
+#pragma unroll
+      for (int part = 0; part < 2; ++part)
+#pragma unroll
+        for (int kk = 0; kk < CH / 16; ++kk) {
+          const uint64_t a = make_smem_desc_sw128(base + part * Cfg::kKBytes + kk * 2048, CH_CHUNK, 1024);
+          const uint64_t b = make_smem_desc_sw128(v_s + z64 * CH_CHUNK + kk * 2048, CH_CHUNK, 1024);
+          umma_bf16(tmem + z64 * 64, a, b, idesc, (part | kk) ? 1u : 0u);
+        }
+    umma_commit(smem_u32(&done));
+  }
+  __syncwarp();
+  bool ok = mbar_wait_bounded(smem_u32(&done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
+  ok = __all_sync(0xffffffffu, ok);
+  tc_fence_after();
+  if (ok) {
+    const int qd = warp & 3, half = warp >> 2;
+    const int r = DK == 128 ? qd * 32 + lane : qd * 16 + lane;        // (a 64-row product: row 16 q + lane in 16 lanes)
+#pragma unroll
+    for (int z64 = 0; z64 < DK / 64; ++z64) {
+      uint32_t v[32];
+      tmem_ld_32x32(tmem + z64 * 64 + half * 32 + ((uint32_t)(qd * 32) << 16), v);
+      tmem_ld_wait();
+      if (DK == 128 || lane < 16) {
+        float4* dst = reinterpret_cast<float4*>(p.u + ((ch * (p.VP / 32) + z64 * 2 + half) * p.KP + r) * 32);
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          dst[i] = make_float4(__uint_as_float(v[4 * i]), __uint_as_float(v[4 * i + 1]), __uint_as_float(v[4 * i + 2]), __uint_as_float(v[4 * i + 3]));
+      }
+    }
+    tc_fence_before();
+  }
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, Cfg::kCols);
+  }
+}
+
+// The state in front of every chunk, and behind the portion: as recurrent_chunk_chain_kernel, with a decay per key row.
+__global__ void __launch_bounds__(256) time_mix_chain_kernel(const MixParams p) {
+  pdl_launch_dependents();
+  const int tiles = p.VP / SC_COLS;
+  const int tile = blockIdx.y % tiles, h = blockIdx.y / tiles, b = blockIdx.z;
+  const int c4 = threadIdx.x & 7, r = blockIdx.x * 32 + (threadIdx.x >> 3);
+  pdl_wait();
+  const int slot = p.slots[b];
+  if (slot < 0 || slot >= p.num_slots) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); return; }
+  const bool fresh = p.seq_lens[b] == p.cu_q[b + 1] - p.cu_q[b];
+  const int c0 = p.seq_chunks[b], c1 = p.seq_chunks[b + 1];
+  float4* st = reinterpret_cast<float4*>(p.s + ((((long long)slot * p.H + h) * tiles + tile) * p.KP + r) * SC_COLS) + c4;
+  const bool live = r < p.dk;
+  float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (!fresh && live) S = *st;
+  for (int cb = c0; cb < c1; cb += CHAIN_AHEAD) {
+    float4 U[CHAIN_AHEAD];
+    float last[CHAIN_AHEAD];
+#pragma unroll
+    for (int i = 0; i < CHAIN_AHEAD; ++i)
+      if (cb + i < c1) {
+        const long long ch = (long long)(cb + i) * p.H + h;
+        U[i] = *(reinterpret_cast<const float4*>(p.u + ((ch * tiles + tile) * p.KP + r) * SC_COLS) + c4);
+        last[i] = p.last[ch * p.KP + r];
+      }
+#pragma unroll
+    for (int i = 0; i < CHAIN_AHEAD; ++i)
+      if (cb + i < c1) {
+        const long long ch = (long long)(cb + i) * p.H + h;
+        const uint32_t h0 = pack_bf16x2(S.x, S.y), h1 = pack_bf16x2(S.z, S.w);
+        const float2 b0 = unpack_bf16x2(h0), b1 = unpack_bf16x2(h1);
+        const long long at = ((ch * (p.VP / 64) + (tile >> 1)) * p.KP + r) * 64 + (tile & 1) * 32 + c4 * 4;
+        *reinterpret_cast<uint2*>(p.s_hi + at) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2*>(p.s_lo + at) = make_uint2(pack_bf16x2(S.x - b0.x, S.y - b0.y), pack_bf16x2(S.z - b1.x, S.w - b1.y));
+        const float a = chunk_exp2(last[i]);
+        S.x = fmaf(a, S.x, U[i].x);
+        S.y = fmaf(a, S.y, U[i].y);
+        S.z = fmaf(a, S.z, U[i].z);
+        S.w = fmaf(a, S.w, U[i].w);
+      }
+  }
+  if (live) *st = S;
+}
+
+__device__ __forceinline__ void mma_16816_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int DK>
+struct MixOutCfg {
+  static constexpr int kTile = CH * DK * 2;                        // r (then r 2^A), k (then V)
+  static constexpr int kA = CH * DK * 4;                           // A, then both parts of the state
+  static constexpr int kSmem = 1024 + 2 * kTile + kA + 2 * CH_CHUNK;
+  static constexpr int kCols = DK;
+};
+
+// Outputs of a chunk of one head. VP == KP == DK.
+template <int DK>
+__global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(const MixParams p) {
+  using Cfg = MixOutCfg<DK>;
+  extern __shared__ __align__(128) uint8_t smem_raw[];
+  __shared__ float row_sum[2][CH];
+  __shared__ __align__(8) uint64_t done;
+  __shared__ uint32_t tmem_base_smem;
+  __shared__ int abort_flag;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  uint8_t* r_p = smem_raw + (base - smem_u32(smem_raw));
+  uint8_t* k_p = r_p + Cfg::kTile;
+  uint8_t* a_p = k_p + Cfg::kTile;
+  uint8_t* w_p = a_p + Cfg::kA;                                    // P [CH, CH]
+  const uint32_t r_s = base, k_s = r_s + Cfg::kTile, a_s = k_s + Cfg::kTile, w_s = a_s + Cfg::kA;
+  if (tid == 0) {
+    abort_flag = 0;
+    mbar_init(smem_u32(&done), 1);
+    fence_mbar_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(&tmem_base_smem), Cfg::kCols);
+    tmem_relinquish();
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x / p.H, h = blockIdx.x % p.H;
+  const int4 ck = p.chunks[c];
+  const int row0 = ck.x, n = ck.y;
+  const long long ch = (long long)c * p.H + h;
+  const __nv_bfloat16* rows = p.proj + (long long)row0 * p.ld;
+  chunk_load<DK>(r_s, rows + h * p.KP, p.ld, n);
+  chunk_load<DK>(k_s, rows + p.k_col + h * p.KP, p.ld, n);
+  {
+    // A: rows of DK floats, 32-byte pieces exchanged by the row's low bits so that eight rows of a fragment meet no bank twice
+    const float* A = p.z + (long long)row0 * p.ldz + h * p.KP;
+#pragma unroll 4
+    for (int i = tid; i < CH * (DK / 4); i += CHT) {
+      const int t = i / (DK / 4), q4 = i % (DK / 4);
+      cp_async16(a_s + t * DK * 4 + ((((q4 >> 1) ^ (t & 7)) << 5) | ((q4 & 1) << 4)), A + (long long)(t < n ? t : 0) * p.ldz + q4 * 4, t < n);
+    }
+  }
+  cp_async_wait_all();
+  __syncthreads();
+  auto a2 = [&](int t, int cc) {                                   // A of channels cc, cc + 1 (cc even); zero in front of the chunk
+    return t < 0 ? make_float2(0.f, 0.f)
+                 : *reinterpret_cast<const float2*>(a_p + t * DK * 4 + ((((cc >> 3) ^ (t & 7)) << 5) | ((cc & 7) << 2)));
+  };
+  auto bf2 = [&](const uint8_t* tile, int t, int cc) {
+    return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(tile + (cc >> 6) * CH_CHUNK + chunk_addr(t, (cc & 63) >> 3) + (cc & 7) * 2));
+  };
+  auto weight_at = [&](int t, int j) { return w_p + (j >> 6) * CH_CHUNK + chunk_addr(t, (j & 63) >> 3) + (j & 7) * 2; };
+  const int g = lane >> 2, cq = 2 * (lane & 3), t0 = warp * 16;    // this warp's block row of P
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {                                    // zero its 16 rows of 256 bytes
+    const int e = lane + i * 32, t = t0 + (e >> 4), u = e & 15;
+    *reinterpret_cast<uint4*>(w_p + (u >> 3) * CH_CHUNK + chunk_addr(t, u & 7)) = make_uint4(0u, 0u, 0u, 0u);
+  }
+  __syncwarp();
+  // r_t 2^(A_(t-1) - A_ref) and k_j 2^(A_ref - A_j) of channels cc, cc + 1
+  auto scaled_r = [&](int t, int cc, float2 ref) {
+    const float2 x = bf2(r_p, t, cc), a = a2(t - 1, cc);
+    return pack_bf16x2(x.x * chunk_exp2(a.x - ref.x), x.y * chunk_exp2(a.y - ref.y));
+  };
+  auto scaled_k = [&](int j, int cc, float2 ref) {
+    const float2 x = bf2(k_p, j, cc), a = a2(j, cc);
+    return pack_bf16x2(x.x * chunk_exp2(ref.x - a.x), x.y * chunk_exp2(ref.y - a.y));
+  };
+  if (t0 < n) {
+    if (warp > 0) {                                                // the blocks left of the diagonal
+      uint32_t fa[DK / 16][4];
+#pragma unroll
+      for (int ks = 0; ks < DK / 16; ++ks) {
+        const int cc = ks * 16 + cq;
+        const float2 ref0 = a2(t0 - 1, cc), ref1 = a2(t0 - 1, cc + 8);
+        fa[ks][0] = scaled_r(t0 + g, cc, ref0);
+        fa[ks][1] = scaled_r(t0 + g + 8, cc, ref0);
+        fa[ks][2] = scaled_r(t0 + g, cc + 8, ref1);
+        fa[ks][3] = scaled_r(t0 + g + 8, cc + 8, ref1);
+      }
+      for (int j0 = 0; j0 < t0; j0 += 8) {
+        float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int ks = 0; ks < DK / 16; ++ks) {
+          const int cc = ks * 16 + cq;
+          mma_16816_bf16(s, fa[ks][0], fa[ks][1], fa[ks][2], fa[ks][3], scaled_k(j0 + g, cc, a2(t0 - 1, cc)),
+                         scaled_k(j0 + g, cc + 8, a2(t0 - 1, cc + 8)));
+        }
+        *reinterpret_cast<uint32_t*>(weight_at(t0 + g, j0 + cq)) = pack_bf16x2(s[0], s[1]);
+        *reinterpret_cast<uint32_t*>(weight_at(t0 + g + 8, j0 + cq)) = pack_bf16x2(s[2], s[3]);
+      }
+    }
+    {                                                              // lower left quarter of the diagonal block
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int ks = 0; ks < DK / 16; ++ks) {
+        const int cc = ks * 16 + cq;
+        const float2 ref0 = a2(t0 + 7, cc), ref1 = a2(t0 + 7, cc + 8);
+        mma_16816_bf16(s, scaled_r(t0 + 8 + g, cc, ref0), 0u, scaled_r(t0 + 8 + g, cc + 8, ref1), 0u, scaled_k(t0 + g, cc, ref0),
+                       scaled_k(t0 + g, cc + 8, ref1));
+      }
+      *reinterpret_cast<uint32_t*>(weight_at(t0 + 8 + g, t0 + cq)) = pack_bf16x2(s[0], s[1]);
+    }
+    if (lane < 28) {                                               // pairs j < t of the two triangles, one per lane
+      int t = 1, j = lane;
+      while (j >= t) { j -= t; ++t; }
+#pragma unroll
+      for (int tri = 0; tri < 2; ++tri) {
+        const int tt = t0 + tri * 8 + t, jj = t0 + tri * 8 + j;
+        float s = 0.f;
+#pragma unroll 4
+        for (int i = 0; i < DK / 2; ++i) {
+          const int cc = 2 * ((i + lane) & (DK / 2 - 1));
+          const float2 x = bf2(r_p, tt, cc), y = bf2(k_p, jj, cc), a = a2(tt - 1, cc), b = a2(jj, cc);
+          s = fmaf(x.x * y.x, chunk_exp2(a.x - b.x), s);
+          s = fmaf(x.y * y.y, chunk_exp2(a.y - b.y), s);
+        }
+        *reinterpret_cast<__nv_bfloat16*>(weight_at(tt, jj)) = __float2bfloat16_rn(s);
+      }
+    }
+    {                                                              // the diagonal: two lanes per token
+      const int t = t0 + (lane & 15);
+      const float* bonus = p.bonus + h * p.KP;
+      float s = 0.f;
+#pragma unroll 4
+      for (int i = 0; i < DK / 4; ++i) {
+        const int cc = (lane >> 4) * (DK / 2) + 2 * i;
+        const float2 x = bf2(r_p, t, cc), y = bf2(k_p, t, cc), u = *reinterpret_cast<const float2*>(bonus + cc);
+        s = fmaf(x.x * y.x, u.x, s);
+        s = fmaf(x.y * y.y, u.y, s);
+      }
+      s += __shfl_xor_sync(0xffffffffu, s, 16);
+      if (lane < 16) *reinterpret_cast<__nv_bfloat16*>(weight_at(t, t)) = __float2bfloat16_rn(s);
+    }
+  }
+  __syncthreads();                                                 // k has been read
+  chunk_load<DK>(k_s, rows + p.v_col + h * p.VP, p.ld, n);
+#pragma unroll 2
+  for (int i = tid; i < CH * (DK / 8); i += CHT) {                 // r 2^A_(t-1), in place
+    const int t = i / (DK / 8), u = i % (DK / 8);
+    uint4* at = reinterpret_cast<uint4*>(r_p + (u >> 3) * CH_CHUNK + chunk_addr(t, u & 7));
+    const uint4 v = *at;
+    auto one = [&](uint32_t x, int cc) {
+      const float2 f = unpack_bf16x2(x), a = a2(t - 1, cc);
+      return pack_bf16x2(f.x * chunk_exp2(a.x), f.y * chunk_exp2(a.y));
+    };
+    *at = make_uint4(one(v.x, u * 8), one(v.y, u * 8 + 2), one(v.z, u * 8 + 4), one(v.w, u * 8 + 6));
+  }
+  __syncthreads();                                                 // A has been read
+  constexpr int PART = DK * DK * 2;                                // one part of the state
+#pragma unroll 4
+  for (int i = tid; i < 2 * (DK / 64) * DK * 8; i += CHT) {        // parts, 64 value channels, key row, 16-byte piece
+    const int part = i / ((DK / 64) * DK * 8), e = i % ((DK / 64) * DK * 8), z64 = e / (DK * 8), r = (e >> 3) % DK, u = e & 7;
+    const __nv_bfloat16* src = (part ? p.s_lo : p.s_hi) + ((ch * (DK / 64) + z64) * DK + r) * 64 + u * 8;
+    cp_async16(a_s + part * PART + z64 * DK * CH_ROWB + chunk_addr(r, u), src, true);
+  }
+  cp_async_wait_all();
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = tmem_base_smem;
+  if (warp == 0 && elect_one_sync()) {
+    constexpr uint32_t idesc = make_idesc_bf16(CH, 64, 0, 1);
+#pragma unroll
+    for (int z64 = 0; z64 < DK / 64; ++z64) {
+#pragma unroll
+      for (int kk = 0; kk < CH / 16; ++kk) {
+        const uint64_t a = make_smem_desc_sw128(w_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+        const uint64_t b = make_smem_desc_sw128(k_s + z64 * CH_CHUNK + kk * 2048, CH_CHUNK, 1024);
+        umma_bf16(tmem + z64 * 64, a, b, idesc, kk ? 1u : 0u);
+      }
+#pragma unroll
+      for (int part = 0; part < 2; ++part)
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk) {
+          const uint64_t a = make_smem_desc_sw128(r_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+          const uint64_t b = make_smem_desc_sw128(a_s + part * PART + z64 * DK * CH_ROWB + kk * 2048, CH_CHUNK, 1024);
+          umma_bf16(tmem + z64 * 64, a, b, idesc, 1u);
+        }
+    }
+    umma_commit(smem_u32(&done));
+  }
+  __syncwarp();
+  const int qd = warp & 3, half = warp >> 2, t = qd * 32 + lane;   // this thread's token; half the channels
+  constexpr int HC = DK / 2;
+  uint4 gate[HC / 8];
+#pragma unroll
+  for (int i = 0; i < HC / 8; ++i) {
+    gate[i] = make_uint4(0u, 0u, 0u, 0u);
+    if (t < n) gate[i] = *reinterpret_cast<const uint4*>(rows + (long long)t * p.ld + p.g_col + h * p.VP + half * HC + i * 8);
+  }
+  bool ok = mbar_wait_bounded(smem_u32(&done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
+  ok = __all_sync(0xffffffffu, ok);
+  tc_fence_after();
+  uint32_t v[HC];
+  float ss = 0.f;
+  if (ok) {
+#pragma unroll
+    for (int i = 0; i < HC / 32; ++i) tmem_ld_32x32(tmem + half * HC + i * 32 + ((uint32_t)(qd * 32) << 16), *reinterpret_cast<uint32_t(*)[32]>(&v[i * 32]));
+    tmem_ld_wait();
+    tc_fence_before();
+#pragma unroll
+    for (int i = 0; i < HC; ++i) ss = fmaf(__uint_as_float(v[i]), __uint_as_float(v[i]), ss);
+    row_sum[half][t] = ss;
+  }
+  __syncthreads();
+  if (ok && t < n) {
+    const float rs = 1.f / sqrtf((row_sum[0][t] + row_sum[1][t]) / (float)p.dk + p.eps);
+    const float* w = p.norm + h * p.VP + half * HC;
+    __nv_bfloat16* dst = p.out + (long long)(row0 + t) * p.ldo + h * p.VP + half * HC;
+#pragma unroll
+    for (int i = 0; i < HC / 8; ++i) {
+      const float4 w0 = *reinterpret_cast<const float4*>(w + i * 8), w1 = *reinterpret_cast<const float4*>(w + i * 8 + 4);
+      auto two = [&](int e, float wx, float wy, uint32_t gz) {
+        const float2 z = unpack_bf16x2(gz);
+        return pack_bf16x2(__uint_as_float(v[i * 8 + e]) * rs * wx * z.x * sigmoid_f(z.x), __uint_as_float(v[i * 8 + e + 1]) * rs * wy * z.y * sigmoid_f(z.y));
+      };
+      *reinterpret_cast<uint4*>(dst + i * 8) = make_uint4(two(0, w0.x, w0.y, gate[i].x), two(2, w0.z, w0.w, gate[i].y), two(4, w1.x, w1.y, gate[i].z),
+                                                          two(6, w1.z, w1.w, gate[i].w));
+    }
+  }
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, Cfg::kCols);
+  }
+}
+
+template <int DK>
+static int launch_time_mix(const MixParams& p, int n_chunks, int n_seq, cudaStream_t stream) {
+  static bool attr[64] = {};
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
+  if (!attr[dev]) {
+    if (cudaFuncSetAttribute(time_mix_state_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixStateCfg<DK>::kSmem) != cudaSuccess ||
+        cudaFuncSetAttribute(time_mix_out_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixOutCfg<DK>::kSmem) != cudaSuccess)
+      return -10;
+    attr[dev] = true;
+  }
+  const dim3 units(n_chunks * p.H);
+  if (launch_kernel(time_mix_state_kernel<DK>, units, dim3(CHT), MixStateCfg<DK>::kSmem, stream, p) != cudaSuccess) return -11;
+  if (launch_kernel(time_mix_chain_kernel, dim3(DK / 32, p.H * (p.VP / SC_COLS), n_seq), dim3(256), 0, stream, p) != cudaSuccess) return -12;
+  return launch_kernel(time_mix_out_kernel<DK>, units, dim3(CHT), MixOutCfg<DK>::kSmem, stream, p) == cudaSuccess ? 0 : -13;
+}
+
+// ------------------------------------------------------------------------------------------
 // out = o / rms * weight * sigmoid(gate), or silu(gate). One CTA per token; a warp takes whole heads. Padding channels of o are zero.
 template <typename T>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ weight,
@@ -1288,6 +1756,37 @@ int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, in
     case 256: return launch_chunks<256>(p, n_chunks, n_seq, stream);
     default: return -1;
   }
+}
+
+// Workspace of the chunked time mixing in bytes.
+long long rb_time_mix_workspace(int n_chunks, int H, int KP) {
+  const long long ch = (long long)n_chunks * H;
+  return ch * ((long long)KP * KP * 8 + KP * 4) + 256;
+}
+
+// Chunked time mixing of whole portions, as rb_recurrent_chunks, down to the normed and gated output rows (bf16). z [T, ldz] is
+// overwritten. KP is 64 or 128; values have as many channels as keys.
+int rb_time_mix_chunks(const void* proj, long long ld, int k_col, int v_col, int g_col, float* z, long long ldz, const float* w0, const float* bonus,
+                       float* s, const void* chunks, const int* seq_chunks, const int* slots, const int* cu_q, const int* seq_lens, const float* norm,
+                       float eps, void* out, long long ldo, void* workspace, int n_chunks, int n_seq, int H, int dk, int KP, int num_slots, int* status,
+                       cudaStream_t stream) {
+  if (n_chunks <= 0 || n_seq <= 0) return 0;
+  if (H <= 0 || H * (KP / SC_COLS) > 65535 || n_seq > 65535 || dk <= 0 || dk > KP || ld % 8 != 0 || ldo % 8 != 0 || ldz % 4 != 0 || workspace == nullptr ||
+      (k_col | v_col | g_col) % 8 != 0)
+    return -1;
+  const long long ch = (long long)n_chunks * H;
+  MixParams p{};
+  p.proj = (const __nv_bfloat16*)proj; p.ld = ld; p.k_col = k_col; p.v_col = v_col; p.g_col = g_col;
+  p.z = z; p.ldz = ldz; p.w0 = w0; p.bonus = bonus; p.chunks = (const int4*)chunks; p.seq_chunks = seq_chunks; p.slots = slots;
+  p.seq_lens = seq_lens; p.cu_q = cu_q; p.s = s; p.norm = norm; p.eps = eps; p.out = (__nv_bfloat16*)out; p.ldo = ldo;
+  p.H = H; p.dk = dk; p.KP = KP; p.VP = KP; p.num_slots = num_slots; p.status = status;
+  float* w = (float*)workspace;
+  p.u = w; w += ch * KP * KP;
+  p.s_hi = (__nv_bfloat16*)w; w += ch * KP * KP / 2;
+  p.s_lo = (__nv_bfloat16*)w; w += ch * KP * KP / 2;
+  p.last = w;
+  if (KP == 64) return launch_time_mix<64>(p, n_chunks, n_seq, stream);
+  return KP == 128 ? launch_time_mix<128>(p, n_chunks, n_seq, stream) : -1;
 }
 
 int rb_gated_norm(const float* o, long long ldo, const float* weight, const void* gate, long long ldg, void* out, long long ldy, int H, int dv,

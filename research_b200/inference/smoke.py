@@ -13,6 +13,7 @@ def engine_smoke(device: torch.device) -> None:
     _run(device, get_preset("tiny-qwen2", num_layers=2))
     _run(device, get_preset("tiny-lulezen"))      # latent attention: prefill and decode kernels, 32-bit residual stream
     _run(device, get_preset("tiny-zamusun"))      # recurrent state, keys-as-values attention, routed experts, looped layers
+    _run(device, get_preset("tiny-fogurax"))      # convolutions, chunks, attention beside time mixing, shared expert, token input
 
 
 def _run(device: torch.device, cfg) -> None:

@@ -11,7 +11,7 @@ import torch
 
 from ... import ops
 from ...models.stack import LightningSpec, MatrixMemorySpec, TimeMixSpec
-from ...ops.recurrent import MAX_DIM, ChunkTable, RecurrentGeometry, RecurrentState, TimeMix, chunk_workspace, chunked_supported
+from ...ops.recurrent import MAX_DIM, ChunkTable, RecurrentGeometry, RecurrentState, TimeMix, chunk_workspace, chunked_supported, time_mix_chunked_supported, time_mix_workspace
 from .base import Part, load_head_columns, load_head_vector, load_heads, up
 
 SCAN_PORTION = 16            # new tokens of a sequence up to which the recurrence runs token by token
@@ -199,29 +199,45 @@ class TimeMixPart(Part):
 
     def mix(self, w: TimeMixWeights, cache: TimeMixState, inp, out, b, plan) -> None:
         """Normed and gated heads' outputs into ``out [T, H * vp]``."""
-        T, g = b.num_tokens, w.geo
-        n = g.heads * g.kp
+        T = b.num_tokens
         ops.token_shift(inp, w.mu, self.mixed, cache.history, b.cu_q, b.positions, b.state_slots)
+        self.recur(w, cache, self.project_mixes(w, T), self.decay_logits(w, T), out, b, plan)
+
+    def project_mixes(self, w: TimeMixWeights, T: int) -> torch.Tensor:
+        """``r | k | v | gate`` of the mixes."""
+        n = w.geo.heads * w.geo.kp
         proj = self.proj[:self.r.rows * 4 * n].view(-1, 4 * n)
         if T < WIDE_BATCH:
             ops.head_gemm_expand(self.mixed[:4], w.wproj, proj, T)       # (the whole buffer: its destination table is kept)
-        proj = proj[:T]
-        if T >= WIDE_BATCH:
-            for i in range(4):
-                ops.gemm(self.mixed[i, :T], w.wproj[i * n:(i + 1) * n], out=proj[:, i * n:(i + 1) * n])
+            return proj[:T]
+        for i in range(4):
+            ops.gemm(self.mixed[i, :T], w.wproj[i * n:(i + 1) * n], out=proj[:T, i * n:(i + 1) * n])
+        return proj[:T]
+
+    def decay_logits(self, w: TimeMixWeights, T: int) -> torch.Tensor:
+        """``W_w2 tanh(W_w1 mix)`` in fp32."""
+        n = w.geo.heads * w.geo.kp
         inner, tanh = self.inner[:T * w.rank].view(T, -1), self.tanh[:T * w.rank * self.parts].view(T, -1)
-        z, o = self.z[:T * n].view(T, n), self.o[:T * n].view(T, n)
         ops.gemm(self.mixed[4, :T], w.w1, out=inner, out_f32=True)
         ops.tanh_parts(inner, tanh)
-        ops.gemm(tanh, w.w2, out=z, out_f32=True)
+        return ops.gemm(tanh, w.w2, out=self.z[:T * n].view(T, n), out_f32=True)
+
+    def recur(self, w: TimeMixWeights, cache: TimeMixState, proj, z, out, b, plan) -> None:
+        T, g, eps = b.num_tokens, w.geo, self.r.cfg.norm_eps
+        o = self.o[:T * g.heads * g.vp].view(T, -1)
         mix = TimeMix(z, w.w0, w.bonus)
+        n_seq, rows, table = plan if time_mix_chunked_supported(g) else (b.rows, T, None)
+        single = b.rows if b.cu_q is None else b.n_single
         args = (proj, None, g, None, None, None, 1.0, cache.state, b.state_slots)
-        if b.cu_q is None or b.n_single > 0:
-            single = b.rows if b.cu_q is None else b.n_single
+        if single > 0:
             ops.recurrent_scan(*args, None, b.seq_lens, o, single, single, mix=mix)
-        if b.cu_q is not None and b.rows > b.n_single:
-            ops.recurrent_scan(*args, b.cu_q, b.seq_lens, o, T, b.rows, b.n_single, mix=mix)
-        ops.gated_norm(o, w.norm, proj[:, g.offsets[3]:], g, self.r.cfg.norm_eps, out, True, silu=True)
+        if n_seq > single:
+            ops.recurrent_scan(*args, b.cu_q, b.seq_lens, o, rows, n_seq, single, mix=mix)
+        if rows > 0:
+            ops.gated_norm(o[:rows], w.norm, proj[:, g.offsets[3]:], g, eps, out, True, silu=True)
+        if table is not None:
+            room = torch.empty(time_mix_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=o.device)
+            ops.time_mix_chunks(proj, g, mix, cache.state, b.state_slots, b.cu_q, b.seq_lens, w.norm, eps, out, table, room)
 
     def forward(self, w: TimeMixWeights, cache: TimeMixState, inp, y, b, plan, small=None) -> None:
         T, n = b.num_tokens, w.geo.heads * w.geo.vp

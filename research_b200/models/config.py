@@ -13,8 +13,9 @@ import json
 from dataclasses import asdict, dataclass, field, replace
 from pathlib import Path
 
-from .stack import (ClampedGluSpec, ExpertsSpec, KeyValueAttentionSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec, LoopSpec,
-                    MatrixMemorySpec, QueryTemperature, RotarySpec, uniform_stack)
+from .stack import (DESIGNS, BandScaling, ClampedGluSpec, ExpertsRouting, ExpertsSpec, GluSpec, GroupedAttentionSpec, KeyValueAttentionSpec,
+                    LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec, LoopSpec, MatrixMemorySpec, ParallelSpec, QueryTemperature,
+                    RotarySpec, TimeMixSpec, TokenSideSpec, YarnScaling, uniform_stack)
 
 
 @dataclass(frozen=True)
@@ -156,6 +157,25 @@ def _keyvalue(heads: int, kv_heads: int, dim: int, every: int) -> KeyValueAttent
     return KeyValueAttentionSpec(heads, kv_heads, dim, dim ** -0.5, QueryTemperature(0.1, every))
 
 
+def _conv_attention(heads: int, kv_heads: int, dim: int, vdim: int, rot: int, taps: int, original: int) -> GroupedAttentionSpec:
+    return GroupedAttentionSpec(DESIGNS["Fogurax"].mixers["attention"], heads, kv_heads, dim, vdim, dim ** -0.5,
+                                RotarySpec(rot, 5e5, True, BandScaling(8.0, 1.0, 4.0, original)), taps)
+
+
+def _chunk_attention(heads: int, kv_heads: int, dim: int, vdim: int, rot: int, size: int, original: int) -> GroupedAttentionSpec:
+    return GroupedAttentionSpec(DESIGNS["Fogurax"].mixers["attention_2"], heads, kv_heads, dim, vdim, dim ** -0.5,
+                                RotarySpec(rot, 5e5, False, YarnScaling(4.0, original, 32.0, 1.0)), 1, size)
+
+
+def _attention_beside_time_mix(heads: int, kv_heads: int, dim: int, rot: int, size: int, mix_heads: int, mix_dim: int, rank: int) -> ParallelSpec:
+    left = GroupedAttentionSpec(DESIGNS["Fogurax"].mixers["parallel"].left, heads, kv_heads, dim, dim, dim ** -0.5, RotarySpec(rot, 5e5, True), 1, size)
+    return ParallelSpec("parallel", left, TimeMixSpec(mix_heads, mix_dim, rank), 1.0, 1.0)
+
+
+def _shared_experts(experts: int, top: int, ff: int, shared: int) -> ExpertsSpec:
+    return ExpertsSpec(experts, top, GluSpec(ff), ExpertsRouting("sigmoid", False, True), GluSpec(shared))
+
+
 PRESETS: dict[str, ModelConfig | LayerStackConfig] = {
     # tiny CPU plumbing model: Qwen2-style, vocab 4096, 4 layers, d 256, 4q/2kv heads
     "tiny-qwen2": ModelConfig(),
@@ -195,6 +215,15 @@ PRESETS: dict[str, ModelConfig | LayerStackConfig] = {
     "zamusun-4b": LayerStackConfig("Zamusun", 128256, 2048, tuple(
         LayerSpec((_memory(16, 128, 128), _lightning(16, 128, 128), _keyvalue(16, 4, 128, 1024))[i % 3], ExpertsSpec(64, 8, ClampedGluSpec(768, 7.0)))
         for i in range(12)), loop=LoopSpec(0, 3, 2)),
+    # layer stacks with short convolutions, chunked attention, attention beside time mixing, a shared expert, a per-layer token input
+    "tiny-fogurax": LayerStackConfig("Fogurax", 4096, 160, (
+        LayerSpec(_chunk_attention(5, 1, 32, 24, 16, 40, 64), GluSpec(288)),
+        LayerSpec(_conv_attention(4, 2, 24, 40, 24, 4, 64), _shared_experts(6, 2, 64, 80)),
+        LayerSpec(_attention_beside_time_mix(3, 3, 40, 24, 50, 4, 32, 24), None)), residual_mult=0.8, token_side=TokenSideSpec(16), init_std=0.05),
+    "fogurax-4b": LayerStackConfig("Fogurax", 128256, 2048, tuple(
+        LayerSpec((_chunk_attention(16, 4, 128, 128, 64, 4096, 4096), _conv_attention(16, 4, 128, 128, 64, 4, 8192),
+                   _attention_beside_time_mix(16, 4, 128, 64, 2048, 32, 64, 64))[i % 3],
+                  GluSpec(8192) if i % 3 == 0 else _shared_experts(64, 8, 768, 1536)) for i in range(15)), residual_mult=0.5, token_side=TokenSideSpec(256)),
 }
 
 

@@ -111,8 +111,11 @@ def _lib() -> ctypes.CDLL:
         lib.rb_recurrent_chunks.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float, c_float] + [c_vp] * 9 + [c_ll, c_vp]
                                             + [c_int] * 8 + [c_vp, c_vp])
         lib.rb_recurrent_chunk_workspace.argtypes, lib.rb_recurrent_chunk_workspace.restype = [c_int] * 4, c_ll
+        lib.rb_time_mix_chunks.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 9 + [c_float, c_vp, c_ll, c_vp] + [c_int] * 6
+                                           + [c_vp, c_vp])
+        lib.rb_time_mix_workspace.argtypes, lib.rb_time_mix_workspace.restype = [c_int] * 3, c_ll
         lib.rb_gated_norm.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_ll] + [c_int] * 7 + [c_float, c_vp]
-        for f in ("rb_recurrent_scan", "rb_recurrent_chunks", "rb_gated_norm", "rb_token_shift", "rb_tanh_parts"):
+        for f in ("rb_recurrent_scan", "rb_recurrent_chunks", "rb_gated_norm", "rb_token_shift", "rb_tanh_parts", "rb_time_mix_chunks"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -234,6 +237,29 @@ def recurrent_chunks(proj, small, geo: RecurrentGeometry, decay, bias_i, bias_f,
 
 def chunk_workspace(n_chunks: int, geo: RecurrentGeometry) -> int:
     return int(_lib().rb_recurrent_chunk_workspace(n_chunks, geo.heads, geo.kp, geo.vp))
+
+
+def time_mix_chunked_supported(geo: RecurrentGeometry) -> bool:
+    return geo.kp in (64, 128) and geo.kp == geo.vp
+
+
+def time_mix_chunks(proj, geo: RecurrentGeometry, mix: TimeMix, state: RecurrentState, slots, cu_q, seq_lens, norm, eps: float, out, table: ChunkTable,
+                    workspace) -> None:
+    """Time mixing over the sequences of ``table`` in chunks of 128 tokens, norm per head and SiLU gate included (bf16 activations on the
+    GPU): rows ``cu_q[first] ..`` of ``out [T, H*vp]``, state updated. Their rows of ``mix.z`` are overwritten."""
+    _, ok, ov, og = geo.offsets
+    n, B, f = table.chunks.shape[0], table.seq_chunks.shape[0] - 1, table.first
+    assert proj.is_cuda and proj.dtype == out.dtype == torch.bfloat16 and proj.stride(1) == out.stride(1) == 1
+    assert workspace.numel() * workspace.element_size() >= time_mix_workspace(n, geo)
+    rc = _lib().rb_time_mix_chunks(ptr(proj), proj.stride(0), ok, ov, og, ptr(mix.z), mix.z.stride(0), ptr(mix.w0), ptr(mix.bonus), ptr(state.s),
+                                   ptr(table.chunks), ptr(table.seq_chunks), ptr(slots[f:]), ptr(cu_q[f:]), ptr(seq_lens[f:]), ptr(norm), eps, ptr(out),
+                                   out.stride(0), ptr(workspace), n, B, geo.heads, geo.dim, geo.kp, state.s.shape[0],
+                                   ptr(status_tensor(proj.device)), stream_handle(proj.device))
+    check_rc(rc, "rb_time_mix_chunks", 3)
+
+
+def time_mix_workspace(n_chunks: int, geo: RecurrentGeometry) -> int:
+    return int(_lib().rb_time_mix_workspace(n_chunks, geo.heads, geo.kp))
 
 
 def token_shift(h, mu, out, history, cu_q, positions, state_slots) -> None:

@@ -2,7 +2,8 @@
 
 ``bench.py --workload stack`` runs it (``--designs``, ``--sizes`` choose). For every size two engines are built with random
 weights: Lulezen (latent attention) beside a Llama-type model, Zamusun (recurrent mixers, keys-as-values attention, routed
-experts, a looped pair of layers) beside a Qwen3-MoE-type model, each with the same width, layer runs, feed-forward,
+experts, a looped pair of layers) and Fogurax (grouped attention with convolutions or chunks, attention beside time mixing, routed and
+shared experts, a per-layer token input) beside a Qwen3-MoE-type model, each with the same width, layer runs, feed-forward,
 vocabulary and heads (grouped queries, head size 128). Measured with CUDA events, after warm-up:
 
 * decode: one captured decode step at the given batch and context, replayed;
@@ -24,8 +25,10 @@ from .. import ops
 from ..inference import EngineConfig, InferenceEngine
 from ..models import LazyRandomWeights
 from ..models.config import ModelConfig
-from ..models.stack import (ClampedGluSpec, ExpertsSpec, KeyValueAttentionSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec,
-                            LoopSpec, MatrixMemorySpec, QueryTemperature, RotarySpec, uniform_stack)
+from ..models.stack import (DESIGNS as STACK_DESIGNS, BandScaling, ClampedGluSpec, ExpertsRouting, ExpertsSpec, GluSpec, GroupedAttentionSpec,
+                            KeyValueAttentionSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec, LoopSpec, MatrixMemorySpec,
+                            ParallelSpec, QueryTemperature, RotarySpec, TimeMixSpec, TokenSideSpec, YarnScaling, uniform_stack)
+from ..inference.stack_parts import DensePart
 from ..ops import experts as ex
 from .timing import flush_l2, time_cuda
 
@@ -93,6 +96,29 @@ def expert_configs(s: ExpertSize):
                       head_dim=128, intermediate_size=s.ff, rope_theta=5e5, tie_word_embeddings=True, attention_bias=False, qk_norm=True,
                       num_experts=s.experts, num_experts_per_tok=s.top, moe_intermediate_size=s.ff)
     return stack, moe
+
+
+def fogurax_stack(s: ExpertSize, layers: int, conv: int = 4, reach: int = 4096, side: int = 256) -> LayerStackConfig:
+    """Every third layer has attention in chunks, convolutions on the projections, or attention beside time mixing; heads of 128
+    channels in attention and 64 in time mixing."""
+    H, G, kinds = s.heads, s.kv_heads, STACK_DESIGNS["Fogurax"].mixers
+
+    def rot(interleaved, scaling=None):
+        return RotarySpec(64, 5e5, interleaved, scaling)
+
+    def heads(form, r, taps=1, size=0):
+        return GroupedAttentionSpec(form, H, G, 128, 128, 128 ** -0.5, r, taps, size)
+
+    chunked = heads(kinds["attention_2"], rot(False, YarnScaling(4.0, 4096, 32.0, 1.0)), size=reach)
+    conved = heads(kinds["attention"], rot(True, BandScaling(8.0, 1.0, 4.0, 8192)), conv)
+    both = ParallelSpec("parallel", heads(kinds["parallel"].left, rot(True), size=reach), TimeMixSpec(2 * H, 64, 64), 1.0, 1.0)
+    mlp = ExpertsSpec(s.experts, s.top, GluSpec(s.ff), ExpertsRouting("sigmoid", False, True), GluSpec(s.ff))
+    return LayerStackConfig("Fogurax", s.vocab, s.width, tuple(LayerSpec((chunked, conved, both)[i % 3], mlp) for i in range(layers)),
+                            residual_mult=0.5, token_side=TokenSideSpec(side))
+
+
+def fogurax_configs(s: ExpertSize):
+    return fogurax_stack(s, s.runs), expert_configs(s)[1]
 
 
 def _engine(cfg, batch: int, context: int, prompt: int) -> InferenceEngine:
@@ -240,14 +266,7 @@ def expert_stack_kernels(eng: InferenceEngine, T: int, context: int, decode: boo
     d, eps = cfg.hidden_size, cfg.norm_eps
     x, h, y = r.x[:T], r.xb[:T], r.y[:T]
     h.normal_()
-    i32 = dict(dtype=torch.int32, device="cuda")
-    if decode:
-        b = r._decode_batch(T)
-    else:
-        pos = torch.arange(T, **i32)
-        b = type(r._decode_batch(2))(rows=1, num_tokens=T, padded=T, max_new=T, tokens=pos, positions=pos, slots=pos, cu_q=torch.tensor([0, T], **i32),
-                                     seq_lens=torch.tensor([T], **i32), block_tables=torch.arange(-(-T // 16), **i32)[None].contiguous(),
-                                     host_cu_q=[0, T], host_seq_lens=[T], state_slots=torch.zeros(1, **i32), n_single=0)
+    b = r._decode_batch(T) if decode else _prompt_batch(r, T)
     seen = set()
     for run in r.runs:
         lw = run.layer
@@ -295,6 +314,92 @@ def expert_stack_kernels(eng: InferenceEngine, T: int, context: int, decode: boo
         lg = r.logits_padded[:T]
         t.gemm("head", T, r.vp, r.wp, lambda: r._head(r.hl[:T], lg), 4)
     return t.rows
+
+
+def fogurax_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict:
+    """The first layer of every kind of mixer, the experts, the token input and what joins them."""
+    r, cfg, t = eng.runner, eng.runner.cfg, _Table()
+    d, eps, m = cfg.hidden_size, cfg.norm_eps, cfg.residual_mult
+    x, h, y = r.x[:T], r.xb[:T], r.y[:T]
+    h.normal_()
+    b = r._decode_batch(T) if decode else _prompt_batch(r, T)
+    seen = set()
+    for run in r.runs:
+        lw = run.layer
+        kind = lw.spec.mixer.type
+        if kind in seen:
+            continue
+        seen.add(kind)
+        both = kind == "parallel"
+        w, part, cache = (lw.mix.left, lw.mixer.left, run.cache[0]) if both else (lw.mix, lw.mixer, run.cache)
+        g, plan = w.geo, part.planned(b)
+        H, G, D, n = g.heads, g.kv_heads, g.dp, g.heads * g.dp
+        proj, q = part._projected(w, T), part.q[:T * n].view(T, n)
+        out = lw.mixer.out[:T * lw.mix.wo.shape[1]].view(T, -1)
+        t.gemm(f"{kind}: joint projection", T, w.wproj.shape[0], r.wp, lambda: r._project(lw, h))
+        small = r._project(lw, h)
+        t.add(f"{kind}: norm + rotation + append", lambda: ops.grouped_append(
+            proj, g, conv=w.conv, cache=cache, cu_q=b.cu_q, positions=b.positions, state_slots=b.state_slots, slots=b.slots, q_norm=w.q_norm,
+            k_norm=w.k_norm, eps=eps, table=w.table, q=q), 2 * T * (g.channels * 2 + (g.history if decode else 0) * 2), 0)
+        fn = lambda: ops.grouped_attention(q, g, cache, b.block_tables, b.cu_q, b.seq_lens, out[:, :n], scale=w.spec.scale, rows=T, max_q=b.max_new,
+                                           n_single=b.n_single, gate=small if w.spec.form.gate else None, workspace=part.workspace, splits=plan.get(g, 1))
+        reach = g.reach or max(context, T)
+        if decode:
+            span = (context - 1) % g.chunk + 1 if g.chunk else min(context, reach)
+            t.add(f"{kind}: attention", fn, 2 * T * (2 * span * G * D + 2 * H * D), 4.0 * T * H * span * D)
+        else:
+            pairs = sum(i % g.chunk + 1 if g.chunk else min(i + 1, reach) for i in range(T))
+            t.add(f"{kind}: attention", fn, 2 * T * D * (2 * H + 2 * G), 4.0 * pairs * H * D)
+        if both:
+            _time_mix_rows(t, r, lw.mixer.right, lw.mix.right, run.cache[1], h, out[:, n:], b, T, decode)
+        t.gemm(f"{kind}: output projection", T, r.wp, out.shape[1], lambda: ops.gemm(out, lw.mix.wo, out=y, out_f32=True), 4)
+    lw = r.layers[0]
+    logits = r._project(lw, h)[:, lw.mix_small:]
+    w, g = lw.ff, lw.ff.geo
+    sc = lw.feed_forward.scratch[g]
+    _routed(t, T, g.experts, g.top, d, g.ff, lambda: ex.experts_up(g, sc, w.wgu, T), lambda: ex.experts_down(g, sc, w.wd), None,
+            {"experts route + plan": (lambda: ex.experts_plan(logits, g, sc), T * (4 * g.experts + 8 * g.top)),
+             "experts gather": (lambda: (ex.experts_plan(logits, g, sc), ex.experts_gather(h, g, sc)), 2 * 2 * T * g.top * d)})
+    shared = w.shared
+    act = r._part(DensePart).act[:T * shared.ffp].view(T, shared.ffp)
+    t.gemm("shared gate|up + unit", T, 2 * shared.ffp, r.wp, lambda: ops.gemm(h, shared.wgu, out=act, bn=256, swiglu=True), 2, shared.ffp)
+    t.gemm("shared down", T, r.wp, shared.ffp, lambda: ops.gemm(act, shared.wd, out=r.y2[:T], out_f32=True), 4)
+    t.add("residual + experts' sum", lambda: ops.stream_norm(x, d, y1=y, y2=r.y2[:T], experts=sc.y[:T * g.top], top=g.top, mult=m, copy=h),
+          T * d * (4 * 4 + 2 + 2 * g.top), 0)
+    z, a = r.side_z[:T], r.side_a[:T]
+    t.gemm("token input: gate", T, r.sp, r.wp, lambda: ops.gemm(h, lw.side.gate, out=z, out_f32=True), 4)
+    t.add("token input: unit", lambda: ops.token_side(z, b.tokens[:T], r.side_embed, 0, a, r.side_dim), T * r.side_dim * 8, 0)
+    t.gemm("token input: projection", T, r.wp, r.sp, lambda: ops.gemm(a, lw.side.proj, out=y, out_f32=True), 4)
+    t.add("token input's norm + residual + norm", lambda: ops.stream_norm(x, d, side=y, side_weight=lw.side.norm, mult=m, weight=lw.norm1[0], eps=eps, h=h),
+          T * d * (4 * 3 + 2), 0)
+    if decode:
+        lg = r.logits_padded[:T]
+        t.gemm("head", T, r.vp, r.wp, lambda: r._head(r.hl[:T], lg), 4)
+    return t.rows
+
+
+def _time_mix_rows(t: _Table, r, part, w, cache, h, out, b, T: int, decode: bool) -> None:
+    g, eps = w.geo, r.cfg.norm_eps
+    n = g.heads * g.kp
+    mixed, plan = part.mixed, part.planned(b)
+    t.add("time mixing: shift", lambda: ops.token_shift(h, w.mu, mixed, cache.history, b.cu_q, b.positions, b.state_slots), 2 * T * r.wp * 6, 0)
+    proj = part.project_mixes(w, T)
+    t.gemm("time mixing: r, k, v, gate", T, 4 * n, r.wp, lambda: part.project_mixes(w, T))
+    t.add("time mixing: decay's products", lambda: part.decay_logits(w, T), 2 * T * r.wp + 2 * w.rank * (r.wp + 2 * n) + 4 * T * n,
+          2.0 * T * w.rank * (r.wp + 2 * n))
+    z = part.decay_logits(w, T)
+    state = 2 * 4 * n * g.vp
+    t.add("time mixing: recurrence + norm + gate", lambda: part.recur(w, cache, proj, z, out, b, plan), T * n * (2 * 5 + 4) + state * b.rows,
+          T * g.heads * (4.0 * g.kp * g.vp + (0 if decode else 2.0 * 64 * (g.kp + g.vp))))
+
+
+def _prompt_batch(r, T: int):
+    """One whole prompt of T tokens."""
+    i32 = dict(dtype=torch.int32, device="cuda")
+    pos = torch.arange(T, **i32)
+    return type(r._decode_batch(2))(rows=1, num_tokens=T, padded=T, max_new=T, tokens=pos, positions=pos, slots=pos, cu_q=torch.tensor([0, T], **i32),
+                                    seq_lens=torch.tensor([T], **i32), block_tables=torch.arange(-(-T // 16), **i32)[None].contiguous(),
+                                    host_cu_q=[0, T], host_seq_lens=[T], state_slots=torch.zeros(1, **i32), n_single=0)
 
 
 def hf_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict:
@@ -346,7 +451,8 @@ def hf_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict
 
 # design -> (sizes, pair of configurations, labels and kernel tables)
 DESIGNS = {"lulezen": (SIZES, configs, (("lulezen", latent_kernels), ("llama", hf_kernels))),
-           "zamusun": (EXPERT_SIZES, expert_configs, (("zamusun", expert_stack_kernels), ("qwen3_moe", hf_kernels)))}
+           "zamusun": (EXPERT_SIZES, expert_configs, (("zamusun", expert_stack_kernels), ("qwen3_moe", hf_kernels))),
+           "fogurax": (EXPERT_SIZES, fogurax_configs, (("fogurax", fogurax_kernels), ("qwen3_moe", hf_kernels)))}
 
 
 def run(sizes: tuple[str, ...] = (), batches: tuple[int, ...] = (1, 64, 256), context: int = 2048, prompts: tuple[int, ...] = (512, 4096),
