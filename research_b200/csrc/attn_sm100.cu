@@ -1153,7 +1153,7 @@ __global__ void kv_gate_kernel(__nv_bfloat16* __restrict__ out, const float* __r
 }
 
 // ------------------------------------------------------------------------------------------
-// Grouped attention with cached keys and values: everything between the joint projection and the attention, one CTA per token.
+// Grouped attention with cached keys and values: everything between the joint projection and the attention.
 // Every projected channel goes through its causal convolution (if there is one), queries and keys through the norm and the rotation;
 // queries land in a buffer with heads padded to DP channels, keys and values in the cache. Look back: history.cuh, over the raw
 // projected values.
@@ -1183,6 +1183,16 @@ struct GroupedAppend {
   int* status;
 };
 
+__device__ __forceinline__ void store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(a, b); }
+__device__ __forceinline__ void store8(float* p, const float (&x)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(x[0], x[1], x[2], x[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(x[4], x[5], x[6], x[7]);
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&x)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(x[0], x[1]), pack_bf16x2(x[2], x[3]), pack_bf16x2(x[4], x[5]), pack_bf16x2(x[6], x[7]));
+}
+
 template <typename T>
 __device__ __forceinline__ void load8(const T* p, float (&x)[8]) {
   constexpr int V = 16 / sizeof(T);
@@ -1195,131 +1205,194 @@ __device__ __forceinline__ void load8(const T* p, float (&x)[8]) {
   }
 }
 
-template <typename T>
+// TOK rows per CTA (the convolution's weights are loaded once for them); STEPS: 64 channels of a padded head each.
+template <typename T, int TOK, int STEPS>
 __global__ void __launch_bounds__(GA_THREADS) grouped_append_kernel(const GroupedAppend p) {
-  extern __shared__ float ga_row[];                       // q and k channels, laid out as in the projection
-  __shared__ float red[2][GA_THREADS / 32];
+  extern __shared__ float ga_rows[];                      // [TOK][v_col] q and k channels, laid out as in the projection
+  __shared__ float red[TOK][2][GA_THREADS / 32];
+  __shared__ RowPlace places[TOK];
+  __shared__ int dests[TOK];
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t0 = blockIdx.x * TOK, n_tok = min(TOK, p.T - t0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* rows = reinterpret_cast<const T*>(p.proj);
   T* hist = reinterpret_cast<T*>(p.hist);
-  RowPlace place{0, p.rows.positions[t], -1};
-  if (p.taps > 1) place = row_place(p.rows, t, p.status);
-  int slot = p.slots[t];
-  if (slot >= 0 && slot / KV_BLOCK >= p.num_blocks) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); slot = -1; }
-  const long long krow = slot >= 0 ? ((long long)(slot / KV_BLOCK) * p.G * KV_BLOCK + slot % KV_BLOCK) * p.DP : 0;
-  T* vcache = reinterpret_cast<T*>(p.values) + krow;      // + head * 16 * DP
-  float ssq = 0.f, ssk = 0.f;
+  if (threadIdx.x < n_tok) {
+    const int t = t0 + threadIdx.x;
+    RowPlace place{0, p.rows.positions[t], -1};
+    if (p.taps > 1) place = row_place(p.rows, t, p.status);
+    int slot = p.slots[t];
+    if (slot >= 0 && slot / KV_BLOCK >= p.num_blocks) { set_status(p.status, ST_BAD_INDEX); slot = -1; }
+    if (place.position < 0 || place.position >= p.max_pos) { set_status(p.status, ST_BAD_INDEX); place.position = 0; }
+    places[threadIdx.x] = place;
+    dests[threadIdx.x] = slot;
+  }
+  __syncthreads();
+  auto cache_row = [&](int slot) { return ((long long)(slot / KV_BLOCK) * p.G * KV_BLOCK + slot % KV_BLOCK) * p.DP; };   // + head * 16 * DP
+  float ssq[TOK], ssk[TOK];
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) ssq[i] = ssk[i] = 0.f;
   const int nq = p.H * p.dim, nk = p.G * p.dim, nv = p.G * p.vdim;
   for (int c = threadIdx.x * 8; c < p.channels; c += GA_THREADS * 8) {
-    float x[8];
-    load8(rows + (long long)t * p.ld + c, x);
+    float x[TOK][8], u[8];
+#pragma unroll
+    for (int i = 0; i < TOK; ++i)
+      if (i < n_tok) load8(rows + (long long)(t0 + i) * p.ld + c, x[i]);
     if (p.conv != nullptr) {
-      float u[8];
+      if (TOK == 1)
 #pragma unroll
-      for (int i = 0; i < 8; ++i) { u[i] = x[i]; x[i] *= p.conv[(long long)(p.taps - 1) * p.channels + c + i]; }
-      for (int d = 1; d < p.taps; ++d) {
-        const T* back = row_before(place, d, rows, p.ld, t, (const T*)hist, p.taps - 1, p.channels);
-        if (back == nullptr) break;                       // (nothing further back either)
-        float y[8];
-        load8(back + c, y);
-        const float* w = p.conv + (long long)(p.taps - 1 - d) * p.channels + c;
+        for (int j = 0; j < 8; ++j) u[j] = x[0][j];
+      for (int d = 0; d < p.taps; ++d) {
+        float w[8];
+        load8(p.conv + (long long)(p.taps - 1 - d) * p.channels + c, w);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) x[i] = fmaf(w[i], y[i], x[i]);
+        for (int i = 0; i < TOK; ++i) {
+          if (i >= n_tok) continue;
+          if (d == 0) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[i][j] *= w[j];
+          } else {
+            const T* back = row_before(places[i], d, rows, p.ld, t0 + i, (const T*)hist, p.taps - 1, p.channels);
+            if (back != nullptr) {
+              float y[8];
+              load8(back + c, y);
+#pragma unroll
+              for (int j = 0; j < 8; ++j) x[i][j] = fmaf(w[j], y[j], x[i][j]);
+            }
+          }
+        }
       }
-      if (p.taps > 1 && p.rows.cu_q == nullptr && place.slot >= 0) {    // one row per sequence: this thread moves its own channels on
-        T* mine = hist + (long long)place.slot * (p.taps - 1) * p.channels + c;
+      if (TOK == 1 && p.taps > 1 && p.rows.cu_q == nullptr && places[0].slot >= 0) {    // one row per sequence: this thread moves its own channels on
+        T* mine = hist + (long long)places[0].slot * (p.taps - 1) * p.channels + c;
         for (int d = p.taps - 2; d >= 1; --d)
 #pragma unroll
           for (int i = 0; i < (int)(8 * sizeof(T) / 16); ++i)
             reinterpret_cast<uint4*>(mine + (long long)d * p.channels)[i] = reinterpret_cast<const uint4*>(mine + (long long)(d - 1) * p.channels)[i];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) kv_store(mine + i, u[i]);
+        store8(mine, u);
       }
     }
     if (c >= p.v_col) {
       const int v0 = c - p.v_col;
-      if (slot >= 0) {
-        if (p.vdim % 8 == 0) {
-          if (v0 < nv) {
-            T* dst = vcache + (long long)(v0 / p.vdim) * KV_BLOCK * p.DP + v0 % p.vdim;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) kv_store(dst + i, x[i]);
-          }
+      for (int i = 0; i < TOK; ++i) {
+        if (i >= n_tok || dests[i] < 0) continue;
+        T* vcache = reinterpret_cast<T*>(p.values) + cache_row(dests[i]);
+        if (p.vdim % 8 == 0) {
+          if (v0 < nv) store8(vcache + (long long)(v0 / p.vdim) * KV_BLOCK * p.DP + v0 % p.vdim, x[i]);
         } else {
 #pragma unroll
-          for (int i = 0; i < 8; ++i)
-            if (v0 + i < nv) kv_store(vcache + (long long)((v0 + i) / p.vdim) * KV_BLOCK * p.DP + (v0 + i) % p.vdim, x[i]);
+          for (int j = 0; j < 8; ++j)
+            if (v0 + j < nv) kv_store(vcache + (long long)((v0 + j) / p.vdim) * KV_BLOCK * p.DP + (v0 + j) % p.vdim, x[i][j]);
         }
       }
     } else {
       const bool is_k = c >= p.k_col;
       const int n = is_k ? nk : nq, c0 = c - (is_k ? p.k_col : 0);
+#pragma unroll
+      for (int i = 0; i < TOK; ++i) {
+        if (i >= n_tok) continue;
+        float4* dst = reinterpret_cast<float4*>(ga_rows + i * p.v_col + c);
+        dst[0] = make_float4(x[i][0], x[i][1], x[i][2], x[i][3]);
+        dst[1] = make_float4(x[i][4], x[i][5], x[i][6], x[i][7]);
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (c0 + j < n) s = fmaf(x[i][j], x[i][j], s);
+        if (is_k) ssk[i] += s; else ssq[i] += s;
+      }
+    }
+  }
+  if (p.norm == GA_NORM_PROJECTION)
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+      const float q = warp_sum(ssq[i]), k = warp_sum(ssk[i]);
+      if (lane == 0) { red[i][0][warp] = q; red[i][1][warp] = k; }
+    }
+  __syncthreads();
+  if (p.norm == GA_NORM_PROJECTION) {                     // sums -> factors, a thread each
+    if (threadIdx.x < 2 * TOK) {
+      const int i = threadIdx.x >> 1, is_k = threadIdx.x & 1;
       float s = 0.f;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        ga_row[c + i] = x[i];
-        if (c0 + i < n) s = fmaf(x[i], x[i], s);
-      }
-      if (is_k) ssk += s; else ssq += s;
+      for (int w = 0; w < GA_THREADS / 32; ++w) s += red[i][is_k][w];
+      red[i][is_k][0] = 1.f / sqrtf(s / (float)(is_k ? nk : nq) + p.eps);
     }
+    __syncthreads();
   }
-  if (p.norm == GA_NORM_PROJECTION) {
-    ssq = warp_sum(ssq);
-    ssk = warp_sum(ssk);
-    if (lane == 0) { red[0][warp] = ssq; red[1][warp] = ssk; }
-  }
-  __syncthreads();
-  float rq = 1.f, rk = 1.f;
-  if (p.norm == GA_NORM_PROJECTION) {
-    ssq = ssk = 0.f;
-#pragma unroll
-    for (int i = 0; i < GA_THREADS / 32; ++i) { ssq += red[0][i]; ssk += red[1][i]; }
-    rq = 1.f / sqrtf(ssq / (float)nq + p.eps);
-    rk = 1.f / sqrtf(ssk / (float)nk + p.eps);
-  }
-  int pos = place.position;
-  if (pos < 0 || pos >= p.max_pos) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); pos = 0; }
-  const float2* table = reinterpret_cast<const float2*>(p.table) + (long long)pos * p.half;
-  // a warp per head, two channels per lane and step
-  for (int hd = warp; hd < p.H + p.G; hd += GA_THREADS / 32) {
+  // A warp per head: lane e takes a pair of channels that the rotation turns, (2e, 2e + 1) or (e, e + half), or two that pass.
+  const int heads = p.H + p.G;
+  for (int u = warp; u < n_tok * heads; u += GA_THREADS / 32) {
+    const int i = u / heads, hd = u - i * heads;
     const bool is_k = hd >= p.H;
     const int head = is_k ? hd - p.H : hd;
-    if (is_k && slot < 0) continue;
-    const float* src = ga_row + (is_k ? p.k_col : 0) + head * p.dim;
-    const float* w = p.norm == GA_NORM_PROJECTION ? (is_k ? p.k_norm : p.q_norm) + head * p.dim : nullptr;
-    const float r = is_k ? rk : rq;
-    auto at = [&](int d) { return w != nullptr ? src[d] * r * w[d] : src[d]; };
-    auto rotated = [&](int d) {
-      if (d >= 2 * p.half) return d < p.dim ? at(d) : 0.f;
-      const int i = p.interleaved ? d >> 1 : d < p.half ? d : d - p.half;
-      const bool first = p.interleaved ? (d & 1) == 0 : d < p.half;
-      const float2 cs = table[i];
-      const float u = at(p.interleaved ? 2 * i : i), v = at(p.interleaved ? 2 * i + 1 : i + p.half);
-      return first ? u * cs.x - v * cs.y : v * cs.x + u * cs.y;
-    };
-    float y[GA_MAX_DP / 64][2], ss = 0.f;
+    if (is_k && dests[i] < 0) continue;
+    const float* src = ga_rows + i * p.v_col + (is_k ? p.k_col : 0) + head * p.dim;
+    const float* w = (is_k ? p.k_norm : p.q_norm) + head * p.dim;
+    const float r = p.norm == GA_NORM_PROJECTION ? red[i][is_k][0] : 1.f;
+    const float2* table = reinterpret_cast<const float2*>(p.table) + (long long)places[i].position * p.half;
+    float y[STEPS][2], ss = 0.f;
+    int at0[STEPS], at1[STEPS];
 #pragma unroll
-    for (int j = 0; j < GA_MAX_DP / 64; ++j) {
-      const int d = lane * 2 + j * 64;
-      y[j][0] = y[j][1] = 0.f;
-      if (d < p.DP) {
-        y[j][0] = rotated(d);
-        y[j][1] = rotated(d + 1);
-        ss += y[j][0] * y[j][0] + y[j][1] * y[j][1];
+    for (int j = 0; j < STEPS; ++j) {
+      const int e = lane + j * 32;
+      const bool turned = e < p.half, split = turned && !p.interleaved;
+      at0[j] = split ? e : 2 * e;
+      at1[j] = split ? e + p.half : 2 * e + 1;
+      float a = at0[j] < p.dim ? src[at0[j]] : 0.f, b = at1[j] < p.dim ? src[at1[j]] : 0.f;
+      if (p.norm == GA_NORM_PROJECTION) {
+        if (at0[j] < p.dim) a *= r * w[at0[j]];
+        if (at1[j] < p.dim) b *= r * w[at1[j]];
+      }
+      if (turned) {
+        const float2 cs = table[e];
+        const float a0 = a;
+        a = a0 * cs.x - b * cs.y;
+        b = b * cs.x + a0 * cs.y;
+      }
+      y[j][0] = a;
+      y[j][1] = b;
+      ss = fmaf(a, a, fmaf(b, b, ss));
+    }
+    if (p.norm == GA_NORM_HEAD) {
+      const float f = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+#pragma unroll
+      for (int j = 0; j < STEPS; ++j) { y[j][0] *= f; y[j][1] *= f; }
+    }
+    T* dst = is_k ? reinterpret_cast<T*>(p.keys) + cache_row(dests[i]) + (long long)head * KV_BLOCK * p.DP
+                  : reinterpret_cast<T*>(p.q) + ((long long)(t0 + i) * p.H + head) * p.DP;
+#pragma unroll
+    for (int j = 0; j < STEPS; ++j) {
+      if (at1[j] >= p.DP) continue;
+      if (at1[j] == at0[j] + 1 && (at0[j] & 1) == 0) {
+        store2(dst + at0[j], y[j][0], y[j][1]);
+      } else {
+        kv_store(dst + at0[j], y[j][0]);
+        kv_store(dst + at1[j], y[j][1]);
       }
     }
-    float f = 1.f;
-    if (p.norm == GA_NORM_HEAD) f = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
-    T* dst = is_k ? reinterpret_cast<T*>(p.keys) + krow + (long long)head * KV_BLOCK * p.DP
-                  : reinterpret_cast<T*>(p.q) + ((long long)t * p.H + head) * p.DP;
-#pragma unroll
-    for (int j = 0; j < GA_MAX_DP / 64; ++j) {
-      const int d = lane * 2 + j * 64;
-      if (d < p.DP) { kv_store(dst + d, y[j][0] * f); kv_store(dst + d + 1, y[j][1] * f); }
-    }
   }
+}
+
+template <typename T>
+static cudaError_t launch_grouped_append(const GroupedAppend& p, cudaStream_t stream) {
+  const int dev = current_device_index();
+  if (dev < 0) return cudaErrorInvalidDevice;
+  const size_t row = (size_t)p.v_col * 4;
+  const bool several = p.rows.cu_q != nullptr && p.T >= 592 && 4 * row <= 100 * 1024;      // (rows of one sequence lie together)
+#define RB_APPEND(TOK, STEPS)                                                                                                  \
+  do {                                                                                                                         \
+    static bool attr[RB_MAX_DEVICES] = {};                                                                                     \
+    if (!attr[dev]) {                                                                                                          \
+      const cudaError_t e = cudaFuncSetAttribute(grouped_append_kernel<T, TOK, STEPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+      if (e != cudaSuccess) return e;                                                                                          \
+      attr[dev] = true;                                                                                                        \
+    }                                                                                                                          \
+    return launch_kernel(grouped_append_kernel<T, TOK, STEPS>, dim3((p.T + TOK - 1) / TOK), dim3(GA_THREADS), TOK * row, stream, p); \
+  } while (0)
+  if (p.DP == 64) { if (several) RB_APPEND(4, 1); else RB_APPEND(1, 1); }
+  if (p.DP == 128) { if (several) RB_APPEND(4, 2); else RB_APPEND(1, 2); }
+  if (several) RB_APPEND(4, GA_MAX_DP / 64); else RB_APPEND(1, GA_MAX_DP / 64);
+#undef RB_APPEND
 }
 
 template <int D, bool SHARED>
@@ -1345,8 +1418,7 @@ extern "C" int rb_grouped_append(const GroupedAppendArgs* a, cudaStream_t stream
   if (a->DP > GA_MAX_DP || a->DP % 64 != 0 || a->dim > a->DP || a->vdim > a->DP || a->G <= 0 || a->H % a->G != 0 || a->taps < 1) return -1;
   if (a->taps > 1 && (a->conv == nullptr || a->hist == nullptr || a->state_slots == nullptr)) return -1;
   if (a->k_col % 8 != 0 || a->v_col % 8 != 0 || a->channels % 8 != 0 || a->ld % 8 != 0 || 2 * a->half > a->dim) return -1;
-  const size_t smem = (size_t)a->v_col * 4;
-  if (smem > 200 * 1024) return -1;
+  if ((size_t)a->v_col * 4 > 200 * 1024) return -1;
   GroupedAppend p;
   p.proj = a->proj; p.ld = a->ld; p.k_col = a->k_col; p.v_col = a->v_col; p.channels = a->channels;
   p.conv = a->conv; p.taps = a->taps; p.hist = a->hist;
@@ -1355,17 +1427,7 @@ extern "C" int rb_grouped_append(const GroupedAppendArgs* a, cudaStream_t stream
   p.table = a->table; p.half = a->half; p.interleaved = a->interleaved; p.max_pos = a->max_pos;
   p.q = a->q; p.keys = a->keys; p.values = a->values; p.num_blocks = a->num_blocks;
   p.H = a->H; p.G = a->G; p.dim = a->dim; p.vdim = a->vdim; p.DP = a->DP; p.T = a->T; p.status = a->status;
-  const int dev = current_device_index();
-  if (dev < 0) return -10;
-  static bool attr[RB_MAX_DEVICES] = {};
-  if (!attr[dev]) {
-    if (cudaFuncSetAttribute(grouped_append_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess ||
-        cudaFuncSetAttribute(grouped_append_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
-      return -10;
-    attr[dev] = true;
-  }
-  cudaError_t e = a->dtype == 0 ? launch_kernel(grouped_append_kernel<__nv_bfloat16>, dim3(a->T), dim3(GA_THREADS), smem, stream, p)
-                                : launch_kernel(grouped_append_kernel<float>, dim3(a->T), dim3(GA_THREADS), smem, stream, p);
+  cudaError_t e = a->dtype == 0 ? launch_grouped_append<__nv_bfloat16>(p, stream) : launch_grouped_append<float>(p, stream);
   if (e == cudaSuccess && a->cu_q != nullptr && a->taps > 1)
     e = a->dtype == 0 ? launch_history_update((const __nv_bfloat16*)a->proj, a->ld, p.rows, (__nv_bfloat16*)a->hist, a->channels, stream)
                       : launch_history_update((const float*)a->proj, a->ld, p.rows, (float*)a->hist, a->channels, stream);

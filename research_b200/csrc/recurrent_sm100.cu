@@ -9,6 +9,7 @@
 //   chunked     long portions, 128 tokens at a time on the tensor cores (tcgen05), in four launches: the gates, what every chunk
 //               adds to the state (all chunks at once), the state in front of every chunk (one pass over the chunks), the
 //               outputs (all chunks at once)
+//   time mixing, one token per sequence: as decode, a whole head at a time, with the head's norm and the output gate
 //   time mixing of long portions: chunked in the same way, in three launches
 //   gated_norm  RMS norm per head or over all heads, times sigmoid(gate), to the activation type
 //
@@ -1550,6 +1551,178 @@ static int launch_time_mix(const MixParams& p, int n_chunks, int n_seq, cudaStre
 }
 
 // ------------------------------------------------------------------------------------------
+// Time mixing, one token per sequence, heads of up to 64 channels (KP = VP = 64): a unit is a whole head of a sequence, so that its
+// norm and the output gate are finished here too. As recurrent_decode_kernel: persistent CTAs, a ring of bulk copies in both
+// directions, the unit's vectors fetched one unit ahead. Threads: 16 groups of 4 value channels x 8 of key rows.
+// ------------------------------------------------------------------------------------------
+constexpr int MD_THREADS = 128, MD_STAGES = 4, MD_DIM = 64;
+constexpr int MD_BYTES = MD_DIM * MD_DIM * 4;
+
+struct MixDecodeParams {
+  const void* proj;              // [B, ld]: r | k | v | gate
+  long long ld;
+  int k_col, v_col, g_col;
+  const float* z;                // [B, ldz]
+  long long ldz;
+  const float* w0;               // [H * 64]
+  const float* bonus;
+  const float* norm;
+  float eps;
+  float* s;                      // [slots, H, 2, 64, 32]
+  const int* slots;
+  const int* seq_lens;
+  void* out;                     // [B, ldo]
+  long long ldo;
+  int H, dk, num_slots;
+  int* status;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(MD_THREADS) time_mix_decode_kernel(const MixDecodeParams p, int units) {
+  extern __shared__ __align__(128) uint8_t smem_raw[];       // MD_STAGES x [2, 64, 32] fp32
+  __shared__ __align__(16) float4 rows_s[MD_DIM];            // r, k, decay, bonus of a key row
+  __shared__ __align__(16) float vs[MD_DIM];
+  __shared__ __align__(16) float red[MD_THREADS / 32][MD_DIM];
+  __shared__ __align__(8) uint64_t full[MD_STAGES];
+  __shared__ int abort_flag;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c4 = tid & 15, r0 = tid >> 4;
+  const uint32_t ring = smem_u32(smem_raw);
+  if (tid == 0) {
+    abort_flag = 0;
+    for (int i = 0; i < MD_STAGES; ++i) mbar_init(smem_u32(&full[i]), 1);
+    fence_mbar_init();
+  }
+  __syncthreads();
+  pdl_launch_dependents();
+  pdl_wait();
+  struct Unit { int b, h, slot; bool fresh; };
+  auto unit_of = [&](int u) {
+    Unit x;
+    x.b = u / p.H;
+    x.h = u - x.b * p.H;
+    x.slot = __ldg(p.slots + x.b);
+    if (x.slot >= p.num_slots) { set_status(p.status, ST_BAD_INDEX); x.slot = -1; }
+    x.fresh = __ldg(p.seq_lens + x.b) == 1;
+    return x;
+  };
+  auto state_of = [&](const Unit& x) { return p.s + ((long long)max(x.slot, 0) * p.H + x.h) * (MD_DIM * MD_DIM); };   // padding rows read slot 0
+  constexpr int MOVER = MD_THREADS - 32;                     // the thread that issues the copies (the first warp finishes the outputs)
+  int issued = 0;
+  auto load = [&](int i) {                                   // MOVER: state of this CTA's i-th unit
+    const int u = blockIdx.x + i * gridDim.x;
+    if (u >= units) return;
+    const uint32_t bar = smem_u32(&full[i % MD_STAGES]);
+    mbar_expect_tx(bar, MD_BYTES);
+    bulk_load(ring + (i % MD_STAGES) * MD_BYTES, state_of(unit_of(u)), MD_BYTES, bar);
+    issued = i + 1;
+  };
+  if (tid == MOVER)
+    for (int i = 0; i < MD_STAGES - 1; ++i) load(i);
+  float4 mine = make_float4(0.f, 0.f, 0.f, 0.f);             // threads below 64: the row's vectors; the others: v in .x
+  float2 gate = make_float2(0.f, 0.f), weight = make_float2(0.f, 0.f);     // first warp: two channels of the outputs
+  Unit x{};
+  auto fetch = [&](int u) {
+    x = unit_of(u);
+    const T* row = reinterpret_cast<const T*>(p.proj) + x.b * p.ld + x.h * MD_DIM;
+    const int c = x.h * MD_DIM;
+    if (tid < MD_DIM) {
+      mine = make_float4(to_f<T>(row[tid]), to_f<T>(row[p.k_col + tid]), p.z[x.b * p.ldz + c + tid] + p.w0[c + tid], p.bonus[c + tid]);
+    } else {
+      mine.x = to_f<T>(row[p.v_col + tid - MD_DIM]);
+    }
+    if (warp == 0) {
+      gate = make_float2(to_f<T>(row[p.g_col + 2 * lane]), to_f<T>(row[p.g_col + 2 * lane + 1]));
+      weight = *reinterpret_cast<const float2*>(p.norm + c + 2 * lane);
+    }
+  };
+  if ((int)blockIdx.x < units) fetch(blockIdx.x);
+  bool ok = true;
+  int it = 0;
+  for (int u = blockIdx.x; u < units; u += gridDim.x, ++it) {
+    const Unit cur = x;
+    const float2 g = gate, w = weight;
+    if (tid < MD_DIM) rows_s[tid] = make_float4(mine.x, mine.y, channel_decay(mine.z), mine.w);
+    else vs[tid - MD_DIM] = mine.x;
+    const int stage = it % MD_STAGES;
+    ok = mbar_wait_bounded(smem_u32(&full[stage]), (uint32_t)((it / MD_STAGES) & 1), &abort_flag, p.status, ST_TIMEOUT_SMEM_FULL);
+    ok = __syncthreads_and(ok);
+    if (!ok) break;
+    if (u + (int)gridDim.x < units) fetch(u + gridDim.x);
+    float4* S = reinterpret_cast<float4*>(smem_raw + stage * MD_BYTES) + (c4 >> 3) * (MD_DIM * 8) + (c4 & 7);     // row r at S[8 r]
+    const float4 v = *reinterpret_cast<const float4*>(&vs[c4 * 4]);
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < MD_DIM / 8; ++i) {
+      const int r = r0 + i * 8;
+      float4 s = cur.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : S[r * 8];
+      const float4 q = rows_s[r];
+      const float4 kv = make_float4(q.y * v.x, q.y * v.y, q.y * v.z, q.y * v.w);
+      acc.x = fmaf(q.x, fmaf(q.w, kv.x, s.x), acc.x);
+      acc.y = fmaf(q.x, fmaf(q.w, kv.y, s.y), acc.y);
+      acc.z = fmaf(q.x, fmaf(q.w, kv.z, s.z), acc.z);
+      acc.w = fmaf(q.x, fmaf(q.w, kv.w, s.w), acc.w);
+      s.x = fmaf(q.z, s.x, kv.x);
+      s.y = fmaf(q.z, s.y, kv.y);
+      s.z = fmaf(q.z, s.z, kv.z);
+      s.w = fmaf(q.z, s.w, kv.w);
+      S[r * 8] = s;
+    }
+    fence_proxy_async_smem();
+    acc.x += __shfl_xor_sync(0xffffffffu, acc.x, 16);
+    acc.y += __shfl_xor_sync(0xffffffffu, acc.y, 16);
+    acc.z += __shfl_xor_sync(0xffffffffu, acc.z, 16);
+    acc.w += __shfl_xor_sync(0xffffffffu, acc.w, 16);
+    if (lane < 16) *reinterpret_cast<float4*>(&red[warp][c4 * 4]) = acc;
+    __syncthreads();
+    if (tid == MOVER) {
+      if (cur.slot >= 0) bulk_store(state_of(cur), ring + stage * MD_BYTES, MD_BYTES);
+      else asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+      asm volatile("cp.async.bulk.wait_group.read 1;" ::: "memory");     // the state stored one unit ago has left its stage
+      load(it + MD_STAGES - 1);
+    }
+    if (warp == 0) {
+      float2 o = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int i = 0; i < MD_THREADS / 32; ++i) {
+        const float2 part = *reinterpret_cast<const float2*>(&red[i][2 * lane]);
+        o.x += part.x;
+        o.y += part.y;
+      }
+      const float rs = cur.slot < 0 ? 0.f : 1.f / sqrtf(warp_sum(o.x * o.x + o.y * o.y) / (float)p.dk + p.eps);
+      const float y0 = o.x * rs * w.x * g.x * sigmoid_f(g.x), y1 = o.y * rs * w.y * g.y * sigmoid_f(g.y);
+      T* dst = reinterpret_cast<T*>(p.out) + cur.b * p.ldo + cur.h * MD_DIM + 2 * lane;
+      if constexpr (sizeof(T) == 4) *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
+      else *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(y0, y1);
+    }
+  }
+  if (tid == MOVER) {
+    if (!ok)                                                 // no copy may land after the CTA has gone
+      for (int i = it; i < issued; ++i) {
+        const uint64_t t0 = globaltimer_ns();
+        while (!mbar_try_wait(smem_u32(&full[i % MD_STAGES]), (uint32_t)((i / MD_STAGES) & 1)))
+          if (globaltimer_ns() - t0 > 50000000ull) break;
+      }
+    asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+  }
+}
+
+template <typename T>
+static int launch_time_mix_decode(const MixDecodeParams& p, int B, cudaStream_t stream) {
+  static int sms[64] = {};
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
+  if (sms[dev] == 0) {
+    int n = 0;
+    if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess ||
+        cudaFuncSetAttribute(time_mix_decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, MD_STAGES * MD_BYTES) != cudaSuccess)
+      return -10;
+    sms[dev] = n;
+  }
+  const int units = B * p.H, grid = units < sms[dev] * 3 ? units : sms[dev] * 3;
+  return launch_kernel(time_mix_decode_kernel<T>, dim3(grid), dim3(MD_THREADS), MD_STAGES * MD_BYTES, stream, p, units) == cudaSuccess ? 0 : -11;
+}
+
+// ------------------------------------------------------------------------------------------
 // out = o / rms * weight * sigmoid(gate), or silu(gate). One CTA per token; a warp takes whole heads. Padding channels of o are zero.
 template <typename T>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ weight,
@@ -1756,6 +1929,17 @@ int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, in
     case 256: return launch_chunks<256>(p, n_chunks, n_seq, stream);
     default: return -1;
   }
+}
+
+// Time mixing of one token per sequence down to the normed and gated output rows; heads padded to 64 channels. Activations and out
+// in bf16 (dtype 0) or fp32.
+int rb_time_mix_decode(const void* proj, long long ld, int k_col, int v_col, int g_col, const float* z, long long ldz, const float* w0,
+                       const float* bonus, const float* norm, float eps, float* s, const int* slots, const int* seq_lens, void* out, long long ldo,
+                       int B, int H, int dk, int num_slots, int dtype, int* status, cudaStream_t stream) {
+  if (B <= 0) return 0;
+  if (H <= 0 || dk <= 0 || dk > MD_DIM || ldo % 2 != 0) return -1;
+  const MixDecodeParams p{proj, ld, k_col, v_col, g_col, z, ldz, w0, bonus, norm, eps, s, slots, seq_lens, out, ldo, H, dk, num_slots, status};
+  return dtype == 0 ? launch_time_mix_decode<__nv_bfloat16>(p, B, stream) : launch_time_mix_decode<float>(p, B, stream);
 }
 
 // Workspace of the chunked time mixing in bytes.

@@ -224,19 +224,17 @@ class TimeMixPart(Part):
 
     def recur(self, w: TimeMixWeights, cache: TimeMixState, proj, z, out, b, plan) -> None:
         T, g, eps = b.num_tokens, w.geo, self.r.cfg.norm_eps
-        o = self.o[:T * g.heads * g.vp].view(T, -1)
         mix = TimeMix(z, w.w0, w.bonus)
         n_seq, rows, table = plan if time_mix_chunked_supported(g) else (b.rows, T, None)
         single = b.rows if b.cu_q is None else b.n_single
-        args = (proj, None, g, None, None, None, 1.0, cache.state, b.state_slots)
         if single > 0:
-            ops.recurrent_scan(*args, None, b.seq_lens, o, single, single, mix=mix)
+            ops.time_mix_decode(proj, g, mix, cache.state, b.state_slots, b.seq_lens, w.norm, eps, out, single)
         if n_seq > single:
-            ops.recurrent_scan(*args, b.cu_q, b.seq_lens, o, rows, n_seq, single, mix=mix)
-        if rows > 0:
-            ops.gated_norm(o[:rows], w.norm, proj[:, g.offsets[3]:], g, eps, out, True, silu=True)
+            o = self.o[:T * g.heads * g.vp].view(T, -1)
+            ops.recurrent_scan(proj, None, g, None, None, None, 1.0, cache.state, b.state_slots, b.cu_q, b.seq_lens, o, rows, n_seq, single, mix=mix)
+            ops.gated_norm(o[single:rows], w.norm, proj[single:, g.offsets[3]:], g, eps, out[single:], True, silu=True)
         if table is not None:
-            room = torch.empty(time_mix_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=o.device)
+            room = torch.empty(time_mix_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=out.device)
             ops.time_mix_chunks(proj, g, mix, cache.state, b.state_slots, b.cu_q, b.seq_lens, w.norm, eps, out, table, room)
 
     def forward(self, w: TimeMixWeights, cache: TimeMixState, inp, y, b, plan, small=None) -> None:

@@ -113,9 +113,11 @@ def _lib() -> ctypes.CDLL:
         lib.rb_recurrent_chunk_workspace.argtypes, lib.rb_recurrent_chunk_workspace.restype = [c_int] * 4, c_ll
         lib.rb_time_mix_chunks.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 9 + [c_float, c_vp, c_ll, c_vp] + [c_int] * 6
                                            + [c_vp, c_vp])
+        lib.rb_time_mix_decode.argtypes = ([c_vp, c_ll] + [c_int] * 3 + [c_vp, c_ll] + [c_vp] * 3 + [c_float] + [c_vp] * 4 + [c_ll] + [c_int] * 5
+                                           + [c_vp, c_vp])
         lib.rb_time_mix_workspace.argtypes, lib.rb_time_mix_workspace.restype = [c_int] * 3, c_ll
         lib.rb_gated_norm.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_ll] + [c_int] * 7 + [c_float, c_vp]
-        for f in ("rb_recurrent_scan", "rb_recurrent_chunks", "rb_gated_norm", "rb_token_shift", "rb_tanh_parts", "rb_time_mix_chunks"):
+        for f in ("rb_recurrent_scan", "rb_recurrent_chunks", "rb_gated_norm", "rb_token_shift", "rb_tanh_parts", "rb_time_mix_chunks", "rb_time_mix_decode"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -239,6 +241,22 @@ def chunk_workspace(n_chunks: int, geo: RecurrentGeometry) -> int:
     return int(_lib().rb_recurrent_chunk_workspace(n_chunks, geo.heads, geo.kp, geo.vp))
 
 
+def time_mix_decode(proj, geo: RecurrentGeometry, mix: TimeMix, state: RecurrentState, slots, seq_lens, norm, eps: float, out, n: int) -> None:
+    """Time mixing of the first ``n`` sequences, one row each, norm per head and SiLU gate included: rows of ``out [>= n, H*vp]`` in the
+    activation type, state updated."""
+    _, ok, ov, og = geo.offsets
+    if not proj.is_cuda or geo.kp != 64:
+        o = torch.empty(n, geo.heads * geo.vp, dtype=torch.float32, device=proj.device)
+        recurrent_scan(proj, None, geo, None, None, None, 1.0, state, slots, None, seq_lens, o, n, n, mix=mix)
+        gated_norm(o, norm, proj[:, og:], geo, eps, out, True, silu=True)
+        return
+    assert proj.stride(1) == out.stride(1) == 1 and proj.dtype == out.dtype and mix.z.dtype == norm.dtype == torch.float32
+    rc = _lib().rb_time_mix_decode(ptr(proj), proj.stride(0), ok, ov, og, ptr(mix.z), mix.z.stride(0), ptr(mix.w0), ptr(mix.bonus), ptr(norm), eps,
+                                   ptr(state.s), ptr(slots), ptr(seq_lens), ptr(out), out.stride(0), n, geo.heads, geo.dim, state.s.shape[0],
+                                   _DT[proj.dtype], ptr(status_tensor(proj.device)), stream_handle(proj.device))
+    check_rc(rc, "rb_time_mix_decode")
+
+
 def time_mix_chunked_supported(geo: RecurrentGeometry) -> bool:
     return geo.kp in (64, 128) and geo.kp == geo.vp
 
@@ -300,6 +318,7 @@ def gated_norm(o, weight, gate, geo: RecurrentGeometry, eps: float, out, per_hea
     head's ``vdim`` channels (``per_head``) or over all heads'."""
     T, H, VP = o.shape[0], geo.heads, geo.vp
     if not o.is_cuda:
+        gate = gate[:T]
         x = o.view(T, H, VP)
         ms = x.pow(2).sum(-1) / geo.vdim if per_head else (x.pow(2).sum((1, 2)) / (H * geo.vdim))[:, None].expand(T, H)
         y = x * torch.rsqrt(ms + eps)[..., None] * weight.view(1, H, VP) * (torch.nn.functional.silu if silu else torch.sigmoid)(gate.float().reshape(T, H, VP))

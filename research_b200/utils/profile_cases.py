@@ -303,6 +303,92 @@ def case_keyvalue_decode() -> None:
     print("ok")
 
 
+def _time_mix(T: int, seqs: int):
+    """32 heads of 64 channels: activations of T rows, state of ``seqs`` sequences."""
+    from ..ops.recurrent import RecurrentGeometry, RecurrentState, TimeMix
+
+    geo = RecurrentGeometry(32, 64, 64, silu=False, gated=False)
+    proj, norm = torch.randn(T, geo.proj, device="cuda").bfloat16(), torch.ones(2048, device="cuda")
+    mix = TimeMix(torch.randn(T, 2048, device="cuda") - 3, torch.zeros(2048, device="cuda"), torch.randn(2048, device="cuda"))
+    return proj, geo, mix, RecurrentState.zeros(geo, seqs, "cuda"), torch.arange(seqs, dtype=torch.int32, device="cuda"), norm
+
+
+def case_time_mix_decode() -> None:
+    """Time mixing, one token for each of 256 sequences: 32 heads of 64 x 64 (134 MB of state)."""
+    proj, geo, mix, state, slots, norm = _time_mix(256, 256)
+    lens, out = torch.full((256,), 100, dtype=torch.int32, device="cuda"), torch.empty(256, 2048, dtype=torch.bfloat16, device="cuda")
+    for _ in range(3):
+        ops.time_mix_decode(proj, geo, mix, state, slots, lens, norm, 1e-6, out, 256)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def case_time_mix_prefill() -> None:
+    """Time mixing in chunks: one portion of 4096 tokens, 32 heads of 64 x 64."""
+    from ..ops.recurrent import ChunkTable, time_mix_workspace
+
+    T = 4096
+    proj, geo, mix, state, slots, norm = _time_mix(T, 1)
+    cu, lens = torch.tensor([0, T], dtype=torch.int32, device="cuda"), torch.tensor([T], dtype=torch.int32, device="cuda")
+    table, out = ChunkTable.make([0, T], 0, "cuda"), torch.empty(T, 2048, dtype=torch.bfloat16, device="cuda")
+    room = torch.empty(time_mix_workspace(table.chunks.shape[0], geo), dtype=torch.uint8, device="cuda")
+    z = mix.z.clone()
+    for _ in range(3):
+        mix.z.copy_(z)
+        ops.time_mix_chunks(proj, geo, mix, state, slots, cu, lens, norm, 1e-6, out, table, room)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def _grouped(T: int, rows_cached: int, conv: bool):
+    from ..ops.grouped import GroupedCache, GroupedGeometry
+
+    geo = GroupedGeometry(16, 4, 128, 128, 4 if conv else 1, conv, "head" if conv else "projection", 64, conv)
+    cache = GroupedCache(*(torch.randn(rows_cached // 16, 4, 16, 128, device="cuda").bfloat16() for _ in range(2)),
+                         torch.zeros(2, 3, geo.channels, device="cuda").bfloat16() if conv else None)
+    return geo, cache, torch.randn(T, geo.proj, device="cuda").bfloat16(), torch.empty(T, 2048, dtype=torch.bfloat16, device="cuda")
+
+
+def _case_append(conv: bool) -> None:
+    T = 4096
+    geo, cache, proj, q = _grouped(T, T, conv)
+    pos = torch.arange(T, dtype=torch.int32, device="cuda")
+    cu, slot = torch.tensor([0, T], dtype=torch.int32, device="cuda"), torch.zeros(1, dtype=torch.int32, device="cuda")
+    ones, table = torch.ones(2048, device="cuda"), ops.frequency_table(T, [0.9 ** i for i in range(32)], 1.0, "cuda")
+    for _ in range(3):
+        ops.grouped_append(proj, geo, conv=torch.ones(4, geo.channels, device="cuda") if conv else None, cache=cache, cu_q=cu, positions=pos, state_slots=slot,
+                           slots=pos, q_norm=None if conv else ones, k_norm=None if conv else ones, eps=1e-6, table=table, q=q)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def case_grouped_append() -> None:
+    """Norm over the projection, rotation and cache append of 4096 tokens: 16 query heads on 4 kv heads of 128 channels."""
+    _case_append(False)
+
+
+def case_grouped_append_conv() -> None:
+    """The same with convolutions of 4 taps and a norm per head."""
+    _case_append(True)
+
+
+def case_grouped_decode() -> None:
+    """Attention over cached keys and values: 256 sequences x 2048 keys, 16 query heads on 4 kv heads of 128 channels (1 GB of cache)."""
+    B, L = 256, 2048
+    geo, cache, _, q = _grouped(B, B * L, False)
+    bt = torch.randperm(B * L // 16, device="cuda").int().view(B, -1)
+    lens, out = torch.full((B,), L, dtype=torch.int32, device="cuda"), torch.empty(B, 2048, dtype=torch.bfloat16, device="cuda")
+    q.normal_()
+    for _ in range(3):
+        ops.grouped_attention(q, geo, cache, bt, None, lens, out, scale=0.09, rows=B, max_q=1, n_single=B)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
 CASES = {k[5:]: v for k, v in globals().items() if k.startswith("case_")}
 
 if __name__ == "__main__":

@@ -119,6 +119,41 @@ def test_append_in_portions(place, shape):
         assert (cache.history[free] == 9.0).all()
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("shape", APPENDS)
+def test_append_of_a_large_batch(cuda_device, dtype, shape):
+    """Hundreds of rows of unlike sequences at once, some behind a history, some without a place in the cache: as the CPU twin."""
+    H, G, D, E, taps, conv, norm, rot, inter = shape
+    geo = GroupedGeometry(H, G, D, E, taps, conv, norm, rot, inter)
+    lens, done, nb = [1, 2, 1, 3, 300, 290, 7, 5], [0, 4, 1, 0, 0, 33, 2, 0], 60
+    cu = [0]
+    for n in lens:
+        cu.append(cu[-1] + n)
+    T = cu[-1]
+    proj = torch.zeros(T, geo.proj)
+    for col, n in ((0, H * D), (geo.k_col, G * D), (geo.v_col, G * E)):
+        proj[:, col:col + n] = rand(T, n, seed=col + 1, dtype=torch.bfloat16)
+    slots = torch.randperm(nb * KV_BLOCK, generator=torch.Generator().manual_seed(3))[:T].int()
+    slots[::9] = -1
+    positions = torch.cat([torch.arange(d, d + n) for n, d in zip(lens, done)]).int()
+    state_slots = torch.tensor([6, 2, 0, 8, 1, 3, 9, 5], dtype=torch.int32)
+    weights = rand(taps, geo.channels, seed=7) if conv else None
+    qn, kn = (rand(n * D, seed=8 + i) + 1.5 if norm == "projection" else None for i, n in enumerate((H, G)))
+    table = ops.frequency_table(400, [0.9 ** i for i in range(rot // 2)], 1.2)
+    res = []
+    for dev, dt in (("cpu", torch.float32), (cuda_device, dtype)):
+        cache = GroupedCache(*(torch.zeros(nb, G, KV_BLOCK, geo.dp, dtype=dt, device=dev) for _ in range(2)),
+                             rand(10, taps - 1, geo.channels, seed=4, dtype=torch.bfloat16).to(dt).to(dev) if taps > 1 else None)
+        q = torch.zeros(T, H * geo.dp, dtype=dt, device=dev)
+        to = lambda t: t.to(dev) if t is not None else None
+        ops.grouped_append(proj.to(dt).to(dev), geo, conv=to(weights), cache=cache, cu_q=i32(cu, dev), positions=to(positions), state_slots=to(state_slots),
+                           slots=to(slots), q_norm=to(qn), k_norm=to(kn), eps=1e-4, table=to(table), q=q)
+        res.append((q, cache.keys, cache.values) + ((cache.history,) if taps > 1 else ()))
+    for want, got in zip(*res):
+        close(got, want, dtype)
+
+
 @pytest.mark.parametrize("place", PLACES)
 def test_append_skips_padding_rows(place):
     dev, dt = place
@@ -297,11 +332,10 @@ def test_time_mixing_in_portions_slots_and_batches(place, shape, strong):
         chunks = dt == torch.bfloat16 and dev == "cuda" and time_mix_chunked_supported(geo)
         short = next((i for i, b in enumerate(order) if parts[b] > 16), len(order)) if chunks else len(order)
         if single:
-            ops.recurrent_scan(*a, None, sl, o, single, single, mix=mix)
+            ops.time_mix_decode(proj, geo, mix, state, a[-1], sl, flat["norm"], eps, out, single)
         if short > single:
             ops.recurrent_scan(*a, cut, sl, o, cu[short], short, single, mix=mix)
-        if cu[short]:
-            ops.gated_norm(o[:cu[short]], flat["norm"], proj[:, geo.offsets[3]:], geo, eps, out, True, silu=True)
+            ops.gated_norm(o[single:cu[short]], flat["norm"], proj[single:, geo.offsets[3]:], geo, eps, out[single:], True, silu=True)
         if short < len(order):
             table = ChunkTable.make(cu, short, dev)
             room = torch.empty(time_mix_workspace(table.chunks.shape[0], geo), dtype=torch.uint8, device=dev)
@@ -317,6 +351,37 @@ def test_time_mixing_in_portions_slots_and_batches(place, shape, strong):
         close(o[..., :D].reshape(n, -1), want[b], dt, (shape, b))
     for part in (1, 3):         # slots nobody owns keep what they held
         assert (state.s[part] == 7.0).all()
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,D,B", [(6, 40, 300), (32, 64, 64), (1, 64, 1), (3, 128, 50)])
+def test_decode_of_many_sequences(cuda_device, dtype, H, D, B):
+    """More heads than CTAs, fresh and continued sequences and padding rows: the one-token kernels equal the scan."""
+    geo = RecurrentGeometry(H, D, D, silu=False, gated=False)
+    n, dev = H * geo.kp, cuda_device
+    r, k, v, g, z = mix_case(geo, [B], 3, False)
+    proj = torch.cat([padded(x, geo.kp) for x in (r, k, v, g)], 1).to(dtype).to(dev)
+    mix = TimeMix(padded(z, geo.kp).to(dev), padded(rand(1, H, D, seed=8), geo.kp).view(-1).to(dev), padded(rand(1, H, D, seed=4), geo.kp).view(-1).to(dev))
+    norm = padded(rand(1, H, D, seed=9) + 1.0, geo.kp).view(-1).to(dev)
+    states = [RecurrentState.zeros(geo, B + 3, dev) for _ in range(2)]
+    start = torch.zeros(B + 3, H, geo.kp, geo.vp)
+    start[:, :, :D, :D] = rand(B + 3, H, D, D, seed=5)
+    for s in states:
+        s.s.copy_(start.view(B + 3, H, geo.kp, geo.tiles, 32).permute(0, 1, 3, 2, 4))
+    slots = (torch.randperm(B, generator=torch.Generator().manual_seed(1)) + 2).int()
+    lens = torch.where(torch.arange(B) % 5 == 3, 1, 20).int()
+    if B > 2:
+        slots[B // 2], slots[B - 1] = -1, -1
+    slots, lens = slots.to(dev), lens.to(dev)
+    o, outs = torch.zeros(B, n, device=dev), [torch.zeros(B, n, dtype=dtype, device=dev) for _ in range(2)]
+    ops.recurrent_scan(proj, None, geo, None, None, None, 1.0, states[0], slots, torch.arange(B + 1, dtype=torch.int32, device=dev), lens, o, B, B, mix=mix)
+    ops.gated_norm(o, norm, proj[:, 3 * n:], geo, 1e-5, outs[0], True, silu=True)
+    ops.time_mix_decode(proj, geo, mix, states[1], slots, lens, norm, 1e-5, outs[1], B)
+    ops.check_status()
+    close(outs[1], outs[0].cpu(), dtype)
+    close(states[1].s, states[0].s.cpu(), torch.float32)
+    assert B <= 2 or outs[1][B - 1].abs().max() == 0
 
 
 @pytest.mark.gpu
