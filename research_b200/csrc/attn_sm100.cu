@@ -1205,60 +1205,73 @@ __device__ __forceinline__ void load8(const T* p, float (&x)[8]) {
   }
 }
 
-// TOK rows per CTA (the convolution's weights are loaded once for them); STEPS: 64 channels of a padded head each.
-template <typename T, int TOK, int STEPS>
-__global__ void __launch_bounds__(GA_THREADS) grouped_append_kernel(const GroupedAppend p) {
+// TOK rows per CTA (the convolution's weights are loaded once for them); STEPS: 64 channels of a padded head each; WHOLE: heads of
+// queries, keys and values have DP channels, none of them padding.
+template <typename T, int TOK, int STEPS, bool WHOLE>
+__global__ void __launch_bounds__(GA_THREADS, 4) grouped_append_kernel(const GroupedAppend p) {
   extern __shared__ float ga_rows[];                      // [TOK][v_col] q and k channels, laid out as in the projection
   __shared__ float red[TOK][2][GA_THREADS / 32];
   __shared__ RowPlace places[TOK];
   __shared__ int dests[TOK];
+  __shared__ long long caches[TOK];                       // element of the row in the caches, + head * 16 * DP
+  const int DP = WHOLE ? STEPS * 64 : p.DP, dim = WHOLE ? DP : p.dim, vdim = WHOLE ? DP : p.vdim;
   pdl_launch_dependents();
   pdl_wait();
   const int t0 = blockIdx.x * TOK, n_tok = min(TOK, p.T - t0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* rows = reinterpret_cast<const T*>(p.proj);
   T* hist = reinterpret_cast<T*>(p.hist);
-  if (threadIdx.x < n_tok) {
-    const int t = t0 + threadIdx.x;
-    RowPlace place{0, p.rows.positions[t], -1};
-    if (p.taps > 1) place = row_place(p.rows, t, p.status);
-    int slot = p.slots[t];
-    if (slot >= 0 && slot / KV_BLOCK >= p.num_blocks) { set_status(p.status, ST_BAD_INDEX); slot = -1; }
-    if (place.position < 0 || place.position >= p.max_pos) { set_status(p.status, ST_BAD_INDEX); place.position = 0; }
+  if (threadIdx.x < TOK) {
+    RowPlace place{0, 0, -1};
+    int slot = -1;
+    if (threadIdx.x < n_tok) {
+      const int t = t0 + threadIdx.x;
+      place.position = p.rows.positions[t];
+      if (p.taps > 1) place = row_place(p.rows, t, p.status);
+      slot = p.slots[t];
+      if (slot >= 0 && slot / KV_BLOCK >= p.num_blocks) { set_status(p.status, ST_BAD_INDEX); slot = -1; }
+      if (place.position < 0 || place.position >= p.max_pos) { set_status(p.status, ST_BAD_INDEX); place.position = 0; }
+    }
     places[threadIdx.x] = place;
     dests[threadIdx.x] = slot;
+    caches[threadIdx.x] = slot < 0 ? 0 : ((long long)(slot / KV_BLOCK) * p.G * KV_BLOCK + slot % KV_BLOCK) * DP;
   }
   __syncthreads();
-  auto cache_row = [&](int slot) { return ((long long)(slot / KV_BLOCK) * p.G * KV_BLOCK + slot % KV_BLOCK) * p.DP; };   // + head * 16 * DP
+  bool near = true;                                       // every row's look back lies in the batch
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) near = near && (i >= n_tok || places[i].offset >= p.taps - 1);
   float ssq[TOK], ssk[TOK];
 #pragma unroll
   for (int i = 0; i < TOK; ++i) ssq[i] = ssk[i] = 0.f;
-  const int nq = p.H * p.dim, nk = p.G * p.dim, nv = p.G * p.vdim;
+  const int nq = p.H * dim, nk = p.G * dim, nv = p.G * vdim;
   for (int c = threadIdx.x * 8; c < p.channels; c += GA_THREADS * 8) {
     float x[TOK][8], u[8];
+    const T* first = rows + (long long)t0 * p.ld + c;
 #pragma unroll
     for (int i = 0; i < TOK; ++i)
-      if (i < n_tok) load8(rows + (long long)(t0 + i) * p.ld + c, x[i]);
+      if (i < n_tok) load8(first + i * p.ld, x[i]);
     if (p.conv != nullptr) {
       if (TOK == 1)
 #pragma unroll
         for (int j = 0; j < 8; ++j) u[j] = x[0][j];
-      for (int d = 0; d < p.taps; ++d) {
-        float w[8];
-        load8(p.conv + (long long)(p.taps - 1 - d) * p.channels + c, w);
+      const float* taps = p.conv + (long long)(p.taps - 1) * p.channels + c;
+      float w[8];
+      load8(taps, w);
+#pragma unroll
+      for (int i = 0; i < TOK; ++i)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[i][j] *= w[j];
+      for (int d = 1; d < p.taps; ++d) {
+        taps -= p.channels;
+        load8(taps, w);
 #pragma unroll
         for (int i = 0; i < TOK; ++i) {
           if (i >= n_tok) continue;
-          if (d == 0) {
+          const T* back = near ? first + (i - d) * p.ld : row_before(places[i], d, rows + c, p.ld, t0 + i, (const T*)hist + c, p.taps - 1, p.channels);
+          if (near || back != nullptr) {
+            float y[8];
+            load8(back, y);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) x[i][j] *= w[j];
-          } else {
-            const T* back = row_before(places[i], d, rows, p.ld, t0 + i, (const T*)hist, p.taps - 1, p.channels);
-            if (back != nullptr) {
-              float y[8];
-              load8(back + c, y);
-#pragma unroll
-              for (int j = 0; j < 8; ++j) x[i][j] = fmaf(w[j], y[j], x[i][j]);
-            }
+            for (int j = 0; j < 8; ++j) x[i][j] = fmaf(w[j], y[j], x[i][j]);
           }
         }
       }
@@ -1273,32 +1286,39 @@ __global__ void __launch_bounds__(GA_THREADS) grouped_append_kernel(const Groupe
     }
     if (c >= p.v_col) {
       const int v0 = c - p.v_col;
+      if (WHOLE || vdim % 8 == 0) {
+        const int at = v0 / vdim * KV_BLOCK * DP + v0 % vdim;
+        if (v0 < nv)
 #pragma unroll
-      for (int i = 0; i < TOK; ++i) {
-        if (i >= n_tok || dests[i] < 0) continue;
-        T* vcache = reinterpret_cast<T*>(p.values) + cache_row(dests[i]);
-        if (p.vdim % 8 == 0) {
-          if (v0 < nv) store8(vcache + (long long)(v0 / p.vdim) * KV_BLOCK * p.DP + v0 % p.vdim, x[i]);
-        } else {
-#pragma unroll
+          for (int i = 0; i < TOK; ++i)
+            if (dests[i] >= 0) store8(reinterpret_cast<T*>(p.values) + caches[i] + at, x[i]);
+      } else {
+#pragma unroll 1
+        for (int i = 0; i < TOK; ++i)
           for (int j = 0; j < 8; ++j)
-            if (v0 + j < nv) kv_store(vcache + (long long)((v0 + j) / p.vdim) * KV_BLOCK * p.DP + (v0 + j) % p.vdim, x[i][j]);
-        }
+            if (dests[i] >= 0 && v0 + j < nv) {
+              float one = 0.f;
+#pragma unroll
+              for (int k = 0; k < TOK * 8; ++k)
+                if (k == i * 8 + j) one = x[k >> 3][k & 7];
+              kv_store(reinterpret_cast<T*>(p.values) + caches[i] + (v0 + j) / vdim * KV_BLOCK * DP + (v0 + j) % vdim, one);
+            }
       }
     } else {
       const bool is_k = c >= p.k_col;
       const int n = is_k ? nk : nq, c0 = c - (is_k ? p.k_col : 0);
 #pragma unroll
       for (int i = 0; i < TOK; ++i) {
-        if (i >= n_tok) continue;
         float4* dst = reinterpret_cast<float4*>(ga_rows + i * p.v_col + c);
         dst[0] = make_float4(x[i][0], x[i][1], x[i][2], x[i][3]);
         dst[1] = make_float4(x[i][4], x[i][5], x[i][6], x[i][7]);
-        float s = 0.f;
+        if (p.norm == GA_NORM_PROJECTION) {
+          float s = 0.f;
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
-          if (c0 + j < n) s = fmaf(x[i][j], x[i][j], s);
-        if (is_k) ssk[i] += s; else ssq[i] += s;
+          for (int j = 0; j < 8; ++j)
+            if (WHOLE || c0 + j < n) s = fmaf(x[i][j], x[i][j], s);
+          if (is_k) ssk[i] += s; else ssq[i] += s;
+        }
       }
     }
   }
@@ -1320,56 +1340,71 @@ __global__ void __launch_bounds__(GA_THREADS) grouped_append_kernel(const Groupe
     __syncthreads();
   }
   // A warp per head: lane e takes a pair of channels that the rotation turns, (2e, 2e + 1) or (e, e + half), or two that pass.
-  const int heads = p.H + p.G;
-  for (int u = warp; u < n_tok * heads; u += GA_THREADS / 32) {
-    const int i = u / heads, hd = u - i * heads;
+  const int heads = p.H + p.G, half = p.half;
+  int i = 0, hd = warp;
+  while (hd >= heads) { hd -= heads; ++i; }
+  while (i < n_tok) {
     const bool is_k = hd >= p.H;
     const int head = is_k ? hd - p.H : hd;
-    if (is_k && dests[i] < 0) continue;
-    const float* src = ga_rows + i * p.v_col + (is_k ? p.k_col : 0) + head * p.dim;
-    const float* w = (is_k ? p.k_norm : p.q_norm) + head * p.dim;
-    const float r = p.norm == GA_NORM_PROJECTION ? red[i][is_k][0] : 1.f;
-    const float2* table = reinterpret_cast<const float2*>(p.table) + (long long)places[i].position * p.half;
-    float y[STEPS][2], ss = 0.f;
-    int at0[STEPS], at1[STEPS];
+    if (!is_k || dests[i] >= 0) {
+      const float* src = ga_rows + i * p.v_col + (is_k ? p.k_col : 0) + head * dim;
+      const float* w = p.norm == GA_NORM_PROJECTION ? (is_k ? p.k_norm : p.q_norm) + head * dim : nullptr;
+      const float r = w != nullptr ? red[i][is_k][0] : 1.f;
+      const float2* table = reinterpret_cast<const float2*>(p.table) + (long long)places[i].position * half;
+      T* dst = is_k ? reinterpret_cast<T*>(p.keys) + caches[i] + head * KV_BLOCK * DP : reinterpret_cast<T*>(p.q) + ((long long)(t0 + i) * p.H + head) * DP;
+      float y[STEPS][2], ss = 0.f;
 #pragma unroll
-    for (int j = 0; j < STEPS; ++j) {
-      const int e = lane + j * 32;
-      const bool turned = e < p.half, split = turned && !p.interleaved;
-      at0[j] = split ? e : 2 * e;
-      at1[j] = split ? e + p.half : 2 * e + 1;
-      float a = at0[j] < p.dim ? src[at0[j]] : 0.f, b = at1[j] < p.dim ? src[at1[j]] : 0.f;
-      if (p.norm == GA_NORM_PROJECTION) {
-        if (at0[j] < p.dim) a *= r * w[at0[j]];
-        if (at1[j] < p.dim) b *= r * w[at1[j]];
+      for (int j = 0; j < STEPS; ++j) {
+        const int e = lane + j * 32;
+        const bool turned = e < half;
+        float a, b;
+        if (turned && !p.interleaved) {
+          a = src[e];
+          b = src[e + half];
+          if (w != nullptr) { a *= r * w[e]; b *= r * w[e + half]; }
+        } else if (WHOLE) {
+          const float2 v = *reinterpret_cast<const float2*>(src + 2 * e);
+          a = v.x;
+          b = v.y;
+          if (w != nullptr) {
+            const float2 f = *reinterpret_cast<const float2*>(w + 2 * e);
+            a *= r * f.x;
+            b *= r * f.y;
+          }
+        } else {
+          a = 2 * e < dim ? src[2 * e] : 0.f;
+          b = 2 * e + 1 < dim ? src[2 * e + 1] : 0.f;
+          if (w != nullptr) {
+            if (2 * e < dim) a *= r * w[2 * e];
+            if (2 * e + 1 < dim) b *= r * w[2 * e + 1];
+          }
+        }
+        if (turned) {
+          const float2 cs = table[e];
+          const float a0 = a;
+          a = a0 * cs.x - b * cs.y;
+          b = b * cs.x + a0 * cs.y;
+        }
+        y[j][0] = a;
+        y[j][1] = b;
+        ss = fmaf(a, a, fmaf(b, b, ss));
       }
-      if (turned) {
-        const float2 cs = table[e];
-        const float a0 = a;
-        a = a0 * cs.x - b * cs.y;
-        b = b * cs.x + a0 * cs.y;
-      }
-      y[j][0] = a;
-      y[j][1] = b;
-      ss = fmaf(a, a, fmaf(b, b, ss));
-    }
-    if (p.norm == GA_NORM_HEAD) {
-      const float f = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+      float f = 1.f;
+      if (p.norm == GA_NORM_HEAD) f = 1.f / sqrtf(warp_sum(ss) / (float)dim + p.eps);
 #pragma unroll
-      for (int j = 0; j < STEPS; ++j) { y[j][0] *= f; y[j][1] *= f; }
-    }
-    T* dst = is_k ? reinterpret_cast<T*>(p.keys) + cache_row(dests[i]) + (long long)head * KV_BLOCK * p.DP
-                  : reinterpret_cast<T*>(p.q) + ((long long)(t0 + i) * p.H + head) * p.DP;
-#pragma unroll
-    for (int j = 0; j < STEPS; ++j) {
-      if (at1[j] >= p.DP) continue;
-      if (at1[j] == at0[j] + 1 && (at0[j] & 1) == 0) {
-        store2(dst + at0[j], y[j][0], y[j][1]);
-      } else {
-        kv_store(dst + at0[j], y[j][0]);
-        kv_store(dst + at1[j], y[j][1]);
+      for (int j = 0; j < STEPS; ++j) {
+        const int e = lane + j * 32;
+        if (!WHOLE && 2 * e >= DP) continue;
+        if (e < half && !p.interleaved) {
+          kv_store(dst + e, y[j][0] * f);
+          kv_store(dst + e + half, y[j][1] * f);
+        } else {
+          store2(dst + 2 * e, y[j][0] * f, y[j][1] * f);
+        }
       }
     }
+    hd += GA_THREADS / 32;
+    while (hd >= heads) { hd -= heads; ++i; }
   }
 }
 
@@ -1378,20 +1413,29 @@ static cudaError_t launch_grouped_append(const GroupedAppend& p, cudaStream_t st
   const int dev = current_device_index();
   if (dev < 0) return cudaErrorInvalidDevice;
   const size_t row = (size_t)p.v_col * 4;
-  const bool several = p.rows.cu_q != nullptr && p.T >= 592 && 4 * row <= 100 * 1024;      // (rows of one sequence lie together)
-#define RB_APPEND(TOK, STEPS)                                                                                                  \
+  const bool several = p.rows.cu_q != nullptr && p.T >= 592 && 2 * row <= 100 * 1024;      // (rows of one sequence lie together)
+  const bool whole = p.dim == p.DP && p.vdim == p.DP && p.H * p.dim == p.k_col;
+#define RB_APPEND(TOK, STEPS, WHOLE)                                                                                           \
   do {                                                                                                                         \
     static bool attr[RB_MAX_DEVICES] = {};                                                                                     \
     if (!attr[dev]) {                                                                                                          \
-      const cudaError_t e = cudaFuncSetAttribute(grouped_append_kernel<T, TOK, STEPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+      const cudaError_t e = cudaFuncSetAttribute(grouped_append_kernel<T, TOK, STEPS, WHOLE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
       if (e != cudaSuccess) return e;                                                                                          \
       attr[dev] = true;                                                                                                        \
     }                                                                                                                          \
-    return launch_kernel(grouped_append_kernel<T, TOK, STEPS>, dim3((p.T + TOK - 1) / TOK), dim3(GA_THREADS), TOK * row, stream, p); \
+    return launch_kernel(grouped_append_kernel<T, TOK, STEPS, WHOLE>, dim3((p.T + TOK - 1) / TOK), dim3(GA_THREADS), TOK * row, stream, p); \
   } while (0)
-  if (p.DP == 64) { if (several) RB_APPEND(4, 1); else RB_APPEND(1, 1); }
-  if (p.DP == 128) { if (several) RB_APPEND(4, 2); else RB_APPEND(1, 2); }
-  if (several) RB_APPEND(4, GA_MAX_DP / 64); else RB_APPEND(1, GA_MAX_DP / 64);
+#define RB_APPEND_SIZE(STEPS, WHOLE)                                                                                           \
+  do {                                                                                                                         \
+    if (several) RB_APPEND(2, STEPS, WHOLE);                                                                                   \
+    RB_APPEND(1, STEPS, WHOLE);                                                                                                \
+  } while (0)
+  if (p.DP == 64 && whole) RB_APPEND_SIZE(1, true);
+  if (p.DP == 64) RB_APPEND_SIZE(1, false);
+  if (p.DP == 128 && whole) RB_APPEND_SIZE(2, true);
+  if (p.DP == 128) RB_APPEND_SIZE(2, false);
+  RB_APPEND_SIZE(GA_MAX_DP / 64, false);
+#undef RB_APPEND_SIZE
 #undef RB_APPEND
 }
 

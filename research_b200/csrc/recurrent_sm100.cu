@@ -1092,8 +1092,8 @@ static int launch_chunks(const ChunkParams& p, int n_chunks, int n_seq, cudaStre
 //
 // Every exponent above is <= 0, but P does not factor over t and j without one that is not: 2^-A_j overflows. So P is made in
 // blocks of 16 x 16 below the diagonal, whose two factors are taken relative to the token in front of the block row, both <= 1
-// (mma.sync, their operands are made in registers); of a block on the diagonal the lower left quarter goes the same way
-// and the two 8 x 8 triangles pair by pair in fp32. P V and the state's part run on tcgen05. Three launches: what every chunk
+// (mma.sync, their operands are made in registers); of a block on the diagonal the lower left quarter and the lower left quarters
+// of the other two go the same way, and the four 4 x 4 triangles pair by pair in fp32. P V and the state's part run on tcgen05. Three launches: what every chunk
 // adds to the state (z becomes A on the way), the chain of states, outputs with the head's norm and the output gate.
 // ------------------------------------------------------------------------------------------
 constexpr float MIX_MOST = 64.f;      // a token that keeps less than 2^-64 keeps nothing; larger sums would cost A its last digits
@@ -1135,9 +1135,9 @@ struct MixStateCfg {
 template <int DK>
 __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_state_kernel(const MixParams p) {
   using Cfg = MixStateCfg<DK>;
-  constexpr int SEGS = CHT / DK, SEG = CH / SEGS;       // a thread has one channel of SEG tokens
+  constexpr int SEGS = 2 * CHT / DK, SEG = CH / SEGS;   // a thread has two channels of SEG tokens
   extern __shared__ __align__(128) uint8_t smem_raw[];
-  __shared__ float sums[SEGS][DK];
+  __shared__ __align__(8) float sums[SEGS][DK];
   __shared__ __align__(8) uint64_t done;
   __shared__ uint32_t tmem_base_smem;
   __shared__ int abort_flag;
@@ -1163,40 +1163,51 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_state_kernel(c
   const long long ch = (long long)c * p.H + h;
   const __nv_bfloat16* rows = p.proj + (long long)row0 * p.ld;
   chunk_load<DK>(v_s, rows + p.v_col + h * p.VP, p.ld, n);
-  const int col = tid % DK, seg = tid / DK, t0 = seg * SEG;
-  float* z = p.z + (long long)row0 * p.ldz + h * p.KP + col;
-  const __nv_bfloat16* k = rows + p.k_col + h * p.KP + col;
-  const float w0 = p.w0[h * p.KP + col];
-  float A[SEG], run = 0.f;
+  const int col = 2 * (tid % (DK / 2)), seg = tid / (DK / 2), t0 = seg * SEG;
+  float* z = p.z + (long long)(row0 + t0) * p.ldz + h * p.KP + col;
+  const __nv_bfloat16* k = rows + (long long)t0 * p.ld + p.k_col + h * p.KP + col;
+  // exp(z + w0) log2(e) as one power of two
+  const float w0 = fmaf(p.w0[h * p.KP + col], LOG2E, 0.52876637f), w1 = fmaf(p.w0[h * p.KP + col + 1], LOG2E, 0.52876637f);
+  float2 A[SEG];
+  uint32_t keys[SEG];                                   // (fetched before anything is stored: the stores could alias)
+  const int mine = min(SEG, n - t0);
 #pragma unroll
-  for (int i = 0; i < SEG; ++i) A[i] = t0 + i < n ? z[(long long)(t0 + i) * p.ldz] : 0.f;
+  for (int i = 0; i < SEG; ++i) A[i] = i < mine ? *reinterpret_cast<const float2*>(z + (long long)i * p.ldz) : make_float2(0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < SEG; ++i) keys[i] = i < mine ? *reinterpret_cast<const uint32_t*>(k + (long long)i * p.ld) : 0u;
+  float2 run = make_float2(0.f, 0.f);
 #pragma unroll
   for (int i = 0; i < SEG; ++i) {
-    if (t0 + i < n) run -= fminf(expf(A[i] + w0) * LOG2E, MIX_MOST);
+    if (i < mine) {
+      run.x -= fminf(chunk_exp2(fmaf(A[i].x, LOG2E, w0)), MIX_MOST);
+      run.y -= fminf(chunk_exp2(fmaf(A[i].y, LOG2E, w1)), MIX_MOST);
+    }
     A[i] = run;
   }
-  sums[seg][col] = run;
+  sums[seg][col] = run.x;
+  sums[seg][col + 1] = run.y;
   __syncthreads();
-  float before = 0.f, total = 0.f;
+  float2 before = make_float2(0.f, 0.f), total = before;
 #pragma unroll
   for (int i = 0; i < SEGS; ++i) {
-    if (i < seg) before += sums[i][col];
-    total += sums[i][col];
+    const float2 x = *reinterpret_cast<const float2*>(&sums[i][col]);
+    if (i < seg) { before.x += x.x; before.y += x.y; }
+    total.x += x.x;
+    total.y += x.y;
   }
-  if (seg == 0) p.last[ch * p.KP + col] = total;
+  if (seg == 0) *reinterpret_cast<float2*>(p.last + ch * p.KP + col) = total;
 #pragma unroll
   for (int i = 0; i < SEG; ++i) {
-    const int t = t0 + i;
-    float x = 0.f;
-    if (t < n) {
-      A[i] += before;
-      z[(long long)t * p.ldz] = A[i];
-      x = __bfloat162float(k[(long long)t * p.ld]) * chunk_exp2(total - A[i]);
-    }
-    const __nv_bfloat16 a = __float2bfloat16_rn(x);
-    const uint32_t at = (col >> 6) * CH_CHUNK + chunk_addr(t, (col & 63) >> 3) + (col & 7) * 2;
-    *reinterpret_cast<__nv_bfloat16*>(hi + at) = a;
-    *reinterpret_cast<__nv_bfloat16*>(lo + at) = __float2bfloat16_rn(x - __bfloat162float(a));
+    A[i].x += before.x;
+    A[i].y += before.y;
+    if (i < mine) *reinterpret_cast<float2*>(z + (long long)i * p.ldz) = A[i];
+    const float2 f = unpack_bf16x2(keys[i]);
+    const float x = f.x * chunk_exp2(total.x - A[i].x), y = f.y * chunk_exp2(total.y - A[i].y);
+    const uint32_t high = pack_bf16x2(x, y);
+    const float2 back = unpack_bf16x2(high);
+    const uint32_t at = (col >> 6) * CH_CHUNK + chunk_addr(t0 + i, (col & 63) >> 3) + (col & 7) * 2;
+    *reinterpret_cast<uint32_t*>(hi + at) = high;
+    *reinterpret_cast<uint32_t*>(lo + at) = pack_bf16x2(x - back.x, y - back.y);
   }
   cp_async_wait_all();
   fence_proxy_async_smem();
@@ -1347,15 +1358,11 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
       cp_async16(a_s + t * DK * 4 + ((((q4 >> 1) ^ (t & 7)) << 5) | ((q4 & 1) << 4)), A + (long long)(t < n ? t : 0) * p.ldz + q4 * 4, t < n);
     }
   }
-  cp_async_wait_all();
-  __syncthreads();
-  auto a2 = [&](int t, int cc) {                                   // A of channels cc, cc + 1 (cc even); zero in front of the chunk
-    return t < 0 ? make_float2(0.f, 0.f)
-                 : *reinterpret_cast<const float2*>(a_p + t * DK * 4 + ((((cc >> 3) ^ (t & 7)) << 5) | ((cc & 7) << 2)));
-  };
-  auto bf2 = [&](const uint8_t* tile, int t, int cc) {
-    return unpack_bf16x2(*reinterpret_cast<const uint32_t*>(tile + (cc >> 6) * CH_CHUNK + chunk_addr(t, (cc & 63) >> 3) + (cc & 7) * 2));
-  };
+  // Addresses: row t of A is at a_p + t * 4 DK, its 32-byte piece u (channels 8u ..) at ((u ^ (t & 7)) << 5); of a tile's chunk of 64
+  // channels row t is at + 128 t, its 16-byte piece u at ((u ^ (t & 7)) << 4). (Pieces beyond the eighth only have higher bits more.)
+  auto a_row = [&](int t) { return a_p + t * (DK * 4); };
+  auto a_piece = [&](int t, int u) { return (u ^ (t & 7)) << 5; };
+  auto b_piece = [&](int t, int u) { return (u >> 3) * CH_CHUNK + (((u & 7) ^ (t & 7)) << 4); };
   auto weight_at = [&](int t, int j) { return w_p + (j >> 6) * CH_CHUNK + chunk_addr(t, (j & 63) >> 3) + (j & 7) * 2; };
   const int g = lane >> 2, cq = 2 * (lane & 3), t0 = warp * 16;    // this warp's block row of P
 #pragma unroll
@@ -1363,78 +1370,127 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
     const int e = lane + i * 32, t = t0 + (e >> 4), u = e & 15;
     *reinterpret_cast<uint4*>(w_p + (u >> 3) * CH_CHUNK + chunk_addr(t, u & 7)) = make_uint4(0u, 0u, 0u, 0u);
   }
-  __syncwarp();
-  // r_t 2^(A_(t-1) - A_ref) and k_j 2^(A_ref - A_j) of channels cc, cc + 1
-  auto scaled_r = [&](int t, int cc, float2 ref) {
-    const float2 x = bf2(r_p, t, cc), a = a2(t - 1, cc);
+  cp_async_wait_all();
+  __syncthreads();
+  auto two_a = [&](int t, int u) {                                 // A of channels 8u + cq, 8u + cq + 1; zero in front of the chunk
+    return t < 0 ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(a_row(t) + a_piece(t, u) + cq * 4);
+  };
+  // r_t 2^(A_(t-1) - A_ref) and k_j 2^(A_ref - A_j) of those channels
+  auto scaled_r = [&](int t, int u, float2 ref) {
+    const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_p + t * CH_ROWB + b_piece(t, u) + cq * 2)), a = two_a(t - 1, u);
     return pack_bf16x2(x.x * chunk_exp2(a.x - ref.x), x.y * chunk_exp2(a.y - ref.y));
   };
-  auto scaled_k = [&](int j, int cc, float2 ref) {
-    const float2 x = bf2(k_p, j, cc), a = a2(j, cc);
+  auto scaled_k = [&](const uint8_t* k_row, const uint8_t* arow, int kb, int ab, float2 ref) {
+    const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_row + kb)), a = *reinterpret_cast<const float2*>(arow + ab);
     return pack_bf16x2(x.x * chunk_exp2(ref.x - a.x), x.y * chunk_exp2(ref.y - a.y));
   };
-  if (t0 < n) {
-    if (warp > 0) {                                                // the blocks left of the diagonal
+  // The blocks left of the diagonal, 8 columns at a time: rows w and 7 - w have 14 such pieces together, half of them for either warp.
+  {
+    int kb[DK / 8], ab[DK / 8];                                    // pieces of a row j with j % 8 == g
+#pragma unroll
+    for (int u = 0; u < DK / 8; ++u) { kb[u] = b_piece(g, u); ab[u] = a_piece(g, u); }
+    const uint8_t* k0 = k_p + g * CH_ROWB + cq * 2;
+    const uint8_t* a0 = a_row(g) + cq * 4;
+    auto blocks = [&](int b0, int from, int to) {                  // block row at token b0, columns 8 from .. 8 to
+      if (b0 >= n || from >= to) return;
       uint32_t fa[DK / 16][4];
+      float2 ref[DK / 8];
 #pragma unroll
-      for (int ks = 0; ks < DK / 16; ++ks) {
-        const int cc = ks * 16 + cq;
-        const float2 ref0 = a2(t0 - 1, cc), ref1 = a2(t0 - 1, cc + 8);
-        fa[ks][0] = scaled_r(t0 + g, cc, ref0);
-        fa[ks][1] = scaled_r(t0 + g + 8, cc, ref0);
-        fa[ks][2] = scaled_r(t0 + g, cc + 8, ref1);
-        fa[ks][3] = scaled_r(t0 + g + 8, cc + 8, ref1);
+      for (int u = 0; u < DK / 8; ++u) {
+        ref[u] = two_a(b0 - 1, u);
+        fa[u / 2][(u & 1) * 2] = scaled_r(b0 + g, u, ref[u]);
+        fa[u / 2][(u & 1) * 2 + 1] = scaled_r(b0 + g + 8, u, ref[u]);
       }
-      for (int j0 = 0; j0 < t0; j0 += 8) {
+      for (int j0 = from * 8; j0 < to * 8; j0 += 8) {
         float s[4] = {0.f, 0.f, 0.f, 0.f};
+        const uint8_t* kr = k0 + j0 * CH_ROWB;
+        const uint8_t* ar = a0 + j0 * (DK * 4);
 #pragma unroll
-        for (int ks = 0; ks < DK / 16; ++ks) {
-          const int cc = ks * 16 + cq;
-          mma_16816_bf16(s, fa[ks][0], fa[ks][1], fa[ks][2], fa[ks][3], scaled_k(j0 + g, cc, a2(t0 - 1, cc)),
-                         scaled_k(j0 + g, cc + 8, a2(t0 - 1, cc + 8)));
-        }
-        *reinterpret_cast<uint32_t*>(weight_at(t0 + g, j0 + cq)) = pack_bf16x2(s[0], s[1]);
-        *reinterpret_cast<uint32_t*>(weight_at(t0 + g + 8, j0 + cq)) = pack_bf16x2(s[2], s[3]);
+        for (int ks = 0; ks < DK / 16; ++ks)
+          mma_16816_bf16(s, fa[ks][0], fa[ks][1], fa[ks][2], fa[ks][3], scaled_k(kr, ar, kb[2 * ks], ab[2 * ks], ref[2 * ks]),
+                         scaled_k(kr, ar, kb[2 * ks + 1], ab[2 * ks + 1], ref[2 * ks + 1]));
+        *reinterpret_cast<uint32_t*>(weight_at(b0 + g, j0 + cq)) = pack_bf16x2(s[0], s[1]);
+        *reinterpret_cast<uint32_t*>(weight_at(b0 + g + 8, j0 + cq)) = pack_bf16x2(s[2], s[3]);
       }
+    };
+#pragma unroll 1
+    for (int part = 0; part < 2; ++part) {
+      const int low = min(warp, 7 - warp), row = part == 0 ? 7 - low : low;        // the longer row of the pair first
+      if (part == 0) blocks(row * 16, warp == low ? 0 : 7 - 2 * low, warp == low ? 7 - 2 * low : 2 * row);
+      else if (warp == low) blocks(row * 16, 0, 2 * row);
     }
+  }
+  if (t0 < n) {
     {                                                              // lower left quarter of the diagonal block
       float s[4] = {0.f, 0.f, 0.f, 0.f};
+      const uint8_t* kr = k_p + (t0 + g) * CH_ROWB + cq * 2;
+      const uint8_t* ar = a_row(t0 + g) + cq * 4;
 #pragma unroll
       for (int ks = 0; ks < DK / 16; ++ks) {
-        const int cc = ks * 16 + cq;
-        const float2 ref0 = a2(t0 + 7, cc), ref1 = a2(t0 + 7, cc + 8);
-        mma_16816_bf16(s, scaled_r(t0 + 8 + g, cc, ref0), 0u, scaled_r(t0 + 8 + g, cc + 8, ref1), 0u, scaled_k(t0 + g, cc, ref0),
-                       scaled_k(t0 + g, cc + 8, ref1));
+        const float2 ref0 = two_a(t0 + 7, 2 * ks), ref1 = two_a(t0 + 7, 2 * ks + 1);
+        mma_16816_bf16(s, scaled_r(t0 + 8 + g, 2 * ks, ref0), 0u, scaled_r(t0 + 8 + g, 2 * ks + 1, ref1), 0u,
+                       scaled_k(kr, ar, b_piece(g, 2 * ks), a_piece(g, 2 * ks), ref0), scaled_k(kr, ar, b_piece(g, 2 * ks + 1), a_piece(g, 2 * ks + 1), ref1));
       }
       *reinterpret_cast<uint32_t*>(weight_at(t0 + 8 + g, t0 + cq)) = pack_bf16x2(s[0], s[1]);
     }
-    if (lane < 28) {                                               // pairs j < t of the two triangles, one per lane
-      int t = 1, j = lane;
-      while (j >= t) { j -= t; ++t; }
+    {                                                              // lower left quarters of the diagonal's two 8 x 8 blocks, in one product
+      const int up = g < 4 ? 0 : 4, t = t0 + 4 + g + up, j = t0 + g + up, ref_row = t0 + 3 + 2 * up;
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int tri = 0; tri < 2; ++tri) {
-        const int tt = t0 + tri * 8 + t, jj = t0 + tri * 8 + j;
-        float s = 0.f;
-#pragma unroll 4
-        for (int i = 0; i < DK / 2; ++i) {
-          const int cc = 2 * ((i + lane) & (DK / 2 - 1));
-          const float2 x = bf2(r_p, tt, cc), y = bf2(k_p, jj, cc), a = a2(tt - 1, cc), b = a2(jj, cc);
-          s = fmaf(x.x * y.x, chunk_exp2(a.x - b.x), s);
-          s = fmaf(x.y * y.y, chunk_exp2(a.y - b.y), s);
-        }
-        *reinterpret_cast<__nv_bfloat16*>(weight_at(tt, jj)) = __float2bfloat16_rn(s);
+      for (int ks = 0; ks < DK / 16; ++ks) {
+        const float2 ref0 = two_a(ref_row, 2 * ks), ref1 = two_a(ref_row, 2 * ks + 1);
+        const uint8_t* kr = k_p + j * CH_ROWB + cq * 2;
+        const uint8_t* ar = a_row(j) + cq * 4;
+        mma_16816_bf16(s, scaled_r(t, 2 * ks, ref0), 0u, scaled_r(t, 2 * ks + 1, ref1), 0u,
+                       scaled_k(kr, ar, b_piece(j, 2 * ks), a_piece(j, 2 * ks), ref0), scaled_k(kr, ar, b_piece(j, 2 * ks + 1), a_piece(j, 2 * ks + 1), ref1));
       }
+      if ((g >> 2) == (cq >> 2)) *reinterpret_cast<uint32_t*>(weight_at(t, t0 + cq + (cq < 4 ? 0 : 4))) = pack_bf16x2(s[0], s[1]);
+    }
+    if (lane < 24) {                                               // pairs j < t of the four 4 x 4 triangles, one per lane
+      const int q = lane % 6, t = q < 1 ? 1 : q < 3 ? 2 : 3, j = q - t * (t - 1) / 2;
+      const int tt = t0 + lane / 6 * 4 + t, jj = t0 + lane / 6 * 4 + j;
+      const uint8_t* rr = r_p + tt * CH_ROWB;
+      const uint8_t* kr = k_p + jj * CH_ROWB;
+      const uint8_t* at = a_row(tt - 1);
+      const uint8_t* aj = a_row(jj);
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll 2
+      for (int i = 0; i < DK / 8; ++i) {                           // eight channels at a time, every lane from a place of its own
+        const int u = (i + lane) & (DK / 8 - 1);
+        const uint4 x = *reinterpret_cast<const uint4*>(rr + b_piece(tt, u)), y = *reinterpret_cast<const uint4*>(kr + b_piece(jj, u));
+        const float4* pa = reinterpret_cast<const float4*>(at + a_piece(tt - 1, u));
+        const float4* pb = reinterpret_cast<const float4*>(aj + a_piece(jj, u));
+        const float4 a = pa[0], b = pb[0], c4 = pa[1], d4 = pb[1];
+        float2 f, h2;
+        f = unpack_bf16x2(x.x); h2 = unpack_bf16x2(y.x);
+        s0 = fmaf(f.x * h2.x, chunk_exp2(a.x - b.x), s0);
+        s1 = fmaf(f.y * h2.y, chunk_exp2(a.y - b.y), s1);
+        f = unpack_bf16x2(x.y); h2 = unpack_bf16x2(y.y);
+        s0 = fmaf(f.x * h2.x, chunk_exp2(a.z - b.z), s0);
+        s1 = fmaf(f.y * h2.y, chunk_exp2(a.w - b.w), s1);
+        f = unpack_bf16x2(x.z); h2 = unpack_bf16x2(y.z);
+        s0 = fmaf(f.x * h2.x, chunk_exp2(c4.x - d4.x), s0);
+        s1 = fmaf(f.y * h2.y, chunk_exp2(c4.y - d4.y), s1);
+        f = unpack_bf16x2(x.w); h2 = unpack_bf16x2(y.w);
+        s0 = fmaf(f.x * h2.x, chunk_exp2(c4.z - d4.z), s0);
+        s1 = fmaf(f.y * h2.y, chunk_exp2(c4.w - d4.w), s1);
+      }
+      *reinterpret_cast<__nv_bfloat16*>(weight_at(tt, jj)) = __float2bfloat16_rn(s0 + s1);
     }
     {                                                              // the diagonal: two lanes per token
       const int t = t0 + (lane & 15);
       const float* bonus = p.bonus + h * p.KP;
       float s = 0.f;
-#pragma unroll 4
-      for (int i = 0; i < DK / 4; ++i) {
-        const int cc = (lane >> 4) * (DK / 2) + 2 * i;
-        const float2 x = bf2(r_p, t, cc), y = bf2(k_p, t, cc), u = *reinterpret_cast<const float2*>(bonus + cc);
-        s = fmaf(x.x * y.x, u.x, s);
-        s = fmaf(x.y * y.y, u.y, s);
+#pragma unroll 2
+      for (int i = 0; i < DK / 16; ++i) {
+        const int u = (lane >> 4) * (DK / 16) + i;
+        const uint4 x = *reinterpret_cast<const uint4*>(r_p + t * CH_ROWB + b_piece(t, u)), y = *reinterpret_cast<const uint4*>(k_p + t * CH_ROWB + b_piece(t, u));
+        const float4 b0 = *reinterpret_cast<const float4*>(bonus + u * 8), b1 = *reinterpret_cast<const float4*>(bonus + u * 8 + 4);
+        float2 f, h2;
+        f = unpack_bf16x2(x.x); h2 = unpack_bf16x2(y.x); s = fmaf(f.x * h2.x, b0.x, fmaf(f.y * h2.y, b0.y, s));
+        f = unpack_bf16x2(x.y); h2 = unpack_bf16x2(y.y); s = fmaf(f.x * h2.x, b0.z, fmaf(f.y * h2.y, b0.w, s));
+        f = unpack_bf16x2(x.z); h2 = unpack_bf16x2(y.z); s = fmaf(f.x * h2.x, b1.x, fmaf(f.y * h2.y, b1.y, s));
+        f = unpack_bf16x2(x.w); h2 = unpack_bf16x2(y.w); s = fmaf(f.x * h2.x, b1.z, fmaf(f.y * h2.y, b1.w, s));
       }
       s += __shfl_xor_sync(0xffffffffu, s, 16);
       if (lane < 16) *reinterpret_cast<__nv_bfloat16*>(weight_at(t, t)) = __float2bfloat16_rn(s);
@@ -1445,13 +1501,17 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
 #pragma unroll 2
   for (int i = tid; i < CH * (DK / 8); i += CHT) {                 // r 2^A_(t-1), in place
     const int t = i / (DK / 8), u = i % (DK / 8);
-    uint4* at = reinterpret_cast<uint4*>(r_p + (u >> 3) * CH_CHUNK + chunk_addr(t, u & 7));
-    const uint4 v = *at;
-    auto one = [&](uint32_t x, int cc) {
-      const float2 f = unpack_bf16x2(x), a = a2(t - 1, cc);
-      return pack_bf16x2(f.x * chunk_exp2(a.x), f.y * chunk_exp2(a.y));
+    if (t == 0) continue;
+    uint4* at = reinterpret_cast<uint4*>(r_p + t * CH_ROWB + b_piece(t, u));
+    const float4* pa = reinterpret_cast<const float4*>(a_row(t - 1) + a_piece(t - 1, u));
+    const float4 a = pa[0], b = pa[1];
+    uint4 v = *at;
+    auto one = [&](uint32_t x, float ax, float ay) {
+      const float2 f = unpack_bf16x2(x);
+      return pack_bf16x2(f.x * chunk_exp2(ax), f.y * chunk_exp2(ay));
     };
-    *at = make_uint4(one(v.x, u * 8), one(v.y, u * 8 + 2), one(v.z, u * 8 + 4), one(v.w, u * 8 + 6));
+    v.x = one(v.x, a.x, a.y); v.y = one(v.y, a.z, a.w); v.z = one(v.z, b.x, b.y); v.w = one(v.w, b.z, b.w);
+    *at = v;
   }
   __syncthreads();                                                 // A has been read
   constexpr int PART = DK * DK * 2;                                // one part of the state
@@ -1521,7 +1581,7 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
       const float4 w0 = *reinterpret_cast<const float4*>(w + i * 8), w1 = *reinterpret_cast<const float4*>(w + i * 8 + 4);
       auto two = [&](int e, float wx, float wy, uint32_t gz) {
         const float2 z = unpack_bf16x2(gz);
-        return pack_bf16x2(__uint_as_float(v[i * 8 + e]) * rs * wx * z.x * sigmoid_f(z.x), __uint_as_float(v[i * 8 + e + 1]) * rs * wy * z.y * sigmoid_f(z.y));
+        return pack_bf16x2(__uint_as_float(v[i * 8 + e]) * rs * wx * silu_fast(z.x), __uint_as_float(v[i * 8 + e + 1]) * rs * wy * silu_fast(z.y));
       };
       *reinterpret_cast<uint4*>(dst + i * 8) = make_uint4(two(0, w0.x, w0.y, gate[i].x), two(2, w0.z, w0.w, gate[i].y), two(4, w1.x, w1.y, gate[i].z),
                                                           two(6, w1.z, w1.w, gate[i].w));
