@@ -16,9 +16,9 @@ append, SwiGLU and sampling are the kernels in csrc/attn_sm100.cu and csrc/ops_s
 
 from __future__ import annotations
 
-import os
-
+import gc
 import math
+import os
 from dataclasses import dataclass
 
 import torch
@@ -161,19 +161,27 @@ class RunnerBase:
         self.d_state_slots.fill_(-1)
         torch.cuda.synchronize(self.device)
         stream = torch.cuda.Stream(self.device)
+        # an abandoned engine's graphs, destroyed by the collector while this one captures, would break the capture
+        gc.collect()
+        collecting = gc.isenabled()
+        gc.disable()
         ops.set_pdl(True)  # decode kernels overlap their prologue with the previous kernel's tail
-        with torch.cuda.stream(stream):
-            for bk in sorted(self.graph_batch_sizes, reverse=True):
-                self._decode_body(bk)  # warm-up: sets kernel attributes outside capture
-                stream.synchronize()
-                g = torch.cuda.CUDAGraph()
-                n0 = LAUNCH_COUNT[0]
-                with torch.cuda.graph(g, pool=self.graph_pool, stream=stream):
-                    self._decode_body(bk)
-                self.launches_per_graph[bk] = LAUNCH_COUNT[0] - n0
-                if self.graph_pool is None:
-                    self.graph_pool = g.pool()
-                self.graphs[bk] = g
+        try:
+            with torch.cuda.stream(stream):
+                for bk in sorted(self.graph_batch_sizes, reverse=True):
+                    self._decode_body(bk)  # warm-up: sets kernel attributes outside capture
+                    stream.synchronize()
+                    g = torch.cuda.CUDAGraph()
+                    n0 = LAUNCH_COUNT[0]
+                    with torch.cuda.graph(g, pool=self.graph_pool, stream=stream):
+                        self._decode_body(bk)
+                    self.launches_per_graph[bk] = LAUNCH_COUNT[0] - n0
+                    if self.graph_pool is None:
+                        self.graph_pool = g.pool()
+                    self.graphs[bk] = g
+        finally:
+            if collecting:
+                gc.enable()
         ops.set_pdl(False)
         torch.cuda.synchronize(self.device)
         ops.check_status(self.device)
