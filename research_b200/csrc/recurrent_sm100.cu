@@ -1,7 +1,7 @@
 // Recurrent mixers with a matrix state per head, for sm_100a.
 //
 //   S_t = a_t S_(t-1) + b_t k_t v_t^T,   o_t = S_t^T q_t        (see ops/recurrent.py)
-//   S_t = diag(w_t) S_(t-1) + k_t v_t^T, o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t        (time mixing: a decay per key channel)
+//   o_t = S_(t-1)^T q_t + (sum_c u_c q_tc k_tc) v_t,  then row c of S decays by its own w_tc and takes k_tc v_t        (time mixing)
 //
 //   scan        token by token: short portions and long ones of the exact mode. One CTA per (sequence, head, 32 value channels);
 //               the state tile stays in registers over the tokens of the portion.

@@ -28,12 +28,11 @@ def linear(x, w, name):
 
 
 def causal_conv(u, taps):
-    """y_t = sum_j taps[:, j] u_(t - n + 1 + j), nothing before the first token."""
-    n, y = taps.shape[1], torch.zeros_like(u)
-    for j in range(n):
-        back = n - 1 - j
-        if back < len(u):
-            y[back:] += taps[:, j] * u[:len(u) - back]
+    """Every channel: the value d tokens back weighs with the d-th tap from the end; nothing lies before the first token."""
+    y = torch.zeros_like(u)
+    for d, tap in enumerate(taps.flip(1).T):
+        if d < len(u):
+            y[d:] += tap * u[:len(u) - d]
     return y
 
 
@@ -162,7 +161,7 @@ def channel_decay(m, w, name):
 
 
 def time_mix_scan(r, k, v, decay, u):
-    """o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t, S_t = diag(decay_t) S_(t-1) + k_t v_t^T;  r, k, decay [t, h, d], v [t, h, e]."""
+    """A matrix per head, read before the token is written into it, the token itself through the bonus;  r, k, decay [t, h, d], v [t, h, e]."""
     S, out = k.new_zeros(k.shape[1], k.shape[2], v.shape[2]), []
     for i in range(len(r)):
         kv = k[i][:, :, None] * v[i][:, None, :]
