@@ -1172,6 +1172,7 @@ struct GroupedAppend {
   const int* slots;        // [T] places in the cache, negative: not stored
   const float* q_norm;     // [H * dim], projection norm
   const float* k_norm;     // [G * dim]
+  const float* q_factor;   // [H] of the queries, or null
   int norm;
   float eps;
   const float* table;      // [positions, half, 2] cos, sin
@@ -1391,6 +1392,7 @@ __global__ void __launch_bounds__(GA_THREADS, 4) grouped_append_kernel(const Gro
       }
       float f = 1.f;
       if (p.norm == GA_NORM_HEAD) f = 1.f / sqrtf(warp_sum(ss) / (float)dim + p.eps);
+      if (!is_k && p.q_factor != nullptr) f *= p.q_factor[head];
 #pragma unroll
       for (int j = 0; j < STEPS; ++j) {
         const int e = lane + j * 32;
@@ -1450,7 +1452,7 @@ constexpr int kv_decode_smem_bytes() {
 
 struct GroupedAppendArgs {       // mirrored by ops/grouped.py
   const void* proj; const float* conv; void* hist; const int* cu_q; const int* positions; const int* state_slots; const int* slots;
-  const float* q_norm; const float* k_norm; const float* table; void* q; void* keys; void* values; int* status;
+  const float* q_norm; const float* k_norm; const float* q_factor; const float* table; void* q; void* keys; void* values; int* status;
   long long ld;
   int k_col, v_col, channels, taps, B, num_state_slots, norm, half, interleaved, max_pos, num_blocks, H, G, dim, vdim, DP, T, dtype;
   float eps;
@@ -1467,7 +1469,7 @@ extern "C" int rb_grouped_append(const GroupedAppendArgs* a, cudaStream_t stream
   p.proj = a->proj; p.ld = a->ld; p.k_col = a->k_col; p.v_col = a->v_col; p.channels = a->channels;
   p.conv = a->conv; p.taps = a->taps; p.hist = a->hist;
   p.rows = History{a->cu_q, a->positions, a->state_slots, a->B, a->taps - 1, a->num_state_slots};
-  p.slots = a->slots; p.q_norm = a->q_norm; p.k_norm = a->k_norm; p.norm = a->norm; p.eps = a->eps;
+  p.slots = a->slots; p.q_norm = a->q_norm; p.k_norm = a->k_norm; p.q_factor = a->q_factor; p.norm = a->norm; p.eps = a->eps;
   p.table = a->table; p.half = a->half; p.interleaved = a->interleaved; p.max_pos = a->max_pos;
   p.q = a->q; p.keys = a->keys; p.values = a->values; p.num_blocks = a->num_blocks;
   p.H = a->H; p.G = a->G; p.dim = a->dim; p.vdim = a->vdim; p.DP = a->DP; p.T = a->T; p.status = a->status;

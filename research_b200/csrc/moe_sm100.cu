@@ -26,18 +26,19 @@ constexpr int MAX_E_PER_LANE = 8;  // up to 256 experts
 
 // n_group > 1 (sigmoid router only): group-limited routing. Experts form n_group contiguous groups, a group scores
 // the sum of its two best choice values, the topk_group best groups stay eligible and the choice values of the
-// other experts become 0 (glm4_moe_functional.py:278-301).
+// other experts become 0 (glm4_moe_functional.py:278-301). The histogram has the first `counted` choices alone (the others are no
+// experts and get no rows).
 __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld, const float* __restrict__ bias, int T, int E,
                                  int k, int sigmoid_router, int norm_topk, float scaling, int* __restrict__ topk_idx,
                                  float* __restrict__ topk_w, int* __restrict__ counts /*[E] histogram, may be null*/,
-                                 int n_group, int topk_group) {
+                                 int n_group, int topk_group, int counted) {
   __shared__ int hist[256];
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (counts != nullptr) {
-    for (int i = threadIdx.x; i < E; i += blockDim.x) hist[i] = 0;
+    for (int i = threadIdx.x; i < counted; i += blockDim.x) hist[i] = 0;
     __syncthreads();
   }
   if (t < T) {
@@ -106,7 +107,8 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
     sum = warp_sum(sum);
     for (int i = 0; i < per; ++i) {
       score[i] /= sum;
-      choice[i] = (lane + 32 * i) < E ? score[i] : -INFINITY;
+      const int e = lane + 32 * i;
+      choice[i] = e < E ? score[i] + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
     }
   }
   float wsum = 0.f;
@@ -141,12 +143,12 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
     if (norm_topk) w = w / (wsum + 1e-20f);
     topk_idx[(long long)t * k + lane] = my_e;
     topk_w[(long long)t * k + lane] = w * scaling;
-    if (counts != nullptr) atomicAdd(&hist[my_e], 1);
+    if (counts != nullptr && my_e < counted) atomicAdd(&hist[my_e], 1);
   }
   }
   if (counts != nullptr) {   // integer adds: the histogram does not depend on their order
     __syncthreads();
-    for (int i = threadIdx.x; i < E; i += blockDim.x)
+    for (int i = threadIdx.x; i < counted; i += blockDim.x)
       if (hist[i]) atomicAdd(&counts[i], hist[i]);
   }
 }
@@ -242,9 +244,9 @@ __global__ void moe_count_kernel(const int* __restrict__ topk_idx, int n, int E,
 
 // Local dispatch: row (t, j) of any 16-byte-multiple width to the next free row of its expert's block (cursor as left by the
 // plan), and the address its result goes to. One warp per pair. With weights (act: 0 bf16, 1 fp32) the row is multiplied by the
-// pair's weight on the way.
+// pair's weight on the way. Choices E .. choices - 1 are no experts: they get no row.
 __global__ void moe_gather_rows_kernel(const uint4* __restrict__ x, long long ld_vec, const int* __restrict__ topk_idx, int n_pairs, int k,
-                                       int row_vec, int E, int* __restrict__ cursor, uint4* __restrict__ xp,
+                                       int row_vec, int E, int choices, int* __restrict__ cursor, uint4* __restrict__ xp,
                                        unsigned long long* __restrict__ ret, unsigned long long y, long long y_row_bytes, int cap,
                                        const float* __restrict__ weights, int act, int* status) {
   pdl_launch_dependents();
@@ -253,7 +255,8 @@ __global__ void moe_gather_rows_kernel(const uint4* __restrict__ x, long long ld
   const int i = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (i >= n_pairs) return;
   const int e = topk_idx[i];
-  if (e < 0 || e >= E) { set_status(status, ST_BAD_INDEX); return; }
+  if (e < 0 || e >= choices) { set_status(status, ST_BAD_INDEX); return; }
+  if (e >= E) return;
   int pos = 0;
   if (lane == 0) pos = cursor[E + e] + atomicAdd(&cursor[e], 1);
   pos = __shfl_sync(0xffffffffu, pos, 0);
@@ -581,7 +584,7 @@ extern "C" int rb_moe_route(const float* logits, const float* bias, int T, int E
                             int norm_topk, float scaling, int* topk_idx, float* topk_w, cudaStream_t s) {
   if (T <= 0) return 0;
   if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E) return -1;
-  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, E, bias, T, E, k, sigmoid_router, norm_topk, scaling, topk_idx, topk_w, nullptr, 1, 1);
+  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, E, bias, T, E, k, sigmoid_router, norm_topk, scaling, topk_idx, topk_w, nullptr, 1, 1, E);
   return RB_OK();
 }
 // Routing plus the per-expert histogram of the choices (added into counts[E], which the caller zeroes).
@@ -589,7 +592,7 @@ extern "C" int rb_moe_route_count(const float* logits, const float* bias, int T,
                                   int norm_topk, float scaling, int* topk_idx, float* topk_w, int* counts, cudaStream_t s) {
   if (T <= 0) return 0;
   if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E || counts == nullptr) return -1;
-  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, E, bias, T, E, k, sigmoid_router, norm_topk, scaling, topk_idx, topk_w, counts, 1, 1);
+  moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, E, bias, T, E, k, sigmoid_router, norm_topk, scaling, topk_idx, topk_w, counts, 1, 1, E);
   return RB_OK();
 }
 // The same with group-limited routing (n_group groups of E / n_group >= 2 experts, topk_group of them eligible).
@@ -601,7 +604,7 @@ extern "C" int rb_moe_route_groups(const float* logits, const float* bias, int T
   if (n_group < 1 || n_group > 32 || topk_group < 1 || topk_group > n_group || E % n_group != 0) return -1;
   if (n_group > 1 && E / n_group < 2) return -1;
   moe_route_kernel<<<(T + 7) / 8, 256, 0, s>>>(logits, E, bias, T, E, k, 1, norm_topk, scaling, topk_idx, topk_w, counts, n_group,
-                                               topk_group);
+                                               topk_group, E);
   return RB_OK();
 }
 extern "C" int rb_moe_count(const int* topk_idx, int n, int E, int* counts, cudaStream_t s) {
@@ -678,14 +681,14 @@ extern "C" int rb_moe_combine(const void* y, const float* w, int T, int k, int d
 // ---------------------------------------------------------------- local expert layer of layer-stack models (ops/experts.py)
 extern "C" void rb_moe_set_pdl(int on) { rb::pdl_enabled() = on != 0; }
 
-// Router on logits with a row stride: softmax or sigmoid scores, the chosen ones divided by their sum or not; histogram added
-// into counts.
-extern "C" int rb_experts_route(const float* logits, long long ld, int T, int E, int k, int sigmoid, int normalize, int* topk_idx, float* topk_w,
-                                int* counts, cudaStream_t s) {
+// Router on logits with a row stride: softmax or sigmoid scores of E choices, the best by score plus `correction` (may be null) chosen,
+// the chosen scores divided by their sum or not; histogram of the first `experts` choices added into counts.
+extern "C" int rb_experts_route(const float* logits, long long ld, const float* correction, int T, int E, int experts, int k, int sigmoid, int normalize,
+                                int* topk_idx, float* topk_w, int* counts, cudaStream_t s) {
   if (T <= 0) return 0;
-  if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E || counts == nullptr) return -1;
-  return launch_kernel(moe_route_kernel, dim3((T + 7) / 8), dim3(256), 0, s, logits, ld, nullptr, T, E, k, sigmoid, normalize, 1.f, topk_idx, topk_w, counts,
-                       1, 1) == cudaSuccess ? 0 : -11;
+  if (E > 32 * MAX_E_PER_LANE || k > 32 || k > E || counts == nullptr || experts <= 0 || experts > E) return -1;
+  return launch_kernel(moe_route_kernel, dim3((T + 7) / 8), dim3(256), 0, s, logits, ld, correction, T, E, k, sigmoid, normalize, 1.f, topk_idx, topk_w, counts,
+                       1, 1, experts) == cudaSuccess ? 0 : -11;
 }
 // Offsets, tile tables and dispatch bases from the histogram, which is zeroed again.
 extern "C" int rb_experts_plan(int* counts, int E, int* expert_offset, int n_gu, int bn_gu, void* tiles_gu, int* ntiles_gu, int n_dn, int bn_dn,
@@ -694,13 +697,13 @@ extern "C" int rb_experts_plan(int* counts, int E, int* expert_offset, int n_gu,
   return launch_kernel(moe_plan_kernel, dim3(1), dim3(256), 0, s, counts, 1, E, 0, E, expert_offset, n_gu, bn_gu, (int4*)tiles_gu, ntiles_gu,
                        n_dn, bn_dn, (int4*)tiles_dn, ntiles_dn, max_tiles, status, 0, cursor, counts) == cudaSuccess ? 0 : -11;
 }
-extern "C" int rb_experts_gather(const void* x, long long ld_bytes, const int* topk_idx, int T, int k, int row_bytes, int E, int* cursor, void* xp,
-                                 void* ret, void* y, long long y_row_bytes, int cap, const float* weights, int act, int* status, cudaStream_t s) {
+extern "C" int rb_experts_gather(const void* x, long long ld_bytes, const int* topk_idx, int T, int k, int row_bytes, int E, int choices, int* cursor,
+                                 void* xp, void* ret, void* y, long long y_row_bytes, int cap, const float* weights, int act, int* status, cudaStream_t s) {
   if (T <= 0) return 0;
   if (ld_bytes % 16 != 0 || row_bytes % 16 != 0) return -1;
   const int n = T * k;
   return launch_kernel(moe_gather_rows_kernel, dim3((n + 7) / 8), dim3(256), 0, s, (const uint4*)x, ld_bytes / 16, topk_idx, n, k, row_bytes / 16, E,
-                       cursor, (uint4*)xp, (unsigned long long*)ret, (unsigned long long)y, y_row_bytes, cap, weights, act, status) == cudaSuccess ? 0 : -11;
+                       choices, cursor, (uint4*)xp, (unsigned long long*)ret, (unsigned long long)y, y_row_bytes, cap, weights, act, status) == cudaSuccess ? 0 : -11;
 }
 
 // ---------------------------------------------------------------- training (expert-grouped rows, padded to 64)

@@ -394,6 +394,170 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamNormParams
   }
 }
 
+// One pass over the fp32 residual stream around a sublayer with a norm before and after it, a CTA per row:
+//   v = y                                                    one output, or
+//   v = pair_scale * (y / rms(y) * w + y2 / rms(y2) * w2)    two mixers side by side, or
+//   v = sigmoid(gate) y + sum_j p[j] e[row * k + j]          a shared expert (its gate may be null) and the routed ones; choices from `experts`
+//                                                            on have no row: their weight goes to `pass`, the sublayer's own input
+//   x += N_post(v), copy = x, h = N_pre(x) in the activation type
+// with N(z) = z / rms(z) * weight, or tanh(alpha z) * weight + bias (BOUNDED). Any of y, h and copy may be null; rows != null: h[i]
+// comes from row rows[i] (no update). Columns are padded to a multiple of 4 with zeros (weights and biases there are zero too).
+struct SandwichNorm { const float* weight; const float* bias; const float* alpha; };
+struct SandwichParams {
+  float* x; long long ldx;
+  const float* y; const float* y2; long long ldy;
+  const float* w; const float* w2;
+  float pair_scale;
+  const float* gate; long long ld_gate;
+  const void* e; long long lde;
+  const float* p; const int* idx; int k, experts;
+  const void* pass; long long ld_pass;
+  SandwichNorm post, pre;
+  void* copy; long long ldc;
+  void* h; long long ldh;
+  const int* rows; int num_src_rows;
+  int d, dp; float eps;
+  int* status;
+};
+
+template <typename TA, bool BOUNDED>
+__global__ void __launch_bounds__(256) stream_sandwich_kernel(const SandwichParams p) {
+  extern __shared__ float4 sw_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long r = blockIdx.x;
+  long long xr = r;
+  if (p.rows != nullptr) {
+    xr = p.rows[r];
+    if (xr < 0 || xr >= p.num_src_rows) { if (threadIdx.x == 0) set_status(p.status, ST_BAD_INDEX); xr = 0; }
+  }
+  float* x = p.x + xr * p.ldx;
+  const float* y = p.y + r * p.ldy;
+  const float* y2 = p.y2 + r * p.ldy;
+  const bool update = p.y != nullptr || p.e != nullptr;
+  auto at4 = [](const float* q, int c) { return *reinterpret_cast<const float4*>(q + c); };
+  auto square = [](float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; };
+  const int step = blockDim.x * 4;
+  float s1 = 1.f, s2 = 0.f;
+  if (p.y2 != nullptr) {
+    float a = 0.f, b = 0.f;
+    for (int c = threadIdx.x * 4; c < p.dp; c += step) { a += square(at4(y, c)); b += square(at4(y2, c)); }
+    s1 = p.pair_scale / sqrtf(block_sum(a, red) / (float)p.d + p.eps);
+    s2 = p.pair_scale / sqrtf(block_sum(b, red) / (float)p.d + p.eps);
+  }
+  if (p.gate != nullptr) s1 = 1.f / (1.f + expf(-p.gate[r * p.ld_gate]));
+  float through = 0.f;
+  if (p.e != nullptr)
+    for (int j = 0; j < p.k; ++j)
+      if (p.idx[r * p.k + j] >= p.experts) through += p.p[r * p.k + j];
+  const TA* e = reinterpret_cast<const TA*>(p.e) + r * p.k * p.lde;
+  const TA* pass = reinterpret_cast<const TA*>(p.pass) + r * p.ld_pass;
+  auto sublayer = [&](int c) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (p.y2 != nullptr) {
+      const float4 a = at4(y, c), b = at4(y2, c), wa = at4(p.w, c), wb = at4(p.w2, c);
+      return make_float4(a.x * s1 * wa.x + b.x * s2 * wb.x, a.y * s1 * wa.y + b.y * s2 * wb.y, a.z * s1 * wa.z + b.z * s2 * wb.z,
+                         a.w * s1 * wa.w + b.w * s2 * wb.w);
+    }
+    if (p.y != nullptr) {
+      const float4 a = at4(y, c);
+      v = make_float4(s1 * a.x, s1 * a.y, s1 * a.z, s1 * a.w);
+    }
+    if (p.e != nullptr) {
+      for (int j = 0; j < p.k; ++j) {
+        if (__ldg(p.idx + r * p.k + j) >= p.experts) continue;
+        const float w = __ldg(p.p + r * p.k + j);
+        const float4 a = load_act4(e + j * p.lde + c);
+        v.x = fmaf(w, a.x, v.x); v.y = fmaf(w, a.y, v.y); v.z = fmaf(w, a.z, v.z); v.w = fmaf(w, a.w, v.w);
+      }
+      if (through != 0.f) {
+        const float4 a = load_act4(pass + c);
+        v.x = fmaf(through, a.x, v.x); v.y = fmaf(through, a.y, v.y); v.z = fmaf(through, a.z, v.z); v.w = fmaf(through, a.w, v.w);
+      }
+    }
+    return v;
+  };
+  auto bounded = [&](const SandwichNorm& n, float alpha, float4 v, int c) {
+    const float4 w = at4(n.weight, c), b = at4(n.bias, c);
+    return make_float4(fmaf(tanhf(alpha * v.x), w.x, b.x), fmaf(tanhf(alpha * v.y), w.y, b.y), fmaf(tanhf(alpha * v.z), w.z, b.z),
+                       fmaf(tanhf(alpha * v.w), w.w, b.w));
+  };
+  TA* h = p.h != nullptr ? reinterpret_cast<TA*>(p.h) + r * p.ldh : nullptr;
+  TA* copy = p.copy != nullptr ? reinterpret_cast<TA*>(p.copy) + r * p.ldc : nullptr;
+  const float post_alpha = BOUNDED && update ? *p.post.alpha : 0.f, pre_alpha = BOUNDED && p.h != nullptr ? *p.pre.alpha : 0.f;
+  float post_scale = 0.f;
+  if (!BOUNDED && update) {
+    float s = 0.f;
+    for (int c = threadIdx.x * 4; c < p.dp; c += step) {
+      const float4 v = sublayer(c);
+      sw_row[c >> 2] = v;
+      s += square(v);
+    }
+    post_scale = 1.f / sqrtf(block_sum(s, red) / (float)p.d + p.eps);
+  }
+  float ss = 0.f;
+  for (int c = threadIdx.x * 4; c < p.dp; c += step) {
+    float4 v = at4(x, c);
+    if (update) {
+      float4 n;
+      if (BOUNDED) {
+        n = bounded(p.post, post_alpha, sublayer(c), c);
+      } else {
+        const float4 a = sw_row[c >> 2], w = at4(p.post.weight, c);
+        n = make_float4(a.x * post_scale * w.x, a.y * post_scale * w.y, a.z * post_scale * w.z, a.w * post_scale * w.w);
+      }
+      v.x += n.x; v.y += n.y; v.z += n.z; v.w += n.w;
+      *reinterpret_cast<float4*>(x + c) = v;
+    }
+    if (copy != nullptr) store_act4(copy + c, v);
+    if (h == nullptr) continue;
+    if (BOUNDED) {
+      store_act4(h + c, bounded(p.pre, pre_alpha, v, c));
+    } else {
+      sw_row[c >> 2] = v;
+      ss += square(v);
+    }
+  }
+  if (BOUNDED || h == nullptr) return;
+  const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)p.d + p.eps);
+  for (int c = threadIdx.x * 4; c < p.dp; c += step) {
+    const float4 v = sw_row[c >> 2], w = at4(p.pre.weight, c);
+    store_act4(h + c, make_float4(v.x * rs * w.x, v.y * rs * w.y, v.z * rs * w.z, v.w * rs * w.w));
+  }
+}
+
+// out = a N(z) + b N(z^2) + c N(z^3) + e on rows of n channels (N: division by the root mean square over the row); act = {a, b, c, e}.
+// Padding columns n .. np - 1 of out become zero.
+template <typename TA>
+__global__ void __launch_bounds__(256) poly_norm_kernel(const TA* __restrict__ z, long long ldz, const float* __restrict__ act, TA* __restrict__ out,
+                                                        long long ldo, int n, int np, float eps) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const TA* row = z + (long long)blockIdx.x * ldz;
+  TA* dst = out + (long long)blockIdx.x * ldo;
+  float m2 = 0.f, m4 = 0.f, m6 = 0.f;
+  auto powers = [&](float v) {
+    const float s = v * v;
+    m2 += s;
+    m4 = fmaf(s, s, m4);
+    m6 = fmaf(s * s, s, m6);
+  };
+  for (int c = threadIdx.x * 4; c < np; c += blockDim.x * 4) {      // (padding columns of z are zero)
+    const float4 v = load_act4(row + c);
+    powers(v.x); powers(v.y); powers(v.z); powers(v.w);
+  }
+  const float inv = 1.f / (float)n;
+  const float a = act[0] / sqrtf(block_sum(m2, red) * inv + eps), b = act[1] / sqrtf(block_sum(m4, red) * inv + eps);
+  const float k = act[2] / sqrtf(block_sum(m6, red) * inv + eps), e = act[3];
+  auto one = [&](float v, int c) { return c < n ? fmaf(v, fmaf(v, fmaf(v, k, b), a), e) : 0.f; };
+  for (int c = threadIdx.x * 4; c < np; c += blockDim.x * 4) {
+    const float4 v = load_act4(row + c);
+    store_act4(dst + c, make_float4(one(v.x, c), one(v.y, c + 1), one(v.z, c + 2), one(v.w, c + 3)));
+  }
+}
+
 // Layer norm of fp32 rows with a two-pass variance; the row is kept in shared memory.
 //   y == nullptr : out = LN(x[rows[i]]) * w + b                     (rows == nullptr: row i)
 //   otherwise    : x += LN(y) * w + b, out = x                      (norm on the sublayer's output, residual add)
@@ -821,6 +985,45 @@ extern "C" int rb_stream_norm(float* x, long long ldx, const float* y1, const fl
   const int threads = dp <= 512 ? 128 : 256;
   cudaError_t err;
   RB_ACT_DISPATCH(dtype, err = launch_kernel(stream_norm_kernel<TA>, dim3(n), dim3(threads), (size_t)dp * 4, stream, p);)
+  return err == cudaSuccess ? 0 : -11;
+}
+
+struct SandwichArgs {            // mirrored by ops/elementwise.py
+  float* x; const float* y; const float* y2; const float* w; const float* w2; const float* gate; const void* e; const float* p; const int* idx;
+  const void* pass; const float* post_weight; const float* post_bias; const float* post_alpha; const float* pre_weight; const float* pre_bias;
+  const float* pre_alpha; void* copy; void* h; const int* rows; int* status;
+  long long ldx, ldy, ld_gate, lde, ld_pass, ldc, ldh;
+  int k, experts, num_src_rows, n, d, dp, bounded, dtype;
+  float pair_scale, eps;
+};
+
+extern "C" int rb_stream_sandwich(const SandwichArgs* a, cudaStream_t stream) {
+  const bool update = a->y != nullptr || a->e != nullptr;
+  if (a->n <= 0 || a->d <= 0 || a->dp < a->d || a->dp % 4 != 0 || a->dp > 12288 || (a->rows != nullptr && update)) return -1;
+  if ((a->ldx | a->ldy | a->lde | a->ld_pass | a->ldc | a->ldh) % 4 != 0 || (a->y2 != nullptr && (a->y == nullptr || a->e != nullptr || a->gate != nullptr))) return -1;
+  if ((a->e != nullptr && (a->p == nullptr || a->idx == nullptr || a->pass == nullptr)) || (update && a->post_weight == nullptr) ||
+      (a->h != nullptr && a->pre_weight == nullptr))
+    return -1;
+  if (a->bounded && ((update && (a->post_bias == nullptr || a->post_alpha == nullptr)) || (a->h != nullptr && (a->pre_bias == nullptr || a->pre_alpha == nullptr)))) return -1;
+  const SandwichParams p{a->x, a->ldx, a->y, a->y2, a->ldy, a->w, a->w2, a->pair_scale, a->gate, a->ld_gate, a->e, a->lde, a->p, a->idx, a->k, a->experts,
+                         a->pass, a->ld_pass, {a->post_weight, a->post_bias, a->post_alpha}, {a->pre_weight, a->pre_bias, a->pre_alpha}, a->copy, a->ldc,
+                         a->h, a->ldh, a->rows, a->num_src_rows, a->d, a->dp, a->eps, a->status};
+  const int threads = a->dp <= 512 ? 128 : 256;
+  const size_t smem = a->bounded ? 0 : (size_t)a->dp * 4;
+  cudaError_t err;
+  RB_ACT_DISPATCH(a->dtype, err = a->bounded ? launch_kernel(stream_sandwich_kernel<TA, true>, dim3(a->n), dim3(threads), smem, stream, p)
+                                             : launch_kernel(stream_sandwich_kernel<TA, false>, dim3(a->n), dim3(threads), smem, stream, p);)
+  return err == cudaSuccess ? 0 : -11;
+}
+
+// z [T, ldz] with np columns, n of them in use -> out [T, ldo].
+extern "C" int rb_poly_norm(const void* z, long long ldz, const float* act, void* out, long long ldo, int T, int n, int np, float eps, int dtype,
+                            cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (n <= 0 || np < n || np % 4 != 0 || ldz % 4 != 0 || ldo % 4 != 0) return -1;
+  const int threads = np <= 512 ? 128 : 256;
+  cudaError_t err;
+  RB_ACT_DISPATCH(dtype, err = launch_kernel(poly_norm_kernel<TA>, dim3(T), dim3(threads), 0, stream, (const TA*)z, ldz, act, (TA*)out, ldo, n, np, eps);)
   return err == cudaSuccess ? 0 : -11;
 }
 

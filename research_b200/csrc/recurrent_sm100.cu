@@ -2,6 +2,8 @@
 //
 //   S_t = a_t S_(t-1) + b_t k_t v_t^T,   o_t = S_t^T q_t        (see ops/recurrent.py)
 //   o_t = S_(t-1)^T q_t + (sum_c u_c q_tc k_tc) v_t,  then row c of S decays by its own w_tc and takes k_tc v_t        (time mixing)
+//   row c of S keeps f_tc of itself and takes (1 - f_tc) v_t,  o_t = S_t^T q_t                                         (forget mixing)
+//   S decays by g_t and takes beta_t k_t (v_t - S^T k_t)^T,  o_t = S_t^T q_t                                           (delta rule)
 //
 //   scan        token by token: short portions and long ones of the exact mode. One CTA per (sequence, head, 32 value channels);
 //               the state tile stays in registers over the tokens of the portion.
@@ -10,7 +12,9 @@
 //               adds to the state (all chunks at once), the state in front of every chunk (one pass over the chunks), the
 //               outputs (all chunks at once)
 //   time mixing, one token per sequence: as decode, a whole head at a time, with the head's norm and the output gate
-//   time mixing of long portions: chunked in the same way, in three launches
+//   time mixing, forget mixing of long portions: chunked in the same way, in three launches
+//   delta rule  short convolutions, SiLU and the heads' norms in a launch of their own; long portions: a triangular inverse per chunk,
+//               one pass over the chunks, outputs
 //   gated_norm  RMS norm per head or over all heads, times sigmoid(gate), to the activation type
 //
 // State: s [slots, H, tiles, KP, 32], n [slots, H, tiles, KP], m [slots, H, tiles], all fp32. A tile of 32 value channels keeps its
@@ -36,6 +40,8 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-
 // log(sigmoid(z)) without cancellation at either end
 __device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
+enum { FORM_PLAIN = 0, FORM_MIX = 1, FORM_FORGET = 2, FORM_DELTA = 3 };
+
 struct ScanParams {
   const void* proj;        // [T, ld]: q | k | v (activation type)
   long long ld;
@@ -55,21 +61,33 @@ struct ScanParams {
   float* out;              // [T, ldo]
   long long ldo;
   int H, dk, KP, VP, num_slots, gated, rows;
-  const float* z;          // [T, ldz] time mixing: w = exp(-exp(z + w0)), column h * KP + key channel
+  const float* z;          // [T, ldz] time mixing: w = exp(-exp(z + w0)), column h * KP + key channel; forget mixing: logits of f
   long long ldz;
   const float* w0;         // [H * KP]
-  const float* bonus;      // [H * KP]
+  const float* bonus;      // [H * KP]; forget mixing: the lower bound of f
   int* status;
+  int ratio;               // heads that share queries and keys
+  const float* units;      // [T, 2 * H / ratio] delta rule: factors of the queries, then of the keys
+  const float* steps;      // [T, 2 * H] delta rule: logarithm of the decay, then the step size
 };
 
 __device__ __forceinline__ float channel_decay(float z) { return expf(-expf(z)); }
 
-// NR: key rows held by a thread (dk <= NR * SC_ROWS); MIX: time mixing
-template <typename T, int NR, bool MIX>
+// Forget gate f = low + (1 - low) sigmoid(z) and what may be written, 1 - f.
+__device__ __forceinline__ float2 forget_gate(float z, float low) {
+  const float e = expf(-fabsf(z)), big = 1.f / (1.f + e), small = e * big;
+  return make_float2(fmaf(1.f - low, z >= 0.f ? big : small, low), (1.f - low) * (z >= 0.f ? small : big));
+}
+
+// NR: key rows held by a thread (dk <= NR * SC_ROWS)
+template <typename T, int NR, int FORM>
 __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanParams p) {
-  __shared__ float qs[NR * SC_ROWS], ks[NR * SC_ROWS], vs[SC_COLS];
-  __shared__ float ws[MIX ? NR * SC_ROWS : 1];
-  __shared__ float red[SC_THREADS / 32][SC_COLS];
+  constexpr bool MIX = FORM == FORM_MIX, FORGET = FORM == FORM_FORGET, DELTA = FORM == FORM_DELTA;
+  __shared__ float qs[NR * SC_ROWS], ks[NR * SC_ROWS];
+  __shared__ __align__(16) float vs[SC_COLS];
+  __shared__ float ws[MIX || FORGET ? NR * SC_ROWS : 1];
+  __shared__ __align__(16) float red[SC_THREADS / 32][SC_COLS];
+  __shared__ __align__(16) float red_k[DELTA ? SC_THREADS / 32 : 1][SC_COLS];
   __shared__ float red_n[SC_THREADS / 32];
   pdl_launch_dependents();
   const int tile = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
@@ -105,22 +123,36 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
   }
   float m = fresh || !p.gated ? 0.f : p.m[unit];
   const T* proj = reinterpret_cast<const T*>(p.proj);
-  const float decay = p.gated || MIX ? 0.f : p.decay[h];
+  const float decay = p.gated || FORM != FORM_PLAIN ? 0.f : p.decay[h];
+  const int hk = h / p.ratio;                      // whose queries and keys
   float bonus[MIX ? NR : 1];
   if (MIX)
 #pragma unroll
     for (int i = 0; i < NR; ++i) bonus[i] = r0 + i * SC_ROWS < p.dk ? p.bonus[h * p.KP + r0 + i * SC_ROWS] : 0.f;
   for (int t = t0; t < t1; ++t) {
     const T* row = proj + t * p.ld;
+    const float* unit_of = DELTA ? p.units + (long long)t * 2 * (p.H / p.ratio) + hk : nullptr;
+    const float q_scale = DELTA ? p.q_scale * unit_of[0] : p.q_scale, k_scale = DELTA ? unit_of[p.H / p.ratio] : 1.f;
     for (int i = tid; i < p.dk; i += SC_THREADS) {
-      qs[i] = to_f<T>(row[p.q_col + h * p.KP + i]) * p.q_scale;
-      ks[i] = to_f<T>(row[p.k_col + h * p.KP + i]);
+      qs[i] = to_f<T>(row[p.q_col + hk * p.KP + i]) * q_scale;
+      if (FORGET) {
+        const float2 f = forget_gate(p.z[t * p.ldz + h * p.KP + i] + p.w0[h * p.KP + i], p.bonus[h * p.KP + i]);
+        ws[i] = f.x;
+        ks[i] = f.y;
+      } else {
+        ks[i] = to_f<T>(row[p.k_col + hk * p.KP + i]) * k_scale;
+      }
       if (MIX) ws[i] = channel_decay(p.z[t * p.ldz + h * p.KP + i] + p.w0[h * p.KP + i]);
     }
     if (tid < SC_COLS) {
       vs[tid] = to_f<T>(row[p.v_col + h * p.VP + tile * SC_COLS + tid]);
     }
     float a = decay, w = 1.f;
+    if (DELTA) {
+      const float* g = p.steps + (long long)t * 2 * p.H + h;
+      a = expf(g[0]);
+      w = g[p.H];
+    }
     if (p.gated) {
       const float* g = p.small + t * p.ld_small;
       const float gi = p.cap * tanhf((g[h] + p.bias_i[h]) / p.cap);
@@ -132,11 +164,35 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
     }
     __syncthreads();
     const float4 v = *reinterpret_cast<const float4*>(&vs[c4 * 4]);
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    float nq = 0.f;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f), acc_k = acc;
+    float nq = 0.f, kr[DELTA ? NR : 1];
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
       const int r = r0 + i * SC_ROWS;
+      if (DELTA) {                                   // S^T k and S^T q of the state in front of the token, and q . k
+        const float k = r < p.dk ? ks[r] : 0.f, q = r < p.dk ? qs[r] : 0.f;
+        kr[DELTA ? i : 0] = k;
+        acc_k.x = fmaf(k, S[i].x, acc_k.x);
+        acc_k.y = fmaf(k, S[i].y, acc_k.y);
+        acc_k.z = fmaf(k, S[i].z, acc_k.z);
+        acc_k.w = fmaf(k, S[i].w, acc_k.w);
+        acc.x = fmaf(q, S[i].x, acc.x);
+        acc.y = fmaf(q, S[i].y, acc.y);
+        acc.z = fmaf(q, S[i].z, acc.z);
+        acc.w = fmaf(q, S[i].w, acc.w);
+        nq = fmaf(q, k, nq);
+      }
+      if (FORGET && r < p.dk) {
+        const float k = ks[r], q = qs[r], d = ws[r];
+        S[i].x = fmaf(d, S[i].x, k * v.x);
+        S[i].y = fmaf(d, S[i].y, k * v.y);
+        S[i].z = fmaf(d, S[i].z, k * v.z);
+        S[i].w = fmaf(d, S[i].w, k * v.w);
+        acc.x = fmaf(q, S[i].x, acc.x);
+        acc.y = fmaf(q, S[i].y, acc.y);
+        acc.z = fmaf(q, S[i].z, acc.z);
+        acc.w = fmaf(q, S[i].w, acc.w);
+      }
       if (MIX && r < p.dk) {
         const float k = ks[r], q = qs[r], d = ws[r], u = bonus[MIX ? i : 0];
         const float4 kv = make_float4(k * v.x, k * v.y, k * v.z, k * v.w);
@@ -149,7 +205,7 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
         S[i].z = fmaf(d, S[i].z, kv.z);
         S[i].w = fmaf(d, S[i].w, kv.w);
       }
-      if (!MIX && r < p.dk) {
+      if (FORM == FORM_PLAIN && r < p.dk) {
         const float kw = w * ks[r], q = qs[r];
         S[i].x = fmaf(a, S[i].x, kw * v.x);
         S[i].y = fmaf(a, S[i].y, kw * v.y);
@@ -171,15 +227,47 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
       acc.z += __shfl_xor_sync(0xffffffffu, acc.z, o);
       acc.w += __shfl_xor_sync(0xffffffffu, acc.w, o);
       nq += __shfl_xor_sync(0xffffffffu, nq, o);
+      if (DELTA) {
+        acc_k.x += __shfl_xor_sync(0xffffffffu, acc_k.x, o);
+        acc_k.y += __shfl_xor_sync(0xffffffffu, acc_k.y, o);
+        acc_k.z += __shfl_xor_sync(0xffffffffu, acc_k.z, o);
+        acc_k.w += __shfl_xor_sync(0xffffffffu, acc_k.w, o);
+      }
     }
-    if (lane < 8) *reinterpret_cast<float4*>(&red[warp][lane * 4]) = acc;
+    if (lane < 8) {
+      *reinterpret_cast<float4*>(&red[warp][lane * 4]) = acc;
+      if (DELTA) *reinterpret_cast<float4*>(&red_k[DELTA ? warp : 0][lane * 4]) = acc_k;
+    }
     if (lane == 0) red_n[warp] = nq;
+    const float my_v = DELTA && tid < SC_COLS ? vs[tid] : 0.f;
     __syncthreads();
-    if (tid < SC_COLS) {
-      float o = 0.f, d = 0.f;
+    if (DELTA) {                                     // (what follows reads the sums alone: the next token's vectors may come)
+      float4 sk = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int i = 0; i < SC_THREADS / 32; ++i) { o += red[i][tid]; d += red_n[i]; }
+      for (int i = 0; i < SC_THREADS / 32; ++i) {
+        const float4 x = *reinterpret_cast<const float4*>(&red_k[DELTA ? i : 0][c4 * 4]);
+        sk.x += x.x; sk.y += x.y; sk.z += x.z; sk.w += x.w;
+      }
+      const float4 u = make_float4(w * (v.x - a * sk.x), w * (v.y - a * sk.y), w * (v.z - a * sk.z), w * (v.w - a * sk.w));
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        const float k = kr[DELTA ? i : 0];
+        S[i].x = fmaf(a, S[i].x, k * u.x);
+        S[i].y = fmaf(a, S[i].y, k * u.y);
+        S[i].z = fmaf(a, S[i].z, k * u.z);
+        S[i].w = fmaf(a, S[i].w, k * u.w);
+      }
+    }
+    if (tid < SC_COLS) {
+      float o = 0.f, d = 0.f, sk = 0.f;
+#pragma unroll
+      for (int i = 0; i < SC_THREADS / 32; ++i) {
+        o += red[i][tid];
+        d += red_n[i];
+        if (DELTA) sk += red_k[DELTA ? i : 0][tid];
+      }
       if (p.gated) o /= fmaxf(fabsf(d), expf(-m)) + 1e-6f;
+      if (DELTA) o = fmaf(a, o, d * (w * (my_v - a * sk)));
       p.out[t * p.ldo + h * p.VP + tile * SC_COLS + tid] = o;
     }
   }
@@ -194,16 +282,16 @@ __global__ void __launch_bounds__(SC_THREADS) recurrent_scan_kernel(const ScanPa
   if (p.gated && tid == 0) p.m[unit] = m;
 }
 
-template <typename T, bool MIX>
+template <typename T, int FORM>
 static int launch_scan(const ScanParams& p, int B, cudaStream_t stream) {
   const dim3 grid(p.VP / SC_COLS, p.H, B);
   const int need = (p.dk + SC_ROWS - 1) / SC_ROWS;
   cudaError_t e;
-  if (need <= 1) e = launch_kernel(recurrent_scan_kernel<T, 1, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
-  else if (need <= 2) e = launch_kernel(recurrent_scan_kernel<T, 2, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
-  else if (need <= 4) e = launch_kernel(recurrent_scan_kernel<T, 4, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
-  else if (need <= 8) e = launch_kernel(recurrent_scan_kernel<T, 8, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
-  else if (need <= 16) e = launch_kernel(recurrent_scan_kernel<T, 16, MIX>, grid, dim3(SC_THREADS), 0, stream, p);
+  if (need <= 1) e = launch_kernel(recurrent_scan_kernel<T, 1, FORM>, grid, dim3(SC_THREADS), 0, stream, p);
+  else if (need <= 2) e = launch_kernel(recurrent_scan_kernel<T, 2, FORM>, grid, dim3(SC_THREADS), 0, stream, p);
+  else if (need <= 4) e = launch_kernel(recurrent_scan_kernel<T, 4, FORM>, grid, dim3(SC_THREADS), 0, stream, p);
+  else if (need <= 8) e = launch_kernel(recurrent_scan_kernel<T, 8, FORM>, grid, dim3(SC_THREADS), 0, stream, p);
+  else if (need <= 16) e = launch_kernel(recurrent_scan_kernel<T, 16, FORM>, grid, dim3(SC_THREADS), 0, stream, p);
   else return -1;
   return e == cudaSuccess ? 0 : -11;
 }
@@ -226,13 +314,15 @@ __device__ __forceinline__ void bulk_store(void* dst, uint32_t src, uint32_t byt
   asm volatile("cp.async.bulk.commit_group;" ::: "memory");
 }
 
-template <typename T, bool MIX>
+template <typename T, int FORM>
 __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const ScanParams p, int B, int units) {
+  constexpr bool MIX = FORM == FORM_MIX, FORGET = FORM == FORM_FORGET, DELTA = FORM == FORM_DELTA;
   extern __shared__ __align__(128) uint8_t smem_raw[];       // RD_STAGES x [dk, 32] fp32, then the sequences' slots
   __shared__ float qs[RD_MAX_DK], ks[RD_MAX_DK];
-  __shared__ float ws[MIX ? RD_MAX_DK : 1], us[MIX ? RD_MAX_DK : 1];
+  __shared__ float ws[MIX || FORGET ? RD_MAX_DK : 1], us[MIX ? RD_MAX_DK : 1];
   __shared__ __align__(16) float vs[SC_COLS];
   __shared__ __align__(16) float red[RD_THREADS / 32][SC_COLS];
+  __shared__ __align__(16) float red_k[DELTA ? RD_THREADS / 32 : 1][SC_COLS];
   __shared__ float red_n[RD_THREADS / 32];
   __shared__ __align__(8) uint64_t full[RD_STAGES];
   __shared__ int abort_flag;
@@ -279,21 +369,24 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
   if (tid == 0)
     for (int i = 0; i < RD_STAGES - 1; ++i) load(i);
   float q[RD_VEC], k[RD_VEC], n[RD_VEC], v = 0.f, gi = 0.f, gf = 0.f, m0 = 0.f;
-  float z[MIX ? RD_VEC : 1], bonus[MIX ? RD_VEC : 1];
+  float z[MIX || FORGET ? RD_VEC : 1], bonus[MIX || FORGET ? RD_VEC : 1];
   Unit x{};
   auto fetch = [&](int u) {
     x = unit_of(u);
     const T* row = reinterpret_cast<const T*>(p.proj) + x.b * p.ld;
     const float* nt = p.n + state_index(x) * p.KP;
+    const int hk = x.h / p.ratio;
+    const float* unit = DELTA ? p.units + (long long)x.b * 2 * (p.H / p.ratio) + hk : nullptr;
+    const float q_scale = DELTA ? p.q_scale * unit[0] : p.q_scale, k_scale = DELTA ? unit[p.H / p.ratio] : 1.f;
 #pragma unroll
     for (int i = 0; i < RD_VEC; ++i) {
       const int r = tid + i * RD_THREADS;
       q[i] = k[i] = n[i] = 0.f;
       if (r < p.dk) {
-        q[i] = to_f<T>(row[p.q_col + x.h * p.KP + r]) * p.q_scale;
-        k[i] = to_f<T>(row[p.k_col + x.h * p.KP + r]);
+        q[i] = to_f<T>(row[p.q_col + hk * p.KP + r]) * q_scale;
+        if (!FORGET) k[i] = to_f<T>(row[p.k_col + hk * p.KP + r]) * k_scale;
         if (p.gated) n[i] = nt[r];
-        if (MIX) {
+        if (MIX || FORGET) {
           z[i] = p.z[x.b * p.ldz + x.h * p.KP + r] + p.w0[x.h * p.KP + r];
           bonus[i] = p.bonus[x.h * p.KP + r];
         }
@@ -304,6 +397,10 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
       gi = p.small[x.b * p.ld_small + x.h];
       gf = p.small[x.b * p.ld_small + p.H + x.h];
       m0 = p.m[state_index(x)];
+    }
+    if (DELTA) {
+      gf = p.steps[(long long)x.b * 2 * p.H + x.h];
+      gi = p.steps[(long long)x.b * 2 * p.H + p.H + x.h];
     }
   };
   if ((int)blockIdx.x < units) fetch(blockIdx.x);
@@ -320,8 +417,12 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
       m = fmaxf(gf + m0, gi);
       a = expf(gf + m0 - m);
       w = expf(gi - m);
-    } else if (!MIX) {
+    } else if (FORM == FORM_PLAIN) {
       a = p.decay[cur.h];
+    }
+    if (DELTA) {
+      a = expf(gf);
+      w = gi;
     }
     const long long si = state_index(cur);
     float nq = 0.f;
@@ -329,10 +430,16 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
     for (int i = 0; i < RD_VEC; ++i) {
       const int r = tid + i * RD_THREADS;
       if (r < p.dk) {
-        const float kw = w * k[i];
+        const float kw = DELTA ? k[i] : w * k[i];
         qs[r] = q[i];
         ks[r] = kw;
-        if (MIX) { ws[r] = channel_decay(z[i]); us[r] = bonus[i]; }
+        if (DELTA) nq = fmaf(q[i], kw, nq);
+        if (MIX) { ws[r] = channel_decay(z[MIX ? i : 0]); us[r] = bonus[MIX ? i : 0]; }
+        if (FORGET) {
+          const float2 f = forget_gate(z[FORGET ? i : 0], bonus[FORGET ? i : 0]);
+          ws[r] = f.x;
+          ks[r] = f.y;
+        }
         if (p.gated) {
           const float nn = fmaf(a, n[i], kw);
           nq = fmaf(q[i], nn, nq);
@@ -348,12 +455,46 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
     if (!ok) break;
     if (u + (int)gridDim.x < units) fetch(u + gridDim.x);
     float4* S = reinterpret_cast<float4*>(smem_raw + stage * tile_bytes);
-    const float4 vv = *reinterpret_cast<const float4*>(&vs[c4 * 4]);
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 vv = *reinterpret_cast<const float4*>(&vs[c4 * 4]);
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f), out_k = acc;
+    const float my_v = DELTA && tid < SC_COLS ? vs[tid] : 0.f;
+    if (DELTA) {                                             // S^T k and S^T q of the state in front of the token
+      if (!zero)
+#pragma unroll 4
+        for (int r = r0; r < p.dk; r += RD_THREADS / 8) {
+          const float4 s = S[r * (SC_COLS / 4) + c4];
+          const float kw = ks[r], qr = qs[r];
+          out_k.x = fmaf(kw, s.x, out_k.x);
+          out_k.y = fmaf(kw, s.y, out_k.y);
+          out_k.z = fmaf(kw, s.z, out_k.z);
+          out_k.w = fmaf(kw, s.w, out_k.w);
+          acc.x = fmaf(qr, s.x, acc.x);
+          acc.y = fmaf(qr, s.y, acc.y);
+          acc.z = fmaf(qr, s.z, acc.z);
+          acc.w = fmaf(qr, s.w, acc.w);
+        }
+#pragma unroll
+      for (int o = 8; o < 32; o <<= 1) {
+        out_k.x += __shfl_xor_sync(0xffffffffu, out_k.x, o);
+        out_k.y += __shfl_xor_sync(0xffffffffu, out_k.y, o);
+        out_k.z += __shfl_xor_sync(0xffffffffu, out_k.z, o);
+        out_k.w += __shfl_xor_sync(0xffffffffu, out_k.w, o);
+      }
+      if (lane < 8) *reinterpret_cast<float4*>(&red_k[DELTA ? warp : 0][lane * 4]) = out_k;
+      __syncthreads();
+      float4 sk = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int i = 0; i < RD_THREADS / 32; ++i) {
+        const float4 y = *reinterpret_cast<const float4*>(&red_k[DELTA ? i : 0][c4 * 4]);
+        sk.x += y.x; sk.y += y.y; sk.z += y.z; sk.w += y.w;
+      }
+      vv = make_float4(w * (vv.x - a * sk.x), w * (vv.y - a * sk.y), w * (vv.z - a * sk.z), w * (vv.w - a * sk.w));
+    }
 #pragma unroll 4
     for (int r = r0; r < p.dk; r += RD_THREADS / 8) {
       float4 s = zero ? make_float4(0.f, 0.f, 0.f, 0.f) : S[r * (SC_COLS / 4) + c4];
-      const float kw = ks[r], qr = qs[r];
+      const float kw = ks[r], qr = DELTA ? 0.f : qs[r];
+      if (FORGET) a = ws[r];
       if (MIX) {                                             // the state in front of the token, and the token with its bonus
         const float bo = us[r];
         acc.x = fmaf(qr, fmaf(bo, kw * vv.x, s.x), acc.x);
@@ -366,7 +507,7 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
       s.y = fmaf(a, s.y, kw * vv.y);
       s.z = fmaf(a, s.z, kw * vv.z);
       s.w = fmaf(a, s.w, kw * vv.w);
-      if (!MIX) {
+      if (!MIX && !DELTA) {
         acc.x = fmaf(qr, s.x, acc.x);
         acc.y = fmaf(qr, s.y, acc.y);
         acc.z = fmaf(qr, s.z, acc.z);
@@ -382,7 +523,7 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
       acc.z += __shfl_xor_sync(0xffffffffu, acc.z, o);
       acc.w += __shfl_xor_sync(0xffffffffu, acc.w, o);
     }
-    if (p.gated) nq = warp_sum(nq);
+    if (p.gated || DELTA) nq = warp_sum(nq);
     if (lane < 8) *reinterpret_cast<float4*>(&red[warp][lane * 4]) = acc;
     if (lane == 0) red_n[warp] = nq;
     __syncthreads();
@@ -393,10 +534,15 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
       load(it + RD_STAGES - 1);
     }
     if (tid < SC_COLS) {
-      float o = 0.f, d = 0.f;
+      float o = 0.f, d = 0.f, sk = 0.f;
 #pragma unroll
-      for (int i = 0; i < RD_THREADS / 32; ++i) { o += red[i][tid]; d += red_n[i]; }
+      for (int i = 0; i < RD_THREADS / 32; ++i) {
+        o += red[i][tid];
+        d += red_n[i];
+        if (DELTA) sk += red_k[DELTA ? i : 0][tid];
+      }
       if (p.gated) o /= fmaxf(fabsf(d), expf(-m)) + 1e-6f;
+      if (DELTA) o = fmaf(a, o, d * (w * (my_v - a * sk)));
       p.out[cur.b * p.ldo + cur.h * p.VP + cur.tile * SC_COLS + tid] = cur.slot < 0 ? 0.f : o;
     }
   }
@@ -411,7 +557,7 @@ __global__ void __launch_bounds__(RD_THREADS) recurrent_decode_kernel(const Scan
   }
 }
 
-template <typename T, bool MIX>
+template <typename T, int FORM>
 static int launch_decode(const ScanParams& p, int B, cudaStream_t stream) {
   static int sms[64] = {};
   int dev = 0;
@@ -420,13 +566,13 @@ static int launch_decode(const ScanParams& p, int B, cudaStream_t stream) {
   if (sms[dev] == 0) {
     int n = 0;
     if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess ||
-        cudaFuncSetAttribute(recurrent_decode_kernel<T, MIX>, cudaFuncAttributeMaxDynamicSharedMemorySize, RD_STAGES * RD_MAX_DK * SC_COLS * 4 + RD_MAX_B * 4) != cudaSuccess)
+        cudaFuncSetAttribute(recurrent_decode_kernel<T, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, RD_STAGES * RD_MAX_DK * SC_COLS * 4 + RD_MAX_B * 4) != cudaSuccess)
       return -10;
     sms[dev] = n;
   }
   const int per_sm = 200 * 1024 / (smem + 7 * 1024) > 6 ? 6 : 200 * 1024 / (smem + 7 * 1024);
   const int units = B * p.H * (p.VP / SC_COLS), grid = units < sms[dev] * per_sm ? units : sms[dev] * per_sm;
-  return launch_kernel(recurrent_decode_kernel<T, MIX>, dim3(grid), dim3(RD_THREADS), smem, stream, p, B, units) == cudaSuccess ? 0 : -11;
+  return launch_kernel(recurrent_decode_kernel<T, FORM>, dim3(grid), dim3(RD_THREADS), smem, stream, p, B, units) == cudaSuccess ? 0 : -11;
 }
 
 // ------------------------------------------------------------------------------------------
@@ -478,6 +624,10 @@ struct ChunkParams {
   long long ldo;
   int H, dk, KP, VP, num_slots, gated;
   int* status;
+  const __nv_bfloat16* v;  // [T, ld_v] values
+  long long ld_v;
+  int ratio;               // heads that share queries and keys
+  int factors;             // the third of a token's gates is a factor of its query
 };
 
 __device__ __forceinline__ float chunk_exp2(float x) {
@@ -636,7 +786,7 @@ __global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_state_
   uint4 raw[UNITS];
   float weight = 0.f;
   auto fetch = [&](const ChunkUnit& x, int buf) {
-    chunk_load<64>(base + 2 * Cfg::kKBytes + buf * CH_CHUNK, p.proj + x.row0 * p.ld + p.v_col + x.h * p.VP + x.z * 64, p.ld, x.n);
+    chunk_load<64>(base + 2 * Cfg::kKBytes + buf * CH_CHUNK, p.v + x.row0 * p.ld_v + x.h * p.VP + x.z * 64, p.ld_v, x.n);
     const __nv_bfloat16* k = p.proj + x.row0 * p.ld + p.k_col + x.h * p.KP;
 #pragma unroll
     for (int i = 0; i < UNITS; ++i) {
@@ -882,13 +1032,13 @@ __global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_out_ke
   };
   auto fetch_first = [&](const ChunkUnit& x) {       // Q, the state's second part, the vectors, V
     const __nv_bfloat16* rows = p.proj + x.row0 * p.ld;
-    chunk_load<DK>(q_s, rows + p.q_col + x.h * p.KP, p.ld, x.n);
+    chunk_load<DK>(q_s, rows + p.q_col + x.h / p.ratio * p.KP, p.ld, x.n);
     load_state(sl_s, p.s_lo, x);
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
       const int e = tid + i * CHT, r = e >> 3;
       vr[i] = make_uint4(0u, 0u, 0u, 0u);
-      if (r < x.n) vr[i] = *reinterpret_cast<const uint4*>(rows + r * p.ld + p.v_col + x.h * p.VP + x.z * 64 + (e & 7) * 8);
+      if (r < x.n) vr[i] = *reinterpret_cast<const uint4*>(p.v + (x.row0 + r) * p.ld_v + x.h * p.VP + x.z * 64 + (e & 7) * 8);
     }
     if (tid < CH) {
       const float* g = p.gates + x.ch * 3 * CH + tid;
@@ -902,7 +1052,7 @@ __global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_out_ke
     }
   };
   auto fetch_second = [&](const ChunkUnit& x) {      // K, the state's first part
-    chunk_load<DK>(k_s, p.proj + x.row0 * p.ld + p.k_col + x.h * p.KP, p.ld, x.n);
+    chunk_load<DK>(k_s, p.proj + x.row0 * p.ld + p.k_col + x.h / p.ratio * p.KP, p.ld, x.n);
     load_state(sv_s, p.s_hi, x);
   };
   ChunkUnit x{};
@@ -1029,6 +1179,7 @@ __global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_out_ke
     __syncwarp();
     if (more) fetch_first(x);
     float f = p.q_scale;
+    if (p.factors) f *= F;
     if (p.gated) f /= fmaxf(fabsf((row_sum[0][t] + row_sum[1][t]) * p.q_scale), chunk_exp2(-(F + B))) + 1e-6f;
     ok = mbar_wait_bounded(smem_u32(&o_done), it & 1, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
     ok = __all_sync(0xffffffffu, ok);
@@ -1095,6 +1246,9 @@ static int launch_chunks(const ChunkParams& p, int n_chunks, int n_seq, cudaStre
 // (mma.sync, their operands are made in registers); of a block on the diagonal the lower left quarter and the lower left quarters
 // of the other two go the same way, and the four 4 x 4 triangles pair by pair in fp32. P V and the state's part run on tcgen05. Three launches: what every chunk
 // adds to the state (z becomes A on the way), the chain of states, outputs with the head's norm and the output gate.
+//
+// Forget mixing is the same with keys 1 - f, weights that end at A_t (a token is written before it is read, P_tt = q_t . k_t) and no
+// output gate.
 // ------------------------------------------------------------------------------------------
 constexpr float MIX_MOST = 64.f;      // a token that keeps less than 2^-64 keeps nothing; larger sums would cost A its last digits
 
@@ -1120,8 +1274,10 @@ struct MixParams {
   float eps;
   __nv_bfloat16* out;            // [T, ldo]
   long long ldo;
-  int H, dk, KP, VP, num_slots;
+  int H, dk, dv, KP, VP, num_slots;
   int* status;
+  __nv_bfloat16* keys;           // [T, ld_keys] forget mixing: 1 - f
+  long long ld_keys;
 };
 
 template <int DK>
@@ -1132,7 +1288,7 @@ struct MixStateCfg {
 };
 
 // What a chunk of one head adds to the state, and A. VP == KP == DK.
-template <int DK>
+template <int DK, bool FORGET>
 __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_state_kernel(const MixParams p) {
   using Cfg = MixStateCfg<DK>;
   constexpr int SEGS = 2 * CHT / DK, SEG = CH / SEGS;   // a thread has two channels of SEG tokens
@@ -1166,19 +1322,31 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_state_kernel(c
   const int col = 2 * (tid % (DK / 2)), seg = tid / (DK / 2), t0 = seg * SEG;
   float* z = p.z + (long long)(row0 + t0) * p.ldz + h * p.KP + col;
   const __nv_bfloat16* k = rows + (long long)t0 * p.ld + p.k_col + h * p.KP + col;
-  // exp(z + w0) log2(e) as one power of two
-  const float w0 = fmaf(p.w0[h * p.KP + col], LOG2E, 0.52876637f), w1 = fmaf(p.w0[h * p.KP + col + 1], LOG2E, 0.52876637f);
+  // exp(z + w0) log2(e) as one power of two; forget mixing: the bias itself
+  const float2 bias = *reinterpret_cast<const float2*>(p.w0 + h * p.KP + col);
+  const float w0 = FORGET ? bias.x : fmaf(bias.x, LOG2E, 0.52876637f), w1 = FORGET ? bias.y : fmaf(bias.y, LOG2E, 0.52876637f);
+  const float2 low = FORGET ? *reinterpret_cast<const float2*>(p.bonus + h * p.KP + col) : make_float2(0.f, 0.f);
   float2 A[SEG];
-  uint32_t keys[SEG];                                   // (fetched before anything is stored: the stores could alias)
+  uint32_t keys[FORGET ? 1 : SEG];                      // (fetched before anything is stored: the stores could alias)
+  float2 fresh[FORGET ? SEG : 1];                       // forget mixing: 1 - f
   const int mine = min(SEG, n - t0);
 #pragma unroll
   for (int i = 0; i < SEG; ++i) A[i] = i < mine ? *reinterpret_cast<const float2*>(z + (long long)i * p.ldz) : make_float2(0.f, 0.f);
+  if (!FORGET)
 #pragma unroll
-  for (int i = 0; i < SEG; ++i) keys[i] = i < mine ? *reinterpret_cast<const uint32_t*>(k + (long long)i * p.ld) : 0u;
+  for (int i = 0; i < SEG; ++i) keys[FORGET ? 0 : i] = i < mine ? *reinterpret_cast<const uint32_t*>(k + (long long)i * p.ld) : 0u;
   float2 run = make_float2(0.f, 0.f);
 #pragma unroll
   for (int i = 0; i < SEG; ++i) {
-    if (i < mine) {
+    if (FORGET) {
+      const float2 x = forget_gate(A[i].x + w0, low.x), y = forget_gate(A[i].y + w1, low.y);
+      fresh[FORGET ? i : 0] = make_float2(i < mine && col < p.dk ? x.y : 0.f, i < mine && col + 1 < p.dk ? y.y : 0.f);
+      auto kept = [](float2 f) { return fminf(-LOG2E * (f.y < 0.5f ? log1pf(-f.y) : logf(f.x)), MIX_MOST); };
+      if (i < mine) {
+        run.x -= kept(x);
+        run.y -= kept(y);
+      }
+    } else if (i < mine) {
       run.x -= fminf(chunk_exp2(fmaf(A[i].x, LOG2E, w0)), MIX_MOST);
       run.y -= fminf(chunk_exp2(fmaf(A[i].y, LOG2E, w1)), MIX_MOST);
     }
@@ -1201,7 +1369,13 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_state_kernel(c
     A[i].x += before.x;
     A[i].y += before.y;
     if (i < mine) *reinterpret_cast<float2*>(z + (long long)i * p.ldz) = A[i];
-    const float2 f = unpack_bf16x2(keys[i]);
+    float2 f;
+    if (FORGET) {
+      f = fresh[FORGET ? i : 0];
+      if (i < mine) *reinterpret_cast<uint32_t*>(p.keys + (long long)(row0 + t0 + i) * p.ld_keys + h * p.KP + col) = pack_bf16x2(f.x, f.y);
+    } else {
+      f = unpack_bf16x2(keys[FORGET ? 0 : i]);
+    }
     const float x = f.x * chunk_exp2(total.x - A[i].x), y = f.y * chunk_exp2(total.y - A[i].y);
     const uint32_t high = pack_bf16x2(x, y);
     const float2 back = unpack_bf16x2(high);
@@ -1316,7 +1490,7 @@ struct MixOutCfg {
 };
 
 // Outputs of a chunk of one head. VP == KP == DK.
-template <int DK>
+template <int DK, bool FORGET>
 __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(const MixParams p) {
   using Cfg = MixOutCfg<DK>;
   extern __shared__ __align__(128) uint8_t smem_raw[];
@@ -1348,7 +1522,9 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
   const long long ch = (long long)c * p.H + h;
   const __nv_bfloat16* rows = p.proj + (long long)row0 * p.ld;
   chunk_load<DK>(r_s, rows + h * p.KP, p.ld, n);
-  chunk_load<DK>(k_s, rows + p.k_col + h * p.KP, p.ld, n);
+  if (FORGET) chunk_load<DK>(k_s, p.keys + (long long)row0 * p.ld_keys + h * p.KP, p.ld_keys, n);
+  else chunk_load<DK>(k_s, rows + p.k_col + h * p.KP, p.ld, n);
+  constexpr int BACK = FORGET ? 0 : 1;                             // queries read the state behind their own token, or in front of it
   {
     // A: rows of DK floats, 32-byte pieces exchanged by the row's low bits so that eight rows of a fragment meet no bank twice
     const float* A = p.z + (long long)row0 * p.ldz + h * p.KP;
@@ -1375,9 +1551,9 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
   auto two_a = [&](int t, int u) {                                 // A of channels 8u + cq, 8u + cq + 1; zero in front of the chunk
     return t < 0 ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(a_row(t) + a_piece(t, u) + cq * 4);
   };
-  // r_t 2^(A_(t-1) - A_ref) and k_j 2^(A_ref - A_j) of those channels
+  // r_t 2^(A_(t-1) - A_ref) (forget mixing: A_t) and k_j 2^(A_ref - A_j) of those channels
   auto scaled_r = [&](int t, int u, float2 ref) {
-    const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_p + t * CH_ROWB + b_piece(t, u) + cq * 2)), a = two_a(t - 1, u);
+    const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_p + t * CH_ROWB + b_piece(t, u) + cq * 2)), a = two_a(t - BACK, u);
     return pack_bf16x2(x.x * chunk_exp2(a.x - ref.x), x.y * chunk_exp2(a.y - ref.y));
   };
   auto scaled_k = [&](const uint8_t* k_row, const uint8_t* arow, int kb, int ab, float2 ref) {
@@ -1451,14 +1627,14 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
       const int tt = t0 + lane / 6 * 4 + t, jj = t0 + lane / 6 * 4 + j;
       const uint8_t* rr = r_p + tt * CH_ROWB;
       const uint8_t* kr = k_p + jj * CH_ROWB;
-      const uint8_t* at = a_row(tt - 1);
+      const uint8_t* at = a_row(tt - BACK);
       const uint8_t* aj = a_row(jj);
       float s0 = 0.f, s1 = 0.f;
 #pragma unroll 2
       for (int i = 0; i < DK / 8; ++i) {                           // eight channels at a time, every lane from a place of its own
         const int u = (i + lane) & (DK / 8 - 1);
         const uint4 x = *reinterpret_cast<const uint4*>(rr + b_piece(tt, u)), y = *reinterpret_cast<const uint4*>(kr + b_piece(jj, u));
-        const float4* pa = reinterpret_cast<const float4*>(at + a_piece(tt - 1, u));
+        const float4* pa = reinterpret_cast<const float4*>(at + a_piece(tt - BACK, u));
         const float4* pb = reinterpret_cast<const float4*>(aj + a_piece(jj, u));
         const float4 a = pa[0], b = pb[0], c4 = pa[1], d4 = pb[1];
         float2 f, h2;
@@ -1485,7 +1661,11 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
       for (int i = 0; i < DK / 16; ++i) {
         const int u = (lane >> 4) * (DK / 16) + i;
         const uint4 x = *reinterpret_cast<const uint4*>(r_p + t * CH_ROWB + b_piece(t, u)), y = *reinterpret_cast<const uint4*>(k_p + t * CH_ROWB + b_piece(t, u));
-        const float4 b0 = *reinterpret_cast<const float4*>(bonus + u * 8), b1 = *reinterpret_cast<const float4*>(bonus + u * 8 + 4);
+        float4 b0 = make_float4(1.f, 1.f, 1.f, 1.f), b1 = b0;
+        if (!FORGET) {
+          b0 = *reinterpret_cast<const float4*>(bonus + u * 8);
+          b1 = *reinterpret_cast<const float4*>(bonus + u * 8 + 4);
+        }
         float2 f, h2;
         f = unpack_bf16x2(x.x); h2 = unpack_bf16x2(y.x); s = fmaf(f.x * h2.x, b0.x, fmaf(f.y * h2.y, b0.y, s));
         f = unpack_bf16x2(x.y); h2 = unpack_bf16x2(y.y); s = fmaf(f.x * h2.x, b0.z, fmaf(f.y * h2.y, b0.w, s));
@@ -1499,11 +1679,11 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
   __syncthreads();                                                 // k has been read
   chunk_load<DK>(k_s, rows + p.v_col + h * p.VP, p.ld, n);
 #pragma unroll 2
-  for (int i = tid; i < CH * (DK / 8); i += CHT) {                 // r 2^A_(t-1), in place
+  for (int i = tid; i < CH * (DK / 8); i += CHT) {                 // r 2^A_(t-1) (forget mixing: A_t), in place
     const int t = i / (DK / 8), u = i % (DK / 8);
-    if (t == 0) continue;
+    if (t < BACK) continue;
     uint4* at = reinterpret_cast<uint4*>(r_p + t * CH_ROWB + b_piece(t, u));
-    const float4* pa = reinterpret_cast<const float4*>(a_row(t - 1) + a_piece(t - 1, u));
+    const float4* pa = reinterpret_cast<const float4*>(a_row(t - BACK) + a_piece(t - BACK, u));
     const float4 a = pa[0], b = pa[1];
     uint4 v = *at;
     auto one = [&](uint32_t x, float ax, float ay) {
@@ -1555,7 +1735,7 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
 #pragma unroll
   for (int i = 0; i < HC / 8; ++i) {
     gate[i] = make_uint4(0u, 0u, 0u, 0u);
-    if (t < n) gate[i] = *reinterpret_cast<const uint4*>(rows + (long long)t * p.ld + p.g_col + h * p.VP + half * HC + i * 8);
+    if (!FORGET && t < n) gate[i] = *reinterpret_cast<const uint4*>(rows + (long long)t * p.ld + p.g_col + h * p.VP + half * HC + i * 8);
   }
   bool ok = mbar_wait_bounded(smem_u32(&done), 0, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
   ok = __all_sync(0xffffffffu, ok);
@@ -1573,7 +1753,7 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
   }
   __syncthreads();
   if (ok && t < n) {
-    const float rs = 1.f / sqrtf((row_sum[0][t] + row_sum[1][t]) / (float)p.dk + p.eps);
+    const float rs = 1.f / sqrtf((row_sum[0][t] + row_sum[1][t]) / (float)p.dv + p.eps);
     const float* w = p.norm + h * p.VP + half * HC;
     __nv_bfloat16* dst = p.out + (long long)(row0 + t) * p.ldo + h * p.VP + half * HC;
 #pragma unroll
@@ -1581,7 +1761,8 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
       const float4 w0 = *reinterpret_cast<const float4*>(w + i * 8), w1 = *reinterpret_cast<const float4*>(w + i * 8 + 4);
       auto two = [&](int e, float wx, float wy, uint32_t gz) {
         const float2 z = unpack_bf16x2(gz);
-        return pack_bf16x2(__uint_as_float(v[i * 8 + e]) * rs * wx * silu_fast(z.x), __uint_as_float(v[i * 8 + e + 1]) * rs * wy * silu_fast(z.y));
+        const float gx = FORGET ? 1.f : silu_fast(z.x), gy = FORGET ? 1.f : silu_fast(z.y);
+        return pack_bf16x2(__uint_as_float(v[i * 8 + e]) * rs * wx * gx, __uint_as_float(v[i * 8 + e + 1]) * rs * wy * gy);
       };
       *reinterpret_cast<uint4*>(dst + i * 8) = make_uint4(two(0, w0.x, w0.y, gate[i].x), two(2, w0.z, w0.w, gate[i].y), two(4, w1.x, w1.y, gate[i].z),
                                                           two(6, w1.z, w1.w, gate[i].w));
@@ -1593,25 +1774,31 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
   }
 }
 
-template <int DK>
+template <int DK, bool FORGET>
 static int launch_time_mix(const MixParams& p, int n_chunks, int n_seq, cudaStream_t stream) {
   static bool attr[64] = {};
   int dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
   if (!attr[dev]) {
-    if (cudaFuncSetAttribute(time_mix_state_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixStateCfg<DK>::kSmem) != cudaSuccess ||
-        cudaFuncSetAttribute(time_mix_out_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixOutCfg<DK>::kSmem) != cudaSuccess)
+    if (cudaFuncSetAttribute(time_mix_state_kernel<DK, FORGET>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixStateCfg<DK>::kSmem) != cudaSuccess ||
+        cudaFuncSetAttribute(time_mix_out_kernel<DK, FORGET>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixOutCfg<DK>::kSmem) != cudaSuccess)
       return -10;
     attr[dev] = true;
   }
   const dim3 units(n_chunks * p.H);
-  if (launch_kernel(time_mix_state_kernel<DK>, units, dim3(CHT), MixStateCfg<DK>::kSmem, stream, p) != cudaSuccess) return -11;
+  if (launch_kernel(time_mix_state_kernel<DK, FORGET>, units, dim3(CHT), MixStateCfg<DK>::kSmem, stream, p) != cudaSuccess) return -11;
   if (launch_kernel(time_mix_chain_kernel, dim3(DK / 32, p.H * (p.VP / SC_COLS), n_seq), dim3(256), 0, stream, p) != cudaSuccess) return -12;
-  return launch_kernel(time_mix_out_kernel<DK>, units, dim3(CHT), MixOutCfg<DK>::kSmem, stream, p) == cudaSuccess ? 0 : -13;
+  return launch_kernel(time_mix_out_kernel<DK, FORGET>, units, dim3(CHT), MixOutCfg<DK>::kSmem, stream, p) == cudaSuccess ? 0 : -13;
 }
 
+}  // namespace rb
+
+#include "delta_rule.cuh"
+
+namespace rb {
+
 // ------------------------------------------------------------------------------------------
-// Time mixing, one token per sequence, heads of up to 64 channels (KP = VP = 64): a unit is a whole head of a sequence, so that its
+// Time or forget mixing, one token per sequence, heads of up to 64 channels (KP = VP = 64): a unit is a whole head of a sequence, so that its
 // norm and the output gate are finished here too. As recurrent_decode_kernel: persistent CTAs, a ring of bulk copies in both
 // directions, the unit's vectors fetched one unit ahead. Threads: 16 groups of 4 value channels x 8 of key rows.
 // ------------------------------------------------------------------------------------------
@@ -1633,11 +1820,11 @@ struct MixDecodeParams {
   const int* seq_lens;
   void* out;                     // [B, ldo]
   long long ldo;
-  int H, dk, num_slots;
+  int H, dk, dv, num_slots;
   int* status;
 };
 
-template <typename T>
+template <typename T, bool FORGET>
 __global__ void __launch_bounds__(MD_THREADS) time_mix_decode_kernel(const MixDecodeParams p, int units) {
   extern __shared__ __align__(128) uint8_t smem_raw[];       // MD_STAGES x [2, 64, 32] fp32
   __shared__ __align__(16) float4 rows_s[MD_DIM];            // r, k, decay, bonus of a key row
@@ -1686,12 +1873,12 @@ __global__ void __launch_bounds__(MD_THREADS) time_mix_decode_kernel(const MixDe
     const T* row = reinterpret_cast<const T*>(p.proj) + x.b * p.ld + x.h * MD_DIM;
     const int c = x.h * MD_DIM;
     if (tid < MD_DIM) {
-      mine = make_float4(to_f<T>(row[tid]), to_f<T>(row[p.k_col + tid]), p.z[x.b * p.ldz + c + tid] + p.w0[c + tid], p.bonus[c + tid]);
+      mine = make_float4(to_f<T>(row[tid]), FORGET ? 0.f : to_f<T>(row[p.k_col + tid]), p.z[x.b * p.ldz + c + tid] + p.w0[c + tid], p.bonus[c + tid]);
     } else {
       mine.x = to_f<T>(row[p.v_col + tid - MD_DIM]);
     }
     if (warp == 0) {
-      gate = make_float2(to_f<T>(row[p.g_col + 2 * lane]), to_f<T>(row[p.g_col + 2 * lane + 1]));
+      if (!FORGET) gate = make_float2(to_f<T>(row[p.g_col + 2 * lane]), to_f<T>(row[p.g_col + 2 * lane + 1]));
       weight = *reinterpret_cast<const float2*>(p.norm + c + 2 * lane);
     }
   };
@@ -1701,8 +1888,14 @@ __global__ void __launch_bounds__(MD_THREADS) time_mix_decode_kernel(const MixDe
   for (int u = blockIdx.x; u < units; u += gridDim.x, ++it) {
     const Unit cur = x;
     const float2 g = gate, w = weight;
-    if (tid < MD_DIM) rows_s[tid] = make_float4(mine.x, mine.y, channel_decay(mine.z), mine.w);
-    else vs[tid - MD_DIM] = mine.x;
+    if (tid < MD_DIM) {
+      if (FORGET) {
+        const float2 f = forget_gate(mine.z, mine.w);
+        rows_s[tid] = tid < p.dk ? make_float4(mine.x, f.y, f.x, 0.f) : make_float4(0.f, 0.f, 0.f, 0.f);
+      } else {
+        rows_s[tid] = make_float4(mine.x, mine.y, channel_decay(mine.z), mine.w);
+      }
+    } else vs[tid - MD_DIM] = mine.x;
     const int stage = it % MD_STAGES;
     ok = mbar_wait_bounded(smem_u32(&full[stage]), (uint32_t)((it / MD_STAGES) & 1), &abort_flag, p.status, ST_TIMEOUT_SMEM_FULL);
     ok = __syncthreads_and(ok);
@@ -1717,14 +1910,22 @@ __global__ void __launch_bounds__(MD_THREADS) time_mix_decode_kernel(const MixDe
       float4 s = cur.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : S[r * 8];
       const float4 q = rows_s[r];
       const float4 kv = make_float4(q.y * v.x, q.y * v.y, q.y * v.z, q.y * v.w);
-      acc.x = fmaf(q.x, fmaf(q.w, kv.x, s.x), acc.x);
-      acc.y = fmaf(q.x, fmaf(q.w, kv.y, s.y), acc.y);
-      acc.z = fmaf(q.x, fmaf(q.w, kv.z, s.z), acc.z);
-      acc.w = fmaf(q.x, fmaf(q.w, kv.w, s.w), acc.w);
+      if (!FORGET) {
+        acc.x = fmaf(q.x, fmaf(q.w, kv.x, s.x), acc.x);
+        acc.y = fmaf(q.x, fmaf(q.w, kv.y, s.y), acc.y);
+        acc.z = fmaf(q.x, fmaf(q.w, kv.z, s.z), acc.z);
+        acc.w = fmaf(q.x, fmaf(q.w, kv.w, s.w), acc.w);
+      }
       s.x = fmaf(q.z, s.x, kv.x);
       s.y = fmaf(q.z, s.y, kv.y);
       s.z = fmaf(q.z, s.z, kv.z);
       s.w = fmaf(q.z, s.w, kv.w);
+      if (FORGET) {
+        acc.x = fmaf(q.x, s.x, acc.x);
+        acc.y = fmaf(q.x, s.y, acc.y);
+        acc.z = fmaf(q.x, s.z, acc.z);
+        acc.w = fmaf(q.x, s.w, acc.w);
+      }
       S[r * 8] = s;
     }
     fence_proxy_async_smem();
@@ -1748,8 +1949,8 @@ __global__ void __launch_bounds__(MD_THREADS) time_mix_decode_kernel(const MixDe
         o.x += part.x;
         o.y += part.y;
       }
-      const float rs = cur.slot < 0 ? 0.f : 1.f / sqrtf(warp_sum(o.x * o.x + o.y * o.y) / (float)p.dk + p.eps);
-      const float y0 = o.x * rs * w.x * g.x * sigmoid_f(g.x), y1 = o.y * rs * w.y * g.y * sigmoid_f(g.y);
+      const float rs = cur.slot < 0 ? 0.f : 1.f / sqrtf(warp_sum(o.x * o.x + o.y * o.y) / (float)p.dv + p.eps);
+      const float y0 = o.x * rs * w.x * (FORGET ? 1.f : g.x * sigmoid_f(g.x)), y1 = o.y * rs * w.y * (FORGET ? 1.f : g.y * sigmoid_f(g.y));
       T* dst = reinterpret_cast<T*>(p.out) + cur.b * p.ldo + cur.h * MD_DIM + 2 * lane;
       if constexpr (sizeof(T) == 4) *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
       else *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(y0, y1);
@@ -1766,7 +1967,7 @@ __global__ void __launch_bounds__(MD_THREADS) time_mix_decode_kernel(const MixDe
   }
 }
 
-template <typename T>
+template <typename T, bool FORGET>
 static int launch_time_mix_decode(const MixDecodeParams& p, int B, cudaStream_t stream) {
   static int sms[64] = {};
   int dev = 0;
@@ -1774,16 +1975,16 @@ static int launch_time_mix_decode(const MixDecodeParams& p, int B, cudaStream_t 
   if (sms[dev] == 0) {
     int n = 0;
     if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess ||
-        cudaFuncSetAttribute(time_mix_decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, MD_STAGES * MD_BYTES) != cudaSuccess)
+        cudaFuncSetAttribute(time_mix_decode_kernel<T, FORGET>, cudaFuncAttributeMaxDynamicSharedMemorySize, MD_STAGES * MD_BYTES) != cudaSuccess)
       return -10;
     sms[dev] = n;
   }
   const int units = B * p.H, grid = units < sms[dev] * 3 ? units : sms[dev] * 3;
-  return launch_kernel(time_mix_decode_kernel<T>, dim3(grid), dim3(MD_THREADS), MD_STAGES * MD_BYTES, stream, p, units) == cudaSuccess ? 0 : -11;
+  return launch_kernel(time_mix_decode_kernel<T, FORGET>, dim3(grid), dim3(MD_THREADS), MD_STAGES * MD_BYTES, stream, p, units) == cudaSuccess ? 0 : -11;
 }
 
 // ------------------------------------------------------------------------------------------
-// out = o / rms * weight * sigmoid(gate), or silu(gate). One CTA per token; a warp takes whole heads. Padding channels of o are zero.
+// out = o / rms * weight * sigmoid(gate), or silu(gate), or without a gate (null). One CTA per token; a warp takes whole heads. Padding channels of o are zero.
 template <typename T>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ weight,
                                                          const T* __restrict__ gate, long long ldg, T* __restrict__ out, long long ldy,
@@ -1823,9 +2024,13 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
       const float4 v = *reinterpret_cast<const float4*>(x + c);
       const float4 w = *reinterpret_cast<const float4*>(weight + c);
       const T* g = gate + t * ldg + c;
-      auto gated = [&](float z) { return silu ? z * sigmoid_f(z) : sigmoid_f(z); };
-      const float y0 = v.x * rs * w.x * gated(to_f<T>(g[0])), y1 = v.y * rs * w.y * gated(to_f<T>(g[1]));
-      const float y2 = v.z * rs * w.z * gated(to_f<T>(g[2])), y3 = v.w * rs * w.w * gated(to_f<T>(g[3]));
+      auto gated = [&](int e) {
+        if (gate == nullptr) return 1.f;
+        const float z = to_f<T>(g[e]);
+        return silu ? z * sigmoid_f(z) : sigmoid_f(z);
+      };
+      const float y0 = v.x * rs * w.x * gated(0), y1 = v.y * rs * w.y * gated(1);
+      const float y2 = v.z * rs * w.z * gated(2), y3 = v.w * rs * w.w * gated(3);
       if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(out + t * ldy + c) = make_float4(y0, y1, y2, y3);
       else *reinterpret_cast<uint2*>(out + t * ldy + c) = make_uint2(pack_bf16x2(y0, y1), pack_bf16x2(y2, y3));
     }
@@ -1935,19 +2140,30 @@ void rb_recurrent_set_pdl(int on) { rb::pdl_enabled() = on != 0; }
 int rb_recurrent_scan(const void* proj, long long ld, int q_col, int k_col, int v_col, const float* small, long long ld_small, const float* decay,
                       const float* bias_i, const float* bias_f, float cap, float q_scale, float* s, float* n, float* m, const int* slots,
                       const int* cu_q, const int* seq_lens, float* out, long long ldo, int H, int dk, int KP, int VP, int B, int num_slots,
-                      int gated, int rows, const float* z, long long ldz, const float* w0, const float* bonus, int dtype, int* status,
-                      cudaStream_t stream) {
+                      int gated, int rows, const float* z, long long ldz, const float* w0, const float* bonus, int form, int ratio,
+                      const float* units, const float* steps, int dtype, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
-  const bool mix = z != nullptr;
-  if (H <= 0 || H > 65535 || B > 65535 || dk <= 0 || dk > KP || VP % SC_COLS != 0) return -1;
-  if (mix ? (gated || w0 == nullptr || bonus == nullptr) : (gated ? small == nullptr : decay == nullptr)) return -1;
+  if (H <= 0 || H > 65535 || B > 65535 || dk <= 0 || dk > KP || VP % SC_COLS != 0 || ratio <= 0 || H % ratio != 0) return -1;
+  if (form == FORM_DELTA ? (gated || units == nullptr || steps == nullptr) : ratio != 1) return -1;
+  if (form == FORM_MIX || form == FORM_FORGET) {
+    if (gated || z == nullptr || w0 == nullptr || bonus == nullptr) return -1;
+  } else if (form == FORM_PLAIN && (gated ? small == nullptr : decay == nullptr)) {
+    return -1;
+  }
   const ScanParams p{proj, ld, q_col, k_col, v_col, small, ld_small, decay, bias_i, bias_f, cap, q_scale, s, n, m, slots, cu_q, seq_lens,
-                     out, ldo, H, dk, KP, VP, num_slots, gated, rows, z, ldz, w0, bonus, status};
-  if (cu_q == nullptr && dk <= RD_MAX_DK && B <= RD_MAX_B)
-    return mix ? (dtype == 0 ? launch_decode<__nv_bfloat16, true>(p, B, stream) : launch_decode<float, true>(p, B, stream))
-               : (dtype == 0 ? launch_decode<__nv_bfloat16, false>(p, B, stream) : launch_decode<float, false>(p, B, stream));
-  return mix ? (dtype == 0 ? launch_scan<__nv_bfloat16, true>(p, B, stream) : launch_scan<float, true>(p, B, stream))
-             : (dtype == 0 ? launch_scan<__nv_bfloat16, false>(p, B, stream) : launch_scan<float, false>(p, B, stream));
+                     out, ldo, H, dk, KP, VP, num_slots, gated, rows, z, ldz, w0, bonus, status, ratio, units, steps};
+  const bool single = cu_q == nullptr && dk <= RD_MAX_DK && B <= RD_MAX_B;
+#define RB_FORM(FORM)                                                                                                                        \
+  return single ? (dtype == 0 ? launch_decode<__nv_bfloat16, FORM>(p, B, stream) : launch_decode<float, FORM>(p, B, stream))               \
+                : (dtype == 0 ? launch_scan<__nv_bfloat16, FORM>(p, B, stream) : launch_scan<float, FORM>(p, B, stream))
+  switch (form) {
+    case FORM_PLAIN: RB_FORM(FORM_PLAIN);
+    case FORM_MIX: RB_FORM(FORM_MIX);
+    case FORM_FORGET: RB_FORM(FORM_FORGET);
+    case FORM_DELTA: RB_FORM(FORM_DELTA);
+    default: return -1;
+  }
+#undef RB_FORM
 }
 
 // Workspace of the chunked form in bytes.
@@ -1973,6 +2189,7 @@ int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, in
   p.chunks = (const int4*)chunks; p.seq_chunks = seq_chunks; p.slots = slots; p.seq_lens = seq_lens; p.cu_q = cu_q;
   p.s = s; p.n = n; p.m = m; p.out = out; p.ldo = ldo;
   p.H = H; p.dk = dk; p.KP = KP; p.VP = VP; p.num_slots = num_slots; p.gated = gated; p.status = status;
+  p.v = p.proj + v_col; p.ld_v = ld; p.ratio = 1;
   float* w = (float*)workspace;
   p.u = w; w += ch * KP * VP;
   p.s_hi = (__nv_bfloat16*)w; w += ch * KP * VP / 2;
@@ -1991,15 +2208,16 @@ int rb_recurrent_chunks(const void* proj, long long ld, int q_col, int k_col, in
   }
 }
 
-// Time mixing of one token per sequence down to the normed and gated output rows; heads padded to 64 channels. Activations and out
+// Time mixing (forget: forget mixing, bonus holds the lower bounds) of one token per sequence down to the normed and gated output rows; heads padded to 64 channels. Activations and out
 // in bf16 (dtype 0) or fp32.
 int rb_time_mix_decode(const void* proj, long long ld, int k_col, int v_col, int g_col, const float* z, long long ldz, const float* w0,
                        const float* bonus, const float* norm, float eps, float* s, const int* slots, const int* seq_lens, void* out, long long ldo,
-                       int B, int H, int dk, int num_slots, int dtype, int* status, cudaStream_t stream) {
+                       int B, int H, int dk, int dv, int num_slots, int forget, int dtype, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
-  if (H <= 0 || dk <= 0 || dk > MD_DIM || ldo % 2 != 0) return -1;
-  const MixDecodeParams p{proj, ld, k_col, v_col, g_col, z, ldz, w0, bonus, norm, eps, s, slots, seq_lens, out, ldo, H, dk, num_slots, status};
-  return dtype == 0 ? launch_time_mix_decode<__nv_bfloat16>(p, B, stream) : launch_time_mix_decode<float>(p, B, stream);
+  if (H <= 0 || dk <= 0 || dk > MD_DIM || dv <= 0 || dv > MD_DIM || ldo % 2 != 0) return -1;
+  const MixDecodeParams p{proj, ld, k_col, v_col, g_col, z, ldz, w0, bonus, norm, eps, s, slots, seq_lens, out, ldo, H, dk, dv, num_slots, status};
+  if (forget) return dtype == 0 ? launch_time_mix_decode<__nv_bfloat16, true>(p, B, stream) : launch_time_mix_decode<float, true>(p, B, stream);
+  return dtype == 0 ? launch_time_mix_decode<__nv_bfloat16, false>(p, B, stream) : launch_time_mix_decode<float, false>(p, B, stream);
 }
 
 // Workspace of the chunked time mixing in bytes.
@@ -2009,32 +2227,95 @@ long long rb_time_mix_workspace(int n_chunks, int H, int KP) {
 }
 
 // Chunked time mixing of whole portions, as rb_recurrent_chunks, down to the normed and gated output rows (bf16). z [T, ldz] is
-// overwritten. KP is 64 or 128; values have as many channels as keys.
+// overwritten. KP is 64 or 128; values have as many (padded) channels as keys. keys not null: forget mixing, which leaves its keys there.
 int rb_time_mix_chunks(const void* proj, long long ld, int k_col, int v_col, int g_col, float* z, long long ldz, const float* w0, const float* bonus,
                        float* s, const void* chunks, const int* seq_chunks, const int* slots, const int* cu_q, const int* seq_lens, const float* norm,
-                       float eps, void* out, long long ldo, void* workspace, int n_chunks, int n_seq, int H, int dk, int KP, int num_slots, int* status,
-                       cudaStream_t stream) {
+                       float eps, void* out, long long ldo, void* workspace, void* keys, long long ld_keys, int n_chunks, int n_seq, int H, int dk,
+                       int dv, int KP, int num_slots, int* status, cudaStream_t stream) {
   if (n_chunks <= 0 || n_seq <= 0) return 0;
   if (H <= 0 || H * (KP / SC_COLS) > 65535 || n_seq > 65535 || dk <= 0 || dk > KP || ld % 8 != 0 || ldo % 8 != 0 || ldz % 4 != 0 || workspace == nullptr ||
-      (k_col | v_col | g_col) % 8 != 0)
+      (k_col | v_col | g_col) % 8 != 0 || dv <= 0 || dv > KP || ld_keys % 8 != 0)
     return -1;
   const long long ch = (long long)n_chunks * H;
   MixParams p{};
   p.proj = (const __nv_bfloat16*)proj; p.ld = ld; p.k_col = k_col; p.v_col = v_col; p.g_col = g_col;
   p.z = z; p.ldz = ldz; p.w0 = w0; p.bonus = bonus; p.chunks = (const int4*)chunks; p.seq_chunks = seq_chunks; p.slots = slots;
   p.seq_lens = seq_lens; p.cu_q = cu_q; p.s = s; p.norm = norm; p.eps = eps; p.out = (__nv_bfloat16*)out; p.ldo = ldo;
-  p.H = H; p.dk = dk; p.KP = KP; p.VP = KP; p.num_slots = num_slots; p.status = status;
+  p.H = H; p.dk = dk; p.dv = dv; p.KP = KP; p.VP = KP; p.num_slots = num_slots; p.status = status;
+  p.keys = (__nv_bfloat16*)keys; p.ld_keys = ld_keys;
   float* w = (float*)workspace;
   p.u = w; w += ch * KP * KP;
   p.s_hi = (__nv_bfloat16*)w; w += ch * KP * KP / 2;
   p.s_lo = (__nv_bfloat16*)w; w += ch * KP * KP / 2;
   p.last = w;
-  if (KP == 64) return launch_time_mix<64>(p, n_chunks, n_seq, stream);
-  return KP == 128 ? launch_time_mix<128>(p, n_chunks, n_seq, stream) : -1;
+  const bool forget = keys != nullptr;
+  if (KP == 64) return forget ? launch_time_mix<64, true>(p, n_chunks, n_seq, stream) : launch_time_mix<64, false>(p, n_chunks, n_seq, stream);
+  if (KP == 128) return forget ? launch_time_mix<128, true>(p, n_chunks, n_seq, stream) : launch_time_mix<128, false>(p, n_chunks, n_seq, stream);
+  return -1;
+}
+
+// Rows of the delta rule between the joint projection and the recurrence (see DeltaRows); cu_q null: one row per sequence. With cu_q the
+// histories move on in a second launch.
+int rb_delta_rows(const void* proj, long long ld, const float* conv, int taps, void* hist, const int* cu_q, const int* positions, const int* slots, int B,
+                  int num_slots, void* out, long long ldo, const float* small, long long ld_small, const float* rate, const float* dt_bias, float* units,
+                  float* steps, int G, int H, int KP, int VP, int T, int dtype, int* status, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (G <= 0 || H <= 0 || H % G != 0 || KP % 64 != 0 || VP % 64 != 0 || KP > 512 || VP > 512 || taps < 1 || taps > 16 || (taps > 1 && hist == nullptr) ||
+      ld % 8 != 0 || ldo % 8 != 0 || B <= 0)
+    return -1;
+  DeltaRows p{proj, ld, conv, taps, hist, History{cu_q, positions, slots, B, taps - 1, num_slots}, out, ldo, small, ld_small, rate, dt_bias, units, steps,
+              G, H, KP, VP, T, 1, status};
+  if (cu_q != nullptr) {                                   // long enough runs that a look back is seldom fetched, enough of them to fill the machine
+    const long long run = (long long)T * (2 * G + H) / (148 * 32);
+    p.run = run < 1 ? 1 : run > 16 ? 16 : (int)run;
+  }
+  cudaError_t e = dtype == 0 ? launch_delta_rows<__nv_bfloat16>(p, stream) : launch_delta_rows<float>(p, stream);
+  const int channels = 2 * G * KP + H * VP;
+  if (e == cudaSuccess && cu_q != nullptr && taps > 1)
+    e = dtype == 0 ? launch_history_update((const __nv_bfloat16*)proj, ld, p.rows, (__nv_bfloat16*)hist, channels, stream)
+                   : launch_history_update((const float*)proj, ld, p.rows, (float*)hist, channels, stream);
+  return e == cudaSuccess ? 0 : -11;
+}
+
+// Workspace of the chunked delta rule in bytes.
+long long rb_delta_workspace(int n_chunks, int H, int KP, int VP) {
+  const long long ch = (long long)n_chunks * H;
+  return ch * ((long long)KP * VP * 4 + CH * KP * 4 + CH * VP * 4 + 3 * CH * 4 + 8) + 256;
+}
+
+// The delta rule over whole portions in chunks, as rb_recurrent_chunks. rows [T, q | k | v] bf16, `values` [T, H * VP] bf16 is room for what is
+// written into the state. KP is 64 or 128.
+int rb_delta_chunks(const void* rows, long long ld, int k_col, int v_col, const float* units, const float* steps, float q_scale, float* s, const void* chunks,
+                    const int* seq_chunks, const int* slots, const int* cu_q, const int* seq_lens, void* values, long long ld_values, float* out,
+                    long long ldo, void* workspace, int n_chunks, int n_seq, int H, int ratio, int dk, int KP, int VP, int num_slots, int* status,
+                    cudaStream_t stream) {
+  if (n_chunks <= 0 || n_seq <= 0) return 0;
+  if (H <= 0 || H > 65535 || n_seq > 65535 || ratio <= 0 || H % ratio != 0 || dk <= 0 || dk > KP || VP % 64 != 0 || ld % 8 != 0 || ld_values % 8 != 0 ||
+      ldo % 4 != 0 || k_col % 8 != 0 || v_col % 8 != 0 || workspace == nullptr)
+    return -1;
+  const long long ch = (long long)n_chunks * H;
+  DeltaParams p{};
+  ChunkParams& c = p.c;
+  c.proj = (const __nv_bfloat16*)rows; c.ld = ld; c.q_col = 0; c.k_col = k_col; c.v_col = v_col; c.q_scale = q_scale;
+  c.chunks = (const int4*)chunks; c.seq_chunks = seq_chunks; c.slots = slots; c.seq_lens = seq_lens; c.cu_q = cu_q;
+  c.s = s; c.out = out; c.ldo = ldo;
+  c.H = H; c.dk = dk; c.KP = KP; c.VP = VP; c.num_slots = num_slots; c.status = status;
+  c.v = c.proj + v_col; c.ld_v = ld; c.ratio = ratio; c.factors = 1;
+  p.units = units; p.steps = steps; p.values = (__nv_bfloat16*)values; p.ld_values = ld_values;
+  float* w = (float*)workspace;
+  p.uv = w; w += ch * CH * VP;
+  c.s_hi = (__nv_bfloat16*)w; w += ch * KP * VP / 2;
+  c.s_lo = (__nv_bfloat16*)w; w += ch * KP * VP / 2;
+  p.w_hi = (__nv_bfloat16*)w; w += ch * CH * KP / 2;
+  p.w_lo = (__nv_bfloat16*)w; w += ch * CH * KP / 2;
+  c.gates = w; w += ch * 3 * CH;
+  c.um = (float2*)w;
+  if (KP == 64) return launch_delta_chunks<64>(p, n_chunks, n_seq, stream);
+  return KP == 128 ? launch_delta_chunks<128>(p, n_chunks, n_seq, stream) : -1;
 }
 
 int rb_gated_norm(const float* o, long long ldo, const float* weight, const void* gate, long long ldg, void* out, long long ldy, int H, int dv,
-                  int VP, int per_head, int silu, int T, int dtype, float eps, cudaStream_t stream) {
+                  int VP, int per_head, int silu, int T, int dtype, float eps, cudaStream_t stream) {      // gate may be null
   if (T <= 0) return 0;
   if (VP % 4 != 0 || ldo % 4 != 0 || ldy % 4 != 0) return -1;
   cudaError_t e;

@@ -5,15 +5,16 @@ every layer of its kind (``make`` / ``load``), the cache or state of every run o
 activations (``allocate``), plans a step for all its layers at once (``plan``) and runs one layer (``forward``).
 """
 
-from ...models.stack import (ClampedGluSpec, ExpertsSpec, GluSpec, GroupedAttentionSpec, KeyValueAttentionSpec, LatentAttentionSpec, LightningSpec,
-                             MatrixMemorySpec, ParallelSpec, TimeMixSpec)
-from .feedforward import DensePart, ExpertsPart
+from ...models.stack import (ClampedGluSpec, DeltaRuleSpec, ExpertsSpec, GluSpec, GroupedAttentionSpec, KeyValueAttentionSpec, LatentAttentionSpec,
+                             LightningSpec, MatrixMemorySpec, NormedPairSpec, ParallelSpec, PolyNormSpec, TimeMixSpec)
+from .feedforward import DensePart, ExpertsPart, PolyNormPart
 from .grouped import GroupedPart
 from .keyvalue import KeyValuePart
 from .latent import LatentPart
-from .parallel import ParallelPart
-from .recurrent import RecurrentPart, TimeMixPart
+from .parallel import NormedPairPart, ParallelPart
+from .recurrent import DeltaPart, RecurrentPart, TimeMixPart
 
 MIXER_PARTS = {LatentAttentionSpec: LatentPart, KeyValueAttentionSpec: KeyValuePart, LightningSpec: RecurrentPart, MatrixMemorySpec: RecurrentPart,
-               GroupedAttentionSpec: GroupedPart, TimeMixSpec: TimeMixPart, ParallelSpec: ParallelPart}
-FEED_FORWARD_PARTS = {ClampedGluSpec: DensePart, GluSpec: DensePart, ExpertsSpec: ExpertsPart}
+               GroupedAttentionSpec: GroupedPart, TimeMixSpec: TimeMixPart, ParallelSpec: ParallelPart, NormedPairSpec: NormedPairPart,
+               DeltaRuleSpec: DeltaPart}
+FEED_FORWARD_PARTS = {ClampedGluSpec: DensePart, GluSpec: DensePart, PolyNormSpec: PolyNormPart, ExpertsSpec: ExpertsPart}

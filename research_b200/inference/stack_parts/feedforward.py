@@ -1,12 +1,12 @@
 """Feed-forwards as parts of a layer stack: a gated unit, clamped or plain SiLU, dense (gate|up with the unit in the GEMM's epilogue,
-down) or as routed experts (``ops/experts.py``) with or without a shared one."""
+down) or as routed experts (``ops/experts.py``) with or without a shared one; two matrices with normed powers between them."""
 
 from __future__ import annotations
 
 import torch
 
 from ... import ops
-from ...models.stack import ClampedGluSpec, ExpertsSpec, GluSpec
+from ...models.stack import ClampedGluSpec, ExpertsSpec, GluSpec, PolyNormSpec
 from ...ops.experts import ExpertsGeometry, ExpertsScratch
 from .base import Part, up
 
@@ -57,21 +57,53 @@ class DensePart(Part):
         return {"y2": y}
 
 
+class PolyNormWeights:
+    __slots__ = ("spec", "wu", "wd", "act", "ffp")
+
+
+class PolyNormPart(Part):
+    def make(self, spec: PolyNormSpec) -> PolyNormWeights:
+        w = PolyNormWeights()
+        w.spec, w.ffp = spec, up(spec.ff, 8)
+        w.wu, w.wd = self.zeros(w.ffp, self.r.wp), self.zeros(self.r.wp, w.ffp)
+        w.act = self.zeros(4, dtype=torch.float32)
+        self.layers.append(w)
+        return w
+
+    def allocate(self) -> None:
+        self.z, self.a = (self.zeros(self.r.rows * max(w.ffp for w in self.layers)) for _ in range(2))
+
+    def load(self, w: PolyNormWeights, get, p: str) -> None:
+        ff, d = w.spec.ff, self.r.cfg.hidden_size
+        w.wu[:ff, :d].copy_(get(p + "up"))
+        w.wd[:d, :ff].copy_(get(p + "down"))
+        w.act.copy_(get(p + "act").float())
+
+    def forward(self, w: PolyNormWeights, inp, y, small=None) -> dict:
+        T = inp.shape[0]
+        z, a = (t[:T * w.ffp].view(T, w.ffp) for t in (self.z, self.a))
+        ops.gemm(inp, w.wu, out=z)
+        ops.poly_norm(z, w.act, w.spec.ff, self.r.cfg.norm_eps, a)
+        ops.gemm(a, w.wd, out=y, out_f32=True)
+        return {"y2": y}
+
+
 class ExpertsWeights:
-    __slots__ = ("spec", "geo", "wgu", "wd", "shared")
+    __slots__ = ("spec", "geo", "wgu", "wd", "shared", "correction")
 
 
 class ExpertsPart(Part):
     @staticmethod
     def small_rows(spec: ExpertsSpec) -> int:
-        return spec.experts
+        return spec.choices + int(spec.routing.shared_gate and spec.shared is not None)
 
     def make(self, spec: ExpertsSpec) -> ExpertsWeights:
         r = self.r
         w = ExpertsWeights()
         w.spec = spec
         how = spec.routing
-        w.geo = ExpertsGeometry.make(spec.experts, spec.top, spec.expert.ff, r.wp, spec.expert.limit, r.dtype, how.scores, how.normalize, how.scale_input)
+        w.geo = ExpertsGeometry.make(spec.experts, spec.top, spec.expert.ff, r.wp, spec.expert.limit, r.dtype, how.scores, how.normalize, how.scale_input, spec.identity)
+        w.correction = self.zeros(spec.choices, dtype=torch.float32) if how.correction else None
         w.shared = r._part(DensePart).make(spec.shared) if spec.shared is not None else None
         w.wgu, w.wd = self.zeros(spec.experts * 2 * w.geo.ffp, r.wp), self.zeros(spec.experts * r.wp, w.geo.ffp)
         self.layers.append(w)
@@ -83,13 +115,24 @@ class ExpertsPart(Part):
     def load(self, w: ExpertsWeights, get, p: str) -> None:
         n = range(w.spec.experts)
         ops.pack_experts((get(f"{p}e{e}.gate") for e in n), (get(f"{p}e{e}.up") for e in n), (get(f"{p}e{e}.down") for e in n), w.geo, w.wgu, w.wd)
+        if w.correction is not None:
+            w.correction.copy_(get(p + "correction").float())
         if w.shared is not None:
             self.r._part(DensePart).load(w.shared, get, p + "shared.")
 
     def load_small(self, w: ExpertsWeights, get, p: str, dst: torch.Tensor) -> None:
-        dst[:w.spec.experts, :self.r.cfg.hidden_size].copy_(get(p + "router"))
+        n, d = w.spec.choices, self.r.cfg.hidden_size
+        dst[:n, :d].copy_(get(p + "router"))
+        if self.small_rows(w.spec) > n:
+            dst[n:n + 1, :d].copy_(get(p + "shared.sg"))
 
     def forward(self, w: ExpertsWeights, inp, y, small) -> dict:
-        e, p = ops.experts_forward(inp, small, w.geo, self.scratch[w.geo], w.wgu, w.wd)
-        add = {"experts": e, "expert_weights": p, "top": w.geo.top}
+        sc = self.scratch[w.geo]
+        e, p = ops.experts_forward(inp, small, w.geo, sc, w.wgu, w.wd, w.correction)
+        if self.r.sandwich:
+            add = {"chosen": ops.ChosenExperts(e, p, sc.idx[:inp.shape[0]], w.geo.experts, inp)}
+            if w.shared is not None and w.spec.routing.shared_gate:
+                add["gate"] = small[:, w.spec.choices:]
+        else:
+            add = {"experts": e, "expert_weights": p, "top": w.geo.top}
         return {**self.r._part(DensePart).forward(w.shared, inp, y), **add} if w.shared is not None else add

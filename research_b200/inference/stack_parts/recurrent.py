@@ -10,8 +10,9 @@ from dataclasses import dataclass
 import torch
 
 from ... import ops
-from ...models.stack import LightningSpec, MatrixMemorySpec, TimeMixSpec
-from ...ops.recurrent import MAX_DIM, ChunkTable, RecurrentGeometry, RecurrentState, TimeMix, chunk_workspace, chunked_supported, time_mix_chunked_supported, time_mix_workspace
+from ...models.stack import DeltaRuleSpec, ForgetMixSpec, LightningSpec, MatrixMemorySpec, TimeMixSpec
+from ...ops.recurrent import (MAX_DIM, MAX_TAPS, ChunkTable, DeltaRule, ForgetMix, RecurrentGeometry, RecurrentState, TimeMix, chunk_workspace,
+                              chunked_supported, delta_chunked_supported, delta_workspace, time_mix_chunked_supported, time_mix_workspace)
 from .base import Part, load_head_columns, load_head_vector, load_heads, up
 
 SCAN_PORTION = 16            # new tokens of a sequence up to which the recurrence runs token by token
@@ -241,4 +242,188 @@ class TimeMixPart(Part):
         T, n = b.num_tokens, w.geo.heads * w.geo.vp
         out = self.out[:T * n].view(T, n)
         self.mix(w, cache, inp, out, b, plan)
+        ops.gemm(out, w.wo, out=y, out_f32=True)
+
+
+class ForgetMixWeights:
+    __slots__ = ("geo", "spec", "wproj", "bias", "lower", "norm", "wo")
+
+
+class ForgetMixPart(Part):
+    """Forget mixing beside another mixer (``parallel.py``), which makes the joint projection."""
+
+    @staticmethod
+    def geometry(spec: ForgetMixSpec) -> RecurrentGeometry:
+        return RecurrentGeometry(spec.heads, spec.dim, spec.vdim, silu=True, gated=False, form="forget")
+
+    @staticmethod
+    def state_floats(spec) -> int:
+        return ForgetMixPart.geometry(spec).state_floats
+
+    def make(self, spec: ForgetMixSpec) -> ForgetMixWeights:
+        g, f32 = self.geometry(spec), torch.float32
+        if g.kp > MAX_DIM:
+            raise ValueError(f"the recurrent kernels take up to {MAX_DIM} key channels per head")
+        w = ForgetMixWeights()
+        w.spec, w.geo, w.wproj = spec, g, None
+        w.bias, w.lower = (self.zeros(g.heads * g.kp, dtype=f32) for _ in range(2))
+        w.norm, w.wo = self.zeros(g.heads * g.vp, dtype=f32), self.zeros(self.r.wp, g.heads * g.vp)
+        self.layers.append(w)
+        return w
+
+    def new_cache(self, w: ForgetMixWeights) -> RecurrentState:
+        return RecurrentState.zeros(w.geo, self.r.scratch_state_slot + 1, self.r.device)
+
+    def allocate(self) -> None:
+        r, n = self.r, max(w.geo.heads * w.geo.kp for w in self.layers)
+        self.keys, self.out = self.zeros(r.rows * n), self.zeros(r.rows * n)
+        self.o = self.zeros(r.rows * n, dtype=torch.float32)
+
+    def load(self, w: ForgetMixWeights, get, p: str) -> None:
+        g, (_, _, ov, _) = w.geo, w.geo.offsets
+        load_heads(w.wproj[:ov], get(p + "q"), g.heads, g.dim, g.kp)
+        load_heads(w.wproj[ov:], get(p + "v"), g.heads, g.vdim, g.vp)
+        load_head_vector(w.bias, get(p + "f.b").float(), g.heads, g.dim, g.kp)
+        load_head_vector(w.lower, get(p + "lower").float(), g.heads, g.dim, g.kp)
+        load_head_vector(w.norm, get(p + "norm").float().repeat(g.heads), g.heads, g.vdim, g.vp)
+        load_head_columns(w.wo, get(p + "o"), g.heads, g.vdim, g.vp)
+
+    def load_small(self, w: ForgetMixWeights, get, p: str, dst: torch.Tensor) -> None:
+        load_heads(dst, get(p + "f"), w.geo.heads, w.geo.dim, w.geo.kp)
+
+    plan = RecurrentPart.plan
+
+    def mix(self, w: ForgetMixWeights, state: RecurrentState, proj, z, y, b, plan) -> None:
+        """``y [T, wp]`` from the projected queries and values ``proj`` and the forget gate's logits ``z``."""
+        T, n = b.num_tokens, w.geo.heads * w.geo.vp
+        out = self.out[:T * n].view(T, n)
+        self.recur(w, state, proj, z, out, b, plan)
+        ops.gemm(out, w.wo, out=y, out_f32=True)
+
+    def recur(self, w: ForgetMixWeights, state: RecurrentState, proj, z, out, b, plan) -> None:
+        T, g, eps = b.num_tokens, w.geo, self.r.cfg.norm_eps
+        n = g.heads * g.kp
+        mix = ForgetMix(z, w.bias, w.lower, self.keys[:T * n].view(T, n))
+        n_seq, rows, table = plan if time_mix_chunked_supported(g) else (b.rows, T, None)
+        single = b.rows if b.cu_q is None else b.n_single
+        if single > 0:
+            ops.time_mix_decode(proj, g, mix, state, b.state_slots, b.seq_lens, w.norm, eps, out, single)
+        if n_seq > single:
+            o = self.o[:T * n].view(T, n)
+            ops.recurrent_scan(proj, None, g, None, None, None, 1.0, state, b.state_slots, b.cu_q, b.seq_lens, o, rows, n_seq, single, mix=mix)
+            ops.gated_norm(o[single:rows], w.norm, None, g, eps, out[single:], True)
+        if table is not None:
+            room = torch.empty(time_mix_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=out.device)
+            ops.time_mix_chunks(proj, g, mix, state, b.state_slots, b.cu_q, b.seq_lens, w.norm, eps, out, table, room)
+
+
+class DeltaWeights:
+    __slots__ = ("geo", "spec", "wproj", "conv", "rate", "dt_bias", "norm", "wo")
+
+
+@dataclass
+class DeltaState:
+    state: RecurrentState
+    history: torch.Tensor | None     # [slots, taps - 1, channels], the last projected rows of every sequence, latest first
+
+
+class DeltaPart(Part):
+    """Gated delta rule: joint projection (queries, keys, values, output gate, logits of decay and step size), one kernel for the
+    convolutions and the heads' units, the recurrence, norm and gate, output projection."""
+
+    fuses_tail = True
+
+    @staticmethod
+    def geometry(spec: DeltaRuleSpec) -> RecurrentGeometry:
+        return RecurrentGeometry(spec.heads, spec.dim, spec.vdim, silu=False, gated=False, form="delta", groups=spec.kv_heads)
+
+    @staticmethod
+    def state_floats(spec) -> int:
+        g = DeltaPart.geometry(spec)
+        return g.state_floats + (spec.taps - 1) * g.channels
+
+    @staticmethod
+    def small_rows(spec) -> int:
+        return 2 * spec.heads
+
+    def make(self, spec: DeltaRuleSpec, tail: int = 0) -> DeltaWeights:
+        g, f32 = self.geometry(spec), torch.float32
+        if max(g.kp, g.vp) > MAX_DIM or spec.taps > MAX_TAPS:
+            raise ValueError(f"the delta rule's kernels take up to {MAX_DIM} key channels and value channels per head, convolutions of {MAX_TAPS}")
+        w = DeltaWeights()
+        w.spec, w.geo = spec, g
+        w.wproj, w.wo = self.zeros(g.proj + tail, self.r.wp), self.zeros(self.r.wp, g.heads * g.vp)
+        w.conv, w.norm = self.zeros(spec.taps, g.channels, dtype=f32), self.zeros(g.heads * g.vp, dtype=f32)
+        w.rate, w.dt_bias = (self.zeros(g.heads, dtype=f32) for _ in range(2))
+        self.layers.append(w)
+        return w
+
+    def new_cache(self, w: DeltaWeights) -> DeltaState:
+        slots = self.r.scratch_state_slot + 1
+        history = self.zeros(slots, w.spec.taps - 1, w.geo.channels) if w.spec.taps > 1 else None
+        return DeltaState(RecurrentState.zeros(w.geo, slots, self.r.device), history)
+
+    def allocate(self) -> None:
+        r, f32, geos = self.r, torch.float32, {w.geo for w in self.layers}
+        self.proj, self.rows = self.zeros(r.rows * max(g.proj for g in geos)), self.zeros(r.rows * max(g.channels for g in geos))
+        self.units = self.zeros(r.rows * max(2 * g.key_heads for g in geos), dtype=f32)
+        self.steps = self.zeros(r.rows * max(2 * g.heads for g in geos), dtype=f32)
+        most = r.rows * max(g.heads * g.vp for g in geos)
+        self.values, self.out, self.o = self.zeros(most), self.zeros(most), self.zeros(most, dtype=f32)
+
+    def load(self, w: DeltaWeights, get, p: str) -> None:
+        g = w.geo
+        H, G, (_, ok, ov, og) = g.heads, g.key_heads, g.offsets
+        for name, lo, hi, heads, dim, padded in (("q", 0, ok, G, g.dim, g.kp), ("k", ok, ov, G, g.dim, g.kp), ("v", ov, og, H, g.vdim, g.vp)):
+            load_heads(w.wproj[lo:hi], get(p + name), heads, dim, padded)
+            conv = get(f"{p}{name}.conv").float().T
+            for t in range(w.spec.taps):
+                load_head_vector(w.conv[t, lo:hi], conv[t].contiguous(), heads, dim, padded)
+        load_heads(w.wproj[og:g.proj], get(p + "g"), H, g.vdim, g.vp)
+        load_head_columns(w.wo, get(p + "o"), H, g.vdim, g.vp)
+        load_head_vector(w.norm, get(p + "norm").float().repeat(H), H, g.vdim, g.vp)
+        w.rate.copy_(get(p + "A_log").float().exp())
+        w.dt_bias.copy_(get(p + "dt_bias").float())
+
+    def load_small(self, w: DeltaWeights, get, p: str, dst: torch.Tensor) -> None:
+        H, d = w.geo.heads, self.r.cfg.hidden_size
+        dst[:H, :d].copy_(get(p + "b"))
+        dst[H:2 * H, :d].copy_(get(p + "a"))
+
+    plan = RecurrentPart.plan
+
+    def _projected(self, w: DeltaWeights, T: int) -> torch.Tensor:
+        return self.proj[:T * w.geo.proj].view(T, w.geo.proj)
+
+    def project(self, w: DeltaWeights, inp, tail) -> None:
+        ops.gemm(inp, w.wproj, out=self._projected(w, inp.shape[0]), tail=tail)
+
+    def prepare(self, w: DeltaWeights, cache: DeltaState, small, b) -> tuple[torch.Tensor, DeltaRule]:
+        """What the recurrence reads, after ``project``."""
+        T, g = b.num_tokens, w.geo
+        rows = self.rows[:T * g.channels].view(T, g.channels)
+        rule = DeltaRule(self.units[:T * 2 * g.key_heads].view(T, -1), self.steps[:T * 2 * g.heads].view(T, -1))
+        ops.delta_rows(self._projected(w, T), small, g, w.conv, cache.history, b.cu_q, b.positions, b.state_slots, w.rate, w.dt_bias, rows, rule)
+        return rows, rule
+
+    def recur(self, w: DeltaWeights, cache: DeltaState, rows, rule: DeltaRule, o, b, plan) -> None:
+        T, g = b.num_tokens, w.geo
+        n_seq, ends, table = plan if delta_chunked_supported(g) else (b.rows, T, None)
+        args = (rows, None, g, None, None, None, 1.0, cache.state, b.state_slots)
+        if b.n_single > 0:
+            ops.recurrent_scan(*args, None, b.seq_lens, o, b.n_single, b.n_single, mix=rule)
+        if n_seq > b.n_single:
+            ops.recurrent_scan(*args, b.cu_q, b.seq_lens, o, ends, n_seq, b.n_single, mix=rule)
+        if table is not None:
+            room = torch.empty(delta_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=o.device)
+            values = self.values[:T * g.heads * g.vp].view(T, -1)
+            ops.delta_chunks(rows, g, rule, cache.state, b.state_slots, b.cu_q, b.seq_lens, o, table, values, room)
+
+    def forward(self, w: DeltaWeights, cache: DeltaState, inp, y, b, plan, small=None) -> None:
+        T, g = b.num_tokens, w.geo
+        n = g.heads * g.vp
+        o, out = self.o[:T * n].view(T, n), self.out[:T * n].view(T, n)
+        rows, rule = self.prepare(w, cache, small, b)
+        self.recur(w, cache, rows, rule, o, b, plan)
+        ops.gated_norm(o, w.norm, self._projected(w, T)[:, g.offsets[3]:], g, self.r.cfg.norm_eps, out, True, silu=True)
         ops.gemm(out, w.wo, out=y, out_f32=True)

@@ -2,13 +2,15 @@
 
 Step buffers, graph capture, packed batches and sampling come from ``RunnerBase``, mixers and feed-forwards from
 ``stack_parts``; this file puts layers together. The residual stream is fp32; projections read activations in the serving
-type. Two kinds of layer (``Design.block``):
+type. Three kinds of layer (``Design.block``):
 
 * post_norm: a sublayer reads the stream itself (a copy in the activation type) and its output is layer-normalised on the way
   back; the layer scale is folded into that norm's weight and bias in fp32;
 * parallel: mixer and feed-forward read one RMS norm of the stream; the residual add, the sum over a token's experts and
   the next layer's norm are one kernel. A per-layer token input (``TokenSideSpec``) enters between the add and that norm: two narrow
-  products over the stream, and its own norm in the same kernel as the next layer's.
+  products over the stream, and its own norm in the same kernel as the next layer's;
+* sandwich: every sublayer reads a norm of the stream, and a norm of its output is added. The weighing of a sublayer's parts (experts, two
+  mixers under norms of their own), the norm behind it, the residual add and the next sublayer's norm are one kernel.
 
 Looped layers run several times with the same weights; every run has a cache or state of its own, and a pass starts with a
 product that mixes the embedding output into the stream.
@@ -25,7 +27,7 @@ from typing import Any
 import torch
 
 from .. import ops
-from ..models.stack import LayerSpec, LayerStackConfig
+from ..models.stack import ExpertsSpec, LayerSpec, LayerStackConfig
 from ..ops.latent import live_tables
 from .model_runner import BLOCK, PackedBatch, RunnerBase
 from .stack_parts import FEED_FORWARD_PARTS, MIXER_PARTS
@@ -35,7 +37,7 @@ from .stack_parts.base import Part, up
 class StackLayer:
     """Weights of one layer: those of its mixer and feed-forward parts, the norms, the narrow fp32 projection."""
 
-    __slots__ = ("spec", "mixer", "mix", "feed_forward", "ff", "norm1", "norm2", "wsmall", "wsmall_ff", "mix_small", "side")
+    __slots__ = ("spec", "mixer", "mix", "feed_forward", "ff", "norm1", "norm2", "wsmall", "wsmall_ff", "mix_small", "side", "norm1b", "norm2b")
 
 
 @dataclass
@@ -79,7 +81,9 @@ class StackRunner(RunnerBase):
                             max_prefill_tokens=max_prefill_tokens, use_cuda_graphs=use_cuda_graphs,
                             graph_batch_sizes=graph_batch_sizes, dtype=dtype)
         self.bf16 = self.on_gpu and dtype == torch.bfloat16
-        self.parallel = cfg.design.block == "parallel"
+        self.parallel, self.sandwich = cfg.design.block == "parallel", cfg.design.block == "sandwich"
+        if not self.sandwich and any(isinstance(x.mlp, ExpertsSpec) and (x.mlp.identity or x.mlp.routing.shared_gate) for x in cfg.layers):
+            raise ValueError("identity experts and gated shared experts belong to sandwich blocks")
         self.wp = up(cfg.hidden_size, 8)
         self.vp = up(cfg.vocab_size, 8)
         self.rows = max(max_prefill_tokens, max_batch)
@@ -111,7 +115,10 @@ class StackRunner(RunnerBase):
             return torch.zeros(*shape, dtype=dtype, device=dev)
 
         def norm():
-            return zeros(self.wp, dtype=torch.float32), zeros(self.wp, dtype=torch.float32)
+            vectors = [zeros(self.wp, dtype=torch.float32) for _ in range(2)]
+            if not self.sandwich:
+                return tuple(vectors)
+            return ops.StreamNorm(*vectors, zeros(1, dtype=torch.float32)) if cfg.design.bounded_norms else ops.StreamNorm(vectors[0])
 
         # (a tied head reads the embedding table itself, whose rows are padded like the head's)
         self.embed = zeros(self.vp, self.wp)
@@ -127,6 +134,7 @@ class StackRunner(RunnerBase):
             lw.spec = spec
             lw.mixer = self._part(_mixer_part(spec))
             lw.norm1, lw.norm2 = norm(), None
+            lw.norm1b = lw.norm2b = norm() if self.sandwich else None
             lw.feed_forward = lw.ff = None
             lw.mix_small = up(lw.mixer.small_rows(spec.mixer), 8)
             ff_small = 0
@@ -134,6 +142,7 @@ class StackRunner(RunnerBase):
                 lw.feed_forward = self._part(FEED_FORWARD_PARTS[type(spec.mlp)])
                 lw.ff = lw.feed_forward.make(spec.mlp)
                 lw.norm2 = None if self.parallel else norm()
+                lw.norm2b = norm() if self.sandwich else None
                 ff_small = up(lw.feed_forward.small_rows(spec.mlp), 8)
             # the mixer's gate logits and, where both read the same activations, the router
             n = lw.mix_small + (ff_small if self.parallel else 0)
@@ -173,6 +182,12 @@ class StackRunner(RunnerBase):
             return get(name).float()
 
         def norm_into(dst, name: str, scale: torch.Tensor | None = None) -> None:
+            if self.sandwich:
+                dst.weight[:d].copy_(f32(name) + float(cfg.design.unit_norms))
+                if dst.alpha is not None:
+                    dst.bias[:d].copy_(f32(name + ".b"))
+                    dst.alpha.copy_(f32(name + ".alpha").reshape(1))
+                return
             if self.parallel:          # RMS norm
                 dst[0][:d].copy_(f32(name) + float(cfg.design.unit_norms))
                 return
@@ -193,7 +208,10 @@ class StackRunner(RunnerBase):
         for i, lw in enumerate(self.layers):
             p = f"l{i}."
             lw.mixer.load(lw.mix, get, p + "mix.")
-            norm_into(lw.norm1, p + "norm1", None if self.parallel else f32(p + "ls1"))
+            scaled = not (self.parallel or self.sandwich)
+            norm_into(lw.norm1, p + "norm1", f32(p + "ls1") if scaled else None)
+            if self.sandwich:
+                norm_into(lw.norm1b, p + "norm1b")
             if lw.mix_small:
                 lw.mixer.load_small(lw.mix, get, p + "mix.", lw.wsmall[:lw.mix_small])
             if lw.ff is not None:
@@ -201,7 +219,9 @@ class StackRunner(RunnerBase):
                 if lw.wsmall_ff is not None:
                     lw.feed_forward.load_small(lw.ff, get, p + "mlp.", lw.wsmall_ff)
                 if not self.parallel:
-                    norm_into(lw.norm2, p + "norm2", f32(p + "ls2"))
+                    norm_into(lw.norm2, p + "norm2", f32(p + "ls2") if scaled else None)
+                if self.sandwich:
+                    norm_into(lw.norm2b, p + "norm2b")
             if lw.side is not None:
                 lw.side.gate[:self.side_dim, :d].copy_(get(p + "side.gate"))
                 lw.side.proj[:d, :self.side_dim].copy_(get(p + "side.proj"))
@@ -229,6 +249,8 @@ class StackRunner(RunnerBase):
         plans = {part: part.planned(b) for part in self.parts.values()}
         if self.parallel:
             self._parallel_layers(b, plans)
+        elif self.sandwich:
+            self._sandwich_layers(b, plans)
         else:
             self._post_norm_layers(b, plans)
 
@@ -266,6 +288,33 @@ class StackRunner(RunnerBase):
                 add = {"side": y, "side_weight": lw.side.norm}
         ops.stream_norm(x, d, **add, mult=m, eps=eps)
 
+    def _sandwich_layers(self, b: PackedBatch, plans: dict) -> None:
+        T, d, eps = b.num_tokens, self.cfg.hidden_size, self.cfg.norm_eps
+        x, h, y = self.x[:T], self.xb[:T], self.y[:T]
+        xl = self.x_loop[:T, :self.wp] if self.x_loop is not None else None
+        self._embed(b, xl)
+        add: dict = {}                                 # what the sublayer before leaves for the stream, and the norm behind it
+
+        def left_by(parts: dict | None, norm) -> dict:
+            parts = dict(parts) if parts else {"y1": y}
+            return {"y": parts.pop("y1", None) if "y1" in parts else parts.pop("y2", None), "post": norm, **parts}
+
+        for run in self.runs:
+            lw = run.layer
+            if run.enters:
+                if add:
+                    ops.stream_sandwich(x, d, **add, eps=eps, copy=xl)
+                    add = {}
+                self._enter_pass(T)
+            ops.stream_sandwich(x, d, **add, pre=lw.norm1, eps=eps, h=h)
+            small = self._project(lw, h)
+            add = left_by(lw.mixer.forward(lw.mix, run.cache, h, y, b, plans[lw.mixer], small), lw.norm1b)
+            if lw.ff is not None:
+                ops.stream_sandwich(x, d, **add, pre=lw.norm2, eps=eps, h=h)
+                small = self._small_rows(h, lw.wsmall_ff) if lw.wsmall_ff is not None else None
+                add = left_by(lw.feed_forward.forward(lw.ff, h, y, small), lw.norm2b)
+        ops.stream_sandwich(x, d, **add, eps=eps)
+
     def _token_side(self, w: SideWeights, b: PackedBatch, xb: torch.Tensor, y: torch.Tensor) -> None:
         """``y = W_proj (gelu_tanh(W_gate x) * e)`` with the layer's part ``e`` of the tokens' side embedding."""
         T = b.num_tokens
@@ -297,7 +346,9 @@ class StackRunner(RunnerBase):
 
     def _final_rows(self, x: torch.Tensor, out: torch.Tensor, rows: torch.Tensor | None = None) -> None:
         d, eps = self.cfg.hidden_size, self.cfg.norm_eps
-        if self.parallel:
+        if self.sandwich:
+            ops.stream_sandwich(x, d, pre=self.final_norm, eps=eps, h=out, rows=rows)
+        elif self.parallel:
             ops.stream_norm(x, d, weight=self.final_norm[0], eps=eps, h=out, rows=rows)
         else:
             ops.layernorm_rows(x, self.final_norm[0], self.final_norm[1], eps, out, rows, d)

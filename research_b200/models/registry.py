@@ -30,6 +30,8 @@ ARCHITECTURES: dict[str, Architecture] = {
                             ("rb_engine_core", "rb_gemm", "rb_gemm2", "rb_gemm_f32", "rb_ops", "rb_latent", "rb_flash")),
     "Zamusun": Architecture(LayerStackConfig.from_dict, "research_b200.inference.stack_runner:StackRunner",
                             ("rb_engine_core", "rb_gemm", "rb_gemm2", "rb_gemm_f32", "rb_ops", "rb_recurrent", "rb_attn", "rb_flash", "rb_moe")),
+    "Sumitar": Architecture(LayerStackConfig.from_dict, "research_b200.inference.stack_runner:StackRunner",
+                            ("rb_engine_core", "rb_gemm", "rb_gemm2", "rb_gemm_f32", "rb_ops", "rb_recurrent", "rb_attn", "rb_flash", "rb_moe")),
     "Fogurax": Architecture(LayerStackConfig.from_dict, "research_b200.inference.stack_runner:StackRunner",
                             ("rb_engine_core", "rb_gemm", "rb_gemm2", "rb_gemm_f32", "rb_ops", "rb_recurrent", "rb_attn", "rb_flash", "rb_moe")),
 }

@@ -15,7 +15,8 @@ a layer is put together around them (norms, residual, head), is a row of ``DESIG
 
 Tensors are named ``embed``, ``l<i>.norm1`` / ``.mix.*`` / ``.mlp.*``, ``final.norm``; matrices are stored ``[out, in]``.
 Post-norm designs add ``.norm1.b`` / ``.ls1`` (and ``norm2`` / ``norm2.b`` / ``ls2`` for the feed-forward) and
-``final.norm.b``; designs without tied embeddings have ``head``; looped stacks have ``loop.in``; stacks with a per-layer token
+``final.norm.b``; sandwich designs have ``.norm1`` / ``.norm1b`` around the mixer and ``.norm2`` / ``.norm2b`` around the feed-forward, with a
+bounded norm each of them (and ``final.norm``) comes with ``.alpha`` (a scalar) and ``.b``; designs without tied embeddings have ``head``; looped stacks have ``loop.in``; stacks with a per-layer token
 input have ``side.embed`` and ``l<i>.side.gate`` / ``.proj`` / ``.norm``.
 """
 
@@ -275,6 +276,26 @@ class GluSpec:
 
 
 @dataclass(frozen=True)
+class PolyNormSpec:
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` between two matrices, with the four numbers in a tensor and ``N`` the division by the root mean
+    square over the ``ff`` values."""
+
+    ff: int
+
+    kind = "dense"
+
+    @staticmethod
+    def from_dict(m: dict) -> "PolyNormSpec":
+        return PolyNormSpec(ff=int(m["ff"]))
+
+    def to_dict(self) -> dict:
+        return {"kind": self.kind, "ff": self.ff}
+
+    def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
+        return {p + "up": (self.ff, width), p + "down": (width, self.ff), p + "act": (4,)}
+
+
+@dataclass(frozen=True)
 class ExpertsRouting:
     """How a design weighs the chosen experts: ``scores`` is "softmax" or "sigmoid" of the router's logits; ``normalize``
     divides the chosen scores by their sum; the weight multiplies an expert's output, or its input with ``scale_input``."""
@@ -282,43 +303,57 @@ class ExpertsRouting:
     scores: str = "softmax"
     normalize: bool = True
     scale_input: bool = False
+    correction: bool = False           # the choice (not the weight) goes by score plus a constant per expert
+    shared_gate: bool = False          # the shared unit's output times the sigmoid of one projected number
 
 
 @dataclass(frozen=True)
 class ExpertsSpec:
     """``experts`` gated units of which every token uses the ``top`` with the largest score, weighed as ``routing`` says;
-    ``shared`` is a further unit that every token passes."""
+    ``shared`` is a further unit that every token passes. ``identity`` more choices hand the input on as it is."""
 
     experts: int
     top: int
     expert: ClampedGluSpec | GluSpec
     routing: ExpertsRouting = ExpertsRouting()
     shared: GluSpec | None = None
+    identity: int = 0
 
     kind = "moe"
 
     def __post_init__(self):
-        assert 1 <= self.top <= self.experts
+        assert 1 <= self.top <= self.choices
+        assert not (self.identity and self.routing.scale_input), "a weight on an expert's input is no weight of an identity's output"
+
+    @property
+    def choices(self) -> int:
+        return self.experts + self.identity
 
     @staticmethod
     def from_dict(m: dict, unit=ClampedGluSpec, routing: ExpertsRouting = ExpertsRouting()) -> "ExpertsSpec":
         shared = m.get("shared")
         return ExpertsSpec(int(m["router"]["experts"]), int(m["router"]["top"]), unit.from_dict(m["expert"]), routing,
-                           unit.from_dict(shared) if shared else None)
+                           unit.from_dict(shared) if shared else None, int(m["router"].get("identity") or 0))
 
     def to_dict(self) -> dict:
         def unit(u) -> dict:
             return {k: v for k, v in u.to_dict().items() if k != "kind"}
 
         d = {"kind": self.kind, "router": {"experts": self.experts, "top": self.top}, "expert": unit(self.expert)}
+        if self.identity:
+            d["router"]["identity"] = self.identity
         return {**d, "shared": unit(self.shared)} if self.shared is not None else d
 
     def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
-        out = {p + "router": (self.experts, width)}
+        out = {p + "router": (self.choices, width)}
+        if self.routing.correction:
+            out[p + "correction"] = (self.choices,)
         for e in range(self.experts):
             out.update(self.expert.param_shapes(f"{p}e{e}.", width))
         if self.shared is not None:
             out.update(self.shared.param_shapes(p + "shared.", width))
+            if self.routing.shared_gate:
+                out[p + "shared.sg"] = (1, width)
         return out
 
 
@@ -338,6 +373,7 @@ class AttentionForm:
     scaling: type | None = None        # BandScaling or YarnScaling
     span: str = "all"
     gate: bool = False                 # every head's output times the sigmoid of one projected number
+    temperature: bool = False          # every head's scores times a number of its own
 
     def from_dict(self, m: dict) -> "GroupedAttentionSpec":
         rot, scaling = m["rot"], None
@@ -400,6 +436,8 @@ class GroupedAttentionSpec:
                 out[p + name + ".norm"] = (n,)
         if self.form.gate:
             out[p + "g"] = (self.heads, width)
+        if self.form.temperature:
+            out[p + "temp"] = (self.heads,)
         return {**out, p + "o": (width, self.heads * self.vdim)}
 
 
@@ -437,6 +475,64 @@ class TimeMixSpec:
 
 
 @dataclass(frozen=True)
+class ForgetMixSpec:
+    """Linear attention whose forget gate also decides what is written (HGRN2, see ``ops/recurrent.py``): a key row keeps ``f`` of itself
+    and takes ``1 - f`` of the value, ``f`` between a lower bound per channel and 1; SiLU on the queries, an RMS norm per head with
+    weights that the heads share."""
+
+    heads: int
+    dim: int
+    vdim: int
+
+    type = "forget_mix"
+
+    @staticmethod
+    def from_dict(m: dict) -> "ForgetMixSpec":
+        return ForgetMixSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]))
+
+    def to_dict(self) -> dict:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim}
+
+    def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
+        n, nv = self.heads * self.dim, self.heads * self.vdim
+        return {p + "q": (n, width), p + "f": (n, width), p + "f.b": (n,), p + "lower": (n,), p + "v": (nv, width), p + "norm": (self.vdim,),
+                p + "o": (width, nv)}
+
+
+@dataclass(frozen=True)
+class DeltaRuleSpec:
+    """Gated delta rule (see ``ops/recurrent.py``): short convolutions with SiLU on queries, keys and values, unit queries and keys that
+    groups of heads share, a decay and a step size per head, an RMS norm per head with weights that the heads share, a SiLU gate."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+
+    type = "delta"
+
+    def __post_init__(self):
+        assert self.heads % self.kv_heads == 0, "heads share queries and keys evenly"
+        assert self.taps >= 1
+
+    @staticmethod
+    def from_dict(m: dict) -> "DeltaRuleSpec":
+        return DeltaRuleSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]))
+
+    def to_dict(self) -> dict:
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "conv": self.taps}
+
+    def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
+        H, n, nv = self.heads, self.kv_heads * self.dim, self.heads * self.vdim
+        out: dict[str, tuple[int, ...]] = {}
+        for name, rows in (("q", n), ("k", n), ("v", nv)):
+            out[p + name], out[f"{p}{name}.conv"] = (rows, width), (rows, self.taps)
+        return {**out, p + "b": (H, width), p + "a": (H, width), p + "A_log": (H,), p + "dt_bias": (H,), p + "g": (nv, width), p + "norm": (self.vdim,),
+                p + "o": (width, nv)}
+
+
+@dataclass(frozen=True)
 class ParallelForm:
     """Which mixers a design puts side by side."""
 
@@ -469,18 +565,49 @@ class ParallelSpec:
 
 
 @dataclass(frozen=True)
+class NormedPairForm:
+    """Which mixers a design puts side by side under norms of their own."""
+
+    type: str
+    left: AttentionForm
+    right: type
+
+    def from_dict(self, m: dict) -> "NormedPairSpec":
+        return NormedPairSpec(self.type, self.left.from_dict(m["left"]), self.right.from_dict(m["right"]))
+
+
+@dataclass(frozen=True)
+class NormedPairSpec:
+    """Two mixers that read the same activations: half the sum of their outputs, each RMS-normed over the width with a weight."""
+
+    type: str
+    left: GroupedAttentionSpec
+    right: ForgetMixSpec
+
+    def to_dict(self) -> dict:
+        return {"left": self.left.to_dict(), "right": self.right.to_dict()}
+
+    def param_shapes(self, p: str, width: int) -> dict[str, tuple[int, ...]]:
+        return {**self.left.param_shapes(p + "left.", width), **self.right.param_shapes(p + "right.", width), p + "left.out": (width,),
+                p + "right.out": (width,)}
+
+
+@dataclass(frozen=True)
 class Design:
     """What all models of a design share. ``block`` is "post_norm" (sublayers read the stream; layer norm with bias and layer
-    scale on their outputs) or "parallel" (mixer and feed-forward read one RMS norm, and both are added)."""
+    scale on their outputs), "parallel" (mixer and feed-forward read one RMS norm, and both are added) or "sandwich" (a norm before
+    and after each sublayer: ``x += norm1b(mixer(norm1(x)))``, then ``x += norm2b(ff(norm2(x)))``)."""
 
     block: str
     tied: bool                         # the head is the embedding table
     mixers: dict                       # "type" in config.json -> what reads the layer's "mixer"
     feed_forwards: dict                # "kind" -> function that reads "mlp"
     unit_norms: bool = False           # norm weights are stored around zero
+    bounded_norms: bool = False        # sandwich: norms are tanh(alpha x) * w + b (Dynamic Tanh) instead of RMS norms
 
 
 WINDOW_ATTENTION = AttentionForm("window_attention", norm="projection", interleaved=True, span="window", gate=True)
+TEMPERED_ATTENTION = AttentionForm("tempered_attention", bias=True, span="window", temperature=True)
 
 DESIGNS = {
     "Lulezen": Design("post_norm", False, {"latent_attention": LatentAttentionSpec}, {"dense": ClampedGluSpec.from_dict}),
@@ -491,13 +618,17 @@ DESIGNS = {
                                            AttentionForm("attention_2", norm="projection", scaling=YarnScaling, span="chunk"),
                                            ParallelForm("parallel", WINDOW_ATTENTION, TimeMixSpec))},
                       {"dense": GluSpec.from_dict, "moe": partial(ExpertsSpec.from_dict, unit=GluSpec, routing=ExpertsRouting("sigmoid", False, True))}),
+    "Sumitar": Design("sandwich", True, {"parallel": NormedPairForm("parallel", TEMPERED_ATTENTION, ForgetMixSpec), "delta": DeltaRuleSpec},
+                      {"dense": PolyNormSpec.from_dict,
+                       "moe": partial(ExpertsSpec.from_dict, unit=GluSpec, routing=ExpertsRouting(normalize=False, correction=True, shared_gate=True))},
+                      bounded_norms=True),
 }
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: LatentAttentionSpec | LightningSpec | MatrixMemorySpec | KeyValueAttentionSpec | GroupedAttentionSpec | ParallelSpec
-    mlp: ClampedGluSpec | GluSpec | ExpertsSpec | None = None
+    mixer: LatentAttentionSpec | LightningSpec | MatrixMemorySpec | KeyValueAttentionSpec | GroupedAttentionSpec | ParallelSpec | NormedPairSpec | DeltaRuleSpec
+    mlp: ClampedGluSpec | GluSpec | PolyNormSpec | ExpertsSpec | None = None
 
     @staticmethod
     def from_dict(e: dict, design: Design) -> "LayerSpec":
@@ -583,7 +714,11 @@ class LayerStackConfig:
         return tuple(LayerRun(i, False) for i in range(loop.start)) + body * loop.times + tuple(LayerRun(i, False) for i in range(loop.stop, n))
 
     def param_shapes(self) -> dict[str, tuple[int, ...]]:
-        d, post = self.hidden_size, self.design.block == "post_norm"
+        d, post, sandwich = self.hidden_size, self.design.block == "post_norm", self.design.block == "sandwich"
+
+        def norm(name: str) -> dict[str, tuple[int, ...]]:
+            return {name: (d,), name + ".b": (d,), name + ".alpha": ()} if self.design.bounded_norms else {name: (d,)}
+
         out: dict[str, tuple[int, ...]] = {"embed": (self.vocab_size, d)}
         if self.loop is not None:
             out["loop.in"] = (d, 2 * d)
@@ -591,7 +726,9 @@ class LayerStackConfig:
             p = f"l{i}."
             subs = [("1", "mix.", layer.mixer)] + ([("2", "mlp.", layer.mlp)] if layer.mlp is not None else [])
             for n, sub, spec in subs:
-                if post:
+                if sandwich:
+                    out.update({**norm(p + "norm" + n), **norm(p + "norm" + n + "b")})
+                elif post:
                     out[p + "norm" + n] = out[p + "norm" + n + ".b"] = out[p + "ls" + n] = (d,)
                 elif n == "1":
                     out[p + "norm1"] = (d,)
@@ -600,7 +737,7 @@ class LayerStackConfig:
                 out.update({p + "side.gate": (self.token_side.dim, d), p + "side.proj": (d, self.token_side.dim), p + "side.norm": (d,)})
         if self.token_side is not None:
             out["side.embed"] = (self.vocab_size, self.num_layers * self.token_side.dim)
-        out["final.norm"] = (d,)
+        out.update(norm("final.norm"))
         if post:
             out["final.norm.b"] = (d,)
         if not self.design.tied:
@@ -610,8 +747,16 @@ class LayerStackConfig:
     def fill_value(self, name: str) -> float | None:
         """Constant a freshly initialised tensor starts from (None: random normal)."""
         last = name.rsplit(".", 1)[-1]
-        if last == "b" or last == "sink":
+        if (last == "b" and not name.endswith(".mix.b")) or last in ("sink", "correction", "lower", "A_log"):
             return 0.0
+        if last == "alpha":
+            return 0.5
+        if last in ("temp", "out"):
+            return 1.0
+        if last == "dt_bias":
+            return -4.0
+        if last == "act":
+            return 1 / 3
         if last.startswith("norm") or last.startswith("ls"):
             return 0.0 if self.design.unit_norms and ".mix." not in name else 1.0
         if ".mu." in name or last == "conv":

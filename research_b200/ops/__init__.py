@@ -22,9 +22,13 @@ from .elementwise import (
     rope_kv_append,
     rope_kv_append_reference,
     rope_table,
+    ChosenExperts,
+    StreamNorm,
+    poly_norm,
     softcap,
     stream_embed,
     stream_norm,
+    stream_sandwich,
     token_side,
     frequency_table,
     swiglu,
@@ -58,7 +62,7 @@ from .latent import (
 )
 from .keyvalue import KeyValueGeometry, kv_append, kv_attention, kv_workspace
 from .grouped import GroupedCache, GroupedGeometry, grouped_append, grouped_attention
-from .recurrent import ChunkTable, RecurrentGeometry, RecurrentState, TimeMix, gated_norm, recurrent_chunks, recurrent_scan, tanh_parts, time_mix_chunks, time_mix_decode, token_shift
+from .recurrent import ChunkTable, DeltaRule, ForgetMix, RecurrentGeometry, RecurrentState, TimeMix, delta_chunks, delta_rows, gated_norm, recurrent_chunks, recurrent_scan, tanh_parts, time_mix_chunks, time_mix_decode, token_shift
 from .sampling import sample_with_logprobs, sample_with_logprobs_reference, token_logprobs
 
 def set_pdl(on: bool) -> None:
@@ -84,5 +88,5 @@ __all__ = [
     "head_gemm_absorb", "head_gemm_expand", "latent_append", "latent_attention", "latent_gather", "latent_plan", "latent_query", "latent_units", "latent_workspace",
     "ExpertsGeometry", "ExpertsScratch", "experts_forward", "pack_experts", "KeyValueGeometry", "kv_append", "kv_attention", "kv_workspace",
     "ChunkTable", "RecurrentGeometry", "RecurrentState", "gated_norm", "recurrent_chunks", "recurrent_scan", "stream_embed", "stream_norm",
-    "GroupedCache", "GroupedGeometry", "grouped_append", "grouped_attention", "TimeMix", "tanh_parts", "time_mix_chunks", "time_mix_decode", "token_shift", "token_side", "frequency_table",
+    "GroupedCache", "GroupedGeometry", "grouped_append", "grouped_attention", "TimeMix", "ForgetMix", "DeltaRule", "delta_chunks", "delta_rows", "ChosenExperts", "StreamNorm", "poly_norm", "stream_sandwich", "tanh_parts", "time_mix_chunks", "time_mix_decode", "token_shift", "token_side", "frequency_table",
 ]

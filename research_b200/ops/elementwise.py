@@ -8,6 +8,7 @@ also what the functional oracles in the reference implement
 from __future__ import annotations
 
 import ctypes
+from dataclasses import dataclass
 
 import torch
 
@@ -35,7 +36,9 @@ def _lib() -> ctypes.CDLL:
         lib.rb_stream_norm.argtypes = ([c_vp, c_ll, c_vp, c_vp, c_ll, c_vp, c_vp, c_ll, c_int, c_vp, c_ll, c_vp, c_float, c_vp, c_ll, c_vp, c_ll, c_vp,
                                         c_vp] + [c_int] * 5 + [c_float, c_vp, c_vp])
         lib.rb_token_side.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_int, c_vp, c_ll] + [c_int] * 4 + [c_vp, c_vp]
-        for f in ("rb_token_side", "rb_stream_embed", "rb_stream_norm", "rb_layernorm", "rb_clamped_glu", "rb_softcap", "rb_rmsnorm", "rb_rope_kv_append", "rb_swiglu", "rb_swiglu_bwd", "rb_embedding", "rb_transpose_bf16"):
+        lib.rb_stream_sandwich.argtypes = [ctypes.POINTER(SandwichArgs), c_vp]
+        lib.rb_poly_norm.argtypes = [c_vp, c_ll, c_vp, c_vp, c_ll, c_int, c_int, c_int, c_float, c_int, c_vp]
+        for f in ("rb_stream_sandwich", "rb_poly_norm", "rb_token_side", "rb_stream_embed", "rb_stream_norm", "rb_layernorm", "rb_clamped_glu", "rb_softcap", "rb_rmsnorm", "rb_rope_kv_append", "rb_swiglu", "rb_swiglu_bwd", "rb_embedding", "rb_transpose_bf16"):
             getattr(lib, f).restype = c_int
         lib._rb_typed = True
     return lib
@@ -274,6 +277,113 @@ def stream_norm(x: torch.Tensor, d: int, *, y1=None, y2=None, experts=None, expe
                                ptr(rows), x.shape[0], _ACT[act.dtype], n, d, x.shape[1], eps, ptr(status_tensor(x.device)),
                                stream_handle(x.device))
     check_rc(rc, "rb_stream_norm")
+
+
+class SandwichArgs(ctypes.Structure):
+    _fields_ = ([(n, c_vp) for n in ("x", "y", "y2", "w", "w2", "gate", "e", "p", "idx", "pass_", "post_weight", "post_bias", "post_alpha", "pre_weight",
+                                     "pre_bias", "pre_alpha", "copy", "h", "rows", "status")]
+                + [(n, c_ll) for n in ("ldx", "ldy", "ld_gate", "lde", "ld_pass", "ldc", "ldh")]
+                + [(n, c_int) for n in ("k", "experts", "num_src_rows", "n", "d", "dp", "bounded", "dtype")]
+                + [("pair_scale", c_float), ("eps", c_float)])
+
+
+@dataclass
+class StreamNorm:
+    """A norm of stream rows: RMS norm, or with ``alpha`` (a scalar) ``tanh(alpha x) * weight + bias``; fp32 on the device."""
+
+    weight: torch.Tensor
+    bias: torch.Tensor | None = None
+    alpha: torch.Tensor | None = None
+
+    def reference(self, x: torch.Tensor, d: int, eps: float) -> torch.Tensor:
+        if self.alpha is not None:
+            return torch.tanh(self.alpha * x) * self.weight + self.bias
+        return x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / d + eps) * self.weight
+
+
+@dataclass
+class ChosenExperts:
+    """Results ``e [T * k, dp]`` of the chosen experts with weights ``p`` and choices ``idx [T, k]``; choices from ``experts`` on stand for the
+    rows of ``input``."""
+
+    e: torch.Tensor
+    p: torch.Tensor
+    idx: torch.Tensor
+    experts: int
+    input: torch.Tensor
+
+
+def stream_sandwich(x: torch.Tensor, d: int, *, y=None, pair=None, gate=None, chosen: ChosenExperts | None = None, post: StreamNorm | None = None,
+                    pre: StreamNorm | None = None, eps: float = 0.0, copy=None, h=None, rows=None) -> None:
+    """What happens to the fp32 stream ``x [n, dp]`` around a sublayer with norms before and after it, in one pass: ``x += post(v)``,
+    ``copy = x`` and ``h = pre(x)`` in the activation type, with the sublayer's output ``v``
+
+    * ``y`` times ``sigmoid(gate [n, >= 1])`` (its first column), if there is one, plus the weighted ``chosen`` experts, or
+    * half the sum of two mixers' ``y`` and ``pair[0]``, each divided by its root mean square, times ``pair[1]`` and ``pair[2]``.
+
+    With ``rows`` only ``h[i]`` of row ``rows[i]``."""
+    n = rows.numel() if rows is not None else x.shape[0]
+    update = y is not None or chosen is not None
+    assert not (update and rows is not None) and (pair is None or (gate is None and chosen is None))
+    if not x.is_cuda:
+        src = x if rows is None else x[rows.long()]
+        if update:
+            v = torch.zeros_like(x)
+            if pair is not None:
+                v = 0.5 * sum(StreamNorm(w).reference(t[:n], d, eps) for t, w in ((y, pair[1]), (pair[0], pair[2])))
+            elif y is not None:
+                v = y[:n] if gate is None else y[:n] * torch.sigmoid(gate[:n, :1])
+            if chosen is not None:
+                k = chosen.p.shape[1]
+                plain = (chosen.idx[:n] >= chosen.experts)[..., None]
+                rows_of = torch.where(plain, chosen.input[:n, None].float(), chosen.e[:n * k].view(n, k, -1).float())
+                v = v + (chosen.p[:n, :, None] * rows_of).sum(1)
+            x += post.reference(v, d, eps)
+        if copy is not None:
+            copy[:n] = x.to(copy.dtype)
+        if h is not None:
+            h[:n] = pre.reference(src, d, eps).to(h.dtype)
+        return
+    a = SandwichArgs()
+    assert x.dtype == torch.float32 and x.stride(1) == 1 and (rows is None or rows.dtype == torch.int32)
+    for name, t in (("x", x), ("y", y), ("gate", gate), ("copy", copy), ("h", h), ("rows", rows), ("status", status_tensor(x.device))):
+        setattr(a, name, t.data_ptr() if t is not None else None)
+    a.ldx, a.ldy, a.ld_gate = x.stride(0), y.stride(0) if y is not None else 0, gate.stride(0) if gate is not None else 0
+    a.ldc, a.ldh = copy.stride(0) if copy is not None else 0, h.stride(0) if h is not None else 0
+    if pair is not None:
+        assert pair[0].stride(0) == y.stride(0)
+        a.y2, a.w, a.w2, a.pair_scale = pair[0].data_ptr(), pair[1].data_ptr(), pair[2].data_ptr(), 0.5
+    act = next((t for t in (h, copy) if t is not None), x)
+    if chosen is not None:
+        act = chosen.e
+        assert chosen.e.dtype == chosen.input.dtype and chosen.idx.dtype == torch.int32 and chosen.idx.is_contiguous() and chosen.p.is_contiguous()
+        a.e, a.p, a.idx, a.pass_ = chosen.e.data_ptr(), chosen.p.data_ptr(), chosen.idx.data_ptr(), chosen.input.data_ptr()
+        a.lde, a.ld_pass, a.k, a.experts = chosen.e.stride(0), chosen.input.stride(0), chosen.p.shape[1], chosen.experts
+    assert (h is None or h.dtype == act.dtype) and (copy is None or copy.dtype == act.dtype)
+    for name, norm in (("post", post if update else None), ("pre", pre if h is not None else None)):
+        if norm is not None:
+            for part in ("weight", "bias", "alpha"):
+                t = getattr(norm, part)
+                setattr(a, f"{name}_{part}", t.data_ptr() if t is not None else None)
+    a.num_src_rows, a.n, a.d, a.dp, a.dtype, a.eps = x.shape[0], n, d, x.shape[1], _ACT[act.dtype], eps
+    a.bounded = int(any(m is not None and m.alpha is not None for m in (post, pre)))
+    check_rc(_lib().rb_stream_sandwich(ctypes.byref(a), stream_handle(x.device)), "rb_stream_sandwich")
+
+
+def poly_norm(z: torch.Tensor, act: torch.Tensor, n: int, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """``act[0] N(z) + act[1] N(z^2) + act[2] N(z^3) + act[3]`` on the first ``n`` columns of the rows (zero behind them), ``N`` the division by
+    the root mean square over those columns; ``act`` in fp32."""
+    T = z.shape[0]
+    if not z.is_cuda:
+        v = z[:, :n].float()
+        terms = (a * p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps) for a, p in zip(act, (v, v ** 2, v ** 3)))
+        out[:T].zero_()
+        out[:T, :n] = (sum(terms) + act[3]).to(out.dtype)
+        return out
+    assert z.stride(1) == out.stride(1) == 1 and z.dtype == out.dtype and act.dtype == torch.float32
+    check_rc(_lib().rb_poly_norm(ptr(z), z.stride(0), ptr(act), ptr(out), out.stride(0), T, n, z.shape[1], eps, _ACT[z.dtype], stream_handle(z.device)),
+             "rb_poly_norm")
+    return out
 
 
 def token_side(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col: int, out: torch.Tensor, n: int) -> None:

@@ -4,6 +4,9 @@ A router's logits -> the ``top`` largest softmax or sigmoid scores, divided by t
 expert (times their weight, when it belongs to the input), the gated unit runs as two grouped products (tile tables made on the
 device, so the layer fits a CUDA graph) and the second one stores every result row at its ``(token, choice)`` place. The
 weighted sum over the choices is left to whoever adds the result to the residual stream (``elementwise.stream_norm``).
+
+Choices from ``experts`` on (``identity`` of them) are no experts: they get no rows, and the sum takes the layer's input with their
+weight. A correction per choice may decide together with the score, without entering the weight.
 """
 
 from __future__ import annotations
@@ -29,9 +32,9 @@ def _up(n: int, m: int) -> int:
 def _lib() -> ctypes.CDLL:
     lib = _native.load("rb_moe")
     if not getattr(lib, "_rb_experts_typed", False):
-        lib.rb_experts_route.argtypes = [c_vp, c_ll] + [c_int] * 5 + [c_vp] * 4
+        lib.rb_experts_route.argtypes = [c_vp, c_ll, c_vp] + [c_int] * 6 + [c_vp] * 4
         lib.rb_experts_plan.argtypes = [c_vp, c_int, c_vp, c_int, c_int, c_vp, c_vp, c_int, c_int, c_vp, c_vp, c_int, c_vp, c_vp, c_vp]
-        lib.rb_experts_gather.argtypes = [c_vp, c_ll, c_vp] + [c_int] * 4 + [c_vp] * 4 + [c_ll, c_int, c_vp, c_int, c_vp, c_vp]
+        lib.rb_experts_gather.argtypes = [c_vp, c_ll, c_vp] + [c_int] * 5 + [c_vp] * 4 + [c_ll, c_int, c_vp, c_int, c_vp, c_vp]
         for f in ("rb_experts_route", "rb_experts_plan", "rb_experts_gather"):
             getattr(lib, f).restype = c_int
         lib._rb_experts_typed = True
@@ -50,6 +53,11 @@ class ExpertsGeometry:
     scores: str = "softmax"
     normalize: bool = True
     scale_input: bool = False    # a choice's weight multiplies the expert's input, not its output
+    identity: int = 0            # choices that hand the input on
+
+    @property
+    def choices(self) -> int:
+        return self.experts + self.identity
 
     @property
     def ffp(self) -> int:
@@ -57,11 +65,11 @@ class ExpertsGeometry:
 
     @staticmethod
     def make(experts: int, top: int, ff: int, width: int, limit: float | None, dtype: torch.dtype, scores: str = "softmax", normalize: bool = True,
-             scale_input: bool = False) -> "ExpertsGeometry":
-        if experts > MAX_EXPERTS or top > MAX_TOP:
+             scale_input: bool = False, identity: int = 0) -> "ExpertsGeometry":
+        if experts + identity > MAX_EXPERTS or top > MAX_TOP:
             raise ValueError(f"the expert kernels take up to {MAX_EXPERTS} experts, {MAX_TOP} per token")
         return ExpertsGeometry(experts, top, ff, width, limit, 128 if dtype == torch.bfloat16 else 64, dtype == torch.bfloat16, scores, normalize,
-                               scale_input)
+                               scale_input, identity)
 
 
 class ExpertsScratch:
@@ -96,9 +104,11 @@ def pack_experts(gates, ups, downs, geo: ExpertsGeometry, wgu: torch.Tensor, wd:
         wd3[e, :dn.shape[0], :geo.ff].copy_(dn)
 
 
-def route_reference(logits: torch.Tensor, top: int, scores: str = "softmax", normalize: bool = True) -> tuple[torch.Tensor, torch.Tensor]:
+def route_reference(logits: torch.Tensor, top: int, scores: str = "softmax", normalize: bool = True,
+                    correction: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
     s = logits.float().softmax(-1) if scores == "softmax" else torch.sigmoid(logits.float())
-    w, idx = s.topk(top, -1)
+    idx = (s if correction is None else s + correction).topk(top, -1).indices
+    w = s.gather(-1, idx)
     return idx.to(torch.int32), w / (w.sum(-1, keepdim=True) + 1e-20) if normalize else w
 
 
@@ -125,10 +135,10 @@ def _grouped(a, b, c, geo: ExpertsGeometry, sc: ExpertsScratch, group_n: int, K:
     check_rc(_gemm_lib().rb_gemm_bf16_ex(ctypes.byref(args), stream_handle(a.device)), "rb_gemm_bf16_ex(experts)")
 
 
-def experts_plan(logits, geo: ExpertsGeometry, sc: ExpertsScratch) -> None:
+def experts_plan(logits, geo: ExpertsGeometry, sc: ExpertsScratch, correction=None) -> None:
     """Choices and weights of every token, the experts' row ranges and the tile tables of both products."""
     T, s, st = logits.shape[0], stream_handle(logits.device), ptr(status_tensor(logits.device))
-    check_rc(_lib().rb_experts_route(ptr(logits), logits.stride(0), T, geo.experts, geo.top, int(geo.scores == "sigmoid"), int(geo.normalize), ptr(sc.idx),
+    check_rc(_lib().rb_experts_route(ptr(logits), logits.stride(0), ptr(correction), T, geo.choices, geo.experts, geo.top, int(geo.scores == "sigmoid"), int(geo.normalize), ptr(sc.idx),
                                      ptr(sc.w), ptr(sc.counts), s), "rb_experts_route")
     check_rc(_lib().rb_experts_plan(ptr(sc.counts), geo.experts, ptr(sc.offsets), 2 * geo.ffp, geo.bn, ptr(sc.tiles_gu), ptr(sc.ntiles), geo.width,
                                     geo.bn, ptr(sc.tiles_dn), sc.ntiles.data_ptr() + 4, sc.max_tiles, ptr(sc.cursor), st, s), "rb_experts_plan")
@@ -136,7 +146,7 @@ def experts_plan(logits, geo: ExpertsGeometry, sc: ExpertsScratch) -> None:
 
 def experts_gather(h, geo: ExpertsGeometry, sc: ExpertsScratch) -> None:
     es = h.element_size()
-    check_rc(_lib().rb_experts_gather(ptr(h), h.stride(0) * es, ptr(sc.idx), h.shape[0], geo.top, geo.width * es, geo.experts, ptr(sc.cursor), ptr(sc.xp),
+    check_rc(_lib().rb_experts_gather(ptr(h), h.stride(0) * es, ptr(sc.idx), h.shape[0], geo.top, geo.width * es, geo.experts, geo.choices, ptr(sc.cursor), ptr(sc.xp),
                                       ptr(sc.ret), ptr(sc.y), geo.width * es, sc.cap, ptr(sc.w) if geo.scale_input else None, int(es == 4),
                                        ptr(status_tensor(h.device)), stream_handle(h.device)),
              "rb_experts_gather")
@@ -153,18 +163,19 @@ def experts_down(geo: ExpertsGeometry, sc: ExpertsScratch, wd) -> None:
     _grouped(sc.act, wd, sc.y, geo, sc, geo.width, geo.ffp, sc.tiles_dn, sc.ntiles[1:], False, sc.ret)
 
 
-def experts_forward(h, logits, geo: ExpertsGeometry, sc: ExpertsScratch, wgu, wd) -> tuple[torch.Tensor, torch.Tensor | None]:
+def experts_forward(h, logits, geo: ExpertsGeometry, sc: ExpertsScratch, wgu, wd, correction=None) -> tuple[torch.Tensor, torch.Tensor | None]:
     """Results ``[T * top, width]`` of every token's chosen experts and the weights ``[T, top]`` they are still to be multiplied by
-    (None with ``scale_input``) for ``h [T, width]`` and the router's logits ``[T, >= experts]`` (fp32)."""
+    (None with ``scale_input``) for ``h [T, width]`` and the router's logits ``[T, >= choices]`` (fp32). ``correction [choices]``: see
+    above. The choices are left in ``sc.idx``; rows of choices that are no experts hold nothing."""
     T, k = h.shape[0], geo.top
     assert T * k <= sc.cap and logits.dtype == torch.float32
     if h.is_cuda:
-        experts_plan(logits, geo, sc)
+        experts_plan(logits, geo, sc, correction)
         experts_gather(h, geo, sc)
         experts_up(geo, sc, wgu, T)
         experts_down(geo, sc, wd)
         return sc.y[:T * k], None if geo.scale_input else sc.w[:T]
-    idx, w = route_reference(logits[:, :geo.experts], k, geo.scores, geo.normalize)
+    idx, w = route_reference(logits[:, :geo.choices], k, geo.scores, geo.normalize, correction)
     sc.idx[:T], sc.w[:T] = idx, w
     y = sc.y[:T * k].view(T, k, geo.width)
     gu3, wd3 = wgu.view(geo.experts, 2 * geo.ffp, -1), wd.view(geo.experts, geo.width, geo.ffp)

@@ -1,5 +1,5 @@
 """Attention with grouped heads over cached keys and values: short convolutions on the projections, norms and rotation of queries
-and keys, a window or chunks, a gate per head. Kernels: ``csrc/attn_sm100.cu`` (append, decode, exact mode),
+and keys, a factor per query head, a window or chunks, a gate per head. Kernels: ``csrc/attn_sm100.cu`` (append, decode, exact mode),
 ``csrc/flash_sm100.cu`` (portions); the CPU twins are here too.
 
 The joint projection of a token is ``q [H, dim] | k [G, dim] | v [G, vdim]`` (each part padded to 8 columns); the append kernel
@@ -41,6 +41,7 @@ class GroupedGeometry:
     interleaved: bool = False
     window: int = 0                  # keys a query sees: the last so many (0: all)
     chunk: int = 0                   # or those of its own run of so many positions
+    temperature: bool = False        # queries times a number of their head
 
     @property
     def dp(self) -> int:
@@ -83,8 +84,8 @@ class GroupedCache:
 
 
 class GroupedAppendArgs(ctypes.Structure):
-    _fields_ = ([(n, c_vp) for n in ("proj", "conv", "hist", "cu_q", "positions", "state_slots", "slots", "q_norm", "k_norm", "table", "q", "keys",
-                                     "values", "status")] + [("ld", c_ll)]
+    _fields_ = ([(n, c_vp) for n in ("proj", "conv", "hist", "cu_q", "positions", "state_slots", "slots", "q_norm", "k_norm", "q_factor", "table", "q",
+                                     "keys", "values", "status")] + [("ld", c_ll)]
                 + [(n, c_int) for n in ("k_col", "v_col", "channels", "taps", "B", "num_state_slots", "norm", "half", "interleaved", "max_pos",
                                         "num_blocks", "H", "G", "dim", "vdim", "DP", "T", "dtype")] + [("eps", c_float)])
 
@@ -151,7 +152,7 @@ def _rotate(x, cs, interleaved: bool):
     return out
 
 
-def _append_reference(proj, geo, conv, cache, cu_q, positions, state_slots, slots, q_norm, k_norm, eps, table, q) -> None:
+def _append_reference(proj, geo, conv, cache, cu_q, positions, state_slots, slots, q_norm, k_norm, eps, table, q, q_factor) -> None:
     T, H, G, D, E = proj.shape[0], geo.heads, geo.kv_heads, geo.dim, geo.vdim
     u = proj[:, :geo.channels].float()
     x = u * conv[geo.taps - 1] if geo.conv else u
@@ -168,6 +169,8 @@ def _append_reference(proj, geo, conv, cache, cu_q, positions, state_slots, slot
         if geo.norm == "head":
             x0 = x0 * torch.rsqrt(x0.pow(2).mean(-1, keepdim=True) + eps)
         qk.append(x0)
+    if q_factor is not None:
+        qk[0] = qk[0] * q_factor[:, None]
     q3 = q[:T].view(T, H, geo.dp)
     q3.zero_()
     q3[..., :D] = qk[0].to(q.dtype)
@@ -179,19 +182,20 @@ def _append_reference(proj, geo, conv, cache, cu_q, positions, state_slots, slot
 
 
 def grouped_append(proj, geo: GroupedGeometry, *, conv, cache: GroupedCache, cu_q, positions, state_slots, slots, q_norm, k_norm, eps: float, table,
-                   q) -> None:
+                   q, q_factor=None) -> None:
     """From the joint projection ``proj [T, >= channels]`` of the packed new tokens: convolved, normed and rotated queries into
     ``q [T, H * dp]``, keys and values into the cache rows ``slots`` (negative: skipped). ``conv [taps, channels]`` fp32, latest tap
-    last; ``table [positions, rot_dims / 2, 2]``; ``state_slots [B]`` own the convolution's look back, which moves on."""
+    last; ``table [positions, rot_dims / 2, 2]``; ``state_slots [B]`` own the convolution's look back, which moves on; queries times
+    ``q_factor [H]`` (fp32, or None)."""
     T = proj.shape[0]
     if not proj.is_cuda:
-        _append_reference(proj, geo, conv, cache, cu_q, positions, state_slots, slots, q_norm, k_norm, eps, table, q)
+        _append_reference(proj, geo, conv, cache, cu_q, positions, state_slots, slots, q_norm, k_norm, eps, table, q, q_factor)
         return
     assert proj.stride(1) == 1 and q.is_contiguous() and cache.keys.is_contiguous() and cache.values.is_contiguous() and table.is_contiguous()
     a = GroupedAppendArgs()
     assert (conv is not None) == geo.conv and (geo.conv or geo.taps == 1)
     for name, t in (("proj", proj), ("conv", conv), ("hist", cache.history), ("cu_q", cu_q), ("positions", positions), ("state_slots", state_slots),
-                    ("slots", slots), ("q_norm", q_norm), ("k_norm", k_norm), ("table", table), ("q", q), ("keys", cache.keys),
+                    ("slots", slots), ("q_norm", q_norm), ("k_norm", k_norm), ("q_factor", q_factor), ("table", table), ("q", q), ("keys", cache.keys),
                     ("values", cache.values), ("status", status_tensor(proj.device))):
         setattr(a, name, t.data_ptr() if t is not None else None)
     a.ld, a.k_col, a.v_col, a.channels, a.taps = proj.stride(0), geo.k_col, geo.v_col, geo.channels, geo.taps
