@@ -13,9 +13,9 @@ import json
 from dataclasses import asdict, dataclass, field, replace
 from pathlib import Path
 
-from .stack import (DESIGNS, BandScaling, ClampedGluSpec, ExpertsRouting, ExpertsSpec, GluSpec, GroupedAttentionSpec, KeyValueAttentionSpec,
-                    LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec, LoopSpec, MatrixMemorySpec, ParallelSpec, QueryTemperature,
-                    RotarySpec, TimeMixSpec, TokenSideSpec, YarnScaling, uniform_stack)
+from .stack import (DESIGNS, BandScaling, ClampedGluSpec, DeltaRuleSpec, ExpertsRouting, ExpertsSpec, ForgetMixSpec, GluSpec, GroupedAttentionSpec,
+                    KeyValueAttentionSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec, LoopSpec, MatrixMemorySpec,
+                    NormedPairSpec, ParallelSpec, PolyNormSpec, QueryTemperature, RotarySpec, TimeMixSpec, TokenSideSpec, YarnScaling, uniform_stack)
 
 
 @dataclass(frozen=True)
@@ -172,6 +172,16 @@ def _attention_beside_time_mix(heads: int, kv_heads: int, dim: int, rot: int, si
     return ParallelSpec("parallel", left, TimeMixSpec(mix_heads, mix_dim, rank), 1.0, 1.0)
 
 
+def _attention_beside_forget_mix(heads: int, kv_heads: int, dim: int, vdim: int, rot: int, size: int, mix_heads: int, mix_dim: int,
+                                 mix_vdim: int) -> NormedPairSpec:
+    left = GroupedAttentionSpec(DESIGNS["Sumitar"].mixers["parallel"].left, heads, kv_heads, dim, vdim, dim ** -0.5, RotarySpec(rot, 5e5), 1, size)
+    return NormedPairSpec("parallel", left, ForgetMixSpec(mix_heads, mix_dim, mix_vdim))
+
+
+def _corrected_experts(experts: int, identity: int, top: int, ff: int, shared: int) -> ExpertsSpec:
+    return ExpertsSpec(experts, top, GluSpec(ff), ExpertsRouting(normalize=False, correction=True, shared_gate=True), GluSpec(shared), identity)
+
+
 def _shared_experts(experts: int, top: int, ff: int, shared: int) -> ExpertsSpec:
     return ExpertsSpec(experts, top, GluSpec(ff), ExpertsRouting("sigmoid", False, True), GluSpec(shared))
 
@@ -224,6 +234,14 @@ PRESETS: dict[str, ModelConfig | LayerStackConfig] = {
         LayerSpec((_chunk_attention(16, 4, 128, 128, 64, 4096, 4096), _conv_attention(16, 4, 128, 128, 64, 4, 8192),
                    _attention_beside_time_mix(16, 4, 128, 64, 2048, 32, 64, 64))[i % 3],
                   GluSpec(8192) if i % 3 == 0 else _shared_experts(64, 8, 768, 1536)) for i in range(15)), residual_mult=0.5, token_side=TokenSideSpec(256)),
+    # layer stacks between two norms a sublayer: windowed attention beside forget mixing, gated delta rule, normed powers, identity experts
+    "tiny-sumitar": LayerStackConfig("Sumitar", 4096, 176, (
+        LayerSpec(_attention_beside_forget_mix(5, 1, 24, 40, 16, 50, 3, 40, 24), PolyNormSpec(288)),
+        LayerSpec(DeltaRuleSpec(4, 2, 48, 32, 3), _corrected_experts(6, 3, 3, 64, 80)),
+        LayerSpec(DeltaRuleSpec(3, 3, 32, 40, 4), None)), init_std=0.05),
+    "sumitar-4b": LayerStackConfig("Sumitar", 128256, 2048, tuple(
+        LayerSpec(_attention_beside_forget_mix(16, 4, 128, 128, 64, 2048, 16, 128, 128) if i % 3 == 2 else DeltaRuleSpec(32, 16, 128, 128, 4),
+                  PolyNormSpec(8192) if i % 3 == 0 else _corrected_experts(60, 4, 8, 768, 1536)) for i in range(15))),
 }
 
 

@@ -133,7 +133,7 @@ def save_safetensors(tensors: dict[str, torch.Tensor], path: str | Path, metadat
     blobs = []
     for name in sorted(tensors):
         t = tensors[name].detach().contiguous().cpu()
-        raw = t.view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         header[name] = {"dtype": _DT_INV[t.dtype], "shape": list(t.shape), "data_offsets": [offset, offset + len(raw)]}
         offset += len(raw)
         blobs.append(raw)
