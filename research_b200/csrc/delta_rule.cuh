@@ -195,12 +195,6 @@ struct DeltaSolveCfg {
   static constexpr int kCols = 256;
 };
 
-__device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(x, y);
-  const float2 b = unpack_bf16x2(hi);
-  lo = pack_bf16x2(x - b.x, y - b.y);
-}
-
 // A 16 x 16 block as first operand of mma.sync (and, four accumulators of an n = 8 product after the other, as its result).
 struct Block16 {
   uint32_t hi[4], lo[4];

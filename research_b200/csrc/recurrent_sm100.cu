@@ -1248,7 +1248,7 @@ static int launch_chunks(const ChunkParams& p, int n_chunks, int n_seq, cudaStre
 // adds to the state (z becomes A on the way), the chain of states, outputs with the head's norm and the output gate.
 //
 // Forget mixing is the same with keys 1 - f, weights that end at A_t (a token is written before it is read, P_tt = q_t . k_t) and no
-// output gate.
+// output gate. Its keys are gates, no rounded activations: they, and what is scaled by a power of A, go into every product in two parts.
 // ------------------------------------------------------------------------------------------
 constexpr float MIX_MOST = 64.f;      // a token that keeps less than 2^-64 keeps nothing; larger sums would cost A its last digits
 
@@ -1276,9 +1276,16 @@ struct MixParams {
   long long ldo;
   int H, dk, dv, KP, VP, num_slots;
   int* status;
-  __nv_bfloat16* keys;           // [T, ld_keys] forget mixing: 1 - f
+  __nv_bfloat16* keys;           // [T, ld_keys] forget mixing: 1 - f [H * KP], and what bf16 lacks of it [H * KP]
   long long ld_keys;
 };
+
+// Two values as two bf16 parts each.
+__device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(x, y);
+  const float2 b = unpack_bf16x2(hi);
+  lo = pack_bf16x2(x - b.x, y - b.y);
+}
 
 template <int DK>
 struct MixStateCfg {
@@ -1372,7 +1379,13 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_state_kernel(c
     float2 f;
     if (FORGET) {
       f = fresh[FORGET ? i : 0];
-      if (i < mine) *reinterpret_cast<uint32_t*>(p.keys + (long long)(row0 + t0 + i) * p.ld_keys + h * p.KP + col) = pack_bf16x2(f.x, f.y);
+      if (i < mine) {
+        uint32_t* key = reinterpret_cast<uint32_t*>(p.keys + (long long)(row0 + t0 + i) * p.ld_keys + h * p.KP + col);
+        uint32_t hi_part, lo_part;
+        split_bf16x2(f.x, f.y, hi_part, lo_part);
+        key[0] = hi_part;
+        key[p.H * p.KP / 2] = lo_part;
+      }
     } else {
       f = unpack_bf16x2(keys[FORGET ? 0 : i]);
     }
@@ -1481,18 +1494,21 @@ __device__ __forceinline__ void mma_16816_bf16(float (&c)[4], uint32_t a0, uint3
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-template <int DK>
+template <int DK, bool FORGET>
 struct MixOutCfg {
   static constexpr int kTile = CH * DK * 2;                        // r (then r 2^A), k (then V)
   static constexpr int kA = CH * DK * 4;                           // A, then both parts of the state
-  static constexpr int kSmem = 1024 + 2 * kTile + kA + 2 * CH_CHUNK;
+  static constexpr int kState = 2 * DK * DK * 2;
+  static constexpr int kRest = 2 * kTile + kA + 2 * CH_CHUNK;      // forget mixing: what bf16 lacks of r 2^A, behind the state where it fits
+  static constexpr int kRLow = kState + kTile <= kA ? 2 * kTile + kState : kRest;
+  static constexpr int kSmem = 1024 + kRest + (FORGET && kRLow == kRest ? kTile : 0);
   static constexpr int kCols = DK;
 };
 
 // Outputs of a chunk of one head. VP == KP == DK.
 template <int DK, bool FORGET>
 __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(const MixParams p) {
-  using Cfg = MixOutCfg<DK>;
+  using Cfg = MixOutCfg<DK, FORGET>;
   extern __shared__ __align__(128) uint8_t smem_raw[];
   __shared__ float row_sum[2][CH];
   __shared__ __align__(8) uint64_t done;
@@ -1551,14 +1567,41 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
   auto two_a = [&](int t, int u) {                                 // A of channels 8u + cq, 8u + cq + 1; zero in front of the chunk
     return t < 0 ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(a_row(t) + a_piece(t, u) + cq * 4);
   };
-  // r_t 2^(A_(t-1) - A_ref) (forget mixing: A_t) and k_j 2^(A_ref - A_j) of those channels
+  // r_t 2^(A_(t-1) - A_ref) (forget mixing: A_t) and k_j 2^(A_ref - A_j) of those channels, as bf16 {value, what it lacks (forget mixing)}
+  auto parts = [](float x, float y) {
+    uint2 v = make_uint2(0u, 0u);
+    if (FORGET) split_bf16x2(x, y, v.x, v.y);
+    else v.x = pack_bf16x2(x, y);
+    return v;
+  };
   auto scaled_r = [&](int t, int u, float2 ref) {
     const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(r_p + t * CH_ROWB + b_piece(t, u) + cq * 2)), a = two_a(t - BACK, u);
-    return pack_bf16x2(x.x * chunk_exp2(a.x - ref.x), x.y * chunk_exp2(a.y - ref.y));
+    return parts(x.x * chunk_exp2(a.x - ref.x), x.y * chunk_exp2(a.y - ref.y));
   };
-  auto scaled_k = [&](const uint8_t* k_row, const uint8_t* arow, int kb, int ab, float2 ref) {
-    const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_row + kb)), a = *reinterpret_cast<const float2*>(arow + ab);
-    return pack_bf16x2(x.x * chunk_exp2(ref.x - a.x), x.y * chunk_exp2(ref.y - a.y));
+  const __nv_bfloat16* key_rest = FORGET ? p.keys + (long long)row0 * p.ld_keys + (p.H + h) * p.KP : nullptr;      // what bf16 lacks of the keys
+  auto rest_row = [&](int j) { return FORGET ? key_rest + (long long)min(j, n - 1) * p.ld_keys : nullptr; };
+  auto scaled_k = [&](const uint8_t* k_row, const uint8_t* arow, const __nv_bfloat16* rest, int kb, int ab, int u, float2 ref) {
+    float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(k_row + kb));
+    const float2 a = *reinterpret_cast<const float2*>(arow + ab);
+    if (FORGET) {
+      const float2 y = unpack_bf16x2(__ldg(reinterpret_cast<const uint32_t*>(rest + 8 * u + cq)));
+      x.x += y.x;
+      x.y += y.y;
+    }
+    return parts(x.x * chunk_exp2(ref.x - a.x), x.y * chunk_exp2(ref.y - a.y));
+  };
+  // s += a b^T over 16 channels
+  auto product = [&](float (&s)[4], uint2 a0, uint2 a1, uint2 a2, uint2 a3, uint2 b0, uint2 b1) {
+    mma_16816_bf16(s, a0.x, a1.x, a2.x, a3.x, b0.x, b1.x);
+    if (FORGET) {
+      mma_16816_bf16(s, a0.y, a1.y, a2.y, a3.y, b0.x, b1.x);
+      mma_16816_bf16(s, a0.x, a1.x, a2.x, a3.x, b0.y, b1.y);
+    }
+  };
+  const uint2 none = make_uint2(0u, 0u);
+  auto key_of = [](uint32_t high, uint32_t rest) {
+    const float2 x = unpack_bf16x2(high), y = unpack_bf16x2(rest);
+    return FORGET ? make_float2(x.x + y.x, x.y + y.y) : x;
   };
   // The blocks left of the diagonal, 8 columns at a time: rows w and 7 - w have 14 such pieces together, half of them for either warp.
   {
@@ -1569,7 +1612,7 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
     const uint8_t* a0 = a_row(g) + cq * 4;
     auto blocks = [&](int b0, int from, int to) {                  // block row at token b0, columns 8 from .. 8 to
       if (b0 >= n || from >= to) return;
-      uint32_t fa[DK / 16][4];
+      uint2 fa[DK / 16][4];
       float2 ref[DK / 8];
 #pragma unroll
       for (int u = 0; u < DK / 8; ++u) {
@@ -1581,10 +1624,11 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
         float s[4] = {0.f, 0.f, 0.f, 0.f};
         const uint8_t* kr = k0 + j0 * CH_ROWB;
         const uint8_t* ar = a0 + j0 * (DK * 4);
+        const __nv_bfloat16* rest = rest_row(j0 + g);
 #pragma unroll
         for (int ks = 0; ks < DK / 16; ++ks)
-          mma_16816_bf16(s, fa[ks][0], fa[ks][1], fa[ks][2], fa[ks][3], scaled_k(kr, ar, kb[2 * ks], ab[2 * ks], ref[2 * ks]),
-                         scaled_k(kr, ar, kb[2 * ks + 1], ab[2 * ks + 1], ref[2 * ks + 1]));
+          product(s, fa[ks][0], fa[ks][1], fa[ks][2], fa[ks][3], scaled_k(kr, ar, rest, kb[2 * ks], ab[2 * ks], 2 * ks, ref[2 * ks]),
+                  scaled_k(kr, ar, rest, kb[2 * ks + 1], ab[2 * ks + 1], 2 * ks + 1, ref[2 * ks + 1]));
         *reinterpret_cast<uint32_t*>(weight_at(b0 + g, j0 + cq)) = pack_bf16x2(s[0], s[1]);
         *reinterpret_cast<uint32_t*>(weight_at(b0 + g + 8, j0 + cq)) = pack_bf16x2(s[2], s[3]);
       }
@@ -1601,11 +1645,13 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
       float s[4] = {0.f, 0.f, 0.f, 0.f};
       const uint8_t* kr = k_p + (t0 + g) * CH_ROWB + cq * 2;
       const uint8_t* ar = a_row(t0 + g) + cq * 4;
+      const __nv_bfloat16* rest = rest_row(t0 + g);
 #pragma unroll
       for (int ks = 0; ks < DK / 16; ++ks) {
         const float2 ref0 = two_a(t0 + 7, 2 * ks), ref1 = two_a(t0 + 7, 2 * ks + 1);
-        mma_16816_bf16(s, scaled_r(t0 + 8 + g, 2 * ks, ref0), 0u, scaled_r(t0 + 8 + g, 2 * ks + 1, ref1), 0u,
-                       scaled_k(kr, ar, b_piece(g, 2 * ks), a_piece(g, 2 * ks), ref0), scaled_k(kr, ar, b_piece(g, 2 * ks + 1), a_piece(g, 2 * ks + 1), ref1));
+        product(s, scaled_r(t0 + 8 + g, 2 * ks, ref0), none, scaled_r(t0 + 8 + g, 2 * ks + 1, ref1), none,
+                scaled_k(kr, ar, rest, b_piece(g, 2 * ks), a_piece(g, 2 * ks), 2 * ks, ref0),
+                scaled_k(kr, ar, rest, b_piece(g, 2 * ks + 1), a_piece(g, 2 * ks + 1), 2 * ks + 1, ref1));
       }
       *reinterpret_cast<uint32_t*>(weight_at(t0 + 8 + g, t0 + cq)) = pack_bf16x2(s[0], s[1]);
     }
@@ -1617,8 +1663,10 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
         const float2 ref0 = two_a(ref_row, 2 * ks), ref1 = two_a(ref_row, 2 * ks + 1);
         const uint8_t* kr = k_p + j * CH_ROWB + cq * 2;
         const uint8_t* ar = a_row(j) + cq * 4;
-        mma_16816_bf16(s, scaled_r(t, 2 * ks, ref0), 0u, scaled_r(t, 2 * ks + 1, ref1), 0u,
-                       scaled_k(kr, ar, b_piece(j, 2 * ks), a_piece(j, 2 * ks), ref0), scaled_k(kr, ar, b_piece(j, 2 * ks + 1), a_piece(j, 2 * ks + 1), ref1));
+        const __nv_bfloat16* rest = rest_row(j);
+        product(s, scaled_r(t, 2 * ks, ref0), none, scaled_r(t, 2 * ks + 1, ref1), none,
+                scaled_k(kr, ar, rest, b_piece(j, 2 * ks), a_piece(j, 2 * ks), 2 * ks, ref0),
+                scaled_k(kr, ar, rest, b_piece(j, 2 * ks + 1), a_piece(j, 2 * ks + 1), 2 * ks + 1, ref1));
       }
       if ((g >> 2) == (cq >> 2)) *reinterpret_cast<uint32_t*>(weight_at(t, t0 + cq + (cq < 4 ? 0 : 4))) = pack_bf16x2(s[0], s[1]);
     }
@@ -1637,17 +1685,18 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
         const float4* pa = reinterpret_cast<const float4*>(at + a_piece(tt - BACK, u));
         const float4* pb = reinterpret_cast<const float4*>(aj + a_piece(jj, u));
         const float4 a = pa[0], b = pb[0], c4 = pa[1], d4 = pb[1];
+        const uint4 z = FORGET ? __ldg(reinterpret_cast<const uint4*>(rest_row(jj) + 8 * u)) : make_uint4(0u, 0u, 0u, 0u);
         float2 f, h2;
-        f = unpack_bf16x2(x.x); h2 = unpack_bf16x2(y.x);
+        f = unpack_bf16x2(x.x); h2 = key_of(y.x, z.x);
         s0 = fmaf(f.x * h2.x, chunk_exp2(a.x - b.x), s0);
         s1 = fmaf(f.y * h2.y, chunk_exp2(a.y - b.y), s1);
-        f = unpack_bf16x2(x.y); h2 = unpack_bf16x2(y.y);
+        f = unpack_bf16x2(x.y); h2 = key_of(y.y, z.y);
         s0 = fmaf(f.x * h2.x, chunk_exp2(a.z - b.z), s0);
         s1 = fmaf(f.y * h2.y, chunk_exp2(a.w - b.w), s1);
-        f = unpack_bf16x2(x.z); h2 = unpack_bf16x2(y.z);
+        f = unpack_bf16x2(x.z); h2 = key_of(y.z, z.z);
         s0 = fmaf(f.x * h2.x, chunk_exp2(c4.x - d4.x), s0);
         s1 = fmaf(f.y * h2.y, chunk_exp2(c4.y - d4.y), s1);
-        f = unpack_bf16x2(x.w); h2 = unpack_bf16x2(y.w);
+        f = unpack_bf16x2(x.w); h2 = key_of(y.w, z.w);
         s0 = fmaf(f.x * h2.x, chunk_exp2(c4.z - d4.z), s0);
         s1 = fmaf(f.y * h2.y, chunk_exp2(c4.w - d4.w), s1);
       }
@@ -1666,11 +1715,12 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
           b0 = *reinterpret_cast<const float4*>(bonus + u * 8);
           b1 = *reinterpret_cast<const float4*>(bonus + u * 8 + 4);
         }
+        const uint4 z = FORGET ? __ldg(reinterpret_cast<const uint4*>(rest_row(t) + 8 * u)) : make_uint4(0u, 0u, 0u, 0u);
         float2 f, h2;
-        f = unpack_bf16x2(x.x); h2 = unpack_bf16x2(y.x); s = fmaf(f.x * h2.x, b0.x, fmaf(f.y * h2.y, b0.y, s));
-        f = unpack_bf16x2(x.y); h2 = unpack_bf16x2(y.y); s = fmaf(f.x * h2.x, b0.z, fmaf(f.y * h2.y, b0.w, s));
-        f = unpack_bf16x2(x.z); h2 = unpack_bf16x2(y.z); s = fmaf(f.x * h2.x, b1.x, fmaf(f.y * h2.y, b1.y, s));
-        f = unpack_bf16x2(x.w); h2 = unpack_bf16x2(y.w); s = fmaf(f.x * h2.x, b1.z, fmaf(f.y * h2.y, b1.w, s));
+        f = unpack_bf16x2(x.x); h2 = key_of(y.x, z.x); s = fmaf(f.x * h2.x, b0.x, fmaf(f.y * h2.y, b0.y, s));
+        f = unpack_bf16x2(x.y); h2 = key_of(y.y, z.y); s = fmaf(f.x * h2.x, b0.z, fmaf(f.y * h2.y, b0.w, s));
+        f = unpack_bf16x2(x.z); h2 = key_of(y.z, z.z); s = fmaf(f.x * h2.x, b1.x, fmaf(f.y * h2.y, b1.y, s));
+        f = unpack_bf16x2(x.w); h2 = key_of(y.w, z.w); s = fmaf(f.x * h2.x, b1.z, fmaf(f.y * h2.y, b1.w, s));
       }
       s += __shfl_xor_sync(0xffffffffu, s, 16);
       if (lane < 16) *reinterpret_cast<__nv_bfloat16*>(weight_at(t, t)) = __float2bfloat16_rn(s);
@@ -1678,9 +1728,11 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
   }
   __syncthreads();                                                 // k has been read
   chunk_load<DK>(k_s, rows + p.v_col + h * p.VP, p.ld, n);
-#pragma unroll 2
-  for (int i = tid; i < CH * (DK / 8); i += CHT) {                 // r 2^A_(t-1) (forget mixing: A_t), in place
-    const int t = i / (DK / 8), u = i % (DK / 8);
+  constexpr int PIECES = CH * (DK / 8) / CHT;
+  uint4 rest_r[FORGET ? PIECES : 1];                               // forget mixing: what bf16 lacks of r 2^A
+#pragma unroll
+  for (int k = 0; k < PIECES; ++k) {                               // r 2^A_(t-1) (forget mixing: A_t), in place
+    const int i = tid + k * CHT, t = i / (DK / 8), u = i % (DK / 8);
     if (t < BACK) continue;
     uint4* at = reinterpret_cast<uint4*>(r_p + t * CH_ROWB + b_piece(t, u));
     const float4* pa = reinterpret_cast<const float4*>(a_row(t - BACK) + a_piece(t - BACK, u));
@@ -1688,12 +1740,19 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
     uint4 v = *at;
     auto one = [&](uint32_t x, float ax, float ay) {
       const float2 f = unpack_bf16x2(x);
-      return pack_bf16x2(f.x * chunk_exp2(ax), f.y * chunk_exp2(ay));
+      return parts(f.x * chunk_exp2(ax), f.y * chunk_exp2(ay));
     };
-    v.x = one(v.x, a.x, a.y); v.y = one(v.y, a.z, a.w); v.z = one(v.z, b.x, b.y); v.w = one(v.w, b.z, b.w);
-    *at = v;
+    const uint2 x = one(v.x, a.x, a.y), y = one(v.y, a.z, a.w), z = one(v.z, b.x, b.y), w = one(v.w, b.z, b.w);
+    *at = make_uint4(x.x, y.x, z.x, w.x);
+    if (FORGET) rest_r[FORGET ? k : 0] = make_uint4(x.y, y.y, z.y, w.y);
   }
   __syncthreads();                                                 // A has been read
+  if (FORGET)
+#pragma unroll
+    for (int k = 0; k < PIECES; ++k) {
+      const int i = tid + k * CHT, t = i / (DK / 8), u = i % (DK / 8);
+      *reinterpret_cast<uint4*>(r_p + Cfg::kRLow + t * CH_ROWB + b_piece(t, u)) = rest_r[FORGET ? k : 0];
+    }
   constexpr int PART = DK * DK * 2;                                // one part of the state
 #pragma unroll 4
   for (int i = tid; i < 2 * (DK / 64) * DK * 8; i += CHT) {        // parts, 64 value channels, key row, 16-byte piece
@@ -1723,6 +1782,13 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_out_kernel(con
         for (int kk = 0; kk < DK / 16; ++kk) {
           const uint64_t a = make_smem_desc_sw128(r_s + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
           const uint64_t b = make_smem_desc_sw128(a_s + part * PART + z64 * DK * CH_ROWB + kk * 2048, CH_CHUNK, 1024);
+          umma_bf16(tmem + z64 * 64, a, b, idesc, 1u);
+        }
+      if (FORGET)
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk) {
+          const uint64_t a = make_smem_desc_sw128(r_s + Cfg::kRLow + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+          const uint64_t b = make_smem_desc_sw128(a_s + z64 * DK * CH_ROWB + kk * 2048, CH_CHUNK, 1024);
           umma_bf16(tmem + z64 * 64, a, b, idesc, 1u);
         }
     }
@@ -1781,14 +1847,14 @@ static int launch_time_mix(const MixParams& p, int n_chunks, int n_seq, cudaStre
   if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return -10;
   if (!attr[dev]) {
     if (cudaFuncSetAttribute(time_mix_state_kernel<DK, FORGET>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixStateCfg<DK>::kSmem) != cudaSuccess ||
-        cudaFuncSetAttribute(time_mix_out_kernel<DK, FORGET>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixOutCfg<DK>::kSmem) != cudaSuccess)
+        cudaFuncSetAttribute(time_mix_out_kernel<DK, FORGET>, cudaFuncAttributeMaxDynamicSharedMemorySize, MixOutCfg<DK, FORGET>::kSmem) != cudaSuccess)
       return -10;
     attr[dev] = true;
   }
   const dim3 units(n_chunks * p.H);
   if (launch_kernel(time_mix_state_kernel<DK, FORGET>, units, dim3(CHT), MixStateCfg<DK>::kSmem, stream, p) != cudaSuccess) return -11;
   if (launch_kernel(time_mix_chain_kernel, dim3(DK / 32, p.H * (p.VP / SC_COLS), n_seq), dim3(256), 0, stream, p) != cudaSuccess) return -12;
-  return launch_kernel(time_mix_out_kernel<DK, FORGET>, units, dim3(CHT), MixOutCfg<DK>::kSmem, stream, p) == cudaSuccess ? 0 : -13;
+  return launch_kernel(time_mix_out_kernel<DK, FORGET>, units, dim3(CHT), MixOutCfg<DK, FORGET>::kSmem, stream, p) == cudaSuccess ? 0 : -13;
 }
 
 }  // namespace rb
@@ -2234,7 +2300,7 @@ int rb_time_mix_chunks(const void* proj, long long ld, int k_col, int v_col, int
                        int dv, int KP, int num_slots, int* status, cudaStream_t stream) {
   if (n_chunks <= 0 || n_seq <= 0) return 0;
   if (H <= 0 || H * (KP / SC_COLS) > 65535 || n_seq > 65535 || dk <= 0 || dk > KP || ld % 8 != 0 || ldo % 8 != 0 || ldz % 4 != 0 || workspace == nullptr ||
-      (k_col | v_col | g_col) % 8 != 0 || dv <= 0 || dv > KP || ld_keys % 8 != 0)
+      (k_col | v_col | g_col) % 8 != 0 || dv <= 0 || dv > KP || ld_keys % 8 != 0 || (keys != nullptr && ld_keys < 2 * H * KP))
     return -1;
   const long long ch = (long long)n_chunks * H;
   MixParams p{};

@@ -276,7 +276,7 @@ class ForgetMixPart(Part):
 
     def allocate(self) -> None:
         r, n = self.r, max(w.geo.heads * w.geo.kp for w in self.layers)
-        self.keys, self.out = self.zeros(r.rows * n), self.zeros(r.rows * n)
+        self.keys, self.out = self.zeros(r.rows * 2 * n), self.zeros(r.rows * n)
         self.o = self.zeros(r.rows * n, dtype=torch.float32)
 
     def load(self, w: ForgetMixWeights, get, p: str) -> None:
@@ -303,7 +303,7 @@ class ForgetMixPart(Part):
     def recur(self, w: ForgetMixWeights, state: RecurrentState, proj, z, out, b, plan) -> None:
         T, g, eps = b.num_tokens, w.geo, self.r.cfg.norm_eps
         n = g.heads * g.kp
-        mix = ForgetMix(z, w.bias, w.lower, self.keys[:T * n].view(T, n))
+        mix = ForgetMix(z, w.bias, w.lower, self.keys[:T * 2 * n].view(T, 2 * n))
         n_seq, rows, table = plan if time_mix_chunked_supported(g) else (b.rows, T, None)
         single = b.rows if b.cu_q is None else b.n_single
         if single > 0:

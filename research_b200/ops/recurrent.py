@@ -121,8 +121,8 @@ class TimeMix:
 
 @dataclass
 class ForgetMix:
-    """Forget mixing: ``z [T, H*kp]`` fp32 with ``f = lower + (1 - lower) sigmoid(z + bias)``; ``keys [>= T, H*kp]`` is room for the chunked
-    form."""
+    """Forget mixing: ``z [T, H*kp]`` fp32 with ``f = lower + (1 - lower) sigmoid(z + bias)``; ``keys [>= T, 2 H*kp]`` is room for the
+    chunked form."""
 
     z: torch.Tensor
     bias: torch.Tensor           # [H*kp]

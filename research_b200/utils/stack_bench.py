@@ -3,7 +3,8 @@
 ``bench.py --workload stack`` runs it (``--designs``, ``--sizes`` choose). For every size two engines are built with random
 weights: Lulezen (latent attention) beside a Llama-type model, Zamusun (recurrent mixers, keys-as-values attention, routed
 experts, a looped pair of layers) and Fogurax (grouped attention with convolutions or chunks, attention beside time mixing, routed and
-shared experts, a per-layer token input) beside a Qwen3-MoE-type model, each with the same width, layer runs, feed-forward,
+shared experts, a per-layer token input) beside a Qwen3-MoE-type model, Sumitar (gated delta rule, attention beside forget mixing, identity
+experts, normed powers) beside Fogurax, each with the same width, layer runs, feed-forward,
 vocabulary and heads (grouped queries, head size 128). Measured with CUDA events, after warm-up:
 
 * decode: one captured decode step at the given batch and context, replayed;
@@ -25,9 +26,10 @@ from .. import ops
 from ..inference import EngineConfig, InferenceEngine
 from ..models import LazyRandomWeights
 from ..models.config import ModelConfig
-from ..models.stack import (DESIGNS as STACK_DESIGNS, BandScaling, ClampedGluSpec, ExpertsRouting, ExpertsSpec, GluSpec, GroupedAttentionSpec,
-                            KeyValueAttentionSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec, LoopSpec, MatrixMemorySpec,
-                            ParallelSpec, QueryTemperature, RotarySpec, TimeMixSpec, TokenSideSpec, YarnScaling, uniform_stack)
+from ..models.stack import (DESIGNS as STACK_DESIGNS, BandScaling, ClampedGluSpec, DeltaRuleSpec, ExpertsRouting, ExpertsSpec, ForgetMixSpec, GluSpec,
+                            GroupedAttentionSpec, KeyValueAttentionSpec, LatentAttentionSpec, LayerSpec, LayerStackConfig, LightningSpec, LoopSpec,
+                            MatrixMemorySpec, NormedPairSpec, ParallelSpec, PolyNormSpec, QueryTemperature, RotarySpec, TimeMixSpec, TokenSideSpec,
+                            YarnScaling, uniform_stack)
 from ..inference.stack_parts import DensePart
 from ..ops import experts as ex
 from .timing import flush_l2, time_cuda
@@ -119,6 +121,23 @@ def fogurax_stack(s: ExpertSize, layers: int, conv: int = 4, reach: int = 4096, 
 
 def fogurax_configs(s: ExpertSize):
     return fogurax_stack(s, s.runs), expert_configs(s)[1]
+
+
+def sumitar_stack(s: ExpertSize, layers: int, conv: int = 4, reach: int = 4096) -> LayerStackConfig:
+    """Two layers of the delta rule (heads of 128 channels, two share queries and keys), then attention beside forget mixing; the first feed-forward
+    has normed powers, the others route, one choice in sixteen an identity."""
+    H, kinds = s.heads, STACK_DESIGNS["Sumitar"].mixers
+    rule = DeltaRuleSpec(H, H // 2, 128, 128, conv)
+    left = GroupedAttentionSpec(kinds["parallel"].left, H, s.kv_heads, 128, 128, 128 ** -0.5, RotarySpec(64, 5e5), 1, reach)
+    both = NormedPairSpec("parallel", left, ForgetMixSpec(H, 128, 128))
+    plain = s.experts // 16
+    mlp = ExpertsSpec(s.experts - plain, s.top, GluSpec(s.ff), ExpertsRouting(normalize=False, correction=True, shared_gate=True), GluSpec(s.ff), plain)
+    return LayerStackConfig("Sumitar", s.vocab, s.width, tuple(LayerSpec(both if i % 3 == 2 else rule, PolyNormSpec(s.top * s.ff) if i == 0 else mlp)
+                                                               for i in range(layers)))
+
+
+def sumitar_configs(s: ExpertSize):
+    return sumitar_stack(s, s.runs), fogurax_stack(s, s.runs)
 
 
 def _engine(cfg, batch: int, context: int, prompt: int) -> InferenceEngine:
@@ -378,6 +397,83 @@ def fogurax_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) ->
     return t.rows
 
 
+def sumitar_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict:
+    """The first layer of every kind of mixer and feed-forward, and what joins them."""
+    r, cfg, t = eng.runner, eng.runner.cfg, _Table()
+    d, eps = cfg.hidden_size, cfg.norm_eps
+    x, h, y, y2 = r.x[:T], r.xb[:T], r.y[:T], r.y2[:T]
+    h.normal_()
+    b = r._decode_batch(T) if decode else _prompt_batch(r, T)
+    run = next(x for x in r.runs if x.layer.spec.mixer.type == "delta")
+    lw, w, part, cache = run.layer, run.layer.mix, run.layer.mixer, run.cache
+    g, plan = w.geo, part.planned(b)
+    H, n = g.heads, g.heads * g.vp
+    t.gemm("delta: joint projection", T, w.wproj.shape[0], r.wp, lambda: r._project(lw, h))
+    small = r._project(lw, h)
+    rows, rule = part.prepare(w, cache, small, b)
+    t.add("delta: convolution + units", lambda: part.prepare(w, cache, small, b), 2 * T * g.channels * (2 + ((w.spec.taps - 1) * 2 if decode else 0)), 0)
+    o, out = part.o[:T * n].view(T, n), part.out[:T * n].view(T, n)
+    t.add("delta: recurrence", lambda: part.recur(w, cache, rows, rule, o, b, plan), T * (2 * g.channels + 4 * n) + 2 * 4 * H * g.kp * g.vp * b.rows,
+          T * H * ((6.0 if decode else 8.0) * g.kp * g.vp + (0 if decode else 2.0 * 64 * (3 * g.kp + 2 * g.vp))))
+    t.add("delta: norm + gate", lambda: ops.gated_norm(o, w.norm, part._projected(w, T)[:, g.offsets[3]:], g, eps, out, True, silu=True), T * n * 8, 0)
+    t.gemm("delta: output projection", T, r.wp, n, lambda: ops.gemm(out, w.wo, out=y, out_f32=True), 4)
+
+    run = next(x for x in r.runs if x.layer.spec.mixer.type == "parallel")
+    pair, left, right = run.layer.mix, run.layer.mixer.left, run.layer.mixer.right
+    w, g, plan = pair.left, pair.left.geo, left.planned(b)
+    H, G, D, n = g.heads, g.kv_heads, g.dp, g.heads * g.dp
+    t.gemm("parallel: joint projection", T, pair.wproj.shape[0], r.wp, lambda: r._project(run.layer, h))
+    small = r._project(run.layer, h)
+    proj = run.layer.mixer._projected(pair, T)
+    q, out = left.q[:T * n].view(T, n), left.out[:T * n].view(T, n)
+    t.add("parallel: rotation + append", lambda: ops.grouped_append(
+        proj[:, pair.right.geo.proj:], g, conv=None, cache=run.cache[0], cu_q=b.cu_q, positions=b.positions, state_slots=b.state_slots, slots=b.slots,
+        q_norm=None, k_norm=None, eps=eps, table=w.table, q=q, q_factor=w.temp), 2 * T * g.channels * 2, 0)
+    fn = lambda: ops.grouped_attention(q, g, run.cache[0], b.block_tables, b.cu_q, b.seq_lens, out, scale=w.spec.scale, rows=T, max_q=b.max_new,
+                                       n_single=b.n_single, workspace=left.workspace, splits=plan.get(g, 1))
+    if decode:
+        span = min(context, g.window)
+        t.add("parallel: attention", fn, 2 * T * (2 * span * G * D + 2 * H * D), 4.0 * T * H * span * D)
+    else:
+        t.add("parallel: attention", fn, 2 * T * D * (2 * H + 2 * G), 4.0 * sum(min(i + 1, g.window) for i in range(T)) * H * D)
+    t.gemm("parallel: output projection, attention", T, r.wp, n, lambda: ops.gemm(out, w.wo, out=y, out_f32=True), 4)
+    rw, rg = pair.right, pair.right.geo
+    m = rg.heads * rg.vp
+    mixed = right.out[:T * m].view(T, m)
+    t.add("parallel: forget mixing + norm", lambda: right.recur(rw, run.cache[1], proj, small, mixed, b, right.planned(b)),
+          T * m * (2 * 3 + 4) + 2 * 4 * m * rg.kp * b.rows, T * rg.heads * (4.0 * rg.kp * rg.vp + (0 if decode else 2.0 * 64 * (rg.kp + rg.vp))))
+    t.gemm("parallel: output projection, forget mixing", T, r.wp, m, lambda: ops.gemm(mixed, rw.wo, out=y2, out_f32=True), 4)
+    norms = dict(post=lw.norm1b, pre=lw.norm2, eps=eps, h=h)
+    t.add("halves' norms + residual + norm", lambda: ops.stream_sandwich(x, d, y=y, pair=(y2, pair.left_out, pair.right_out), **norms), T * d * (4 * 4 + 2), 0)
+    t.add("norm + residual + norm", lambda: ops.stream_sandwich(x, d, y=y, **norms), T * d * (4 * 3 + 2), 0)
+
+    lw = r.layers[0]
+    w, act = lw.ff, lw.feed_forward
+    z, a = act.z[:T * w.ffp].view(T, w.ffp), act.a[:T * w.ffp].view(T, w.ffp)
+    t.gemm("dense: up", T, w.ffp, r.wp, lambda: ops.gemm(h, w.wu, out=z))
+    t.add("dense: normed powers", lambda: ops.poly_norm(z, w.act, w.spec.ff, eps, a), T * w.ffp * 4, 0)
+    t.gemm("dense: down", T, r.wp, w.ffp, lambda: ops.gemm(a, w.wd, out=y, out_f32=True), 4)
+    lw = next(x for x in r.layers if x.spec.mlp.kind == "moe")
+    small = r._small_rows(h, lw.wsmall_ff)
+    e, g = lw.ff, lw.ff.geo
+    sc = lw.feed_forward.scratch[g]
+    t.gemm("router", T, lw.wsmall_ff.shape[0], r.wp, lambda: r._small_rows(h, lw.wsmall_ff), 4)
+    _routed(t, T, g.experts, g.top, d, g.ff, lambda: ex.experts_up(g, sc, e.wgu, T), lambda: ex.experts_down(g, sc, e.wd), None,
+            {"experts route + plan": (lambda: ex.experts_plan(small, g, sc, e.correction), T * (4 * g.choices + 8 * g.top)),
+             "experts gather": (lambda: (ex.experts_plan(small, g, sc, e.correction), ex.experts_gather(h, g, sc)), 2 * 2 * T * g.top * d)})
+    shared = e.shared
+    act = r._part(DensePart).act[:T * shared.ffp].view(T, shared.ffp)
+    t.gemm("shared gate|up + unit", T, 2 * shared.ffp, r.wp, lambda: ops.gemm(h, shared.wgu, out=act, bn=256, swiglu=True), 2, shared.ffp)
+    t.gemm("shared down", T, r.wp, shared.ffp, lambda: ops.gemm(act, shared.wd, out=y, out_f32=True), 4)
+    chosen = ops.ChosenExperts(sc.y[:T * g.top], sc.w[:T], sc.idx[:T], g.experts, h)
+    t.add("experts' sum + norm + residual + norm", lambda: ops.stream_sandwich(x, d, y=y, gate=small[:, g.choices:], chosen=chosen, **norms),
+          T * d * (4 * 3 + 2 + 2 * g.top), 0)
+    if decode:
+        lg = r.logits_padded[:T]
+        t.gemm("head", T, r.vp, r.wp, lambda: r._head(r.hl[:T], lg), 4)
+    return t.rows
+
+
 def _time_mix_rows(t: _Table, r, part, w, cache, h, out, b, T: int, decode: bool) -> None:
     g, eps = w.geo, r.cfg.norm_eps
     n = g.heads * g.kp
@@ -452,7 +548,8 @@ def hf_kernels(eng: InferenceEngine, T: int, context: int, decode: bool) -> dict
 # design -> (sizes, pair of configurations, labels and kernel tables)
 DESIGNS = {"lulezen": (SIZES, configs, (("lulezen", latent_kernels), ("llama", hf_kernels))),
            "zamusun": (EXPERT_SIZES, expert_configs, (("zamusun", expert_stack_kernels), ("qwen3_moe", hf_kernels))),
-           "fogurax": (EXPERT_SIZES, fogurax_configs, (("fogurax", fogurax_kernels), ("qwen3_moe", hf_kernels)))}
+           "fogurax": (EXPERT_SIZES, fogurax_configs, (("fogurax", fogurax_kernels), ("qwen3_moe", hf_kernels))),
+           "sumitar": (EXPERT_SIZES, sumitar_configs, (("sumitar", sumitar_kernels), ("fogurax", fogurax_kernels)))}
 
 
 def run(sizes: tuple[str, ...] = (), batches: tuple[int, ...] = (1, 64, 256), context: int = 2048, prompts: tuple[int, ...] = (512, 4096),

@@ -90,7 +90,7 @@ def test_forget_mixing_in_portions_slots_and_batches(place, shape):
         b = bt.step(parts, dt == torch.bfloat16 and dev == "cuda" and time_mix_chunked_supported(geo))
         q, v, z = (b.rows([d[i] for d in data]) for i in range(3))
         proj = torch.cat([padded(q, geo.kp), padded(v, geo.vp), torch.full((b.T, 8), 9.0)], 1).to(dt).to(dev)
-        mix = ForgetMix(padded(z, geo.kp).to(dev), bias_p, lower_p, torch.full((b.T, n), 3.0, dtype=dt, device=dev))
+        mix = ForgetMix(padded(z, geo.kp).to(dev), bias_p, lower_p, torch.full((b.T, 2 * n), 3.0, dtype=dt, device=dev))
         o, out = torch.full((b.T, H * geo.vp), 9.0, device=dev), torch.full((b.T, H * geo.vp + 8), 9.0, dtype=dt, device=dev)[:, :H * geo.vp]
         if b.single:
             ops.time_mix_decode(proj, geo, mix, state, b.state_slots, b.seq_lens, norm_p, eps, out, b.single)
