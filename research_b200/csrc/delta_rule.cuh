@@ -169,19 +169,19 @@ static cudaError_t launch_delta_rows(const DeltaRows& p, cudaStream_t stream) {
 // second one goes over a sequence's chunks with U = T diag(beta) V - W S, and the outputs are recurrent_chunk_out_kernel's with U for
 // the values. All factors of the keys are applied in fp32 outside the products; T, W, U and S go in as two bf16 parts each.
 //
-// The inverse: its eight 16 x 16 blocks on the diagonal by substitution in fp32, the others by mma.sync with operands in two parts.
-// Warp j makes column j of blocks, transposed, X_ij^T = -(sum_(j <= k < i) X_kj^T L_ik^T) X_ii^T, so that every result is the next
-// product's first operand as it lies in the registers.
+// The inverse X: its eight 16 x 16 blocks on the diagonal by substitution in fp32, the others by mma.sync with operands in two parts.
+// Warp j makes column j of blocks, transposed, X_ij^T = -(sum_(j <= k < i) X_kj^T L_ik^T) X_ii^T, and leaves it in fp32 where L has nothing:
+// L fills the blocks below the diagonal of one square, X^T the others.
 // ------------------------------------------------------------------------------------------
 struct DeltaParams {
   ChunkParams c;
   const float* units;      // [T, 2 G]
   const float* steps;      // [T, 2 H]
-  __nv_bfloat16* w_hi;     // [chunks, H, KP / 64, CH, 64]
+  __nv_bfloat16* w_hi;     // [chunks, H, KP / 64, CH, 64], tiles as they lie in shared memory (chunk_addr)
   __nv_bfloat16* w_lo;
-  float* uv;               // [chunks, H, VP / 64, CH, 64]
-  __nv_bfloat16* values;   // [T, ld_values] U
-  long long ld_values;
+  __nv_bfloat16* keys;     // [chunks, G, KP / 64, CH, 64], so too
+  float* uv;               // [chunks, H, VP / 64, 16, CH, 4]
+  __nv_bfloat16* values;   // [chunks, H, VP / 64, 8, CH, 8] U
 };
 
 // Place of L[t][j]: groups of eight exchanged by the row's low bits, so that four rows of a fragment meet no bank twice.
@@ -195,20 +195,16 @@ struct DeltaSolveCfg {
   static constexpr int kCols = 256;
 };
 
-// A 16 x 16 block as first operand of mma.sync (and, four accumulators of an n = 8 product after the other, as its result).
+// A 16 x 16 block as first operand of mma.sync, in two parts, from pairs (row g, columns c, c + 1), (g + 8, ..), (g, c + 8 ..), (g + 8, c + 8 ..).
 struct Block16 {
   uint32_t hi[4], lo[4];
-  __device__ __forceinline__ void set(const float (&lower)[4], const float (&upper)[4], float sign) {      // columns 0 .. 7, 8 .. 15
-    split_bf16x2(sign * lower[0], sign * lower[1], hi[0], lo[0]);
-    split_bf16x2(sign * lower[2], sign * lower[3], hi[1], lo[1]);
-    split_bf16x2(sign * upper[0], sign * upper[1], hi[2], lo[2]);
-    split_bf16x2(sign * upper[2], sign * upper[3], hi[3], lo[3]);
-  }
+  __device__ __forceinline__ void set(int e, float x, float y) { split_bf16x2(x, y, hi[e], lo[e]); }
 };
 
-// acc[2] += a m^T for a block m of fp32 rows: column n of the product goes with row n of m. `m(row, column)` is the address of two elements.
+// acc += a m^T for a block m of fp32 rows, the two halves of the columns and the three products of parts apart: column n of the product goes
+// with row n of m. `m(row, column)` is the address of two elements.
 template <typename Block>
-__device__ __forceinline__ void block_product(float (&acc)[2][4], const Block16& a, Block m, int lane) {
+__device__ __forceinline__ void block_product(float (&acc)[2][3][4], const Block16& a, Block m, int lane) {
   const int g = lane >> 2, c = 2 * (lane & 3);
 #pragma unroll
   for (int q = 0; q < 2; ++q) {
@@ -216,9 +212,9 @@ __device__ __forceinline__ void block_product(float (&acc)[2][4], const Block16&
     uint32_t h0, l0, h1, l1;
     split_bf16x2(x.x, x.y, h0, l0);
     split_bf16x2(y.x, y.y, h1, l1);
-    mma_16816_bf16(acc[q], a.hi[0], a.hi[1], a.hi[2], a.hi[3], h0, h1);
-    mma_16816_bf16(acc[q], a.lo[0], a.lo[1], a.lo[2], a.lo[3], h0, h1);
-    mma_16816_bf16(acc[q], a.hi[0], a.hi[1], a.hi[2], a.hi[3], l0, l1);
+    mma_16816_bf16(acc[q][0], a.hi[0], a.hi[1], a.hi[2], a.hi[3], h0, h1);
+    mma_16816_bf16(acc[q][1], a.lo[0], a.lo[1], a.lo[2], a.lo[3], h0, h1);
+    mma_16816_bf16(acc[q][2], a.hi[0], a.hi[1], a.hi[2], a.hi[3], l0, l1);
   }
 }
 
@@ -305,6 +301,7 @@ __global__ void __launch_bounds__(CHT, 2) delta_solve_kernel(const DeltaParams p
     umma_commit(smem_u32(&done));
   }
   __syncwarp();
+  if (tid == 32 && h % c.ratio == 0) bulk_store(p.keys + ((long long)chunk * G + hk) * DK * CH, k_s, Cfg::kKBytes);
   const int qd = warp & 3, half = warp >> 2, t = qd * 32 + lane;
   const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
   int phase = 0;
@@ -335,69 +332,92 @@ __global__ void __launch_bounds__(CHT, 2) delta_solve_kernel(const DeltaParams p
   }
   ok = __syncthreads_and(ok);
   if (ok) {
+    auto at = [&](int row, int col) { return L + inverse_at(row, col); };
+    const int j16 = warp * 16;
     {                                                    // the warp's diagonal block, a column per lane
       float x[16];
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         float s = 0.f;
 #pragma unroll
-        for (int j = 0; j < i; ++j) s = fmaf(L[inverse_at(warp * 16 + i, warp * 16 + j)], x[j], s);
+        for (int j = 0; j < i; j += 4) {
+          const float4 l = *reinterpret_cast<const float4*>(at(j16 + i, j16 + j));
+          s = fmaf(l.x, x[j], s);
+          if (j + 1 < i) s = fmaf(l.y, x[j + 1 < i ? j + 1 : 0], s);
+          if (j + 2 < i) s = fmaf(l.z, x[j + 2 < i ? j + 2 : 0], s);
+          if (j + 3 < i) s = fmaf(l.w, x[j + 3 < i ? j + 3 : 0], s);
+        }
         x[i] = (i == (lane & 15) ? 1.f : 0.f) - s;
       }
-      if (lane < 16)
+      __syncwarp();
+      if (lane < 16) {
 #pragma unroll
         for (int i = 0; i < 16; ++i) diag[warp][i][lane] = x[i];
+#pragma unroll
+        for (int i = 0; i < 16; i += 4) *reinterpret_cast<float4*>(at(j16 + lane, j16 + i)) = make_float4(x[i], x[i + 1], x[i + 2], x[i + 3]);
+      }
     }
     __syncthreads();
-    Block16 Y[8];                                        // X_ij^T of this warp's j
     const int g = lane >> 2, cq = 2 * (lane & 3);
-    {
-      float lower[4], upper[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int m = g + (e >> 1) * 8, k = cq + (e & 1);
-        lower[e] = diag[warp][k][m];
-        upper[e] = diag[warp][k + 8][m];
-      }
-#pragma unroll
-      for (int i = 0; i < 8; ++i)
-        if (i == warp) Y[i].set(lower, upper, 1.f);
-    }
-#pragma unroll
-    for (int i = 1; i < 8; ++i) {
-      if (i <= warp) continue;
-      float acc[2][4] = {};
-#pragma unroll
-      for (int k = 0; k < i; ++k)
-        if (k >= warp) block_product(acc, Y[k], [&](int row, int col) { return L + inverse_at(i * 16 + row, k * 16 + col); }, lane);
-      Block16 sum;
-      sum.set(acc[0], acc[1], -1.f);
-      float x[2][4] = {};
-      block_product(x, sum, [&](int row, int col) { return &diag[i][row][col]; }, lane);
-      Y[i].set(x[0], x[1], 1.f);
-    }
-    __syncthreads();                                     // L has been read
-    // T^T with its rows (columns of T) scaled, in two parts, [CH, CH] as two tiles of 64 columns each
-    auto store_inverse = [&](float s0, float s1) {       // factors of rows 16 warp + g and + 8
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
+#pragma unroll 1
+    for (int i16 = j16 + 16; i16 < CH; i16 += 16) {
+      float acc[2][3][4] = {};
+#pragma unroll 2
+      for (int k16 = j16; k16 < i16; k16 += 16) {
+        Block16 a;
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int row = warp * 16 + g + (e & 1) * 8, col = i * 16 + (e >> 1) * 8 + cq;
-          uint32_t hi = 0u, lo = 0u;
-          if (i >= warp) {
-            const float2 a = unpack_bf16x2(Y[i].hi[e]), b = unpack_bf16x2(Y[i].lo[e]);
-            const float s = e & 1 ? s1 : s0;
-            split_bf16x2((a.x + b.x) * s, (a.y + b.y) * s, hi, lo);
-          }
-          uint8_t* at = t_p + (col >> 6) * CH_CHUNK + chunk_addr(row, (col & 63) >> 3) + (col & 7) * 2;
-          *reinterpret_cast<uint32_t*>(at) = hi;
-          *reinterpret_cast<uint32_t*>(at + 2 * CH_CHUNK) = lo;
+          const float2 v = *reinterpret_cast<const float2*>(at(j16 + g + (e & 1) * 8, k16 + cq + (e >> 1) * 8));
+          a.set(e, v.x, v.y);
         }
+        block_product(acc, a, [&](int row, int col) { return at(i16 + row, k16 + col); }, lane);
+      }
+      Block16 sum;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int q = e >> 1, h2 = (e & 1) * 2;
+        sum.set(e, -(acc[q][0][h2] + acc[q][1][h2] + acc[q][2][h2]), -(acc[q][0][h2 + 1] + acc[q][1][h2 + 1] + acc[q][2][h2 + 1]));
+      }
+      float x[2][3][4] = {};
+      block_product(x, sum, [&](int row, int col) { return &diag[i16 >> 4][row][col]; }, lane);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int q = e >> 1, h2 = (e & 1) * 2;
+        *reinterpret_cast<float2*>(at(j16 + g + (e & 1) * 8, i16 + cq + q * 8)) =
+            make_float2(x[q][0][h2] + x[q][1][h2] + x[q][2][h2], x[q][0][h2 + 1] + x[q][1][h2 + 1] + x[q][2][h2 + 1]);
+      }
+      __syncwarp();
+    }
+    __syncthreads();
+    // X^T with its rows (columns of the inverse) scaled, in two parts, [CH, CH] as two tiles of 64 columns each: the square it comes from is
+    // overwritten, so every thread keeps its eight pieces of eight columns (row 16 k + tid / 16, piece tid % 16).
+    float X[8][8];
+    const int piece = tid & 15;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int row = k * 16 + (tid >> 4);
+#pragma unroll
+      for (int e = 0; e < 8; e += 4) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (piece >> 1 >= k) v = *reinterpret_cast<const float4*>(at(row, piece * 8 + e));
+        X[k][e] = v.x; X[k][e + 1] = v.y; X[k][e + 2] = v.z; X[k][e + 3] = v.w;
+      }
+    }
+    __syncthreads();
+    auto store_inverse = [&](bool keys) {                // for the product with the keys, or with the values
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int row = k * 16 + (tid >> 4);
+        const float f = keys ? betas[row] * rks[row] * chunk_exp2(Fs[row]) : betas[row];
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split_bf16x2(X[k][2 * e] * f, X[k][2 * e + 1] * f, hi[e], lo[e]);
+        uint8_t* dst = t_p + (piece >> 3) * CH_CHUNK + chunk_addr(row, piece & 7);
+        *reinterpret_cast<uint4*>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(dst + 2 * CH_CHUNK) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
       }
     };
-    const int ra = warp * 16 + g, rb8 = ra + 8;
-    store_inverse(betas[ra] * rks[ra] * chunk_exp2(Fs[ra]), betas[rb8] * rks[rb8] * chunk_exp2(Fs[rb8]));
+    store_inverse(true);
     fence_proxy_async_smem();
     tc_fence_before();
     __syncthreads();
@@ -422,6 +442,7 @@ __global__ void __launch_bounds__(CHT, 2) delta_solve_kernel(const DeltaParams p
     __syncwarp();
     phase ^= 1;
     ok = mbar_wait_bounded(smem_u32(&done), phase, &abort_flag, c.status, ST_TIMEOUT_TMEM_FULL);
+    if (tid == 32) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
     ok = __syncthreads_and(ok);                          // K and the inverse have been read
     if (ok) {
       const __nv_bfloat16* v = rows + c.v_col + h * c.VP;
@@ -430,23 +451,31 @@ __global__ void __launch_bounds__(CHT, 2) delta_solve_kernel(const DeltaParams p
         for (int z = z0; z < min(z0 + DK / 64, tiles); ++z) chunk_load<64>(k_s + (z - z0) * CH_CHUNK, v + z * 64, c.ld, n);
       };
       load_values(0);
-      store_inverse(betas[ra], betas[rb8]);
       tc_fence_after();
 #pragma unroll
-      for (int z = 0; z < DK / 64; ++z) {                // W
+      for (int z = 0; z < DK / 64; ++z) {                // W, over the inverse, and from there to global memory as it lies
         uint32_t w[32];
         tmem_ld_32x32(tmem + z * 64 + half * 32 + lane_addr, w);
         tmem_ld_wait();
-        const long long at = ((ch * (DK / 64) + z) * CH + t) * 64 + half * 32;
 #pragma unroll
-        for (int i = 0; i < 32; i += 8) {
+        for (int i = 0; i < 4; ++i) {
           uint32_t hi[4], lo[4];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) split_bf16x2(__uint_as_float(w[i + 2 * e]), __uint_as_float(w[i + 2 * e + 1]), hi[e], lo[e]);
-          *reinterpret_cast<uint4*>(p.w_hi + at + i) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(p.w_lo + at + i) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          for (int e = 0; e < 4; ++e) split_bf16x2(__uint_as_float(w[8 * i + 2 * e]), __uint_as_float(w[8 * i + 2 * e + 1]), hi[e], lo[e]);
+          uint8_t* dst = t_p + z * CH_CHUNK + chunk_addr(t, half * 4 + i);
+          *reinterpret_cast<uint4*>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4*>(dst + Cfg::kKBytes) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         }
       }
+      fence_proxy_async_smem();
+      __syncthreads();
+      if (tid == 32) {
+        bulk_store(p.w_hi + ch * DK * CH, t_s, Cfg::kKBytes);
+        bulk_store(p.w_lo + ch * DK * CH, t_s + Cfg::kKBytes, Cfg::kKBytes);
+        asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
+      }
+      __syncthreads();
+      store_inverse(false);
       for (int z0 = 0; ok && z0 < tiles; z0 += DK / 64) {
         const int have = min(DK / 64, tiles - z0);
         cp_async_wait_all();
@@ -466,16 +495,17 @@ __global__ void __launch_bounds__(CHT, 2) delta_solve_kernel(const DeltaParams p
           uint32_t u[32];
           tmem_ld_32x32(tmem + 128 + z * 64 + half * 32 + lane_addr, u);
           tmem_ld_wait();
-          float4* dst = reinterpret_cast<float4*>(p.uv + ((ch * tiles + z0 + z) * CH + t) * 64 + half * 32);
+          float4* dst = reinterpret_cast<float4*>(p.uv) + ((ch * tiles + z0 + z) * 16 + half * 8) * CH + t;
 #pragma unroll
           for (int i = 0; i < 8; ++i)
-            dst[i] = make_float4(__uint_as_float(u[4 * i]), __uint_as_float(u[4 * i + 1]), __uint_as_float(u[4 * i + 2]), __uint_as_float(u[4 * i + 3]));
+            dst[i * CH] = make_float4(__uint_as_float(u[4 * i]), __uint_as_float(u[4 * i + 1]), __uint_as_float(u[4 * i + 2]), __uint_as_float(u[4 * i + 3]));
         }
       }
       tc_fence_before();
     }
   }
   cp_async_wait_all();
+  if (tid == 32) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
@@ -483,20 +513,25 @@ __global__ void __launch_bounds__(CHT, 2) delta_solve_kernel(const DeltaParams p
   }
 }
 
-// The chunks of a sequence one after the other, 64 value channels of a head per CTA; the state in registers.
+// The chunks of a sequence one after the other, 64 value channels of a head per CTA; the state in registers. A chunk is two products one
+// behind the other (W S, then K^T U), each with both parts of its second operand side by side; what is written to global memory, and
+// the next chunk's vectors, pass while the products run.
+constexpr int DC_THREADS = 512, DC_COLS = 64 / (DC_THREADS / 128);     // value channels of a thread's row
+
 template <int DK>
 struct DeltaChainCfg {
   static constexpr int kWBytes = CH * DK * 2;                      // one part of W; K
   static constexpr int kSBytes = DK * CH_ROWB;                     // one part of the state
   static constexpr int kSmem = 1024 + 3 * kWBytes + 2 * kSBytes + 2 * CH_CHUNK;
-  static constexpr int kCols = 128;                                // W S 64 | K^T U 64
+  static constexpr int kCols = 256;                                // W S, K^T U: with the first and the second part of S, U
 };
 
 template <int DK>
-__global__ void __launch_bounds__(CHT) delta_chain_kernel(const DeltaParams p) {
+__global__ void __launch_bounds__(DC_THREADS) delta_chain_kernel(const DeltaParams p) {
   using Cfg = DeltaChainCfg<DK>;
+  static_assert(DC_COLS == 16, "a thread's row is one TMEM load");
   extern __shared__ __align__(128) uint8_t smem_raw[];
-  __shared__ __align__(8) uint64_t u_done, s_done;
+  __shared__ __align__(8) uint64_t u_done, s_done, w_full, k_full;
   __shared__ uint32_t tmem_base_smem;
   __shared__ int abort_flag;
   const ChunkParams& c = p.c;
@@ -509,6 +544,8 @@ __global__ void __launch_bounds__(CHT) delta_chain_kernel(const DeltaParams p) {
     abort_flag = 0;
     mbar_init(smem_u32(&u_done), 1);
     mbar_init(smem_u32(&s_done), 1);
+    mbar_init(smem_u32(&w_full), 1);
+    mbar_init(smem_u32(&k_full), 1);
     fence_mbar_init();
   }
   if (warp == 1) {
@@ -522,153 +559,187 @@ __global__ void __launch_bounds__(CHT) delta_chain_kernel(const DeltaParams p) {
   pdl_launch_dependents();
   pdl_wait();
   const int z = blockIdx.x, h = blockIdx.y, b = blockIdx.z, hk = h / c.ratio;
-  const int qd = warp & 3, half = warp >> 2, t = qd * 32 + lane;
+  const int qd = warp & 3, col = (warp >> 2) * DC_COLS, t = qd * 32 + lane;
   const uint32_t lane_addr = (uint32_t)(qd * 32) << 16;
   const int slot = c.slots[b];
   if (slot >= 0 && slot < c.num_slots) {
     const bool fresh = c.seq_lens[b] == c.cu_q[b + 1] - c.cu_q[b];
     const int c0 = c.seq_chunks[b], c1 = c.seq_chunks[b + 1];
-    // key row of this thread's 32 value channels (a 64-row product: row 16 q + lane in 16 lanes)
+    // key row of this thread's value channels (a 64-row product: row 16 q + lane in 16 lanes)
     const int r = DK == 128 ? t : qd * 16 + lane;
     const bool holds = DK == 128 || lane < 16, live = holds && r < c.dk;
-    float4* st = reinterpret_cast<float4*>(c.s + ((((long long)slot * c.H + h) * (c.VP / SC_COLS) + z * 2 + half) * c.KP + (holds ? r : 0)) * SC_COLS);
-    float S[32];
+    float4* st = reinterpret_cast<float4*>(c.s + ((((long long)slot * c.H + h) * (c.VP / SC_COLS) + z * 2 + col / SC_COLS) * c.KP + (holds ? r : 0)) * SC_COLS +
+                                           col % SC_COLS);
+    float S[DC_COLS];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < DC_COLS / 4; ++i) {
       float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
       if (live && !fresh) v = st[i];
       S[4 * i] = v.x; S[4 * i + 1] = v.y; S[4 * i + 2] = v.z; S[4 * i + 3] = v.w;
     }
+    int w_loads = 0, k_loads = 0;                        // thread 0: copies on their way or landed
     auto load_w = [&](int k) {
       const long long at = ((long long)k * c.H + h) * DK * CH;
-#pragma unroll 4
-      for (int i = tid; i < 2 * CH * (DK / 8); i += CHT) {         // parts, tiles of 64 columns, rows, pieces
-        const int part = i / (CH * (DK / 8)), e = i % (CH * (DK / 8)), row = (e >> 3) % CH;
-        cp_async16(w_s + part * Cfg::kWBytes + (e >> 3) / CH * CH_CHUNK + chunk_addr(row, e & 7), (part ? p.w_lo : p.w_hi) + at + e * 8, true);
-      }
+      const uint32_t bar = smem_u32(&w_full);
+      mbar_expect_tx(bar, 2 * Cfg::kWBytes);
+      bulk_load(w_s, p.w_hi + at, Cfg::kWBytes, bar);
+      bulk_load(w_s + Cfg::kWBytes, p.w_lo + at, Cfg::kWBytes, bar);
+      ++w_loads;
     };
     auto load_k = [&](int k) {
-      const int4 ck = c.chunks[k];
-      chunk_load<DK>(k_s, c.proj + (long long)ck.x * c.ld + c.k_col + hk * c.KP, c.ld, ck.y);
+      const uint32_t bar = smem_u32(&k_full);
+      mbar_expect_tx(bar, Cfg::kWBytes);
+      bulk_load(k_s, p.keys + ((long long)k * (c.H / c.ratio) + hk) * DK * CH, Cfg::kWBytes, bar);
+      ++k_loads;
     };
     // what a thread needs of a chunk besides: its row of T diag(beta) V, the factor of its key, the chunk's decay
-    float4 uv[8];
+    float4 uv[DC_COLS / 4];
     float factor = 0.f, decay = 0.f;
     auto fetch = [&](int k) {
       const long long ch = (long long)k * c.H + h;
-      const float4* src = reinterpret_cast<const float4*>(p.uv + ((ch * (c.VP / 64) + z) * CH + t) * 64 + half * 32);
+      const float4* src = reinterpret_cast<const float4*>(p.uv) + ((ch * (c.VP / 64) + z) * 16 + col / 4) * CH + t;
 #pragma unroll
-      for (int i = 0; i < 8; ++i) uv[i] = src[i];
+      for (int i = 0; i < DC_COLS / 4; ++i) uv[i] = src[i * CH];
       decay = c.um[ch].x;
       factor = c.gates[ch * 3 * CH + t];
     };
-    if (c0 < c1) { load_w(c0); load_k(c0); fetch(c0); }
+    if (c0 < c1) {
+      if (tid == 0) { load_w(c0); load_k(c0); }
+      fetch(c0);
+    }
     bool ok = true;
+    constexpr int MOVER = DC_THREADS - 32;               // the thread that stores the state's parts
     for (int k = c0; k < c1; ++k) {
       const uint32_t phase = (uint32_t)((k - c0) & 1);
       const long long ch = (long long)k * c.H + h;
-      const int4 ck = c.chunks[k];
+      uint4 hi[2], lo[2];
+      auto split8 = [](const float (&x)[DC_COLS], int i, uint4& a, uint4& d) {
+        split_bf16x2(x[i], x[i + 1], a.x, d.x);
+        split_bf16x2(x[i + 2], x[i + 3], a.y, d.y);
+        split_bf16x2(x[i + 4], x[i + 5], a.z, d.z);
+        split_bf16x2(x[i + 6], x[i + 7], a.w, d.w);
+      };
       if (holds) {
-        const long long at = ((ch * (c.VP / 64) + z) * c.KP + r) * 64 + half * 32;
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          uint32_t hi[4], lo[4];
-#pragma unroll
-          for (int e = 0; e < 4; ++e) split_bf16x2(S[i * 8 + 2 * e], S[i * 8 + 2 * e + 1], hi[e], lo[e]);
-          const uint4 a = make_uint4(hi[0], hi[1], hi[2], hi[3]), d = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-          const uint32_t o = chunk_addr(r, half * 4 + i);
-          *reinterpret_cast<uint4*>(s_p + o) = a;
-          *reinterpret_cast<uint4*>(s_p + Cfg::kSBytes + o) = d;
-          *reinterpret_cast<uint4*>(c.s_hi + at + i * 8) = a;
-          *reinterpret_cast<uint4*>(c.s_lo + at + i * 8) = d;
+        for (int i = 0; i < 2; ++i) {
+          split8(S, i * 8, hi[i], lo[i]);
+          const uint32_t o = chunk_addr(r, col / 8 + i);
+          *reinterpret_cast<uint4*>(s_p + o) = hi[i];
+          *reinterpret_cast<uint4*>(s_p + Cfg::kSBytes + o) = lo[i];
         }
       }
-      cp_async_wait_all();
       fence_proxy_async_smem();
       tc_fence_before();
+      if (warp == 0 && ok) ok = __all_sync(0xffffffffu, mbar_wait_bounded(smem_u32(&w_full), phase, &abort_flag, c.status, ST_TIMEOUT_SMEM_FULL));
       ok = __syncthreads_and(ok);
       if (!ok) break;
       tc_fence_after();
-      if (warp == 0 && elect_one_sync()) {
-        constexpr uint32_t idesc = make_idesc_bf16(CH, 64, 0, 1);
+      if (warp == 0 && elect_one_sync()) {                         // W S without the product of the two small parts
+        constexpr uint32_t both = make_idesc_bf16(CH, 128, 0, 1), one = make_idesc_bf16(CH, 64, 0, 1);
 #pragma unroll
-        for (int part = 0; part < 3; ++part)                       // W S without the product of the two small parts
+        for (int part = 0; part < 2; ++part)
 #pragma unroll
           for (int kk = 0; kk < DK / 16; ++kk) {
-            const uint64_t a = make_smem_desc_sw128(w_s + (part == 1 ? Cfg::kWBytes : 0) + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
-            const uint64_t d = make_smem_desc_sw128(s_s + (part == 2 ? Cfg::kSBytes : 0) + kk * 2048, CH_CHUNK, 1024);
-            umma_bf16(tmem, a, d, idesc, (part | kk) ? 1u : 0u);
+            const uint64_t a = make_smem_desc_sw128(w_s + part * Cfg::kWBytes + (kk >> 2) * CH_CHUNK + (kk & 3) * 32, 16, 1024);
+            const uint64_t d = make_smem_desc_sw128(s_s + kk * 2048, Cfg::kSBytes, 1024);
+            umma_bf16(tmem, a, d, part ? one : both, (part | kk) ? 1u : 0u);
           }
         umma_commit(smem_u32(&u_done));
+      }
+      __syncwarp();
+      const long long tile = ch * (c.VP / 64) + z;
+      if (tid == MOVER) {                                          // the state in front of the chunk, for the outputs
+        bulk_store(c.s_hi + tile * c.KP * 64, s_s, Cfg::kSBytes);
+        bulk_store(c.s_lo + tile * c.KP * 64, s_s + Cfg::kSBytes, Cfg::kSBytes);
+        asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
       }
       __syncwarp();
       const float weight = chunk_exp2(decay + factor), keep = chunk_exp2(decay);
       ok = mbar_wait_bounded(smem_u32(&u_done), phase, &abort_flag, c.status, ST_TIMEOUT_TMEM_FULL);
       ok = __all_sync(0xffffffffu, ok);
       tc_fence_after();
+      uint4 row[2];                                                // U in the activation type
       if (ok) {
-        if (k + 1 < c1) load_w(k + 1);                             // W has been read
-        uint32_t v[32];
-        tmem_ld_32x32(tmem + half * 32 + lane_addr, v);
+        if (tid == 0 && k + 1 < c1) load_w(k + 1);                 // W has been read
+        uint32_t a[DC_COLS], d[DC_COLS];
+        tmem_ld_32x16(tmem + col + lane_addr, a);
+        tmem_ld_32x16(tmem + 64 + col + lane_addr, d);
         tmem_ld_wait();
         tc_fence_before();
-        __nv_bfloat16* dst = p.values + (long long)(ck.x + t) * p.ld_values + h * c.VP + z * 64 + half * 32;
+        float U[DC_COLS];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float4 x = uv[2 * i], y = uv[2 * i + 1];
-          const float U[8] = {x.x - __uint_as_float(v[8 * i]),     x.y - __uint_as_float(v[8 * i + 1]), x.z - __uint_as_float(v[8 * i + 2]),
-                              x.w - __uint_as_float(v[8 * i + 3]), y.x - __uint_as_float(v[8 * i + 4]), y.y - __uint_as_float(v[8 * i + 5]),
-                              y.z - __uint_as_float(v[8 * i + 6]), y.w - __uint_as_float(v[8 * i + 7])};
-          if (t < ck.y)
-            *reinterpret_cast<uint4*>(dst + i * 8) =
-                make_uint4(pack_bf16x2(U[0], U[1]), pack_bf16x2(U[2], U[3]), pack_bf16x2(U[4], U[5]), pack_bf16x2(U[6], U[7]));
-          uint32_t hi[4], lo[4];
-#pragma unroll
-          for (int e = 0; e < 4; ++e) split_bf16x2(weight * U[2 * e], weight * U[2 * e + 1], hi[e], lo[e]);
-          const uint32_t o = chunk_addr(t, half * 4 + i);
-          *reinterpret_cast<uint4*>(u_p + o) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(u_p + CH_CHUNK + o) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        for (int i = 0; i < DC_COLS / 4; ++i) {
+          U[4 * i] = uv[i].x - (__uint_as_float(a[4 * i]) + __uint_as_float(d[4 * i]));
+          U[4 * i + 1] = uv[i].y - (__uint_as_float(a[4 * i + 1]) + __uint_as_float(d[4 * i + 1]));
+          U[4 * i + 2] = uv[i].z - (__uint_as_float(a[4 * i + 2]) + __uint_as_float(d[4 * i + 2]));
+          U[4 * i + 3] = uv[i].w - (__uint_as_float(a[4 * i + 3]) + __uint_as_float(d[4 * i + 3]));
         }
-        if (k + 1 < c1) fetch(k + 1);
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+          row[i] = make_uint4(pack_bf16x2(U[8 * i], U[8 * i + 1]), pack_bf16x2(U[8 * i + 2], U[8 * i + 3]), pack_bf16x2(U[8 * i + 4], U[8 * i + 5]),
+                              pack_bf16x2(U[8 * i + 6], U[8 * i + 7]));
+#pragma unroll
+        for (int i = 0; i < DC_COLS; ++i) U[i] *= weight;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          split8(U, i * 8, hi[i], lo[i]);
+          const uint32_t o = chunk_addr(t, col / 8 + i);
+          *reinterpret_cast<uint4*>(u_p + o) = hi[i];
+          *reinterpret_cast<uint4*>(u_p + CH_CHUNK + o) = lo[i];
+        }
       }
       fence_proxy_async_smem();
       tc_fence_before();
+      if (warp == 0 && ok) ok = __all_sync(0xffffffffu, mbar_wait_bounded(smem_u32(&k_full), phase, &abort_flag, c.status, ST_TIMEOUT_SMEM_FULL));
       ok = __syncthreads_and(ok);
       if (!ok) break;
       tc_fence_after();
       if (warp == 0 && elect_one_sync()) {
-        constexpr uint32_t idesc = make_idesc_bf16(DK, 64, 1, 1);
+        constexpr uint32_t idesc = make_idesc_bf16(DK, 128, 1, 1);
 #pragma unroll
-        for (int part = 0; part < 2; ++part)
-#pragma unroll
-          for (int kk = 0; kk < CH / 16; ++kk) {
-            const uint64_t a = make_smem_desc_sw128(k_s + kk * 2048, CH_CHUNK, 1024);
-            const uint64_t d = make_smem_desc_sw128(u_s + part * CH_CHUNK + kk * 2048, CH_CHUNK, 1024);
-            umma_bf16(tmem + 64, a, d, idesc, (part | kk) ? 1u : 0u);
-          }
+        for (int kk = 0; kk < CH / 16; ++kk) {
+          const uint64_t a = make_smem_desc_sw128(k_s + kk * 2048, CH_CHUNK, 1024);
+          const uint64_t d = make_smem_desc_sw128(u_s + kk * 2048, CH_CHUNK, 1024);
+          umma_bf16(tmem + 128, a, d, idesc, kk ? 1u : 0u);
+        }
         umma_commit(smem_u32(&s_done));
       }
       __syncwarp();
+      {
+        uint4* dst = reinterpret_cast<uint4*>(p.values) + (tile * 8 + col / 8) * CH + t;
+        dst[0] = row[0];
+        dst[CH] = row[1];
+      }
+      if (k + 1 < c1) fetch(k + 1);
       ok = mbar_wait_bounded(smem_u32(&s_done), phase, &abort_flag, c.status, ST_TIMEOUT_TMEM_FULL);
       ok = __all_sync(0xffffffffu, ok);
       tc_fence_after();
       if (ok) {
-        if (k + 1 < c1) load_k(k + 1);                             // K has been read
-        uint32_t v[32];
-        tmem_ld_32x32(tmem + 64 + half * 32 + lane_addr, v);
+        if (tid == 0 && k + 1 < c1) load_k(k + 1);                 // K has been read
+        uint32_t a[DC_COLS], d[DC_COLS];
+        tmem_ld_32x16(tmem + 128 + col + lane_addr, a);
+        tmem_ld_32x16(tmem + 192 + col + lane_addr, d);
         tmem_ld_wait();
         tc_fence_before();
 #pragma unroll
-        for (int i = 0; i < 32; ++i) S[i] = fmaf(keep, S[i], __uint_as_float(v[i]));
+        for (int i = 0; i < DC_COLS; ++i) S[i] = fmaf(keep, S[i], __uint_as_float(a[i]) + __uint_as_float(d[i]));
+      }
+    }
+    if (!ok && tid == 0) {                                         // no copy may land after the CTA has gone
+      const uint64_t since = globaltimer_ns();
+      for (int i = 0; i < 2; ++i) {
+        const int loads = i ? k_loads : w_loads;
+        while (loads > 0 && !mbar_try_wait(smem_u32(i ? &k_full : &w_full), (uint32_t)((loads - 1) & 1)))
+          if (globaltimer_ns() - since > 50000000ull) break;
       }
     }
     if (ok && live)
 #pragma unroll
-      for (int i = 0; i < 8; ++i) st[i] = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
+      for (int i = 0; i < DC_COLS / 4; ++i) st[i] = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
+    if (tid == MOVER) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
   } else if (tid == 0) {
     set_status(c.status, ST_BAD_INDEX);
   }
-  cp_async_wait_all();
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
@@ -694,11 +765,8 @@ static int launch_delta_chunks(const DeltaParams& p, int n_chunks, int n_seq, cu
   const int units = n_chunks * c.H * (c.VP / 64);
   const int most = sms[dev] * (ChunkOutCfg<DK>::kSmem + 5 * 1024 <= 113 * 1024 ? 2 : 1);
   if (launch_kernel(delta_solve_kernel<DK>, dim3(n_chunks * c.H), dim3(CHT), DeltaSolveCfg<DK>::kSmem, stream, p) != cudaSuccess) return -11;
-  if (launch_kernel(delta_chain_kernel<DK>, dim3(c.VP / 64, c.H, n_seq), dim3(CHT), DeltaChainCfg<DK>::kSmem, stream, p) != cudaSuccess) return -12;
-  ChunkParams out = c;
-  out.v = p.values;
-  out.ld_v = p.ld_values;
-  return launch_kernel(recurrent_chunk_out_kernel<DK>, dim3(units < most ? units : most), dim3(CHT), ChunkOutCfg<DK>::kSmem, stream, out, units) == cudaSuccess ? 0 : -13;
+  if (launch_kernel(delta_chain_kernel<DK>, dim3(c.VP / 64, c.H, n_seq), dim3(DC_THREADS), DeltaChainCfg<DK>::kSmem, stream, p) != cudaSuccess) return -12;
+  return launch_kernel(recurrent_chunk_out_kernel<DK>, dim3(units < most ? units : most), dim3(CHT), ChunkOutCfg<DK>::kSmem, stream, c, units) == cudaSuccess ? 0 : -13;
 }
 
 }  // namespace rb

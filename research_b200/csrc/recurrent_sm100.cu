@@ -627,7 +627,9 @@ struct ChunkParams {
   const __nv_bfloat16* v;  // [T, ld_v] values
   long long ld_v;
   int ratio;               // heads that share queries and keys
-  int factors;             // the third of a token's gates is a factor of its query
+  // delta rule: values [chunks, H, VP / 64, 8, CH, 8], the state's parts as they lie in shared memory, and the third of a token's gates is a
+  // factor of its query
+  const __nv_bfloat16* written;
 };
 
 __device__ __forceinline__ float chunk_exp2(float x) {
@@ -1028,7 +1030,7 @@ __global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_out_ke
   auto load_state = [&](uint32_t dst, const __nv_bfloat16* part, const ChunkUnit& x) {
     const __nv_bfloat16* src = part + (x.ch * (p.VP / 64) + x.z) * p.KP * 64;
 #pragma unroll 4
-    for (int i = tid; i < DK * 8; i += CHT) cp_async16(dst + chunk_addr(i >> 3, i & 7), src + i * 8, true);
+    for (int i = tid; i < DK * 8; i += CHT) cp_async16(dst + (p.written ? i * 16 : chunk_addr(i >> 3, i & 7)), src + i * 8, true);
   };
   auto fetch_first = [&](const ChunkUnit& x) {       // Q, the state's second part, the vectors, V
     const __nv_bfloat16* rows = p.proj + x.row0 * p.ld;
@@ -1038,7 +1040,8 @@ __global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_out_ke
     for (int i = 0; i < VPT; ++i) {
       const int e = tid + i * CHT, r = e >> 3;
       vr[i] = make_uint4(0u, 0u, 0u, 0u);
-      if (r < x.n) vr[i] = *reinterpret_cast<const uint4*>(p.v + (x.row0 + r) * p.ld_v + x.h * p.VP + x.z * 64 + (e & 7) * 8);
+      if (p.written) vr[i] = reinterpret_cast<const uint4*>(p.written)[(x.ch * (p.VP / 64) + x.z) * (8 * CH) + e];
+      else if (r < x.n) vr[i] = *reinterpret_cast<const uint4*>(p.v + (x.row0 + r) * p.ld_v + x.h * p.VP + x.z * 64 + (e & 7) * 8);
     }
     if (tid < CH) {
       const float* g = p.gates + x.ch * 3 * CH + tid;
@@ -1157,7 +1160,7 @@ __global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_out_ke
 #pragma unroll
       for (int i = 0; i < VPT; ++i) {
         const int e = tid + i * CHT;
-        *reinterpret_cast<uint4*>(sv_p + chunk_addr(e >> 3, e & 7)) = vr[i];
+        *reinterpret_cast<uint4*>(sv_p + (p.written ? chunk_addr(e % CH, e / CH) : chunk_addr(e >> 3, e & 7))) = vr[i];
       }
     }
     row_sum[half][t] = sum + c_in * qn;
@@ -1179,7 +1182,7 @@ __global__ void __launch_bounds__(CHT, DK <= 128 ? 2 : 1) recurrent_chunk_out_ke
     __syncwarp();
     if (more) fetch_first(x);
     float f = p.q_scale;
-    if (p.factors) f *= F;
+    if (p.written) f *= F;
     if (p.gated) f /= fmaxf(fabsf((row_sum[0][t] + row_sum[1][t]) * p.q_scale), chunk_exp2(-(F + B))) + 1e-6f;
     ok = mbar_wait_bounded(smem_u32(&o_done), it & 1, &abort_flag, p.status, ST_TIMEOUT_TMEM_FULL);
     ok = __all_sync(0xffffffffu, ok);
@@ -1287,6 +1290,27 @@ __device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uin
   lo = pack_bf16x2(x - b.x, y - b.y);
 }
 
+// Forget gate for the chunked form: {log2 f (at least -MIX_MOST), 1 - f} from z log2(e), with errors of a few fp32 roundings.
+// For f near 1: -log1p(-k) = 2 atanh(w) with w = k / (2 - k), and the series of atanh (w <= 1/3).
+__device__ __forceinline__ float2 chunk_forget(float z2, float low) {
+  const float e = chunk_exp2(-fabsf(z2)), big = __fdividef(1.f, 1.f + e), small = e * big;
+  const float k = (1.f - low) * (z2 >= 0.f ? small : big);
+  float kept;
+  if (k < 0.5f) {
+    const float w = __fdividef(k, 2.f - k), x = w * w;
+    float s = fmaf(x, 1.f / 13.f, 1.f / 11.f);
+    s = fmaf(x, s, 1.f / 9.f);
+    s = fmaf(x, s, 1.f / 7.f);
+    s = fmaf(x, s, 1.f / 5.f);
+    s = fmaf(x, s, 1.f / 3.f);
+    kept = -2.f * LOG2E * fmaf(w * x, s, w);
+  } else {
+    const float f = fmaf(1.f - low, z2 >= 0.f ? big : small, low);
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(kept) : "f"(f));
+  }
+  return make_float2(fmaxf(kept, -MIX_MOST), k);
+}
+
 template <int DK>
 struct MixStateCfg {
   static constexpr int kKBytes = CH * DK * 2;
@@ -1346,12 +1370,11 @@ __global__ void __launch_bounds__(CHT, DK == 64 ? 2 : 1) time_mix_state_kernel(c
 #pragma unroll
   for (int i = 0; i < SEG; ++i) {
     if (FORGET) {
-      const float2 x = forget_gate(A[i].x + w0, low.x), y = forget_gate(A[i].y + w1, low.y);
+      const float2 x = chunk_forget((A[i].x + w0) * LOG2E, low.x), y = chunk_forget((A[i].y + w1) * LOG2E, low.y);
       fresh[FORGET ? i : 0] = make_float2(i < mine && col < p.dk ? x.y : 0.f, i < mine && col + 1 < p.dk ? y.y : 0.f);
-      auto kept = [](float2 f) { return fminf(-LOG2E * (f.y < 0.5f ? log1pf(-f.y) : logf(f.x)), MIX_MOST); };
       if (i < mine) {
-        run.x -= kept(x);
-        run.y -= kept(y);
+        run.x += x.x;
+        run.y += y.x;
       }
     } else if (i < mine) {
       run.x -= fminf(chunk_exp2(fmaf(A[i].x, LOG2E, w0)), MIX_MOST);
@@ -2346,17 +2369,16 @@ int rb_delta_rows(const void* proj, long long ld, const float* conv, int taps, v
 // Workspace of the chunked delta rule in bytes.
 long long rb_delta_workspace(int n_chunks, int H, int KP, int VP) {
   const long long ch = (long long)n_chunks * H;
-  return ch * ((long long)KP * VP * 4 + CH * KP * 4 + CH * VP * 4 + 3 * CH * 4 + 8) + 256;
+  return ch * ((long long)KP * VP * 4 + CH * KP * 6 + CH * VP * 6 + 3 * CH * 4 + 8) + 256;      // (room for a key head per head)
 }
 
-// The delta rule over whole portions in chunks, as rb_recurrent_chunks. rows [T, q | k | v] bf16, `values` [T, H * VP] bf16 is room for what is
-// written into the state. KP is 64 or 128.
+// The delta rule over whole portions in chunks, as rb_recurrent_chunks. rows [T, q | k | v] bf16. KP is 64 or 128.
 int rb_delta_chunks(const void* rows, long long ld, int k_col, int v_col, const float* units, const float* steps, float q_scale, float* s, const void* chunks,
-                    const int* seq_chunks, const int* slots, const int* cu_q, const int* seq_lens, void* values, long long ld_values, float* out,
-                    long long ldo, void* workspace, int n_chunks, int n_seq, int H, int ratio, int dk, int KP, int VP, int num_slots, int* status,
+                    const int* seq_chunks, const int* slots, const int* cu_q, const int* seq_lens, float* out, long long ldo,
+                    void* workspace, int n_chunks, int n_seq, int H, int ratio, int dk, int KP, int VP, int num_slots, int* status,
                     cudaStream_t stream) {
   if (n_chunks <= 0 || n_seq <= 0) return 0;
-  if (H <= 0 || H > 65535 || n_seq > 65535 || ratio <= 0 || H % ratio != 0 || dk <= 0 || dk > KP || VP % 64 != 0 || ld % 8 != 0 || ld_values % 8 != 0 ||
+  if (H <= 0 || H > 65535 || n_seq > 65535 || ratio <= 0 || H % ratio != 0 || dk <= 0 || dk > KP || VP % 64 != 0 || ld % 8 != 0 ||
       ldo % 4 != 0 || k_col % 8 != 0 || v_col % 8 != 0 || workspace == nullptr)
     return -1;
   const long long ch = (long long)n_chunks * H;
@@ -2366,14 +2388,17 @@ int rb_delta_chunks(const void* rows, long long ld, int k_col, int v_col, const 
   c.chunks = (const int4*)chunks; c.seq_chunks = seq_chunks; c.slots = slots; c.seq_lens = seq_lens; c.cu_q = cu_q;
   c.s = s; c.out = out; c.ldo = ldo;
   c.H = H; c.dk = dk; c.KP = KP; c.VP = VP; c.num_slots = num_slots; c.status = status;
-  c.v = c.proj + v_col; c.ld_v = ld; c.ratio = ratio; c.factors = 1;
-  p.units = units; p.steps = steps; p.values = (__nv_bfloat16*)values; p.ld_values = ld_values;
+  c.v = c.proj + v_col; c.ld_v = ld; c.ratio = ratio;
+  p.units = units; p.steps = steps;
   float* w = (float*)workspace;
   p.uv = w; w += ch * CH * VP;
   c.s_hi = (__nv_bfloat16*)w; w += ch * KP * VP / 2;
   c.s_lo = (__nv_bfloat16*)w; w += ch * KP * VP / 2;
   p.w_hi = (__nv_bfloat16*)w; w += ch * CH * KP / 2;
   p.w_lo = (__nv_bfloat16*)w; w += ch * CH * KP / 2;
+  p.keys = (__nv_bfloat16*)w; w += ch * CH * KP / 2;
+  p.values = (__nv_bfloat16*)w; w += ch * CH * VP / 2;
+  c.written = p.values;
   c.gates = w; w += ch * 3 * CH;
   c.um = (float2*)w;
   if (KP == 64) return launch_delta_chunks<64>(p, n_chunks, n_seq, stream);

@@ -369,7 +369,7 @@ class DeltaPart(Part):
         self.units = self.zeros(r.rows * max(2 * g.key_heads for g in geos), dtype=f32)
         self.steps = self.zeros(r.rows * max(2 * g.heads for g in geos), dtype=f32)
         most = r.rows * max(g.heads * g.vp for g in geos)
-        self.values, self.out, self.o = self.zeros(most), self.zeros(most), self.zeros(most, dtype=f32)
+        self.out, self.o = self.zeros(most), self.zeros(most, dtype=f32)
 
     def load(self, w: DeltaWeights, get, p: str) -> None:
         g = w.geo
@@ -416,8 +416,7 @@ class DeltaPart(Part):
             ops.recurrent_scan(*args, b.cu_q, b.seq_lens, o, ends, n_seq, b.n_single, mix=rule)
         if table is not None:
             room = torch.empty(delta_workspace(table.chunks.shape[0], g), dtype=torch.uint8, device=o.device)
-            values = self.values[:T * g.heads * g.vp].view(T, -1)
-            ops.delta_chunks(rows, g, rule, cache.state, b.state_slots, b.cu_q, b.seq_lens, o, table, values, room)
+            ops.delta_chunks(rows, g, rule, cache.state, b.state_slots, b.cu_q, b.seq_lens, o, table, room)
 
     def forward(self, w: DeltaWeights, cache: DeltaState, inp, y, b, plan, small=None) -> None:
         T, g = b.num_tokens, w.geo

@@ -152,7 +152,7 @@ def _lib() -> ctypes.CDLL:
                                           + [c_vp, c_ll] + [c_int] * 8 + [c_vp, c_ll, c_vp, c_vp, c_int, c_int, c_vp, c_vp, c_int, c_vp, c_vp])
         lib.rb_delta_rows.argtypes = ([c_vp, c_ll, c_vp, c_int] + [c_vp] * 4 + [c_int, c_int, c_vp, c_ll, c_vp, c_ll] + [c_vp] * 4 + [c_int] * 6
                                       + [c_vp, c_vp])
-        lib.rb_delta_chunks.argtypes = ([c_vp, c_ll, c_int, c_int, c_vp, c_vp, c_float] + [c_vp] * 7 + [c_ll, c_vp, c_ll, c_vp] + [c_int] * 8
+        lib.rb_delta_chunks.argtypes = ([c_vp, c_ll, c_int, c_int, c_vp, c_vp, c_float] + [c_vp] * 7 + [c_ll, c_vp] + [c_int] * 8
                                         + [c_vp, c_vp])
         lib.rb_delta_workspace.argtypes, lib.rb_delta_workspace.restype = [c_int] * 4, c_ll
         lib.rb_token_shift.argtypes = [c_vp, c_ll, c_vp, c_int, c_vp, c_ll, c_ll, c_vp, c_vp, c_vp, c_vp] + [c_int] * 5 + [c_vp, c_vp]
@@ -394,16 +394,16 @@ def delta_chunked_supported(geo: RecurrentGeometry) -> bool:
     return geo.kp in (64, 128)
 
 
-def delta_chunks(rows, geo: RecurrentGeometry, mix: DeltaRule, state: RecurrentState, slots, cu_q, seq_lens, out, table: ChunkTable, values,
+def delta_chunks(rows, geo: RecurrentGeometry, mix: DeltaRule, state: RecurrentState, slots, cu_q, seq_lens, out, table: ChunkTable,
                  workspace) -> None:
     """The delta rule over the sequences of ``table`` in chunks of 128 tokens (bf16 rows on the GPU): fp32 rows ``cu_q[first] ..`` of ``out``, state
-    updated. ``values [>= T, H*vp]`` (bf16) and ``workspace`` (``delta_workspace`` bytes) are room to work in."""
+    updated. ``workspace``: ``delta_workspace`` bytes."""
     _, ok, ov, _ = geo.offsets
     n, B, f = table.chunks.shape[0], table.seq_chunks.shape[0] - 1, table.first
-    assert rows.is_cuda and rows.dtype == values.dtype == torch.bfloat16 and rows.stride(1) == out.stride(1) == values.stride(1) == 1
+    assert rows.is_cuda and rows.dtype == torch.bfloat16 and rows.stride(1) == out.stride(1) == 1
     assert out.dtype == torch.float32 and workspace.numel() * workspace.element_size() >= delta_workspace(n, geo)
     rc = _lib().rb_delta_chunks(ptr(rows), rows.stride(0), ok, ov, ptr(mix.units), ptr(mix.steps), geo.q_scale, ptr(state.s), ptr(table.chunks),
-                                ptr(table.seq_chunks), ptr(slots[f:]), ptr(cu_q[f:]), ptr(seq_lens[f:]), ptr(values), values.stride(0), ptr(out),
+                                ptr(table.seq_chunks), ptr(slots[f:]), ptr(cu_q[f:]), ptr(seq_lens[f:]), ptr(out),
                                 out.stride(0), ptr(workspace), n, B, geo.heads, geo.heads // geo.key_heads, geo.dim, geo.kp, geo.vp, state.s.shape[0],
                                 ptr(status_tensor(rows.device)), stream_handle(rows.device))
     check_rc(rc, "rb_delta_chunks", 3)

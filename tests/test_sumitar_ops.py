@@ -203,8 +203,7 @@ def test_delta_rule_in_portions_slots_and_batches(place, shape):
             ops.recurrent_scan(*a, b.cut, b.seq_lens, out, b.cu[b.short], b.short, b.single, mix=rule)
         if b.table is not None:
             room = torch.empty(delta_workspace(b.table.chunks.shape[0], geo), dtype=torch.uint8, device=dev)
-            values = torch.full((b.T, H * geo.vp), 3.0, dtype=dt, device=dev)
-            ops.delta_chunks(rows, geo, rule, state, b.state_slots, b.cut, b.seq_lens, out, b.table, values, room)
+            ops.delta_chunks(rows, geo, rule, state, b.state_slots, b.cut, b.seq_lens, out, b.table, room)
         b.split(out, got)
     for i, m in enumerate(LENS):
         o = torch.cat(got[i]).view(m, H, geo.vp)
@@ -237,10 +236,10 @@ def test_delta_chunks_equal_the_scan(cuda_device, H, G, D, E):
     outs = [torch.zeros(T, H * geo.vp, device=dev) for _ in range(2)]
     ops.recurrent_scan(rows, None, geo, None, None, None, 1.0, states[0], slots, cut, lens_t, outs[0], T, 6, mix=rule)
     table = ChunkTable.make(cu, 0, dev)
-    room, values = torch.empty(delta_workspace(table.chunks.shape[0], geo), dtype=torch.uint8, device=dev), torch.zeros(T, H * geo.vp, dtype=torch.bfloat16, device=dev)
+    room = torch.empty(delta_workspace(table.chunks.shape[0], geo), dtype=torch.uint8, device=dev)
     for _ in range(2):          # (twice: nothing is left behind in the workspace)
         states[1].s.copy_(start.view(8, H, geo.kp, geo.tiles, 32).permute(0, 1, 3, 2, 4))
-        ops.delta_chunks(rows, geo, rule, states[1], slots, cut, lens_t, outs[1], table, values, room)
+        ops.delta_chunks(rows, geo, rule, states[1], slots, cut, lens_t, outs[1], table, room)
         ops.check_status()
         close(outs[1], outs[0].cpu(), torch.bfloat16)
         close(states[1].s, states[0].s.cpu(), torch.float32, tol=1e-4)
