@@ -814,7 +814,7 @@ def main() -> None:
                          "serving = batch 64, prompts of 2048 tokens, 256 new tokens (the tensor-parallel serving case); "
                          "stack = prefill and decode of layer-stack models beside the closest model of equal size, kernel by kernel")
     ap.add_argument("--sizes", default="", help="stack: comma-separated sizes (default: all)")
-    ap.add_argument("--designs", default="", help="stack: comma-separated designs, lulezen, zamusun or fogurax (default: all)")
+    ap.add_argument("--designs", default="", help="stack: comma-separated designs, lulezen, zamusun, fogurax or sumitar (default: all)")
     ap.add_argument("--model", default=None, help="model preset (default: llama-3-8b for train / serving, qwen2.5-0.5b for rollout)")
     ap.add_argument("--seq", type=int, default=TRAIN_SEQ, help="train: tokens per sequence")
     ap.add_argument("--batch", type=int, default=TRAIN_BATCH_PER_GPU, help="train: sequences per GPU per step")

@@ -222,7 +222,7 @@ template <int DK>
 __global__ void __launch_bounds__(CHT, 2) delta_solve_kernel(const DeltaParams p) {
   using Cfg = DeltaSolveCfg<DK>;
   extern __shared__ __align__(128) uint8_t smem_raw[];
-  __shared__ float Fs[CH], betas[CH], rks[CH];
+  __shared__ float Fs[CH], betas[CH], rks[CH], sums[4];
   __shared__ __align__(8) float diag[8][16][18];
   __shared__ __align__(8) uint64_t done;
   __shared__ uint32_t tmem_base_smem;
@@ -254,37 +254,33 @@ __global__ void __launch_bounds__(CHT, 2) delta_solve_kernel(const DeltaParams p
   const long long ch = (long long)chunk * c.H + h;
   const __nv_bfloat16* rows = c.proj + (long long)row0 * c.ld;
   chunk_load<DK>(k_s, rows + c.k_col + hk * c.KP, c.ld, n);
-  if (warp == 0) {                                       // F, step sizes, factors: four tokens per lane
-    float lf[4], run = 0.f;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int t = lane * 4 + i;
-      const long long r = row0 + min(t, n - 1);
-      const bool in = t < n;
-      run += in ? fmaxf(p.steps[r * 2 * c.H + h] * LOG2E, -MIX_MOST) : 0.f;
-      lf[i] = run;
-      betas[t] = in ? p.steps[r * 2 * c.H + c.H + h] : 0.f;
-      rks[t] = in ? p.units[r * 2 * G + G + hk] : 0.f;
+  float run = 0.f, q_factor = 0.f, k_factor = 0.f, step = 0.f;       // a token per thread of the first four warps: F, step sizes, factors
+  if (tid < CH) {
+    if (tid < n) {
+      const long long r = row0 + tid;
+      run = fmaxf(p.steps[r * 2 * c.H + h] * LOG2E, -MIX_MOST);
+      step = p.steps[r * 2 * c.H + c.H + h];
+      q_factor = p.units[r * 2 * G + hk];
+      k_factor = p.units[r * 2 * G + G + hk];
     }
-    float before = run;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float y = __shfl_up_sync(0xffffffffu, before, o);
-      if (lane >= o) before += y;
+      const float y = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += y;
     }
-    const float total = __shfl_sync(0xffffffffu, before, 31);
-    before -= run;
-    float* gates = c.gates + ch * 3 * CH;                // log2 of a key's factor, the row's reference, the query's factor
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int t = lane * 4 + i;
-      const float F = lf[i] + before;
-      Fs[t] = F;
-      gates[t] = t < n ? log2f(rks[t]) - F : -INFINITY;
-      gates[CH + t] = -F;
-      gates[2 * CH + t] = t < n ? p.units[(long long)(row0 + t) * 2 * G + hk] : 0.f;
-    }
-    if (lane == 0) c.um[ch] = make_float2(total, 0.f);
+    if (lane == 31) sums[warp] = run;
+  }
+  __syncthreads();
+  if (tid < CH) {
+    for (int w = 0; w < warp; ++w) run += sums[w];
+    Fs[tid] = run;
+    betas[tid] = step;
+    rks[tid] = k_factor;
+    float* gates = c.gates + ch * 3 * CH + tid;          // log2 of a key's factor, the row's reference, the query's factor
+    gates[0] = tid < n ? log2f(k_factor) - run : -INFINITY;
+    gates[CH] = -run;
+    gates[2 * CH] = q_factor;
+    if (tid == CH - 1) c.um[ch] = make_float2(run, 0.f);
   }
   cp_async_wait_all();
   fence_proxy_async_smem();

@@ -14,6 +14,7 @@ def engine_smoke(device: torch.device) -> None:
     _run(device, get_preset("tiny-lulezen"))      # latent attention: prefill and decode kernels, 32-bit residual stream
     _run(device, get_preset("tiny-zamusun"))      # recurrent state, keys-as-values attention, routed experts, looped layers
     _run(device, get_preset("tiny-fogurax"))      # convolutions, chunks, attention beside time mixing, shared expert, token input
+    _run(device, get_preset("tiny-sumitar"))      # sandwich norms, attention beside forget mixing, delta rule, identity experts, normed powers
 
 
 def _run(device: torch.device, cfg) -> None:

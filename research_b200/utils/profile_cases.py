@@ -342,6 +342,77 @@ def case_time_mix_prefill() -> None:
     print("ok")
 
 
+def case_forget_mix_prefill() -> None:
+    """Forget mixing in chunks: one portion of 4096 tokens, 32 heads of 64 x 64."""
+    from ..ops.recurrent import ChunkTable, ForgetMix, RecurrentGeometry, RecurrentState, time_mix_workspace
+
+    T, n = 4096, 2048
+    geo = RecurrentGeometry(32, 64, 64, silu=True, gated=False, form="forget")
+    proj, z = torch.randn(T, geo.proj, device="cuda").bfloat16(), torch.randn(T, n, device="cuda") + 3
+    mix = ForgetMix(z.clone(), torch.zeros(n, device="cuda"), torch.rand(n, device="cuda") * 0.5, torch.empty(T, 2 * n, dtype=torch.bfloat16, device="cuda"))
+    state, slots = RecurrentState.zeros(geo, 1, "cuda"), torch.zeros(1, dtype=torch.int32, device="cuda")
+    cu, lens = torch.tensor([0, T], dtype=torch.int32, device="cuda"), torch.tensor([T], dtype=torch.int32, device="cuda")
+    table, out, norm = ChunkTable.make([0, T], 0, "cuda"), torch.empty(T, n, dtype=torch.bfloat16, device="cuda"), torch.ones(n, device="cuda")
+    room = torch.empty(time_mix_workspace(table.chunks.shape[0], geo), dtype=torch.uint8, device="cuda")
+    for _ in range(3):
+        mix.z.copy_(z)
+        ops.time_mix_chunks(proj, geo, mix, state, slots, cu, lens, norm, 1e-6, out, table, room)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def _delta(T: int, seqs: int):
+    """16 heads of 128 channels: rows, factors and steps of T tokens, state of ``seqs`` sequences."""
+    from ..ops.recurrent import DeltaRule, RecurrentGeometry, RecurrentState
+
+    geo = RecurrentGeometry(16, 128, 128, silu=False, gated=False, form="delta", groups=16)
+    rows = torch.randn(T, geo.channels, device="cuda").bfloat16()
+    rule = DeltaRule(torch.full((T, 32), 128 ** -0.5, device="cuda"), torch.cat([-torch.rand(T, 16, device="cuda") * 0.1, torch.rand(T, 16, device="cuda")], 1))
+    return rows, geo, rule, RecurrentState.zeros(geo, seqs, "cuda"), torch.arange(seqs, dtype=torch.int32, device="cuda")
+
+
+def case_delta_prefill() -> None:
+    """Delta rule in chunks: one portion of 4096 tokens, 16 heads of 128 x 128."""
+    from ..ops.recurrent import ChunkTable, delta_workspace
+
+    T = 4096
+    rows, geo, rule, state, slots = _delta(T, 1)
+    cu, lens = torch.tensor([0, T], dtype=torch.int32, device="cuda"), torch.tensor([T], dtype=torch.int32, device="cuda")
+    table, out = ChunkTable.make([0, T], 0, "cuda"), torch.empty(T, 2048, device="cuda")
+    room = torch.empty(delta_workspace(table.chunks.shape[0], geo), dtype=torch.uint8, device="cuda")
+    for _ in range(3):
+        ops.delta_chunks(rows, geo, rule, state, slots, cu, lens, out, table, room)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def case_delta_decode() -> None:
+    """Delta rule, one token for each of 256 sequences: 16 heads of 128 x 128 (268 MB of state)."""
+    rows, geo, rule, state, slots = _delta(256, 256)
+    lens, out = torch.full((256,), 100, dtype=torch.int32, device="cuda"), torch.empty(256, 2048, device="cuda")
+    for _ in range(3):
+        ops.recurrent_scan(rows, None, geo, None, None, None, 1.0, state, slots, None, lens, out, 256, 256, mix=rule)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
+def case_delta_rows() -> None:
+    """Convolutions of 4 taps, SiLU and units of 4096 tokens: 16 heads of 128 channels each of queries, keys and values."""
+    T = 4096
+    rows, geo, rule, _, slots = _delta(T, 1)
+    proj, small = torch.randn(T, geo.proj, device="cuda").bfloat16(), torch.randn(T, 32, device="cuda")
+    hist, ones = torch.zeros(2, 3, geo.channels, dtype=torch.bfloat16, device="cuda"), torch.ones(16, device="cuda")
+    cu, pos = torch.tensor([0, T], dtype=torch.int32, device="cuda"), torch.arange(T, dtype=torch.int32, device="cuda")
+    for _ in range(3):
+        ops.delta_rows(proj, small, geo, torch.ones(4, geo.channels, device="cuda"), hist, cu, pos, slots, ones, ones, rows, rule)
+    torch.cuda.synchronize()
+    ops.check_status()
+    print("ok")
+
+
 def _grouped(T: int, rows_cached: int, conv: bool):
     from ..ops.grouped import GroupedCache, GroupedGeometry
 

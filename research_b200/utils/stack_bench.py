@@ -124,12 +124,12 @@ def fogurax_configs(s: ExpertSize):
 
 
 def sumitar_stack(s: ExpertSize, layers: int, conv: int = 4, reach: int = 4096) -> LayerStackConfig:
-    """Two layers of the delta rule (heads of 128 channels, two share queries and keys), then attention beside forget mixing; the first feed-forward
-    has normed powers, the others route, one choice in sixteen an identity."""
+    """Two layers of the delta rule (heads of 128 channels), then attention beside forget mixing (heads of 64); the first feed-forward has normed
+    powers, the others route, one choice in sixteen an identity."""
     H, kinds = s.heads, STACK_DESIGNS["Sumitar"].mixers
-    rule = DeltaRuleSpec(H, H // 2, 128, 128, conv)
+    rule = DeltaRuleSpec(H, H, 128, 128, conv)
     left = GroupedAttentionSpec(kinds["parallel"].left, H, s.kv_heads, 128, 128, 128 ** -0.5, RotarySpec(64, 5e5), 1, reach)
-    both = NormedPairSpec("parallel", left, ForgetMixSpec(H, 128, 128))
+    both = NormedPairSpec("parallel", left, ForgetMixSpec(2 * H, 64, 64))
     plain = s.experts // 16
     mlp = ExpertsSpec(s.experts - plain, s.top, GluSpec(s.ff), ExpertsRouting(normalize=False, correction=True, shared_gate=True), GluSpec(s.ff), plain)
     return LayerStackConfig("Sumitar", s.vocab, s.width, tuple(LayerSpec(both if i % 3 == 2 else rule, PolyNormSpec(s.top * s.ff) if i == 0 else mlp)
