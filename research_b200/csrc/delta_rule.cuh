@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rows_kernel(const DeltaRows 
       float s = weight[0][j] * x[j];
 #pragma unroll
       for (int d = 1; d < TAPS; ++d) s = fmaf(weight[d][j], back[d - 1][j], s);
-      y[j] = s * sigmoid_f(s);
+      y[j] = sizeof(T) == 4 ? s * sigmoid_f(s) : silu_fast(s);
     }
     if (active) lane_store<T, CPL>(reinterpret_cast<T*>(p.out) + (long long)t * p.ldo + c, y);
     if (!is_v) {
